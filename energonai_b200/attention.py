@@ -96,3 +96,67 @@ def attention_decode(q, k, v, head_dim, kv_len, mask=None, scale=None, out=None,
                                     ptr(kv_len_device), head_dim, float(scale), dtype_code(q.dtype), nsplit, ptr(scratch),
                                     scratch.numel() if scratch is not None else 0, stream_ptr()), "attention_decode")
     return out
+
+
+def attention_prefill_window(q, k, v, head_dim, window, mask=None, scale=None, out=None):
+    """attention_prefill (causal, tensor-core kernel) in which row i sees the keys j with
+    0 <= i - j < window (window 0: all up to i)."""
+    require_cuda(q, k, v, mask, out)
+    B, Sq, HD = q.shape
+    Sk = k.shape[1]
+    if out is None:
+        out = torch.empty((B, Sq, HD), dtype=q.dtype, device=q.device)
+    if mask is not None and (mask.dtype != q.dtype or mask.stride(-1) != 1 or mask.dim() != 2 or mask.shape[1] < Sk):
+        raise RuntimeError("attention: mask must be [batch, kv_len] of the tensor dtype")
+    qs, ks, vs, os_ = (_bsh_strides(t, head_dim) for t in (q, k, v, out))
+    scale = head_dim ** -0.5 if scale is None else scale
+    check(lib().eb_attention_prefill_window_tc(ptr(q), ptr(k), ptr(v), ptr(out), ptr(mask), qs[0], qs[1], ks[0], ks[1], vs[0], vs[1],
+                                               os_[0], os_[1], mask.stride(0) if mask is not None else 0, B, HD // head_dim, Sq, Sk,
+                                               head_dim, int(window), float(scale), dtype_code(q.dtype), stream_ptr()),
+          "attention_prefill_window_tc")
+    return out
+
+
+def attention_plain(q, k, v, heads, k_dim, v_dim, window=0, scale=1.0, first=None, pos_device=None, shared_kv=False):
+    """Windowed causal attention on the CUDA cores, any head sizes, fp32 / fp16 / bf16.  q [B, Sq,
+    heads*k_dim]; k / v [B, rows, heads*dim] or, with shared_kv, [B, rows, dim] shared by the heads.
+    Query row i holds position pos_device + i (None: i), the key of position j is row j mod rows;
+    first [B] int32 is each sequence's first position.  Returns [B, Sq, heads*v_dim]."""
+    require_cuda(q, k, v, first, pos_device)
+    B, Sq, _ = q.shape
+    out = torch.empty((B, Sq, heads * v_dim), dtype=q.dtype, device=q.device)
+    if any(t.stride(2) != 1 for t in (q, k, v)) or k.shape[1] != v.shape[1]:
+        raise RuntimeError("attention: contiguous last dims and one number of key / value rows required")
+    hk, hv = (0, 0) if shared_kv else (k_dim, v_dim)
+    check(lib().eb_attention_plain(ptr(q), ptr(k), ptr(v), ptr(out), q.stride(0), q.stride(1), k_dim, k.stride(0), k.stride(1), hk,
+                                   v.stride(0), v.stride(1), hv, out.stride(0), out.stride(1), v_dim, B, heads, Sq, k_dim, v_dim,
+                                   int(window), k.shape[1], ptr(pos_device), ptr(first), float(scale), dtype_code(q.dtype), stream_ptr()),
+          "attention_plain")
+    return out
+
+
+LATENT_WIDTHS = (64, 128, 256, 384, 512)      # latent widths of the tensor-core generation kernel
+
+
+def pick_latent_nsplit(batch, heads, keys, sm_count=148):
+    """Key splits per (sequence, head tile): what fills the SMs, at least two 64-key tiles each."""
+    ctas = batch * -(-heads // (32 if heads > 16 else 16))
+    tiles = max(1, -(-keys // 64))
+    return max(1, min(sm_count // max(1, ctas), tiles // 2, 64))
+
+
+def latent_decode(q, cache, rank, heads, window, pos_device, scale, first=None, nsplit=None):
+    """Generation step over a latent ring cache: q [B, heads*rank] (absorbed queries), cache [B,
+    rows, rank], pos_device int32 scalar (the query's position).  Returns [B, heads*rank]."""
+    require_cuda(q, cache, pos_device, first)
+    B = q.shape[0]
+    rows = cache.shape[1]
+    out = torch.empty((B, heads * rank), dtype=q.dtype, device=q.device)
+    if nsplit is None:
+        nsplit = pick_latent_nsplit(B, heads, min(window, rows) if window > 0 else rows)
+    nbytes = lib().eb_latent_decode_scratch_bytes(B, heads, rank, nsplit)
+    scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
+    check(lib().eb_latent_decode(ptr(q), q.stride(0), ptr(cache), cache.stride(0), cache.stride(1), rows, ptr(out), out.stride(0), B,
+                                 heads, rank, int(window), ptr(pos_device), ptr(first), float(scale), dtype_code(q.dtype), nsplit,
+                                 ptr(scratch), nbytes, stream_ptr()), "latent_decode", launches=2 if nsplit > 1 else 1)
+    return out

@@ -6,6 +6,7 @@ Every .cu under csrc/ is compiled to an object under build/ (skipped when up to 
 linked into energonai_b200/libenergon_b200.so.  No torch headers are involved.
 """
 import concurrent.futures
+import fcntl
 import os
 import subprocess
 import sys
@@ -34,6 +35,12 @@ def _newer(src_paths, target):
 
 def build(force=False, verbose=False):
     os.makedirs(OBJ_DIR, exist_ok=True)
+    with open(os.path.join(OBJ_DIR, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)          # processes that start together build once
+        return _build(force, verbose)
+
+
+def _build(force, verbose):
     sources = sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
     headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h", ".inc"))]
     headers.append(os.path.join(os.path.dirname(HERE), "include", "energon_b200.h"))

@@ -23,6 +23,9 @@
 // sum is fp32).  The two row tiles alternate on the tensor core: while the softmax warps of one
 // work on their scores, it serves the other.
 //
+// A sliding window (row i sees only the `window` keys up to its own position) shortens the range of
+// key tiles a row tile walks and hides the leading keys of its first tiles; nothing else changes.
+//
 // Every mbarrier wait is bounded; a wait that runs out is recorded, the CTA's roles leave (each
 // decision made uniform over the warp first), copies in flight are given time to land, TMEM is
 // freed and the kernel returns.
@@ -55,6 +58,7 @@ __device__ int g_tc_status[4];             // [0] code, [1] where, [2] block, [3
 
 struct TcParams {
   int B, H, Sq, Sk, causal;
+  int window;                              // > 0: row i sees keys j with i - j < window only (causal)
   int mask_vec;                            // mask rows start on 16-byte boundaries
   float scale_log2;                        // scale * log2(e)
   const void *mask;                        // additive [B][>= Sk] in T, or null
@@ -217,14 +221,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   const int q0 = qb * (kTiles * kRows), shift = p.Sk - p.Sq;
   // key tiles each row tile walks: all of them, or up to its last row's diagonal; none for a
   // row tile that lies wholly behind the end of the sequence
-  int nt[kTiles], nmax = 0;
+  // With a window a row tile starts at the first key its first row sees: tiles [ks[t], nt[t]) of
+  // the CTA's [jmin, nmax).  (The ranges of the two row tiles rise together and leave no gap.)
+  int nt[kTiles], ks[kTiles], nmax = 0, jmin = 0x7fffffff;
 #pragma unroll
   for (int t = 0; t < kTiles; ++t) {
     const int qt0 = q0 + t * kRows;
     const int last_key = p.causal ? min(p.Sk - 1, qt0 + kRows - 1 + shift) : p.Sk - 1;
     nt[t] = (qt0 < p.Sq && last_key >= 0) ? last_key / kKeys + 1 : 0;
+    ks[t] = p.window > 0 ? max(0, qt0 + shift - p.window + 1) / kKeys : 0;
+    if (nt[t] > 0) jmin = min(jmin, ks[t]);
     nmax = max(nmax, nt[t]);
   }
+  if (jmin > nmax) jmin = nmax;
 
   if (threadIdx.x == 0) {
     asm volatile("prefetch.tensormap [%0];" ::"l"(&tm_q) : "memory");
@@ -267,19 +276,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       // K runs one tile ahead of V: its stage is released earlier (after the scores, not after
       // the value product), and the next scores are what the softmax warps wait for
       auto load_k = [&](int j) -> bool {
-        const int ks = j & 1;
-        if (j >= 2 && !bar_wait(k_empty + 8 * ks, ((j >> 1) - 1) & 1, abort_flag, 1)) return false;
-        bar_expect_tx(k_full + 8 * ks, kKBytes);
+        const int i = j - jmin, st = i & 1;
+        if (i >= 2 && !bar_wait(k_empty + 8 * st, ((i >> 1) - 1) & 1, abort_flag, 1)) return false;
+        bar_expect_tx(k_full + 8 * st, kKBytes);
 #pragma unroll
         for (int kb = 0; kb < kSub; ++kb)
-          tma_load_3d(k_addr + ks * kKBytes + kb * kKeys * 128, &tm_k, k_full + 8 * ks, h * D + kb * 64, j * kKeys, b);
+          tma_load_3d(k_addr + st * kKBytes + kb * kKeys * 128, &tm_k, k_full + 8 * st, h * D + kb * 64, j * kKeys, b);
         return true;
       };
-      bool ok = load_k(0);
-      for (int j = 0; j < nmax && ok; ++j) {
-        const int vs = j % kVStages, vu = j / kVStages;
+      bool ok = load_k(jmin);
+      for (int j = jmin; j < nmax && ok; ++j) {
+        const int i = j - jmin, vs = i % kVStages, vu = i / kVStages;
         if (j + 1 < nmax && !load_k(j + 1)) break;
-        if (j >= kVStages && !bar_wait(v_empty + 8 * vs, (vu - 1) & 1, abort_flag, 9)) break;
+        if (i >= kVStages && !bar_wait(v_empty + 8 * vs, (vu - 1) & 1, abort_flag, 9)) break;
         bar_expect_tx(v_full + 8 * vs, kVBytes);
 #pragma unroll
         for (int kb = 0; kb < kSub; ++kb)
@@ -292,29 +301,32 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     // (which also says that S(j) has been read): S(j+1) first, so the softmax warps get their
     // next scores as early as possible, then O += P(j) . V(j).
     if (lane == 0 && nmax > 0) {
-      auto last_reader = [&](int j) { return (kTiles > 1 && j < nt[kTiles - 1]) ? kTiles - 1 : 0; };
+      // (with a window, the second row tile joins at key tile ks[1]: its first scores are issued in
+      // the round before, behind those of the first row tile)
+      auto last_reader = [&](int j) { return (kTiles > 1 && j >= ks[kTiles - 1] && j < nt[kTiles - 1]) ? kTiles - 1 : 0; };
       auto issue_scores = [&](int t, int j) -> bool {
-        const int ks = j & 1;
-        if (!bar_wait(k_full + 8 * ks, (j >> 1) & 1, abort_flag, 3)) return false;
+        const int st = (j - jmin) & 1;
+        if (!bar_wait(k_full + 8 * st, ((j - jmin) >> 1) & 1, abort_flag, 3)) return false;
         tc_fence_after();
 #pragma unroll
         for (int kb = 0; kb < kSub; ++kb) {
-          const uint64_t a = tc_desc(q_addr + t * kQBytes + kb * kRows * 128), bd = tc_desc(k_addr + ks * kKBytes + kb * kKeys * 128);
+          const uint64_t a = tc_desc(q_addr + t * kQBytes + kb * kRows * 128), bd = tc_desc(k_addr + st * kKBytes + kb * kKeys * 128);
 #pragma unroll
           for (int k = 0; k < 4; ++k) tc_mma(tmem + t * kKeys, a + 2 * k, bd + 2 * k, kIdescS, (kb > 0 || k > 0) ? 1u : 0u);
         }
         tc_commit(s_full + 8 * t);
-        if (t == last_reader(j)) tc_commit(k_empty + 8 * ks);
+        if (t == last_reader(j)) tc_commit(k_empty + 8 * st);
         return true;
       };
       bool ok = bar_wait(q_full, 0, abort_flag, 2);
       for (int t = 0; t < kTiles && ok; ++t)
-        if (nt[t] > 0) ok = issue_scores(t, 0);
-      for (int j = 0; j < nmax && ok; ++j) {
-        const int vs = j % kVStages, vu = j / kVStages;
+        if (nt[t] > 0 && ks[t] == jmin) ok = issue_scores(t, jmin);
+      for (int j = jmin; j < nmax && ok; ++j) {
+        const int vs = (j - jmin) % kVStages, vu = (j - jmin) / kVStages;
         for (int t = 0; t < kTiles && ok; ++t) {
-          if (j >= nt[t]) continue;
-          ok = bar_wait(p_full + 8 * t, j & 1, abort_flag, 5);
+          if (nt[t] > 0 && ks[t] == j + 1) ok = issue_scores(t, j + 1);
+          if (j < ks[t] || j >= nt[t]) continue;
+          ok = ok && bar_wait(p_full + 8 * t, (j - ks[t]) & 1, abort_flag, 5);
           if (ok && j + 1 < nt[t]) ok = issue_scores(t, j + 1);
           ok = ok && bar_wait(v_full + 8 * vs, vu & 1, abort_flag, 10);
           if (!ok) break;
@@ -326,7 +338,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
             for (int k = 0; k < 4; ++k) {
               // 16 keys per instruction: two 8-row groups (2048 bytes) down the V tile
               const uint64_t bd = tc_desc_nmajor(v_addr + vs * kVBytes + (a2 * 4 + k) * 2048, kKeys * 128);
-              tc_mma(tmem + kPvCol + t * kKeys, a + 2 * k, bd, kIdescPV, (j > 0 || a2 > 0 || k > 0) ? 1u : 0u);
+              tc_mma(tmem + kPvCol + t * kKeys, a + 2 * k, bd, kIdescPV, (j > ks[t] || a2 > 0 || k > 0) ? 1u : 0u);
             }
           }
           tc_commit(pv_full + 8 * t);
@@ -337,15 +349,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   } else {
     // ---------------- softmax warps: 4 per row tile, thread = query row ----------------
     const int t = (warp - 2) >> 2, quarter = warp & 3, row = quarter * 32 + lane, qi = q0 + t * kRows + row;
-    const int ntiles = nt[t];
+    const int ntiles = nt[t], first_tile = ks[t];
     const uint32_t t_s = tmem + ((uint32_t)(quarter * 32) << 16) + t * kKeys, t_pv = t_s + kPvCol;
     const uint32_t my_s_full = s_full + 8 * t, my_p_full = p_full + 8 * t, my_pv_full = pv_full + 8 * t;
     uint8_t *p_row = p_ptr + t * kPBytes + row * 128;
     const T *mrow = p.mask ? reinterpret_cast<const T *>(p.mask) + (long long)b * p.mask_bs : nullptr;
     const int vis_end = p.causal ? min(p.Sk, qi + shift + 1) : p.Sk;               // keys [0, vis_end) are visible to this row
+    const int vis_begin = p.window > 0 ? qi + shift - p.window + 1 : 0;            // ... from this key on
     float m_ref = -1e30f, l_run = 0.f;      // m_ref: the maximum the accumulated row and l_run are scaled by
     bool alive = ntiles > 0;
-    for (int j = 0; j < ntiles && alive; ++j) {
+    for (int j = first_tile; j < ntiles && alive; ++j) {
       const int key0 = j * kKeys;
       // Work per chunk of 32 keys, decided for the warp as a whole (tensor-memory loads are
       // warp-wide): 0 = hidden from every row of the warp (behind the diagonal or the end of the
@@ -361,11 +374,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         float mv = 0.f;
         if (mrow && kb + lane < p.Sk) mv = to_f32<T>(mrow[kb + lane]) * kLog2eTc;
         mval[c] = mv;
-        const bool hidden = __all_sync(0xffffffffu, kb >= vis_end);
-        const bool simple = __all_sync(0xffffffffu, kb + 32 <= vis_end && mv == 0.f);
+        const bool hidden = __all_sync(0xffffffffu, kb >= vis_end || kb + 32 <= vis_begin);
+        const bool simple = __all_sync(0xffffffffu, kb >= vis_begin && kb + 32 <= vis_end && mv == 0.f);
         cls[c] = hidden ? 0 : (simple ? 1 : 2);
       }
-      if (!__all_sync(0xffffffffu, bar_wait(my_s_full, j & 1, abort_flag, 7))) { alive = false; break; }
+      if (!__all_sync(0xffffffffu, bar_wait(my_s_full, (j - first_tile) & 1, abort_flag, 7))) { alive = false; break; }
       tc_fence_after();
       // pass 1: the row maximum of this tile (log2 domain, masks applied)
       float r0 = -INFINITY, r1 = -INFINITY, r2 = -INFINITY, r3 = -INFINITY, m_tile = -1e30f;
@@ -383,11 +396,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
             r3 = fmaxf(r3, x[e + 3]);
           }
         } else {
-          const int nvis = vis_end - (key0 + c * 32);
+          const int nvis = vis_end - (key0 + c * 32), n0 = vis_begin - (key0 + c * 32);
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
             const float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
-            m_tile = fmaxf(m_tile, e < nvis ? v : -INFINITY);
+            m_tile = fmaxf(m_tile, e < nvis && e >= n0 ? v : -INFINITY);
           }
         }
       }
@@ -396,7 +409,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       // The previous tile's value product must be complete before P is overwritten (it reads P)
       // and before the accumulated row is rescaled; it was issued right behind the scores just
       // read, so this wait is normally over already.
-      if (j > 0 && !__all_sync(0xffffffffu, bar_wait(my_pv_full, (j - 1) & 1, abort_flag, 8))) { alive = false; break; }
+      if (j > first_tile && !__all_sync(0xffffffffu, bar_wait(my_pv_full, (j - 1 - first_tile) & 1, abort_flag, 8))) { alive = false; break; }
       // rescale only when some row of the warp gained more than 2^8 (the loads and stores of
       // tensor memory are warp-wide, so the warp decides together)
       if (__any_sync(0xffffffffu, m_tile > m_ref + kRescaleLog2)) {
@@ -404,7 +417,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         const float alpha = ex2(m_ref - m_new);
         m_ref = m_new;
         l_run *= alpha;
-        if (j > 0) {
+        if (j > first_tile) {
           tc_fence_after();
 #pragma unroll 1
           for (int c = 0; c < D / 32; ++c) {
@@ -434,11 +447,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
 #pragma unroll
           for (int e = 0; e < 32; ++e) x[e] = ex2(fmaf(x[e], p.scale_log2, neg_m));
         } else {
-          const int nvis = vis_end - (key0 + c * 32);
+          const int nvis = vis_end - (key0 + c * 32), n0 = vis_begin - (key0 + c * 32);
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
             const float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
-            x[e] = e < nvis ? ex2(v + neg_m) : 0.f;
+            x[e] = e < nvis && e >= n0 ? ex2(v + neg_m) : 0.f;
           }
         }
 #pragma unroll
@@ -464,7 +477,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       __syncwarp();
       if (lane == 0) bar_arrive(my_p_full);
     }
-    if (alive && !__all_sync(0xffffffffu, bar_wait(my_pv_full, (ntiles - 1) & 1, abort_flag, 11))) alive = false;
+    if (alive && !__all_sync(0xffffffffu, bar_wait(my_pv_full, (ntiles - 1 - first_tile) & 1, abort_flag, 11))) alive = false;
     if (alive) {
       tc_fence_after();
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
@@ -576,12 +589,12 @@ int attention_tc_status(int *out4, bool clear) {
 
 using namespace eb;
 
-extern "C" int eb_attention_prefill_tc(const void *q, const void *k, const void *v, void *out, const void *mask,
+static int prefill_tc_impl(const void *q, const void *k, const void *v, void *out, const void *mask,
                                        long long q_batch_stride, long long q_row_stride, long long k_batch_stride,
                                        long long k_row_stride, long long v_batch_stride, long long v_row_stride,
                                        long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
-                                       int heads, int q_len, int kv_len, int head_dim, int causal, float scale, int dtype,
-                                       void *stream) {
+                                       int heads, int q_len, int kv_len, int head_dim, int causal, int window, float scale,
+                                       int dtype, void *stream) {
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "attention_prefill: fp16 or bf16 only (dtype %d)", dtype);
   EB_REQUIRE(head_dim == 64 || head_dim == 128, "attention_prefill: head_dim %d not supported (64 or 128)", head_dim);
@@ -594,6 +607,7 @@ extern "C" int eb_attention_prefill_tc(const void *q, const void *k, const void 
   for (long long s : strides) EB_REQUIRE(s % 8 == 0, "attention_prefill: strides must be multiples of 8 elements");
   EB_REQUIRE(kv_len >= q_len || !causal, "attention_prefill: causal attention needs kv_len >= q_len");
   EB_REQUIRE(scale > 0.f, "attention_prefill: the scale must be positive");
+  EB_REQUIRE(window >= 0 && (window == 0 || causal), "attention_prefill: a window needs the causal mask");
   cudaStream_t st = as_stream(stream);
   const long long hd = (long long)heads * head_dim;
   CUtensorMap mq, mk, mv;
@@ -602,11 +616,33 @@ extern "C" int eb_attention_prefill_tc(const void *q, const void *k, const void 
   if ((rc = tc_map3(&mq, q, dtype, hd, q_len, batch, q_row_stride, q_batch_stride, kRows))) return rc;
   if ((rc = tc_map3(&mk, k, dtype, hd, kv_len, batch, k_row_stride, k_batch_stride, kKeys))) return rc;
   TcParams p{};
-  p.B = batch; p.H = heads; p.Sq = q_len; p.Sk = kv_len; p.causal = causal;
+  p.B = batch; p.H = heads; p.Sq = q_len; p.Sk = kv_len; p.causal = causal; p.window = window;
   p.scale_log2 = scale * kLog2eTc;
   p.mask = mask; p.mask_bs = mask_batch_stride;
   p.mask_vec = mask && aligned16(mask) && mask_batch_stride % 8 == 0;
   p.o = out; p.o_bs = o_batch_stride; p.o_rs = o_row_stride;
   if (dtype == EB_F16) return head_dim == 64 ? launch_tc<__half, 64>(mq, mk, mv, p, st) : launch_tc<__half, 128>(mq, mk, mv, p, st);
   return head_dim == 64 ? launch_tc<__nv_bfloat16, 64>(mq, mk, mv, p, st) : launch_tc<__nv_bfloat16, 128>(mq, mk, mv, p, st);
+}
+
+extern "C" int eb_attention_prefill_tc(const void *q, const void *k, const void *v, void *out, const void *mask,
+                                       long long q_batch_stride, long long q_row_stride, long long k_batch_stride,
+                                       long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                                       long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
+                                       int heads, int q_len, int kv_len, int head_dim, int causal, float scale, int dtype,
+                                       void *stream) {
+  return prefill_tc_impl(q, k, v, out, mask, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
+                         o_batch_stride, o_row_stride, mask_batch_stride, batch, heads, q_len, kv_len, head_dim, causal, 0, scale, dtype,
+                         stream);
+}
+
+extern "C" int eb_attention_prefill_window_tc(const void *q, const void *k, const void *v, void *out, const void *mask,
+                                       long long q_batch_stride, long long q_row_stride, long long k_batch_stride,
+                                       long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                                       long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
+                                       int heads, int q_len, int kv_len, int head_dim, int window, float scale, int dtype,
+                                       void *stream) {
+  return prefill_tc_impl(q, k, v, out, mask, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
+                         o_batch_stride, o_row_stride, mask_batch_stride, batch, heads, q_len, kv_len, head_dim, 1, window, scale, dtype,
+                         stream);
 }

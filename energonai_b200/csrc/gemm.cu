@@ -34,6 +34,7 @@
 #include <type_traits>
 
 #include "comm.cuh"
+#include "gated.cuh"
 
 namespace eb {
 namespace {
@@ -92,6 +93,13 @@ struct GemmParams {
   const void *ln_x;
   long long ln_ldx;
   float ln_eps;
+  // Normal orientation, grouped (tile_group != null): W holds the [N, K] weights of several groups
+  // one below the other; row tile i of A (128 rows) is multiplied by those of group tile_group[i].
+  // Only the first *live_tiles row tiles are processed.  Both are read at run time.
+  const int *tile_group, *live_tiles;
+  // gated (normal orientation): columns come in blocks of 8 gates and their 8 ups; C is [M, N/2]
+  int gated;
+  float gate_limit, gate_alpha;
 };
 
 // ---- PTX wrappers ---------------------------------------------------------------------------
@@ -246,6 +254,7 @@ template <int BN, bool SWAP> struct Scheduler {
         if (end > tile_start && tile_start > pos) { h0 = tile_start; h1 = end; end = tile_start; }
       }
     } else {
+      if (p.live_tiles) lane_tiles = min(lane_tiles, *p.live_tiles);
       pos = blockIdx.x;
       end = lane_tiles * col_tiles;
     }
@@ -290,6 +299,9 @@ template <int BN, bool SWAP> struct Scheduler {
     return true;
   }
 };
+
+// First weight row of the group that a row tile of A belongs to.
+__device__ __forceinline__ int group_row(const GemmParams &p, int lane_tile) { return p.tile_group ? p.tile_group[lane_tile] * p.N : 0; }
 
 __device__ __forceinline__ float apply_act(float v, int act) {
   if (act == EB_ACT_RELU) return fmaxf(v, 0.f);
@@ -410,7 +422,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
       Scheduler<BN, SWAP> sw(p);
       Segment s;
       while (pre < stages && sw.next(s)) {
-        const int w_row = SWAP ? s.lane_row0 : s.col_tile * BN;
+        const int w_row = SWAP ? s.lane_row0 : s.col_tile * BN + group_row(p, s.lane_tile);
         for (int sk = s.sk0; sk < s.sk1 && pre < stages; ++sk, ++pre) {
           const uint32_t fb = full_bar + 8 * pre;
           if (lane == 0) mbar_expect_tx(fb, sk == nsk - 1 ? last_tx : full_tx);
@@ -427,7 +439,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
     uint32_t phase = 0;
     bool ok = true;
     while (ok && sched.next(s)) {
-      const int w_row = SWAP ? s.lane_row0 : s.col_tile * BN;
+      const int w_row = SWAP ? s.lane_row0 : s.col_tile * BN + group_row(p, s.lane_tile);
       const int x_row = SWAP ? s.col_tile * BN : s.lane_row0;
       for (int sk = s.sk0; sk < s.sk1; ++sk, ++iter) {
         const uint32_t fb = full_bar + 8 * stage;
@@ -624,6 +636,25 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
                   *reinterpret_cast<const uint4 *>(stage + row * kPitch + col);
           }
           __syncwarp();
+        }
+        tcgen05_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(tempty_bar + 8 * acc);
+      } else if (!SWAP && p.gated) {
+        // One output row per thread; 16 accumulator columns are 8 gates and their 8 ups.
+        const int m = s.lane_row0 + lrow;
+        T *c_row_ptr = reinterpret_cast<T *>(p.C) + (long long)m * p.ldc;
+#pragma unroll 2
+        for (int c = 0; c < BN / 16; ++c) {
+          const int n0 = s.col_tile * BN + c * 16;
+          if (n0 >= p.N) break;                              // warp-uniform (N is a multiple of 16)
+          float v[16], y[8];
+          tmem_ld16(t_base + c * 16, v);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) y[j] = gated_value(v[j], v[8 + j], p.gate_limit, p.gate_alpha);
+          Vec16<T> o;
+          o.pack(y);
+          if (m < p.M) o.store(c_row_ptr + n0 / 2);
         }
         tcgen05_fence_before();
         __syncwarp();
@@ -1437,6 +1468,45 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
   const size_t smem = kBarrierBytes + 1024 + (size_t)p.stages * (kLanes * 128 + bn * 128) + (p.rs ? 4 * 32 * 72 * 2 : 0);
   if ((rc = make_map(&tl, A, dtype, M, K, lda, kLanes))) return rc;
   if ((rc = make_map(&tc, W, dtype, N, K, ldw, bn))) return rc;
+  if (bn == 256)
+    return dtype == EB_F16 ? launch<__half, 256, false>(tl, tc, p, grid, smem, st)
+                           : launch<__nv_bfloat16, 256, false>(tl, tc, p, grid, smem, st);
+  return dtype == EB_F16 ? launch<__half, 128, false>(tl, tc, p, grid, smem, st)
+                         : launch<__nv_bfloat16, 128, false>(tl, tc, p, grid, smem, st);
+}
+
+extern "C" int eb_gemm_grouped(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, int M, int N, int K,
+                               int groups, const int32_t *tile_group, const int32_t *live_tiles, int gated, float limit, float alpha,
+                               int dtype, void *stream) {
+  EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "gemm_grouped: operands must be fp16 or bf16 (got dtype %d)", dtype);
+  EB_REQUIRE(M >= 0 && N > 0 && K > 0 && groups > 0, "gemm_grouped: bad size");
+  if (M == 0) return EB_OK;
+  EB_REQUIRE(A && W && C && tile_group && live_tiles, "gemm_grouped: null pointer");
+  EB_REQUIRE(M % kLanes == 0, "gemm_grouped: the rows come in whole tiles of %d (M=%d)", kLanes, M);
+  EB_REQUIRE(K % 8 == 0 && N % (gated ? 16 : 8) == 0, "gemm_grouped: K must be a multiple of 8, N of %d (K=%d N=%d)", gated ? 16 : 8, K, N);
+  EB_REQUIRE(lda >= K && ldw >= K && lda % 8 == 0 && ldw % 8 == 0 && ldc >= (gated ? N / 2 : N) && ldc % 8 == 0,
+             "gemm_grouped: row strides must be multiples of 8 and hold a row");
+  EB_REQUIRE((long long)groups * N < (1ll << 31), "gemm_grouped: too many weight rows");
+  EB_REQUIRE(aligned16(A) && aligned16(W) && aligned16(C), "gemm_grouped: pointers must be 16-byte aligned");
+  cudaStream_t st = as_stream(stream);
+  GemmParams p{};
+  p.M = M; p.N = N; p.K = K;
+  p.kblocks = (K + kBlockK - 1) / kBlockK;
+  p.C = C; p.ldc = ldc;
+  p.lane_rows = M; p.col_rows = N;
+  p.tile_group = tile_group; p.live_tiles = live_tiles;
+  p.gated = gated; p.gate_limit = limit; p.gate_alpha = alpha;
+  p.kpb = 1;
+  const long long lane_tiles = M / kLanes;
+  const int bn = lane_tiles * ((N + 255) / 256) >= sm_count() && N > 128 ? 256 : 128;
+  const long long tiles = lane_tiles * ((N + bn - 1) / bn);
+  const int grid = (int)(tiles < sm_count() ? tiles : sm_count());
+  p.stages = bn == 256 ? 4 : 6;
+  const size_t smem = kBarrierBytes + 1024 + (size_t)p.stages * (kLanes * 128 + bn * 128);
+  CUtensorMap tl, tc;
+  int rc;
+  if ((rc = make_map(&tl, A, dtype, M, K, lda, kLanes))) return rc;
+  if ((rc = make_map(&tc, W, dtype, (long long)groups * N, K, ldw, bn))) return rc;
   if (bn == 256)
     return dtype == EB_F16 ? launch<__half, 256, false>(tl, tc, p, grid, smem, st)
                            : launch<__nv_bfloat16, 256, false>(tl, tc, p, grid, smem, st);

@@ -1,0 +1,300 @@
+// RMS norm and what surrounds it in a decoder whose residual stream is kept in fp32:
+//
+//   rms_norm          y = x / sqrt(mean(x^2) + eps) * (w_offset + w), rows optionally written a
+//                     second time into a ring cache (row of position p = p mod capacity)
+//   rms_residual      x += norm(y), x fp32 in place, plus a copy of the new x in the operand type
+//                     for the products that read it.  y is a plain row, or the weighted sum of the
+//                     rows a mixture of experts produced for the token.  Optionally the router of
+//                     the mixture that follows is evaluated on the new row in the same launch
+//                     (generation steps: the row is already in registers, and one launch less
+//                     lies on the critical path).
+//
+// One CTA per row, the row register-resident in packs of 8; statistics, weights and the residual
+// are fp32 throughout.
+#include "common.cuh"
+#include "router.cuh"
+
+namespace eb {
+namespace {
+
+constexpr int kNormThreads = 256;
+
+template <typename T> __device__ __forceinline__ void load8(const T *p, float (&f)[8]);
+template <> __device__ __forceinline__ void load8<float>(const float *p, float (&f)[8]) {
+  const float4 a = *reinterpret_cast<const float4 *>(p), b = *reinterpret_cast<const float4 *>(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+template <> __device__ __forceinline__ void load8<__half>(const __half *p, float (&f)[8]) {
+  Vec16<__half> v;
+  v.load(p);
+  v.unpack(f);
+}
+template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16 *p, float (&f)[8]) {
+  Vec16<__nv_bfloat16> v;
+  v.load(p);
+  v.unpack(f);
+}
+template <typename T> __device__ __forceinline__ void store8(T *p, const float (&f)[8]);
+template <> __device__ __forceinline__ void store8<float>(float *p, const float (&f)[8]) {
+  *reinterpret_cast<float4 *>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4 *>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+}
+template <> __device__ __forceinline__ void store8<__half>(__half *p, const float (&f)[8]) {
+  Vec16<__half> v;
+  v.pack(f);
+  v.store(p);
+}
+template <> __device__ __forceinline__ void store8<__nv_bfloat16>(__nv_bfloat16 *p, const float (&f)[8]) {
+  Vec16<__nv_bfloat16> v;
+  v.pack(f);
+  v.store(p);
+}
+
+struct RmsParams {
+  const void *x;               // rows ldx apart
+  long long ldx;
+  const void *w;               // [n2] in the output type
+  float w_offset, eps, inv_count;
+  void *y;                     // rows ldy apart, or null
+  long long ldy;
+  int n2;
+  // ring cache: row (b, s) of the n1 = batch * rows_per_batch rows holds position pos0 + s of
+  // sequence b; the last `ring_rows` positions are kept at ring + b*ring_bs + (position mod ring_rows)*ring_ld
+  void *ring;
+  long long ring_bs, ring_ld;
+  int ring_rows, rows_per_batch;
+  const int *pos_dev;          // device scalar with pos0, or null (pos0 = 0)
+};
+
+template <typename TI, typename TO, int PACKS>
+__global__ void __launch_bounds__(kNormThreads) rms_norm_kernel(const RmsParams p) {
+  __shared__ float scratch[kNormThreads / 32];
+  griddep_wait();
+  griddep_launch();
+  const long long row = blockIdx.x;
+  const TI *x = reinterpret_cast<const TI *>(p.x) + row * p.ldx;
+  const TO *w = reinterpret_cast<const TO *>(p.w);
+  const int packs = p.n2 / 8;
+  float v[PACKS][8];
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * kNormThreads;
+    if (c >= packs) break;
+    load8<TI>(x + c * 8, v[i]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq = fmaf(v[i][e], v[i][e], sq);
+  }
+  const float r = rsqrtf(block_sum<kNormThreads>(sq, scratch) * p.inv_count + p.eps);
+  TO *ring = nullptr;
+  if (p.ring) {
+    const long long b = row / p.rows_per_batch;
+    const int s = (int)(row - b * p.rows_per_batch);
+    const int pos = (p.pos_dev ? *p.pos_dev : 0) + s;
+    if (p.rows_per_batch - s <= p.ring_rows && pos >= 0)
+      ring = reinterpret_cast<TO *>(p.ring) + b * p.ring_bs + (long long)(pos % p.ring_rows) * p.ring_ld;
+  }
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * kNormThreads;
+    if (c >= packs) break;
+    float wv[8];
+    load8<TO>(w + c * 8, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) wv[e] = v[i][e] * r * (p.w_offset + wv[e]);
+    if (p.y) store8<TO>(reinterpret_cast<TO *>(p.y) + row * p.ldy + c * 8, wv);
+    if (ring) store8<TO>(ring + c * 8, wv);
+  }
+}
+
+struct ResidualParams {
+  const void *y;               // rows ldy apart (T)
+  long long ldy;
+  // combine: row t of the sublayer's output = sum_k weights[t*top+k] * y[rows ? rows[t*top+k] : t*top+k],
+  // entries with idx < 0 left out
+  const int *idx, *rows;
+  const float *weights;
+  int top;
+  const void *w;               // [n2] T
+  float w_offset, eps, inv_count;
+  float *x;                    // fp32 residual stream, rows ldx apart, updated in place
+  long long ldx;
+  void *xt;                    // the new rows in T, rows ldt apart (null: not written)
+  long long ldt;
+  int n2;
+  // router of the mixture that follows (null: none)
+  const void *router;          // [experts][n2] T
+  int experts, r_top;
+  int *r_idx;
+  float *r_weights;
+};
+
+template <typename T, int PACKS, bool COMBINE>
+__global__ void __launch_bounds__(kNormThreads) rms_residual_kernel(const ResidualParams p) {
+  __shared__ float scratch[kNormThreads / 32];
+  extern __shared__ float dyn[];                   // router: [n2] row, [experts] logits
+  const long long row = blockIdx.x;
+  const T *w = reinterpret_cast<const T *>(p.w);
+  const int packs = p.n2 / 8;
+  griddep_wait();
+  griddep_launch();
+  float v[PACKS][8];
+  float sq = 0.f;
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * kNormThreads;
+    if (c >= packs) break;
+    if (COMBINE) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] = 0.f;
+      for (int k = 0; k < p.top; ++k) {
+        const long long a = row * p.top + k;
+        if (p.idx[a] < 0) continue;
+        const long long src = p.rows ? p.rows[a] : a;
+        const float s = p.weights[a];
+        float f[8];
+        load8<T>(reinterpret_cast<const T *>(p.y) + src * p.ldy + c * 8, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = fmaf(s, f[e], v[i][e]);
+      }
+    } else {
+      load8<T>(reinterpret_cast<const T *>(p.y) + row * p.ldy + c * 8, v[i]);
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq = fmaf(v[i][e], v[i][e], sq);
+  }
+  const float r = rsqrtf(block_sum<kNormThreads>(sq, scratch) * p.inv_count + p.eps);
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * kNormThreads;
+    if (c >= packs) break;
+    float wv[8], xv[8];
+    load8<T>(w + c * 8, wv);
+    load8<float>(p.x + row * p.ldx + c * 8, xv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) xv[e] = fmaf(v[i][e] * r, p.w_offset + wv[e], xv[e]);
+    store8<float>(p.x + row * p.ldx + c * 8, xv);
+    if (p.xt) store8<T>(reinterpret_cast<T *>(p.xt) + row * p.ldt + c * 8, xv);
+    if (p.router) {
+      // the router reads the row as the products do: rounded to the operand type
+#pragma unroll
+      for (int e = 0; e < 8; ++e) dyn[c * 8 + e] = to_f32<T>(from_f32<T>(xv[e]));
+    }
+  }
+  if (!p.router) return;
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float *z = dyn + p.n2;
+  for (int e = warp; e < p.experts; e += kNormThreads / 32) {
+    const T *wr = reinterpret_cast<const T *>(p.router) + (long long)e * p.n2;
+    float acc = 0.f;
+    for (int c = lane; c < packs; c += 32) {
+      float f[8];
+      load8<T>(wr + c * 8, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc = fmaf(f[j], dyn[c * 8 + j], acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) z[e] = acc;
+  }
+  __syncthreads();
+  if (warp == 0) route_warp(z, p.experts, p.r_top, p.r_idx + row * p.r_top, p.r_weights + row * p.r_top, nullptr, nullptr);
+}
+
+template <typename TI, typename TO>
+int launch_rms(const RmsParams &p, int n1, cudaStream_t st) {
+  const int packs = p.n2 / 8, per = (packs + kNormThreads - 1) / kNormThreads;
+  const dim3 g(n1), b(kNormThreads);
+  if (per <= 1) launch_pdl(rms_norm_kernel<TI, TO, 1>, g, b, 0, st, p);
+  else if (per <= 2) launch_pdl(rms_norm_kernel<TI, TO, 2>, g, b, 0, st, p);
+  else if (per <= 4) launch_pdl(rms_norm_kernel<TI, TO, 4>, g, b, 0, st, p);
+  else launch_pdl(rms_norm_kernel<TI, TO, 8>, g, b, 0, st, p);
+  return check_launch("rms_norm");
+}
+
+template <typename T, bool COMBINE>
+int launch_residual(const ResidualParams &p, int n1, cudaStream_t st) {
+  const int packs = p.n2 / 8, per = (packs + kNormThreads - 1) / kNormThreads;
+  const size_t smem = p.router ? (size_t)(p.n2 + p.experts) * sizeof(float) : 0;
+  const dim3 g(n1), b(kNormThreads);
+  auto go = [&](auto kern) -> int {
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+      cudaGetLastError();
+      return fail(EB_ECUDA, "rms_residual: cannot reserve %zu bytes of shared memory", smem);
+    }
+    launch_pdl(kern, g, b, smem, st, p);
+    return check_launch("rms_residual");
+  };
+  if (per <= 1) return go(rms_residual_kernel<T, 1, COMBINE>);
+  if (per <= 2) return go(rms_residual_kernel<T, 2, COMBINE>);
+  if (per <= 4) return go(rms_residual_kernel<T, 4, COMBINE>);
+  return go(rms_residual_kernel<T, 8, COMBINE>);
+}
+
+constexpr int kMaxNormWidth = 8 * 8 * kNormThreads;
+
+}  // namespace
+}  // namespace eb
+
+using namespace eb;
+
+extern "C" int eb_rms_norm(const void *x, long long ldx, int in_dtype, const void *w, float w_offset, float eps, void *y, long long ldy,
+                           int out_dtype, int n1, int n2, int count, void *ring, long long ring_batch_stride, long long ring_ld,
+                           int ring_rows, int rows_per_batch, const int32_t *pos_device, void *stream) {
+  if (n1 == 0) return EB_OK;
+  EB_REQUIRE(dtype_ok(in_dtype) && dtype_ok(out_dtype), "rms_norm: bad dtype %d / %d", in_dtype, out_dtype);
+  EB_REQUIRE(in_dtype == EB_F32 || in_dtype == out_dtype, "rms_norm: the input is fp32 or of the output type");
+  EB_REQUIRE(x && w && (y || ring), "rms_norm: null pointer");
+  EB_REQUIRE(n1 > 0 && n2 > 0 && n2 % 8 == 0 && n2 <= kMaxNormWidth, "rms_norm: width %d must be a multiple of 8, at most %d", n2, kMaxNormWidth);
+  EB_REQUIRE(count > 0 && count <= n2, "rms_norm: the mean is over 1..n2 elements");
+  EB_REQUIRE(ldx >= n2 && ldx % 8 == 0 && (!y || (ldy >= n2 && ldy % 8 == 0)), "rms_norm: row strides must be multiples of 8 and >= n2");
+  EB_REQUIRE(aligned16(x) && aligned16(w) && aligned16(y) && aligned16(ring), "rms_norm: pointers must be 16-byte aligned");
+  if (ring) {
+    EB_REQUIRE(ring_rows > 0 && rows_per_batch > 0 && n1 % rows_per_batch == 0, "rms_norm: the ring needs its rows and rows_per_batch");
+    EB_REQUIRE(ring_ld >= n2 && ring_ld % 8 == 0 && ring_batch_stride % 8 == 0, "rms_norm: ring strides must be multiples of 8");
+  }
+  RmsParams p{};
+  p.x = x; p.ldx = ldx; p.w = w; p.w_offset = w_offset; p.eps = eps; p.inv_count = 1.f / (float)count;
+  p.y = y; p.ldy = ldy; p.n2 = n2;
+  p.ring = ring; p.ring_bs = ring_batch_stride; p.ring_ld = ring_ld; p.ring_rows = ring_rows; p.rows_per_batch = rows_per_batch;
+  p.pos_dev = pos_device;
+  cudaStream_t st = as_stream(stream);
+  if (in_dtype == EB_F32) {
+    if (out_dtype == EB_F32) return launch_rms<float, float>(p, n1, st);
+    if (out_dtype == EB_F16) return launch_rms<float, __half>(p, n1, st);
+    return launch_rms<float, __nv_bfloat16>(p, n1, st);
+  }
+  if (out_dtype == EB_F16) return launch_rms<__half, __half>(p, n1, st);
+  return launch_rms<__nv_bfloat16, __nv_bfloat16>(p, n1, st);
+}
+
+extern "C" int eb_rms_residual(const void *y, long long ldy, int dtype, const int32_t *idx, const int32_t *rows, const float *weights,
+                               int top, const void *w, float w_offset, float eps, float *x, long long ldx, void *xt, long long ldt,
+                               int n1, int n2, int count, const void *router, int experts, int router_top, int32_t *router_idx,
+                               float *router_weights, void *stream) {
+  if (n1 == 0) return EB_OK;
+  EB_REQUIRE(dtype_ok(dtype), "rms_residual: bad dtype %d", dtype);
+  EB_REQUIRE(y && w && x, "rms_residual: null pointer");
+  EB_REQUIRE(n1 > 0 && n2 > 0 && n2 % 8 == 0 && n2 <= kMaxNormWidth, "rms_residual: width %d must be a multiple of 8, at most %d", n2, kMaxNormWidth);
+  EB_REQUIRE(count > 0 && count <= n2, "rms_residual: the mean is over 1..n2 elements");
+  EB_REQUIRE(ldy >= n2 && ldy % 8 == 0 && ldx >= n2 && ldx % 8 == 0 && (!xt || (ldt >= n2 && ldt % 8 == 0)),
+             "rms_residual: row strides must be multiples of 8 and >= n2");
+  EB_REQUIRE(aligned16(y) && aligned16(w) && aligned16(x) && aligned16(xt) && aligned16(router), "rms_residual: pointers must be 16-byte aligned");
+  EB_REQUIRE(!idx || (weights && top > 0), "rms_residual: a combination needs weights and top");
+  if (router) {
+    EB_REQUIRE(router_idx && router_weights, "rms_residual: the router needs its outputs");
+    EB_REQUIRE(experts > 0 && experts <= kMaxExperts && router_top > 0 && router_top <= experts,
+               "rms_residual: bad router (%d experts, top %d)", experts, router_top);
+  }
+  ResidualParams p{};
+  p.y = y; p.ldy = ldy; p.idx = idx; p.rows = rows; p.weights = weights; p.top = top;
+  p.w = w; p.w_offset = w_offset; p.eps = eps; p.inv_count = 1.f / (float)count;
+  p.x = x; p.ldx = ldx; p.xt = xt; p.ldt = ldt; p.n2 = n2;
+  p.router = router; p.experts = experts; p.r_top = router_top; p.r_idx = router_idx; p.r_weights = router_weights;
+  cudaStream_t st = as_stream(stream);
+#define EB_RES(T) (idx ? launch_residual<T, true>(p, n1, st) : launch_residual<T, false>(p, n1, st))
+  if (dtype == EB_F32) return EB_RES(float);
+  if (dtype == EB_F16) return EB_RES(__half);
+  return EB_RES(__nv_bfloat16);
+#undef EB_RES
+}

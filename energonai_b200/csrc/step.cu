@@ -150,8 +150,9 @@ extern "C" int eb_greedy_step(const void *logits, long long ld_logits, int batch
   EB_REQUIRE(logits && out_ids && kv_state && counter, "greedy_step: null pointer");
   EB_REQUIRE(ld_logits >= vocab && ld_out >= out_cols && out_cols >= 0, "greedy_step: leading dimensions smaller than the rows they hold");
   if (word_emb) {
-    EB_REQUIRE(pos_emb && hidden_out && hidden > 0 && vocab_rows > 0 && pos_rows > 0 && ld_hidden >= hidden,
-               "greedy_step: the embedding needs word and position tables, an output and their sizes");
+    EB_REQUIRE(hidden_out && hidden > 0 && vocab_rows > 0 && ld_hidden >= hidden,
+               "greedy_step: the embedding needs a word table, an output and their sizes");
+    EB_REQUIRE(!add_pos || (pos_emb && pos_rows > 0), "greedy_step: the position embedding needs its table and size");
   }
   StepParams p{};
   p.logits = logits; p.ld_logits = ld_logits; p.batch = batch; p.vocab = vocab;

@@ -1,0 +1,200 @@
+"""Latent attention with a sliding window, its ring cache, and the state of a batch of sequences.
+
+Per token a layer keeps one latent row c = RMSNorm(W_dkv h); keys and values of every head are
+linear maps of it, k = W_uk c, v = W_uv c.  Two evaluation orders give the same result:
+
+  prompt           k and v are expanded with one GEMM and a windowed attention kernel runs on them;
+  generation step  W_uk is moved onto the query and W_uv behind the attention, which then reads the
+                   cached latent rows themselves, once for all heads (eb_latent_decode).
+
+A layer may take another layer's latents instead of having its own projection (`kv_from`); it still
+has its own queries, up-projections, window and scale.
+
+Head sizes and the latent width are padded with zeros to what the tensor-core kernels take; zero
+columns change no product.
+"""
+import torch
+from torch import nn
+
+from ..attention import (LATENT_WIDTHS, attention_plain, attention_prefill_window, latent_decode)
+from ..gemm import gemm
+from ..moe import per_head
+from ..nn import RMSNorm1D, init_weight
+from ..norm import rms_norm
+from .attention import KVCache
+
+
+def round_up(n, m):
+    return -(-n // m) * m
+
+
+class LatentCache(KVCache):
+    """[batch, rows, latent] ring of latent rows: position p lives in row p mod rows.  `window` is the
+    longest window of the layers that read it (0: unlimited), so rows = min(positions, window).
+    A ring shorter than its window has never wrapped, which is why it can grow like a KVCache."""
+
+    def __init__(self, width, window, reserve=256):
+        super().__init__(reserve)
+        self.width, self.window = width, window
+
+    def rows_for(self, positions):
+        return min(positions, self.window) if self.window > 0 else positions
+
+    def prepare(self, batch, positions, dtype, device):
+        """For a new batch: room for `positions`; memory kept from an earlier batch of the same size
+        is used again when it has exactly the rows that are needed."""
+        self.reset()
+        rows = self.rows_for(positions)
+        if self.buf is None or self.buf.shape[:2] != (batch, rows) or self.buf.dtype != dtype or self.buf.device != device:
+            self.buf = torch.empty((batch, rows, self.width), dtype=dtype, device=device)
+
+    def grow(self, positions):
+        rows = self.rows_for(positions)
+        if rows > self.buf.shape[1]:
+            self.ensure(self.buf.shape[0], self.rows_for(positions + self.reserve), self.width, self.buf.dtype, self.buf.device, exact=True)
+
+    def keep(self, rows):
+        self.buf = self.buf.index_select(0, rows)
+
+
+class SequenceState:
+    """What a batch of sequences holds between steps: the caches, where each sequence begins in the
+    left-padded batch, and the common position.  `kv_state` = (position of the next token, its
+    successor) lives on the device, where captured steps advance it."""
+
+    def __init__(self, caches):
+        self.caches = caches                    # {layer: LatentCache}
+        self.first = self.kv_state = None
+        self.batch, self.length, self.padded = 0, 0, False
+
+    def begin(self, first, prompt_len, reserve, dtype, device):
+        """first: list with the number of padding positions in front of each sequence."""
+        B = len(first)
+        if self.first is None or self.first.numel() != B or self.first.device != device:
+            self.first = torch.empty(B, dtype=torch.int32, device=device)
+            self.kv_state = torch.empty(2, dtype=torch.int32, device=device)
+        self.first.copy_(torch.tensor(first, dtype=torch.int32))
+        self.kv_state.copy_(torch.tensor([prompt_len, prompt_len + 1], dtype=torch.int32))
+        self.batch, self.length, self.padded = B, prompt_len, any(first)
+        for c in self.caches.values():
+            c.prepare(B, prompt_len + max(0, reserve), dtype, device)
+            c.len = prompt_len
+
+    def ensure(self, positions):
+        for c in self.caches.values():
+            c.grow(positions)
+
+    def capacity(self):
+        """Positions the caches can take; None if every layer's ring holds its whole window."""
+        caps = [c.buf.shape[1] for c in self.caches.values() if c.window <= 0 or c.buf.shape[1] < c.window]
+        return min(caps) if caps else None
+
+    def set_length(self, n):
+        self.length = n
+        for c in self.caches.values():
+            c.len = n
+
+    def advance(self):
+        self.kv_state.add_(1)
+        self.set_length(self.length + 1)
+
+    def keep(self, rows):
+        """Only the sequences `rows` (list of indices) go on; the memory of the others is given back."""
+        if list(rows) == list(range(self.batch)):
+            return
+        sel = torch.tensor(list(rows), dtype=torch.long, device=self.first.device)
+        self.first = self.first.index_select(0, sel)
+        for c in self.caches.values():
+            c.keep(sel)
+        self.batch = len(rows)
+
+    def fork(self, rows):
+        """A state of its own for the sequences `rows`."""
+        out = SequenceState({k: LatentCache(c.width, c.window, c.reserve) for k, c in self.caches.items()})
+        for k, c in self.caches.items():
+            out.caches[k].buf, out.caches[k].len = c.buf, c.len
+        out.first, out.kv_state = self.first, self.kv_state.clone()
+        out.batch, out.length, out.padded = self.batch, self.length, self.padded
+        if list(rows) == list(range(self.batch)):
+            raise RuntimeError("fork: nothing would be left")
+        out.keep(rows)
+        return out
+
+
+class PromptContext:
+    """One prompt pass: shapes, padding, and the latents of the layers run so far."""
+
+    def __init__(self, state, batch, seq, mask):
+        self.state, self.batch, self.seq, self.mask = state, batch, seq, mask
+        self.first = state.first if state.padded else None
+        self.latents = {}
+
+
+class StepContext:
+    """One generation step."""
+
+    def __init__(self, state):
+        self.state, self.batch = state, state.batch
+        self.first = state.first if state.padded else None
+        self.pos = state.kv_state[0:1]
+
+
+class LatentAttention(nn.Module):
+    def __init__(self, layer, width, heads, dim, vdim, kv_rank, window, scale, eps, dtype, kv_from=None, device=None):
+        super().__init__()
+        self.layer, self.width, self.heads, self.dim, self.vdim, self.kv_rank = layer, width, heads, dim, vdim, kv_rank
+        self.window, self.scale, self.kv_from = window, scale, kv_from
+        wide = max(dim, vdim)
+        self.tensor_core_prompt = dtype != torch.float32 and wide <= 128
+        self.dk = self.dv = 64 if wide <= 64 else 128
+        if not self.tensor_core_prompt:
+            self.dk, self.dv = round_up(dim, 8), round_up(vdim, 8)
+        self.tensor_core_step = dtype != torch.float32 and kv_rank <= LATENT_WIDTHS[-1]
+        self.rank = min(w for w in LATENT_WIDTHS if w >= kv_rank) if self.tensor_core_step else round_up(kv_rank, 8)
+        self.q_rows = heads * self.dk
+        own = kv_from is None
+        self.in_proj = init_weight(self.q_rows + (self.rank if own else 0), width, dtype=dtype, device=device)   # queries | latent
+        self.latent_norm = RMSNorm1D(self.rank, eps=eps, count=kv_rank, offset=0.0, dtype=dtype, device=device) if own else None
+        self.kv_up = init_weight(heads * (self.dk + self.dv), self.rank, dtype=dtype, device=device)             # keys | values, head by head
+        self.k_absorb = init_weight(heads, self.rank, self.dk, dtype=dtype, device=device)                       # W_uk of a head, transposed
+        self.out_proj = init_weight(width, heads * self.dv, dtype=dtype, device=device)
+
+    @property
+    def source(self):
+        return self.layer if self.kv_from is None else self.kv_from
+
+    def prompt(self, h, ctx):
+        """h [batch*seq, width] -> [batch*seq, width]; fills this layer's cache."""
+        B, S = ctx.batch, ctx.seq
+        q = gemm(h, self.in_proj, static_weight=True)
+        if self.kv_from is None:
+            n = self.latent_norm
+            ctx.latents[self.layer] = rms_norm(q[:, self.q_rows:], n.weight, n.eps, offset=n.offset, count=n.count,
+                                               ring=ctx.state.caches[self.layer].buf, rows_per_batch=S)
+        c = ctx.latents[self.source]
+        kv = gemm(c, self.kv_up, static_weight=True).view(B, S, -1)
+        q3 = q.view(B, S, -1)[:, :, :self.q_rows]
+        k, v = kv[:, :, :self.q_rows], kv[:, :, self.q_rows:]
+        if self.tensor_core_prompt:
+            o = attention_prefill_window(q3, k, v, self.dk, self.window, mask=ctx.mask, scale=self.scale)
+        else:
+            o = attention_plain(q3, k, v, self.heads, self.dk, self.dv, window=self.window, scale=self.scale, first=ctx.first)
+        return gemm(o.view(B * S, -1), self.out_proj, static_weight=True)
+
+    def step(self, h, ctx):
+        """h [batch, width], one new position per sequence -> [batch, width]."""
+        B = ctx.batch
+        q = gemm(h, self.in_proj, static_weight=True)
+        cache = ctx.state.caches[self.source].buf
+        if self.kv_from is None:
+            n = self.latent_norm
+            rms_norm(q[:, self.q_rows:], n.weight, n.eps, offset=n.offset, count=n.count, write_out=False, ring=cache,
+                     rows_per_batch=1, pos_device=ctx.pos)
+        qa = per_head(q[:, :self.q_rows], self.k_absorb)
+        if self.tensor_core_step:
+            o = latent_decode(qa, cache, self.rank, self.heads, self.window, ctx.pos, self.scale, first=ctx.first)
+        else:
+            o = attention_plain(qa.view(B, 1, -1), cache, cache, self.heads, self.rank, self.rank, window=self.window, scale=self.scale,
+                                first=ctx.first, pos_device=ctx.pos, shared_kv=True).view(B, -1)
+        v = per_head(o, self.kv_up[self.q_rows:].view(self.heads, self.dv, self.rank))
+        return gemm(v, self.out_proj, static_weight=True)

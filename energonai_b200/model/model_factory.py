@@ -1,15 +1,10 @@
 """PipelineModel and the model factories with the reference's interface
 (energonai/model/model_factory.py:43-354), single pipeline stage.
 
-The generation loop keeps the reference's contract (input_ids / attention_mask in, token ids
-extended to max_tokens out; sampling through the same logits warpers; greedy = top_k 1) but
-does the work once: the prompt is embedded and run through the blocks a single time, every
-later step embeds and runs only the new token against the key/value caches, and the final
-norm + LM head see only the last position (the reference re-embeds the whole sequence and
-runs the head on every position each step, model_factory.py:112-131, with the same result for
-the sampled token)."""
+The generation loop is GenerationModel's (generation.py); this class says what a prompt pass and a
+generation step of a pre- / post-LayerNorm transformer are."""
 import os
-from typing import Callable, Optional
+from typing import Callable
 
 import torch
 from torch import dtype, nn
@@ -18,10 +13,11 @@ from ..nn import LayerNorm1D, can_fold
 from .downstream import LMHead1D
 from .embedding import Embedding1D
 from .endecoder import Block1D
+from .generation import GenerationModel
 from .mlp import gelu_impl
 
 
-class PipelineModel(nn.Module):
+class PipelineModel(GenerationModel):
     def __init__(self,
                  vocab_size: int = 50257,
                  num_tokentypes: int = 0,
@@ -48,9 +44,6 @@ class PipelineModel(nn.Module):
         self.hidden_size, self.first, self.last = hidden_size, first, last
         self.max_seq_len, self.model_name = max_seq_len, model_name
         self.disable_past_cache = disable_past_cache
-        self.eos_token_id = 50256          # the reference hard-codes this stop id (model_factory.py:133)
-        self.use_cuda_graph = True         # greedy generation steps are captured once and replayed
-        self.stop_check_every = 16         # replayed steps between two host reads of the stop condition
         # optional: generation steps run each layer as two launches (attention + one chained
         # kernel for the six GEMM / LayerNorm operations around it).  Off by default: measured on
         # OPT-13B, batch 16, the chained step is about 6 % slower than one kernel per operation
@@ -227,156 +220,63 @@ class PipelineModel(nn.Module):
             record.setdefault("hidden", []).append(last_hidden[:, -1, :].clone())
         return self.head(last_hidden)[:, -1, :]
 
-    def _graph_state(self, batch_size, tgt_len, model_dtype, dev, ids_dtype):
-        key = (batch_size, tgt_len, model_dtype, ids_dtype, tuple(b.attn.past_cache.buf.data_ptr() for b in self.blocks))
-        st = getattr(self, "_decode_state", None)
-        if st is None or st["key"] != key:
-            add_mask = torch.zeros((batch_size, tgt_len), dtype=model_dtype, device=dev)
-            st = {"key": key, "graph": None, "add_mask": add_mask, "mask4": add_mask.view(batch_size, 1, 1, tgt_len),
-                  "out_ids": torch.empty((batch_size, tgt_len), dtype=ids_dtype, device=dev),
-                  "tok": torch.empty((batch_size,), dtype=ids_dtype, device=dev),
-                  "kv_state": torch.zeros(2, dtype=torch.int32, device=dev),
-                  "chain_mode": self._chain_mode(batch_size, model_dtype)}
-            # the step's tail as one launch (eb_greedy_step) needs int64 ids, no token-type table
-            # and logits of the embedding's dtype; otherwise the framework's kernels do it
-            if (st["chain_mode"] is None and ids_dtype == torch.int64 and self.embed.tokentype_embeddings is None
-                    and self.embed.position_embeddings.weight.dtype == model_dtype
-                    and os.environ.get("EB_FUSED_TAIL", "1") != "0"):
-                st["hidden"] = torch.empty((batch_size, 1, self.hidden_size), dtype=model_dtype, device=dev)
-                st["step_counter"] = torch.zeros(1, dtype=torch.int32, device=dev)
-            self._decode_state = st
-        return st
+    # ---- what the generation loop (generation.py) asks of this model ----
+    @property
+    def model_dtype(self):
+        return self.norm.module.weight.dtype
 
-    @torch.inference_mode()
-    def forward(self, hidden_states=None, input_ids=None, attention_mask=None, seq_lens=None,
-                max_tokens: Optional[int] = None, top_k: Optional[int] = None, top_p: Optional[float] = None,
-                temperature: Optional[float] = None, record=None):
+    def _cache_key(self):
+        return tuple(b.attn.past_cache.buf.data_ptr() for b in self.blocks)
+
+    def _prompt_logits(self, input_ids, attention_mask, record=None):
         batch_size, cur_len = input_ids.shape
-        tgt_len = cur_len + 1 if not max_tokens else max_tokens
-        if cur_len >= tgt_len:
-            return input_ids
-        if attention_mask is None:
-            attention_mask = torch.ones_like(input_ids)
-        dev = input_ids.device
-        model_dtype = self.norm.module.weight.dtype
-        self.reserve_cache(tgt_len - cur_len)
-        greedy = top_k == 1 and (temperature is None or temperature > 0)
-        step_times = record.setdefault("step_events", []) if record is not None else None
-        from .. import _lib
-        launches0, replayed = _lib.launch_count, 0
-
-        def mark():
-            if step_times is not None:
-                ev = torch.cuda.Event(enable_timing=True)
-                ev.record()
-                step_times.append(ev)
-
-        # ---- prompt pass ----
-        add_mask_prompt = (1.0 - attention_mask.view(batch_size, -1).to(model_dtype)) * -10000.0
-        mark()
+        self._prompt_mask = (1.0 - attention_mask.view(batch_size, -1).to(self.model_dtype)) * -10000.0
         hidden_states = self.embed(input_ids)
-        mask4 = add_mask_prompt.view(batch_size, 1, 1, cur_len)
+        mask4 = self._prompt_mask.view(batch_size, 1, 1, cur_len)
         for block in self.blocks:
             hidden_states = block(hidden_states=hidden_states, attention_mask=mask4, first_cache=True)
         last_hidden = self.norm(hidden_states[:, -1:, :].contiguous())
-        logits = self.head(last_hidden)[:, -1, :]
         if record is not None:
-            record.setdefault("logits", []).append(logits.clone())
             record.setdefault("hidden", []).append(last_hidden[:, -1, :].clone())
-        tok = logits.argmax(-1) if greedy else self.generate(input_ids, logits, top_k=top_k, top_p=top_p,
-                                                             temperature=temperature)
-        mark()
-        if not max_tokens:
-            return tok
-        if torch.all(tok == self.eos_token_id):
-            return input_ids
+        return self.head(last_hidden)[:, -1, :]
 
-        # ---- generation steps ----
+    def _check_capacity(self, tgt_len):
         for blk in self.blocks:
             # steps driven by device-side positions cannot grow the cache: it must hold the whole call
             if not self.disable_past_cache and blk.attn.past_cache.capacity() < tgt_len:
                 raise RuntimeError(f"key/value cache holds {blk.attn.past_cache.capacity()} positions, {tgt_len} needed")
-        st = self._graph_state(batch_size, tgt_len, model_dtype, dev, input_ids.dtype)
+
+    def _new_step_state(self, batch_size, tgt_len, model_dtype, dev, ids_dtype):
+        add_mask = torch.zeros((batch_size, tgt_len), dtype=model_dtype, device=dev)
+        st = {"add_mask": add_mask, "mask4": add_mask.view(batch_size, 1, 1, tgt_len),
+              "kv_state": torch.zeros(2, dtype=torch.int32, device=dev),
+              "chain_mode": self._chain_mode(batch_size, model_dtype)}
+        # the step's tail as one launch (eb_greedy_step) needs int64 ids, no token-type table
+        # and logits of the embedding's dtype; otherwise the framework's kernels do it
+        if (st["chain_mode"] is None and ids_dtype == torch.int64 and self.embed.tokentype_embeddings is None
+                and self.embed.position_embeddings.weight.dtype == model_dtype
+                and os.environ.get("EB_FUSED_TAIL", "1") != "0"):
+            st["hidden"] = torch.empty((batch_size, 1, self.hidden_size), dtype=model_dtype, device=dev)
+            st["step_counter"] = torch.zeros(1, dtype=torch.int32, device=dev)
+        return st
+
+    def _seed_steps(self, st, tok, cur_len):
         st["add_mask"].zero_()
-        st["add_mask"][:, :cur_len] = add_mask_prompt
-        out_ids = st["out_ids"]
-        out_ids[:, :cur_len] = input_ids
-        out_ids[:, cur_len] = tok
-        st["tok"].copy_(tok)
-        st["kv_state"].copy_(torch.tensor([cur_len, cur_len + 1], dtype=torch.int32), non_blocking=False)
+        st["add_mask"][:, :cur_len] = self._prompt_mask
         if st.get("hidden") is not None:    # the first generated token's embedding; later ones come from the step's tail
             st["hidden"].copy_(self.embed(tok.view(-1, 1), past_key_values_length=cur_len))
-        use_graph = greedy and self.use_cuda_graph and (record is None or record.get("allow_graph", False))
-        produced = cur_len + 1
-        checked = cur_len + 1                                  # columns of out_ids already tested for the stop condition
-        for pos in range(cur_len + 1, tgt_len):
-            if use_graph:
-                if st["graph"] is None and pos == cur_len + 1:
-                    before = _lib.launch_count
-                    self._static_step(st)                      # eager once: also warms every kernel up
-                    st["launches"] = _lib.launch_count - before
-                elif st["graph"] is None:
-                    g = torch.cuda.CUDAGraph()
-                    before = _lib.launch_count
-                    with torch.cuda.graph(g):
-                        self._static_step(st)
-                    launches0 += _lib.launch_count - before    # captured, not executed
-                    st["graph"] = g
-                    g.replay()
-                    replayed += st["launches"]
-                else:
-                    st["graph"].replay()
-                    replayed += st["launches"]
-                mark()
-                # The reference stops when every sequence has just produced the stop token
-                # (model_factory.py:133-134).  Asking after every step would make the host wait for
-                # the device once per token; replays are queued ahead instead and the question is
-                # asked for a window of steps at a time.  Steps queued beyond the stopping point
-                # only wrote cache rows and columns that are cut off below.
-                if (pos - cur_len) % self.stop_check_every == 0 or pos == tgt_len - 1:
-                    hit = (out_ids[:, checked:pos + 1] == self.eos_token_id).all(0).nonzero()
-                    if hit.numel():
-                        produced = checked + int(hit[0])
-                        break
-                    checked = pos + 1
-                produced = pos + 1
-                continue
-            hidden_states = self.embed(tok.view(-1, 1), past_key_values_length=pos - 1)
-            mask4 = st["add_mask"][:, :pos].view(batch_size, 1, 1, pos)
-            for block in self.blocks:
-                hidden_states = block(hidden_states=hidden_states, attention_mask=mask4, first_cache=False)
-            logits = self._last_logits(hidden_states, record)
-            if record is not None:
-                record.setdefault("logits", []).append(logits.clone())
-            tok = logits.argmax(-1) if greedy else self.generate(out_ids[:, :pos], logits, top_k=top_k, top_p=top_p,
-                                                                 temperature=temperature)
-            out_ids[:, pos] = tok
-            mark()
-            if torch.all(tok == self.eos_token_id):
-                break
-            produced = pos + 1
+
+    def _eager_step(self, st, tok, pos, record=None):
+        batch_size = tok.shape[0]
+        hidden_states = self.embed(tok.view(-1, 1), past_key_values_length=pos - 1)
+        mask4 = st["add_mask"][:, :pos].view(batch_size, 1, 1, pos)
+        for block in self.blocks:
+            hidden_states = block(hidden_states=hidden_states, attention_mask=mask4, first_cache=False)
+        return self._last_logits(hidden_states, record)
+
+    def _end_generation(self, produced):
         for blk in self.blocks:                                # host bookkeeping of the cache length
             blk.attn.past_cache.len = produced - 1
-        self.launches_last_call = _lib.launch_count - launches0 + replayed   # kernels of this library executed
-        return out_ids[:, :produced].clone()
-
-    def get_logits_processor(self, top_k=None, top_p=None, temperature=None):
-        from transformers.generation import (LogitsProcessorList, TemperatureLogitsWarper, TopKLogitsWarper,
-                                             TopPLogitsWarper)
-        processor_list = LogitsProcessorList()
-        if temperature is not None and temperature != 1.0:
-            processor_list.append(TemperatureLogitsWarper(temperature))
-        if top_k is not None and top_k != 0:
-            processor_list.append(TopKLogitsWarper(top_k))
-        if top_p is not None and top_p < 1.0:
-            processor_list.append(TopPLogitsWarper(top_p))
-        return processor_list
-
-    def generate(self, input_ids, logits, top_k=None, top_p=None, temperature=None):
-        """model_factory.py:153-159 on last-position logits [batch, vocab]."""
-        logits = self.get_logits_processor(top_k, top_p, temperature)(input_ids, logits)
-        probs = torch.softmax(logits, -1, dtype=torch.float)
-        return torch.multinomial(probs, num_samples=1).squeeze(1)
 
 
 def create_pipeline_model(depth: int = 48, layer_partitions=None, **model_kwargs):

@@ -174,6 +174,27 @@ class _LayerNormParams(nn.Module):
         self.bias = nn.Parameter(torch.zeros(n, dtype=dtype, device=device))
 
 
+def init_weight(*shape, dtype=None, device=None, std=0.02):
+    """A weight in the layout of its kernel, N(0, std) until a checkpoint is loaded."""
+    w = nn.Parameter(torch.empty(*shape, dtype=dtype, device=device), requires_grad=False)
+    nn.init.normal_(w, std=std)
+    return w
+
+
+class RMSNorm1D(nn.Module):
+    """Parameters of x / sqrt(mean(x^2) + eps) * (offset + weight): offset 0 for a plain weight, 1 for
+    one stored around zero.  The mean is over the first `count` columns (zero padding follows)."""
+
+    def __init__(self, normalized_shape, eps, count=None, offset=0.0, dtype=None, device=None):
+        super().__init__()
+        self.normalized_shape, self.eps, self.count, self.offset = int(normalized_shape), eps, count or int(normalized_shape), offset
+        self.weight = nn.Parameter(torch.full((self.normalized_shape,), 1.0 - offset, dtype=dtype, device=device), requires_grad=False)
+
+    def forward(self, x):
+        from .norm import rms_norm
+        return rms_norm(_flat(x), self.weight, self.eps, offset=self.offset, count=self.count).view(x.shape)
+
+
 class LayerNorm1D(nn.Module):
     def __init__(self, normalized_shape, eps=1e-5, dtype=None, device=None):
         super().__init__()

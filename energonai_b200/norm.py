@@ -1,0 +1,60 @@
+"""Python entry to the RMS-norm kernels (eb_rms_norm / eb_rms_residual)."""
+import torch
+
+from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
+
+
+def _rows(t, what):
+    if t.dim() != 2 or t.stride(1) != 1:
+        raise RuntimeError(f"{what} must be [rows, width] with contiguous rows")
+    return t.stride(0)
+
+
+def rms_norm(x, weight, eps, offset=0.0, count=None, out=None, write_out=True, ring=None, rows_per_batch=1, pos_device=None):
+    """y = x / sqrt(mean(x^2) + eps) * (offset + weight) over the rows of x [n1, n2] (fp32 or the
+    weight's dtype); the mean is over the first `count` columns (the others are zero padding).
+    ring [batch, rows, >= n2]: the rows are also written to a ring cache, row (b, s) at
+    (position of the first row + s) mod rows, that position from pos_device (int32 scalar; None: 0).
+    Returns y in the weight's dtype (None with write_out=False)."""
+    require_cuda(x, weight, out, ring, pos_device)
+    ldx = _rows(x, "rms_norm: x")
+    n1, n2 = x.shape
+    if weight.numel() != n2:
+        raise RuntimeError("rms_norm: the weight must have one entry per column")
+    if out is None and write_out:
+        out = torch.empty((n1, n2), dtype=weight.dtype, device=x.device)
+    if ring is not None and (ring.dim() != 3 or ring.stride(2) != 1 or ring.dtype != weight.dtype or ring.shape[0] * rows_per_batch != n1
+                             or ring.shape[2] < n2):
+        raise RuntimeError("rms_norm: the ring must be [batch, rows, width] of the weight's dtype")
+    check(lib().eb_rms_norm(ptr(x), ldx, dtype_code(x.dtype), ptr(weight), float(offset), float(eps), ptr(out),
+                            _rows(out, "rms_norm: out") if out is not None else 0, dtype_code(weight.dtype), n1, n2, count or n2,
+                            ptr(ring), ring.stride(0) if ring is not None else 0, ring.stride(1) if ring is not None else 0,
+                            ring.shape[1] if ring is not None else 0, rows_per_batch, ptr(pos_device), stream_ptr()), "rms_norm")
+    return out
+
+
+def rms_residual(y, weight, eps, x, xt=None, offset=0.0, count=None, mix=None, router=None):
+    """x += rms_norm(y) in place, x [n1, n2] fp32; xt (the weight's dtype) receives the new rows.
+    mix = (idx, rows, weights) of a mixture of experts (idx / weights [n1, top], rows or None): the
+    row of y is then the weighted sum of the token's expert rows.  router = (weight [experts, n2],
+    experts, top): also returns (idx, weights) of the mixture that follows."""
+    require_cuda(y, weight, x, xt)
+    n1, n2 = x.shape
+    if x.dtype != torch.float32 or y.dtype != weight.dtype or y.shape[1] != n2 or weight.numel() != n2:
+        raise RuntimeError("rms_residual: x is fp32, y and the weight share a dtype, all of one width")
+    if mix is None and y.shape[0] != n1:
+        raise RuntimeError("rms_residual: one row of y per row of x")
+    idx, rows, mw = mix if mix is not None else (None, None, None)
+    r_idx = r_w = None
+    if router is not None:
+        rw, experts, top = router
+        if rw.shape[1] != n2 or not rw.is_contiguous() or rw.dtype != weight.dtype or rw.shape[0] < experts:
+            raise RuntimeError("rms_residual: the router weight must be contiguous [experts, width]")
+        r_idx = torch.empty((n1, top), dtype=torch.int32, device=x.device)
+        r_w = torch.empty((n1, top), dtype=torch.float32, device=x.device)
+    check(lib().eb_rms_residual(ptr(y), _rows(y, "rms_residual: y"), dtype_code(y.dtype), ptr(idx), ptr(rows), ptr(mw),
+                                idx.shape[1] if idx is not None else 0, ptr(weight), float(offset), float(eps), ptr(x),
+                                _rows(x, "rms_residual: x"), ptr(xt), _rows(xt, "rms_residual: xt") if xt is not None else 0, n1, n2,
+                                count or n2, ptr(router[0]) if router else None, router[1] if router else 0, router[2] if router else 0,
+                                ptr(r_idx), ptr(r_w), stream_ptr()), "rms_residual")
+    return (r_idx, r_w) if router is not None else None

@@ -22,9 +22,10 @@ def greedy_step(logits, out_ids, tok, kv_state, counter, word_emb=None, pos_emb=
     B, V = logits.shape
     hidden = 0
     if word_emb is not None:
-        if not (word_emb.dtype == pos_emb.dtype == hidden_out.dtype):
+        if word_emb.dtype != hidden_out.dtype or (pos_emb is not None and pos_emb.dtype != word_emb.dtype):
             raise RuntimeError("greedy_step: embedding tables and output must share a dtype")
-        if not (word_emb.is_contiguous() and pos_emb.is_contiguous() and hidden_out.stride(-1) == 1):
+        add_pos = add_pos and pos_emb is not None           # models without position embeddings
+        if not (word_emb.is_contiguous() and (pos_emb is None or pos_emb.is_contiguous()) and hidden_out.stride(-1) == 1):
             raise RuntimeError("greedy_step: embedding tables must be contiguous")
         hidden = word_emb.shape[1]
         hidden_out = hidden_out.view(B, hidden) if hidden_out.dim() != 2 else hidden_out

@@ -20,12 +20,15 @@ import torch
 
 from ..sharding import shard_model_state
 from ..tp import get_tp
+from .safetensors_io import load_safetensors
 
 __all__ = ["load_checkpoint", "load_state_dict", "remove_prefix"]
 
 
 def _load_file(path):
     """One checkpoint file as CPU tensors, memory-mapped where the file format allows."""
+    if path.endswith(".safetensors"):
+        return load_safetensors(path)
     try:
         return torch.load(path, map_location="cpu", mmap=True, weights_only=True)
     except (RuntimeError, ValueError):
@@ -41,6 +44,8 @@ def load_state_dict(path):
     if not os.path.isdir(path):
         raise FileNotFoundError(f"checkpoint {path} is neither a file nor a directory")
     files = sorted(os.path.join(path, f) for f in os.listdir(path) if os.path.isfile(os.path.join(path, f)))
+    # a model folder keeps its weights in *.safetensors beside its configuration
+    files = [f for f in files if f.endswith(".safetensors")] or files
     workers = max(1, min(int(os.environ.get("LOAD_N_PROC", "1")), len(files)))
     merged = {}
     if workers > 1:

@@ -335,6 +335,76 @@ EB_API int eb_decode_chain(const eb_chain_op *ops, int n_ops, int M, int dtype, 
                     size_t workspace_bytes, eb_comm *comm, void *stream);
 EB_API size_t eb_decode_chain_workspace_bytes(const eb_chain_op *ops, int n_ops, int M);
 
+/* ---- products of a mixture of experts, 32-bit products ---------------------------------------- */
+
+/* The prompt-orientation GEMM with several groups of weights: row tile i of A (128 rows) is
+ * multiplied by the weights of group tile_group[i].  W holds the groups' [N, K] matrices one below
+ * the other ([groups * N, K], rows ldw apart); only the first *live_tiles row tiles are processed
+ * (both device memory, read at run time).  M, a multiple of 128, is the room A and C have.
+ * gated != 0: the columns of a group come in blocks of 8 gates and their 8 ups and
+ *   C[m][8b + j] = g * sigmoid(alpha * g) * (u + 1),  g = min(gate, limit), u = clamp(up, -limit, limit)
+ * (C is [M, N/2]), the activation in fp32 on the accumulators.  fp16 / bf16. */
+EB_API int eb_gemm_grouped(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, int M, int N, int K,
+                    int groups, const int32_t *tile_group, const int32_t *live_tiles, int gated, float limit, float alpha,
+                    int dtype, void *stream);
+
+/* The same kind of product for a handful of rows per group (generation steps), as one pass over
+ * the weights of the groups that have rows.  idx != NULL: entry i of the list (rows entries)
+ * belongs to group idx[i] (negative: none), reads row i / a_div of A and writes row i of C.  idx
+ * NULL: every group takes all rows, with group strides on A and C (heads of an absorbed attention
+ * projection).  Strides in elements; gated as above. */
+EB_API int eb_grouped_skinny(const void *A, long long lda, long long a_group_stride, int a_div, const void *W,
+                      long long w_group_stride, long long ldw, void *C, long long ldc, long long c_group_stride,
+                      const int32_t *idx, int rows, int groups, int N, int K, int gated, float limit, float alpha, int dtype,
+                      void *stream);
+
+/* C = A . W^T in true 32-bit.  Strided groups, or row tiles with their group (one of the two). */
+EB_API int eb_gemm_f32(const float *A, long long lda, long long a_group_stride, const float *W, long long ldw,
+                long long w_group_stride, float *C, long long ldc, long long c_group_stride, int M, int N, int K, int groups,
+                const int32_t *tile_group, const int32_t *live_tiles, void *stream);
+
+/* The gated activation alone: x [n1, 2*half] in the 8 + 8 column order -> y [n1, half]. */
+EB_API int eb_gated_act(const void *x, long long ldx, void *y, long long ldy, int n1, int half, float limit, float alpha,
+                 int dtype, void *stream);
+
+/* Router of a mixture: idx[t][k], weights[t][k] = the `top` largest softmax scores over all experts
+ * of logits[t] (fp32, not renormalised; the lowest index among equals).  first (or NULL): rows
+ * t with t mod rows_per_batch < first[t / rows_per_batch] are padding and get idx -1.  With counts
+ * (zero on entry), ranks[t][k] = the choice's place among its expert's rows. */
+EB_API int eb_moe_route(const float *logits, long long ld, int tokens, int experts, int top, const int32_t *first,
+                 int rows_per_batch, int32_t *idx, float *weights, int32_t *counts, int32_t *ranks, void *stream);
+
+/* Row layout in which every expert owns whole 128-row tiles: offsets[e], tile_group[] (at most
+ * max_tiles), *live_tiles; counts are zeroed for the next batch. */
+EB_API int eb_moe_plan(int32_t *counts, int experts, int32_t *offsets, int32_t *tile_group, int max_tiles, int32_t *live_tiles,
+                void *stream);
+
+/* rows[t][k] = offsets[idx] + rank (or -1) and out[rows[t][k]] = x[t]; top <= 32. */
+EB_API int eb_moe_permute(const void *x, long long ldx, int n2, int dtype, int tokens, int top, const int32_t *idx,
+                   const int32_t *ranks, const int32_t *offsets, int32_t *rows, void *out, long long ldo, int max_rows,
+                   void *stream);
+
+/* ---- RMS norm ---------------------------------------------------------------------------------- */
+
+/* y = x / sqrt(sum(x^2) / count + eps) * (w_offset + w) over n1 rows of n2 elements (count < n2: the
+ * row is zero-padded).  x is fp32 or of the output type, w of the output type; fp32 inside.  ring
+ * (or NULL): the rows also go to a ring cache, row (b, s) of n1 = batch * rows_per_batch to row
+ * (pos0 + s) mod ring_rows of sequence b, pos0 read from pos_device (NULL: 0); of a longer prompt
+ * only the last ring_rows positions are kept. */
+EB_API int eb_rms_norm(const void *x, long long ldx, int in_dtype, const void *w, float w_offset, float eps, void *y,
+                long long ldy, int out_dtype, int n1, int n2, int count, void *ring, long long ring_batch_stride,
+                long long ring_ld, int ring_rows, int rows_per_batch, const int32_t *pos_device, void *stream);
+
+/* x += norm(y) with the residual stream x in fp32, in place; xt (or NULL) receives the new rows in
+ * `dtype`.  idx != NULL: y is the output of a mixture, the row of token t being
+ * sum_k weights[t][k] * y[rows ? rows[t][k] : t*top + k] over the k with idx[t][k] >= 0.
+ * router (or NULL, [experts][n2]): the router of the mixture that follows is evaluated on the new
+ * row as rounded to `dtype` (as eb_moe_route). */
+EB_API int eb_rms_residual(const void *y, long long ldy, int dtype, const int32_t *idx, const int32_t *rows,
+                    const float *weights, int top, const void *w, float w_offset, float eps, float *x, long long ldx, void *xt,
+                    long long ldt, int n1, int n2, int count, const void *router, int experts, int router_top,
+                    int32_t *router_idx, float *router_weights, void *stream);
+
 /* ---- the tail of a greedy generation step ----------------------------------------------------- */
 
 /* Replaces, per step, the arg-max / concatenate / embed sequence of the reference's generation
@@ -384,6 +454,38 @@ EB_API int eb_attention_prefill_tc(const void *q, const void *k, const void *v, 
                             long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
                             int heads, int q_len, int kv_len, int head_dim, int causal, float scale, int dtype,
                             void *stream);
+
+/* eb_attention_prefill_tc with a sliding window: row i sees the keys j with 0 <= i - j < window
+ * (window 0: all up to i). */
+EB_API int eb_attention_prefill_window_tc(const void *q, const void *k, const void *v, void *out, const void *mask,
+                            long long q_batch_stride, long long q_row_stride, long long k_batch_stride,
+                            long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                            long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
+                            int heads, int q_len, int kv_len, int head_dim, int window, float scale, int dtype,
+                            void *stream);
+
+/* Windowed causal attention for any head sizes and fp32 / fp16 / bf16 on the CUDA cores: query row
+ * i holds position pos0 + i (pos0 from pos_device, NULL: 0) and sees the positions
+ * max(first[b], its own - window + 1) .. its own; the key / value of position j is row
+ * j mod ring_rows.  Head strides may be 0 (keys shared by the heads). */
+EB_API int eb_attention_plain(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+                       long long q_row_stride, long long q_head_stride, long long k_batch_stride, long long k_row_stride,
+                       long long k_head_stride, long long v_batch_stride, long long v_row_stride, long long v_head_stride,
+                       long long o_batch_stride, long long o_row_stride, long long o_head_stride, int batch, int heads,
+                       int q_len, int k_dim, int v_dim, int window, int ring_rows, const int32_t *pos_device,
+                       const int32_t *first, float scale, int dtype, void *stream);
+
+/* Generation step of latent attention with absorbed projections: q [batch][heads * rank] are the
+ * queries in latent space, the cached latent row of a position is key and value of every head,
+ *   out[b][h] = sum_j softmax_j(scale * q[b][h] . c[b][j]) c[b][j]
+ * over the positions max(first[b], pos - window + 1) .. pos (window 0: all), position j in cache row
+ * j mod ring_rows.  rank 64, 128, 256, 384 or 512.  nsplit > 1 splits the positions over that many
+ * CTAs per (sequence, head tile) and merges them in a second launch through `scratch`. */
+EB_API int eb_latent_decode(const void *q, long long q_batch_stride, const void *cache, long long cache_batch_stride,
+                     long long cache_row_stride, int ring_rows, void *out, long long out_batch_stride, int batch, int heads,
+                     int rank, int window, const int32_t *pos_device, const int32_t *first, float scale, int dtype,
+                     int nsplit, void *scratch, size_t scratch_bytes, void *stream);
+EB_API size_t eb_latent_decode_scratch_bytes(int batch, int heads, int rank, int nsplit);
 
 /* The same product for one new query row per sequence against the cached keys/values (the
  * generation step; replaces the torch.cat past_cache reads of attention.py:86-98 followed by
