@@ -95,21 +95,24 @@ moe_permute_kernel(const uint4 *x, long long ldx16, int packs, int tokens, int t
   const int t = blockIdx.x * (kPermuteThreads / 32) + warp;
   if (t >= tokens) return;
   const long long a0 = (long long)t * top;
-  int dest = -1;                                   // lane k: destination of choice k (top <= 32)
-  if (lane < top) {
-    const int e = idx[a0 + lane];
-    if (e >= 0) {
-      dest = offsets[e] + ranks[a0 + lane];
-      if (dest >= max_rows) dest = -1;
+  for (int k0 = 0; k0 < top; k0 += 32) {
+    int dest = -1;                                 // lane k: destination of choice k0 + k
+    if (k0 + lane < top) {
+      const int e = idx[a0 + k0 + lane];
+      if (e >= 0) {
+        dest = offsets[e] + ranks[a0 + k0 + lane];
+        if (dest >= max_rows) dest = -1;
+      }
+      rows[a0 + k0 + lane] = dest;
     }
-    rows[a0 + lane] = dest;
-  }
-  for (int c = lane; c - lane < packs; c += 32) {
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (c < packs) v = x[(long long)t * ldx16 + c];
-    for (int k = 0; k < top; ++k) {
-      const int d = __shfl_sync(0xffffffffu, dest, k);
-      if (d >= 0 && c < packs) out[(long long)d * ldo16 + c] = v;
+    const int n = min(32, top - k0);
+    for (int c = lane; c - lane < packs; c += 32) {
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (c < packs) v = x[(long long)t * ldx16 + c];
+      for (int k = 0; k < n; ++k) {
+        const int d = __shfl_sync(0xffffffffu, dest, k);
+        if (d >= 0 && c < packs) out[(long long)d * ldo16 + c] = v;
+      }
     }
   }
 }
@@ -284,7 +287,7 @@ extern "C" int eb_moe_permute(const void *x, long long ldx, int n2, int dtype, i
   const int per = 16 / dtype_size(dtype);
   EB_REQUIRE(n2 > 0 && n2 % per == 0 && ldx % per == 0 && ldo % per == 0 && ldx >= n2 && ldo >= n2, "moe_permute: rows must be whole 16-byte packs");
   EB_REQUIRE(aligned16(x) && aligned16(out), "moe_permute: pointers must be 16-byte aligned");
-  EB_REQUIRE(tokens > 0 && top > 0 && top <= 32 && max_rows > 0, "moe_permute: bad sizes (top %d, at most 32)", top);
+  EB_REQUIRE(tokens > 0 && top > 0 && max_rows > 0, "moe_permute: bad sizes");
   launch_pdl(moe_permute_kernel, dim3((tokens + 7) / 8), dim3(kPermuteThreads), 0, as_stream(stream), reinterpret_cast<const uint4 *>(x),
              ldx / per, n2 / per, tokens, top, idx, ranks, offsets, rows, reinterpret_cast<uint4 *>(out), ldo / per, max_rows);
   return check_launch("moe_permute");

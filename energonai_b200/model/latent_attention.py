@@ -145,9 +145,10 @@ class LatentAttention(nn.Module):
         self.layer, self.width, self.heads, self.dim, self.vdim, self.kv_rank = layer, width, heads, dim, vdim, kv_rank
         self.window, self.scale, self.kv_from = window, scale, kv_from
         wide = max(dim, vdim)
-        self.tensor_core_prompt = dtype != torch.float32 and wide <= 128
-        self.dk = self.dv = 64 if wide <= 64 else 128
-        if not self.tensor_core_prompt:
+        self.tensor_core_prompt = dtype != torch.float32 and wide <= 128 and scale > 0
+        if self.tensor_core_prompt:
+            self.dk = self.dv = 64 if wide <= 64 else 128
+        else:
             self.dk, self.dv = round_up(dim, 8), round_up(vdim, 8)
         self.tensor_core_step = dtype != torch.float32 and kv_rank <= LATENT_WIDTHS[-1]
         self.rank = min(w for w in LATENT_WIDTHS if w >= kv_rank) if self.tensor_core_step else round_up(kv_rank, 8)
@@ -174,7 +175,7 @@ class LatentAttention(nn.Module):
         c = ctx.latents[self.source]
         kv = gemm(c, self.kv_up, static_weight=True).view(B, S, -1)
         q3 = q.view(B, S, -1)[:, :, :self.q_rows]
-        k, v = kv[:, :, :self.q_rows], kv[:, :, self.q_rows:]
+        k, v = kv[:, :, :self.q_rows], kv[:, :, self.q_rows:]        # (keys have as many rows as queries)
         if self.tensor_core_prompt:
             o = attention_prefill_window(q3, k, v, self.dk, self.window, mask=ctx.mask, scale=self.scale)
         else:

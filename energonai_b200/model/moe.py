@@ -8,7 +8,7 @@ import torch
 from torch import nn
 
 from ..gemm import gemm
-from ..moe import SortedRows, grouped_gemm, route, skinny_experts
+from ..moe import SKINNY_MAX_ENTRIES, SortedRows, grouped_gemm, route, skinny_experts
 from ..nn import init_weight
 from .latent_attention import round_up
 
@@ -18,8 +18,8 @@ SKINNY_MAX_TOKENS = 128      # up to here an expert gets a handful of rows: stre
 class MixtureOfExperts(nn.Module):
     def __init__(self, width, experts, top, ff, limit, alpha, dtype, device=None):
         super().__init__()
-        if not 0 < top <= min(experts, 32):
-            raise ValueError(f"mixture of experts: top {top} of {experts} experts (at most 32)")
+        if not 0 < top <= experts:
+            raise ValueError(f"mixture of experts: top {top} of {experts} experts")
         self.experts, self.top, self.ff, self.gate = experts, top, ff, (limit, alpha)
         self.ff_padded = round_up(ff, 8)
         self.router = init_weight(round_up(experts, 8), width, dtype=dtype, device=device)
@@ -28,7 +28,7 @@ class MixtureOfExperts(nn.Module):
         self._counts = None
 
     def skinny(self, tokens):
-        return tokens <= SKINNY_MAX_TOKENS and self.router.dtype != torch.float32
+        return tokens <= SKINNY_MAX_TOKENS and tokens * self.top <= SKINNY_MAX_ENTRIES and self.router.dtype != torch.float32
 
     def router_for_step(self, tokens):
         """(weight, experts, top) for the residual kernel to evaluate the router itself, or None."""

@@ -6,6 +6,8 @@ from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
 
 ROW_TILE = 128           # rows of one expert come in tiles of this many in the sorted layout
 
+SKINNY_MAX_ENTRIES = 10240   # (token, choice) pairs the weight-streaming product sorts in shared memory
+
 
 def route(logits, experts, top, first=None, rows_per_batch=0, counts=None):
     """logits [T, >= experts] fp32 -> idx [T, top] int32, weights [T, top] fp32 (softmax scores over

@@ -1,0 +1,250 @@
+"""Throughput of the latent-attention / mixture-of-experts decoder at sizes that resemble a real
+model's layers (random weights), beside an OPT-shaped PipelineModel of equal width, heads, depth and
+active feed-forward weights, and the time of every kernel of it next to its roofline and to the like
+kernel of the other model.  `bench.py --design tulezen` prints the result as one JSON line."""
+import json
+import os
+import statistics
+
+import torch
+
+SIZES = {
+    # window, kv_rank, experts ... of a layer; every second layer takes its latents from the one before
+    "2048": dict(width=2048, heads=16, dim=128, kv_rank=512, window=1024, experts=64, top=6, ff=1408, layers=8, vocab=32768),
+    "4096": dict(width=4096, heads=32, dim=128, kv_rank=512, window=4096, experts=32, top=4, ff=2048, layers=6, vocab=32768),
+}
+RUNS = [  # (size, batch, prompt, new tokens)
+    ("2048", 8, 1024, 64), ("2048", 64, 1024, 64), ("4096", 16, 512, 64), ("4096", 2, 4096, 64),
+]
+FLUSH_BYTES = 400 << 20      # a timed kernel cycles through operand copies of at least this size
+
+
+def peaks():
+    path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
+    d = json.load(open(path)) if os.path.exists(path) else {}
+    return {"hbm": d.get("hbm_gbs", 6650.0) * 1e9, "tensor": d.get("bf16_tflops", 1590.0) * 1e12,
+            "kind": "measured" if d else "fallback"}
+
+
+def make_tulezen(z):
+    from ..registry import build_model
+    layer = {"type": "latent_attention",
+             "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["dim"], "kv_rank": z["kv_rank"], "mask": {"size": z["window"]},
+                       "scale": z["dim"] ** -0.5},
+             "mlp": {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["ff"], "limit": 7.0}}}
+    layers = [dict(layer, mixer=dict(layer["mixer"], **({"kv_from": i - 1} if i % 2 else {}))) for i in range(z["layers"])]
+    torch.manual_seed(1)
+    return build_model("Tulezen", config_dict={"vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "layers": layers},
+                       dtype=torch.bfloat16, device="cuda")
+
+
+def make_opt(z, max_len):
+    from ..model import create_pipeline_model
+    torch.manual_seed(1)
+    ffn = (z["top"] * z["ff"] * 3 // 2 + 7) // 8 * 8            # as many feed-forward weights per token
+    with torch.device("cuda"):
+        m = create_pipeline_model(depth=z["layers"], vocab_size=z["vocab"], hidden_size=z["width"], max_seq_len=max_len,
+                                  num_heads=z["heads"], mlp_ratio=ffn / z["width"], activation=torch.nn.functional.relu,
+                                  is_decoder=True, fused_qkv=True, dtype=torch.bfloat16)
+    m.eos_token_id = -1
+    return m.eval()
+
+
+def timed_generation(model, vocab, B, S, new, reps=3):
+    ids = torch.randint(0, vocab, (B, S), device="cuda")
+    mask = torch.ones_like(ids)
+    out = []
+    for i in range(reps + 2):
+        rec = {"allow_graph": True}
+        model(input_ids=ids, attention_mask=mask, max_tokens=S + new, top_k=1, record=rec)
+        torch.cuda.synchronize()
+        if i >= 2:
+            ev = rec["step_events"]
+            steps = [a.elapsed_time(b) for a, b in zip(ev[3:-1], ev[4:])]
+            out.append((ev[0].elapsed_time(ev[1]), statistics.median(steps)))
+    pre, step = statistics.median(o[0] for o in out), statistics.median(o[1] for o in out)
+    return {"prefill_ms": pre, "prefill_tokens_per_s": B * S / pre * 1e3, "step_ms": step, "decode_tokens_per_s": B / step * 1e3}
+
+
+def time_calls(calls, reps=10):
+    """Median time of one call, from replays of a graph that runs all of `calls` (operand copies that
+    together exceed L2) back to back."""
+    for c in calls[:2]:
+        c()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for c in calls:
+            c()
+    ts = []
+    for i in range(reps + 3):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        g.replay()
+        b.record()
+        torch.cuda.synchronize()
+        if i >= 3:
+            ts.append(a.elapsed_time(b) * 1e3 / len(calls))
+    return statistics.median(ts)
+
+
+def copies(nbytes, most=64):
+    return max(2, min(most, -(-FLUSH_BYTES // max(1, int(nbytes)))))
+
+
+def kernel_table(z, B, S, T):
+    """[(phase, kernel, like kernel or None, us, bytes, flops)] for batch B at S cached positions
+    (generation step) and T prompt tokens in sequences of min(S, T)."""
+    from ..attention import (attention_decode, attention_prefill, attention_prefill_window, latent_decode)
+    from ..gemm import gemm
+    from ..kernel.cuda_native.layer_norm import layer_norm_forward
+    from ..moe import SortedRows, grouped_gemm, per_head, route, skinny_experts
+    from ..norm import rms_norm, rms_residual
+    bf, dev = torch.bfloat16, "cuda"
+    W, H, d, R, E, K, ff = z["width"], z["heads"], z["dim"], z["kv_rank"], z["experts"], z["top"], z["ff"]
+    win = z["window"]
+    keys = min(S, win)
+    rnd = lambda *s, dtype=bf: (torch.randn(*s, device=dev, dtype=torch.float32) * 0.05).to(dtype)
+    rows = []
+
+    def add(phase, name, like, us, nbytes, flops=0.0):
+        rows.append((phase, name, like, us, float(nbytes), float(flops)))
+
+    def product(phase, name, M, N, Kd, like=None, out32=False):
+        nb = 2 * (N * Kd + M * Kd) + (4 if out32 else 2) * M * N
+        ws = [rnd(N, Kd) for _ in range(copies(2 * N * Kd, 32))]
+        xs = [rnd(M, Kd) for _ in range(4)]
+        us = time_calls([lambda w=w, x=xs[i % 4]: gemm(x, w, out_dtype=torch.float32 if out32 else None, static_weight=True)
+                         for i, w in enumerate(ws)])
+        add(phase, name, like, us, nb, 2.0 * M * N * Kd)
+
+    # ---- generation step ----
+    product("step", "gemm in_proj", B, H * d + R, W)
+    product("step", "gemm out_proj", B, W, H * d)
+    pos = torch.tensor([S - 1], dtype=torch.int32, device=dev)
+    ring = [rnd(B, keys, R) for _ in range(copies(B * keys * R * 2))]
+    q = rnd(B, H * R)
+    add("step", "latent_decode", "attention_decode (OPT)", time_calls([lambda c=c: latent_decode(q, c, R, H, win, pos, 0.05) for c in ring]),
+        2 * B * keys * R + 4 * B * H * R, 4.0 * B * H * keys * R)
+    kv = [rnd(B, keys, 3 * H * d) for _ in range(copies(B * keys * 2 * H * d * 2))]
+    add("step", "attention_decode (OPT)", None, time_calls([lambda c=c: attention_decode(
+        c[:, :, 2 * H * d:], c[:, :, :H * d], c[:, :, H * d:2 * H * d], d, keys, q_in_cache=True) for c in kv]), 4 * B * keys * H * d)
+    del kv
+    w = rnd(R)
+    x = rnd(B, R)
+    add("step", "rms_norm to ring", "layer_norm (OPT)", time_calls([lambda c=c: rms_norm(x, w, 1e-5, write_out=False, ring=c, pos_device=pos)
+                                                                    for c in ring]), 4 * B * R)
+    del ring
+    ups = [rnd(H, R, d) for _ in range(copies(H * R * d * 2, 48))]
+    qh, o = rnd(B, H * d), rnd(B, H * R)
+    add("step", "per_head key absorb", "gemm out_proj", time_calls([lambda w=w: per_head(qh, w) for w in ups]), 2 * (H * R * d + B * H * (R + d)))
+    add("step", "per_head value up", "gemm out_proj", time_calls([lambda w=w: per_head(o, w.view(H, d, R)) for w in ups]),
+        2 * (H * R * d + B * H * (R + d)))
+    del ups
+    xs, xt, y, nw = torch.randn(B, W, device=dev), rnd(B, W), rnd(B, W), rnd(W)
+    routers = [rnd(E, W) for _ in range(16)]
+    add("step", "rms_residual + router", "layer_norm (OPT)", time_calls([lambda r=r: rms_residual(y, nw, 1e-5, xs, xt=xt, offset=1.0, router=(r, E, K))
+                                                                         for r in routers]), 12 * B * W + 2 * E * W)
+    lw, lb = rnd(W), rnd(W)
+    add("step", "layer_norm (OPT)", None, time_calls([lambda: layer_norm_forward(xt, lw, lb, 1e-5)] * 16), 4 * B * W)
+    g = torch.Generator(device=dev).manual_seed(3)
+    n_w = max(2, min(8, -(-FLUSH_BYTES // (6 * E * ff * W))))
+    gu = [rnd(E, 2 * ff, W) for _ in range(n_w)]
+    dn = [rnd(E, W, ff) for _ in range(n_w)]
+    idx = torch.rand(B, E, device=dev, generator=g).topk(K, -1).indices.to(torch.int32)
+    wts = torch.rand(B, K, device=dev)
+    act_e = int(idx.unique().numel())
+    a = rnd(B * K, ff)
+    add("step", "experts gate_up", "gemm out_proj", time_calls([lambda w=w: skinny_experts(xt, w, idx, K, gate=(7.0, 1.702)) for w in gu]),
+        2 * (act_e * 2 * ff * W + B * W + B * K * ff), 4.0 * B * K * ff * W)
+    add("step", "experts down", "gemm out_proj", time_calls([lambda w=w: skinny_experts(a, w, idx, 1) for w in dn]),
+        2 * (act_e * ff * W + B * K * (W + ff)), 2.0 * B * K * ff * W)
+    ym = rnd(B * K, W)
+    add("step", "rms_residual combine", "layer_norm (OPT)", time_calls([lambda: rms_residual(ym, nw, 1e-5, xs, xt=xt, offset=1.0, mix=(idx, None, wts))] * 16),
+        10 * B * W + 2 * B * K * W)
+
+    # ---- prompt ----
+    seq = min(S, T)
+    nB = T // seq
+    product("prompt", "gemm in_proj", T, H * d + R, W)
+    product("prompt", "gemm kv_up", T, 2 * H * d, R)
+    product("prompt", "gemm out_proj", T, W, H * d)
+    product("prompt", "gemm router", T, E, W, out32=True)
+    q3, kv3 = rnd(nB, seq, H * d), rnd(nB, seq, 2 * H * d)
+    n_c = 4
+    pairs = sum(min(i + 1, win) for i in range(seq))
+    add("prompt", "attention window", "attention causal (OPT)", time_calls([lambda: attention_prefill_window(q3, kv3[:, :, :H * d], kv3[:, :, H * d:], d, win)] * n_c),
+        2 * T * 4 * H * d, 4.0 * nB * H * d * pairs)
+    add("prompt", "attention causal (OPT)", None, time_calls([lambda: attention_prefill(q3, kv3[:, :, :H * d], kv3[:, :, H * d:], d)] * n_c),
+        2 * T * 4 * H * d, 4.0 * nB * H * d * seq * (seq + 1) / 2)
+    c = [rnd(T, R) for _ in range(copies(4 * T * R))]
+    add("prompt", "rms_norm latent", "layer_norm (OPT)", time_calls([lambda t=t: rms_norm(t, w, 1e-5) for t in c]), 4 * T * R)
+    del c
+    xs = [torch.randn(T, W, device=dev) for _ in range(copies(12 * T * W, 8))]
+    xts, ys = [rnd(T, W) for _ in xs], [rnd(T, W) for _ in xs]
+    add("prompt", "rms_residual", "layer_norm (OPT)", time_calls([lambda x=x, t=t, y=y: rms_residual(y, nw, 1e-5, x, xt=t, offset=1.0)
+                                                                  for x, t, y in zip(xs, xts, ys)]), 12 * T * W)
+    add("prompt", "layer_norm (OPT)", None, time_calls([lambda t=t: layer_norm_forward(t, lw, lb, 1e-5) for t in xts + ys]), 4 * T * W)
+    logits = torch.randn(T, E, device=dev)
+    counts = torch.zeros(E, dtype=torch.int32, device=dev)
+    n0, n1 = [torch.zeros(E, dtype=torch.int32, device=dev) for _ in range(2)]
+    add("prompt", "moe route", None, time_calls([lambda: route(logits, E, K, counts=n0)] * 4), 4 * T * E + 12 * T * K)
+    idx, wts, ranks = route(logits, E, K, counts=counts)
+    keep = counts.clone()
+
+    def sort_rows():
+        n1.copy_(keep)
+        return SortedRows(xts[0], idx, ranks, n1)
+    plan = sort_rows()
+    add("prompt", "moe plan + permute", "layer_norm (OPT)", time_calls([sort_rows] * 4), 2 * T * W * (1 + K))
+    live = int(plan.live_tiles.item()) * 128
+    add("prompt", "grouped gate_up", "gemm out_proj", time_calls([lambda w=w: grouped_gemm(plan.x, w, plan, gate=(7.0, 1.702)) for w in gu]),
+        2 * (E * 2 * ff * W + T * K * (W + ff)), 4.0 * T * K * ff * W)
+    act = grouped_gemm(plan.x, gu[0], plan, gate=(7.0, 1.702))
+    add("prompt", "grouped down", "gemm out_proj", time_calls([lambda w=w: grouped_gemm(act, w, plan) for w in dn]),
+        2 * (E * ff * W + T * K * (W + ff)), 2.0 * T * K * ff * W)
+    ym = grouped_gemm(act, dn[0], plan)
+    add("prompt", "rms_residual combine", "layer_norm (OPT)", time_calls([lambda x=x, t=t: rms_residual(ym, nw, 1e-5, x, xt=t, offset=1.0, mix=(idx, plan.rows, wts))
+                                                                          for x, t in zip(xs, xts)]), 10 * T * W + 2 * T * K * W)
+    return rows, {"active_experts": act_e, "sorted_rows": live, "routed_rows": T * K}
+
+
+def table_with_fractions(rows):
+    pk = peaks()
+    out = []
+    for phase, name, like, us, nbytes, flops in rows:
+        roof = max(nbytes / pk["hbm"], flops / pk["tensor"]) * 1e6
+        out.append({"phase": phase, "kernel": name, "us": round(us, 2), "roofline_us": round(roof, 2), "frac": round(roof / us, 3), "like": like,
+                    "bound": "hbm" if nbytes / pk["hbm"] >= flops / pk["tensor"] else "tensor"})
+    by = {(r["phase"], r["kernel"]): r["frac"] for r in out}
+    for r in out:
+        if r["like"]:
+            r["like_frac"] = by[(r["phase"], r["like"])]
+            r["ratio_to_like"] = round(r["frac"] / r["like_frac"], 2)
+    return out
+
+
+def run(kernels=True, generation=True):
+    from ..gemm import device_status
+    res = {"design": "tulezen", "dtype": "bf16", "data": "synthetic, random weights", "peaks": peaks(), "sizes": SIZES, "generation": [],
+           "kernels": {}}
+    if kernels:
+        with torch.inference_mode():
+            for (name, B, S, T) in (("2048", 16, 2048, 8192), ("4096", 16, 4096, 8192)):
+                rows, info = kernel_table(SIZES[name], B, S, T)
+                res["kernels"][f"width {name}, batch {B}, {S} positions, {T} prompt tokens"] = dict(info, table=table_with_fractions(rows))
+                torch.cuda.empty_cache()
+    if generation:
+        for name, B, S, new in RUNS:
+            z = SIZES[name]
+            line = {"size": name, "batch": B, "prompt": S, "new_tokens": new}
+            for what, make in (("tulezen", lambda: make_tulezen(z)), ("opt", lambda: make_opt(z, S + new))):
+                model = make()
+                line[what] = timed_generation(model, z["vocab"], B, S, new)
+                model._decode_state = None
+                del model
+                torch.cuda.empty_cache()
+            res["generation"].append(line)
+    status = device_status()
+    res["device_status"] = list(status)
+    return res

@@ -379,7 +379,7 @@ EB_API int eb_moe_route(const float *logits, long long ld, int tokens, int exper
 EB_API int eb_moe_plan(int32_t *counts, int experts, int32_t *offsets, int32_t *tile_group, int max_tiles, int32_t *live_tiles,
                 void *stream);
 
-/* rows[t][k] = offsets[idx] + rank (or -1) and out[rows[t][k]] = x[t]; top <= 32. */
+/* rows[t][k] = offsets[idx] + rank (or -1) and out[rows[t][k]] = x[t]. */
 EB_API int eb_moe_permute(const void *x, long long ldx, int n2, int dtype, int tokens, int top, const int32_t *idx,
                    const int32_t *ranks, const int32_t *offsets, int32_t *rows, void *out, long long ldo, int max_rows,
                    void *stream);
