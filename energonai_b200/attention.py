@@ -139,10 +139,14 @@ LATENT_WIDTHS = (64, 128, 256, 384, 512)      # latent widths of the tensor-core
 
 
 def pick_latent_nsplit(batch, heads, keys, sm_count=148):
-    """Key splits per (sequence, head tile): what fills the SMs, at least two 64-key tiles each."""
+    """Key splits per (sequence, head tile): what fills the SMs, at least two 64-key tiles each.  2
+    and 4 are clusters that merge in shared memory.  (A cluster of 8 CTAs with a whole SM each finds
+    room in a GPC so rarely that it ran in two waves: 8 splits took 50 us where 9, merged in a
+    second launch, took 33.)"""
     ctas = batch * -(-heads // (32 if heads > 16 else 16))
     tiles = max(1, -(-keys // 64))
-    return max(1, min(sm_count // max(1, ctas), tiles // 2, 64))
+    want = max(1, min(sm_count // max(1, ctas), tiles // 2, 64))
+    return 4 if 4 <= want < 8 else (2 if 2 <= want < 4 else (9 if want == 8 else want))
 
 
 def latent_decode(q, cache, rank, heads, window, pos_device, scale, first=None, nsplit=None):
@@ -158,5 +162,5 @@ def latent_decode(q, cache, rank, heads, window, pos_device, scale, first=None, 
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
     check(lib().eb_latent_decode(ptr(q), q.stride(0), ptr(cache), cache.stride(0), cache.stride(1), rows, ptr(out), out.stride(0), B,
                                  heads, rank, int(window), ptr(pos_device), ptr(first), float(scale), dtype_code(q.dtype), nsplit,
-                                 ptr(scratch), nbytes, stream_ptr()), "latent_decode", launches=2 if nsplit > 1 else 1)
+                                 ptr(scratch), nbytes, stream_ptr()), "latent_decode", launches=2 if nbytes else 1)
     return out

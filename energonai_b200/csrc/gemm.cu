@@ -1318,6 +1318,7 @@ extern "C" size_t eb_gemm_workspace_bytes(int M, int N, int K) {
 
 namespace eb {
 int attention_tc_status(int *out4, bool clear);   // attention_tc.cu
+int latent_status(int *out4, bool clear);         // latent_attention.cu
 }
 
 extern "C" int eb_device_status(int *out4, int clear) {
@@ -1336,6 +1337,12 @@ extern "C" int eb_device_status(int *out4, int clear) {
   if (host[0] == 0 && attn[0] != 0) {
     for (int i = 0; i < 4; ++i) host[i] = attn[i];
     host[1] += 100;
+  }
+  int lat[4] = {0, 0, 0, 0};                       // latent attention: 200+
+  if (eb::latent_status(lat, clear != 0) != EB_OK) return fail(EB_ECUDA, "device_status: cannot read the status word");
+  if (host[0] == 0 && lat[0] != 0) {
+    for (int i = 0; i < 4; ++i) host[i] = lat[i];
+    host[1] += 200;
   }
   if (out4)
     for (int i = 0; i < 4; ++i) out4[i] = host[i];

@@ -46,7 +46,7 @@ moe_route_kernel(const float *logits, long long ld, int tokens, int experts, int
 
 constexpr int kPlanThreads = 1024;
 
-// counts[experts] -> offsets[experts] (first row of the expert, a multiple of 128), tile_group[],
+// counts[experts * kCountStride] -> offsets[experts] (first row of the expert, a multiple of 128), tile_group[],
 // live_tiles; the counts are zeroed for the next batch.
 __global__ void __launch_bounds__(kPlanThreads)
 moe_plan_kernel(int *counts, int experts, int *offsets, int *tile_group, int max_tiles, int *live_tiles) {
@@ -57,7 +57,7 @@ moe_plan_kernel(int *counts, int experts, int *offsets, int *tile_group, int max
   const int per = (experts + kPlanThreads - 1) / kPlanThreads;
   const int e0 = tid * per, e1 = min(experts, e0 + per);
   int mine = 0;
-  for (int e = e0; e < e1; ++e) mine += (counts[e] + 127) / 128;
+  for (int e = e0; e < e1; ++e) mine += (counts[e * kCountStride] + 127) / 128;
   int incl = mine;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) {
@@ -73,12 +73,12 @@ moe_plan_kernel(int *counts, int experts, int *offsets, int *tile_group, int max
   }
   int tile = before + incl - mine;
   for (int e = e0; e < e1; ++e) {
-    const int n = (counts[e] + 127) / 128;
+    const int n = (counts[e * kCountStride] + 127) / 128;
     offsets[e] = tile * 128;
     for (int i = 0; i < n; ++i)
       if (tile + i < max_tiles) tile_group[tile + i] = e;
     tile += n;
-    counts[e] = 0;
+    counts[e * kCountStride] = 0;
   }
   if (tid == 0) *live_tiles = min(total, max_tiles);
 }
@@ -142,6 +142,7 @@ struct SkinnyParams {
   int N, K;
   int gated;
   float limit, alpha;
+  int ksplit;                  // the warps of a CTA share 16 weight rows and take this many columns each (0: own rows, all columns)
 };
 
 template <typename T> __device__ __forceinline__ void mma_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1);
@@ -163,8 +164,10 @@ __device__ __forceinline__ uint4 ld_stream(const void *p) {
 // quartet: lane (g, t) loads 16 bytes of weight rows g and g + 8 and of activation row g at the
 // same 8 columns, and hands them to two MMAs.  Which columns an MMA calls k = 0..15 does not
 // matter as long as both operands agree, so nothing is rearranged.
-template <typename T, int NT, int U>
-__device__ __forceinline__ void skinny_tile(const SkinnyParams &p, int group, int row0, const int *list, int base, int n) {
+// With ksplit the warps of the CTA add their parts up in shared memory, always in the same order.
+template <typename T, int NT, int U, bool SPLIT>
+__device__ __forceinline__ void skinny_tile(const SkinnyParams &p, int group, int row0, const int *list, int base, int n, float *part) {
+  const int warp = threadIdx.x >> 5, k_begin = SPLIT ? warp * p.ksplit : 0, k_end = SPLIT ? min(p.K, k_begin + p.ksplit) : p.K;
   const int lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const T *W = reinterpret_cast<const T *>(p.W) + (long long)group * p.w_gs;
   const T *A = reinterpret_cast<const T *>(p.A) + (long long)group * p.a_gs;
@@ -183,12 +186,12 @@ __device__ __forceinline__ void skinny_tile(const SkinnyParams &p, int group, in
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
   const uint4 zero = make_uint4(0, 0, 0, 0);
-  for (int k0 = 0; k0 < p.K; k0 += 32 * U) {
+  for (int k0 = k_begin; k0 < k_end; k0 += 32 * U) {
     uint4 a[U], b[U], x[U][NT];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int k = k0 + u * 32;
-      const bool ok = k + t * 8 < p.K;
+      const bool ok = k + t * 8 < k_end;
       a[u] = ok ? ld_stream(wa + k) : zero;
       b[u] = ok ? ld_stream(wb + k) : zero;
 #pragma unroll
@@ -201,6 +204,23 @@ __device__ __forceinline__ void skinny_tile(const SkinnyParams &p, int group, in
         mma_16816<T>(acc[j], a[u].x, b[u].x, a[u].y, b[u].y, x[u][j].x, x[u][j].y);
         mma_16816<T>(acc[j], a[u].z, b[u].z, a[u].w, b[u].w, x[u][j].z, x[u][j].w);
       }
+  }
+  if (SPLIT) {
+    const int warps = blockDim.x >> 5;
+    __syncthreads();                               // the parts of an earlier round have been read
+    if (warp > 0) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) part[((warp - 1) * 16 + j * 4 + e) * 32 + lane] = acc[j][e];
+    }
+    __syncthreads();
+    if (warp > 0) return;
+    for (int w = 0; w < warps - 1; ++w)
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[j][e] += part[(w * 16 + j * 4 + e) * 32 + lane];
   }
   T *C = reinterpret_cast<T *>(p.C) + (long long)group * p.c_gs;
 #pragma unroll
@@ -220,10 +240,11 @@ __device__ __forceinline__ void skinny_tile(const SkinnyParams &p, int group, in
     }
 }
 
-template <typename T>
+template <typename T, bool SPLIT>
 __global__ void __launch_bounds__(128) grouped_skinny_kernel(const SkinnyParams p) {
   extern __shared__ int list[];
   __shared__ int s_n;
+  __shared__ float part[SPLIT ? 3 * 16 * 32 : 1];
   griddep_wait();
   griddep_launch();
   const int group = blockIdx.y;
@@ -236,14 +257,14 @@ __global__ void __launch_bounds__(128) grouped_skinny_kernel(const SkinnyParams 
     __syncthreads();
     n = s_n;
   }
-  const int row0 = (blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * 16;
+  const int row0 = (SPLIT ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * 16;
   if (n == 0 || row0 >= p.N) return;
   const int *l = p.idx ? list : nullptr;
   for (int base = 0; base < n; base += 32) {
     const int m = min(32, n - base);
-    if (m <= 8) skinny_tile<T, 1, 8>(p, group, row0, l, base, m);
-    else if (m <= 16) skinny_tile<T, 2, 4>(p, group, row0, l, base, m);
-    else skinny_tile<T, 4, 2>(p, group, row0, l, base, m);
+    if (m <= 8) skinny_tile<T, 1, 8, SPLIT>(p, group, row0, l, base, m, part);
+    else if (m <= 16) skinny_tile<T, 2, 4, SPLIT>(p, group, row0, l, base, m, part);
+    else skinny_tile<T, 4, 2, SPLIT>(p, group, row0, l, base, m, part);
   }
 }
 
@@ -324,14 +345,18 @@ extern "C" int eb_grouped_skinny(const void *A, long long lda, long long a_group
   p.A = A; p.lda = lda; p.a_gs = a_group_stride; p.a_div = a_div; p.W = W; p.w_gs = w_group_stride; p.ldw = ldw;
   p.C = C; p.ldc = ldc; p.c_gs = c_group_stride; p.idx = idx; p.rows = rows; p.N = N; p.K = K;
   p.gated = gated; p.limit = limit; p.alpha = alpha;
-  // warps per CTA: fewer when that is what it takes to give every SM work
+  // Too few strips to give every SM a CTA of four: with many columns the four warps share a strip
+  // and split its columns, with few the CTAs get fewer warps.  (The choice depends on the weights'
+  // shape alone, so a row's result does not change with the batch.)
   const int strips = (N + 15) / 16;
   int warps = 4;
-  while (warps > 1 && (long long)((strips + warps - 1) / warps) * groups < 2ll * sm_count()) warps >>= 1;
-  const dim3 g((strips + warps - 1) / warps, groups), b(warps * 32);
+  const bool few = (long long)((strips + warps - 1) / warps) * groups < 2ll * sm_count(), split = few && K >= 256;
+  if (split) p.ksplit = ((K + warps - 1) / warps + 31) / 32 * 32;
+  while (!split && warps > 1 && (long long)((strips + warps - 1) / warps) * groups < 2ll * sm_count()) warps >>= 1;
+  const dim3 g(split ? strips : (strips + warps - 1) / warps, groups), b(warps * 32);
   const size_t smem = idx ? (size_t)rows * sizeof(int) : 0;
   cudaStream_t st = as_stream(stream);
-  if (dtype == EB_F16) launch_pdl(grouped_skinny_kernel<__half>, g, b, smem, st, p);
-  else launch_pdl(grouped_skinny_kernel<__nv_bfloat16>, g, b, smem, st, p);
+  if (dtype == EB_F16) launch_pdl(split ? grouped_skinny_kernel<__half, true> : grouped_skinny_kernel<__half, false>, g, b, smem, st, p);
+  else launch_pdl(split ? grouped_skinny_kernel<__nv_bfloat16, true> : grouped_skinny_kernel<__nv_bfloat16, false>, g, b, smem, st, p);
   return check_launch("grouped_skinny");
 }

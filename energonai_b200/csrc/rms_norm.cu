@@ -57,7 +57,7 @@ struct RmsParams {
   float w_offset, eps, inv_count;
   void *y;                     // rows ldy apart, or null
   long long ldy;
-  int n2;
+  int n1, n2;
   // ring cache: row (b, s) of the n1 = batch * rows_per_batch rows holds position pos0 + s of
   // sequence b; the last `ring_rows` positions are kept at ring + b*ring_bs + (position mod ring_rows)*ring_ld
   void *ring;
@@ -66,12 +66,15 @@ struct RmsParams {
   const int *pos_dev;          // device scalar with pos0, or null (pos0 = 0)
 };
 
-template <typename TI, typename TO, int PACKS>
+// THREADS per row: the CTA, or (rows of at most 1024 elements) one of its warps.
+template <typename TI, typename TO, int PACKS, int THREADS>
 __global__ void __launch_bounds__(kNormThreads) rms_norm_kernel(const RmsParams p) {
   __shared__ float scratch[kNormThreads / 32];
   griddep_wait();
   griddep_launch();
-  const long long row = blockIdx.x;
+  const int tid = THREADS == 32 ? threadIdx.x & 31 : threadIdx.x;
+  const long long row = THREADS == 32 ? (long long)blockIdx.x * (kNormThreads / 32) + (threadIdx.x >> 5) : blockIdx.x;
+  if (row >= p.n1) return;                         // (a whole warp, and only where a warp is a row)
   const TI *x = reinterpret_cast<const TI *>(p.x) + row * p.ldx;
   const TO *w = reinterpret_cast<const TO *>(p.w);
   const int packs = p.n2 / 8;
@@ -79,13 +82,13 @@ __global__ void __launch_bounds__(kNormThreads) rms_norm_kernel(const RmsParams 
   float sq = 0.f;
 #pragma unroll
   for (int i = 0; i < PACKS; ++i) {
-    const int c = threadIdx.x + i * kNormThreads;
+    const int c = tid + i * THREADS;
     if (c >= packs) break;
     load8<TI>(x + c * 8, v[i]);
 #pragma unroll
     for (int e = 0; e < 8; ++e) sq = fmaf(v[i][e], v[i][e], sq);
   }
-  const float r = rsqrtf(block_sum<kNormThreads>(sq, scratch) * p.inv_count + p.eps);
+  const float r = rsqrtf(block_sum<THREADS>(sq, scratch) * p.inv_count + p.eps);
   TO *ring = nullptr;
   if (p.ring) {
     const long long b = row / p.rows_per_batch;
@@ -96,7 +99,7 @@ __global__ void __launch_bounds__(kNormThreads) rms_norm_kernel(const RmsParams 
   }
 #pragma unroll
   for (int i = 0; i < PACKS; ++i) {
-    const int c = threadIdx.x + i * kNormThreads;
+    const int c = tid + i * THREADS;
     if (c >= packs) break;
     float wv[8];
     load8<TO>(w + c * 8, wv);
@@ -129,9 +132,10 @@ struct ResidualParams {
   float *r_weights;
 };
 
-template <typename T, int PACKS, bool COMBINE>
-__global__ void __launch_bounds__(kNormThreads) rms_residual_kernel(const ResidualParams p) {
-  __shared__ float scratch[kNormThreads / 32];
+// THREADS: 256, or 1024 with a router (few rows then, and the router's weights to read per row)
+template <typename T, int PACKS, bool COMBINE, int THREADS>
+__global__ void __launch_bounds__(THREADS) rms_residual_kernel(const ResidualParams p) {
+  __shared__ float scratch[THREADS / 32];
   extern __shared__ float dyn[];                   // router: [n2] row, [experts] logits
   const long long row = blockIdx.x;
   const T *w = reinterpret_cast<const T *>(p.w);
@@ -142,7 +146,7 @@ __global__ void __launch_bounds__(kNormThreads) rms_residual_kernel(const Residu
   float sq = 0.f;
 #pragma unroll
   for (int i = 0; i < PACKS; ++i) {
-    const int c = threadIdx.x + i * kNormThreads;
+    const int c = threadIdx.x + i * THREADS;
     if (c >= packs) break;
     if (COMBINE) {
 #pragma unroll
@@ -163,10 +167,10 @@ __global__ void __launch_bounds__(kNormThreads) rms_residual_kernel(const Residu
 #pragma unroll
     for (int e = 0; e < 8; ++e) sq = fmaf(v[i][e], v[i][e], sq);
   }
-  const float r = rsqrtf(block_sum<kNormThreads>(sq, scratch) * p.inv_count + p.eps);
+  const float r = rsqrtf(block_sum<THREADS>(sq, scratch) * p.inv_count + p.eps);
 #pragma unroll
   for (int i = 0; i < PACKS; ++i) {
-    const int c = threadIdx.x + i * kNormThreads;
+    const int c = threadIdx.x + i * THREADS;
     if (c >= packs) break;
     float wv[8], xv[8];
     load8<T>(w + c * 8, wv);
@@ -185,9 +189,10 @@ __global__ void __launch_bounds__(kNormThreads) rms_residual_kernel(const Residu
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float *z = dyn + p.n2;
-  for (int e = warp; e < p.experts; e += kNormThreads / 32) {
+  for (int e = warp; e < p.experts; e += THREADS / 32) {
     const T *wr = reinterpret_cast<const T *>(p.router) + (long long)e * p.n2;
     float acc = 0.f;
+#pragma unroll 4
     for (int c = lane; c < packs; c += 32) {
       float f[8];
       load8<T>(wr + c * 8, f);
@@ -205,18 +210,22 @@ template <typename TI, typename TO>
 int launch_rms(const RmsParams &p, int n1, cudaStream_t st) {
   const int packs = p.n2 / 8, per = (packs + kNormThreads - 1) / kNormThreads;
   const dim3 g(n1), b(kNormThreads);
-  if (per <= 1) launch_pdl(rms_norm_kernel<TI, TO, 1>, g, b, 0, st, p);
-  else if (per <= 2) launch_pdl(rms_norm_kernel<TI, TO, 2>, g, b, 0, st, p);
-  else if (per <= 4) launch_pdl(rms_norm_kernel<TI, TO, 4>, g, b, 0, st, p);
-  else launch_pdl(rms_norm_kernel<TI, TO, 8>, g, b, 0, st, p);
+  const dim3 gw((n1 + kNormThreads / 32 - 1) / (kNormThreads / 32));
+  if (packs <= 32) launch_pdl(rms_norm_kernel<TI, TO, 1, 32>, gw, b, 0, st, p);
+  else if (packs <= 64) launch_pdl(rms_norm_kernel<TI, TO, 2, 32>, gw, b, 0, st, p);
+  else if (packs <= 128) launch_pdl(rms_norm_kernel<TI, TO, 4, 32>, gw, b, 0, st, p);
+  else if (per <= 1) launch_pdl(rms_norm_kernel<TI, TO, 1, kNormThreads>, g, b, 0, st, p);
+  else if (per <= 2) launch_pdl(rms_norm_kernel<TI, TO, 2, kNormThreads>, g, b, 0, st, p);
+  else if (per <= 4) launch_pdl(rms_norm_kernel<TI, TO, 4, kNormThreads>, g, b, 0, st, p);
+  else launch_pdl(rms_norm_kernel<TI, TO, 8, kNormThreads>, g, b, 0, st, p);
   return check_launch("rms_norm");
 }
 
 template <typename T, bool COMBINE>
 int launch_residual(const ResidualParams &p, int n1, cudaStream_t st) {
-  const int packs = p.n2 / 8, per = (packs + kNormThreads - 1) / kNormThreads;
+  const int packs = p.n2 / 8, threads = p.router ? 1024 : kNormThreads, per = (packs + threads - 1) / threads;
   const size_t smem = p.router ? (size_t)(p.n2 + p.experts) * sizeof(float) : 0;
-  const dim3 g(n1), b(kNormThreads);
+  const dim3 g(n1), b(threads);
   auto go = [&](auto kern) -> int {
     if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       cudaGetLastError();
@@ -225,10 +234,11 @@ int launch_residual(const ResidualParams &p, int n1, cudaStream_t st) {
     launch_pdl(kern, g, b, smem, st, p);
     return check_launch("rms_residual");
   };
-  if (per <= 1) return go(rms_residual_kernel<T, 1, COMBINE>);
-  if (per <= 2) return go(rms_residual_kernel<T, 2, COMBINE>);
-  if (per <= 4) return go(rms_residual_kernel<T, 4, COMBINE>);
-  return go(rms_residual_kernel<T, 8, COMBINE>);
+  if (p.router) return per <= 1 ? go(rms_residual_kernel<T, 1, COMBINE, 1024>) : go(rms_residual_kernel<T, 2, COMBINE, 1024>);
+  if (per <= 1) return go(rms_residual_kernel<T, 1, COMBINE, kNormThreads>);
+  if (per <= 2) return go(rms_residual_kernel<T, 2, COMBINE, kNormThreads>);
+  if (per <= 4) return go(rms_residual_kernel<T, 4, COMBINE, kNormThreads>);
+  return go(rms_residual_kernel<T, 8, COMBINE, kNormThreads>);
 }
 
 constexpr int kMaxNormWidth = 8 * 8 * kNormThreads;
@@ -255,7 +265,7 @@ extern "C" int eb_rms_norm(const void *x, long long ldx, int in_dtype, const voi
   }
   RmsParams p{};
   p.x = x; p.ldx = ldx; p.w = w; p.w_offset = w_offset; p.eps = eps; p.inv_count = 1.f / (float)count;
-  p.y = y; p.ldy = ldy; p.n2 = n2;
+  p.y = y; p.ldy = ldy; p.n1 = n1; p.n2 = n2;
   p.ring = ring; p.ring_bs = ring_batch_stride; p.ring_ld = ring_ld; p.ring_rows = ring_rows; p.rows_per_batch = rows_per_batch;
   p.pos_dev = pos_device;
   cudaStream_t st = as_stream(stream);

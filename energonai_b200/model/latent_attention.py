@@ -46,12 +46,14 @@ class LatentCache(KVCache):
         self.reset()
         rows = self.rows_for(positions)
         if self.buf is None or self.buf.shape[:2] != (batch, rows) or self.buf.dtype != dtype or self.buf.device != device:
-            self.buf = torch.empty((batch, rows, self.width), dtype=dtype, device=device)
+            self.buf = torch.zeros((batch, rows, self.width), dtype=dtype, device=device)     # (unwritten rows must be finite)
 
     def grow(self, positions):
         rows = self.rows_for(positions)
-        if rows > self.buf.shape[1]:
+        have = self.buf.shape[1]
+        if rows > have:
             self.ensure(self.buf.shape[0], self.rows_for(positions + self.reserve), self.width, self.buf.dtype, self.buf.device, exact=True)
+            self.buf[:, have:].zero_()
 
     def keep(self, rows):
         self.buf = self.buf.index_select(0, rows)

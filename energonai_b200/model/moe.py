@@ -8,7 +8,7 @@ import torch
 from torch import nn
 
 from ..gemm import gemm
-from ..moe import SKINNY_MAX_ENTRIES, SortedRows, grouped_gemm, route, skinny_experts
+from ..moe import SKINNY_MAX_ENTRIES, SortedRows, grouped_gemm, new_counts, route, skinny_experts
 from ..nn import init_weight
 from .latent_attention import round_up
 
@@ -44,7 +44,7 @@ class MixtureOfExperts(nn.Module):
             act = skinny_experts(h, self.gate_up, idx, self.top, gate=self.gate)
             return skinny_experts(act, self.down, idx, 1), (idx, None, w)
         if self._counts is None or self._counts.device != h.device:
-            self._counts = torch.zeros(self.experts, dtype=torch.int32, device=h.device)
+            self._counts = new_counts(self.experts, h.device)
         logits = gemm(h, self.router, out_dtype=torch.float32, static_weight=True)
         idx, w, ranks = route(logits, self.experts, self.top, first, rows_per_batch, counts=self._counts)
         plan = SortedRows(h, idx, ranks, self._counts)

@@ -4,15 +4,21 @@ import torch
 
 from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
 
+COUNT_STRIDE = 32        # EB_MOE_COUNT_STRIDE
 ROW_TILE = 128           # rows of one expert come in tiles of this many in the sorted layout
 
 SKINNY_MAX_ENTRIES = 10240   # (token, choice) pairs the weight-streaming product sorts in shared memory
 
 
+def new_counts(experts, device):
+    """Zeroed row counters of the experts; route() fills them, SortedRows zeroes them again."""
+    return torch.zeros(experts * COUNT_STRIDE, dtype=torch.int32, device=device)
+
+
 def route(logits, experts, top, first=None, rows_per_batch=0, counts=None):
     """logits [T, >= experts] fp32 -> idx [T, top] int32, weights [T, top] fp32 (softmax scores over
     all experts, not renormalised).  first [batch] int32: rows before it in their sequence are
-    padding (idx -1).  With counts [experts] int32 (zero) also ranks [T, top]."""
+    padding (idx -1).  With counts (new_counts) also ranks [T, top]."""
     require_cuda(logits, first, counts)
     if logits.dim() != 2 or logits.dtype != torch.float32 or logits.stride(1) != 1:
         raise RuntimeError("moe route: logits must be fp32 [tokens, experts]")
@@ -30,7 +36,7 @@ class SortedRows:
 
     def __init__(self, x, idx, ranks, counts):
         T, top = idx.shape
-        experts = counts.numel()
+        experts = counts.numel() // COUNT_STRIDE
         self.max_tiles = (T * top) // ROW_TILE + min(experts, T * top)
         dev = x.device
         i32 = lambda n: torch.empty(n, dtype=torch.int32, device=dev)

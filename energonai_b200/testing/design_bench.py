@@ -98,7 +98,7 @@ def kernel_table(z, B, S, T):
     from ..attention import (attention_decode, attention_prefill, attention_prefill_window, latent_decode)
     from ..gemm import gemm
     from ..kernel.cuda_native.layer_norm import layer_norm_forward
-    from ..moe import SortedRows, grouped_gemm, per_head, route, skinny_experts
+    from ..moe import SortedRows, grouped_gemm, new_counts, per_head, route, skinny_experts
     from ..norm import rms_norm, rms_residual
     bf, dev = torch.bfloat16, "cuda"
     W, H, d, R, E, K, ff = z["width"], z["heads"], z["dim"], z["kv_rank"], z["experts"], z["top"], z["ff"]
@@ -186,8 +186,7 @@ def kernel_table(z, B, S, T):
                                                                   for x, t, y in zip(xs, xts, ys)]), 12 * T * W)
     add("prompt", "layer_norm (OPT)", None, time_calls([lambda t=t: layer_norm_forward(t, lw, lb, 1e-5) for t in xts + ys]), 4 * T * W)
     logits = torch.randn(T, E, device=dev)
-    counts = torch.zeros(E, dtype=torch.int32, device=dev)
-    n0, n1 = [torch.zeros(E, dtype=torch.int32, device=dev) for _ in range(2)]
+    counts, n0, n1 = [new_counts(E, dev) for _ in range(3)]
     add("prompt", "moe route", None, time_calls([lambda: route(logits, E, K, counts=n0)] * 4), 4 * T * E + 12 * T * K)
     idx, wts, ranks = route(logits, E, K, counts=counts)
     keep = counts.clone()
@@ -230,7 +229,7 @@ def run(kernels=True, generation=True):
            "kernels": {}}
     if kernels:
         with torch.inference_mode():
-            for (name, B, S, T) in (("2048", 16, 2048, 8192), ("4096", 16, 4096, 8192)):
+            for (name, B, S, T) in (("2048", 64, 2048, 8192), ("4096", 16, 4096, 8192)):
                 rows, info = kernel_table(SIZES[name], B, S, T)
                 res["kernels"][f"width {name}, batch {B}, {S} positions, {T} prompt tokens"] = dict(info, table=table_with_fractions(rows))
                 torch.cuda.empty_cache()

@@ -370,7 +370,9 @@ EB_API int eb_gated_act(const void *x, long long ldx, void *y, long long ldy, in
 /* Router of a mixture: idx[t][k], weights[t][k] = the `top` largest softmax scores over all experts
  * of logits[t] (fp32, not renormalised; the lowest index among equals).  first (or NULL): rows
  * t with t mod rows_per_batch < first[t / rows_per_batch] are padding and get idx -1.  With counts
- * (zero on entry), ranks[t][k] = the choice's place among its expert's rows. */
+ * (one int every 32, EB_MOE_COUNT_STRIDE; zero on entry), ranks[t][k] = the choice's place among its
+ * expert's rows. */
+#define EB_MOE_COUNT_STRIDE 32
 EB_API int eb_moe_route(const float *logits, long long ld, int tokens, int experts, int top, const int32_t *first,
                  int rows_per_batch, int32_t *idx, float *weights, int32_t *counts, int32_t *ranks, void *stream);
 
@@ -479,8 +481,11 @@ EB_API int eb_attention_plain(const void *q, const void *k, const void *v, void 
  * queries in latent space, the cached latent row of a position is key and value of every head,
  *   out[b][h] = sum_j softmax_j(scale * q[b][h] . c[b][j]) c[b][j]
  * over the positions max(first[b], pos - window + 1) .. pos (window 0: all), position j in cache row
- * j mod ring_rows.  rank 64, 128, 256, 384 or 512.  nsplit > 1 splits the positions over that many
- * CTAs per (sequence, head tile) and merges them in a second launch through `scratch`. */
+ * j mod ring_rows.  rank 64, 128, 256, 384 or 512.  Every cache row must hold finite numbers, also
+ * those no position has been written to yet (they are multiplied by a weight of exactly 0).
+ * nsplit > 1 splits the positions over that many CTAs per (sequence, head tile): 2, 4 or 8 are
+ * clusters that merge their parts on chip, any other number merges in a second launch through
+ * `scratch` (eb_latent_decode_scratch_bytes).  Waits are bounded ("where" codes 200 and up). */
 EB_API int eb_latent_decode(const void *q, long long q_batch_stride, const void *cache, long long cache_batch_stride,
                      long long cache_row_stride, int ring_rows, void *out, long long out_batch_stride, int batch, int heads,
                      int rank, int window, const int32_t *pos_device, const int32_t *first, float scale, int dtype,
