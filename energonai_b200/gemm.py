@@ -39,11 +39,8 @@ def gemm(a, w, bias=None, act=None, residual=None, out=None, out_dtype=None, out
     require_cuda(a, w, bias, residual, out)
     if a.dim() != 2 or w.dim() != 2 or a.shape[1] != w.shape[1]:
         raise RuntimeError(f"gemm: shapes {tuple(a.shape)} x {tuple(w.shape)}^T do not match")
-    if a.dtype == torch.float32 and w.dtype == torch.float32:
-        return _gemm_f32(a, w, out, bias is None and residual is None and peer is None and ln_fold is None
-                         and act in (None, "none", ACT_NONE) and out_rows_per_batch == 0 and out_row_offset_device is None)
     if a.dtype != w.dtype or a.dtype not in (torch.float16, torch.bfloat16):
-        raise RuntimeError("gemm: fp16, bf16 or fp32 operands of one dtype required")
+        raise RuntimeError("gemm: fp16 or bf16 operands of one dtype required")
     if a.stride(1) != 1:
         a = a.contiguous()
     if w.stride(1) != 1:
@@ -90,10 +87,11 @@ def gemm(a, w, bias=None, act=None, residual=None, out=None, out_dtype=None, out
     return out
 
 
-def _gemm_f32(a, w, out, plain):
-    """The true 32-bit product of models run in fp32 (CUDA cores, no reduced-precision mode)."""
-    if not plain:
-        raise RuntimeError("gemm: the fp32 product has no epilogue (bias, activation, residual, row mapping)")
+def gemm_f32(a, w, out=None):
+    """a [M,K] @ w [N,K].T in true 32-bit (CUDA cores, no reduced-precision mode)."""
+    require_cuda(a, w, out)
+    if a.dim() != 2 or w.dim() != 2 or a.shape[1] != w.shape[1] or a.dtype != torch.float32 or w.dtype != torch.float32:
+        raise RuntimeError("gemm_f32: fp32 a [M,K] and w [N,K] required")
     a, w = (t if t.stride(1) == 1 else t.contiguous() for t in (a, w))
     (M, K), N = a.shape, w.shape[0]
     if out is None:
@@ -101,6 +99,11 @@ def _gemm_f32(a, w, out, plain):
     check(lib().eb_gemm_f32(ptr(a), a.stride(0), 0, ptr(w), w.stride(0), 0, ptr(out), out.stride(0), 0, M, N, K, 1, None, None,
                             stream_ptr()), "gemm_f32")
     return out
+
+
+def project(x, w, out_dtype=None):
+    """x @ w.T with a model's weight: the tensor-core GEMM, or the 32-bit one for models run in fp32."""
+    return gemm_f32(x, w) if w.dtype == torch.float32 else gemm(x, w, out_dtype=out_dtype, static_weight=True)
 
 
 LN_FOLD_MAX_ROWS = 32

@@ -17,7 +17,7 @@ import torch
 from torch import nn
 
 from ..attention import (LATENT_WIDTHS, attention_plain, attention_prefill_window, latent_decode)
-from ..gemm import gemm
+from ..gemm import project
 from ..moe import per_head
 from ..nn import RMSNorm1D, init_weight
 from ..norm import rms_norm
@@ -169,25 +169,25 @@ class LatentAttention(nn.Module):
     def prompt(self, h, ctx):
         """h [batch*seq, width] -> [batch*seq, width]; fills this layer's cache."""
         B, S = ctx.batch, ctx.seq
-        q = gemm(h, self.in_proj, static_weight=True)
+        q = project(h, self.in_proj)
         if self.kv_from is None:
             n = self.latent_norm
             ctx.latents[self.layer] = rms_norm(q[:, self.q_rows:], n.weight, n.eps, offset=n.offset, count=n.count,
                                                ring=ctx.state.caches[self.layer].buf, rows_per_batch=S)
         c = ctx.latents[self.source]
-        kv = gemm(c, self.kv_up, static_weight=True).view(B, S, -1)
+        kv = project(c, self.kv_up).view(B, S, -1)
         q3 = q.view(B, S, -1)[:, :, :self.q_rows]
         k, v = kv[:, :, :self.q_rows], kv[:, :, self.q_rows:]        # (keys have as many rows as queries)
         if self.tensor_core_prompt:
             o = attention_prefill_window(q3, k, v, self.dk, self.window, mask=ctx.mask, scale=self.scale)
         else:
             o = attention_plain(q3, k, v, self.heads, self.dk, self.dv, window=self.window, scale=self.scale, first=ctx.first)
-        return gemm(o.view(B * S, -1), self.out_proj, static_weight=True)
+        return project(o.view(B * S, -1), self.out_proj)
 
     def step(self, h, ctx):
         """h [batch, width], one new position per sequence -> [batch, width]."""
         B = ctx.batch
-        q = gemm(h, self.in_proj, static_weight=True)
+        q = project(h, self.in_proj)
         cache = ctx.state.caches[self.source].buf
         if self.kv_from is None:
             n = self.latent_norm
@@ -200,4 +200,4 @@ class LatentAttention(nn.Module):
             o = attention_plain(qa.view(B, 1, -1), cache, cache, self.heads, self.rank, self.rank, window=self.window, scale=self.scale,
                                 first=ctx.first, pos_device=ctx.pos, shared_kv=True).view(B, -1)
         v = per_head(o, self.kv_up[self.q_rows:].view(self.heads, self.dv, self.rank))
-        return gemm(v, self.out_proj, static_weight=True)
+        return project(v, self.out_proj)

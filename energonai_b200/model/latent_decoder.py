@@ -9,7 +9,7 @@ import os
 import torch
 from torch import nn
 
-from ..gemm import gemm
+from ..gemm import project
 from ..nn import RMSNorm1D, init_weight
 from ..norm import rms_norm, rms_residual
 from ..step import greedy_step
@@ -142,7 +142,7 @@ class LatentDecoder(GenerationModel):
         """Final norm and head of rows of the residual stream -> fp32 [rows, vocab]."""
         n = self.norm
         h = rms_norm(x, n.weight, n.eps, offset=n.offset, count=n.count)
-        return gemm(h, self.head, out_dtype=torch.float32, static_weight=True)[:, :self.vocab]
+        return project(h, self.head, out_dtype=torch.float32)[:, :self.vocab]
 
     # ---- what the generation loop asks for ----
     @property

@@ -7,7 +7,7 @@ kernel needs to form the weighted sum of a token's expert rows itself."""
 import torch
 from torch import nn
 
-from ..gemm import gemm
+from ..gemm import project
 from ..moe import SKINNY_MAX_ENTRIES, SortedRows, grouped_gemm, new_counts, route, skinny_experts
 from ..nn import init_weight
 from .latent_attention import round_up
@@ -39,13 +39,13 @@ class MixtureOfExperts(nn.Module):
         evaluated already.  first: padding positions per sequence, which get no expert."""
         T = h.shape[0]
         if self.skinny(T):
-            idx, w = routed if routed is not None else route(gemm(h, self.router, out_dtype=torch.float32, static_weight=True),
+            idx, w = routed if routed is not None else route(project(h, self.router, out_dtype=torch.float32),
                                                              self.experts, self.top, first, rows_per_batch)
             act = skinny_experts(h, self.gate_up, idx, self.top, gate=self.gate)
             return skinny_experts(act, self.down, idx, 1), (idx, None, w)
         if self._counts is None or self._counts.device != h.device:
             self._counts = new_counts(self.experts, h.device)
-        logits = gemm(h, self.router, out_dtype=torch.float32, static_weight=True)
+        logits = project(h, self.router, out_dtype=torch.float32)
         idx, w, ranks = route(logits, self.experts, self.top, first, rows_per_batch, counts=self._counts)
         plan = SortedRows(h, idx, ranks, self._counts)
         act = grouped_gemm(plan.x, self.gate_up, plan, gate=self.gate)

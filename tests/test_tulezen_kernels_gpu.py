@@ -172,10 +172,10 @@ def test_per_head_product(B, dtype):
 
 
 def test_gemm_f32_is_true_32_bit():
-    from energonai_b200.gemm import gemm
+    from energonai_b200.gemm import gemm_f32
     for M, N, K in ((1, 5, 7), (70, 65, 130), (300, 448, 256)):
         a, w = rnd(M, K, dtype=F32), rnd(N, K, seed=1, dtype=F32)
-        close(gemm(a, w), a.double().cpu() @ w.double().cpu().T, 1e-6)
+        close(gemm_f32(a, w), a.double().cpu() @ w.double().cpu().T, 1e-6)
 
 
 # ---- windowed prompt attention ---------------------------------------------------------------------------
