@@ -3,10 +3,10 @@
 // Both operands are K-major 16-bit matrices (A [M,K], W [N,K]); accumulation is fp32 in
 // tensor memory.  One kernel template serves two orientations:
 //
-//   normal (M > 128): TMEM lanes = 128 rows of A, TMEM columns = BN rows of W.  Persistent
+//   normal (M > 32): TMEM lanes = 128 rows of A, TMEM columns = BN rows of W.  Persistent
 //       CTAs walk 128 x BN output tiles in a grouped raster so that concurrently running CTAs
 //       share A and W panels in L2.
-//   swapped (M <= 128, generation steps): TMEM lanes = 128 rows of W, TMEM columns = the (padded)
+//   swapped (M <= 32, generation steps; up to 128 with the exchange): TMEM lanes = 128 rows of W, TMEM columns = the (padded)
 //       M rows of A.  The work is one pass over W (HBM-bound).  An MMA over 128 lanes costs the
 //       same however many lanes carry useful rows, so W is always taken in full 128-row tiles,
 //       and the (tile, k) space is cut stream-K style into equal contiguous ranges, one per CTA:
@@ -1419,7 +1419,12 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
 
   CUtensorMap tl, tc;
   int rc;
-  if (M <= kLanes) {
+  // Between 33 and 128 rows the swapped orientation holds 64 or 128 batch values per thread in its
+  // epilogue and sums as many partials per shared tile: 49 us (64 rows) and 240 us (128 rows) for
+  // a 2560 x 2048 weight that the normal orientation multiplies in 16 us, its row tile mostly
+  // padding.  The swapped one stays for shapes the other cannot store and for the fused exchange.
+  const bool normal_ok = !comm && N % 8 == 0 && ldc % 8 == 0 && (!residual || ldr % 8 == 0) && (c_rows_per_batch == 0 || c_batch_stride % 8 == 0);
+  if (M <= 32 || (M <= kLanes && !normal_ok)) {
     // swapped orientation: lanes = rows of W, columns = rows of A
     const int bn = swap_bn(M);
     int grid;

@@ -236,7 +236,8 @@ EB_API int eb_allreduce(eb_comm *comm, void *buf, size_t count, int dtype, void 
  * The kernel is launched so that it may begin before the preceding kernel of the stream has
  * finished; it reads A, bias and residual only after that kernel completed, and W too unless
  * flags has EB_GEMM_STATIC_W.
- * For M <= 128 (generation steps) the kernel streams W exactly once, split evenly over all SMs
+ * For M <= 32 (generation steps; up to 128 where the output's strides are not multiples of 8) the
+ * kernel streams W exactly once, split evenly over all SMs
  * (stream-K over 128-row tiles; a K of at most 1280 is not cut, one CTA per tile), and combines
  * the partial sums of tiles shared by several CTAs
  * through `workspace`: at least eb_gemm_workspace_bytes(M,N,K) bytes, 16-byte aligned,
