@@ -117,20 +117,27 @@ def attention_prefill_window(q, k, v, head_dim, window, mask=None, scale=None, o
     return out
 
 
-def attention_plain(q, k, v, heads, k_dim, v_dim, window=0, scale=1.0, first=None, pos_device=None, shared_kv=False):
+def attention_plain(q, k, v, heads, k_dim, v_dim, window=0, scale=1.0, first=None, pos_device=None, shared_kv=False,
+                    kv_heads=None, bias=None, sink=False):
     """Windowed causal attention on the CUDA cores, any head sizes, fp32 / fp16 / bf16.  q [B, Sq,
     heads*k_dim]; k / v [B, rows, heads*dim] or, with shared_kv, [B, rows, dim] shared by the heads.
     Query row i holds position pos_device + i (None: i), the key of position j is row j mod rows;
-    first [B] int32 is each sequence's first position.  Returns [B, Sq, heads*v_dim]."""
-    require_cuda(q, k, v, first, pos_device)
+    first [B] int32 is each sequence's first position.  kv_heads: heads of k / v, each shared by
+    heads / kv_heads query heads.  bias = (r1, r2), fp32 per query head: r1 * ln(1 + r2 * distance) is
+    taken off the scaled score.  sink: one is added to the softmax denominator.  Returns [B, Sq, heads*v_dim]."""
+    r1, r2 = bias if bias is not None else (None, None)
+    require_cuda(q, k, v, first, pos_device, r1, r2)
+    if bias is not None and any(r.dtype != torch.float32 or r.numel() != heads or not r.is_contiguous() for r in bias):
+        raise RuntimeError("attention: the distance bias has two fp32 numbers per query head")
     B, Sq, _ = q.shape
     out = torch.empty((B, Sq, heads * v_dim), dtype=q.dtype, device=q.device)
     if any(t.stride(2) != 1 for t in (q, k, v)) or k.shape[1] != v.shape[1]:
         raise RuntimeError("attention: contiguous last dims and one number of key / value rows required")
     hk, hv = (0, 0) if shared_kv else (k_dim, v_dim)
     check(lib().eb_attention_plain(ptr(q), ptr(k), ptr(v), ptr(out), q.stride(0), q.stride(1), k_dim, k.stride(0), k.stride(1), hk,
-                                   v.stride(0), v.stride(1), hv, out.stride(0), out.stride(1), v_dim, B, heads, Sq, k_dim, v_dim,
-                                   int(window), k.shape[1], ptr(pos_device), ptr(first), float(scale), dtype_code(q.dtype), stream_ptr()),
+                                   v.stride(0), v.stride(1), hv, out.stride(0), out.stride(1), v_dim, B, heads,
+                                   heads // (kv_heads or heads), Sq, k_dim, v_dim, int(window), k.shape[1], ptr(pos_device), ptr(first),
+                                   ptr(r1), ptr(r2), 1 if sink else 0, float(scale), dtype_code(q.dtype), stream_ptr()),
           "attention_plain")
     return out
 
@@ -164,3 +171,31 @@ def latent_decode(q, cache, rank, heads, window, pos_device, scale, first=None, 
                                  heads, rank, int(window), ptr(pos_device), ptr(first), float(scale), dtype_code(q.dtype), nsplit,
                                  ptr(scratch), nbytes, stream_ptr()), "latent_decode", launches=2 if nbytes else 1)
     return out
+
+
+def attention_inputs(proj, heads, kv_heads, dk, dv, q_norm, q_count, k_norm, k_count, eps, k_cache, v_cache, rows_per_batch, temp=None,
+                     vmix=None, v_first=None, pos_device=None, first=None):
+    """Rows [q | k | v | ...] of a projection -> normalised queries [rows, heads*dk]; keys and values go
+    to their cache rows.  q and k are normalised over all heads at once (q_count / k_count columns are
+    real); temp = (coef, every): q times 1 + coef * ln(floor((p + 1) / every) + 1); vmix (fp32 scalar) and
+    v_first (another layer's v_cache): v = (1 - vmix) v + vmix v_first of the same token."""
+    require_cuda(proj, q_norm, k_norm, k_cache, v_cache, vmix, v_first, pos_device, first)
+    n1 = proj.shape[0]
+    if any(t.dtype != proj.dtype for t in (q_norm, k_norm, k_cache, v_cache)) or (v_first is not None and v_first.dtype != proj.dtype):
+        raise RuntimeError("attention_inputs: one dtype required")
+    if proj.dim() != 2 or proj.stride(1) != 1 or q_norm.numel() != heads * dk or k_norm.numel() != kv_heads * dk:
+        raise RuntimeError("attention_inputs: rows [q | k | v], one norm entry per column of q and of k")
+    B = n1 // rows_per_batch
+    for t, w in ((k_cache, kv_heads * dk), (v_cache, kv_heads * dv), (v_first, kv_heads * dv)):
+        if t is not None and (t.dim() != 3 or t.stride(2) != 1 or t.shape[0] != B or t.shape[2] != w or t.shape[1] != k_cache.shape[1]):
+            raise RuntimeError("attention_inputs: caches are [batch, rows, kv_heads*dim]")
+    if vmix is not None and (vmix.dtype != torch.float32 or v_first is None):
+        raise RuntimeError("attention_inputs: vmix is an fp32 scalar and goes with v_first")
+    q = torch.empty((n1, heads * dk), dtype=proj.dtype, device=proj.device)
+    coef, every = temp if temp is not None else (0.0, 0)
+    check(lib().eb_attention_inputs(ptr(proj), proj.stride(0), heads, kv_heads, dk, dv, ptr(q_norm), int(q_count), ptr(k_norm), int(k_count),
+                                    float(eps), float(coef), int(every), ptr(vmix), ptr(v_first), v_first.stride(0) if vmix is not None else 0,
+                                    v_first.stride(1) if vmix is not None else 0, ptr(q), q.stride(0), ptr(k_cache), k_cache.stride(0),
+                                    k_cache.stride(1), ptr(v_cache), v_cache.stride(0), v_cache.stride(1), k_cache.shape[1], n1, rows_per_batch,
+                                    ptr(pos_device), ptr(first), dtype_code(proj.dtype), stream_ptr()), "attention_inputs")
+    return q

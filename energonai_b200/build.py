@@ -19,6 +19,13 @@ LIB_PATH = os.path.join(HERE, "libenergon_b200.so")
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
               "-diag-suppress", "177,550"]
+# Recurrences add up the logarithms of their gates over a whole sequence: an approximation's bias would
+# add up with them, so these files get the accurate functions.
+ACCURATE = {"matrix_memory.cu"}
+
+
+def nvcc_flags(source):
+    return [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and source in ACCURATE)]
 
 
 def _nvcc():
@@ -48,7 +55,7 @@ def _build(force, verbose):
     for s in sources:
         src, obj = os.path.join(CSRC, s), os.path.join(OBJ_DIR, s[:-3] + ".o")
         if force or _newer([src] + headers, obj):
-            jobs.append([_nvcc()] + NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else []) + ["-c", src, "-o", obj])
+            jobs.append([_nvcc()] + nvcc_flags(s) + (["-Xptxas", "-v"] if verbose else []) + ["-c", src, "-o", obj])
 
     def run(cmd):
         r = subprocess.run(cmd, capture_output=True, text=True)

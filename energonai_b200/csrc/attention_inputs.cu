@@ -1,0 +1,156 @@
+// What lies between the projection of an attention layer and the attention itself, one row per CTA:
+// RMS norm of the whole query and of the whole key (before they are heads), a query temperature that
+// grows with the position, values mixed with those an earlier layer cached for the same token, and the
+// stores into the key / value cache.  Statistics and factors are fp32.
+#include "common.cuh"
+
+namespace eb {
+namespace {
+
+struct InputParams {
+  const void *proj;
+  long long ldp;
+  int nq, nk, nv;              // columns of q, k, v
+  const void *wq, *wk;
+  float inv_q, inv_k, eps, coef;
+  int every;
+  const float *vmix;
+  const void *vf;
+  long long vf_bs, vf_rs;
+  void *q;
+  long long ldq;
+  void *k, *v;
+  long long k_bs, k_rs, v_bs, v_rs;
+  int cache_rows, rows_per_batch;
+  const int *pos_dev, *first;
+};
+
+template <typename T> struct Pack8 {               // 8 elements of T
+  static __device__ __forceinline__ void load(const T *p, float (&f)[8]) {
+    constexpr int N = Vec16<T>::N;
+#pragma unroll
+    for (int i = 0; i < 8 / N; ++i) {
+      Vec16<T> a;
+      float t[N];
+      a.load(p + i * N);
+      a.unpack(t);
+#pragma unroll
+      for (int e = 0; e < N; ++e) f[i * N + e] = t[e];
+    }
+  }
+  static __device__ __forceinline__ void store(T *p, const float (&f)[8]) {
+    constexpr int N = Vec16<T>::N;
+#pragma unroll
+    for (int i = 0; i < 8 / N; ++i) {
+      Vec16<T> a;
+      float t[N];
+#pragma unroll
+      for (int e = 0; e < N; ++e) t[e] = f[i * N + e];
+      a.pack(t);
+      a.store(p + i * N);
+    }
+  }
+};
+
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS) attention_inputs_kernel(const InputParams p) {
+  __shared__ float scratch[2][THREADS / 32];
+  griddep_wait();
+  griddep_launch();
+  const long long row = blockIdx.x;
+  const long long b = row / p.rows_per_batch;
+  const int col = (p.pos_dev ? *p.pos_dev : 0) + (int)(row - b * p.rows_per_batch);
+  const T *x = reinterpret_cast<const T *>(p.proj) + row * p.ldp;
+  const int nq = p.nq / 8, nk = p.nk / 8, nv = p.nv / 8;
+  float sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x; c < nq + nk; c += THREADS) {
+    float f[8];
+    Pack8<T>::load(x + c * 8, f);
+    float s = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s = fmaf(f[e], f[e], s);
+    if (c < nq) sq += s; else sk += s;
+  }
+  sq = block_sum<THREADS>(sq, scratch[0]);
+  sk = block_sum<THREADS>(sk, scratch[1]);
+  float rq = rsqrtf(sq * p.inv_q + p.eps);
+  const float rk = rsqrtf(sk * p.inv_k + p.eps);
+  if (p.every > 0) {
+    const int pos = max(0, col - (p.first ? p.first[b] : 0));
+    rq *= 1.f + p.coef * logf((float)((pos + 1) / p.every + 1));
+  }
+  const bool keep = col >= 0 && col < p.cache_rows;
+  T *q = reinterpret_cast<T *>(p.q) + row * p.ldq;
+  T *k = reinterpret_cast<T *>(p.k) + b * p.k_bs + (long long)col * p.k_rs;
+  T *v = reinterpret_cast<T *>(p.v) + b * p.v_bs + (long long)col * p.v_rs;
+  const T *vf = p.vmix ? reinterpret_cast<const T *>(p.vf) + b * p.vf_bs + (long long)col * p.vf_rs : nullptr;
+  const float lambda = p.vmix ? *p.vmix : 0.f;
+  for (int c = threadIdx.x; c < nq + nk + nv; c += THREADS) {
+    float f[8], w[8];
+    Pack8<T>::load(x + c * 8, f);
+    if (c < nq) {
+      Pack8<T>::load(reinterpret_cast<const T *>(p.wq) + c * 8, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] *= rq * w[e];
+      Pack8<T>::store(q + c * 8, f);
+    } else if (c < nq + nk) {
+      if (!keep) continue;
+      Pack8<T>::load(reinterpret_cast<const T *>(p.wk) + (c - nq) * 8, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] *= rk * w[e];
+      Pack8<T>::store(k + (c - nq) * 8, f);
+    } else {
+      if (!keep) continue;
+      const int o = (c - nq - nk) * 8;
+      if (vf) {
+        Pack8<T>::load(vf + o, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = fmaf(lambda, w[e], (1.f - lambda) * f[e]);
+      }
+      Pack8<T>::store(v + o, f);
+    }
+  }
+}
+
+template <typename T> int launch_inputs(const InputParams &p, int n1, cudaStream_t st) {
+  if (p.nq + p.nk + p.nv <= 2048) launch_pdl(attention_inputs_kernel<T, 128>, dim3(n1), dim3(128), 0, st, p);
+  else launch_pdl(attention_inputs_kernel<T, 256>, dim3(n1), dim3(256), 0, st, p);
+  return check_launch("attention_inputs");
+}
+
+}  // namespace
+}  // namespace eb
+
+using namespace eb;
+
+extern "C" int eb_attention_inputs(const void *proj, long long ldp, int heads, int kv_heads, int dk, int dv, const void *q_norm, int q_count,
+                                   const void *k_norm, int k_count, float eps, float temp_coef, int temp_every, const float *vmix,
+                                   const void *v_first, long long vf_batch_stride, long long vf_row_stride, void *q_out, long long ldq,
+                                   void *k_cache, long long k_batch_stride, long long k_row_stride, void *v_cache, long long v_batch_stride,
+                                   long long v_row_stride, int cache_rows, int n1, int rows_per_batch, const int32_t *pos_device,
+                                   const int32_t *first, int dtype, void *stream) {
+  if (n1 == 0) return EB_OK;
+  EB_REQUIRE(dtype_ok(dtype), "attention_inputs: bad dtype %d", dtype);
+  EB_REQUIRE(proj && q_norm && k_norm && q_out && k_cache && v_cache, "attention_inputs: null pointer");
+  EB_REQUIRE(heads > 0 && kv_heads > 0 && dk > 0 && dv > 0 && dk % 8 == 0 && dv % 8 == 0, "attention_inputs: head sizes must be multiples of 8 (%d, %d)", dk, dv);
+  EB_REQUIRE((long long)heads * dk < (1 << 24) && (long long)kv_heads * (dk > dv ? dk : dv) < (1 << 24), "attention_inputs: too many columns");
+  const int nq = heads * dk, nk = kv_heads * dk, nv = kv_heads * dv;
+  EB_REQUIRE(q_count > 0 && q_count <= nq && k_count > 0 && k_count <= nk, "attention_inputs: the means are over 1..all columns");
+  EB_REQUIRE(temp_every >= 0 && (!vmix || v_first), "attention_inputs: bad temperature step, or a mix without the other values");
+  EB_REQUIRE(n1 > 0 && rows_per_batch > 0 && n1 % rows_per_batch == 0 && cache_rows > 0, "attention_inputs: bad row counts");
+  const long long strides[] = {ldp, ldq, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride, vmix ? vf_batch_stride : 0, vmix ? vf_row_stride : 0};
+  for (long long s : strides) EB_REQUIRE(s % 8 == 0, "attention_inputs: strides must be multiples of 8 elements");
+  EB_REQUIRE(ldp >= nq + nk + nv && ldq >= nq && k_row_stride >= nk && v_row_stride >= nv, "attention_inputs: row strides smaller than the rows they hold");
+  EB_REQUIRE(aligned16(proj) && aligned16(q_norm) && aligned16(k_norm) && aligned16(q_out) && aligned16(k_cache) && aligned16(v_cache) &&
+                 aligned16(v_first), "attention_inputs: pointers must be 16-byte aligned");
+  InputParams p{};
+  p.proj = proj; p.ldp = ldp; p.nq = nq; p.nk = nk; p.nv = nv; p.wq = q_norm; p.wk = k_norm;
+  p.inv_q = 1.f / (float)q_count; p.inv_k = 1.f / (float)k_count; p.eps = eps; p.coef = temp_coef; p.every = temp_every;
+  p.vmix = vmix; p.vf = v_first; p.vf_bs = vf_batch_stride; p.vf_rs = vf_row_stride;
+  p.q = q_out; p.ldq = ldq; p.k = k_cache; p.k_bs = k_batch_stride; p.k_rs = k_row_stride; p.v = v_cache; p.v_bs = v_batch_stride; p.v_rs = v_row_stride;
+  p.cache_rows = cache_rows; p.rows_per_batch = rows_per_batch; p.pos_dev = pos_device; p.first = first;
+  cudaStream_t st = as_stream(stream);
+  if (dtype == EB_F32) return launch_inputs<float>(p, n1, st);
+  if (dtype == EB_F16) return launch_inputs<__half>(p, n1, st);
+  return launch_inputs<__nv_bfloat16>(p, n1, st);
+}

@@ -35,6 +35,7 @@
 
 #include "comm.cuh"
 #include "gated.cuh"
+#include "xielu.cuh"
 
 namespace eb {
 namespace {
@@ -100,6 +101,10 @@ struct GemmParams {
   // gated (normal orientation): columns come in blocks of 8 gates and their 8 ups; C is [M, N/2]
   int gated;
   float gate_limit, gate_alpha;
+  // the activation serves the output columns below act_cols (a multiple of 8); act_params: its two
+  // numbers on the device (EB_ACT_XIELU)
+  int act_cols;
+  const float *act_params;
 };
 
 // ---- PTX wrappers ---------------------------------------------------------------------------
@@ -303,7 +308,8 @@ template <int BN, bool SWAP> struct Scheduler {
 // First weight row of the group that a row tile of A belongs to.
 __device__ __forceinline__ int group_row(const GemmParams &p, int lane_tile) { return p.tile_group ? p.tile_group[lane_tile] * p.N : 0; }
 
-__device__ __forceinline__ float apply_act(float v, int act) {
+__device__ __forceinline__ float apply_act(float v, int act, float a0 = 0.f, float a1 = 0.f) {
+  if (act == EB_ACT_XIELU) return xielu_fast(v, a0, a1);
   if (act == EB_ACT_RELU) return fmaxf(v, 0.f);
   if (act == EB_ACT_GELU_TANH) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * v * (1.f + 0.044715f * v * v)));
   if (act == EB_ACT_GELU_ERF) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
@@ -668,7 +674,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
         const bool m_ok = m < p.M && row_in_limit(p, p.c_row_offset_dev ? __ldg(p.c_row_offset_dev) : 0);
         const long long c_off = m_ok ? c_row_offset(p, m) : 0;
         const int n_base = s.col_tile * BN;
-        const int act = p.act;
+        float act0 = 0.f, act1 = 0.f;
+        if (p.act_params) { act0 = __ldg(p.act_params); act1 = __ldg(p.act_params + 1); }
         const bool out_f32 = p.out_f32 != 0;
         const T *res_row = (res && m_ok) ? res + (long long)m * p.ldr : nullptr;
         constexpr int kChunks = BN / 16;
@@ -708,12 +715,13 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
                     rq[i][h].unpack(rf);
 #pragma unroll
                     for (int j = 0; j < 8; ++j) vv[j] += bf[j];
+                    const int act = n < p.act_cols ? p.act : EB_ACT_NONE;
                     if (act == EB_ACT_RELU) {
 #pragma unroll
                       for (int j = 0; j < 8; ++j) vv[j] = fmaxf(vv[j], 0.f);
                     } else if (act != EB_ACT_NONE) {
 #pragma unroll
-                      for (int j = 0; j < 8; ++j) vv[j] = apply_act(vv[j], act);
+                      for (int j = 0; j < 8; ++j) vv[j] = apply_act(vv[j], act, act0, act1);
                     }
 #pragma unroll
                     for (int j = 0; j < 8; ++j) vv[j] += rf[j];
@@ -956,7 +964,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
           // hides a branch, and a handful of branches per row was a third of a short launch.
           const int rows = p.M;
           const long long ldc = p.ldc;
-          const int act = p.act;
+          const int act = n < p.act_cols ? p.act : EB_ACT_NONE;
+          float act0 = 0.f, act1 = 0.f;
+          if (p.act_params) { act0 = __ldg(p.act_params); act1 = __ldg(p.act_params + 1); }
           const bool out_f32 = p.out_f32 != 0;
 #pragma unroll
           for (int m0 = 0; m0 < BN; m0 += 16) {
@@ -989,7 +999,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
               for (int j = 0; j < 16; ++j) y[j] = fmaxf(y[j], 0.f);
             } else if (act != EB_ACT_NONE) {
 #pragma unroll
-              for (int j = 0; j < 16; ++j) y[j] = apply_act(y[j], act);
+              for (int j = 0; j < 16; ++j) y[j] = apply_act(y[j], act, act0, act1);
             }
 #pragma unroll
             for (int j = 0; j < 16; ++j) y[j] += r[j];
@@ -1355,7 +1365,7 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
                      const int32_t *c_row_offset_device, int c_row_offset_limit, int flags, void *workspace,
                      size_t workspace_bytes, void *stream, const eb_comm *comm, const float *ln_colsum = nullptr,
                      const float *ln_bias = nullptr, double ln_eps = 0.0, bool reduce_scatter = false,
-                     size_t rs_stage_offset = 0) {
+                     size_t rs_stage_offset = 0, int act_cols = 0x7fffffff, const float *act_params = nullptr) {
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "gemm: operands must be fp16 or bf16 (got dtype %d)", dtype);
   if (ln_colsum || ln_bias) {
     EB_REQUIRE(ln_colsum && ln_bias, "gemm_ln: ln_colsum and ln_bias go together");
@@ -1366,7 +1376,7 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
   }
   EB_REQUIRE(out_dtype == dtype || out_dtype == EB_F32, "gemm: output must be the input type or fp32");
   EB_REQUIRE(M >= 0 && N >= 0 && K >= 0, "gemm: negative size");
-  EB_REQUIRE(act >= EB_ACT_NONE && act <= EB_ACT_GELU_ERF, "gemm: unknown activation %d", act);
+  EB_REQUIRE(act >= EB_ACT_NONE && (act <= EB_ACT_GELU_ERF || (act == EB_ACT_XIELU && act_params)), "gemm: unknown activation %d", act);
   EB_REQUIRE((flags & ~EB_GEMM_STATIC_W) == 0, "gemm: unknown flag bits 0x%x", flags);
   if (M == 0 || N == 0) return EB_OK;
   EB_REQUIRE(A && W && (C || reduce_scatter), "gemm: null operand");
@@ -1415,7 +1425,7 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
                comm->world, comm->recv_bytes / 2);
     p.comm = comm_dev(comm);
   }
-  p.bias = bias; p.residual = residual; p.ldr = ldr; p.act = act; p.out_f32 = out_dtype == EB_F32 && dtype != EB_F32;
+  p.bias = bias; p.residual = residual; p.ldr = ldr; p.act = act; p.act_cols = act_cols; p.act_params = act_params; p.out_f32 = out_dtype == EB_F32 && dtype != EB_F32;
 
   CUtensorMap tl, tc;
   int rc;
@@ -1534,6 +1544,15 @@ extern "C" int eb_gemm(const void *A, long long lda, const void *W, long long ld
   return gemm_impl(A, lda, W, ldw, C, ldc, bias, residual, ldr, M, N, K, dtype, out_dtype, act, c_rows_per_batch,
                    c_batch_stride, c_row_offset_device, c_row_offset_limit, flags, workspace, workspace_bytes, stream,
                    nullptr);
+}
+
+extern "C" int eb_gemm_xielu(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, const void *bias, int M,
+                             int N, int K, int act_cols, const float *act_params, int dtype, int out_dtype, int flags, void *workspace,
+                             size_t workspace_bytes, void *stream) {
+  EB_REQUIRE(act_params && (uintptr_t)act_params % 4 == 0, "gemm_xielu: the activation's two numbers are required");
+  EB_REQUIRE(act_cols >= 0 && act_cols % 8 == 0, "gemm_xielu: the activation covers a multiple of 8 columns (got %d)", act_cols);
+  return gemm_impl(A, lda, W, ldw, C, ldc, bias, nullptr, 0, M, N, K, dtype, out_dtype, EB_ACT_XIELU, 0, 0, nullptr, 0, flags, workspace,
+                   workspace_bytes, stream, nullptr, nullptr, nullptr, 0.0, false, 0, act_cols, act_params);
 }
 
 extern "C" int eb_gemm_ln(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc,

@@ -580,6 +580,9 @@ struct PlainParams {
   const int *pos_dev;          // position of query row 0, or null (0)
   const int *first;
   float scale_log2;
+  int group;                   // query heads per key / value head
+  const float *r1, *r2;        // per head: r1 * ln(1 + r2 * distance) is taken off the score, or null
+  int sink;                    // one is added to the softmax denominator
 };
 
 template <typename T>
@@ -599,8 +602,9 @@ __global__ void attention_plain_kernel(const PlainParams p) {
   int lo = p.first ? p.first[b] : 0;
   if (p.window > 0) lo = max(lo, pos - p.window + 1);
   lo = max(lo, max(0, pos - p.ring_rows + 1));
-  const T *K = reinterpret_cast<const T *>(p.k) + b * p.k_bs + h * p.k_hs, *V = reinterpret_cast<const T *>(p.v) + b * p.v_bs + h * p.v_hs;
-  float m = -1e30f, l = 0.f;
+  const T *K = reinterpret_cast<const T *>(p.k) + b * p.k_bs + h / p.group * p.k_hs, *V = reinterpret_cast<const T *>(p.v) + b * p.v_bs + h / p.group * p.v_hs;
+  const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
+  float m = p.sink ? 0.f : -1e30f, l = p.sink ? 1.f : 0.f;      // the sink: a score of 0 without a value
   for (int j0 = lo; j0 <= pos; j0 += 32) {
     const int j = j0 + lane;
     float s = -INFINITY;
@@ -609,6 +613,7 @@ __global__ void attention_plain_kernel(const PlainParams p) {
       float a = 0.f;
       for (int d = 0; d < p.dk; ++d) a = fmaf(sq[d], to_f32<T>(kr[d]), a);
       s = a * p.scale_log2;
+      if (p.r1) s -= r1 * log2f(fmaf(r2, (float)(pos - j), 1.f));
     }
     const float mn = fmaxf(m, warp_max(s)), alpha = exp2f(m - mn), pj = exp2f(s - mn);
     m = mn;
@@ -696,15 +701,18 @@ extern "C" int eb_latent_decode(const void *q, long long q_batch_stride, const v
 extern "C" int eb_attention_plain(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
                                   long long q_head_stride, long long k_batch_stride, long long k_row_stride, long long k_head_stride,
                                   long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
-                                  long long o_row_stride, long long o_head_stride, int batch, int heads, int q_len, int k_dim, int v_dim,
-                                  int window, int ring_rows, const int32_t *pos_device, const int32_t *first, float scale, int dtype,
-                                  void *stream) {
+                                  long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
+                                  int v_dim, int window, int ring_rows, const int32_t *pos_device, const int32_t *first, const float *bias_r1,
+                                  const float *bias_r2, int sink, float scale, int dtype, void *stream) {
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype_ok(dtype), "attention_plain: bad dtype %d", dtype);
   EB_REQUIRE(q && k && v && out, "attention_plain: null pointer");
   EB_REQUIRE(batch > 0 && batch <= 65535 && heads > 0 && heads <= 65535 && q_len > 0 && k_dim > 0 && v_dim > 0 && window >= 0 && ring_rows > 0,
              "attention_plain: bad sizes");
+  EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_plain: %d heads do not share keys in groups of %d", heads, kv_group);
+  EB_REQUIRE((bias_r1 == nullptr) == (bias_r2 == nullptr), "attention_plain: the distance bias has two numbers per head");
   PlainParams p{};
+  p.group = kv_group; p.r1 = bias_r1; p.r2 = bias_r2; p.sink = sink;
   p.q = q; p.k = k; p.v = v; p.o = out;
   p.q_bs = q_batch_stride; p.q_rs = q_row_stride; p.q_hs = q_head_stride;
   p.k_bs = k_batch_stride; p.k_rs = k_row_stride; p.k_hs = k_head_stride;

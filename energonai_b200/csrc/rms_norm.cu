@@ -8,6 +8,11 @@
 //                     the mixture that follows is evaluated on the new row in the same launch
 //                     (generation steps: the row is already in registers, and one launch less
 //                     lies on the critical path).
+//   stream_update     the residual step of blocks that normalise in front of AND behind a
+//                     sublayer: x += norm(y * sigmoid(gate)) * w_out, then h = norm(x) * w_next for
+//                     the sublayer that follows, and optionally a few more products of h whose
+//                     results stay in fp32 (the gates of a recurrence that follows).  With `src` it
+//                     starts the stream instead: x = scale * src.
 //
 // One CTA per row, the row register-resident in packs of 8; statistics, weights and the residual
 // are fp32 throughout.
@@ -206,6 +211,133 @@ __global__ void __launch_bounds__(THREADS) rms_residual_kernel(const ResidualPar
   if (warp == 0) route_warp(z, p.experts, p.r_top, p.r_idx + row * p.r_top, p.r_weights + row * p.r_top, nullptr, nullptr);
 }
 
+struct StreamParams {
+  const void *src;             // T rows lds apart: x = src_scale * src instead of x as it is (null: x as it is)
+  long long lds;
+  float src_scale;
+  const void *y, *gate;        // T rows; y null: nothing is added; gate null: no gate
+  long long ldy, ldg;
+  const float *w_out;          // [n2]
+  float *x;                    // fp32 stream, rows ldx apart
+  long long ldx;
+  const void *w_next;          // [n2] T, or null: no h
+  void *h;
+  long long ldh;
+  const void *proj;            // [n_proj][n2] T, or null
+  int n_proj;
+  float *proj_out;             // rows ldp apart
+  long long ldp;
+  float eps, inv_count;
+  int n2;
+};
+
+template <typename T, int PACKS, int THREADS>
+__global__ void __launch_bounds__(THREADS) stream_update_kernel(const StreamParams p) {
+  __shared__ float scratch[THREADS / 32];
+  extern __shared__ float dyn[];                   // the row of h, for the small products
+  const long long row = blockIdx.x;
+  const int packs = p.n2 / 8;
+  griddep_wait();
+  griddep_launch();
+  float v[PACKS][8];
+  float r = 0.f;
+  if (p.y) {
+    float sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < PACKS; ++i) {
+      const int c = threadIdx.x + i * THREADS;
+      if (c >= packs) break;
+      load8<T>(reinterpret_cast<const T *>(p.y) + row * p.ldy + c * 8, v[i]);
+      if (p.gate) {
+        float g[8];
+        load8<T>(reinterpret_cast<const T *>(p.gate) + row * p.ldg + c * 8, g);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = v[i][e] / (1.f + __expf(-g[e]));
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sq = fmaf(v[i][e], v[i][e], sq);
+    }
+    r = rsqrtf(block_sum<THREADS>(sq, scratch) * p.inv_count + p.eps);
+  }
+  float sx = 0.f;
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= packs) break;
+    float xv[8];
+    if (p.src) {
+      load8<T>(reinterpret_cast<const T *>(p.src) + row * p.lds + c * 8, xv);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) xv[e] *= p.src_scale;
+    } else {
+      load8<float>(p.x + row * p.ldx + c * 8, xv);
+    }
+    if (p.y) {
+      float wv[8];
+      load8<float>(p.w_out + c * 8, wv);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) xv[e] = fmaf(v[i][e] * r, wv[e], xv[e]);
+    }
+    store8<float>(p.x + row * p.ldx + c * 8, xv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      sx = fmaf(xv[e], xv[e], sx);
+      v[i][e] = xv[e];
+    }
+  }
+  if (!p.w_next) return;
+  r = rsqrtf(block_sum<THREADS>(sx, scratch) * p.inv_count + p.eps);
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= packs) break;
+    float wv[8];
+    load8<T>(reinterpret_cast<const T *>(p.w_next) + c * 8, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) wv[e] *= v[i][e] * r;
+    store8<T>(reinterpret_cast<T *>(p.h) + row * p.ldh + c * 8, wv);
+    if (p.proj) {
+      // the products read h as every other product does: rounded to the operand type
+#pragma unroll
+      for (int e = 0; e < 8; ++e) dyn[c * 8 + e] = to_f32<T>(from_f32<T>(wv[e]));
+    }
+  }
+  if (!p.proj) return;
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int e = warp; e < p.n_proj; e += THREADS / 32) {
+    const T *wr = reinterpret_cast<const T *>(p.proj) + (long long)e * p.n2;
+    float acc = 0.f;
+#pragma unroll 4
+    for (int c = lane; c < packs; c += 32) {
+      float f[8];
+      load8<T>(wr + c * 8, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc = fmaf(f[j], dyn[c * 8 + j], acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) p.proj_out[row * p.ldp + e] = acc;
+  }
+}
+
+template <typename T> int launch_stream(const StreamParams &p, int n1, cudaStream_t st) {
+  const int packs = p.n2 / 8, threads = p.proj ? 1024 : kNormThreads, per = (packs + threads - 1) / threads;
+  const size_t smem = p.proj ? (size_t)p.n2 * sizeof(float) : 0;
+  auto go = [&](auto kern) -> int {
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+      cudaGetLastError();
+      return fail(EB_ECUDA, "stream_update: cannot reserve %zu bytes of shared memory", smem);
+    }
+    launch_pdl(kern, dim3(n1), dim3(threads), smem, st, p);
+    return check_launch("stream_update");
+  };
+  if (p.proj) return per <= 1 ? go(stream_update_kernel<T, 1, 1024>) : go(stream_update_kernel<T, 2, 1024>);
+  if (per <= 1) return go(stream_update_kernel<T, 1, kNormThreads>);
+  if (per <= 2) return go(stream_update_kernel<T, 2, kNormThreads>);
+  if (per <= 4) return go(stream_update_kernel<T, 4, kNormThreads>);
+  return go(stream_update_kernel<T, 8, kNormThreads>);
+}
+
 template <typename TI, typename TO>
 int launch_rms(const RmsParams &p, int n1, cudaStream_t st) {
   const int packs = p.n2 / 8, per = (packs + kNormThreads - 1) / kNormThreads;
@@ -307,4 +439,31 @@ extern "C" int eb_rms_residual(const void *y, long long ldy, int dtype, const in
   if (dtype == EB_F16) return EB_RES(__half);
   return EB_RES(__nv_bfloat16);
 #undef EB_RES
+}
+
+extern "C" int eb_stream_update(const void *src, long long lds, float src_scale, const void *y, long long ldy, const void *gate, long long ldg,
+                                const float *w_out, float *x, long long ldx, const void *w_next, void *h, long long ldh, const void *proj,
+                                int n_proj, float *proj_out, long long ldp, float eps, int n1, int n2, int count, int dtype, void *stream) {
+  if (n1 == 0) return EB_OK;
+  EB_REQUIRE(dtype_ok(dtype), "stream_update: bad dtype %d", dtype);
+  EB_REQUIRE(x && (src || y || w_next), "stream_update: null pointer");
+  EB_REQUIRE(n1 > 0 && n2 > 0 && n2 % 8 == 0 && n2 <= kMaxNormWidth, "stream_update: width %d must be a multiple of 8, at most %d", n2, kMaxNormWidth);
+  EB_REQUIRE(count > 0 && count <= n2, "stream_update: the mean is over 1..n2 elements");
+  EB_REQUIRE(ldx >= n2 && ldx % 8 == 0 && (!src || (lds >= n2 && lds % 8 == 0)) && (!y || (ldy >= n2 && ldy % 8 == 0)) &&
+                 (!gate || (ldg >= n2 && ldg % 8 == 0)) && (!w_next || (ldh >= n2 && ldh % 8 == 0)),
+             "stream_update: row strides must be multiples of 8 and >= n2");
+  EB_REQUIRE(!y || w_out, "stream_update: the added row needs its weight");
+  EB_REQUIRE(!gate || y, "stream_update: a gate without a row");
+  EB_REQUIRE(!w_next || h, "stream_update: no place for the normalised row");
+  EB_REQUIRE(!proj || (w_next && proj_out && n_proj > 0 && ldp >= n_proj), "stream_update: the small products need the normalised row and their output");
+  EB_REQUIRE(aligned16(src) && aligned16(y) && aligned16(gate) && aligned16(w_out) && aligned16(x) && aligned16(w_next) && aligned16(h) &&
+                 aligned16(proj), "stream_update: pointers must be 16-byte aligned");
+  StreamParams p{};
+  p.src = src; p.lds = lds; p.src_scale = src_scale; p.y = y; p.ldy = ldy; p.gate = gate; p.ldg = ldg; p.w_out = w_out;
+  p.x = x; p.ldx = ldx; p.w_next = w_next; p.h = h; p.ldh = ldh; p.proj = proj; p.n_proj = n_proj; p.proj_out = proj_out; p.ldp = ldp;
+  p.eps = eps; p.inv_count = 1.f / (float)count; p.n2 = n2;
+  cudaStream_t st = as_stream(stream);
+  if (dtype == EB_F32) return launch_stream<float>(p, n1, st);
+  if (dtype == EB_F16) return launch_stream<__half>(p, n1, st);
+  return launch_stream<__nv_bfloat16>(p, n1, st);
 }

@@ -87,23 +87,54 @@ def gemm(a, w, bias=None, act=None, residual=None, out=None, out_dtype=None, out
     return out
 
 
-def gemm_f32(a, w, out=None):
-    """a [M,K] @ w [N,K].T in true 32-bit (CUDA cores, no reduced-precision mode)."""
-    require_cuda(a, w, out)
-    if a.dim() != 2 or w.dim() != 2 or a.shape[1] != w.shape[1] or a.dtype != torch.float32 or w.dtype != torch.float32:
-        raise RuntimeError("gemm_f32: fp32 a [M,K] and w [N,K] required")
+def gemm_xielu(a, w, bias, act_params, act_cols, static_weight=False):
+    """a [M,K] @ w [N,K].T + bias with xIELU on the columns below act_cols (a multiple of 8); act_params:
+    device fp32 (softplus(p), 1/2 + softplus(q)), see xielu_params()."""
+    require_cuda(a, w, bias, act_params)
+    if a.dim() != 2 or w.dim() != 2 or a.shape[1] != w.shape[1] or a.dtype != w.dtype or a.dtype not in (torch.float16, torch.bfloat16):
+        raise RuntimeError("gemm_xielu: fp16 or bf16 a [M,K] and w [N,K] of one dtype required")
+    if act_params.dtype != torch.float32 or act_params.numel() != 2 or (bias is not None and (bias.dtype != a.dtype or bias.numel() != w.shape[0])):
+        raise RuntimeError("gemm_xielu: two fp32 numbers, and a bias of the operand dtype with one entry per column")
     a, w = (t if t.stride(1) == 1 else t.contiguous() for t in (a, w))
     (M, K), N = a.shape, w.shape[0]
-    if out is None:
-        out = torch.empty((M, N), dtype=torch.float32, device=a.device)
-    check(lib().eb_gemm_f32(ptr(a), a.stride(0), 0, ptr(w), w.stride(0), 0, ptr(out), out.stride(0), 0, M, N, K, 1, None, None,
-                            stream_ptr()), "gemm_f32")
+    out = torch.empty((M, N), dtype=a.dtype, device=a.device)
+    nbytes = lib().eb_gemm_workspace_bytes(M, N, K)
+    ws = workspace(a.device, nbytes) if nbytes else None
+    check(lib().eb_gemm_xielu(ptr(a), a.stride(0), ptr(w), w.stride(0), ptr(out), N, ptr(bias), M, N, K, int(act_cols), ptr(act_params),
+                              dtype_code(a.dtype), dtype_code(a.dtype), 1 if static_weight else 0, ptr(ws),
+                              ws.numel() if ws is not None else 0, stream_ptr()), "gemm_xielu")
     return out
 
 
-def project(x, w, out_dtype=None):
-    """x @ w.T with a model's weight: the tensor-core GEMM, or the 32-bit one for models run in fp32."""
-    return gemm_f32(x, w) if w.dtype == torch.float32 else gemm(x, w, out_dtype=out_dtype, static_weight=True)
+def xielu_params(p, q):
+    """(softplus(p), 1/2 + softplus(q)) as the fp32 pair the kernels take."""
+    s = torch.nn.functional.softplus(torch.tensor([float(p), float(q)], dtype=torch.float64))
+    return torch.stack([s[0], 0.5 + s[1]]).float()
+
+
+def gemm_f32(a, w, bias=None, xielu=None):
+    """a [M,K] @ w [N,K].T (+ bias) in true 32-bit (CUDA cores, no reduced-precision mode); xielu =
+    (act_params, act_cols) as in gemm_xielu."""
+    act_params, act_cols = xielu if xielu is not None else (None, 0)
+    require_cuda(a, w, bias, act_params)
+    if a.dim() != 2 or w.dim() != 2 or a.shape[1] != w.shape[1] or any(t is not None and t.dtype != torch.float32 for t in (a, w, bias, act_params)):
+        raise RuntimeError("gemm_f32: fp32 a [M,K] and w [N,K] required")
+    a, w = (t if t.stride(1) == 1 else t.contiguous() for t in (a, w))
+    (M, K), N = a.shape, w.shape[0]
+    out = torch.empty((M, N), dtype=torch.float32, device=a.device)
+    check(lib().eb_gemm_f32(ptr(a), a.stride(0), 0, ptr(w), w.stride(0), 0, ptr(out), out.stride(0), 0, M, N, K, 1, None, None, ptr(bias),
+                            int(act_cols), ptr(act_params), stream_ptr()), "gemm_f32")
+    return out
+
+
+def project(x, w, out_dtype=None, bias=None, xielu=None):
+    """x @ w.T (+ bias) with a model's weight: the tensor-core GEMM, or the 32-bit one for models run in
+    fp32.  xielu = (act_params, act_cols): that activation on the first columns."""
+    if w.dtype == torch.float32:
+        return gemm_f32(x, w, bias=bias, xielu=xielu)
+    if xielu is not None:
+        return gemm_xielu(x, w, bias, *xielu, static_weight=True)
+    return gemm(x, w, bias=bias, out_dtype=out_dtype, static_weight=True)
 
 
 LN_FOLD_MAX_ROWS = 32

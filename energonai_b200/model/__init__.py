@@ -1,14 +1,19 @@
 """Layer modules and model factories with the interfaces of the reference's `energonai.model`."""
 from .attention import MultiHeadAttention1D
-from .mlp import MLP1D, gelu_impl
+from .mlp import MLP1D, XIELUFeedForward, gelu_impl
 from .endecoder import Block1D
 from .embedding import Embedding1D
 from .downstream import LMHead1D
 from .generation import GenerationModel
-from .config import LatentDecoderConfig
-from .latent_attention import LatentAttention, LatentCache, SequenceState
+from .config import LatentDecoderConfig, SandwichDecoderConfig
+from .sequence_state import RecurrentState, RingCache, SequenceState
+from .latent_attention import LatentAttention
 from .moe import MixtureOfExperts
+from .layered_decoder import LayeredDecoder
 from .latent_decoder import LatentDecoder, OutputNormBlock
+from .grouped_attention import GroupedAttention
+from .matrix_memory import MatrixMemory
+from .sandwich_decoder import SandwichBlock, SandwichDecoder
 from .model_factory import (PipelineModel, create_pipeline_model, gpt2_small, gpt2_large, gpt2_8B, gpt3, hf_gpt2,
                             bert_small, bert_large, bert_8B, bert_175B, opt_125M, opt_6B, opt_13B, opt_30B, opt_66B,
                             opt_175B)
@@ -16,5 +21,6 @@ from .model_factory import (PipelineModel, create_pipeline_model, gpt2_small, gp
 __all__ = ["MultiHeadAttention1D", "MLP1D", "Block1D", "Embedding1D", "LMHead1D", "PipelineModel", "gelu_impl",
            "create_pipeline_model", "gpt2_small", "gpt2_large", "gpt2_8B", "gpt3", "hf_gpt2", "bert_small",
            "bert_large", "bert_8B", "bert_175B", "opt_125M", "opt_6B", "opt_13B", "opt_30B", "opt_66B", "opt_175B",
-           "GenerationModel", "LatentDecoderConfig", "LatentDecoder", "LatentAttention", "LatentCache", "SequenceState",
-           "MixtureOfExperts", "OutputNormBlock"]
+           "GenerationModel", "LatentDecoderConfig", "LatentDecoder", "LatentAttention", "RingCache", "RecurrentState",
+           "SequenceState", "MixtureOfExperts", "OutputNormBlock", "LayeredDecoder", "GroupedAttention", "MatrixMemory", "SandwichBlock",
+           "SandwichDecoder", "SandwichDecoderConfig", "XIELUFeedForward"]

@@ -1,4 +1,4 @@
-"""Latent attention with a sliding window, its ring cache, and the state of a batch of sequences.
+"""Latent attention with a sliding window over a ring cache of latent rows.
 
 Per token a layer keeps one latent row c = RMSNorm(W_dkv h); keys and values of every head are
 linear maps of it, k = W_uk c, v = W_uv c.  Two evaluation orders give the same result:
@@ -21,124 +21,7 @@ from ..gemm import project
 from ..moe import per_head
 from ..nn import RMSNorm1D, init_weight
 from ..norm import rms_norm
-from .attention import KVCache
-
-
-def round_up(n, m):
-    return -(-n // m) * m
-
-
-class LatentCache(KVCache):
-    """[batch, rows, latent] ring of latent rows: position p lives in row p mod rows.  `window` is the
-    longest window of the layers that read it (0: unlimited), so rows = min(positions, window).
-    A ring shorter than its window has never wrapped, which is why it can grow like a KVCache."""
-
-    def __init__(self, width, window, reserve=256):
-        super().__init__(reserve)
-        self.width, self.window = width, window
-
-    def rows_for(self, positions):
-        return min(positions, self.window) if self.window > 0 else positions
-
-    def prepare(self, batch, positions, dtype, device):
-        """For a new batch: room for `positions`; memory kept from an earlier batch of the same size
-        is used again when it has exactly the rows that are needed."""
-        self.reset()
-        rows = self.rows_for(positions)
-        if self.buf is None or self.buf.shape[:2] != (batch, rows) or self.buf.dtype != dtype or self.buf.device != device:
-            self.buf = torch.zeros((batch, rows, self.width), dtype=dtype, device=device)     # (unwritten rows must be finite)
-
-    def grow(self, positions):
-        rows = self.rows_for(positions)
-        have = self.buf.shape[1]
-        if rows > have:
-            self.ensure(self.buf.shape[0], self.rows_for(positions + self.reserve), self.width, self.buf.dtype, self.buf.device, exact=True)
-            self.buf[:, have:].zero_()
-
-    def keep(self, rows):
-        self.buf = self.buf.index_select(0, rows)
-
-
-class SequenceState:
-    """What a batch of sequences holds between steps: the caches, where each sequence begins in the
-    left-padded batch, and the common position.  `kv_state` = (position of the next token, its
-    successor) lives on the device, where captured steps advance it."""
-
-    def __init__(self, caches):
-        self.caches = caches                    # {layer: LatentCache}
-        self.first = self.kv_state = None
-        self.batch, self.length, self.padded = 0, 0, False
-
-    def begin(self, first, prompt_len, reserve, dtype, device):
-        """first: list with the number of padding positions in front of each sequence."""
-        B = len(first)
-        if self.first is None or self.first.numel() != B or self.first.device != device:
-            self.first = torch.empty(B, dtype=torch.int32, device=device)
-            self.kv_state = torch.empty(2, dtype=torch.int32, device=device)
-        self.first.copy_(torch.tensor(first, dtype=torch.int32))
-        self.kv_state.copy_(torch.tensor([prompt_len, prompt_len + 1], dtype=torch.int32))
-        self.batch, self.length, self.padded = B, prompt_len, any(first)
-        for c in self.caches.values():
-            c.prepare(B, prompt_len + max(0, reserve), dtype, device)
-            c.len = prompt_len
-
-    def ensure(self, positions):
-        for c in self.caches.values():
-            c.grow(positions)
-
-    def capacity(self):
-        """Positions the caches can take; None if every layer's ring holds its whole window."""
-        caps = [c.buf.shape[1] for c in self.caches.values() if c.window <= 0 or c.buf.shape[1] < c.window]
-        return min(caps) if caps else None
-
-    def set_length(self, n):
-        self.length = n
-        for c in self.caches.values():
-            c.len = n
-
-    def advance(self):
-        self.kv_state.add_(1)
-        self.set_length(self.length + 1)
-
-    def keep(self, rows):
-        """Only the sequences `rows` (list of indices) go on; the memory of the others is given back."""
-        if list(rows) == list(range(self.batch)):
-            return
-        sel = torch.tensor(list(rows), dtype=torch.long, device=self.first.device)
-        self.first = self.first.index_select(0, sel)
-        for c in self.caches.values():
-            c.keep(sel)
-        self.batch = len(rows)
-
-    def fork(self, rows):
-        """A state of its own for the sequences `rows`."""
-        out = SequenceState({k: LatentCache(c.width, c.window, c.reserve) for k, c in self.caches.items()})
-        for k, c in self.caches.items():
-            out.caches[k].buf, out.caches[k].len = c.buf, c.len
-        out.first, out.kv_state = self.first, self.kv_state.clone()
-        out.batch, out.length, out.padded = self.batch, self.length, self.padded
-        if list(rows) == list(range(self.batch)):
-            raise RuntimeError("fork: nothing would be left")
-        out.keep(rows)
-        return out
-
-
-class PromptContext:
-    """One prompt pass: shapes, padding, and the latents of the layers run so far."""
-
-    def __init__(self, state, batch, seq, mask):
-        self.state, self.batch, self.seq, self.mask = state, batch, seq, mask
-        self.first = state.first if state.padded else None
-        self.latents = {}
-
-
-class StepContext:
-    """One generation step."""
-
-    def __init__(self, state):
-        self.state, self.batch = state, state.batch
-        self.first = state.first if state.padded else None
-        self.pos = state.kv_state[0:1]
+from .sequence_state import round_up
 
 
 class LatentAttention(nn.Module):

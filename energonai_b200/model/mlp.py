@@ -6,7 +6,9 @@ from typing import Callable, Optional
 import torch
 from torch import dtype, nn
 
-from ..nn import Linear1D_Col, Linear1D_Row
+from ..gemm import project, xielu_params
+from ..nn import Linear1D_Col, Linear1D_Row, init_weight
+from .sequence_state import round_up
 
 
 def gelu_impl(x):
@@ -50,3 +52,22 @@ class MLP1D(nn.Module):
             residual = residual[:, -1:, :] if residual is not None else None
         inter = self.dense_1(hidden_states, act=self.act_code, fold_norm=fold_norm)
         return self.dense_2(inter, residual=residual, transient_ok=transient_ok)
+
+
+class XIELUFeedForward(nn.Module):
+    """W_down xIELU(W_up h), with the pre-activation of a residual gate, W_gate h + b, from the same
+    product (the activation covers its first columns only)."""
+
+    def __init__(self, width, ff, dtype, device=None):
+        super().__init__()
+        kw = dict(dtype=dtype, device=device)
+        self.ff, self.ff_padded = ff, round_up(ff, 8)
+        self.up = init_weight(self.ff_padded + width, width, **kw)              # up | residual gate
+        self.bias = init_weight(self.ff_padded + width, std=0.0, **kw)
+        self.act = nn.Parameter(xielu_params(0.8, 0.8).to(device), requires_grad=False)
+        self.down = init_weight(width, self.ff_padded, **kw)
+
+    def forward(self, h):
+        """-> (y, pre-activation of its gate)."""
+        u = project(h, self.up, bias=self.bias, xielu=(self.act, self.ff_padded))
+        return project(u[:, :self.ff_padded], self.down), u[:, self.ff_padded:]

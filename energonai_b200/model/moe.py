@@ -10,7 +10,7 @@ from torch import nn
 from ..gemm import project
 from ..moe import SKINNY_MAX_ENTRIES, SortedRows, grouped_gemm, new_counts, route, skinny_experts
 from ..nn import init_weight
-from .latent_attention import round_up
+from .sequence_state import round_up
 
 SKINNY_MAX_TOKENS = 128      # up to here an expert gets a handful of rows: stream its weights instead
 

@@ -62,7 +62,7 @@ def grouped_gemm(a, w, plan, gate=None):
     if a.dtype == torch.float32:
         out = torch.empty((M, N), dtype=a.dtype, device=a.device)
         check(lib().eb_gemm_f32(ptr(a), a.stride(0), 0, ptr(w), K, N * K, ptr(out), N, 0, M, N, K, 1, ptr(plan.tile_group),
-                                ptr(plan.live_tiles), stream_ptr()), "gemm_f32")
+                                ptr(plan.live_tiles), None, 0, None, stream_ptr()), "gemm_f32")
         return gated_act(out, limit, alpha) if gate is not None else out
     out = torch.empty((M, N // 2 if gate is not None else N), dtype=a.dtype, device=a.device)
     check(lib().eb_gemm_grouped(ptr(a), a.stride(0), ptr(w), K, ptr(out), out.stride(0), M, N, K, E, ptr(plan.tile_group),
@@ -108,8 +108,8 @@ def per_head(a, w):
         raise RuntimeError("per_head: a [rows, heads*K] and contiguous w [heads, N, K] of one dtype required")
     out = torch.empty((B, H * N), dtype=a.dtype, device=a.device)
     if a.dtype == torch.float32:
-        check(lib().eb_gemm_f32(ptr(a), a.stride(0), K, ptr(w), K, N * K, ptr(out), H * N, N, B, N, K, H, None, None, stream_ptr()),
-              "gemm_f32")
+        check(lib().eb_gemm_f32(ptr(a), a.stride(0), K, ptr(w), K, N * K, ptr(out), H * N, N, B, N, K, H, None, None, None, 0, None,
+                                stream_ptr()), "gemm_f32")
     else:
         check(lib().eb_grouped_skinny(ptr(a), a.stride(0), K, 1, ptr(w), N * K, K, ptr(out), H * N, N, None, B, H, N, K, 0, 0.0, 0.0,
                                       dtype_code(a.dtype), stream_ptr()), "grouped_skinny")

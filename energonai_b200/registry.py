@@ -79,10 +79,13 @@ def _populate():
         return
     _done = True
     from . import model as M
-    from .model.config import LatentDecoderConfig
+    from .model.config import LatentDecoderConfig, SandwichDecoderConfig
     from .model.latent_decoder import LatentDecoder
+    from .model.sandwich_decoder import SandwichDecoder
+    from .utils.checkpointing_mutolix import processing_Mutolix
     from .utils.checkpointing_tulezen import processing_Tulezen
     for name in ("opt_125M", "opt_6B", "opt_13B", "opt_30B", "opt_66B", "opt_175B", "gpt2_small", "gpt2_large", "gpt2_8B", "gpt3",
                  "hf_gpt2", "bert_small", "bert_large", "bert_8B", "bert_175B"):
         register_factory(name, getattr(M, name))
     register_architecture("Tulezen", LatentDecoderConfig, LatentDecoder, processing_Tulezen)
+    register_architecture("Mutolix", SandwichDecoderConfig, SandwichDecoder, processing_Mutolix)

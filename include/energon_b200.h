@@ -46,6 +46,7 @@ extern "C" {
 #define EB_ACT_RELU 1
 #define EB_ACT_GELU_TANH 2 /* energonai/model/model_factory.py:32-35 (gelu_impl)            */
 #define EB_ACT_GELU_ERF 3  /* torch.nn.functional.gelu                                      */
+#define EB_ACT_XIELU 4     /* eb_gemm_xielu, eb_gemm_f32                                    */
 
 /* flags for eb_gemm */
 #define EB_GEMM_STATIC_W 1 /* W is constant (model weights): the kernel may start reading it while
@@ -250,6 +251,14 @@ EB_API int eb_gemm(const void *A, long long lda, const void *W, long long ldw, v
             int c_row_offset_limit, int flags, void *workspace, size_t workspace_bytes, void *stream);
 EB_API size_t eb_gemm_workspace_bytes(int M, int N, int K);
 
+/* eb_gemm (no residual, plain rows) whose activation is xIELU on the columns below act_cols, a
+ * multiple of 8; the other columns get their bias only.  act_params: device floats
+ * (softplus(p), 1/2 + softplus(q)) of
+ *   z > 0: softplus(p) z^2 + z/2;   z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2. */
+EB_API int eb_gemm_xielu(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, const void *bias,
+                  int M, int N, int K, int act_cols, const float *act_params, int dtype, int out_dtype, int flags,
+                  void *workspace, size_t workspace_bytes, void *stream);
+
 /* Row-parallel GEMM with the tensor-parallel all-reduce fused into its epilogue, for the
  * generation orientation (M <= 128).  Replaces "F.linear, then dist.all_reduce, then + bias" of
  * colossalai's Linear1D_Row (the row-parallel layers constructed at
@@ -359,10 +368,13 @@ EB_API int eb_grouped_skinny(const void *A, long long lda, long long a_group_str
                       const int32_t *idx, int rows, int groups, int N, int K, int gated, float limit, float alpha, int dtype,
                       void *stream);
 
-/* C = A . W^T in true 32-bit.  Strided groups, or row tiles with their group (one of the two). */
+/* C = A . W^T in true 32-bit.  Strided groups, or row tiles with their group (one of the two).  A single
+ * product may add bias [N] and apply xIELU to the columns below act_cols (act_params as
+ * eb_gemm_xielu; either NULL: left out). */
 EB_API int eb_gemm_f32(const float *A, long long lda, long long a_group_stride, const float *W, long long ldw,
                 long long w_group_stride, float *C, long long ldc, long long c_group_stride, int M, int N, int K, int groups,
-                const int32_t *tile_group, const int32_t *live_tiles, void *stream);
+                const int32_t *tile_group, const int32_t *live_tiles, const float *bias, int act_cols, const float *act_params,
+                void *stream);
 
 /* The gated activation alone: x [n1, 2*half] in the 8 + 8 column order -> y [n1, half]. */
 EB_API int eb_gated_act(const void *x, long long ldx, void *y, long long ldy, int n1, int half, float limit, float alpha,
@@ -407,6 +419,61 @@ EB_API int eb_rms_residual(const void *y, long long ldy, int dtype, const int32_
                     const float *weights, int top, const void *w, float w_offset, float eps, float *x, long long ldx, void *xt,
                     long long ldt, int n1, int n2, int count, const void *router, int experts, int router_top,
                     int32_t *router_idx, float *router_weights, void *stream);
+
+/* The residual step of blocks with a norm in front of and behind every sublayer, per row of n2 elements
+ * (means over the first `count`; norm(z) = z / sqrt(mean(z^2) + eps)):
+ *   x = src_scale * src          if src (the embedding rows, `dtype`), else x as it is (fp32)
+ *   x += norm(y * sigmoid(gate)) * w_out        if y  (gate NULL: 1; w_out fp32)
+ *   h = norm(x) * w_next                        if w_next; h in `dtype`
+ *   proj_out[row][e] = h . proj[e], e < n_proj  if proj; h as rounded, fp32 results */
+EB_API int eb_stream_update(const void *src, long long lds, float src_scale, const void *y, long long ldy, const void *gate,
+                     long long ldg, const float *w_out, float *x, long long ldx, const void *w_next, void *h, long long ldh,
+                     const void *proj, int n_proj, float *proj_out, long long ldp, float eps, int n1, int n2, int count,
+                     int dtype, void *stream);
+
+/* Queries, keys and values of a projected row [q: heads*dk | k: kv_heads*dk | v: kv_heads*dv] made ready
+ * for attention.  q and k are divided by the root mean square over ALL their rows (counts q_count and
+ * k_count: heads may be zero-padded) and multiplied by q_norm / k_norm; q also by
+ *   1 + temp_coef * ln(floor((p + 1) / temp_every) + 1)      at position p (temp_every 0: 1);
+ * with vmix (device scalar) v becomes (1 - vmix) v + vmix v_first, v_first the cached value row of the
+ * same token in another layer's cache.  q goes to q_out, k and v to cache row col = pos0 + s of
+ * sequence b (row b*rows_per_batch + s of n1; pos0 from pos_device, NULL: 0); nothing is stored for
+ * col >= cache_rows.  p = col - first[b]. */
+EB_API int eb_attention_inputs(const void *proj, long long ldp, int heads, int kv_heads, int dk, int dv, const void *q_norm,
+                        int q_count, const void *k_norm, int k_count, float eps, float temp_coef, int temp_every,
+                        const float *vmix, const void *v_first, long long vf_batch_stride, long long vf_row_stride,
+                        void *q_out, long long ldq, void *k_cache, long long k_batch_stride, long long k_row_stride,
+                        void *v_cache, long long v_batch_stride, long long v_row_stride, int cache_rows, int n1,
+                        int rows_per_batch, const int32_t *pos_device, const int32_t *first, int dtype, void *stream);
+
+/* ---- matrix memory ------------------------------------------------------------------------------ */
+
+/* A recurrent layer whose state per head is a matrix S [dk][dv], a vector n [dk] and a scalar m.  With
+ *   i = cap tanh((a_i + bias_i) / cap),  f = logsigmoid(cap tanh((a_f + bias_f) / cap)):
+ *   m' = max(f + m, i);  S' = exp(f + m - m') S + exp(i - m') k v^T;  n' likewise with k alone;
+ *   o = S'^T (q scale) / (max(|n' . q scale|, exp(-m')) + 1e-6)
+ * all in fp32.  gates: fp32 rows ldg apart, a_i of head h at column h, a_f at column heads + h.
+ * q, k (heads*dk), v (heads*dv) and o are column ranges of rows ldp / ldo apart.  The state is
+ * S [batch][heads][dk][dv], n [batch][heads][dk], m [batch][heads], fp32.
+ *
+ * eb_memory_scan: a whole prompt, rows b*seq + s, from an empty state; rows s < first[b] are padding
+ * and leave it empty; CUDA cores, any sizes, token by token. */
+EB_API int eb_memory_scan(const void *q, const void *k, const void *v, long long ldp, const float *gates, long long ldg,
+                   const float *bias_i, const float *bias_f, float cap, float scale, const int32_t *first, void *o,
+                   long long ldo, float *S, float *n, float *m, int batch, int seq, int heads, int dk, int dv, int dtype,
+                   void *stream);
+
+/* One token per sequence: the state goes on by one step, and
+ *   out[h] = unit(o_h) * norm * sigmoid(g), unit(o) = o / sqrt(mean over dv_count of o^2 + eps). */
+EB_API int eb_memory_step(const void *q, const void *k, const void *v, const void *g, long long ldp, const float *gates,
+                   long long ldg, const float *bias_i, const float *bias_f, float cap, float scale, const void *norm,
+                   int dv_count, float eps, void *out, long long ldo, float *S, float *n, float *m, int batch, int heads,
+                   int dk, int dv, int dtype, void *stream);
+
+/* The same tail for the rows of a prompt: out[h] = unit(o_h) * norm * sigmoid(g) per head of dv elements
+ * (dv_count of them real). */
+EB_API int eb_head_norm_gate(const void *o, long long ldo, const void *g, long long ldg, const void *norm, float eps, void *out,
+                      long long ld_out, int rows, int heads, int dv, int dv_count, int dtype, void *stream);
 
 /* ---- the tail of a greedy generation step ----------------------------------------------------- */
 
@@ -470,13 +537,16 @@ EB_API int eb_attention_prefill_window_tc(const void *q, const void *k, const vo
 /* Windowed causal attention for any head sizes and fp32 / fp16 / bf16 on the CUDA cores: query row
  * i holds position pos0 + i (pos0 from pos_device, NULL: 0) and sees the positions
  * max(first[b], its own - window + 1) .. its own; the key / value of position j is row
- * j mod ring_rows.  Head strides may be 0 (keys shared by the heads). */
+ * j mod ring_rows.  Head strides may be 0 (keys shared by the heads); kv_group query heads share a
+ * key / value head.  bias_r1 / bias_r2 (or NULL): per query head, r1 * ln(1 + r2 * distance) is taken off
+ * the scaled score.  sink != 0 adds one to the softmax denominator (a key of score 0 without a value). */
 EB_API int eb_attention_plain(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
                        long long q_row_stride, long long q_head_stride, long long k_batch_stride, long long k_row_stride,
                        long long k_head_stride, long long v_batch_stride, long long v_row_stride, long long v_head_stride,
                        long long o_batch_stride, long long o_row_stride, long long o_head_stride, int batch, int heads,
-                       int q_len, int k_dim, int v_dim, int window, int ring_rows, const int32_t *pos_device,
-                       const int32_t *first, float scale, int dtype, void *stream);
+                       int kv_group, int q_len, int k_dim, int v_dim, int window, int ring_rows, const int32_t *pos_device,
+                       const int32_t *first, const float *bias_r1, const float *bias_r2, int sink, float scale, int dtype,
+                       void *stream);
 
 /* Generation step of latent attention with absorbed projections: q [batch][heads * rank] are the
  * queries in latent space, the cached latent row of a position is key and value of every head,

@@ -8,7 +8,7 @@ import torch
 import tulezen_plain as P
 from energonai_b200 import _lib, registry
 from energonai_b200.attention import pick_latent_nsplit
-from energonai_b200.model import LatentCache, LatentDecoder, LatentDecoderConfig, PipelineModel, GenerationModel, SequenceState
+from energonai_b200.model import GenerationModel, LatentDecoder, LatentDecoderConfig, PipelineModel, RingCache, SequenceState
 from energonai_b200.trace import TraceSession
 from energonai_b200.utils import load_checkpoint, load_safetensors, load_state_dict, processing_Tulezen
 
@@ -153,7 +153,7 @@ def test_cache_is_a_ring_as_long_as_the_longest_window_of_its_readers():
 
 
 def test_state_keeps_and_forks_sequences():
-    s = SequenceState({0: LatentCache(8, 4)})
+    s = SequenceState({0: RingCache(8, 4)})
     s.begin([2, 0, 1], 6, 3, torch.float32, torch.device("cpu"))
     s.caches[0].buf.copy_(torch.arange(3.)[:, None, None].expand_as(s.caches[0].buf))
     two = s.fork([1])
@@ -235,12 +235,12 @@ def test_kernels_validate_before_any_cuda_call():
     assert L.eb_gemm_grouped(a, 8, a, 8, a, 8, 64, 16, 8, 1, a, a, 0, 0.0, 0.0, B16, None) == -1 and "whole tiles" in _lib.last_error()
     assert L.eb_gemm_grouped(a, 8, a, 8, a, 8, 128, 24, 8, 1, a, a, 1, 1.0, 1.0, B16, None) == -1
     assert L.eb_grouped_skinny(a, 8, 0, 1, a, 8, 8, a, 8, 0, None, 1, 1, 8, 12, 0, 0.0, 0.0, B16, None) == -1
-    assert L.eb_gemm_f32(a, 4, 0, a, 8, 0, a, 8, 0, 1, 8, 8, 1, None, None, None) == -1
+    assert L.eb_gemm_f32(a, 4, 0, a, 8, 0, a, 8, 0, 1, 8, 8, 1, None, None, None, 0, None, None) == -1
     latent = lambda rank=64, dtype=B16, nsplit=1: L.eb_latent_decode(a, 64, a, 640, 64, 10, a, 64, 1, 1, rank, 4, a, None, 1.0, dtype, nsplit,
                                                                      None, 0, None)
     assert latent(rank=96) == -1 and "latent width" in _lib.last_error()
     assert latent(dtype=F32) == -1 and latent(nsplit=3) == -1 and "scratch" in _lib.last_error()
     assert L.eb_latent_decode_scratch_bytes(2, 3, 64, 4) == 0 and L.eb_latent_decode_scratch_bytes(2, 3, 64, 3) == 2 * 3 * 3 * 66 * 4
-    assert L.eb_attention_plain(a, a, a, None, *[8] * 12, 1, 1, 1, 8, 8, 0, 4, None, None, 1.0, F32, None) == -1
+    assert L.eb_attention_plain(a, a, a, None, *[8] * 12, 1, 1, 1, 1, 8, 8, 0, 4, None, None, None, None, 0, 1.0, F32, None) == -1
     args = [a, a, a, a, None, 64, 64, 64, 64, 64, 64, 64, 64, 0, 1, 1, 8, 8, 64]
     assert L.eb_attention_prefill_window_tc(*args, -1, 0.1, B16, None) == -1 and "window" in _lib.last_error()
