@@ -5,7 +5,7 @@ import torch
 
 from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
 
-_scratch = {}
+_scratch, _outgrown = {}, []
 TC_MIN_ROWS = 128        # below this many query rows the 256-row CTAs of the tensor-core kernel are mostly padding
 
 
@@ -13,6 +13,8 @@ def _get_scratch(device, nbytes):
     key = torch.device(device).index
     buf = _scratch.get(key)
     if buf is None or buf.numel() < nbytes:
+        if buf is not None:
+            _outgrown.append(buf)            # captured steps may still hold its address
         buf = torch.zeros(max(nbytes, 1 << 20), dtype=torch.uint8, device=device)
         _scratch[key] = buf
     return buf
@@ -199,3 +201,62 @@ def attention_inputs(proj, heads, kv_heads, dk, dv, q_norm, q_count, k_norm, k_c
                                     k_cache.stride(1), ptr(v_cache), v_cache.stride(0), v_cache.stride(1), k_cache.shape[1], n1, rows_per_batch,
                                     ptr(pos_device), ptr(first), dtype_code(proj.dtype), stream_ptr()), "attention_inputs")
     return q
+
+
+def distance_bias(r1, r2, distances):
+    """Table [heads, >= distances] of r1 * log2(1 + r2 * d) for attention_prefill_biased."""
+    require_cuda(r1, r2)
+    n = distances + 256                              # (rows behind the end of a sequence read on)
+    table = torch.empty((r1.numel(), n), dtype=torch.float32, device=r1.device)
+    check(lib().eb_distance_bias(ptr(r1), ptr(r2), r1.numel(), n, ptr(table), stream_ptr()), "distance_bias")
+    return table
+
+
+def attention_prefill_biased(q, k, v, head_dim, bias_table, sink=True, window=0, mask=None, scale=None, out=None):
+    """attention_prefill_window for q [B, Sq, H*D] and k / v [B, Sk, G*D] (G heads, each shared by H/G
+    query heads); the distance bias of bias_table (distance_bias()) is taken off the scores; sink: one is
+    added to the softmax denominator."""
+    require_cuda(q, k, v, mask, out, bias_table)
+    B, Sq, HD = q.shape
+    Sk, H, G = k.shape[1], HD // head_dim, k.shape[2] // head_dim
+    if out is None:
+        out = torch.empty((B, Sq, HD), dtype=q.dtype, device=q.device)
+    if mask is not None and (mask.dtype != q.dtype or mask.stride(-1) != 1 or mask.dim() != 2 or mask.shape[1] < Sk):
+        raise RuntimeError("attention: mask must be [batch, kv_len] of the tensor dtype")
+    if bias_table.dtype != torch.float32 or bias_table.dim() != 2 or not bias_table.is_contiguous() or bias_table.shape[0] != H or H % G:
+        raise RuntimeError("attention: a bias table with one row per query head, query heads in equal groups")
+    qs, ks, vs, os_ = (_bsh_strides(t, head_dim) for t in (q, k, v, out))
+    scale = head_dim ** -0.5 if scale is None else scale
+    check(lib().eb_attention_prefill_biased_tc(ptr(q), ptr(k), ptr(v), ptr(out), ptr(mask), qs[0], qs[1], ks[0], ks[1], vs[0], vs[1],
+                                               os_[0], os_[1], mask.stride(0) if mask is not None else 0, B, H, H // G, Sq, Sk, head_dim,
+                                               int(window), ptr(bias_table), bias_table.shape[1], 1 if sink else 0, float(scale),
+                                               dtype_code(q.dtype), stream_ptr()), "attention_prefill_biased_tc")
+    return out
+
+
+def pick_group_nsplit(batch, units, keys, sm_count=148):
+    """Key splits per (sequence, group of heads): what gives every SM two CTAs, at least 256 keys each."""
+    want = -(-2 * sm_count // max(1, batch * units))
+    return max(1, min(want, keys // 256, 64))
+
+
+def attention_group_decode(q, k, v, head_dim, pos_device, scale, first=None, bias=None, sink=True, nsplit=None):
+    """Generation step: q [B, H*D], k / v [B, rows, G*D] cache views, pos_device int32 scalar (the query's
+    position).  bias = (r1, r2) fp32 per query head.  Returns [B, H*D]."""
+    r1, r2 = bias if bias is not None else (None, None)
+    require_cuda(q, k, v, pos_device, first, r1, r2)
+    B, HD = q.shape
+    H, G, rows = HD // head_dim, k.shape[2] // head_dim, k.shape[1]
+    if bias is not None and any(r.dtype != torch.float32 or r.numel() != H or not r.is_contiguous() for r in bias):
+        raise RuntimeError("attention: the distance bias has two fp32 numbers per query head")
+    ks, vs = _bsh_strides(k, head_dim), _bsh_strides(v, head_dim)
+    out = torch.empty((B, HD), dtype=q.dtype, device=q.device)
+    if nsplit is None:
+        nsplit = pick_group_nsplit(B, G * -(-(H // G) // 16), rows)
+    nbytes = lib().eb_attention_group_decode_scratch_bytes(B, H, G, head_dim, nsplit)
+    scratch = _get_scratch(q.device, nbytes) if nbytes else None
+    check(lib().eb_attention_group_decode(ptr(q), ptr(k), ptr(v), ptr(out), q.stride(0), ks[0], ks[1], vs[0], vs[1], out.stride(0), B, H, G,
+                                          head_dim, rows, ptr(pos_device), ptr(first), ptr(r1), ptr(r2), 1 if sink else 0, float(scale),
+                                          dtype_code(q.dtype), nsplit, ptr(scratch), scratch.numel() if scratch is not None else 0,
+                                          stream_ptr()), "attention_group_decode")
+    return out

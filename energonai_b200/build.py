@@ -21,7 +21,7 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "-diag-suppress", "177,550"]
 # Recurrences add up the logarithms of their gates over a whole sequence: an approximation's bias would
 # add up with them, so these files get the accurate functions.
-ACCURATE = {"matrix_memory.cu"}
+ACCURATE = {"matrix_memory.cu", "matrix_memory_tc.cu"}
 
 
 def nvcc_flags(source):

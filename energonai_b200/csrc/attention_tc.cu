@@ -23,22 +23,25 @@
 // sum is fp32).  The two row tiles alternate on the tensor core: while the softmax warps of one
 // work on their scores, it serves the other.
 //
+// Query heads may share a key / value head in groups.  A biased form takes r1 ln(1 + r2 distance) off
+// every score, read from a table per head (a row's 32 scores of a chunk are 32 consecutive entries, the
+// lanes of a warp one entry apart: loads that coalesce, where a logarithm per score would double the
+// work of the special-function unit), and may add one to the softmax denominator (a sink of score 0).
+//
 // A sliding window (row i sees only the `window` keys up to its own position) shortens the range of
 // key tiles a row tile walks and hides the leading keys of its first tiles; nothing else changes.
 //
 // Every mbarrier wait is bounded; a wait that runs out is recorded, the CTA's roles leave (each
 // decision made uniform over the warp first), copies in flight are given time to land, TMEM is
 // freed and the kernel returns.
-#include <cuda.h>
-
 #include <type_traits>
 
-#include "common.cuh"
+#include "tc_ops.cuh"
 
 namespace eb {
 namespace {
 
-constexpr int kRows = 128;                 // query rows per row tile = UMMA M = TMEM lanes
+// (kRows of tc_ops.cuh: query rows per row tile)
 constexpr int kTiles = 2;                  // row tiles per CTA, each with its own four softmax warps
 constexpr int kKeys = 128;                 // keys per tile
 constexpr int kTcThreads = 64 + kTiles * 128;
@@ -52,13 +55,14 @@ template <int D> struct TcSmem {
 };
 constexpr float kLog2eTc = 1.4426950408889634f;
 constexpr float kRescaleLog2 = 8.f;         // the accumulated row is rescaled when its maximum grows by more than 2^8
-constexpr unsigned long long kTcWaitNs = 1000ull * 1000ull * 1000ull;
-
-__device__ int g_tc_status[4];             // [0] code, [1] where, [2] block, [3] detail
 
 struct TcParams {
   int B, H, Sq, Sk, causal;
   int window;                              // > 0: row i sees keys j with i - j < window only (causal)
+  int group;                               // query heads per key / value head
+  const float *bias;                       // biased form: [H][bias_ld], r1 * log2(1 + r2 * distance)
+  long long bias_ld;
+  int sink;
   int mask_vec;                            // mask rows start on 16-byte boundaries
   float scale_log2;                        // scale * log2(e)
   const void *mask;                        // additive [B][>= Sk] in T, or null
@@ -67,130 +71,11 @@ struct TcParams {
   long long o_bs, o_rs;
 };
 
-// ---- PTX wrappers (the same forms the GEMM uses) ----------------------------------------------
-__device__ __forceinline__ uint32_t s32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ unsigned long long gtimer() {
-  unsigned long long t;
-  asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
-  return t;
-}
-__device__ __forceinline__ void bar_init(uint32_t bar, uint32_t count) {
-  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count) : "memory");
-}
-__device__ __forceinline__ void bar_expect_tx(uint32_t bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void bar_arrive(uint32_t bar) {
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ bool bar_try(uint32_t bar, uint32_t parity) {
-  uint32_t ok;
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "mbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
-      "selp.u32 %0, 1, 0, p;\n\t}"
-      : "=r"(ok)
-      : "r"(bar), "r"(parity)
-      : "memory");
-  return ok != 0;
-}
-__device__ __noinline__ bool bar_wait_slow(uint32_t bar, uint32_t parity, volatile int *abort_flag, int where) {
-  const unsigned long long t0 = gtimer();
-  for (unsigned it = 1;; ++it) {
-    if (bar_try(bar, parity)) return true;
-    if ((it & 63u) == 0) {
-      if (*abort_flag) return false;
-      if (gtimer() - t0 > kTcWaitNs) {
-        *abort_flag = 1;
-        if (atomicCAS(&g_tc_status[0], 0, EB_ETIMEDOUT) == 0) {
-          g_tc_status[1] = where;
-          g_tc_status[2] = blockIdx.x;
-          g_tc_status[3] = (int)parity;
-        }
-        return false;
-      }
-    }
-  }
-}
-__device__ __forceinline__ bool bar_wait(uint32_t bar, uint32_t parity, volatile int *abort_flag, int where) {
-  if (bar_try(bar, parity)) return true;
-  return bar_wait_slow(bar, parity, abort_flag, where);
-}
-__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap *map, uint32_t bar, int x, int y, int z) {
-  asm volatile(
-      "cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-      ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar)
-      : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_commit(uint32_t bar) {
-  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void tc_mma(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-  asm volatile(
-      "{\n\t.reg .pred p;\n\t"
-      "setp.ne.b32 p, %4, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-      ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-__device__ __forceinline__ void tc_ld32(uint32_t taddr, float *v) {
-  uint32_t r[32];
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,"
-      "%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]),
-        "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]),
-        "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-      : "r"(taddr));
-  asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-  for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-}
-__device__ __forceinline__ void tc_st32(uint32_t taddr, const float *v) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,"
-      "%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};"
-      ::"r"(taddr), "r"(__float_as_uint(v[0])), "r"(__float_as_uint(v[1])), "r"(__float_as_uint(v[2])), "r"(__float_as_uint(v[3])),
-        "r"(__float_as_uint(v[4])), "r"(__float_as_uint(v[5])), "r"(__float_as_uint(v[6])), "r"(__float_as_uint(v[7])),
-        "r"(__float_as_uint(v[8])), "r"(__float_as_uint(v[9])), "r"(__float_as_uint(v[10])), "r"(__float_as_uint(v[11])),
-        "r"(__float_as_uint(v[12])), "r"(__float_as_uint(v[13])), "r"(__float_as_uint(v[14])), "r"(__float_as_uint(v[15])),
-        "r"(__float_as_uint(v[16])), "r"(__float_as_uint(v[17])), "r"(__float_as_uint(v[18])), "r"(__float_as_uint(v[19])),
-        "r"(__float_as_uint(v[20])), "r"(__float_as_uint(v[21])), "r"(__float_as_uint(v[22])), "r"(__float_as_uint(v[23])),
-        "r"(__float_as_uint(v[24])), "r"(__float_as_uint(v[25])), "r"(__float_as_uint(v[26])), "r"(__float_as_uint(v[27])),
-        "r"(__float_as_uint(v[28])), "r"(__float_as_uint(v[29])), "r"(__float_as_uint(v[30])), "r"(__float_as_uint(v[31]))
-      : "memory");
-}
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ void tc_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-// K-major tile of 128-byte rows with the 128-byte swizzle; 8-row groups 1024 bytes apart.
-__device__ __forceinline__ uint64_t tc_desc(uint32_t addr) {
-  return (uint64_t)((addr & 0x3FFFFu) >> 4) | ((uint64_t)1 << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) |
-         ((uint64_t)2 << 61);
-}
-// N-major B operand (the contraction index runs down the rows of the tile): 64-column atoms of
-// 8 rows x 128 bytes, swizzled; atoms along N lie atom_stride bytes apart (leading offset), 8-row
-// groups along K 1024 bytes apart.
-__device__ __forceinline__ uint64_t tc_desc_nmajor(uint32_t addr, uint32_t atom_stride) {
-  return (uint64_t)((addr & 0x3FFFFu) >> 4) | ((uint64_t)(atom_stride >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) |
-         ((uint64_t)2 << 61);
-}
-// kind::f16, fp32 accumulate, both operands K-major, M = 128.
-__host__ __device__ constexpr uint32_t tc_idesc(int n, int is_bf16) {
-  return (1u << 4) | ((uint32_t)is_bf16 << 7) | ((uint32_t)is_bf16 << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(kRows >> 4) << 24);
-}
-
 // ---- the attention kernel ----------------------------------------------------------------------
 // Shared memory (1024-aligned): [1 KB barriers, TMEM slot, abort flag][Q: 2 row tiles x D/64
 // sub-tiles of 128 rows x 128 B][K ring: 2 x D/64 sub-tiles][V ring: kVStages x D/64 sub-tiles
 // of 128 key rows x 128 B][P: 2 row tiles x 2 sub-tiles of 128 rows x 128 B].
-template <typename T, int D>
+template <typename T, int D, bool BIAS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                             const __grid_constant__ CUtensorMap tm_v, const TcParams p) {
@@ -217,7 +102,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   uint8_t *p_ptr = smem + 1024 + kTiles * kQBytes + 2 * kKBytes + kVStages * kVBytes;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int qb = gridDim.x - 1 - blockIdx.x, h = blockIdx.y, b = blockIdx.z;   // longest (latest, under the causal mask) blocks first
+  const int qb = gridDim.x - 1 - blockIdx.x, h = blockIdx.y, hk = h / p.group, b = blockIdx.z;   // longest (latest, under the causal mask) blocks first
   const int q0 = qb * (kTiles * kRows), shift = p.Sk - p.Sq;
   // key tiles each row tile walks: all of them, or up to its last row's diagonal; none for a
   // row tile that lies wholly behind the end of the sequence
@@ -281,7 +166,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         bar_expect_tx(k_full + 8 * st, kKBytes);
 #pragma unroll
         for (int kb = 0; kb < kSub; ++kb)
-          tma_load_3d(k_addr + st * kKBytes + kb * kKeys * 128, &tm_k, k_full + 8 * st, h * D + kb * 64, j * kKeys, b);
+          tma_load_3d(k_addr + st * kKBytes + kb * kKeys * 128, &tm_k, k_full + 8 * st, hk * D + kb * 64, j * kKeys, b);
         return true;
       };
       bool ok = load_k(jmin);
@@ -292,7 +177,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         bar_expect_tx(v_full + 8 * vs, kVBytes);
 #pragma unroll
         for (int kb = 0; kb < kSub; ++kb)
-          tma_load_3d(v_addr + vs * kVBytes + kb * kKeys * 128, &tm_v, v_full + 8 * vs, h * D + kb * 64, j * kKeys, b);
+          tma_load_3d(v_addr + vs * kVBytes + kb * kKeys * 128, &tm_v, v_full + 8 * vs, hk * D + kb * 64, j * kKeys, b);
       }
     }
   } else if (warp == 1) {
@@ -356,7 +241,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     const T *mrow = p.mask ? reinterpret_cast<const T *>(p.mask) + (long long)b * p.mask_bs : nullptr;
     const int vis_end = p.causal ? min(p.Sk, qi + shift + 1) : p.Sk;               // keys [0, vis_end) are visible to this row
     const int vis_begin = p.window > 0 ? qi + shift - p.window + 1 : 0;            // ... from this key on
-    float m_ref = -1e30f, l_run = 0.f;      // m_ref: the maximum the accumulated row and l_run are scaled by
+    // m_ref: the maximum the accumulated row and l_run are scaled by (a sink is a score of 0 seen already)
+    float m_ref = BIAS && p.sink ? 0.f : -1e30f, l_run = BIAS && p.sink ? 1.f : 0.f;
+    // A bias that only lowers scores need not enter the maximum: any reference that is not below the
+    // largest score will do as long as the probabilities keep their precision, which bf16 does over its
+    // whole range.  fp16 does not, and a negative r1 raises scores: there the maximum includes it.
+    const float *bias = BIAS ? p.bias + (long long)h * p.bias_ld : nullptr;
+    const bool bias_in_max = BIAS && (!kBf16 || bias[1] < 0.f);
     bool alive = ntiles > 0;
     for (int j = first_tile; j < ntiles && alive; ++j) {
       const int key0 = j * kKeys;
@@ -387,7 +278,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         if (cls[c] == 0) continue;
         float x[32];
         tc_ld32(t_s + c * 32, x);
-        if (cls[c] == 1) {
+        const int gap = qi + shift - (key0 + c * 32);                 // distance to the chunk's first key
+        if (cls[c] == 1 && bias_in_max) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) m_tile = fmaxf(m_tile, fmaf(x[e], p.scale_log2, -__ldg(bias + gap - e)));
+        } else if (cls[c] == 1) {
 #pragma unroll
           for (int e = 0; e < 32; e += 4) {
             r0 = fmaxf(r0, x[e]);
@@ -399,7 +294,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           const int nvis = vis_end - (key0 + c * 32), n0 = vis_begin - (key0 + c * 32);
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
-            const float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
+            float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
+            if (bias_in_max) v -= __ldg(bias + max(0, gap - e));
             m_tile = fmaxf(m_tile, e < nvis && e >= n0 ? v : -INFINITY);
           }
         }
@@ -441,16 +337,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           for (int g = 0; g < 4; ++g) *reinterpret_cast<uint4 *>(dst + ((((c & 1) * 4 + g) ^ (row & 7)) << 4)) = make_uint4(0, 0, 0, 0);
           continue;
         }
-        float x[32];
+        const int gap = qi + shift - (key0 + c * 32);
+        float x[32], bt[BIAS ? 32 : 1];
+        if (BIAS && cls[c] == 1) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) bt[BIAS ? e : 0] = __ldg(bias + gap - e);
+        }
         tc_ld32(t_s + c * 32, x);
         if (cls[c] == 1) {
 #pragma unroll
-          for (int e = 0; e < 32; ++e) x[e] = ex2(fmaf(x[e], p.scale_log2, neg_m));
+          for (int e = 0; e < 32; ++e) x[e] = ex2(fmaf(x[e], p.scale_log2, BIAS ? neg_m - bt[BIAS ? e : 0] : neg_m));
         } else {
           const int nvis = vis_end - (key0 + c * 32), n0 = vis_begin - (key0 + c * 32);
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
-            const float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
+            float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
+            if (BIAS) v -= __ldg(bias + max(0, gap - e));
             x[e] = e < nvis && e >= n0 ? ex2(v + neg_m) : 0.f;
           }
         }
@@ -517,42 +419,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
 }
 
 // ---- host side ---------------------------------------------------------------------------------
-typedef CUresult (*EncodeFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *,
-                             const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave, CUtensorMapSwizzle,
-                             CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeFn tc_encode_fn() {
-  static EncodeFn fn = nullptr;
-  if (!fn) {
-    void *sym = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &q) == cudaSuccess && q == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<EncodeFn>(sym);
-  }
-  return fn;
+// out[h][d] = r1[h] * log2(1 + r2[h] * d)
+__global__ void distance_bias_kernel(const float *r1, const float *r2, int len, float *out) {
+  griddep_wait();
+  griddep_launch();
+  const int d = blockIdx.x * blockDim.x + threadIdx.x, h = blockIdx.y;
+  if (d < len) out[(long long)h * len + d] = r1[h] * log2f(fmaf(r2[h], (float)d, 1.f));
 }
 
-// 3-D map over [batch][rows][cols] (cols contiguous), box 64 x box_rows x 1, 128-byte swizzle,
-// out-of-bounds elements read as zero.  Strides in elements.
-int tc_map3(CUtensorMap *map, const void *base, int dtype, long long cols, long long rows, long long batch, long long row_stride,
-            long long batch_stride, int box_rows) {
-  EncodeFn fn = tc_encode_fn();
-  if (!fn) return fail(EB_ECUDA, "attention_prefill: cuTensorMapEncodeTiled is not available from the driver");
-  cuuint64_t dims[3] = {(cuuint64_t)cols, (cuuint64_t)rows, (cuuint64_t)batch};
-  cuuint64_t strides[2] = {(cuuint64_t)row_stride * 2, (cuuint64_t)batch_stride * 2};
-  cuuint32_t box[3] = {64, (cuuint32_t)box_rows, 1};
-  cuuint32_t estr[3] = {1, 1, 1};
-  CUresult r = fn(map, dtype == EB_BF16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, const_cast<void *>(base),
-                  dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
-                  CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-  if (r != CUDA_SUCCESS) return fail(EB_ECUDA, "attention_prefill: cuTensorMapEncodeTiled failed with CUresult %d", (int)r);
-  return EB_OK;
-}
-
-template <typename T, int D>
+template <typename T, int D, bool BIAS>
 int launch_tc(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const TcParams &p, cudaStream_t st) {
   constexpr size_t smem = TcSmem<D>::kTotal;
-  auto kern = attention_prefill_tc_kernel<T, D>;
+  auto kern = attention_prefill_tc_kernel<T, D, BIAS>;
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -571,19 +449,7 @@ int launch_tc(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &m
 }  // namespace
 
 // Status words of this file's kernels, for eb_device_status.
-int attention_tc_status(int *out4, bool clear) {
-  int host[4] = {0, 0, 0, 0};
-  if (cudaMemcpyFromSymbol(host, g_tc_status, sizeof(host)) != cudaSuccess) {
-    cudaGetLastError();
-    return EB_ECUDA;
-  }
-  for (int i = 0; i < 4; ++i) out4[i] = host[i];
-  if (clear && host[0] != 0) {
-    int zero[4] = {0, 0, 0, 0};
-    cudaMemcpyToSymbol(g_tc_status, zero, sizeof(zero));
-  }
-  return EB_OK;
-}
+int attention_tc_status(int *out4, bool clear) { return tc_status(out4, clear); }
 
 }  // namespace eb
 
@@ -594,7 +460,8 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
                                        long long k_row_stride, long long v_batch_stride, long long v_row_stride,
                                        long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
                                        int heads, int q_len, int kv_len, int head_dim, int causal, int window, float scale,
-                                       int dtype, void *stream) {
+                                       int dtype, void *stream, int kv_group = 1, const float *bias = nullptr, long long bias_ld = 0,
+                                       int sink = 0) {
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "attention_prefill: fp16 or bf16 only (dtype %d)", dtype);
   EB_REQUIRE(head_dim == 64 || head_dim == 128, "attention_prefill: head_dim %d not supported (64 or 128)", head_dim);
@@ -609,20 +476,23 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   EB_REQUIRE(scale > 0.f, "attention_prefill: the scale must be positive");
   EB_REQUIRE(window >= 0 && (window == 0 || causal), "attention_prefill: a window needs the causal mask");
   cudaStream_t st = as_stream(stream);
-  const long long hd = (long long)heads * head_dim;
+  const long long hd = (long long)heads * head_dim, hkd = hd / kv_group;
   CUtensorMap mq, mk, mv;
   int rc;
-  if ((rc = tc_map3(&mv, v, dtype, hd, kv_len, batch, v_row_stride, v_batch_stride, kKeys))) return rc;
+  if ((rc = tc_map3(&mv, v, dtype, hkd, kv_len, batch, v_row_stride, v_batch_stride, kKeys))) return rc;
   if ((rc = tc_map3(&mq, q, dtype, hd, q_len, batch, q_row_stride, q_batch_stride, kRows))) return rc;
-  if ((rc = tc_map3(&mk, k, dtype, hd, kv_len, batch, k_row_stride, k_batch_stride, kKeys))) return rc;
+  if ((rc = tc_map3(&mk, k, dtype, hkd, kv_len, batch, k_row_stride, k_batch_stride, kKeys))) return rc;
   TcParams p{};
   p.B = batch; p.H = heads; p.Sq = q_len; p.Sk = kv_len; p.causal = causal; p.window = window;
   p.scale_log2 = scale * kLog2eTc;
   p.mask = mask; p.mask_bs = mask_batch_stride;
   p.mask_vec = mask && aligned16(mask) && mask_batch_stride % 8 == 0;
   p.o = out; p.o_bs = o_batch_stride; p.o_rs = o_row_stride;
-  if (dtype == EB_F16) return head_dim == 64 ? launch_tc<__half, 64>(mq, mk, mv, p, st) : launch_tc<__half, 128>(mq, mk, mv, p, st);
-  return head_dim == 64 ? launch_tc<__nv_bfloat16, 64>(mq, mk, mv, p, st) : launch_tc<__nv_bfloat16, 128>(mq, mk, mv, p, st);
+  p.group = kv_group; p.bias = bias; p.bias_ld = bias_ld; p.sink = sink;
+#define EB_TC(T, D) (bias ? launch_tc<T, D, true>(mq, mk, mv, p, st) : launch_tc<T, D, false>(mq, mk, mv, p, st))
+  if (dtype == EB_F16) return head_dim == 64 ? EB_TC(__half, 64) : EB_TC(__half, 128);
+  return head_dim == 64 ? EB_TC(__nv_bfloat16, 64) : EB_TC(__nv_bfloat16, 128);
+#undef EB_TC
 }
 
 extern "C" int eb_attention_prefill_tc(const void *q, const void *k, const void *v, void *out, const void *mask,
@@ -645,4 +515,25 @@ extern "C" int eb_attention_prefill_window_tc(const void *q, const void *k, cons
   return prefill_tc_impl(q, k, v, out, mask, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
                          o_batch_stride, o_row_stride, mask_batch_stride, batch, heads, q_len, kv_len, head_dim, 1, window, scale, dtype,
                          stream);
+}
+
+extern "C" int eb_distance_bias(const float *r1, const float *r2, int heads, int len, float *table, void *stream) {
+  if (heads == 0 || len == 0) return EB_OK;
+  EB_REQUIRE(r1 && r2 && table && heads > 0 && heads <= 65535 && len > 0, "distance_bias: bad arguments");
+  launch_pdl(distance_bias_kernel, dim3((len + 255) / 256, heads), dim3(256), 0, as_stream(stream), r1, r2, len, table);
+  return check_launch("distance_bias");
+}
+
+extern "C" int eb_attention_prefill_biased_tc(const void *q, const void *k, const void *v, void *out, const void *mask,
+                                       long long q_batch_stride, long long q_row_stride, long long k_batch_stride,
+                                       long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                                       long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
+                                       int heads, int kv_group, int q_len, int kv_len, int head_dim, int window, const float *bias_table,
+                                       int bias_len, int sink, float scale, int dtype, void *stream) {
+  EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_prefill: %d heads do not share keys in groups of %d", heads, kv_group);
+  EB_REQUIRE(bias_table && bias_len >= kv_len + kTiles * kRows, "attention_prefill: the bias table needs %d distances, has %d",
+             kv_len + kTiles * kRows, bias_len);
+  return prefill_tc_impl(q, k, v, out, mask, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
+                         o_batch_stride, o_row_stride, mask_batch_stride, batch, heads, q_len, kv_len, head_dim, 1, window, scale, dtype,
+                         stream, kv_group, bias_table, bias_len, sink);
 }

@@ -1329,6 +1329,7 @@ extern "C" size_t eb_gemm_workspace_bytes(int M, int N, int K) {
 namespace eb {
 int attention_tc_status(int *out4, bool clear);   // attention_tc.cu
 int latent_status(int *out4, bool clear);         // latent_attention.cu
+int memory_tc_status(int *out4, bool clear);      // matrix_memory_tc.cu
 }
 
 extern "C" int eb_device_status(int *out4, int clear) {
@@ -1353,6 +1354,12 @@ extern "C" int eb_device_status(int *out4, int clear) {
   if (host[0] == 0 && lat[0] != 0) {
     for (int i = 0; i < 4; ++i) host[i] = lat[i];
     host[1] += 200;
+  }
+  int mem[4] = {0, 0, 0, 0};                       // matrix memory: 300+
+  if (eb::memory_tc_status(mem, clear != 0) != EB_OK) return fail(EB_ECUDA, "device_status: cannot read the status word");
+  if (host[0] == 0 && mem[0] != 0) {
+    for (int i = 0; i < 4; ++i) host[i] = mem[i];
+    host[1] += 300;
   }
   if (out4)
     for (int i = 0; i < 4; ++i) out4[i] = host[i];

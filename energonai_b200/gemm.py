@@ -5,7 +5,7 @@ from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda, ACT_NON
 
 ACT_CODES = {None: ACT_NONE, "none": ACT_NONE, "relu": ACT_RELU, "gelu_tanh": ACT_GELU_TANH, "gelu": ACT_GELU_ERF}
 
-_workspaces = {}
+_workspaces, _outgrown = {}, []
 
 
 def workspace(device, nbytes):
@@ -14,6 +14,8 @@ def workspace(device, nbytes):
     key = torch.device(device).index
     ws = _workspaces.get(key)
     if ws is None or ws.numel() < nbytes:
+        if ws is not None:
+            _outgrown.append(ws)             # captured steps may still hold its address
         ws = torch.zeros(max(nbytes, 1 << 20), dtype=torch.uint8, device=device)
         _workspaces[key] = ws
     return ws

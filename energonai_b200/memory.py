@@ -25,8 +25,12 @@ def _gates(gates, bias, heads, rows):
         raise RuntimeError("matrix memory: one fp32 bias per head and gate")
 
 
-def memory_scan(q, k, v, gates, bias, cap, scale, state, heads, first=None):
-    """A prompt through the recurrence, token by token: q, k [batch*seq, heads*dk], v [batch*seq,
+MEMORY_KEY_HEADS = (64, 128)      # key head sizes of the chunked tensor-core kernel
+
+
+def memory_prompt(q, k, v, gates, bias, cap, scale, state, heads, first=None, chunked=False):
+    """A prompt through the recurrence, token by token on the CUDA cores, or (chunked: bf16, key heads
+    of MEMORY_KEY_HEADS) 128 tokens at a time on the tensor cores: q, k [batch*seq, heads*dk], v [batch*seq,
     heads*dv] (column views of one projection), gates fp32 [batch*seq, >= 2*heads] (input gates, forget
     gates), bias (input, forget) fp32 [heads].  state = (S, n, m) is overwritten with the state behind
     the last token; first [batch] int32: padding rows in front.  Returns [batch*seq, heads*dv]."""
@@ -37,9 +41,9 @@ def memory_scan(q, k, v, gates, bias, cap, scale, state, heads, first=None):
     if T % B:
         raise RuntimeError("matrix memory: whole sequences required")
     o = torch.empty((T, heads * dv), dtype=q.dtype, device=q.device)
-    check(lib().eb_memory_scan(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(gates), gates.stride(0), ptr(bias[0]), ptr(bias[1]), float(cap),
-                               float(scale), ptr(first), ptr(o), o.stride(0), *(ptr(t) for t in state), B, T // B, heads, dk, dv,
-                               dtype_code(q.dtype), stream_ptr()), "memory_scan")
+    run, name = (lib().eb_memory_chunks, "memory_chunks") if chunked else (lib().eb_memory_scan, "memory_scan")
+    check(run(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(gates), gates.stride(0), ptr(bias[0]), ptr(bias[1]), float(cap), float(scale),
+              ptr(first), ptr(o), o.stride(0), *(ptr(t) for t in state), B, T // B, heads, dk, dv, dtype_code(q.dtype), stream_ptr()), name)
     return o
 
 

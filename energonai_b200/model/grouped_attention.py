@@ -8,7 +8,7 @@ the padding."""
 import torch
 from torch import nn
 
-from ..attention import attention_inputs, attention_plain
+from ..attention import (attention_group_decode, attention_inputs, attention_plain, attention_prefill_biased, distance_bias)
 from ..gemm import project
 from ..nn import init_weight
 from .sequence_state import RingCache, round_up
@@ -66,6 +66,12 @@ class GroupedAttention(nn.Module):
         q = attention_inputs(proj, H, G, self.dk, self.dv, self.q_norm, H * self.dim, self.k_norm, G * self.dim, self.eps, k, v, S,
                              temp=self.temp, vmix=self.vmix if mix else None, v_first=self._keys_values(ctx, self.v_from)[1] if mix else None,
                              pos_device=ctx.pos, first=ctx.first).view(B, S, -1)
-        o = attention_plain(q, k, v, H, self.dk, self.dv, scale=self.scale, first=ctx.first, pos_device=ctx.pos, kv_heads=G,
-                            bias=(self.r1, self.r2), sink=True)
+        bias = (self.r1, self.r2)
+        if not self.tensor_core:
+            o = attention_plain(q, k, v, H, self.dk, self.dv, scale=self.scale, first=ctx.first, pos_device=ctx.pos, kv_heads=G, bias=bias,
+                                sink=True)
+        elif ctx.is_prompt:
+            o = attention_prefill_biased(q, k[:, :S], v[:, :S], self.dk, distance_bias(*bias, S), mask=ctx.mask, scale=self.scale)
+        else:
+            o = attention_group_decode(q.view(B, -1), k, v, self.dk, ctx.pos, self.scale, first=ctx.first, bias=bias)
         return project(o.view(B * S, -1), self.out_proj), proj[:, proj.shape[1] - self.width:]

@@ -8,7 +8,7 @@ import torch
 from torch import nn
 
 from ..gemm import project
-from ..memory import head_norm_gate, memory_scan, memory_step
+from ..memory import MEMORY_KEY_HEADS, head_norm_gate, memory_prompt, memory_step
 from ..nn import init_weight
 from .sequence_state import RecurrentState, round_up
 
@@ -19,7 +19,9 @@ class MatrixMemory(nn.Module):
         kw = dict(dtype=dtype, device=device)
         self.layer, self.width, self.heads, self.dim, self.vdim, self.cap, self.eps = layer, width, heads, dim, vdim, gate_cap, eps
         self.scale = dim ** -0.5
-        self.dk, self.dv = round_up(dim, 8), round_up(vdim, 8)
+        self.chunked = dtype == torch.bfloat16 and dim <= MEMORY_KEY_HEADS[-1]      # prompts on the tensor cores
+        self.dk = min(n for n in MEMORY_KEY_HEADS if n >= dim) if self.chunked else round_up(dim, 8)
+        self.dv = round_up(vdim, 8)
         qk, vg = heads * self.dk, heads * self.dv
         self.splits = [qk, qk, vg, vg, width]
         self.in_proj = init_weight(sum(self.splits), width, **kw)               # q | k | v | output gate | residual gate
@@ -44,7 +46,7 @@ class MatrixMemory(nn.Module):
             gates = project(h, self.gates, out_dtype=torch.float32)
         bias = self.gate_bias.unbind(0)
         if ctx.is_prompt:
-            o = memory_scan(q, k, v, gates, bias, self.cap, self.scale, state, self.heads, first=ctx.first)
+            o = memory_prompt(q, k, v, gates, bias, self.cap, self.scale, state, self.heads, first=ctx.first, chunked=self.chunked)
             y = head_norm_gate(o, g, self.norm, self.heads, self.vdim, self.eps)
         else:
             y = memory_step(q, k, v, g, gates, bias, self.cap, self.scale, self.norm, self.vdim, self.eps, state, self.heads)

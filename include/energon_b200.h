@@ -463,6 +463,14 @@ EB_API int eb_memory_scan(const void *q, const void *k, const void *v, long long
                    long long ldo, float *S, float *n, float *m, int batch, int seq, int heads, int dk, int dv, int dtype,
                    void *stream);
 
+/* eb_memory_scan on the tensor cores, 128 tokens at a time: bf16, dk 64 or 128 (heads zero-padded to it).
+ * State and gates are fp32; what enters or leaves the state as an operand is split into two bf16
+ * parts, a weighted score is rounded to one.  Waits are bounded ("where" codes 300 and up). */
+EB_API int eb_memory_chunks(const void *q, const void *k, const void *v, long long ldp, const float *gates, long long ldg,
+                     const float *bias_i, const float *bias_f, float cap, float scale, const int32_t *first, void *o,
+                     long long ldo, float *S, float *n, float *m, int batch, int seq, int heads, int dk, int dv, int dtype,
+                     void *stream);
+
 /* One token per sequence: the state goes on by one step, and
  *   out[h] = unit(o_h) * norm * sigmoid(g), unit(o) = o / sqrt(mean over dv_count of o^2 + eps). */
 EB_API int eb_memory_step(const void *q, const void *k, const void *v, const void *g, long long ldp, const float *gates,
@@ -533,6 +541,33 @@ EB_API int eb_attention_prefill_window_tc(const void *q, const void *k, const vo
                             long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
                             int heads, int q_len, int kv_len, int head_dim, int window, float scale, int dtype,
                             void *stream);
+
+/* table[h][d] = r1[h] log2(1 + r2[h] d), d < len: the distance bias of eb_attention_prefill_biased_tc. */
+EB_API int eb_distance_bias(const float *r1, const float *r2, int heads, int len, float *table, void *stream);
+
+/* eb_attention_prefill_window_tc in which kv_group query heads share a key / value head (k and v have
+ * heads / kv_group heads), bias_table[h][i - j] * ln 2 is taken off the scaled score, and sink != 0 adds
+ * one to the softmax denominator.  bias_table: fp32 [heads][bias_len] from eb_distance_bias, at
+ * least kv_len + 256 distances. */
+EB_API int eb_attention_prefill_biased_tc(const void *q, const void *k, const void *v, void *out, const void *mask,
+                            long long q_batch_stride, long long q_row_stride, long long k_batch_stride,
+                            long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                            long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
+                            int heads, int kv_group, int q_len, int kv_len, int head_dim, int window, const float *bias_table,
+                            int bias_len, int sink, float scale, int dtype, void *stream);
+
+/* Generation step for query heads in groups that share a key / value head: q [batch][heads*head_dim], one
+ * row per sequence at position pos (device scalar); k / v rows first[b] .. pos of the cache,
+ *   s_j = scale q.k_j - r1[h] ln(1 + r2[h] (pos - j));   out = sum_j exp(s_j) v_j / ([sink] + sum_j exp(s_j)).
+ * The keys and values of a group are read once for all its heads.  nsplit > 1 splits the positions over
+ * that many CTAs; the last to arrive merges them through `scratch`
+ * (eb_attention_group_decode_scratch_bytes, zero-filled once; calls sharing it must not overlap). */
+EB_API int eb_attention_group_decode(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+                              long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                              long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int cache_rows,
+                              const int32_t *pos_device, const int32_t *first, const float *bias_r1, const float *bias_r2,
+                              int sink, float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes, void *stream);
+EB_API size_t eb_attention_group_decode_scratch_bytes(int batch, int heads, int kv_heads, int head_dim, int nsplit);
 
 /* Windowed causal attention for any head sizes and fp32 / fp16 / bf16 on the CUDA cores: query row
  * i holds position pos0 + i (pos0 from pos_device, NULL: 0) and sees the positions
