@@ -235,9 +235,11 @@ def attention_prefill_biased(q, k, v, head_dim, bias_table, sink=True, window=0,
 
 
 def pick_group_nsplit(batch, units, keys, sm_count=148):
-    """Key splits per (sequence, group of heads): what gives every SM two CTAs, at least 256 keys each."""
-    want = -(-2 * sm_count // max(1, batch * units))
-    return max(1, min(want, keys // 256, 64))
+    """Key splits per (sequence, group of heads), of at least 256 keys each: enough for two CTAs per SM,
+    then what spreads the CTAs over the SMs most evenly, each further split counted as 4 % (its merge)."""
+    n, most = max(1, batch * units), max(1, min(keys // 256, 64))
+    least = min(most, -(-2 * sm_count // n))
+    return min(range(least, most + 1), key=lambda s: -(-n * s // sm_count) / (n * s) * (1 + 0.04 * s))
 
 
 def attention_group_decode(q, k, v, head_dim, pos_device, scale, first=None, bias=None, sink=True, nsplit=None):

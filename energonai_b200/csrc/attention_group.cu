@@ -27,10 +27,11 @@ struct GroupParams {
   int *counters;
 };
 
-template <typename T, int D>
+// WIDE: groups of more than 8 heads; else the second half of the tile's rows is not looked at.
+template <typename T, int D, bool WIDE>
 __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(const GroupParams p) {
   extern __shared__ __align__(128) uint8_t smem[];
-  constexpr int kTileBytes = kTile * D * 2, kLd = D + 2;
+  constexpr int kTileBytes = kTile * D * 2, kLd = D + 2, kHalves = WIDE ? 2 : 1;
   const uint32_t k_s = (uint32_t)__cvta_generic_to_shared(smem), v_s = k_s + kStages * kTileBytes;
   float *red = reinterpret_cast<float *>(smem);     // after the key loop: [4 warps][16][D + 2]
   __shared__ int s_last;
@@ -58,7 +59,7 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
     cp_async_commit();
   }
   uint32_t qf[D / 16][4];
-  const bool row_ok[2] = {g < nh, g + 8 < nh};
+  const bool row_ok[2] = {g < nh, WIDE && g + 8 < nh};
 #pragma unroll
   for (int kk = 0; kk < D / 16; ++kk)
 #pragma unroll
@@ -93,9 +94,9 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
       mma16816<T>(s[0], qf[kk], kf[0], kf[1]);
       mma16816<T>(s[1], qf[kk], kf[2], kf[3]);
     }
-    float corr[2];
+    float corr[2] = {1.f, 1.f};
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
+    for (int r = 0; r < kHalves; ++r) {
       float mx = -INFINITY;
 #pragma unroll
       for (int i = 0; i < 2; ++i)
@@ -124,9 +125,13 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
     }
     if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
 #pragma unroll
-      for (int i = 0; i < D / 8; ++i) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+      for (int i = 0; i < D / 8; ++i) {
+        o[i][0] *= corr[0]; o[i][1] *= corr[0];
+        if (WIDE) { o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+      }
     }
-    uint32_t pf[4] = {eb::pack2<T>(s[0][0], s[0][1]), eb::pack2<T>(s[0][2], s[0][3]), eb::pack2<T>(s[1][0], s[1][1]), eb::pack2<T>(s[1][2], s[1][3])};
+    const uint32_t pf[4] = {eb::pack2<T>(s[0][0], s[0][1]), WIDE ? eb::pack2<T>(s[0][2], s[0][3]) : 0u, eb::pack2<T>(s[1][0], s[1][1]),
+                            WIDE ? eb::pack2<T>(s[1][2], s[1][3]) : 0u};
 #pragma unroll
     for (int db = 0; db < D / 16; ++db) {
       uint32_t vf[4];
@@ -139,7 +144,7 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   cp_async_wait<0>();
   __syncthreads();                                  // all tiles are consumed: their memory takes the partial rows
 #pragma unroll
-  for (int r = 0; r < 2; ++r) {
+  for (int r = 0; r < kHalves; ++r) {
     float l = l_run[r];
     l += __shfl_xor_sync(0xffffffffu, l, 1);
     l += __shfl_xor_sync(0xffffffffu, l, 2);
@@ -207,9 +212,9 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   }
 }
 
-template <typename T, int D> int launch_group(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
+template <typename T, int D, bool WIDE> int launch_group_as(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
   constexpr size_t smem = 2 * kStages * (size_t)kTile * D * 2;
-  auto kern = attention_group_decode_kernel<T, D>;
+  auto kern = attention_group_decode_kernel<T, D, WIDE>;
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -222,6 +227,10 @@ template <typename T, int D> int launch_group(const GroupParams &p, int kv_heads
   }
   launch_pdl(kern, dim3(p.nsplit, kv_heads * p.blocks, B), dim3(kGroupThreads), smem, st, p);
   return check_launch("attention_group_decode");
+}
+
+template <typename T, int D> int launch_group(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
+  return p.group > 8 ? launch_group_as<T, D, true>(p, kv_heads, B, st) : launch_group_as<T, D, false>(p, kv_heads, B, st);
 }
 
 inline int head_blocks(int heads, int kv_heads) { return (heads / kv_heads + kRowsPerCta - 1) / kRowsPerCta; }

@@ -26,20 +26,22 @@ struct InputParams {
 };
 
 template <typename T> struct Pack8 {               // 8 elements of T
-  static __device__ __forceinline__ void load(const T *p, float (&f)[8]) {
-    constexpr int N = Vec16<T>::N;
+  static constexpr int N = Vec16<T>::N;
+  Vec16<T> part[8 / N];
+  __device__ __forceinline__ void load(const T *p) {
+#pragma unroll
+    for (int i = 0; i < 8 / N; ++i) part[i].load(p + i * N);
+  }
+  __device__ __forceinline__ void unpack(float (&f)[8]) const {
 #pragma unroll
     for (int i = 0; i < 8 / N; ++i) {
-      Vec16<T> a;
       float t[N];
-      a.load(p + i * N);
-      a.unpack(t);
+      part[i].unpack(t);
 #pragma unroll
       for (int e = 0; e < N; ++e) f[i * N + e] = t[e];
     }
   }
   static __device__ __forceinline__ void store(T *p, const float (&f)[8]) {
-    constexpr int N = Vec16<T>::N;
 #pragma unroll
     for (int i = 0; i < 8 / N; ++i) {
       Vec16<T> a;
@@ -52,69 +54,94 @@ template <typename T> struct Pack8 {               // 8 elements of T
   }
 };
 
-template <typename T, int THREADS>
+// PACKS packs of 8 columns per thread stay in registers, beside what each is multiplied by or mixed
+// with: everything a row needs is requested before the two sums are formed.
+template <typename T, int PACKS, int THREADS>
 __global__ void __launch_bounds__(THREADS) attention_inputs_kernel(const InputParams p) {
-  __shared__ float scratch[2][THREADS / 32];
+  __shared__ float2 scratch[THREADS / 32];
   griddep_wait();
   griddep_launch();
   const long long row = blockIdx.x;
   const long long b = row / p.rows_per_batch;
   const int col = (p.pos_dev ? *p.pos_dev : 0) + (int)(row - b * p.rows_per_batch);
   const T *x = reinterpret_cast<const T *>(p.proj) + row * p.ldp;
-  const int nq = p.nq / 8, nk = p.nk / 8, nv = p.nv / 8;
-  float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x; c < nq + nk; c += THREADS) {
-    float f[8];
-    Pack8<T>::load(x + c * 8, f);
-    float s = 0.f;
+  const int nq = p.nq / 8, nk = p.nk / 8, all = nq + nk + p.nv / 8;
+  const bool keep = col >= 0 && col < p.cache_rows;
+  const T *vf = p.vmix && keep ? reinterpret_cast<const T *>(p.vf) + b * p.vf_bs + (long long)col * p.vf_rs : nullptr;
+  Pack8<T> xv[PACKS], wv[PACKS];
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= all) break;
+    xv[i].load(x + c * 8);
+    if (c < nq) wv[i].load(reinterpret_cast<const T *>(p.wq) + c * 8);
+    else if (c < nq + nk) wv[i].load(reinterpret_cast<const T *>(p.wk) + (c - nq) * 8);
+    else if (vf) wv[i].load(vf + (c - nq - nk) * 8);
+  }
+  const float lambda = vf ? *p.vmix : 0.f;
+  const int first = p.first ? p.first[b] : 0;
+  float2 sq = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= nq + nk) break;
+    float f[8], s = 0.f;
+    xv[i].unpack(f);
 #pragma unroll
     for (int e = 0; e < 8; ++e) s = fmaf(f[e], f[e], s);
-    if (c < nq) sq += s; else sk += s;
+    if (c < nq) sq.x += s; else sq.y += s;
   }
-  sq = block_sum<THREADS>(sq, scratch[0]);
-  sk = block_sum<THREADS>(sk, scratch[1]);
-  float rq = rsqrtf(sq * p.inv_q + p.eps);
-  const float rk = rsqrtf(sk * p.inv_k + p.eps);
-  if (p.every > 0) {
-    const int pos = max(0, col - (p.first ? p.first[b] : 0));
-    rq *= 1.f + p.coef * logf((float)((pos + 1) / p.every + 1));
+  sq.x = warp_sum(sq.x);
+  sq.y = warp_sum(sq.y);
+  if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = sq;
+  __syncthreads();
+  sq = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < THREADS / 32; ++i) {
+    sq.x += scratch[i].x;
+    sq.y += scratch[i].y;
   }
-  const bool keep = col >= 0 && col < p.cache_rows;
+  float rq = rsqrtf(sq.x * p.inv_q + p.eps);
+  const float rk = rsqrtf(sq.y * p.inv_k + p.eps);
+  if (p.every > 0) rq *= 1.f + p.coef * logf((float)((max(0, col - first) + 1) / p.every + 1));
   T *q = reinterpret_cast<T *>(p.q) + row * p.ldq;
   T *k = reinterpret_cast<T *>(p.k) + b * p.k_bs + (long long)col * p.k_rs;
   T *v = reinterpret_cast<T *>(p.v) + b * p.v_bs + (long long)col * p.v_rs;
-  const T *vf = p.vmix ? reinterpret_cast<const T *>(p.vf) + b * p.vf_bs + (long long)col * p.vf_rs : nullptr;
-  const float lambda = p.vmix ? *p.vmix : 0.f;
-  for (int c = threadIdx.x; c < nq + nk + nv; c += THREADS) {
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= all) break;
     float f[8], w[8];
-    Pack8<T>::load(x + c * 8, f);
+    xv[i].unpack(f);
+    wv[i].unpack(w);
     if (c < nq) {
-      Pack8<T>::load(reinterpret_cast<const T *>(p.wq) + c * 8, w);
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] *= rq * w[e];
       Pack8<T>::store(q + c * 8, f);
     } else if (c < nq + nk) {
-      if (!keep) continue;
-      Pack8<T>::load(reinterpret_cast<const T *>(p.wk) + (c - nq) * 8, w);
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[e] *= rk * w[e];
-      Pack8<T>::store(k + (c - nq) * 8, f);
+      if (keep) Pack8<T>::store(k + (c - nq) * 8, f);
     } else {
-      if (!keep) continue;
-      const int o = (c - nq - nk) * 8;
       if (vf) {
-        Pack8<T>::load(vf + o, w);
 #pragma unroll
         for (int e = 0; e < 8; ++e) f[e] = fmaf(lambda, w[e], (1.f - lambda) * f[e]);
       }
-      Pack8<T>::store(v + o, f);
+      if (keep) Pack8<T>::store(v + (c - nq - nk) * 8, f);
     }
   }
 }
 
 template <typename T> int launch_inputs(const InputParams &p, int n1, cudaStream_t st) {
-  if (p.nq + p.nk + p.nv <= 2048) launch_pdl(attention_inputs_kernel<T, 128>, dim3(n1), dim3(128), 0, st, p);
-  else launch_pdl(attention_inputs_kernel<T, 256>, dim3(n1), dim3(256), 0, st, p);
+  const int packs = (p.nq + p.nk + p.nv) / 8;
+  const dim3 g(n1);
+  if (packs <= 128) launch_pdl(attention_inputs_kernel<T, 1, 128>, g, dim3(128), 0, st, p);
+  else if (packs <= 256) launch_pdl(attention_inputs_kernel<T, 1, 256>, g, dim3(256), 0, st, p);
+  else if (packs <= 512) launch_pdl(attention_inputs_kernel<T, 2, 256>, g, dim3(256), 0, st, p);
+  else if (packs <= 1024) launch_pdl(attention_inputs_kernel<T, 4, 256>, g, dim3(256), 0, st, p);
+  else if (packs <= 2048) launch_pdl(attention_inputs_kernel<T, 4, 512>, g, dim3(512), 0, st, p);
+  else if (packs <= 4096) launch_pdl(attention_inputs_kernel<T, 4, 1024>, g, dim3(1024), 0, st, p);
+  else return fail(EB_EUNSUPPORTED, "attention_inputs: %d columns are too many (32768)", packs * 8);
   return check_launch("attention_inputs");
 }
 

@@ -54,6 +54,9 @@ template <int D> struct TcSmem {
   static constexpr size_t kTotal = 1024 + 1024 + (size_t)kTiles * kQBytes + 2 * kKBytes + (size_t)kVStages * kVBytes + (size_t)kTiles * kPBytes;
 };
 constexpr float kLog2eTc = 1.4426950408889634f;
+// From this distance on r1 log2(1 + r2 d) is interpolated between d, d - 16 and d - 32: the third derivative
+// is at most 2 r1 / (ln 2 d^3), so the parabola is off by less than 1e-5 r1.
+constexpr int kFarKeys = 512;
 constexpr float kRescaleLog2 = 8.f;         // the accumulated row is rescaled when its maximum grows by more than 2^8
 
 struct TcParams {
@@ -257,8 +260,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       // multiply-add and one exponential per key, most chunks of a long prompt; 2 = per-key
       // work (the chunk the diagonal crosses, chunks with mask values).  Lane l keeps the mask
       // value of key l of each chunk, in the log2 domain.
+      // (The biased form keeps its chunk loops rolled: unrolled, its body outgrew the instruction cache,
+      // which was the largest stall.  So it packs the classes and reads mask values again.)
       int cls[kKeys / 32];
       float mval[kKeys / 32];
+      uint32_t classes = 0;
 #pragma unroll
       for (int c = 0; c < kKeys / 32; ++c) {
         const int kb = key0 + c * 32;
@@ -268,21 +274,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         const bool hidden = __all_sync(0xffffffffu, kb >= vis_end || kb + 32 <= vis_begin);
         const bool simple = __all_sync(0xffffffffu, kb >= vis_begin && kb + 32 <= vis_end && mv == 0.f);
         cls[c] = hidden ? 0 : (simple ? 1 : 2);
+        if (BIAS) classes |= (uint32_t)cls[c] << (2 * c);
       }
+      auto mask_value = [&](int c) { return mrow && key0 + c * 32 + lane < p.Sk ? to_f32<T>(mrow[key0 + c * 32 + lane]) * kLog2eTc : 0.f; };
       if (!__all_sync(0xffffffffu, bar_wait(my_s_full, (j - first_tile) & 1, abort_flag, 7))) { alive = false; break; }
       tc_fence_after();
       // pass 1: the row maximum of this tile (log2 domain, masks applied)
       float r0 = -INFINITY, r1 = -INFINITY, r2 = -INFINITY, r3 = -INFINITY, m_tile = -1e30f;
-#pragma unroll
-      for (int c = 0; c < kKeys / 32; ++c) {
-        if (cls[c] == 0) continue;
+      auto maximum = [&](int c, int kind, float mv) {
+        if (kind == 0) return;
         float x[32];
         tc_ld32(t_s + c * 32, x);
         const int gap = qi + shift - (key0 + c * 32);                 // distance to the chunk's first key
-        if (cls[c] == 1 && bias_in_max) {
+        if (kind == 1 && bias_in_max) {
 #pragma unroll
           for (int e = 0; e < 32; ++e) m_tile = fmaxf(m_tile, fmaf(x[e], p.scale_log2, -__ldg(bias + gap - e)));
-        } else if (cls[c] == 1) {
+        } else if (kind == 1) {
 #pragma unroll
           for (int e = 0; e < 32; e += 4) {
             r0 = fmaxf(r0, x[e]);
@@ -294,11 +301,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           const int nvis = vis_end - (key0 + c * 32), n0 = vis_begin - (key0 + c * 32);
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
-            float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
+            float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mv, e));
             if (bias_in_max) v -= __ldg(bias + max(0, gap - e));
             m_tile = fmaxf(m_tile, e < nvis && e >= n0 ? v : -INFINITY);
           }
         }
+      };
+      if constexpr (BIAS) {
+#pragma unroll 1
+        for (int c = 0; c < kKeys / 32; ++c) maximum(c, (classes >> (2 * c)) & 3, mask_value(c));
+      } else {
+#pragma unroll
+        for (int c = 0; c < kKeys / 32; ++c) maximum(c, cls[c], mval[c]);
       }
       r0 = fmaxf(fmaxf(r0, r1), fmaxf(r2, r3));
       if (r0 > -INFINITY) m_tile = fmaxf(m_tile, r0 * p.scale_log2);   // the scale is positive: the maximum commutes with it
@@ -329,29 +343,46 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       // pass 2: probabilities -> the 16-bit A operand of the second product (swizzled rows of 128 bytes)
       float l0 = 0.f, l1 = 0.f;
       const float neg_m = -m_ref;
-#pragma unroll
-      for (int c = 0; c < kKeys / 32; ++c) {
+      auto weights = [&](int c, int kind, float mv) {
         uint8_t *dst = p_row + (c >> 1) * (kRows * 128);
-        if (cls[c] == 0) {
+        if (kind == 0) {
 #pragma unroll
           for (int g = 0; g < 4; ++g) *reinterpret_cast<uint4 *>(dst + ((((c & 1) * 4 + g) ^ (row & 7)) << 4)) = make_uint4(0, 0, 0, 0);
-          continue;
+          return;
         }
-        const int gap = qi + shift - (key0 + c * 32);
-        float x[32], bt[BIAS ? 32 : 1];
-        if (BIAS && cls[c] == 1) {
-#pragma unroll
-          for (int e = 0; e < 32; ++e) bt[BIAS ? e : 0] = __ldg(bias + gap - e);
-        }
+        float x[32];
         tc_ld32(t_s + c * 32, x);
-        if (cls[c] == 1) {
+        const int gap = qi + shift - (key0 + c * 32);
+        if (kind == 1 && BIAS) {
+          // far from the diagonal the bias of a chunk's 32 keys is a parabola through three of them
+          if (q0 + t * kRows + quarter * 32 + shift - (key0 + c * 32) - 32 >= kFarKeys) {
+            const float b0 = __ldg(bias + gap), b1 = __ldg(bias + gap - 16), b2 = __ldg(bias + gap - 32);
+            const float c0 = neg_m - b0, c1 = (3.f * b0 + b2 - 4.f * b1) * (1.f / 32.f), c2 = (2.f * b1 - b0 - b2) * (1.f / 512.f);
 #pragma unroll
-          for (int e = 0; e < 32; ++e) x[e] = ex2(fmaf(x[e], p.scale_log2, BIAS ? neg_m - bt[BIAS ? e : 0] : neg_m));
+            for (int e = 0; e < 32; e += 2) {
+              float s0, s1;
+              fma2(s0, s1, (float)e, (float)(e + 1), c2, c2, c1, c1);
+              fma2(s0, s1, s0, s1, (float)e, (float)(e + 1), c0, c0);
+              fma2(x[e], x[e + 1], x[e], x[e + 1], p.scale_log2, p.scale_log2, s0, s1);
+            }
+          } else {
+#pragma unroll
+            for (int e = 0; e < 32; e += 2) {
+              float s0, s1;
+              add2(s0, s1, neg_m, neg_m, -__ldg(bias + gap - e), -__ldg(bias + gap - e - 1));
+              fma2(x[e], x[e + 1], x[e], x[e + 1], p.scale_log2, p.scale_log2, s0, s1);
+            }
+          }
+#pragma unroll
+          for (int e = 0; e < 32; ++e) x[e] = ex2(x[e]);
+        } else if (kind == 1) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) x[e] = ex2(fmaf(x[e], p.scale_log2, neg_m));
         } else {
           const int nvis = vis_end - (key0 + c * 32), n0 = vis_begin - (key0 + c * 32);
 #pragma unroll
           for (int e = 0; e < 32; ++e) {
-            float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mval[c], e));
+            float v = fmaf(x[e], p.scale_log2, __shfl_sync(0xffffffffu, mv, e));
             if (BIAS) v -= __ldg(bias + max(0, gap - e));
             x[e] = e < nvis && e >= n0 ? ex2(v + neg_m) : 0.f;
           }
@@ -370,6 +401,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           }
           *reinterpret_cast<uint4 *>(dst + ((((c & 1) * 4 + g) ^ (row & 7)) << 4)) = w;
         }
+      };
+      if constexpr (BIAS) {
+#pragma unroll 1
+        for (int c = 0; c < kKeys / 32; ++c) weights(c, (classes >> (2 * c)) & 3, mask_value(c));
+      } else {
+#pragma unroll
+        for (int c = 0; c < kKeys / 32; ++c) weights(c, cls[c], mval[c]);
       }
       l_run += l0 + l1;
       // P is complete for this warp's 32 rows: make it visible to the tensor core's reads.  The

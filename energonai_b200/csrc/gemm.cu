@@ -105,6 +105,10 @@ struct GemmParams {
   // numbers on the device (EB_ACT_XIELU)
   int act_cols;
   const float *act_params;
+  // columns from tail_col on (a multiple of 8) go, in fp32, to `tail` instead of C
+  int tail_col;
+  float *tail;
+  long long ld_tail;
 };
 
 // ---- PTX wrappers ---------------------------------------------------------------------------
@@ -308,8 +312,7 @@ template <int BN, bool SWAP> struct Scheduler {
 // First weight row of the group that a row tile of A belongs to.
 __device__ __forceinline__ int group_row(const GemmParams &p, int lane_tile) { return p.tile_group ? p.tile_group[lane_tile] * p.N : 0; }
 
-__device__ __forceinline__ float apply_act(float v, int act, float a0 = 0.f, float a1 = 0.f) {
-  if (act == EB_ACT_XIELU) return xielu_fast(v, a0, a1);
+__device__ __forceinline__ float apply_act(float v, int act) {
   if (act == EB_ACT_RELU) return fmaxf(v, 0.f);
   if (act == EB_ACT_GELU_TANH) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * v * (1.f + 0.044715f * v * v)));
   if (act == EB_ACT_GELU_ERF) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
@@ -719,13 +722,20 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
                     if (act == EB_ACT_RELU) {
 #pragma unroll
                       for (int j = 0; j < 8; ++j) vv[j] = fmaxf(vv[j], 0.f);
+                    } else if (act == EB_ACT_XIELU) {
+#pragma unroll
+                      for (int j = 0; j < 8; ++j) vv[j] = xielu_fast(vv[j], act0, act1);
                     } else if (act != EB_ACT_NONE) {
 #pragma unroll
-                      for (int j = 0; j < 8; ++j) vv[j] = apply_act(vv[j], act, act0, act1);
+                      for (int j = 0; j < 8; ++j) vv[j] = apply_act(vv[j], act);
                     }
 #pragma unroll
                     for (int j = 0; j < 8; ++j) vv[j] += rf[j];
-                    if (out_f32) {
+                    if (n >= p.tail_col) {
+                      float4 *o = reinterpret_cast<float4 *>(p.tail + (long long)m * p.ld_tail + (n - p.tail_col));
+                      o[0] = make_float4(vv[0], vv[1], vv[2], vv[3]);
+                      o[1] = make_float4(vv[4], vv[5], vv[6], vv[7]);
+                    } else if (out_f32) {
                       float4 *o = reinterpret_cast<float4 *>(reinterpret_cast<float *>(p.C) + c_off + n);
                       o[0] = make_float4(vv[0], vv[1], vv[2], vv[3]);
                       o[1] = make_float4(vv[4], vv[5], vv[6], vv[7]);
@@ -997,13 +1007,20 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
             if (act == EB_ACT_RELU) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) y[j] = fmaxf(y[j], 0.f);
+            } else if (act == EB_ACT_XIELU) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) y[j] = xielu_fast(y[j], act0, act1);
             } else if (act != EB_ACT_NONE) {
 #pragma unroll
-              for (int j = 0; j < 16; ++j) y[j] = apply_act(y[j], act, act0, act1);
+              for (int j = 0; j < 16; ++j) y[j] = apply_act(y[j], act);
             }
 #pragma unroll
             for (int j = 0; j < 16; ++j) y[j] += r[j];
-            if (out_f32) {
+            if (n >= p.tail_col) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j)
+                if (m0 + j < rows) p.tail[(long long)(m0 + j) * p.ld_tail + (n - p.tail_col)] = y[j];
+            } else if (out_f32) {
               float *c = reinterpret_cast<float *>(p.C);
 #pragma unroll
               for (int j = 0; j < 16; ++j) {
@@ -1372,7 +1389,8 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
                      const int32_t *c_row_offset_device, int c_row_offset_limit, int flags, void *workspace,
                      size_t workspace_bytes, void *stream, const eb_comm *comm, const float *ln_colsum = nullptr,
                      const float *ln_bias = nullptr, double ln_eps = 0.0, bool reduce_scatter = false,
-                     size_t rs_stage_offset = 0, int act_cols = 0x7fffffff, const float *act_params = nullptr) {
+                     size_t rs_stage_offset = 0, int act_cols = 0x7fffffff, const float *act_params = nullptr,
+                     int tail_col = 0x7fffffff, float *tail = nullptr, long long ld_tail = 0) {
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "gemm: operands must be fp16 or bf16 (got dtype %d)", dtype);
   if (ln_colsum || ln_bias) {
     EB_REQUIRE(ln_colsum && ln_bias, "gemm_ln: ln_colsum and ln_bias go together");
@@ -1390,7 +1408,7 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
   // the generation orientation (M <= 128) writes C one element at a time: any N will do there
   EB_REQUIRE(K >= 8 && K % 8 == 0 && (N % 8 == 0 || M <= kLanes), "gemm: K, and N for M > 128, must be positive multiples of 8 (K=%d N=%d)", K, N);
   EB_REQUIRE(lda >= K && ldw >= K && lda % 8 == 0 && ldw % 8 == 0, "gemm: lda/ldw must be multiples of 8 and >= K");
-  EB_REQUIRE(ldc >= N && (ldc % 8 == 0 || M <= kLanes) && (!residual || (ldr >= N && (ldr % 8 == 0 || M <= kLanes))),
+  EB_REQUIRE(ldc >= (N < tail_col ? N : tail_col) && (ldc % 8 == 0 || M <= kLanes) && (!residual || (ldr >= N && (ldr % 8 == 0 || M <= kLanes))),
              "gemm: ldc/ldr must be >= N (and multiples of 8 for M > 128)");
   EB_REQUIRE(c_rows_per_batch >= 0 && (c_rows_per_batch == 0 || c_batch_stride % 8 == 0 || M <= kLanes), "gemm: bad batch mapping of C");
   EB_REQUIRE(c_row_offset_limit >= 0, "gemm: negative row-offset limit");
@@ -1432,7 +1450,8 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
                comm->world, comm->recv_bytes / 2);
     p.comm = comm_dev(comm);
   }
-  p.bias = bias; p.residual = residual; p.ldr = ldr; p.act = act; p.act_cols = act_cols; p.act_params = act_params; p.out_f32 = out_dtype == EB_F32 && dtype != EB_F32;
+  p.bias = bias; p.residual = residual; p.ldr = ldr; p.act = act; p.act_cols = act_cols; p.act_params = act_params;
+  p.tail_col = tail_col; p.tail = tail; p.ld_tail = ld_tail; p.out_f32 = out_dtype == EB_F32 && dtype != EB_F32;
 
   CUtensorMap tl, tc;
   int rc;
@@ -1525,6 +1544,7 @@ extern "C" int eb_gemm_grouped(const void *A, long long lda, const void *W, long
   p.lane_rows = M; p.col_rows = N;
   p.tile_group = tile_group; p.live_tiles = live_tiles;
   p.gated = gated; p.gate_limit = limit; p.gate_alpha = alpha;
+  p.act_cols = p.tail_col = 0x7fffffff;
   p.kpb = 1;
   const long long lane_tiles = M / kLanes;
   const int bn = lane_tiles * ((N + 255) / 256) >= sm_count() && N > 128 ? 256 : 128;
@@ -1553,13 +1573,15 @@ extern "C" int eb_gemm(const void *A, long long lda, const void *W, long long ld
                    nullptr);
 }
 
-extern "C" int eb_gemm_xielu(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, const void *bias, int M,
-                             int N, int K, int act_cols, const float *act_params, int dtype, int out_dtype, int flags, void *workspace,
-                             size_t workspace_bytes, void *stream) {
-  EB_REQUIRE(act_params && (uintptr_t)act_params % 4 == 0, "gemm_xielu: the activation's two numbers are required");
-  EB_REQUIRE(act_cols >= 0 && act_cols % 8 == 0, "gemm_xielu: the activation covers a multiple of 8 columns (got %d)", act_cols);
-  return gemm_impl(A, lda, W, ldw, C, ldc, bias, nullptr, 0, M, N, K, dtype, out_dtype, EB_ACT_XIELU, 0, 0, nullptr, 0, flags, workspace,
-                   workspace_bytes, stream, nullptr, nullptr, nullptr, 0.0, false, 0, act_cols, act_params);
+extern "C" int eb_gemm_parts(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, const void *bias, int M,
+                             int N, int K, int act_cols, const float *act_params, int tail_col, float *tail, long long ld_tail, int dtype,
+                             int flags, void *workspace, size_t workspace_bytes, void *stream) {
+  EB_REQUIRE((uintptr_t)act_params % 4 == 0 && act_cols >= 0 && act_cols % 8 == 0, "gemm_parts: the activation covers a multiple of 8 columns (got %d)", act_cols);
+  EB_REQUIRE(!tail || (tail_col >= 0 && tail_col <= N && tail_col % 8 == 0 && aligned16(tail) && ld_tail % 4 == 0 && ld_tail >= N - tail_col),
+             "gemm_parts: the fp32 tail begins at a multiple of 8 columns (got %d of %d) and holds whole rows", tail_col, N);
+  return gemm_impl(A, lda, W, ldw, C, ldc, bias, nullptr, 0, M, N, K, dtype, dtype, act_params ? EB_ACT_XIELU : EB_ACT_NONE, 0, 0, nullptr, 0, flags,
+                   workspace, workspace_bytes, stream, nullptr, nullptr, nullptr, 0.0, false, 0, act_params ? act_cols : 0x7fffffff, act_params,
+                   tail ? tail_col : 0x7fffffff, tail, ld_tail);
 }
 
 extern "C" int eb_gemm_ln(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc,

@@ -9,15 +9,11 @@
 //                   forms the head's norm through distributed shared memory, so that the output
 //                   gate and the projection's operand come out of the same launch.
 //   head_norm_gate  that tail alone, for the rows of a prompt.
-#include <cooperative_groups.h>
-
 #include "common.cuh"
 #include "memory_gates.cuh"
 
 namespace eb {
 namespace {
-
-namespace cg = cooperative_groups;
 
 template <typename T> __device__ __forceinline__ T store_cast(float v) { return from_f32<T>(v); }
 template <> __device__ __forceinline__ __half store_cast<__half>(float v) { return __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f)); }
@@ -134,12 +130,27 @@ struct StepParams {
   int heads, dk, dv, cols;     // cols: columns per CTA, a multiple of 4
 };
 
+__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+
 template <typename T>
-__global__ void __launch_bounds__(kStepThreads) memory_step_kernel(const StepParams p) {
+__global__ void __launch_bounds__(kStepThreads, 4) memory_step_kernel(const StepParams p) {
   extern __shared__ float sm[];
   float *qs = sm, *ks = qs + p.dk, *ns = ks + p.dk, *vs = ns + p.dk, *red = vs + p.cols;      // red: [row groups][cols]
-  __shared__ float scratch[kStepThreads / 32], head_sq;
-  cg::cluster_group cluster = cg::this_cluster();
+  // The CTAs of a head show each other their sums of squares: every one sends its own to all with an
+  // asynchronous store that completes on the receiver's mbarrier.  (A cluster barrier would do, but its
+  // release waits for the stores of the whole state.)
+  __shared__ float scratch[kStepThreads / 32], part_sq[8];
+  __shared__ __align__(8) uint64_t arrived;
+  const int peers = gridDim.x;
+  if (peers > 1) {
+    if (threadIdx.x == 0) {
+      asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(smem_addr(&arrived)) : "memory");
+      asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+      asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_addr(&arrived)), "r"(peers * 4) : "memory");
+    }
+    __syncwarp();
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+  }
   griddep_wait();
   griddep_launch();
   const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
@@ -147,6 +158,18 @@ __global__ void __launch_bounds__(kStepThreads) memory_step_kernel(const StepPar
   const long long bh = (long long)b * p.heads + h;
   const T *q = reinterpret_cast<const T *>(p.q) + b * p.ldp + h * p.dk, *k = reinterpret_cast<const T *>(p.k) + b * p.ldp + h * p.dk,
           *v = reinterpret_cast<const T *>(p.v) + b * p.ldp + h * p.dv + c0, *g = reinterpret_cast<const T *>(p.g) + b * p.ldp + h * p.dv + c0;
+  // thread = 4 columns of every R-th row; kStepBatch rows of the state in flight per thread, the first of
+  // them requested before anything else is worked out
+  const int groups = p.cols / 4, R = kStepThreads / groups, cg4 = tid % groups, rg = tid / groups;
+  const bool active = rg < R && cg4 * 4 < width;
+  float *S = p.S + bh * p.dk * p.dv + c0 + cg4 * 4;
+  float4 s[kStepBatch];
+  auto fetch = [&](int d0) {
+#pragma unroll
+    for (int i = 0; i < kStepBatch; ++i)
+      if (d0 + i * R < p.dk) s[i] = __ldcs(reinterpret_cast<const float4 *>(S + (long long)(d0 + i * R) * p.dv));
+  };
+  if (active) fetch(rg);
   const float m0 = p.m[bh];
   const float li = log_input_gate(p.gates[b * p.ldg + h], p.bias_i[h], p.cap), lf = log_forget_gate(p.gates[b * p.ldg + p.heads + h], p.bias_f[h], p.cap);
   const float m1 = fmaxf(lf + m0, li), a = expf(lf + m0 - m1), w = expf(li - m1);
@@ -162,17 +185,11 @@ __global__ void __launch_bounds__(kStepThreads) memory_step_kernel(const StepPar
   nq = block_sum<kStepThreads>(nq, scratch);                                   // (also makes qs, ks, vs visible)
   const float den = fmaxf(fabsf(nq), expf(-m1)) + kMemoryDenomEps;
 
-  // thread = 4 columns of every R-th row; kStepBatch rows of the state in flight per thread
-  const int groups = p.cols / 4, R = kStepThreads / groups, cg4 = tid % groups, rg = tid / groups;
   float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (rg < R && cg4 * 4 < width) {
+  if (active) {
     const float4 vv = *reinterpret_cast<const float4 *>(vs + cg4 * 4);
-    float *S = p.S + bh * p.dk * p.dv + c0 + cg4 * 4;
     for (int d0 = rg; d0 < p.dk; d0 += R * kStepBatch) {
-      float4 s[kStepBatch];
-#pragma unroll
-      for (int i = 0; i < kStepBatch; ++i)
-        if (d0 + i * R < p.dk) s[i] = __ldcs(reinterpret_cast<const float4 *>(S + (long long)(d0 + i * R) * p.dv));
+      if (d0 != rg) fetch(d0);
 #pragma unroll
       for (int i = 0; i < kStepBatch; ++i) {
         const int d = d0 + i * R;
@@ -198,20 +215,33 @@ __global__ void __launch_bounds__(kStepThreads) memory_step_kernel(const StepPar
     sq = fmaf(x, x, sq);
   }
   sq = block_sum<kStepThreads>(sq, scratch);
-  if (tid == 0) head_sq = sq;
-  cluster.sync();                                   // every CTA of the head has read n and m, and shows its sum of squares
-  const int peers = cluster.num_blocks();
-  float total = 0.f;
-  for (int r = 0; r < peers; ++r) total += *cluster.map_shared_rank(&head_sq, r);
-  const float rs = rsqrtf(total * p.inv_count + p.eps);
+  if (peers > 1) {
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");         // every CTA's mbarrier is set up
+    if (tid < peers) {
+      uint32_t dst, bar;
+      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(dst) : "r"(smem_addr(&part_sq[blockIdx.x])), "r"(tid));
+      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(bar) : "r"(smem_addr(&arrived)), "r"(tid));
+      asm volatile("st.async.shared::cluster.mbarrier::complete_tx::bytes.b32 [%0], %1, [%2];" ::"r"(dst), "r"(__float_as_uint(sq)), "r"(bar) : "memory");
+    }
+    // (the sums of all CTAs arrive without further waits of theirs; the limit only keeps a defect from hanging)
+    for (int it = 0; it < (1 << 20); ++it) {
+      uint32_t ok;
+      asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], 0;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+                   : "=r"(ok) : "r"(smem_addr(&arrived)) : "memory");
+      if (ok) break;
+    }
+    sq = 0.f;
+    for (int r = 0; r < peers; ++r) sq += part_sq[r];
+  }
+  const float rs = rsqrtf(sq * p.inv_count + p.eps);
   T *out = reinterpret_cast<T *>(p.out) + b * p.ldo + h * p.dv + c0;
   const T *norm = reinterpret_cast<const T *>(p.norm) + h * p.dv + c0;
   for (int c = tid; c < width; c += kStepThreads) out[c] = from_f32<T>(red[c] * rs * to_f32<T>(norm[c]) * sigmoid(to_f32<T>(g[c])));
+  // every CTA of the head has read n and m: its sum, which depends on them, is here
   if (blockIdx.x == 0) {
     for (int d = tid; d < p.dk; d += kStepThreads) p.n[bh * p.dk + d] = ns[d];
     if (tid == 0) p.m[bh] = m1;
   }
-  cluster.sync();                                   // no CTA leaves while its sum may still be read
 }
 
 template <typename T> int launch_step(StepParams p, int B, cudaStream_t st) {

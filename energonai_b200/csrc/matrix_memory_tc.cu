@@ -18,10 +18,14 @@
 // keeps 16 bits of mantissa where a single operand would have 8; a weighted score is rounded once, as
 // attention weights are.
 //
-// Warp roles (384 threads): 0 TMA, 1 MMA issue, 2 the gates (one chunk ahead: gate functions, running
-// sums and maxima, 4 tokens per lane), 3 idle, 4-7 thread = token: weights the scores, forms the
-// denominator, stores the output, 8-11 weight the keys and sum them into n (thread = 8 columns of every
-// 8th or 16th row), then thread = value column: decays the state and writes its operand copies.
+// Warp roles (512 threads): 0 TMA, 1 MMA issue, 2 the gates (one chunk ahead: gate functions, running
+// sums and maxima, 32 tokens at a time), 3 idle; 4-7 thread = token: weights the scores, forms the
+// denominator, stores the output (turned around in shared memory: rows of 128 bytes); 8-11 q.n for the
+// denominator; 12-15 thread = value column: decays the state and writes its operand copies; then 8-15
+// together weight the keys and sum them into n (thread = 8 columns of every 8th or 16th row).
+//
+// The chain from chunk to chunk is: keys arrive, A, keys weighted, state updated.  So the state's product
+// is issued before those of the output, which fill the tensor core while the next keys arrive.
 //
 // Every mbarrier wait is bounded, as in attention_tc.cu ("where" codes 300 and up).
 #include <type_traits>
@@ -34,7 +38,7 @@ namespace {
 
 constexpr int kChunk = kRows;              // tokens per chunk
 constexpr int kCols = 128;                 // value columns per CTA
-constexpr int kMemThreads = 384;
+constexpr int kMemThreads = 512;
 constexpr float kLog2eMem = 1.4426950408889634f;
 
 struct MemTcParams {
@@ -56,13 +60,14 @@ struct GateBuf {
   float inter[kChunk];         // exp(m - M_t)
   float floor_[kChunk];        // exp(-m_t)
   float w[kChunk];             // exp(u_s - M_end)
-  float decay, m_next, pad[2]; // exp(m - M_end), M_end + F_end
+  float decay, pad[3];         // exp(m - M_end)
 };
 
 template <int DK> struct MemSmem {
   static constexpr uint32_t kOp = (DK / 64) * kRows * 128, kV = 2 * kRows * 128;          // a [128][DK] operand, a [128][128] one
-  static constexpr uint32_t kGates = 256, kN = kGates + 2 * sizeof(GateBuf), kRed = kN + 2 * DK * 4, kHead = (kRed + 4 * DK * 4 + 1023) / 1024 * 1024;
-  static constexpr size_t kTotal = 1024 + kHead + 5 * (size_t)kOp + kV;
+  static constexpr uint32_t kGates = 256, kN = kGates + 2 * sizeof(GateBuf), kQn = kN + 2 * DK * 4, kRed = kQn + 2 * kChunk * 4,
+                            kHead = (kRed + 2 * 8 * DK * 4 + 1023) / 1024 * 1024, kStage = 4 * 32 * 128;
+  static constexpr size_t kTotal = 1024 + kHead + 5 * (size_t)kOp + kV + kStage;
 };
 
 template <int DK>
@@ -81,15 +86,15 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   const uint32_t raw = s32(smem_raw);
   uint8_t *smem = smem_raw + (((raw + 1023u) & ~1023u) - raw);
   const uint32_t bar0 = s32(smem);
-  const uint32_t q_full = bar0, q_empty = bar0 + 8, k_full = bar0 + 16, v_full = bar0 + 24, kv_empty = bar0 + 32, s_full = bar0 + 40, p_full = bar0 + 48,
+  const uint32_t q_full = bar0, q_empty = bar0 + 8, k_full = bar0 + 16, v_full = bar0 + 24, k_empty = bar0 + 32, s_full = bar0 + 40, p_full = bar0 + 48,
                  o_full = bar0 + 56, o_empty = bar0 + 64, state_full = bar0 + 72, kw_full = bar0 + 80, delta_full = bar0 + 88, g_full = bar0 + 96,
-                 g_empty = bar0 + 112, red_full = bar0 + 128;
-  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(smem + 192);
-  volatile int *abort_flag = reinterpret_cast<volatile int *>(smem + 200);
+                 g_empty = bar0 + 112, red_full = bar0 + 128, v_empty = bar0 + 136, qs_full = bar0 + 144, qn_full = bar0 + 152, n_full = bar0 + 160;
+  uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(smem + 224);
+  volatile int *abort_flag = reinterpret_cast<volatile int *>(smem + 232);
   GateBuf *gate_buf = reinterpret_cast<GateBuf *>(smem + L::kGates);
-  float *n_buf = reinterpret_cast<float *>(smem + L::kN), *red = reinterpret_cast<float *>(smem + L::kRed);
+  float *n_buf = reinterpret_cast<float *>(smem + L::kN), *qn_buf = reinterpret_cast<float *>(smem + L::kQn), *red = reinterpret_cast<float *>(smem + L::kRed);
   uint8_t *q_ptr = smem + L::kHead, *k_ptr = q_ptr + L::kOp, *lo_ptr = k_ptr + L::kOp, *shi_ptr = lo_ptr + L::kOp, *slo_ptr = shi_ptr + L::kOp,
-          *v_ptr = slo_ptr + L::kOp;
+          *v_ptr = slo_ptr + L::kOp, *stage_ptr = v_ptr + L::kV;
   const uint32_t q_addr = s32(q_ptr), k_addr = s32(k_ptr), lo_addr = s32(lo_ptr), shi_addr = s32(shi_ptr), slo_addr = s32(slo_ptr), v_addr = s32(v_ptr);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -104,18 +109,22 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     bar_init(q_empty, 1 + 4);                // the products' commit, and the warps that read q for the denominator
     bar_init(k_full, 1);
     bar_init(v_full, 1);
-    bar_init(kv_empty, 1);
+    bar_init(k_empty, 1);
+    bar_init(v_empty, 1);
     bar_init(s_full, 1);
     bar_init(p_full, 4);
     bar_init(o_full, 1);
     bar_init(o_empty, 4);
     bar_init(state_full, 4);
-    bar_init(kw_full, 4);
+    bar_init(kw_full, 8);
     bar_init(delta_full, 1);
-    bar_init(red_full, 4);
+    bar_init(red_full, 8);
+    bar_init(qs_full, 1);
+    bar_init(qn_full, 4);
+    bar_init(n_full, 4);
     for (int i = 0; i < 2; ++i) {
       bar_init(g_full + 8 * i, 1);
-      bar_init(g_empty + 8 * i, 8);
+      bar_init(g_empty + 8 * i, 12);
     }
     *abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -129,7 +138,7 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = *tmem_slot;
+  const uint32_t tmem = __shfl_sync(0xffffffffu, *tmem_slot, 0);
   griddep_launch();
   griddep_wait();
 
@@ -141,59 +150,71 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         bar_expect_tx(q_full, L::kOp);
 #pragma unroll
         for (int i = 0; i < kSub; ++i) tma_load_3d(q_addr + i * kAtom, &tm_q, q_full, h * DK + i * 64, c * kChunk, b);
-        if (c > 0 && !bar_wait(kv_empty, (c - 1) & 1, abort_flag, 2)) break;
+        if (c > 0 && !bar_wait(k_empty, (c - 1) & 1, abort_flag, 2)) break;
         bar_expect_tx(k_full, L::kOp);
 #pragma unroll
         for (int i = 0; i < kSub; ++i) tma_load_3d(k_addr + i * kAtom, &tm_k, k_full, h * DK + i * 64, c * kChunk, b);
+        if (c > 0 && !bar_wait(v_empty, (c - 1) & 1, abort_flag, 24)) break;
         bar_expect_tx(v_full, L::kV);
 #pragma unroll
         for (int i = 0; i < 2; ++i) tma_load_3d(v_addr + i * kAtom, &tm_v, v_full, h * p.dv + slice * kCols + i * 64, c * kChunk, b);
+        // the stages are single: what can be had ahead is that the next chunk's rows wait in L2
+        if (c + 1 < nc) {
+#pragma unroll
+          for (int i = 0; i < kSub; ++i) {
+            tma_prefetch_3d(&tm_q, h * DK + i * 64, (c + 1) * kChunk, b);
+            tma_prefetch_3d(&tm_k, h * DK + i * 64, (c + 1) * kChunk, b);
+          }
+#pragma unroll
+          for (int i = 0; i < 2; ++i) tma_prefetch_3d(&tm_v, h * p.dv + slice * kCols + i * 64, (c + 1) * kChunk, b);
+        }
       }
     }
   } else if (warp == 1) {
     // ---------------- MMA issuer ----------------
-    if (lane == 0) {
+    // (the whole warp goes along, see tc_mma_warp)
+    {
+      auto wait = [&](uint32_t bar, int parity, int where) { return __all_sync(0xffffffffu, bar_wait(bar, parity, abort_flag, where)); };
       for (int c = 0; c < nc; ++c) {
         const int ph = c & 1, before = (c - 1) & 1;
-        if (!bar_wait(q_full, ph, abort_flag, 3) || !bar_wait(k_full, ph, abort_flag, 4)) break;
-        if (c > 0 && !bar_wait(o_full, before, abort_flag, 5)) break;          // the weighted scores of the last chunk lie where A goes
+        if (!wait(q_full, ph, 3) || !wait(k_full, ph, 4)) break;
+        if (c > 0 && !wait(o_full, before, 5)) break;          // the weighted scores of the last chunk lie where A goes
         tc_fence_after();
 #pragma unroll
-        for (int i = 0; i < kSub; ++i) {
-          const uint64_t a = tc_desc(q_addr + i * kAtom), bd = tc_desc(k_addr + i * kAtom);
-#pragma unroll
-          for (int k = 0; k < 4; ++k) tc_mma(tmem + kColA, a + 2 * k, bd + 2 * k, kIdescA, (i > 0 || k > 0) ? 1u : 0u);
+        for (int k = 0; k < DK / 16; ++k) {
+          const uint32_t at = (k >> 2) * kAtom + (k & 3) * 32;
+          tc_mma_warp(tmem + kColA, tc_desc(q_addr + at), tc_desc(k_addr + at), kIdescA, k > 0 ? 1u : 0u);
         }
-        tc_commit(s_full);
+        tc_commit_warp(s_full);
+        if (!wait(v_full, ph, 8) || !wait(kw_full, ph, 10)) break;
+        if (c > 0 && !wait(state_full, before, 6)) break;
+        tc_fence_after();
+#pragma unroll
+        for (int k = 0; k < 2 * kChunk / 16; ++k) {    // 16 tokens per instruction: two 8-row groups of V and of w K
+          const uint32_t at = (k % (kChunk / 16)) * 2048;
+          tc_mma_warp(tmem + kColS, tc_desc_nmajor(v_addr + at, kAtom), tc_desc_nmajor((k < kChunk / 16 ? k_addr : lo_addr) + at, kAtom), kIdescS,
+                      (c > 0 || k > 0) ? 1u : 0u);
+        }
+        tc_commit_warp(delta_full);
+        tc_commit_warp(k_empty);
         if (c > 0) {
-          if (!bar_wait(state_full, before, abort_flag, 6) || !bar_wait(o_empty, before, abort_flag, 7)) break;
+          if (!wait(o_empty, before, 7)) break;
           tc_fence_after();
 #pragma unroll
-          for (int part = 0; part < 2; ++part)
-#pragma unroll
-            for (int i = 0; i < kSub; ++i) {
-              const uint64_t a = tc_desc(q_addr + i * kAtom), bd = tc_desc((part ? slo_addr : shi_addr) + i * kAtom);
-#pragma unroll
-              for (int k = 0; k < 4; ++k) tc_mma(tmem + kColO1, a + 2 * k, bd + 2 * k, kIdescO, (part > 0 || i > 0 || k > 0) ? 1u : 0u);
-            }
+          for (int k = 0; k < 2 * DK / 16; ++k) {
+            const uint32_t at = ((k >> 2) % kSub) * kAtom + (k & 3) * 32;
+            tc_mma_warp(tmem + kColO1, tc_desc(q_addr + at), tc_desc((k < DK / 16 ? shi_addr : slo_addr) + at), kIdescO, k > 0 ? 1u : 0u);
+          }
         }
-        tc_commit(q_empty);
-        if (!bar_wait(v_full, ph, abort_flag, 8) || !bar_wait(p_full, ph, abort_flag, 9)) break;
+        tc_commit_warp(q_empty);
+        tc_commit_warp(qs_full);
+        if (!wait(p_full, ph, 9)) break;
         tc_fence_after();
 #pragma unroll
-        for (int k = 0; k < kChunk / 16; ++k)          // 16 tokens per instruction: 8 columns of P, two 8-row groups of V
-          tc_mma_ts(tmem + kColO2, tmem + kColA + 8 * k, tc_desc_nmajor(v_addr + k * 2048, kAtom), kIdescPV, k > 0 ? 1u : 0u);
-        tc_commit(o_full);
-        if (!bar_wait(kw_full, ph, abort_flag, 10)) break;
-        tc_fence_after();
-#pragma unroll
-        for (int part = 0; part < 2; ++part)
-#pragma unroll
-          for (int k = 0; k < kChunk / 16; ++k)
-            tc_mma(tmem + kColS, tc_desc_nmajor(v_addr + k * 2048, kAtom), tc_desc_nmajor((part ? lo_addr : k_addr) + k * 2048, kAtom), kIdescS,
-                   (c > 0 || part > 0 || k > 0) ? 1u : 0u);
-        tc_commit(delta_full);
-        tc_commit(kv_empty);
+        for (int k = 0; k < kChunk / 16; ++k)          // 8 columns of P per instruction
+          tc_mma_ts_warp(tmem + kColO2, tmem + kColA + 8 * k, tc_desc_nmajor(v_addr + k * 2048, kAtom), kIdescPV, k > 0 ? 1u : 0u);
+        tc_commit_warp(o_full);
+        tc_commit_warp(v_empty);
       }
     }
   } else if (warp == 2) {
@@ -201,61 +222,51 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     const float bi = p.bias_i[h], bf = p.bias_f[h];
     const int t_first = p.first ? p.first[b] : 0;
     float m = 0.f;
-    for (int c = 0; c < nc; ++c) {
+    // pre-activations are requested 32 tokens ahead
+    float ai, af;
+    auto fetch = [&](int t) {
+      const float *g = p.gates + ((long long)b * p.seq + min(t, p.seq - 1)) * p.ldg;
+      ai = g[h];
+      af = g[p.heads + h];
+    };
+    fetch(lane);
+    bool alive = true;
+    for (int c = 0; c < nc && alive; ++c) {
       const int slot = c & 1;
-      float li[4], F[4];
-      float run = 0.f;
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int t = c * kChunk + lane * 4 + j;
-        li[j] = -INFINITY;                             // padding, or behind the end: adds nothing, forgets nothing
-        if (t >= t_first && t < p.seq) {
-          const float *g = p.gates + ((long long)b * p.seq + t) * p.ldg;
-          li[j] = log_input_gate(g[h], bi, p.cap);
-          run += log_forget_gate(g[p.heads + h], bf, p.cap);
-        }
-        F[j] = run;
-      }
-      float base = run;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float x = __shfl_up_sync(0xffffffffu, base, o);
-        if (lane >= o) base += x;
-      }
-      const float F_end = __shfl_sync(0xffffffffu, base, 31);
-      base -= run;
-      float u[4], top = -INFINITY;
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        F[j] += base;
-        u[j] = li[j] - F[j];
-        top = fmaxf(top, u[j]);
-      }
-      float upto = top;
-#pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float x = __shfl_up_sync(0xffffffffu, upto, o);
-        if (lane >= o) upto = fmaxf(upto, x);
-      }
-      const float M_end = fmaxf(m, __shfl_sync(0xffffffffu, upto, 31));
-      float prev = __shfl_up_sync(0xffffffffu, upto, 1);
-      float M = lane == 0 ? m : fmaxf(m, prev);
-      if (c >= 2 && !__all_sync(0xffffffffu, bar_wait(g_empty + 8 * slot, ((c >> 1) - 1) & 1, abort_flag, 11))) break;
+      if (c >= 2 && !__all_sync(0xffffffffu, bar_wait(g_empty + 8 * slot, ((c >> 1) - 1) & 1, abort_flag, 11))) { alive = false; break; }
       GateBuf &gb = gate_buf[slot];
+      float F_end = 0.f, M_end = m;                    // of the tokens so far
+#pragma unroll 1
+      for (int j = 0; j < kChunk; j += 32) {
+        const int t = c * kChunk + j + lane;
+        const bool live = t >= t_first && t < p.seq;   // padding, or behind the end: adds nothing, forgets nothing
+        const float li = live ? log_input_gate(ai, bi, p.cap) : -INFINITY;
+        float F = live ? log_forget_gate(af, bf, p.cap) : 0.f;
+        fetch(t + 32);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int t = lane * 4 + j;
-        M = fmaxf(M, u[j]);
-        gb.u2[t] = u[j] * kLog2eMem;
-        gb.M2[t] = M * kLog2eMem;
-        gb.inter[t] = expf(m - M);
-        gb.floor_[t] = expf(-(M + F[j]));
-        gb.w[t] = expf(u[j] - M_end);
+        for (int o = 1; o < 32; o <<= 1) {
+          const float x = __shfl_up_sync(0xffffffffu, F, o);
+          if (lane >= o) F += x;
+        }
+        F += F_end;
+        F_end = __shfl_sync(0xffffffffu, F, 31);
+        const float u = li - F;
+        float M = u;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+          const float x = __shfl_up_sync(0xffffffffu, M, o);
+          if (lane >= o) M = fmaxf(M, x);
+        }
+        M = fmaxf(M, M_end);
+        M_end = __shfl_sync(0xffffffffu, M, 31);
+        gb.u2[j + lane] = u * kLog2eMem;
+        gb.M2[j + lane] = M * kLog2eMem;
+        gb.inter[j + lane] = ex2((m - M) * kLog2eMem);
+        gb.floor_[j + lane] = ex2(-(M + F) * kLog2eMem);
       }
-      if (lane == 0) {
-        gb.decay = expf(m - M_end);
-        gb.m_next = M_end + F_end;
-      }
+#pragma unroll 1
+      for (int j = lane; j < kChunk; j += 32) gb.w[j] = ex2(gb.u2[j] - M_end * kLog2eMem);   // (this lane's own entries)
+      if (lane == 0) gb.decay = ex2((m - M_end) * kLog2eMem);
       m = M_end + F_end;
       __syncwarp();
       if (lane == 0) bar_arrive(g_full + 8 * slot);
@@ -265,17 +276,17 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
     // ---------------- scores and output: thread = token ----------------
     const int quarter = warp & 3, row = quarter * 32 + lane;
     const uint32_t t_lane = tmem + ((uint32_t)(quarter * 32) << 16);
-    const uint8_t *q_row = q_ptr + row * 128;
+    uint8_t *stage = stage_ptr + quarter * (32 * 128);
     bool alive = true;
     for (int c = 0; c < nc && alive; ++c) {
-      const int ph = c & 1, before = (c - 1) & 1, slot = c & 1;
+      const int ph = c & 1, slot = c & 1;
       if (!__all_sync(0xffffffffu, bar_wait(g_full + 8 * slot, (c >> 1) & 1, abort_flag, 12))) { alive = false; break; }
       const GateBuf &gb = gate_buf[slot];
       const float M2 = gb.M2[row], inter = gb.inter[row], floor_ = gb.floor_[row];
       if (!__all_sync(0xffffffffu, bar_wait(s_full, ph, abort_flag, 13))) { alive = false; break; }
       tc_fence_after();
-      float sum = 0.f;
-#pragma unroll
+      float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll 1
       for (int cc = 0; cc < kChunk / 32; ++cc) {
         uint32_t packed[16];
         if (cc > quarter) {                            // behind the diagonal for every row of the warp
@@ -286,8 +297,11 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           tc_ld32(t_lane + kColA + cc * 32, x);
 #pragma unroll
           for (int e = 0; e < 32; e += 4) {
-            const float4 u = *reinterpret_cast<const float4 *>(gb.u2 + cc * 32 + e);
-            x[e] *= ex2(u.x - M2); x[e + 1] *= ex2(u.y - M2); x[e + 2] *= ex2(u.z - M2); x[e + 3] *= ex2(u.w - M2);
+            float4 u = *reinterpret_cast<const float4 *>(gb.u2 + cc * 32 + e);
+            add2(u.x, u.y, u.x, u.y, -M2, -M2);
+            add2(u.z, u.w, u.z, u.w, -M2, -M2);
+            mul2(x[e], x[e + 1], x[e], x[e + 1], ex2(u.x), ex2(u.y));
+            mul2(x[e + 2], x[e + 3], x[e + 2], x[e + 3], ex2(u.z), ex2(u.w));
           }
           if (cc == quarter) {
 #pragma unroll
@@ -295,22 +309,88 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           }
 #pragma unroll
           for (int e = 0; e < 32; e += 2) {
-            sum += x[e] + x[e + 1];
+            add2(sum0, sum1, sum0, sum1, x[e], x[e + 1]);
             packed[e / 2] = pack2<T>(x[e], x[e + 1]);
           }
         }
         tc_st16(t_lane + kColA + cc * 16, packed);     // over scores of this row that have been read
       }
       tc_st_wait();
-      // the chunk's first state: its part of the denominator is q . n
-      float qn = 0.f;
-      if (c > 0) {
-        if (!__all_sync(0xffffffffu, bar_wait(state_full, before, abort_flag, 14)) || !__all_sync(0xffffffffu, bar_wait(q_full, ph, abort_flag, 15))) {
-          alive = false;
-          break;
-        }
-        const float *n = n_buf + slot * DK;
+      // the part of the chunk's first state in the denominator
+      if (!__all_sync(0xffffffffu, bar_wait(qn_full, ph, abort_flag, 14))) { alive = false; break; }
+      const float qn = qn_buf[slot * kChunk + row];
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) {
+        bar_arrive(p_full);
+        bar_arrive(g_empty + 8 * slot);
+      }
+      const float den = fmaxf(fabsf(p.scale * fmaf(inter, qn, sum0 + sum1)), floor_) + kMemoryDenomEps;
+      const float f2 = p.scale / den, f1 = f2 * inter;
+      if (!__all_sync(0xffffffffu, bar_wait(o_full, ph, abort_flag, 16))) { alive = false; break; }
+      tc_fence_after();
+      T *ob = reinterpret_cast<T *>(p.o) + ((long long)b * p.seq + c * kChunk + quarter * 32) * p.ldo + h * p.dv + slice * kCols;
+      const int left = p.dv - slice * kCols;           // value columns of this slice that exist (a multiple of 8)
+      const int rows = p.seq - c * kChunk - quarter * 32;
+#pragma unroll 1
+      for (int cc = 0; cc < kCols / 32; ++cc) {
+        uint32_t xr[32], yr[32];
+        float x[32];
+        tc_ld32_issue(t_lane + kColO2 + cc * 32, xr);
+        tc_ld32_issue(t_lane + kColO1 + cc * 32, yr);
+        tc_ld_wait();
 #pragma unroll
+        for (int e = 0; e < 32; e += 2) mul2(x[e], x[e + 1], __uint_as_float(xr[e]), __uint_as_float(xr[e + 1]), f2, f2);
+        if (c > 0) {                                   // (the first chunk begins with nothing; O1 is not defined)
+#pragma unroll
+          for (int e = 0; e < 32; e += 2)
+            fma2(x[e], x[e + 1], __uint_as_float(yr[e]), __uint_as_float(yr[e + 1]), f1, f1, x[e], x[e + 1]);
+        }
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          uint4 w;
+          w.x = pack2<T>(x[g * 8 + 0], x[g * 8 + 1]);
+          w.y = pack2<T>(x[g * 8 + 2], x[g * 8 + 3]);
+          w.z = pack2<T>(x[g * 8 + 4], x[g * 8 + 5]);
+          w.w = pack2<T>(x[g * 8 + 6], x[g * 8 + 7]);
+          *reinterpret_cast<uint4 *>(stage + lane * 128 + ((((cc & 1) * 4 + g) ^ (lane & 7)) << 4)) = w;
+        }
+        if ((cc & 1) == 0) continue;
+        // 64 columns of the warp's 32 rows: 8 lanes store a row
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          const int r = i * 4 + (lane >> 3), col = (cc >> 1) * 64 + (lane & 7) * 8;
+          const uint4 w = *reinterpret_cast<const uint4 *>(stage + r * 128 + (((lane & 7) ^ (r & 7)) << 4));
+          if (r < rows && col < left) *reinterpret_cast<uint4 *>(ob + (long long)r * p.ldo + col) = w;
+        }
+        __syncwarp();
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) bar_arrive(o_empty);
+    }
+  } else if (warp >= 8) {
+    // ---------------- q.n (warps 8-11), state (12-15), weighted keys (all) ----------------
+    const int half = (warp - 8) >> 2, tid = threadIdx.x - 256 - half * 128, quarter = warp & 3, row = quarter * 32 + lane;
+    const uint32_t t_state = tmem + ((uint32_t)(quarter * 32) << 16) + kColS;
+    constexpr int kPieces = DK / 8, kRowStep = 128 / kPieces;                   // 16-byte pieces of a row; rows a pass of 128 threads covers
+    const int piece = tid % kPieces, r0 = half * (kChunk / 2) + tid / kPieces;  // each half of the warps takes half of the rows
+    const uint32_t piece_off = (uint32_t)(piece >> 3) * kAtom;
+    bool alive = true;
+    for (int c = 0; c < nc && alive; ++c) {
+      const int ph = c & 1, before = (c - 1) & 1, slot = c & 1;
+      auto wait = [&](uint32_t bar, int parity, int where) { return __all_sync(0xffffffffu, bar_wait(bar, parity, abort_flag, where)) != 0; };
+      if (!wait(g_full + 8 * slot, (c >> 1) & 1, 17)) { alive = false; break; }
+      const GateBuf &gb = gate_buf[slot];
+      const float decay = gb.decay;
+      if (half == 0) {
+        // (p_full of the chunk before: the last q.n has been read)
+        if ((c > 0 && (!wait(p_full, before, 18) || !wait(n_full, before, 19))) || !wait(q_full, ph, 20)) { alive = false; break; }
+        const uint8_t *q_row = q_ptr + row * 128;
+        const float *n = n_buf + slot * DK;
+        float qn[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
         for (int i = 0; i < DK / 8; ++i) {
           const uint4 w = *reinterpret_cast<const uint4 *>(q_row + (i >> 3) * kAtom + (((i & 7) ^ (row & 7)) << 4));
           const uint32_t ww[4] = {w.x, w.y, w.z, w.w};
@@ -319,70 +399,19 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const float2 f = unpack2<T>(ww[e]);
-            qn = fmaf(f.x, nn[2 * e], qn);
-            qn = fmaf(f.y, nn[2 * e + 1], qn);
+            fma2(qn[(e & 1) * 2], qn[(e & 1) * 2 + 1], f.x, f.y, nn[2 * e], nn[2 * e + 1], qn[(e & 1) * 2], qn[(e & 1) * 2 + 1]);
           }
         }
-      }
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) {
-        bar_arrive(p_full);
-        bar_arrive(q_empty);
-        bar_arrive(g_empty + 8 * slot);
-      }
-      const float den = fmaxf(fabsf(p.scale * fmaf(inter, qn, sum)), floor_) + kMemoryDenomEps;
-      const float f2 = p.scale / den, f1 = f2 * inter;
-      if (!__all_sync(0xffffffffu, bar_wait(o_full, ph, abort_flag, 16))) { alive = false; break; }
-      tc_fence_after();
-      const int t = c * kChunk + row;
-      T *orow = reinterpret_cast<T *>(p.o) + ((long long)b * p.seq + t) * p.ldo + h * p.dv + slice * kCols;
-      const int left = p.dv - slice * kCols;           // value columns of this slice that exist (a multiple of 8)
-#pragma unroll 1
-      for (int cc = 0; cc < kCols / 32; ++cc) {
-        float x[32];
-        tc_ld32(t_lane + kColO2 + cc * 32, x);
-#pragma unroll
-        for (int e = 0; e < 32; ++e) x[e] *= f2;
-        if (c > 0) {
-          float y[32];
-          tc_ld32(t_lane + kColO1 + cc * 32, y);
-#pragma unroll
-          for (int e = 0; e < 32; ++e) x[e] = fmaf(y[e], f1, x[e]);
+        qn_buf[slot * kChunk + row] = (qn[0] + qn[1]) + (qn[2] + qn[3]);
+        __syncwarp();
+        if (lane == 0) {
+          bar_arrive(qn_full);
+          bar_arrive(q_empty);
         }
-        if (t < p.seq) {
-#pragma unroll
-          for (int g = 0; g < 4; ++g) {
-            if (cc * 32 + g * 8 >= left) break;
-            uint4 w;
-            w.x = pack2<T>(x[g * 8 + 0], x[g * 8 + 1]);
-            w.y = pack2<T>(x[g * 8 + 2], x[g * 8 + 3]);
-            w.z = pack2<T>(x[g * 8 + 4], x[g * 8 + 5]);
-            w.w = pack2<T>(x[g * 8 + 6], x[g * 8 + 7]);
-            *reinterpret_cast<uint4 *>(orow + cc * 32 + g * 8) = w;
-          }
-        }
-      }
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) bar_arrive(o_empty);
-    }
-  } else if (warp >= 8) {
-    // ---------------- keys and state ----------------
-    const int tid = threadIdx.x - 256, quarter = warp & 3, row = quarter * 32 + lane;
-    const uint32_t t_state = tmem + ((uint32_t)(quarter * 32) << 16) + kColS;
-    constexpr int kPieces = DK / 8, kRowStep = 128 / kPieces;                   // 16-byte pieces of a row; rows a pass covers
-    const int piece = tid % kPieces, r0 = tid / kPieces;
-    const uint32_t piece_off = (uint32_t)(piece >> 3) * kAtom;
-    bool alive = true;
-    for (int c = 0; c < nc && alive; ++c) {
-      const int ph = c & 1, before = (c - 1) & 1, slot = c & 1;
-      if (!__all_sync(0xffffffffu, bar_wait(g_full + 8 * slot, (c >> 1) & 1, abort_flag, 17))) { alive = false; break; }
-      const GateBuf &gb = gate_buf[slot];
-      const float decay = gb.decay;
-      if (c > 0) {
-        // the state this chunk begins with: operand copies for Q S, and the master decayed for what is added to it
-        if (!__all_sync(0xffffffffu, bar_wait(delta_full, before, abort_flag, 18))) { alive = false; break; }
+      } else if (c > 0) {
+        // the state this chunk begins with: operand copies for Q S (the last ones have been read), and the
+        // master decayed for what is added to it
+        if (!wait(delta_full, before, 21) || !wait(qs_full, before, 22)) { alive = false; break; }
         tc_fence_after();
 #pragma unroll 1
         for (int cc = 0; cc < DK / 32; ++cc) {
@@ -394,17 +423,18 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
             uint32_t hi[4], lo[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-              const float a = x[g * 8 + 2 * e], d = x[g * 8 + 2 * e + 1];
+              float a = x[g * 8 + 2 * e], d = x[g * 8 + 2 * e + 1];
               hi[e] = pack2<T>(a, d);
               const float2 r = unpack2<T>(hi[e]);
-              lo[e] = pack2<T>(a - r.x, d - r.y);
+              add2(a, d, a, d, -r.x, -r.y);
+              lo[e] = pack2<T>(a, d);
             }
             const uint32_t at = off + ((((cc & 1) * 4 + g) ^ (row & 7)) << 4);
             *reinterpret_cast<uint4 *>(shi_ptr + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
             *reinterpret_cast<uint4 *>(slo_ptr + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
           }
 #pragma unroll
-          for (int e = 0; e < 32; ++e) x[e] *= decay;
+          for (int e = 0; e < 32; e += 2) mul2(x[e], x[e + 1], x[e], x[e + 1], decay, decay);
           tc_st32(t_state + cc * 32, x);
         }
         tc_st_wait();
@@ -413,33 +443,41 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
         __syncwarp();
         if (lane == 0) bar_arrive(state_full);
       }
-      if (!__all_sync(0xffffffffu, bar_wait(k_full, ph, abort_flag, 19)) || !__all_sync(0xffffffffu, bar_wait(s_full, ph, abort_flag, 20))) {
-        alive = false;
-        break;
-      }
+      if (!wait(k_full, ph, 23) || !wait(s_full, ph, 24)) { alive = false; break; }
       float acc[8] = {};
+#pragma unroll 1
+      for (int i0 = 0; i0 < kChunk / 2 / kRowStep; i0 += 4) {
+        uint4 kv[4];
+        float w[4];
 #pragma unroll
-      for (int i = 0; i < kChunk / kRowStep; ++i) {
-        const int r = r0 + i * kRowStep;
-        const uint32_t at = piece_off + r * 128 + (((piece & 7) ^ (r & 7)) << 4);
-        const uint4 kv = *reinterpret_cast<const uint4 *>(k_ptr + at);
-        const uint32_t kk[4] = {kv.x, kv.y, kv.z, kv.w};
-        const float w = gb.w[r];
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float2 f = unpack2<T>(kk[e]);
-          const float a = w * f.x, d = w * f.y;
-          acc[2 * e] += a;
-          acc[2 * e + 1] += d;
-          hi[e] = pack2<T>(a, d);
-          const float2 x = unpack2<T>(hi[e]);
-          lo[e] = pack2<T>(a - x.x, d - x.y);
+        for (int i = 0; i < 4; ++i) {                  // the rows of a batch are read before any of them is written
+          const int r = r0 + (i0 + i) * kRowStep;
+          kv[i] = *reinterpret_cast<const uint4 *>(k_ptr + piece_off + r * 128 + (((piece & 7) ^ (r & 7)) << 4));
+          w[i] = gb.w[r];
         }
-        *reinterpret_cast<uint4 *>(k_ptr + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        *reinterpret_cast<uint4 *>(lo_ptr + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int r = r0 + (i0 + i) * kRowStep;
+          const uint32_t kk[4] = {kv[i].x, kv[i].y, kv[i].z, kv[i].w};
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            float2 f = unpack2<T>(kk[e]);
+            mul2(f.x, f.y, f.x, f.y, w[i], w[i]);
+            add2(acc[2 * e], acc[2 * e + 1], acc[2 * e], acc[2 * e + 1], f.x, f.y);
+            hi[e] = pack2<T>(f.x, f.y);
+            const float2 x = unpack2<T>(hi[e]);
+            add2(f.x, f.y, f.x, f.y, -x.x, -x.y);
+            lo[e] = pack2<T>(f.x, f.y);
+          }
+          const uint32_t at = piece_off + r * 128 + (((piece & 7) ^ (r & 7)) << 4);
+          *reinterpret_cast<uint4 *>(k_ptr + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+          *reinterpret_cast<uint4 *>(lo_ptr + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        }
       }
       asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      __syncwarp();
+      if (lane == 0) bar_arrive(kw_full);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
 #pragma unroll
@@ -447,20 +485,29 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
       }
       if (lane < kPieces) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) red[quarter * DK + piece * 8 + e] = acc[e];
+        for (int e = 0; e < 8; ++e) red[(slot * 8 + warp - 8) * DK + piece * 8 + e] = acc[e];
       }
       __syncwarp();
       if (lane == 0) bar_arrive(red_full);
-      if (!__all_sync(0xffffffffu, bar_wait(red_full, ph, abort_flag, 22))) { alive = false; break; }
-      if (tid < DK)
-        n_buf[(slot ^ 1) * DK + tid] = fmaf(decay, n_buf[slot * DK + tid], red[tid] + red[DK + tid] + red[2 * DK + tid] + red[3 * DK + tid]);
-      __syncwarp();
-      if (lane == 0) {
-        bar_arrive(kw_full);
-        bar_arrive(g_empty + 8 * slot);
+      if (half == 0) {
+        if (!wait(red_full, ph, 25)) { alive = false; break; }
+        if (tid < DK) {
+          float sum = 0.f;
+#pragma unroll
+          for (int i = 0; i < 8; ++i) sum += red[(slot * 8 + i) * DK + tid];
+          n_buf[(slot ^ 1) * DK + tid] = fmaf(decay, n_buf[slot * DK + tid], sum);
+        }
+        __syncwarp();
+        if (lane == 0) bar_arrive(n_full);
       }
+      __syncwarp();
+      if (lane == 0) bar_arrive(g_empty + 8 * slot);
     }
-    if (alive && !__all_sync(0xffffffffu, bar_wait(delta_full, (nc - 1) & 1, abort_flag, 21))) alive = false;
+    if (half == 0) {
+      if (alive && slice == 0 && tid < DK) p.n[((long long)b * p.heads + h) * DK + tid] = n_buf[(nc & 1) * DK + tid];
+      alive = false;                                   // (the state is the other half's)
+    }
+    if (alive && !__all_sync(0xffffffffu, bar_wait(delta_full, (nc - 1) & 1, abort_flag, 26))) alive = false;
     if (alive) {
       tc_fence_after();
       const long long bh = (long long)b * p.heads + h;
@@ -475,7 +522,6 @@ memory_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_const
           for (int e = 0; e < 32; ++e) S[(long long)e * p.dv] = x[e];
         }
       }
-      if (slice == 0 && tid < DK) p.n[bh * DK + tid] = n_buf[(nc & 1) * DK + tid];
     }
   }
 

@@ -10,9 +10,7 @@
 //                     lies on the critical path).
 //   stream_update     the residual step of blocks that normalise in front of AND behind a
 //                     sublayer: x += norm(y * sigmoid(gate)) * w_out, then h = norm(x) * w_next for
-//                     the sublayer that follows, and optionally a few more products of h whose
-//                     results stay in fp32 (the gates of a recurrence that follows).  With `src` it
-//                     starts the stream instead: x = scale * src.
+//                     the sublayer that follows.  With `src` it starts the stream: x = scale * src.
 //
 // One CTA per row, the row register-resident in packs of 8; statistics, weights and the residual
 // are fp32 throughout.
@@ -223,18 +221,14 @@ struct StreamParams {
   const void *w_next;          // [n2] T, or null: no h
   void *h;
   long long ldh;
-  const void *proj;            // [n_proj][n2] T, or null
-  int n_proj;
-  float *proj_out;             // rows ldp apart
-  long long ldp;
   float eps, inv_count;
   int n2;
 };
 
-template <typename T, int PACKS, int THREADS>
-__global__ void __launch_bounds__(THREADS) stream_update_kernel(const StreamParams p) {
+template <typename T, int PACKS>
+__global__ void __launch_bounds__(kNormThreads) stream_update_kernel(const StreamParams p) {
+  constexpr int THREADS = kNormThreads;
   __shared__ float scratch[THREADS / 32];
-  extern __shared__ float dyn[];                   // the row of h, for the small products
   const long long row = blockIdx.x;
   const int packs = p.n2 / 8;
   griddep_wait();
@@ -296,46 +290,17 @@ __global__ void __launch_bounds__(THREADS) stream_update_kernel(const StreamPara
 #pragma unroll
     for (int e = 0; e < 8; ++e) wv[e] *= v[i][e] * r;
     store8<T>(reinterpret_cast<T *>(p.h) + row * p.ldh + c * 8, wv);
-    if (p.proj) {
-      // the products read h as every other product does: rounded to the operand type
-#pragma unroll
-      for (int e = 0; e < 8; ++e) dyn[c * 8 + e] = to_f32<T>(from_f32<T>(wv[e]));
-    }
-  }
-  if (!p.proj) return;
-  __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int e = warp; e < p.n_proj; e += THREADS / 32) {
-    const T *wr = reinterpret_cast<const T *>(p.proj) + (long long)e * p.n2;
-    float acc = 0.f;
-#pragma unroll 4
-    for (int c = lane; c < packs; c += 32) {
-      float f[8];
-      load8<T>(wr + c * 8, f);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) acc = fmaf(f[j], dyn[c * 8 + j], acc);
-    }
-    acc = warp_sum(acc);
-    if (lane == 0) p.proj_out[row * p.ldp + e] = acc;
   }
 }
 
 template <typename T> int launch_stream(const StreamParams &p, int n1, cudaStream_t st) {
-  const int packs = p.n2 / 8, threads = p.proj ? 1024 : kNormThreads, per = (packs + threads - 1) / threads;
-  const size_t smem = p.proj ? (size_t)p.n2 * sizeof(float) : 0;
-  auto go = [&](auto kern) -> int {
-    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
-      cudaGetLastError();
-      return fail(EB_ECUDA, "stream_update: cannot reserve %zu bytes of shared memory", smem);
-    }
-    launch_pdl(kern, dim3(n1), dim3(threads), smem, st, p);
-    return check_launch("stream_update");
-  };
-  if (p.proj) return per <= 1 ? go(stream_update_kernel<T, 1, 1024>) : go(stream_update_kernel<T, 2, 1024>);
-  if (per <= 1) return go(stream_update_kernel<T, 1, kNormThreads>);
-  if (per <= 2) return go(stream_update_kernel<T, 2, kNormThreads>);
-  if (per <= 4) return go(stream_update_kernel<T, 4, kNormThreads>);
-  return go(stream_update_kernel<T, 8, kNormThreads>);
+  const int packs = p.n2 / 8, per = (packs + kNormThreads - 1) / kNormThreads;
+  const dim3 g(n1), b(kNormThreads);
+  if (per <= 1) launch_pdl(stream_update_kernel<T, 1>, g, b, 0, st, p);
+  else if (per <= 2) launch_pdl(stream_update_kernel<T, 2>, g, b, 0, st, p);
+  else if (per <= 4) launch_pdl(stream_update_kernel<T, 4>, g, b, 0, st, p);
+  else launch_pdl(stream_update_kernel<T, 8>, g, b, 0, st, p);
+  return check_launch("stream_update");
 }
 
 template <typename TI, typename TO>
@@ -442,8 +407,7 @@ extern "C" int eb_rms_residual(const void *y, long long ldy, int dtype, const in
 }
 
 extern "C" int eb_stream_update(const void *src, long long lds, float src_scale, const void *y, long long ldy, const void *gate, long long ldg,
-                                const float *w_out, float *x, long long ldx, const void *w_next, void *h, long long ldh, const void *proj,
-                                int n_proj, float *proj_out, long long ldp, float eps, int n1, int n2, int count, int dtype, void *stream) {
+                                const float *w_out, float *x, long long ldx, const void *w_next, void *h, long long ldh, float eps, int n1, int n2, int count, int dtype, void *stream) {
   if (n1 == 0) return EB_OK;
   EB_REQUIRE(dtype_ok(dtype), "stream_update: bad dtype %d", dtype);
   EB_REQUIRE(x && (src || y || w_next), "stream_update: null pointer");
@@ -455,12 +419,11 @@ extern "C" int eb_stream_update(const void *src, long long lds, float src_scale,
   EB_REQUIRE(!y || w_out, "stream_update: the added row needs its weight");
   EB_REQUIRE(!gate || y, "stream_update: a gate without a row");
   EB_REQUIRE(!w_next || h, "stream_update: no place for the normalised row");
-  EB_REQUIRE(!proj || (w_next && proj_out && n_proj > 0 && ldp >= n_proj), "stream_update: the small products need the normalised row and their output");
-  EB_REQUIRE(aligned16(src) && aligned16(y) && aligned16(gate) && aligned16(w_out) && aligned16(x) && aligned16(w_next) && aligned16(h) &&
-                 aligned16(proj), "stream_update: pointers must be 16-byte aligned");
+  EB_REQUIRE(aligned16(src) && aligned16(y) && aligned16(gate) && aligned16(w_out) && aligned16(x) && aligned16(w_next) && aligned16(h),
+             "stream_update: pointers must be 16-byte aligned");
   StreamParams p{};
   p.src = src; p.lds = lds; p.src_scale = src_scale; p.y = y; p.ldy = ldy; p.gate = gate; p.ldg = ldg; p.w_out = w_out;
-  p.x = x; p.ldx = ldx; p.w_next = w_next; p.h = h; p.ldh = ldh; p.proj = proj; p.n_proj = n_proj; p.proj_out = proj_out; p.ldp = ldp;
+  p.x = x; p.ldx = ldx; p.w_next = w_next; p.h = h; p.ldh = ldh;
   p.eps = eps; p.inv_count = 1.f / (float)count; p.n2 = n2;
   cudaStream_t st = as_stream(stream);
   if (dtype == EB_F32) return launch_stream<float>(p, n1, st);

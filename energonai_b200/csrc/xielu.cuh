@@ -5,9 +5,11 @@
 
 namespace eb {
 
-// for 16-bit results: the cancellation in exp(z) - 1 near zero is below their resolution
+// for 16-bit results (the cancellation in exp(z) - 1 near zero is below their resolution); no branch:
+// each half vanishes on the other side of zero
 __device__ __forceinline__ float xielu_fast(float z, float up, float down) {
-  return 0.5f * z + (z > 0.f ? up * z * z : down * (__expf(fminf(z, 0.f)) - 1.f - z));
+  const float pos = fmaxf(z, 0.f), neg = fminf(z, 0.f);
+  return fmaf(up * pos, pos, fmaf(down, (__expf(neg) - 1.f) - neg, 0.5f * z));
 }
 __device__ __forceinline__ float xielu_exact(float z, float up, float down) {
   return 0.5f * z + (z > 0.f ? up * z * z : down * (expm1f(fminf(z, 0.f)) - z));

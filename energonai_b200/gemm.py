@@ -89,23 +89,28 @@ def gemm(a, w, bias=None, act=None, residual=None, out=None, out_dtype=None, out
     return out
 
 
-def gemm_xielu(a, w, bias, act_params, act_cols, static_weight=False):
-    """a [M,K] @ w [N,K].T + bias with xIELU on the columns below act_cols (a multiple of 8); act_params:
-    device fp32 (softplus(p), 1/2 + softplus(q)), see xielu_params()."""
+def gemm_parts(a, w, bias=None, xielu=None, tail_col=None, static_weight=False):
+    """a [M,K] @ w [N,K].T + bias for stacked weights: xielu = (act_params, act_cols), that activation on
+    the columns below act_cols (act_params: device fp32 pair, see xielu_params()); tail_col: the columns
+    from there on are returned in fp32.  Returns out, or (out, tail) with tail_col."""
+    act_params, act_cols = xielu if xielu is not None else (None, 0)
     require_cuda(a, w, bias, act_params)
     if a.dim() != 2 or w.dim() != 2 or a.shape[1] != w.shape[1] or a.dtype != w.dtype or a.dtype not in (torch.float16, torch.bfloat16):
-        raise RuntimeError("gemm_xielu: fp16 or bf16 a [M,K] and w [N,K] of one dtype required")
-    if act_params.dtype != torch.float32 or act_params.numel() != 2 or (bias is not None and (bias.dtype != a.dtype or bias.numel() != w.shape[0])):
-        raise RuntimeError("gemm_xielu: two fp32 numbers, and a bias of the operand dtype with one entry per column")
+        raise RuntimeError("gemm_parts: fp16 or bf16 a [M,K] and w [N,K] of one dtype required")
+    if act_params is not None and (act_params.dtype != torch.float32 or act_params.numel() != 2):
+        raise RuntimeError("gemm_parts: the activation has two fp32 numbers")
+    if bias is not None and (bias.dtype != a.dtype or bias.numel() != w.shape[0]):
+        raise RuntimeError("gemm_parts: the bias has the operand dtype and one entry per column")
     a, w = (t if t.stride(1) == 1 else t.contiguous() for t in (a, w))
     (M, K), N = a.shape, w.shape[0]
-    out = torch.empty((M, N), dtype=a.dtype, device=a.device)
+    out = torch.empty((M, N if tail_col is None else tail_col), dtype=a.dtype, device=a.device)
+    tail = torch.empty((M, N - tail_col), dtype=torch.float32, device=a.device) if tail_col is not None else None
     nbytes = lib().eb_gemm_workspace_bytes(M, N, K)
     ws = workspace(a.device, nbytes) if nbytes else None
-    check(lib().eb_gemm_xielu(ptr(a), a.stride(0), ptr(w), w.stride(0), ptr(out), N, ptr(bias), M, N, K, int(act_cols), ptr(act_params),
-                              dtype_code(a.dtype), dtype_code(a.dtype), 1 if static_weight else 0, ptr(ws),
-                              ws.numel() if ws is not None else 0, stream_ptr()), "gemm_xielu")
-    return out
+    check(lib().eb_gemm_parts(ptr(a), a.stride(0), ptr(w), w.stride(0), ptr(out), out.shape[1], ptr(bias), M, N, K, int(act_cols),
+                              ptr(act_params), tail_col or 0, ptr(tail), tail.shape[1] if tail is not None else 0, dtype_code(a.dtype),
+                              1 if static_weight else 0, ptr(ws), ws.numel() if ws is not None else 0, stream_ptr()), "gemm_parts")
+    return out if tail is None else (out, tail)
 
 
 def xielu_params(p, q):
@@ -116,7 +121,7 @@ def xielu_params(p, q):
 
 def gemm_f32(a, w, bias=None, xielu=None):
     """a [M,K] @ w [N,K].T (+ bias) in true 32-bit (CUDA cores, no reduced-precision mode); xielu =
-    (act_params, act_cols) as in gemm_xielu."""
+    (act_params, act_cols) as in gemm_parts."""
     act_params, act_cols = xielu if xielu is not None else (None, 0)
     require_cuda(a, w, bias, act_params)
     if a.dim() != 2 or w.dim() != 2 or a.shape[1] != w.shape[1] or any(t is not None and t.dtype != torch.float32 for t in (a, w, bias, act_params)):
@@ -129,14 +134,18 @@ def gemm_f32(a, w, bias=None, xielu=None):
     return out
 
 
-def project(x, w, out_dtype=None, bias=None, xielu=None):
+def project(x, w, out_dtype=None, bias=None):
     """x @ w.T (+ bias) with a model's weight: the tensor-core GEMM, or the 32-bit one for models run in
-    fp32.  xielu = (act_params, act_cols): that activation on the first columns."""
-    if w.dtype == torch.float32:
-        return gemm_f32(x, w, bias=bias, xielu=xielu)
-    if xielu is not None:
-        return gemm_xielu(x, w, bias, *xielu, static_weight=True)
-    return gemm(x, w, bias=bias, out_dtype=out_dtype, static_weight=True)
+    fp32."""
+    return gemm_f32(x, w, bias=bias) if w.dtype == torch.float32 else gemm(x, w, bias=bias, out_dtype=out_dtype, static_weight=True)
+
+
+def project_parts(x, w, bias=None, xielu=None, tail_col=None):
+    """gemm_parts with a model's weight, or its 32-bit form."""
+    if w.dtype != torch.float32:
+        return gemm_parts(x, w, bias, xielu, tail_col, static_weight=True)
+    out = gemm_f32(x, w, bias=bias, xielu=xielu)
+    return out if tail_col is None else (out[:, :tail_col], out[:, tail_col:])
 
 
 LN_FOLD_MAX_ROWS = 32

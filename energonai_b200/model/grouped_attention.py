@@ -45,9 +45,6 @@ class GroupedAttention(nn.Module):
         self.r1, self.r2, self.vmix = fp32(H), fp32(H), fp32(1)
         self.out_proj = init_weight(width, H * self.dv, **kw)
 
-    def step_products(self):
-        return None
-
     def cache(self):
         return RingCache(self.kv_heads * (self.dk + self.dv))
 
@@ -57,7 +54,7 @@ class GroupedAttention(nn.Module):
         n = buf.shape[2] - self.kv_heads * self.dv
         return buf[:, :, :n], buf[:, :, n:]
 
-    def forward(self, h, ctx, _=None):
+    def forward(self, h, ctx):
         """h [rows, width] -> (y, pre-activation of the residual gate); keys and values are cached."""
         B, S, H, G = ctx.batch, ctx.seq, self.heads, self.kv_heads
         proj = project(h, self.in_proj, bias=self.bias)

@@ -1,13 +1,12 @@
 """Matrix-memory mixer: per head a matrix state S with a normaliser n and a running maximum m of its log
 gates, carried in fp32 from token to token (the equations are with eb_memory_scan in the header).
 
-One product of h gives queries, keys, values, output gates and the pre-activation of the residual gate;
-the two recurrence gates are products of their own, whose results stay in fp32.  In a generation step
-they come from the launch that normalised h."""
+One product of h gives queries, keys, values, output gates, the pre-activation of the residual gate and,
+in fp32, those of the two recurrence gates."""
 import torch
 from torch import nn
 
-from ..gemm import project
+from ..gemm import project, project_parts
 from ..memory import MEMORY_KEY_HEADS, head_norm_gate, memory_prompt, memory_step
 from ..nn import init_weight
 from .sequence_state import RecurrentState, round_up
@@ -24,26 +23,22 @@ class MatrixMemory(nn.Module):
         self.dv = round_up(vdim, 8)
         qk, vg = heads * self.dk, heads * self.dv
         self.splits = [qk, qk, vg, vg, width]
-        self.in_proj = init_weight(sum(self.splits), width, **kw)               # q | k | v | output gate | residual gate
-        self.bias = init_weight(sum(self.splits), std=0.0, **kw)
-        self.gates = init_weight(round_up(2 * heads, 8), width, **kw)           # input gates | forget gates
+        self.tail = sum(self.splits)
+        # q | k | v | output gate | residual gate || input gates | forget gates
+        self.in_proj = init_weight(self.tail + round_up(2 * heads, 8), width, **kw)
+        self.bias = init_weight(self.in_proj.shape[0], std=0.0, **kw)           # (the recurrence gates' is gate_bias)
         self.gate_bias = nn.Parameter(torch.zeros(2, heads, dtype=torch.float32, device=device), requires_grad=False)
         self.norm = nn.Parameter(torch.ones(vg, dtype=dtype, device=device), requires_grad=False)
         self.out_proj = init_weight(width, vg, **kw)
 
-    def step_products(self):
-        """Weight of the fp32 products that the launch before a generation step's mixer can take along."""
-        return self.gates
-
     def cache(self):
         return RecurrentState([(self.heads, self.dk, self.dv), (self.heads, self.dk), (self.heads,)])
 
-    def forward(self, h, ctx, gates=None):
+    def forward(self, h, ctx):
         """h [rows, width] -> (y, pre-activation of the residual gate); the state goes on."""
         state = ctx.state.caches[self.layer].tensors
-        q, k, v, g, rg = project(h, self.in_proj, bias=self.bias).split(self.splits, 1)
-        if gates is None:
-            gates = project(h, self.gates, out_dtype=torch.float32)
+        rows, gates = project_parts(h, self.in_proj, bias=self.bias, tail_col=self.tail)
+        q, k, v, g, rg = rows.split(self.splits, 1)
         bias = self.gate_bias.unbind(0)
         if ctx.is_prompt:
             o = memory_prompt(q, k, v, gates, bias, self.cap, self.scale, state, self.heads, first=ctx.first, chunked=self.chunked)

@@ -6,7 +6,7 @@ from typing import Callable, Optional
 import torch
 from torch import dtype, nn
 
-from ..gemm import project, xielu_params
+from ..gemm import project, project_parts, xielu_params
 from ..nn import Linear1D_Col, Linear1D_Row, init_weight
 from .sequence_state import round_up
 
@@ -69,5 +69,5 @@ class XIELUFeedForward(nn.Module):
 
     def forward(self, h):
         """-> (y, pre-activation of its gate)."""
-        u = project(h, self.up, bias=self.bias, xielu=(self.act, self.ff_padded))
+        u = project_parts(h, self.up, bias=self.bias, xielu=(self.act, self.ff_padded))
         return project(u[:, :self.ff_padded], self.down), u[:, self.ff_padded:]

@@ -4,8 +4,8 @@ sublayer, a gate on the sublayer's result, a scale per element:
     x += norm_out(mixer(h) * sigmoid(W h + b)) * scale,  h = norm_in(x)
 
 and the same for the feed-forward.  Everything between two sublayers is one launch (stream_update): gate,
-norm, scale and residual sum of the one, norm of the next and, in generation steps, the recurrence
-gates of a matrix memory that follows.  The scale is multiplied into the output norm's weight, in fp32."""
+norm, scale and residual sum of the one, norm of the next.  The scale is multiplied into the output
+norm's weight, in fp32."""
 import torch
 from torch import nn
 
@@ -15,9 +15,6 @@ from .grouped_attention import GroupedAttention, padded_head
 from .layered_decoder import LayeredDecoder
 from .matrix_memory import MatrixMemory
 from .mlp import XIELUFeedForward
-
-STEP_PRODUCTS_MAX_ROWS = 128      # beyond, the gates of a step are a product of their own
-
 
 class SandwichBlock(nn.Module):
     def __init__(self, mixer, mlp, padded, dtype, device=None):
@@ -48,23 +45,17 @@ class SandwichDecoder(LayeredDecoder):
     def run(self, rows, ctx, on_layer=None):
         eps, count = self.config.eps, self.width
         x = torch.empty(rows.shape, dtype=torch.float32, device=rows.device)
-        take_along = not ctx.is_prompt and rows.shape[0] <= STEP_PRODUCTS_MAX_ROWS
-        last = self.norm.weight if not ctx.is_prompt else None         # (of a prompt only some rows go on to the head)
-
-        def to_layer(i, **kw):
-            if i == len(self.layers):
-                return stream_update(x, eps, count, w_next=last, **kw)
-            blk = self.layers[i]
-            return stream_update(x, eps, count, w_next=blk.norm1, products=blk.mixer.step_products() if take_along else None, **kw)
-        h, extra = to_layer(0, src=rows, src_scale=self.config.embed_scale)
+        # behind the last layer: the final norm of a step (of a prompt only some rows go on to the head)
+        into = [blk.norm1 for blk in self.layers] + [None if ctx.is_prompt else self.norm.weight]
+        h = stream_update(x, eps, count, src=rows, src_scale=self.config.embed_scale, w_next=into[0])
         for i, blk in enumerate(self.layers):
-            y, gate = blk.mixer(h, ctx, extra)
+            y, gate = blk.mixer(h, ctx)
             w_out = blk.out1
             if blk.mlp is not None:
-                h, _ = stream_update(x, eps, count, y=y, gate=gate, w_out=w_out, w_next=blk.norm2)
+                h = stream_update(x, eps, count, y=y, gate=gate, w_out=w_out, w_next=blk.norm2)
                 y, gate = blk.mlp(h)
                 w_out = blk.out2
-            h, extra = to_layer(i + 1, y=y, gate=gate, w_out=w_out)
+            h = stream_update(x, eps, count, y=y, gate=gate, w_out=w_out, w_next=into[i + 1])
             if on_layer is not None:
                 on_layer(i, x)
         return x, h

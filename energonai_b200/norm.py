@@ -60,25 +60,22 @@ def rms_residual(y, weight, eps, x, xt=None, offset=0.0, count=None, mix=None, r
     return (r_idx, r_w) if router is not None else None
 
 
-def stream_update(x, eps, count=None, src=None, src_scale=1.0, y=None, gate=None, w_out=None, w_next=None, products=None):
+def stream_update(x, eps, count=None, src=None, src_scale=1.0, y=None, gate=None, w_out=None, w_next=None):
     """The residual step of blocks that normalise in front of and behind a sublayer; x [n1, n2] fp32 in
     place:  x = src_scale * src (if src is given);  x += norm(y * sigmoid(gate)) * w_out (if y is; w_out
-    fp32);  h = norm(x) * w_next (if w_next is);  products [P, n2]: also h @ products.T in fp32.
-    Returns (h, products' result), None for what was not asked for."""
-    require_cuda(x, src, y, gate, w_out, w_next, products)
+    fp32);  returns h = norm(x) * w_next (None without w_next)."""
+    require_cuda(x, src, y, gate, w_out, w_next)
     n1, n2 = x.shape
     t = next((a for a in (src, y, w_next) if a is not None), None)
-    if t is None or x.dtype != torch.float32 or any(a is not None and a.dtype != t.dtype for a in (src, y, gate, w_next, products)):
+    if t is None or x.dtype != torch.float32 or any(a is not None and a.dtype != t.dtype for a in (src, y, gate, w_next)):
         raise RuntimeError("stream_update: x is fp32, the other rows and weights share a dtype")
-    if any(a is not None and tuple(a.shape) != (n1, n2) for a in (src, y, gate)) or any(a is not None and a.shape[-1] != n2 for a in (w_out, w_next, products)):
+    if any(a is not None and tuple(a.shape) != (n1, n2) for a in (src, y, gate)) or any(a is not None and a.shape[-1] != n2 for a in (w_out, w_next)):
         raise RuntimeError("stream_update: everything is [rows, width] of one width")
-    if w_out is not None and w_out.dtype != torch.float32 or products is not None and not products.is_contiguous():
-        raise RuntimeError("stream_update: w_out is fp32, the products' weight contiguous")
+    if w_out is not None and w_out.dtype != torch.float32:
+        raise RuntimeError("stream_update: w_out is fp32")
     h = torch.empty((n1, n2), dtype=t.dtype, device=x.device) if w_next is not None else None
-    out = torch.empty((n1, products.shape[0]), dtype=torch.float32, device=x.device) if products is not None else None
     ld = lambda a, what: _rows(a, f"stream_update: {what}") if a is not None else 0
     check(lib().eb_stream_update(ptr(src), ld(src, "src"), float(src_scale), ptr(y), ld(y, "y"), ptr(gate), ld(gate, "gate"), ptr(w_out), ptr(x),
-                                 ld(x, "x"), ptr(w_next), ptr(h), n2, ptr(products), products.shape[0] if products is not None else 0, ptr(out),
-                                 out.shape[1] if out is not None else 0, float(eps), n1, n2, count or n2, dtype_code(t.dtype), stream_ptr()),
+                                 ld(x, "x"), ptr(w_next), ptr(h), n2, float(eps), n1, n2, count or n2, dtype_code(t.dtype), stream_ptr()),
           "stream_update")
-    return h, out
+    return h

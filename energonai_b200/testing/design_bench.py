@@ -1,7 +1,8 @@
-"""Throughput of the latent-attention / mixture-of-experts decoder at sizes that resemble a real
-model's layers (random weights), beside an OPT-shaped PipelineModel of equal width, heads, depth and
-active feed-forward weights, and the time of every kernel of it next to its roofline and to the like
-kernel of the other model.  `bench.py --design tulezen` prints the result as one JSON line."""
+"""Throughput of the layer-listed decoders (latent attention / mixture of experts, matrix memory / grouped
+attention) at sizes that resemble a real model's layers (random weights), beside an OPT-shaped
+PipelineModel of equal width, heads, depth and weights per token, and the time of every kernel next to
+its roofline and to the like kernel of the other model.  `bench.py --design tulezen | mutolix` prints
+the result as one JSON line."""
 import json
 import os
 import statistics
@@ -50,6 +51,33 @@ def make_opt(z, max_len):
     return m.eval()
 
 
+MUTOLIX_SIZES = {
+    # alternating matrix-memory layers (no feed-forward) and attention layers (with one); m*: the memory's heads
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, mheads=8, mdim=128, mvdim=256, ff=8192, layers=8, vocab=32768),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, mheads=16, mdim=128, mvdim=256, ff=16384, layers=6, vocab=32768),
+}
+
+
+def make_mutolix(z):
+    from ..registry import build_model
+    memory = {"type": "mlstm", "mixer": {"heads": z["mheads"], "dim": z["mdim"], "vdim": z["mvdim"], "gate_cap": 15.0}, "mlp": None}
+    attention = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"],
+                                                "scale": z["dim"] ** -0.5, "q_temp": {"coef": 0.1, "every": 512}, "v_mix": True},
+                 "mlp": {"kind": "dense", "ff": z["ff"]}}
+    torch.manual_seed(1)
+    return build_model("Mutolix", config_dict={"vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+                                               "layers": [memory, attention] * (z["layers"] // 2)}, dtype=torch.bfloat16, device="cuda")
+
+
+def mutolix_as_opt(z):
+    """The feed-forward size with which an OPT layer has as many weights as a layer here has on average."""
+    w, h = z["width"], z["heads"] * z["dim"]
+    memory = w * (2 * z["mheads"] * z["mdim"] + 3 * z["mheads"] * z["mvdim"] + w)
+    attention = w * (2 * h + 2 * z["kv_heads"] * z["dim"] + 2 * w + 2 * z["ff"])
+    ffn = ((memory + attention) / 2 / w - 4 * w) / 2
+    return dict(z, top=1, ff=int(ffn / 1.5))
+
+
 def timed_generation(model, vocab, B, S, new, reps=3):
     ids = torch.randint(0, vocab, (B, S), device="cuda")
     mask = torch.ones_like(ids)
@@ -68,7 +96,8 @@ def timed_generation(model, vocab, B, S, new, reps=3):
 
 def time_calls(calls, reps=10):
     """Median time of one call, from replays of a graph that runs all of `calls` (operand copies that
-    together exceed L2) back to back."""
+    together exceed L2) back to back, at least eight of them."""
+    calls = list(calls) * -(-8 // len(calls))
     for c in calls[:2]:
         c()
     torch.cuda.synchronize()
@@ -208,6 +237,125 @@ def kernel_table(z, B, S, T):
     return rows, {"active_experts": act_e, "sorted_rows": live, "routed_rows": T * K}
 
 
+def mutolix_kernel_table(z, B, S, T):
+    """As kernel_table, for the matrix-memory / grouped-attention decoder."""
+    from ..attention import (attention_decode, attention_group_decode, attention_inputs, attention_prefill, attention_prefill_biased, distance_bias)
+    from ..gemm import gemm, project_parts
+    from ..kernel.cuda_native.layer_norm import layer_norm_forward
+    from ..memory import head_norm_gate, memory_prompt, memory_step
+    from ..norm import stream_update
+    bf, dev = torch.bfloat16, "cuda"
+    W, H, G, d, ff = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
+    MH, md, mv = z["mheads"], z["mdim"], z["mvdim"]
+    rnd = lambda *s, dtype=bf: (torch.randn(*s, device=dev, dtype=torch.float32) * 0.05).to(dtype)
+    rows = []
+
+    def add(phase, name, like, us, nbytes, flops=0.0):
+        rows.append((phase, name, like, us, float(nbytes), float(flops)))
+
+    def product(phase, name, M, N, Kd, like=None, act=None, xielu=0, tail=0):
+        N += tail
+        nb = 2 * (N * Kd + M * Kd) + 2 * M * (N + tail)
+        ws = [rnd(N, Kd) for _ in range(copies(2 * N * Kd, 32))]
+        xs = [rnd(M, Kd) for _ in range(4)]
+        bias, par = rnd(N), torch.tensor([0.7, 0.9], device=dev)
+        if xielu or tail:
+            call = lambda w, x: project_parts(x, w, bias=bias, xielu=(par, xielu) if xielu else None, tail_col=N - tail if tail else None)
+        else:
+            call = lambda w, x: gemm(x, w, bias=bias if act else None, act=act, static_weight=True)
+        us = time_calls([lambda w=w, x=xs[i % 4]: call(w, x) for i, w in enumerate(ws)])
+        add(phase, name, like, us, nb, 2.0 * M * N * Kd)
+
+    qk, vg = MH * md, MH * mv
+    n_mem, n_att = 2 * qk + 2 * vg + W, (H + 2 * G) * d + W
+    nw, w32, lw, lb = rnd(W), torch.ones(W, device=dev), rnd(W), rnd(W)
+    bias_h = tuple(torch.rand(H, device=dev) for _ in range(2))
+    mbias = tuple(torch.zeros(MH, device=dev) + x for x in (0.0, 4.0))
+
+    # ---- generation step ----
+    product("step", "gemm in_proj (memory)", B, n_mem, W, tail=-(-2 * MH // 8) * 8)
+    product("step", "gemm in_proj (attention)", B, n_att, W)
+    product("step", "gemm out_proj", B, W, H * d)
+    product("step", "gemm up + xielu", B, ff + W, W, like="gemm fc1 relu (OPT)", xielu=ff)
+    product("step", "gemm fc1 relu (OPT)", B, ff + W, W, act="relu")
+    product("step", "gemm down", B, W, ff)
+    nb = 8 * B * MH * (md * mv + md)
+    states = [[rnd(B, MH, md, mv, dtype=torch.float32), rnd(B, MH, md, dtype=torch.float32), torch.zeros(B, MH, device=dev)] for _ in range(copies(nb / 2))]
+    row = rnd(B, 2 * qk + 2 * vg)
+    gates, mnorm = rnd(B, 2 * MH, dtype=torch.float32), rnd(vg)
+    q, k, v, g = row.split([qk, qk, vg, vg], 1)
+    add("step", "memory_step", "attention_decode (OPT)", time_calls([lambda s=s: memory_step(q, k, v, g, gates, mbias, 15.0, md ** -0.5, mnorm, mv, 1e-6, s, MH)
+                                                                     for s in states]), nb + 2 * B * (2 * qk + 3 * vg))
+    del states
+    pos = torch.tensor([S - 1], dtype=torch.int32, device=dev)
+    kv = [rnd(B, S, 2 * G * d) for _ in range(copies(B * S * 2 * G * d * 2))]
+    qr = rnd(B, H * d)
+    add("step", "attention_group_decode", "attention_decode (OPT)", time_calls([lambda c=c: attention_group_decode(
+        qr, c[:, :, :G * d], c[:, :, G * d:], d, pos, 0.09, bias=bias_h) for c in kv]), 4 * B * S * G * d + 4 * B * H * d)
+    pr, qn, kn, lam = rnd(B, n_att), rnd(H * d), rnd(G * d), torch.full((1,), 0.5, device=dev)
+    add("step", "attention_inputs", "layer_norm (OPT)", time_calls([lambda c=c: attention_inputs(
+        pr, H, G, d, d, qn, H * d, kn, G * d, 1e-6, c[:, :, :G * d], c[:, :, G * d:], 1, temp=(0.1, 512), vmix=lam, v_first=kv[0][:, :, G * d:],
+        pos_device=pos) for c in kv[1:]]), 4 * B * (H + 2 * G) * d + 2 * B * G * d)
+    del kv
+    kv = [rnd(B, S, 3 * H * d) for _ in range(copies(B * S * 2 * H * d * 2))]
+    add("step", "attention_decode (OPT)", None, time_calls([lambda c=c: attention_decode(
+        c[:, :, 2 * H * d:], c[:, :, :H * d], c[:, :, H * d:2 * H * d], d, S, q_in_cache=True) for c in kv]), 4 * B * S * H * d)
+    del kv
+    x, y, gr = torch.randn(B, W, device=dev), rnd(B, W), rnd(B, n_mem)[:, :W]
+    add("step", "stream_update", "layer_norm (OPT)", time_calls([lambda: stream_update(x, 1e-6, y=y, gate=gr, w_out=w32, w_next=nw)] * 16), 14 * B * W)
+    xt = rnd(B, W)
+    add("step", "layer_norm (OPT)", None, time_calls([lambda: layer_norm_forward(xt, lw, lb, 1e-5)] * 16), 4 * B * W)
+
+    # ---- prompt ----
+    seq = min(S, T)
+    nB = T // seq
+    product("prompt", "gemm in_proj (memory)", T, n_mem, W, tail=-(-2 * MH // 8) * 8)
+    product("prompt", "gemm in_proj (attention)", T, n_att, W)
+    product("prompt", "gemm out_proj", T, W, H * d)
+    product("prompt", "gemm up + xielu", T, ff + W, W, like="gemm fc1 relu (OPT)", xielu=ff)
+    product("prompt", "gemm fc1 relu (OPT)", T, ff + W, W, act="relu")
+    product("prompt", "gemm down", T, W, ff)
+    projs = [rnd(T, n_mem) for _ in range(3)]
+    gates = rnd(T, 2 * MH, dtype=torch.float32)
+    state = [torch.empty(nB, MH, md, mv, device=dev), torch.empty(nB, MH, md, device=dev), torch.empty(nB, MH, device=dev)]
+    add("prompt", "memory_chunks", "attention causal (OPT)", time_calls([lambda r=r: memory_prompt(
+        *r[:, :2 * qk + vg].split([qk, qk, vg], 1), gates, mbias, 15.0, md ** -0.5, state, MH, chunked=True) for r in projs]),
+        4 * T * (qk + vg) + 8 * T * MH + 4 * nB * MH * md * mv, 4.0 * T * MH * md * mv)
+    os_ = [rnd(T, vg) for _ in range(4)]
+    add("prompt", "head_norm_gate", "layer_norm (OPT)", time_calls([lambda o=o: head_norm_gate(o, projs[0][:, 2 * qk + vg:2 * qk + 2 * vg], mnorm, MH, mv, 1e-6)
+                                                                    for o in os_]), 6 * T * vg)
+    del projs, os_
+    projs = [rnd(T, n_att) for _ in range(3)]
+    caches = [rnd(nB, seq, 2 * G * d) for _ in range(2)]
+    kc, vc = caches[0][:, :, :G * d], caches[0][:, :, G * d:]
+    add("prompt", "attention_inputs", "layer_norm (OPT)", time_calls([lambda r=r: attention_inputs(
+        r, H, G, d, d, qn, H * d, kn, G * d, 1e-6, kc, vc, seq, temp=(0.1, 512), vmix=lam, v_first=caches[1][:, :, G * d:]) for r in projs]),
+        4 * T * (H + 2 * G) * d + 2 * T * G * d)
+    del projs
+    q3, kv3 = rnd(nB, seq, H * d), rnd(nB, seq, 2 * H * d)
+    flops = 4.0 * nB * H * d * seq * (seq + 1) / 2
+    add("prompt", "attention biased", "attention causal (OPT)", time_calls([lambda: attention_prefill_biased(q3, kc, vc, d, table)] * 4)
+        if (table := distance_bias(*bias_h, seq)) is not None else 0.0, 2 * T * (2 * H + 2 * G) * d, flops)
+    add("prompt", "distance_bias", None, time_calls([lambda: distance_bias(*bias_h, seq)] * 8), 4 * H * (seq + 256))
+    add("prompt", "attention causal (OPT)", None, time_calls([lambda: attention_prefill(q3, kv3[:, :, :H * d], kv3[:, :, H * d:], d)] * 4),
+        2 * T * 4 * H * d, flops)
+    del q3, kv3, caches
+    xs = [torch.randn(T, W, device=dev) for _ in range(copies(14 * T * W, 8))]
+    ys = [rnd(T, W) for _ in xs]
+    gs = [rnd(T, n_att)[:, -W:] for _ in range(2)]
+    add("prompt", "stream_update", "layer_norm (OPT)", time_calls([lambda x=x, y=y, g=gs[i % 2]: stream_update(x, 1e-6, y=y, gate=g, w_out=w32, w_next=nw)
+                                                                   for i, (x, y) in enumerate(zip(xs, ys))]), 14 * T * W)
+    lns = [rnd(T, W) for _ in range(copies(4 * T * W, 8))]
+    add("prompt", "layer_norm (OPT)", None, time_calls([lambda t=t: layer_norm_forward(t, lw, lb, 1e-5) for t in lns]), 4 * T * W)
+    return rows, {}
+
+
+DESIGNS = {
+    "tulezen": dict(sizes=SIZES, runs=RUNS, make=make_tulezen, as_opt=lambda z: z, table=kernel_table),
+    "mutolix": dict(sizes=MUTOLIX_SIZES, runs=RUNS, make=make_mutolix, as_opt=mutolix_as_opt, table=mutolix_kernel_table),
+}
+
+
 def table_with_fractions(rows):
     pk = peaks()
     out = []
@@ -223,21 +371,22 @@ def table_with_fractions(rows):
     return out
 
 
-def run(kernels=True, generation=True):
+def run(design="tulezen", kernels=True, generation=True):
     from ..gemm import device_status
-    res = {"design": "tulezen", "dtype": "bf16", "data": "synthetic, random weights", "peaks": peaks(), "sizes": SIZES, "generation": [],
+    D = DESIGNS[design]
+    res = {"design": design, "dtype": "bf16", "data": "synthetic, random weights", "peaks": peaks(), "sizes": D["sizes"], "generation": [],
            "kernels": {}}
     if kernels:
         with torch.inference_mode():
             for (name, B, S, T) in (("2048", 64, 2048, 8192), ("4096", 16, 4096, 8192)):
-                rows, info = kernel_table(SIZES[name], B, S, T)
+                rows, info = D["table"](D["sizes"][name], B, S, T)
                 res["kernels"][f"width {name}, batch {B}, {S} positions, {T} prompt tokens"] = dict(info, table=table_with_fractions(rows))
                 torch.cuda.empty_cache()
     if generation:
-        for name, B, S, new in RUNS:
-            z = SIZES[name]
+        for name, B, S, new in D["runs"]:
+            z = D["sizes"][name]
             line = {"size": name, "batch": B, "prompt": S, "new_tokens": new}
-            for what, make in (("tulezen", lambda: make_tulezen(z)), ("opt", lambda: make_opt(z, S + new))):
+            for what, make in ((design, lambda: D["make"](z)), ("opt", lambda: make_opt(D["as_opt"](z), S + new))):
                 model = make()
                 line[what] = timed_generation(model, z["vocab"], B, S, new)
                 model._decode_state = None

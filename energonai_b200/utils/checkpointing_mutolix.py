@@ -65,9 +65,9 @@ def processing_Mutolix(state_dict, model):
         H = m.heads
         q, k = (heads(rows(take(p + n, H * m.dim, w)), H, m.dim, at.dk) for n in ("q", "k"))
         v, g = (heads(rows(take(p + n, H * m.vdim, w)), H, m.vdim, at.dv) for n in ("v", "g"))
-        out[o + "in_proj"] = torch.cat([q, k, v, g, gate])
-        out[o + "bias"] = torch.cat([torch.zeros(at.in_proj.shape[0] - W, dtype=gate_bias.dtype), gate_bias])
-        out[o + "gates"] = _pad(torch.cat([take(p + "i", H, w), take(p + "f", H, w)]), *at.gates.shape)
+        gates = _pad(torch.cat([take(p + "i", H, w), take(p + "f", H, w)]), at.in_proj.shape[0] - at.tail, W)
+        out[o + "in_proj"] = torch.cat([q, k, v, g, gate, gates])
+        out[o + "bias"] = torch.cat([gate_bias.new_zeros(at.tail - W), gate_bias, gate_bias.new_zeros(gates.shape[0])])
         out[o + "gate_bias"] = torch.stack([take(p + "i.b", H), take(p + "f.b", H)])
         out[o + "norm"] = heads(take(p + "norm", H * m.vdim), H, m.vdim, at.dv)
         out[o + "out_proj"] = columns(take(p + "o", w, H * m.vdim), H, m.vdim, at.dv)

@@ -46,7 +46,7 @@ extern "C" {
 #define EB_ACT_RELU 1
 #define EB_ACT_GELU_TANH 2 /* energonai/model/model_factory.py:32-35 (gelu_impl)            */
 #define EB_ACT_GELU_ERF 3  /* torch.nn.functional.gelu                                      */
-#define EB_ACT_XIELU 4     /* eb_gemm_xielu, eb_gemm_f32                                    */
+#define EB_ACT_XIELU 4     /* eb_gemm_parts, eb_gemm_f32                                    */
 
 /* flags for eb_gemm */
 #define EB_GEMM_STATIC_W 1 /* W is constant (model weights): the kernel may start reading it while
@@ -251,13 +251,15 @@ EB_API int eb_gemm(const void *A, long long lda, const void *W, long long ldw, v
             int c_row_offset_limit, int flags, void *workspace, size_t workspace_bytes, void *stream);
 EB_API size_t eb_gemm_workspace_bytes(int M, int N, int K);
 
-/* eb_gemm (no residual, plain rows) whose activation is xIELU on the columns below act_cols, a
- * multiple of 8; the other columns get their bias only.  act_params: device floats
+/* eb_gemm (no residual, plain rows) for several things at once that read the same A, their weights
+ * stacked in W.  act_params (or NULL): xIELU on the columns below act_cols, a multiple of 8; device floats
  * (softplus(p), 1/2 + softplus(q)) of
- *   z > 0: softplus(p) z^2 + z/2;   z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2. */
-EB_API int eb_gemm_xielu(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, const void *bias,
-                  int M, int N, int K, int act_cols, const float *act_params, int dtype, int out_dtype, int flags,
-                  void *workspace, size_t workspace_bytes, void *stream);
+ *   z > 0: softplus(p) z^2 + z/2;   z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2.
+ * tail (or NULL): the columns from tail_col on, a multiple of 8, go there in fp32, rows ld_tail apart;
+ * C then holds the tail_col columns before them.  bias [N] or NULL. */
+EB_API int eb_gemm_parts(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, const void *bias,
+                  int M, int N, int K, int act_cols, const float *act_params, int tail_col, float *tail, long long ld_tail,
+                  int dtype, int flags, void *workspace, size_t workspace_bytes, void *stream);
 
 /* Row-parallel GEMM with the tensor-parallel all-reduce fused into its epilogue, for the
  * generation orientation (M <= 128).  Replaces "F.linear, then dist.all_reduce, then + bias" of
@@ -370,7 +372,7 @@ EB_API int eb_grouped_skinny(const void *A, long long lda, long long a_group_str
 
 /* C = A . W^T in true 32-bit.  Strided groups, or row tiles with their group (one of the two).  A single
  * product may add bias [N] and apply xIELU to the columns below act_cols (act_params as
- * eb_gemm_xielu; either NULL: left out). */
+ * eb_gemm_parts; either NULL: left out). */
 EB_API int eb_gemm_f32(const float *A, long long lda, long long a_group_stride, const float *W, long long ldw,
                 long long w_group_stride, float *C, long long ldc, long long c_group_stride, int M, int N, int K, int groups,
                 const int32_t *tile_group, const int32_t *live_tiles, const float *bias, int act_cols, const float *act_params,
@@ -424,12 +426,10 @@ EB_API int eb_rms_residual(const void *y, long long ldy, int dtype, const int32_
  * (means over the first `count`; norm(z) = z / sqrt(mean(z^2) + eps)):
  *   x = src_scale * src          if src (the embedding rows, `dtype`), else x as it is (fp32)
  *   x += norm(y * sigmoid(gate)) * w_out        if y  (gate NULL: 1; w_out fp32)
- *   h = norm(x) * w_next                        if w_next; h in `dtype`
- *   proj_out[row][e] = h . proj[e], e < n_proj  if proj; h as rounded, fp32 results */
+ *   h = norm(x) * w_next                        if w_next; h in `dtype` */
 EB_API int eb_stream_update(const void *src, long long lds, float src_scale, const void *y, long long ldy, const void *gate,
                      long long ldg, const float *w_out, float *x, long long ldx, const void *w_next, void *h, long long ldh,
-                     const void *proj, int n_proj, float *proj_out, long long ldp, float eps, int n1, int n2, int count,
-                     int dtype, void *stream);
+                     float eps, int n1, int n2, int count, int dtype, void *stream);
 
 /* Queries, keys and values of a projected row [q: heads*dk | k: kv_heads*dk | v: kv_heads*dv] made ready
  * for attention.  q and k are divided by the root mean square over ALL their rows (counts q_count and

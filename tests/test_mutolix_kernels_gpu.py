@@ -23,13 +23,20 @@ def rel(got, want):
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16, torch.float16])
 @pytest.mark.parametrize("M,N,K,cols", [(1, 48, 40, 24), (17, 136, 264, 136), (32, 72, 64, 0), (64, 264, 96, 128), (300, 520, 200, 264)])
 def test_product_with_bias_and_xielu_on_its_first_columns(dtype, M, N, K, cols):
-    from energonai_b200.gemm import project, xielu_params
+    from energonai_b200.gemm import project_parts, xielu_params
     x, w, b = rnd(M, K, seed=1).to(dtype), rnd(N, K, seed=2, scale=K ** -0.5).to(dtype), rnd(N, seed=3).to(dtype)
     act = xielu_params(0.7, -1.1)
-    got = project(x.cuda(), w.cuda(), bias=b.cuda(), xielu=(act.cuda(), cols))
     z = x.double() @ w.double().T + b.double()
-    z[:, :cols] = P.xielu(z[:, :cols], torch.tensor(0.7, dtype=torch.float64), torch.tensor(-1.1, dtype=torch.float64))
-    assert got.dtype == dtype and rel(got, z) < {torch.float32: 1e-6, torch.bfloat16: 6e-3, torch.float16: 1e-3}[dtype]
+    want = z.clone()
+    want[:, :cols] = P.xielu(z[:, :cols], torch.tensor(0.7, dtype=torch.float64), torch.tensor(-1.1, dtype=torch.float64))
+    tol = {torch.float32: 1e-6, torch.bfloat16: 6e-3, torch.float16: 1e-3}[dtype]
+    got = project_parts(x.cuda(), w.cuda(), bias=b.cuda(), xielu=(act.cuda(), cols))
+    assert got.dtype == dtype and rel(got, want) < tol
+    # the last columns in fp32, with and without activation
+    got, tail = project_parts(x.cuda(), w.cuda(), bias=b.cuda(), xielu=(act.cuda(), cols), tail_col=N - 16)
+    assert tail.dtype == torch.float32 and rel(got, want[:, :N - 16]) < tol and rel(tail, want[:, N - 16:]) < (1e-6 if dtype == torch.float32 else 2e-6 if cols <= N - 16 else 1e-4)
+    got, tail = project_parts(x.cuda(), w.cuda(), tail_col=8)
+    assert rel(got, z[:, :8] - b.double()[:8]) < tol and rel(tail, z[:, 8:] - b.double()[8:]) < 2e-6
 
 
 # ---- norms around a sublayer ----------------------------------------------------------------------------
@@ -39,28 +46,27 @@ def test_stream_update(dtype, rows, width, count):
     from energonai_b200.norm import stream_update
     pad = lambda t: torch.nn.functional.pad(t, (0, width - count))
     y, g, src, x0 = (pad(rnd(rows, count, seed=s)).to(dtype) for s in (1, 2, 3, 4))
-    wo, wn, pr = pad(1 + rnd(count, seed=5)), pad(1 + rnd(count, seed=6)).to(dtype), pad(rnd(11, count, seed=7)).to(dtype)
+    wo, wn = pad(1 + rnd(count, seed=5)), pad(1 + rnd(count, seed=6)).to(dtype)
     eps, tol = 1e-3, 3e-6 if dtype == torch.float32 else 6e-3
     d = lambda t: t[..., :count].double()
     dev = lambda t: t.cuda()
     # start of the stream
     x = torch.empty(rows, width, device="cuda")
-    h, z = stream_update(x, eps, count, src=dev(src), src_scale=2.5, w_next=dev(wn), products=dev(pr))
+    h = stream_update(x, eps, count, src=dev(src), src_scale=2.5, w_next=dev(wn))
     want = d(src) * 2.5
     assert rel(x[:, :count], want) < 1e-6 and float(x[:, count:].abs().sum()) == 0
     want_h = P.rms_norm(want, d(wn), eps)
     assert rel(h[:, :count], want_h) < tol
-    assert z.dtype == torch.float32 and rel(z, h[:, :count].double().cpu() @ d(pr).T) < 1e-5
     # between two sublayers, with and without gate
     for gate in (g, None):
         x = x0.float().cuda()
-        h, z = stream_update(x, eps, count, y=dev(y), gate=dev(gate) if gate is not None else None, w_out=dev(wo), w_next=dev(wn))
+        h = stream_update(x, eps, count, y=dev(y), gate=dev(gate) if gate is not None else None, w_out=dev(wo), w_next=dev(wn))
         s = d(y) * torch.sigmoid(d(gate)) if gate is not None else d(y)
         want = d(x0) + P.rms_norm(s, d(wo), eps)
-        assert z is None and rel(x[:, :count], want) < 3e-6 and rel(h[:, :count], P.rms_norm(want, d(wn), eps)) < tol
+        assert rel(x[:, :count], want) < 3e-6 and rel(h[:, :count], P.rms_norm(want, d(wn), eps)) < tol
     # the last one
     x = x0.float().cuda()
-    assert stream_update(x, eps, count, y=dev(y), gate=dev(g), w_out=dev(wo)) == (None, None)
+    assert stream_update(x, eps, count, y=dev(y), gate=dev(g), w_out=dev(wo)) is None
     assert rel(x[:, :count], d(x0) + P.rms_norm(d(y) * torch.sigmoid(d(g)), d(wo), eps)) < 3e-6
 
 
