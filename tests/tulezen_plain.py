@@ -145,7 +145,7 @@ def save_safetensors(path, tensors):
     names = {torch.bfloat16: "BF16", torch.float32: "F32", torch.float16: "F16", torch.int32: "I32", torch.int64: "I64"}
     head, blobs, at = {}, [], 0
     for k, v in tensors.items():
-        raw = v.contiguous().view(torch.uint8).numpy().tobytes() if v.numel() else b""
+        raw = v.contiguous().reshape(-1).view(torch.uint8).numpy().tobytes() if v.numel() else b""
         head[k] = {"dtype": names[v.dtype], "shape": list(v.shape), "data_offsets": [at, at + len(raw)]}
         blobs.append(raw)
         at += len(raw)
