@@ -6,6 +6,7 @@ the result as one JSON line."""
 import json
 import os
 import statistics
+import time
 
 import torch
 
@@ -105,6 +106,7 @@ def time_calls(calls, reps=10):
     with torch.cuda.graph(g):
         for c in calls:
             c()
+    time.sleep(0.3)              # a kernel timed right behind a run of large products would find the clock lowered by the power cap
     ts = []
     for i in range(reps + 3):
         a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
