@@ -119,14 +119,22 @@ def attention_prefill_window(q, k, v, head_dim, window, mask=None, scale=None, o
     return out
 
 
+def _check_sinks(sinks, heads):
+    require_cuda(sinks)
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != heads or not sinks.is_contiguous()):
+        raise RuntimeError("attention: one fp32 sink per query head")
+
+
 def attention_plain(q, k, v, heads, k_dim, v_dim, window=0, scale=1.0, first=None, pos_device=None, shared_kv=False,
-                    kv_heads=None, bias=None, sink=False):
+                    kv_heads=None, bias=None, sink=False, chunk=None, sinks=None):
     """Windowed causal attention on the CUDA cores, any head sizes, fp32 / fp16 / bf16.  q [B, Sq,
     heads*k_dim]; k / v [B, rows, heads*dim] or, with shared_kv, [B, rows, dim] shared by the heads.
     Query row i holds position pos_device + i (None: i), the key of position j is row j mod rows;
     first [B] int32 is each sequence's first position.  kv_heads: heads of k / v, each shared by
     heads / kv_heads query heads.  bias = (r1, r2), fp32 per query head: r1 * ln(1 + r2 * distance) is
-    taken off the scaled score.  sink: one is added to the softmax denominator.  Returns [B, Sq, heads*v_dim]."""
+    taken off the scaled score.  sink: one is added to the softmax denominator.  chunk (0: none; instead of
+    window and bias): a position sees only its own chunk of so many, counted from first; sinks fp32 [heads] or
+    None: exp of it joins the denominator.  Returns [B, Sq, heads*v_dim]."""
     r1, r2 = bias if bias is not None else (None, None)
     require_cuda(q, k, v, first, pos_device, r1, r2)
     if bias is not None and any(r.dtype != torch.float32 or r.numel() != heads or not r.is_contiguous() for r in bias):
@@ -136,6 +144,15 @@ def attention_plain(q, k, v, heads, k_dim, v_dim, window=0, scale=1.0, first=Non
     if any(t.stride(2) != 1 for t in (q, k, v)) or k.shape[1] != v.shape[1]:
         raise RuntimeError("attention: contiguous last dims and one number of key / value rows required")
     hk, hv = (0, 0) if shared_kv else (k_dim, v_dim)
+    if chunk is not None:
+        if bias is not None or window or sink:
+            raise RuntimeError("attention: a chunk goes without window, bias and constant sink")
+        _check_sinks(sinks, heads)
+        check(lib().eb_attention_plain_chunk(ptr(q), ptr(k), ptr(v), ptr(out), q.stride(0), q.stride(1), k_dim, k.stride(0), k.stride(1), hk,
+                                             v.stride(0), v.stride(1), hv, out.stride(0), out.stride(1), v_dim, B, heads,
+                                             heads // (kv_heads or heads), Sq, k_dim, v_dim, int(chunk), k.shape[1], ptr(pos_device), ptr(first),
+                                             ptr(sinks), float(scale), dtype_code(q.dtype), stream_ptr()), "attention_plain_chunk")
+        return out
     check(lib().eb_attention_plain(ptr(q), ptr(k), ptr(v), ptr(out), q.stride(0), q.stride(1), k_dim, k.stride(0), k.stride(1), hk,
                                    v.stride(0), v.stride(1), hv, out.stride(0), out.stride(1), v_dim, B, heads,
                                    heads // (kv_heads or heads), Sq, k_dim, v_dim, int(window), k.shape[1], ptr(pos_device), ptr(first),
@@ -261,4 +278,66 @@ def attention_group_decode(q, k, v, head_dim, pos_device, scale, first=None, bia
                                           head_dim, rows, ptr(pos_device), ptr(first), ptr(r1), ptr(r2), 1 if sink else 0, float(scale),
                                           dtype_code(q.dtype), nsplit, ptr(scratch), scratch.numel() if scratch is not None else 0,
                                           stream_ptr()), "attention_group_decode")
+    return out
+
+
+def attention_rotary(proj, heads, kv_heads, dk, dim, q_norm, k_norm, eps, freq, k_cache, v_cache, rows_per_batch, pos_device=None, first=None,
+                     keys=False):
+    """Rows [q | k | ...] of a projection -> queries [rows, heads*dk], normalised head by head over `dim` columns
+    and rotated (freq fp32: angle per position of each leading pair); keys, treated alike, and values, the
+    keys as projected, go to the ring caches.  keys: also returns the keys as rows (else None)."""
+    require_cuda(proj, q_norm, k_norm, freq, k_cache, v_cache, pos_device, first)
+    n1 = proj.shape[0]
+    if any(t.dtype != proj.dtype for t in (q_norm, k_norm, k_cache, v_cache)) or freq.dtype != torch.float32 or not freq.is_contiguous():
+        raise RuntimeError("attention_rotary: one dtype required, frequencies in fp32")
+    if proj.dim() != 2 or proj.stride(1) != 1 or q_norm.numel() != dk or k_norm.numel() != dk:
+        raise RuntimeError("attention_rotary: rows [q | k], one norm entry per column of a head")
+    B = n1 // rows_per_batch
+    for t in (k_cache, v_cache):
+        if t.dim() != 3 or t.stride(2) != 1 or t.shape[0] != B or t.shape[2] != kv_heads * dk or t.shape[1] != k_cache.shape[1]:
+            raise RuntimeError("attention_rotary: caches are [batch, rows, kv_heads*dk]")
+    q = torch.empty((n1, heads * dk), dtype=proj.dtype, device=proj.device)
+    k = torch.empty((n1, kv_heads * dk), dtype=proj.dtype, device=proj.device) if keys else None
+    check(lib().eb_attention_rotary(ptr(proj), proj.stride(0), heads, kv_heads, dk, int(dim), ptr(q_norm), ptr(k_norm), float(eps), ptr(freq),
+                                    freq.numel(), ptr(q), q.stride(0), ptr(k), k.stride(0) if keys else 0, ptr(k_cache), k_cache.stride(0),
+                                    k_cache.stride(1), ptr(v_cache), v_cache.stride(0), v_cache.stride(1), k_cache.shape[1], n1, rows_per_batch,
+                                    ptr(pos_device), ptr(first), dtype_code(proj.dtype), stream_ptr()), "attention_rotary")
+    return q, k
+
+
+def attention_prefill_chunk(q, k, v, head_dim, chunk, sinks=None, first=None, scale=None, out=None):
+    """Prompt attention (tensor-core kernel): q [B, S, H*D], k / v [B, S, G*D]; row i sees the keys up to itself in
+    its own chunk (0: no chunks) counted from first[b]; exp(sinks[h]) joins the denominator."""
+    require_cuda(q, k, v, first, out)
+    B, S, HD = q.shape
+    H, G = HD // head_dim, k.shape[2] // head_dim
+    if k.shape[1] != S or v.shape != k.shape or H % G:
+        raise RuntimeError("attention: a whole prompt with query heads in equal groups")
+    _check_sinks(sinks, H)
+    if out is None:
+        out = torch.empty((B, S, HD), dtype=q.dtype, device=q.device)
+    qs, ks, vs, os_ = (_bsh_strides(t, head_dim) for t in (q, k, v, out))
+    scale = head_dim ** -0.5 if scale is None else scale
+    check(lib().eb_attention_prefill_chunk_tc(ptr(q), ptr(k), ptr(v), ptr(out), *qs, *ks, *vs, *os_, B, H, H // G, S, head_dim, int(chunk),
+                                              ptr(first), ptr(sinks), float(scale), dtype_code(q.dtype), stream_ptr()), "attention_prefill_chunk_tc")
+    return out
+
+
+def attention_group_decode_chunk(q, k, v, head_dim, pos_device, scale, chunk, sinks=None, first=None, nsplit=None):
+    """Generation step of attention_prefill_chunk: q [B, H*D], k / v [B, rows, G*D] cache views (rings if chunk > 0),
+    pos_device int32 scalar (the query's position).  Returns [B, H*D]."""
+    require_cuda(q, k, v, pos_device, first)
+    B, HD = q.shape
+    H, G, rows = HD // head_dim, k.shape[2] // head_dim, k.shape[1]
+    _check_sinks(sinks, H)
+    ks, vs = _bsh_strides(k, head_dim), _bsh_strides(v, head_dim)
+    out = torch.empty((B, HD), dtype=q.dtype, device=q.device)
+    if nsplit is None:
+        nsplit = pick_group_nsplit(B, G * -(-(H // G) // 16), rows)
+    nbytes = lib().eb_attention_group_decode_scratch_bytes(B, H, G, head_dim, nsplit)
+    scratch = _get_scratch(q.device, nbytes) if nbytes else None
+    check(lib().eb_attention_group_decode_chunk(ptr(q), ptr(k), ptr(v), ptr(out), q.stride(0), ks[0], ks[1], vs[0], vs[1], out.stride(0), B, H, G,
+                                                head_dim, rows, int(chunk), ptr(pos_device), ptr(first), ptr(sinks), float(scale),
+                                                dtype_code(q.dtype), nsplit, ptr(scratch), scratch.numel() if scratch is not None else 0,
+                                                stream_ptr()), "attention_group_decode_chunk")
     return out

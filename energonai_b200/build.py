@@ -20,8 +20,8 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
               "-diag-suppress", "177,550"]
 # Recurrences add up the logarithms of their gates over a whole sequence: an approximation's bias would
-# add up with them, so these files get the accurate functions.
-ACCURATE = {"matrix_memory.cu", "matrix_memory_tc.cu"}
+# add up with them, so these files get the accurate functions; so do angles that grow with the position.
+ACCURATE = {"matrix_memory.cu", "matrix_memory_tc.cu", "decay_memory.cu", "decay_memory_tc.cu", "attention_rotary.cu"}
 
 
 def nvcc_flags(source):

@@ -4,7 +4,11 @@
 // 64-key tile and loads, waits for and consumes only those; two tiles are in flight per CTA.  The
 // position range of a (sequence, group) may be split over CTAs, merged by the last to arrive.
 //
-// Scores: scale q.k - r1 ln(1 + r2 distance), optionally a sink (one more in the denominator), all fp32;
+// A chunk mask (a position sees only its own chunk of so many positions, counted from the sequence's first)
+// goes with a ring cache: position p in row p mod rows.
+//
+// Scores: scale q.k - r1 ln(1 + r2 distance), optionally a sink (one more in the denominator, or exp of a
+// number per head), all fp32;
 // an attention weight is rounded once, as an operand of the value product.
 #include "attention_mma.cuh"
 
@@ -19,6 +23,8 @@ struct GroupParams {
   const void *q, *k, *v;
   void *o;
   long long q_bs, k_bs, k_rs, v_bs, v_rs, o_bs;
+  const float *sinks;                               // per head, or null (with sink: 0)
+  int chunk;                                        // RING: positions of a chunk
   int group, blocks, cache_rows, nsplit, sink;      // blocks: CTAs of up to 16 heads per group
   const int *pos_dev, *first;
   const float *r1, *r2;
@@ -28,7 +34,7 @@ struct GroupParams {
 };
 
 // WIDE: groups of more than 8 heads; else the second half of the tile's rows is not looked at.
-template <typename T, int D, bool WIDE>
+template <typename T, int D, bool WIDE, bool RING>
 __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(const GroupParams p) {
   extern __shared__ __align__(128) uint8_t smem[];
   constexpr int kTileBytes = kTile * D * 2, kLd = D + 2, kHalves = WIDE ? 2 : 1;
@@ -42,17 +48,25 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   const int split = blockIdx.x, hk = blockIdx.y / p.blocks, hb = blockIdx.y % p.blocks, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int h0 = hk * p.group + hb * kRowsPerCta, nh = min(kRowsPerCta, p.group - hb * kRowsPerCta);
-  const int pos = min(max(*p.pos_dev, 0), p.cache_rows - 1), Sk = pos + 1;
-  const int lo = p.first ? min(max(p.first[b], 0), pos) : 0;
-  const int tile_lo = lo / kTile, tiles = (Sk + kTile - 1) / kTile - tile_lo, per = (tiles + p.nsplit - 1) / p.nsplit;
-  const int tile0 = tile_lo + split * per, tile1 = min(tile_lo + tiles, tile0 + per);
+  const int pos = RING ? max(*p.pos_dev, 0) : min(max(*p.pos_dev, 0), p.cache_rows - 1), Sk = pos + 1;
+  int lo = p.first ? min(max(p.first[b], 0), pos) : 0;
+  if (RING) lo = max(lo + (pos - lo) / p.chunk * p.chunk, pos - p.cache_rows + 1);
+  // tile n holds the positions from base + 64 n on
+  const int base = RING ? lo : lo / kTile * kTile, tiles = (Sk - base + kTile - 1) / kTile, per = (tiles + p.nsplit - 1) / p.nsplit;
+  const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
+  const int r0 = RING ? base % p.cache_rows : 0;
 
   const T *qb = reinterpret_cast<const T *>(p.q) + b * p.q_bs + (long long)h0 * D;
   const T *kb = reinterpret_cast<const T *>(p.k) + b * p.k_bs + hk * D;
   const T *vb = reinterpret_cast<const T *>(p.v) + b * p.v_bs + hk * D;
   auto load_kv = [&](int n, int buf) {
-    load_warp_rows<T, D>(k_s + buf * kTileBytes, kb, p.k_rs, n * kTile, Sk, warp, lane);
-    load_warp_rows<T, D>(v_s + buf * kTileBytes, vb, p.v_rs, n * kTile, Sk, warp, lane);
+    if (RING) {
+      load_warp_ring<T, D>(k_s + buf * kTileBytes, kb, p.k_rs, n * kTile, Sk - base, r0, p.cache_rows, warp, lane);
+      load_warp_ring<T, D>(v_s + buf * kTileBytes, vb, p.v_rs, n * kTile, Sk - base, r0, p.cache_rows, warp, lane);
+      return;
+    }
+    load_warp_rows<T, D>(k_s + buf * kTileBytes, kb, p.k_rs, base + n * kTile, Sk, warp, lane);
+    load_warp_rows<T, D>(v_s + buf * kTileBytes, vb, p.v_rs, base + n * kTile, Sk, warp, lane);
   };
   for (int i = 0; i < kStages - 1; ++i) {
     if (tile0 + i < tile1) load_kv(tile0 + i, i);
@@ -102,7 +116,7 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int j = n * kTile + warp * 16 + i * 8 + 2 * t + e;
+          const int j = base + n * kTile + warp * 16 + i * 8 + 2 * t + e;
           float x = s[i][2 * r + e] * p.scale_log2 - r1[r] * log2f(fmaf(r2[r], (float)max(pos - j, 0), 1.f));
           if (j > pos || j < lo || !row_ok[r]) x = -INFINITY;
           s[i][2 * r + e] = x;
@@ -155,11 +169,13 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   }
   __syncthreads();
   // row by row: the parts of the warps, or of the splits, in one scale; the sink joins the last merge
+  auto sink_score = [&](int row) { return !p.sink ? -INFINITY : p.sinks ? p.sinks[h0 + row] * kLog2eGroup : 0.f; };
   auto merge = [&](const float *parts, int count, long long stride, int row, int d, bool sink, float &m_out, float &l_out) {
-    float m = sink ? 0.f : -INFINITY;
+    const float sc = sink ? sink_score(row) : -INFINITY;
+    float m = sc;
     for (int i = 0; i < count; ++i) m = fmaxf(m, __ldcg(parts + i * stride + row * kLd + D));
     const float ref = m == -INFINITY ? 0.f : m;
-    float l = sink ? exp2f(-ref) : 0.f, acc = 0.f;
+    float l = exp2f(sc - ref), acc = 0.f;
     for (int i = 0; i < count; ++i) {
       const float w = exp2f(__ldcg(parts + i * stride + row * kLd + D) - ref);
       l = fmaf(__ldcg(parts + i * stride + row * kLd + D + 1), w, l);
@@ -175,11 +191,12 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   for (int i = threadIdx.x; i < nh * D; i += kGroupThreads) {
     const int row = i / D, d = i % D;
     // (shared memory: plain loads)
-    float m = p.nsplit == 1 && p.sink ? 0.f : -INFINITY;
+    const float sc = p.nsplit == 1 ? sink_score(row) : -INFINITY;
+    float m = sc;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, red[(w * kRowsPerCta + row) * kLd + D]);
     const float ref = m == -INFINITY ? 0.f : m;
-    float l = p.nsplit == 1 && p.sink ? exp2f(-ref) : 0.f, acc = 0.f;
+    float l = exp2f(sc - ref), acc = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float *part = red + (w * kRowsPerCta + row) * kLd;
@@ -212,9 +229,9 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   }
 }
 
-template <typename T, int D, bool WIDE> int launch_group_as(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
+template <typename T, int D, bool WIDE, bool RING> int launch_group_as(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
   constexpr size_t smem = 2 * kStages * (size_t)kTile * D * 2;
-  auto kern = attention_group_decode_kernel<T, D, WIDE>;
+  auto kern = attention_group_decode_kernel<T, D, WIDE, RING>;
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -230,7 +247,8 @@ template <typename T, int D, bool WIDE> int launch_group_as(const GroupParams &p
 }
 
 template <typename T, int D> int launch_group(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
-  return p.group > 8 ? launch_group_as<T, D, true>(p, kv_heads, B, st) : launch_group_as<T, D, false>(p, kv_heads, B, st);
+  if (p.chunk > 0) return p.group > 8 ? launch_group_as<T, D, true, true>(p, kv_heads, B, st) : launch_group_as<T, D, false, true>(p, kv_heads, B, st);
+  return p.group > 8 ? launch_group_as<T, D, true, false>(p, kv_heads, B, st) : launch_group_as<T, D, false, false>(p, kv_heads, B, st);
 }
 
 inline int head_blocks(int heads, int kv_heads) { return (heads / kv_heads + kRowsPerCta - 1) / kRowsPerCta; }
@@ -245,11 +263,12 @@ extern "C" size_t eb_attention_group_decode_scratch_bytes(int batch, int heads, 
   return kCounterSlots * sizeof(int) + (size_t)batch * kv_heads * head_blocks(heads, kv_heads) * nsplit * kRowsPerCta * (head_dim + 2) * sizeof(float);
 }
 
-extern "C" int eb_attention_group_decode(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+static int group_decode_impl(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
                                          long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
                                          long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int cache_rows,
                                          const int32_t *pos_device, const int32_t *first, const float *bias_r1, const float *bias_r2, int sink,
-                                         float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes, void *stream) {
+                                         const float *sinks, int chunk, float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes,
+                                         void *stream) {
   if (batch == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "attention_group_decode: fp16 or bf16 only (dtype %d)", dtype);
   EB_REQUIRE(head_dim == 64 || head_dim == 128, "attention_group_decode: head_dim %d not supported (64 or 128)", head_dim);
@@ -263,7 +282,7 @@ extern "C" int eb_attention_group_decode(const void *q, const void *k, const voi
   GroupParams p{};
   p.q = q; p.k = k; p.v = v; p.o = out; p.q_bs = q_batch_stride; p.k_bs = k_batch_stride; p.k_rs = k_row_stride; p.v_bs = v_batch_stride;
   p.v_rs = v_row_stride; p.o_bs = out_batch_stride; p.group = heads / kv_heads; p.blocks = head_blocks(heads, kv_heads);
-  p.cache_rows = cache_rows; p.nsplit = nsplit; p.sink = sink; p.pos_dev = pos_device; p.first = first; p.r1 = bias_r1; p.r2 = bias_r2;
+  p.cache_rows = cache_rows; p.nsplit = nsplit; p.sink = sink; p.sinks = sinks; p.chunk = chunk; p.pos_dev = pos_device; p.first = first; p.r1 = bias_r1; p.r2 = bias_r2;
   p.scale_log2 = scale * kLog2eGroup;
   EB_REQUIRE((long long)kv_heads * p.blocks <= 65535, "attention_group_decode: too many heads");
   if (nsplit > 1) {
@@ -276,4 +295,25 @@ extern "C" int eb_attention_group_decode(const void *q, const void *k, const voi
   cudaStream_t st = as_stream(stream);
   if (dtype == EB_F16) return head_dim == 64 ? launch_group<__half, 64>(p, kv_heads, batch, st) : launch_group<__half, 128>(p, kv_heads, batch, st);
   return head_dim == 64 ? launch_group<__nv_bfloat16, 64>(p, kv_heads, batch, st) : launch_group<__nv_bfloat16, 128>(p, kv_heads, batch, st);
+}
+
+extern "C" int eb_attention_group_decode(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+                                         long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                                         long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int cache_rows,
+                                         const int32_t *pos_device, const int32_t *first, const float *bias_r1, const float *bias_r2, int sink,
+                                         float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes, void *stream) {
+  return group_decode_impl(q, k, v, out, q_batch_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride, out_batch_stride, batch, heads,
+                           kv_heads, head_dim, cache_rows, pos_device, first, bias_r1, bias_r2, sink, nullptr, 0, scale, dtype, nsplit, scratch,
+                           scratch_bytes, stream);
+}
+
+extern "C" int eb_attention_group_decode_chunk(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+                                         long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                                         long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int ring_rows, int chunk,
+                                         const int32_t *pos_device, const int32_t *first, const float *sinks, float scale, int dtype,
+                                         int nsplit, void *scratch, size_t scratch_bytes, void *stream) {
+  EB_REQUIRE(chunk >= 0, "attention_group_decode: a chunk of %d positions", chunk);
+  return group_decode_impl(q, k, v, out, q_batch_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride, out_batch_stride, batch, heads,
+                           kv_heads, head_dim, ring_rows, pos_device, first, nullptr, nullptr, sinks ? 1 : 0, sinks, chunk, scale, dtype, nsplit, scratch,
+                           scratch_bytes, stream);
 }

@@ -67,5 +67,21 @@ __device__ __forceinline__ void load_warp_rows(uint32_t tile, const T *base, lon
   }
 }
 
+// The same for a ring of R rows: entry i of the tile is position rel0 + i of `count`, the first of them in
+// row r0 (count <= R, so a position wraps at most once).
+template <typename T, int D>
+__device__ __forceinline__ void load_warp_ring(uint32_t tile, const T *base, long long rs, int rel0, int count, int r0, int R, int warp, int lane) {
+  constexpr int kChunks = D / 8, kRowStep = 32 / kChunks, kIters = 16 / kRowStep;
+  const int c = lane % kChunks, rl = lane / kChunks;
+#pragma unroll
+  for (int k = 0; k < kIters; ++k) {
+    const int i = warp * 16 + rl + k * kRowStep, rel = rel0 + i;
+    const bool ok = rel < count;
+    int r = r0 + rel;
+    if (r >= R) r -= R;
+    cp_async16(tile + tile_off<D>(i, c), ok ? base + (long long)r * rs + c * 8 : base, ok);
+  }
+}
+
 }  // namespace
 }  // namespace eb

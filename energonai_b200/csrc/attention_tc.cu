@@ -29,7 +29,10 @@
 // work of the special-function unit), and may add one to the softmax denominator (a sink of score 0).
 //
 // A sliding window (row i sees only the `window` keys up to its own position) shortens the range of
-// key tiles a row tile walks and hides the leading keys of its first tiles; nothing else changes.
+// key tiles a row tile walks and hides the leading keys of its first tiles; nothing else changes.  Chunks
+// (a row sees only its own chunk of so many positions, counted from the sequence's first row behind the
+// padding) do the same with another lower bound, and a number per head may join the softmax as a
+// score without a value.
 //
 // Every mbarrier wait is bounded; a wait that runs out is recorded, the CTA's roles leave (each
 // decision made uniform over the warp first), copies in flight are given time to land, TMEM is
@@ -66,6 +69,9 @@ struct TcParams {
   const float *bias;                       // biased form: [H][bias_ld], r1 * log2(1 + r2 * distance)
   long long bias_ld;
   int sink;
+  const float *sinks;                      // plain form: per head, a score without a value (null: none)
+  int chunk;                               // > 0: row i sees only the keys of its chunk, counted from `first`
+  const int *first;                        // [B] padding rows in front of each sequence (they see themselves), or null
   int mask_vec;                            // mask rows start on 16-byte boundaries
   float scale_log2;                        // scale * log2(e)
   const void *mask;                        // additive [B][>= Sk] in T, or null
@@ -107,6 +113,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int qb = gridDim.x - 1 - blockIdx.x, h = blockIdx.y, hk = h / p.group, b = blockIdx.z;   // longest (latest, under the causal mask) blocks first
   const int q0 = qb * (kTiles * kRows), shift = p.Sk - p.Sq;
+  if (p.first) griddep_wait();
+  const int first = p.first ? p.first[b] : 0;
+  // first key that the row at position i sees
+  auto seen_from = [&](int i) {
+    if (p.window > 0) return i - p.window + 1;
+    const int f = min(first, max(i, 0));
+    return p.chunk > 0 && i > f ? f + (i - f) / p.chunk * p.chunk : f;
+  };
   // key tiles each row tile walks: all of them, or up to its last row's diagonal; none for a
   // row tile that lies wholly behind the end of the sequence
   // With a window a row tile starts at the first key its first row sees: tiles [ks[t], nt[t]) of
@@ -117,7 +131,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     const int qt0 = q0 + t * kRows;
     const int last_key = p.causal ? min(p.Sk - 1, qt0 + kRows - 1 + shift) : p.Sk - 1;
     nt[t] = (qt0 < p.Sq && last_key >= 0) ? last_key / kKeys + 1 : 0;
-    ks[t] = p.window > 0 ? max(0, qt0 + shift - p.window + 1) / kKeys : 0;
+    ks[t] = max(0, seen_from(qt0 + shift)) / kKeys;
     if (nt[t] > 0) jmin = min(jmin, ks[t]);
     nmax = max(nmax, nt[t]);
   }
@@ -243,9 +257,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     uint8_t *p_row = p_ptr + t * kPBytes + row * 128;
     const T *mrow = p.mask ? reinterpret_cast<const T *>(p.mask) + (long long)b * p.mask_bs : nullptr;
     const int vis_end = p.causal ? min(p.Sk, qi + shift + 1) : p.Sk;               // keys [0, vis_end) are visible to this row
-    const int vis_begin = p.window > 0 ? qi + shift - p.window + 1 : 0;            // ... from this key on
+    const int vis_begin = seen_from(qi + shift);                                   // ... from this key on
     // m_ref: the maximum the accumulated row and l_run are scaled by (a sink is a score of 0 seen already)
     float m_ref = BIAS && p.sink ? 0.f : -1e30f, l_run = BIAS && p.sink ? 1.f : 0.f;
+    if (!BIAS && p.sinks) {
+      m_ref = p.sinks[h] * kLog2eTc;
+      l_run = 1.f;
+    }
     // A bias that only lowers scores need not enter the maximum: any reference that is not below the
     // largest score will do as long as the probabilities keep their precision, which bf16 does over its
     // whole range.  fp16 does not, and a negative r1 raises scores: there the maximum includes it.
@@ -499,7 +517,7 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
                                        long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
                                        int heads, int q_len, int kv_len, int head_dim, int causal, int window, float scale,
                                        int dtype, void *stream, int kv_group = 1, const float *bias = nullptr, long long bias_ld = 0,
-                                       int sink = 0) {
+                                       int sink = 0, const float *sinks = nullptr, int chunk = 0, const int32_t *first = nullptr) {
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "attention_prefill: fp16 or bf16 only (dtype %d)", dtype);
   EB_REQUIRE(head_dim == 64 || head_dim == 128, "attention_prefill: head_dim %d not supported (64 or 128)", head_dim);
@@ -527,6 +545,7 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   p.mask_vec = mask && aligned16(mask) && mask_batch_stride % 8 == 0;
   p.o = out; p.o_bs = o_batch_stride; p.o_rs = o_row_stride;
   p.group = kv_group; p.bias = bias; p.bias_ld = bias_ld; p.sink = sink;
+  p.sinks = sinks; p.chunk = chunk; p.first = first;
 #define EB_TC(T, D) (bias ? launch_tc<T, D, true>(mq, mk, mv, p, st) : launch_tc<T, D, false>(mq, mk, mv, p, st))
   if (dtype == EB_F16) return head_dim == 64 ? EB_TC(__half, 64) : EB_TC(__half, 128);
   return head_dim == 64 ? EB_TC(__nv_bfloat16, 64) : EB_TC(__nv_bfloat16, 128);
@@ -574,4 +593,16 @@ extern "C" int eb_attention_prefill_biased_tc(const void *q, const void *k, cons
   return prefill_tc_impl(q, k, v, out, mask, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
                          o_batch_stride, o_row_stride, mask_batch_stride, batch, heads, q_len, kv_len, head_dim, 1, window, scale, dtype,
                          stream, kv_group, bias_table, bias_len, sink);
+}
+
+extern "C" int eb_attention_prefill_chunk_tc(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+                                       long long q_row_stride, long long k_batch_stride, long long k_row_stride,
+                                       long long v_batch_stride, long long v_row_stride, long long o_batch_stride,
+                                       long long o_row_stride, int batch, int heads, int kv_group, int len, int head_dim, int chunk,
+                                       const int32_t *first, const float *sinks, float scale, int dtype, void *stream) {
+  EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_prefill: %d heads do not share keys in groups of %d", heads, kv_group);
+  EB_REQUIRE(chunk >= 0, "attention_prefill: a chunk of %d positions", chunk);
+  return prefill_tc_impl(q, k, v, out, nullptr, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
+                         o_batch_stride, o_row_stride, 0, batch, heads, len, len, head_dim, 1, 0, scale, dtype, stream, kv_group, nullptr, 0, 0,
+                         sinks, chunk, first);
 }

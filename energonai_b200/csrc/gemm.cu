@@ -98,7 +98,7 @@ struct GemmParams {
   // one below the other; row tile i of A (128 rows) is multiplied by those of group tile_group[i].
   // Only the first *live_tiles row tiles are processed.  Both are read at run time.
   const int *tile_group, *live_tiles;
-  // gated (normal orientation): columns come in blocks of 8 gates and their 8 ups; C is [M, N/2]
+  // gated (EB_UNIT_CLAMPED or EB_UNIT_GEGLU): columns come in blocks of 8 gates and their 8 ups; C is [M, N/2]
   int gated;
   float gate_limit, gate_alpha;
   // the activation serves the output columns below act_cols (a multiple of 8); act_params: its two
@@ -659,8 +659,13 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
           if (n0 >= p.N) break;                              // warp-uniform (N is a multiple of 16)
           float v[16], y[8];
           tmem_ld16(t_base + c * 16, v);
+          if (p.gated == EB_UNIT_GEGLU) {
 #pragma unroll
-          for (int j = 0; j < 8; ++j) y[j] = gated_value(v[j], v[8 + j], p.gate_limit, p.gate_alpha);
+            for (int j = 0; j < 8; ++j) y[j] = gelu_tanh_value(v[j]) * v[8 + j];
+          } else {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) y[j] = gated_value(v[j], v[8 + j], p.gate_limit, p.gate_alpha);
+          }
           Vec16<T> o;
           o.pack(y);
           if (m < p.M) o.store(c_row_ptr + n0 / 2);
@@ -962,10 +967,15 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
         // a peer's lines never came: the whole warp leaves together (lanes without a column of
         // their own, beyond N, did not wait and must not be left behind at the next tile)
         if (p.comm.world >= 1 && __any_sync(0xffffffffu, lost)) { alive = false; continue; }
-        if (do_epilogue && n_ok && row_ok) {
+        // gated: the up of gate row n is row n + 8, eight lanes on (a block of 16 rows never straddles a warp)
+        if (p.gated && do_epilogue) {                   // (warp-uniform)
+#pragma unroll
+          for (int m = 0; m < BN; ++m) v[m] = unit_value(p.gated, v[m], __shfl_xor_sync(0xffffffffu, v[m], 8), p.gate_limit, p.gate_alpha);
+        }
+        if (do_epilogue && n_ok && row_ok && !(p.gated && (n & 8))) {
           // offset of row m of C, advanced row by row (a division per row by the run-time
           // rows-per-batch cost 0.1 us each: 2 us per tile)
-          long long row_off = c_extra + n;
+          long long row_off = c_extra + (p.gated ? (n >> 4) * 8 + (n & 7) : n);
           const int rpb = p.c_rows_per_batch;
           const long long batch_step = rpb > 0 ? p.c_batch_stride - (long long)(rpb - 1) * p.ldc : p.ldc;
           int row_in_batch = 0;
@@ -1390,7 +1400,8 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
                      size_t workspace_bytes, void *stream, const eb_comm *comm, const float *ln_colsum = nullptr,
                      const float *ln_bias = nullptr, double ln_eps = 0.0, bool reduce_scatter = false,
                      size_t rs_stage_offset = 0, int act_cols = 0x7fffffff, const float *act_params = nullptr,
-                     int tail_col = 0x7fffffff, float *tail = nullptr, long long ld_tail = 0) {
+                     int tail_col = 0x7fffffff, float *tail = nullptr, long long ld_tail = 0, int unit = EB_UNIT_NONE,
+                     float gate_limit = 0.f, float gate_alpha = 0.f) {
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "gemm: operands must be fp16 or bf16 (got dtype %d)", dtype);
   if (ln_colsum || ln_bias) {
     EB_REQUIRE(ln_colsum && ln_bias, "gemm_ln: ln_colsum and ln_bias go together");
@@ -1408,7 +1419,7 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
   // the generation orientation (M <= 128) writes C one element at a time: any N will do there
   EB_REQUIRE(K >= 8 && K % 8 == 0 && (N % 8 == 0 || M <= kLanes), "gemm: K, and N for M > 128, must be positive multiples of 8 (K=%d N=%d)", K, N);
   EB_REQUIRE(lda >= K && ldw >= K && lda % 8 == 0 && ldw % 8 == 0, "gemm: lda/ldw must be multiples of 8 and >= K");
-  EB_REQUIRE(ldc >= (N < tail_col ? N : tail_col) && (ldc % 8 == 0 || M <= kLanes) && (!residual || (ldr >= N && (ldr % 8 == 0 || M <= kLanes))),
+  EB_REQUIRE(ldc >= (unit != EB_UNIT_NONE ? N / 2 : N < tail_col ? N : tail_col) && (ldc % 8 == 0 || M <= kLanes) && (!residual || (ldr >= N && (ldr % 8 == 0 || M <= kLanes))),
              "gemm: ldc/ldr must be >= N (and multiples of 8 for M > 128)");
   EB_REQUIRE(c_rows_per_batch >= 0 && (c_rows_per_batch == 0 || c_batch_stride % 8 == 0 || M <= kLanes), "gemm: bad batch mapping of C");
   EB_REQUIRE(c_row_offset_limit >= 0, "gemm: negative row-offset limit");
@@ -1451,6 +1462,7 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
     p.comm = comm_dev(comm);
   }
   p.bias = bias; p.residual = residual; p.ldr = ldr; p.act = act; p.act_cols = act_cols; p.act_params = act_params;
+  p.gated = unit; p.gate_limit = gate_limit; p.gate_alpha = gate_alpha;
   p.tail_col = tail_col; p.tail = tail; p.ld_tail = ld_tail; p.out_f32 = out_dtype == EB_F32 && dtype != EB_F32;
 
   CUtensorMap tl, tc;
@@ -1524,8 +1536,10 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
 }
 
 extern "C" int eb_gemm_grouped(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, int M, int N, int K,
-                               int groups, const int32_t *tile_group, const int32_t *live_tiles, int gated, float limit, float alpha,
+                               int groups, const int32_t *tile_group, const int32_t *live_tiles, int unit, float limit, float alpha,
                                int dtype, void *stream) {
+  const int gated = unit == EB_UNIT_CLAMPED || unit == EB_UNIT_GEGLU ? unit : 0;
+  EB_REQUIRE(unit >= EB_UNIT_NONE && unit <= EB_UNIT_GELU, "gemm_grouped: unknown unit %d", unit);
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "gemm_grouped: operands must be fp16 or bf16 (got dtype %d)", dtype);
   EB_REQUIRE(M >= 0 && N > 0 && K > 0 && groups > 0, "gemm_grouped: bad size");
   if (M == 0) return EB_OK;
@@ -1543,7 +1557,7 @@ extern "C" int eb_gemm_grouped(const void *A, long long lda, const void *W, long
   p.C = C; p.ldc = ldc;
   p.lane_rows = M; p.col_rows = N;
   p.tile_group = tile_group; p.live_tiles = live_tiles;
-  p.gated = gated; p.gate_limit = limit; p.gate_alpha = alpha;
+  p.gated = gated; p.gate_limit = limit; p.gate_alpha = alpha; p.act = unit == EB_UNIT_GELU ? EB_ACT_GELU_ERF : EB_ACT_NONE;
   p.act_cols = p.tail_col = 0x7fffffff;
   p.kpb = 1;
   const long long lane_tiles = M / kLanes;
@@ -1582,6 +1596,15 @@ extern "C" int eb_gemm_parts(const void *A, long long lda, const void *W, long l
   return gemm_impl(A, lda, W, ldw, C, ldc, bias, nullptr, 0, M, N, K, dtype, dtype, act_params ? EB_ACT_XIELU : EB_ACT_NONE, 0, 0, nullptr, 0, flags,
                    workspace, workspace_bytes, stream, nullptr, nullptr, nullptr, 0.0, false, 0, act_params ? act_cols : 0x7fffffff, act_params,
                    tail ? tail_col : 0x7fffffff, tail, ld_tail);
+}
+
+extern "C" int eb_gemm_gated(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, int M, int N, int K, int unit,
+                             float limit, float alpha, int dtype, int flags, void *workspace, size_t workspace_bytes, void *stream) {
+  EB_REQUIRE(unit == EB_UNIT_CLAMPED || unit == EB_UNIT_GEGLU, "gemm_gated: unit %d has no gate", unit);
+  EB_REQUIRE(N % 16 == 0 && ldc % 8 == 0, "gemm_gated: N must be a multiple of 16 and ldc of 8 (N=%d)", N);
+  return gemm_impl(A, lda, W, ldw, C, ldc, nullptr, nullptr, 0, M, N, K, dtype, dtype, EB_ACT_NONE, 0, 0, nullptr, 0, flags, workspace,
+                   workspace_bytes, stream, nullptr, nullptr, nullptr, 0.0, false, 0, 0x7fffffff, nullptr, 0x7fffffff, nullptr, 0, unit, limit,
+                   alpha);
 }
 
 extern "C" int eb_gemm_ln(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc,

@@ -583,6 +583,8 @@ struct PlainParams {
   int group;                   // query heads per key / value head
   const float *r1, *r2;        // per head: r1 * ln(1 + r2 * distance) is taken off the score, or null
   int sink;                    // one is added to the softmax denominator
+  const float *sinks;          // per head: exp of it is (instead of one)
+  int chunk;                   // > 0: a position sees only its own chunk of so many, counted from first
 };
 
 template <typename T>
@@ -601,10 +603,11 @@ __global__ void attention_plain_kernel(const PlainParams p) {
   const int pos = (p.pos_dev ? *p.pos_dev : 0) + i;
   int lo = p.first ? p.first[b] : 0;
   if (p.window > 0) lo = max(lo, pos - p.window + 1);
+  if (p.chunk > 0 && pos > lo) lo += (pos - lo) / p.chunk * p.chunk;
   lo = max(lo, max(0, pos - p.ring_rows + 1));
   const T *K = reinterpret_cast<const T *>(p.k) + b * p.k_bs + h / p.group * p.k_hs, *V = reinterpret_cast<const T *>(p.v) + b * p.v_bs + h / p.group * p.v_hs;
   const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
-  float m = p.sink ? 0.f : -1e30f, l = p.sink ? 1.f : 0.f;      // the sink: a score of 0 without a value
+  float m = p.sinks ? p.sinks[h] * kLog2eLat : p.sink ? 0.f : -1e30f, l = p.sinks || p.sink ? 1.f : 0.f;      // the sink: a score without a value
   for (int j0 = lo; j0 <= pos; j0 += 32) {
     const int j = j0 + lane;
     float s = -INFINITY;
@@ -698,12 +701,12 @@ extern "C" int eb_latent_decode(const void *q, long long q_batch_stride, const v
   return dtype == EB_F16 ? launch_latent_r<__half>(map, p, batch, rank, st) : launch_latent_r<__nv_bfloat16>(map, p, batch, rank, st);
 }
 
-extern "C" int eb_attention_plain(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
+static int plain_impl(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
                                   long long q_head_stride, long long k_batch_stride, long long k_row_stride, long long k_head_stride,
                                   long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
                                   long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
                                   int v_dim, int window, int ring_rows, const int32_t *pos_device, const int32_t *first, const float *bias_r1,
-                                  const float *bias_r2, int sink, float scale, int dtype, void *stream) {
+                                  const float *bias_r2, int sink, const float *sinks, int chunk, float scale, int dtype, void *stream) {
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype_ok(dtype), "attention_plain: bad dtype %d", dtype);
   EB_REQUIRE(q && k && v && out, "attention_plain: null pointer");
@@ -712,7 +715,7 @@ extern "C" int eb_attention_plain(const void *q, const void *k, const void *v, v
   EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_plain: %d heads do not share keys in groups of %d", heads, kv_group);
   EB_REQUIRE((bias_r1 == nullptr) == (bias_r2 == nullptr), "attention_plain: the distance bias has two numbers per head");
   PlainParams p{};
-  p.group = kv_group; p.r1 = bias_r1; p.r2 = bias_r2; p.sink = sink;
+  p.group = kv_group; p.r1 = bias_r1; p.r2 = bias_r2; p.sink = sink; p.sinks = sinks; p.chunk = chunk;
   p.q = q; p.k = k; p.v = v; p.o = out;
   p.q_bs = q_batch_stride; p.q_rs = q_row_stride; p.q_hs = q_head_stride;
   p.k_bs = k_batch_stride; p.k_rs = k_row_stride; p.k_hs = k_head_stride;
@@ -724,4 +727,27 @@ extern "C" int eb_attention_plain(const void *q, const void *k, const void *v, v
   if (dtype == EB_F32) return launch_plain<float>(p, batch, st);
   if (dtype == EB_F16) return launch_plain<__half>(p, batch, st);
   return launch_plain<__nv_bfloat16>(p, batch, st);
+}
+
+extern "C" int eb_attention_plain(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
+                                  long long q_head_stride, long long k_batch_stride, long long k_row_stride, long long k_head_stride,
+                                  long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
+                                  long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
+                                  int v_dim, int window, int ring_rows, const int32_t *pos_device, const int32_t *first, const float *bias_r1,
+                                  const float *bias_r2, int sink, float scale, int dtype, void *stream) {
+  return plain_impl(q, k, v, out, q_batch_stride, q_row_stride, q_head_stride, k_batch_stride, k_row_stride, k_head_stride, v_batch_stride,
+                    v_row_stride, v_head_stride, o_batch_stride, o_row_stride, o_head_stride, batch, heads, kv_group, q_len, k_dim, v_dim, window,
+                    ring_rows, pos_device, first, bias_r1, bias_r2, sink, nullptr, 0, scale, dtype, stream);
+}
+
+extern "C" int eb_attention_plain_chunk(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
+                                  long long q_head_stride, long long k_batch_stride, long long k_row_stride, long long k_head_stride,
+                                  long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
+                                  long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
+                                  int v_dim, int chunk, int ring_rows, const int32_t *pos_device, const int32_t *first,
+                                  const float *sinks, float scale, int dtype, void *stream) {
+  EB_REQUIRE(chunk >= 0, "attention_plain: a chunk of %d positions", chunk);
+  return plain_impl(q, k, v, out, q_batch_stride, q_row_stride, q_head_stride, k_batch_stride, k_row_stride, k_head_stride, v_batch_stride,
+                    v_row_stride, v_head_stride, o_batch_stride, o_row_stride, o_head_stride, batch, heads, kv_group, q_len, k_dim, v_dim, 0,
+                    ring_rows, pos_device, first, nullptr, nullptr, 0, sinks, chunk, scale, dtype, stream);
 }

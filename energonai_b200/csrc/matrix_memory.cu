@@ -11,14 +11,13 @@
 //   head_norm_gate  that tail alone, for the rows of a prompt.
 #include "common.cuh"
 #include "memory_gates.cuh"
+#include "state_pass.cuh"
 
 namespace eb {
 namespace {
 
 template <typename T> __device__ __forceinline__ T store_cast(float v) { return from_f32<T>(v); }
 template <> __device__ __forceinline__ __half store_cast<__half>(float v) { return __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f)); }
-
-__device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
 // ---- prompt, token by token ------------------------------------------------------------------------
 constexpr int kScanCols = 32, kScanThreads = 256, kScanWarps = kScanThreads / 32;
@@ -113,8 +112,6 @@ template <typename T> int launch_scan(const ScanParams &p, int B, cudaStream_t s
 }
 
 // ---- one token per sequence ------------------------------------------------------------------------
-constexpr int kStepThreads = 256, kStepBatch = 8;
-
 struct StepParams {
   const void *q, *k, *v, *g;
   long long ldp;
@@ -130,27 +127,14 @@ struct StepParams {
   int heads, dk, dv, cols;     // cols: columns per CTA, a multiple of 4
 };
 
-__device__ __forceinline__ uint32_t smem_addr(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
 template <typename T>
 __global__ void __launch_bounds__(kStepThreads, 4) memory_step_kernel(const StepParams p) {
   extern __shared__ float sm[];
   float *qs = sm, *ks = qs + p.dk, *ns = ks + p.dk, *vs = ns + p.dk, *red = vs + p.cols;      // red: [row groups][cols]
-  // The CTAs of a head show each other their sums of squares: every one sends its own to all with an
-  // asynchronous store that completes on the receiver's mbarrier.  (A cluster barrier would do, but its
-  // release waits for the stores of the whole state.)
-  __shared__ float scratch[kStepThreads / 32], part_sq[8];
-  __shared__ __align__(8) uint64_t arrived;
+  __shared__ float scratch[kStepThreads / 32];
+  __shared__ __align__(8) ClusterSum head_sum;
   const int peers = gridDim.x;
-  if (peers > 1) {
-    if (threadIdx.x == 0) {
-      asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(smem_addr(&arrived)) : "memory");
-      asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-      asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_addr(&arrived)), "r"(peers * 4) : "memory");
-    }
-    __syncwarp();
-    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
-  }
+  cluster_sum_begin(head_sum, peers);
   griddep_wait();
   griddep_launch();
   const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x;
@@ -158,18 +142,8 @@ __global__ void __launch_bounds__(kStepThreads, 4) memory_step_kernel(const Step
   const long long bh = (long long)b * p.heads + h;
   const T *q = reinterpret_cast<const T *>(p.q) + b * p.ldp + h * p.dk, *k = reinterpret_cast<const T *>(p.k) + b * p.ldp + h * p.dk,
           *v = reinterpret_cast<const T *>(p.v) + b * p.ldp + h * p.dv + c0, *g = reinterpret_cast<const T *>(p.g) + b * p.ldp + h * p.dv + c0;
-  // thread = 4 columns of every R-th row; kStepBatch rows of the state in flight per thread, the first of
-  // them requested before anything else is worked out
-  const int groups = p.cols / 4, R = kStepThreads / groups, cg4 = tid % groups, rg = tid / groups;
-  const bool active = rg < R && cg4 * 4 < width;
-  float *S = p.S + bh * p.dk * p.dv + c0 + cg4 * 4;
-  float4 s[kStepBatch];
-  auto fetch = [&](int d0) {
-#pragma unroll
-    for (int i = 0; i < kStepBatch; ++i)
-      if (d0 + i * R < p.dk) s[i] = __ldcs(reinterpret_cast<const float4 *>(S + (long long)(d0 + i * R) * p.dv));
-  };
-  if (active) fetch(rg);
+  StatePass pass(p.S + bh * p.dk * p.dv + c0, p.dk, p.dv, p.cols, width);
+  pass.begin();
   const float m0 = p.m[bh];
   const float li = log_input_gate(p.gates[b * p.ldg + h], p.bias_i[h], p.cap), lf = log_forget_gate(p.gates[b * p.ldg + p.heads + h], p.bias_f[h], p.cap);
   const float m1 = fmaxf(lf + m0, li), a = expf(lf + m0 - m1), w = expf(li - m1);
@@ -185,54 +159,18 @@ __global__ void __launch_bounds__(kStepThreads, 4) memory_step_kernel(const Step
   nq = block_sum<kStepThreads>(nq, scratch);                                   // (also makes qs, ks, vs visible)
   const float den = fmaxf(fabsf(nq), expf(-m1)) + kMemoryDenomEps;
 
-  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (active) {
-    const float4 vv = *reinterpret_cast<const float4 *>(vs + cg4 * 4);
-    for (int d0 = rg; d0 < p.dk; d0 += R * kStepBatch) {
-      if (d0 != rg) fetch(d0);
-#pragma unroll
-      for (int i = 0; i < kStepBatch; ++i) {
-        const int d = d0 + i * R;
-        if (d < p.dk) {
-          const float kd = ks[d], qd = qs[d];
-          s[i].x = fmaf(a, s[i].x, kd * vv.x); s[i].y = fmaf(a, s[i].y, kd * vv.y);
-          s[i].z = fmaf(a, s[i].z, kd * vv.z); s[i].w = fmaf(a, s[i].w, kd * vv.w);
-          __stcs(reinterpret_cast<float4 *>(S + (long long)d * p.dv), s[i]);
-          acc.x = fmaf(s[i].x, qd, acc.x); acc.y = fmaf(s[i].y, qd, acc.y);
-          acc.z = fmaf(s[i].z, qd, acc.z); acc.w = fmaf(s[i].w, qd, acc.w);
-        }
-      }
-    }
-  }
-  if (rg < R) *reinterpret_cast<float4 *>(red + rg * p.cols + cg4 * 4) = acc;
+  pass.run([a](int) { return a; }, ks, qs, vs, red);
   __syncthreads();
   float sq = 0.f;
   for (int c = tid; c < width; c += kStepThreads) {
     float x = 0.f;
-    for (int r = 0; r < R; ++r) x += red[r * p.cols + c];
+    for (int r = 0; r < pass.R; ++r) x += red[r * p.cols + c];
     x /= den;
     red[c] = x;                                     // (row group 0: only this thread has read column c of it)
     sq = fmaf(x, x, sq);
   }
   sq = block_sum<kStepThreads>(sq, scratch);
-  if (peers > 1) {
-    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");         // every CTA's mbarrier is set up
-    if (tid < peers) {
-      uint32_t dst, bar;
-      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(dst) : "r"(smem_addr(&part_sq[blockIdx.x])), "r"(tid));
-      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(bar) : "r"(smem_addr(&arrived)), "r"(tid));
-      asm volatile("st.async.shared::cluster.mbarrier::complete_tx::bytes.b32 [%0], %1, [%2];" ::"r"(dst), "r"(__float_as_uint(sq)), "r"(bar) : "memory");
-    }
-    // (the sums of all CTAs arrive without further waits of theirs; the limit only keeps a defect from hanging)
-    for (int it = 0; it < (1 << 20); ++it) {
-      uint32_t ok;
-      asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], 0;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-                   : "=r"(ok) : "r"(smem_addr(&arrived)) : "memory");
-      if (ok) break;
-    }
-    sq = 0.f;
-    for (int r = 0; r < peers; ++r) sq += part_sq[r];
-  }
+  sq = cluster_sum(head_sum, peers, sq);
   const float rs = rsqrtf(sq * p.inv_count + p.eps);
   T *out = reinterpret_cast<T *>(p.out) + b * p.ldo + h * p.dv + c0;
   const T *norm = reinterpret_cast<const T *>(p.norm) + h * p.dv + c0;
@@ -245,31 +183,13 @@ __global__ void __launch_bounds__(kStepThreads, 4) memory_step_kernel(const Step
 }
 
 template <typename T> int launch_step(StepParams p, int B, cudaStream_t st) {
-  // columns of a head over as many CTAs as it takes to have two per SM, at least 32 columns each;
-  // more where a CTA would hold more than 1024
-  int split = 1;
-  while (split < 8 && ((long long)B * p.heads * split < 2 * sm_count() || p.dv > 1024 * split) && (p.dv + 2 * split - 1) / (2 * split) >= 32) split *= 2;
+  const int split = state_split((long long)B * p.heads, p.dv);
   p.cols = ((p.dv + split - 1) / split + 3) / 4 * 4;
   if (p.cols > 4 * kStepThreads) return fail(EB_EUNSUPPORTED, "memory_step: value head size %d is too large", p.dv);
   const int R = kStepThreads / (p.cols / 4);
   const size_t smem = (size_t)(3 * p.dk + p.cols + R * p.cols) * sizeof(float);
   if (smem > 48 * 1024) return fail(EB_EUNSUPPORTED, "memory_step: head sizes %d / %d are too large", p.dk, p.dv);
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(split, p.heads, B);
-  cfg.blockDim = dim3(kStepThreads);
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = st;
-  cudaLaunchAttribute attr[2];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = split;
-  attr[0].val.clusterDim.y = 1;
-  attr[0].val.clusterDim.z = 1;
-  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[1].val.programmaticStreamSerializationAllowed = pdl_enabled() ? 1 : 0;
-  cfg.attrs = attr;
-  cfg.numAttrs = 2;
-  cudaLaunchKernelEx(&cfg, memory_step_kernel<T>, p);
-  return check_launch("memory_step");
+  return launch_state_step("memory_step", memory_step_kernel<T>, p, dim3(split, p.heads, B), split, smem, st);
 }
 
 // ---- the tail of a prompt's rows ---------------------------------------------------------------------
@@ -278,7 +198,7 @@ struct HeadNormParams {
   long long ldo, ldg, ld_out;
   void *out;
   float inv_count, eps;
-  int rows, heads, dv;
+  int rows, heads, dv, silu;   // silu: the gate is g * sigmoid(g)
 };
 
 // A warp per (row, head), heads in packs of 8 elements.
@@ -326,7 +246,7 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const HeadNormParam
     wv.load(norm + c * N);
     wv.unpack(wf);
 #pragma unroll
-    for (int e = 0; e < N; ++e) f[e] = f[e] * rs * wf[e] * __fdividef(1.f, 1.f + __expf(-gf[e]));
+    for (int e = 0; e < N; ++e) f[e] = f[e] * rs * wf[e] * __fdividef(p.silu ? gf[e] : 1.f, 1.f + __expf(-gf[e]));
     y.pack(f);
     y.store(out + c * N);
   };
@@ -393,8 +313,8 @@ extern "C" int eb_memory_step(const void *q, const void *k, const void *v, const
   return launch_step<__nv_bfloat16>(p, batch, st);
 }
 
-extern "C" int eb_head_norm_gate(const void *o, long long ldo, const void *g, long long ldg, const void *norm, float eps, void *out,
-                                 long long ld_out, int rows, int heads, int dv, int dv_count, int dtype, void *stream) {
+extern "C" int eb_head_norm_gate_act(const void *o, long long ldo, const void *g, long long ldg, const void *norm, float eps, void *out,
+                                     long long ld_out, int rows, int heads, int dv, int dv_count, int silu, int dtype, void *stream) {
   if (rows == 0) return EB_OK;
   EB_REQUIRE(dtype_ok(dtype), "head_norm_gate: bad dtype %d", dtype);
   EB_REQUIRE(o && g && norm && out, "head_norm_gate: null pointer");
@@ -405,11 +325,16 @@ extern "C" int eb_head_norm_gate(const void *o, long long ldo, const void *g, lo
   EB_REQUIRE(((long long)rows * heads + 7) / 8 < (1ll << 31), "head_norm_gate: too many rows");
   HeadNormParams p{};
   p.o = o; p.g = g; p.norm = norm; p.ldo = ldo; p.ldg = ldg; p.ld_out = ld_out; p.out = out;
-  p.inv_count = 1.f / (float)dv_count; p.eps = eps; p.rows = rows; p.heads = heads; p.dv = dv;
+  p.inv_count = 1.f / (float)dv_count; p.eps = eps; p.rows = rows; p.heads = heads; p.dv = dv; p.silu = silu;
   const dim3 grid((unsigned)(((long long)rows * heads + 7) / 8)), block(256);
   cudaStream_t st = as_stream(stream);
   if (dtype == EB_F32) launch_pdl(head_norm_gate_kernel<float>, grid, block, 0, st, p);
   else if (dtype == EB_F16) launch_pdl(head_norm_gate_kernel<__half>, grid, block, 0, st, p);
   else launch_pdl(head_norm_gate_kernel<__nv_bfloat16>, grid, block, 0, st, p);
   return check_launch("head_norm_gate");
+}
+
+extern "C" int eb_head_norm_gate(const void *o, long long ldo, const void *g, long long ldg, const void *norm, float eps, void *out,
+                                 long long ld_out, int rows, int heads, int dv, int dv_count, int dtype, void *stream) {
+  return eb_head_norm_gate_act(o, ldo, g, ldg, norm, eps, out, ld_out, rows, heads, dv, dv_count, 0, dtype, stream);
 }

@@ -8,7 +8,7 @@
 //   grouped_skinny  one product per group (an expert, or a head of an absorbed attention
 //                 projection) for a handful of rows each: a pass over the weights of the groups
 //                 that have rows, each weight read once
-//   gated_act     the expert activation on its own (fp32 path)
+//   unit_act      the expert activation on its own (fp32 path)
 //
 // Gate and up projections are interleaved in blocks of 8 rows (8 gates, then their 8 ups), so
 // that an epilogue holds both halves of a pair in one thread.
@@ -22,9 +22,11 @@ namespace {
 // ---- routing of prompt-sized batches ------------------------------------------------------------
 constexpr int kRouteWarps = 4;
 
+// RULE: the choice follows `rule` (router.cuh); `experts` are the choices, those from `rule.real` on have no rows.
+template <bool RULE>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 moe_route_kernel(const float *logits, long long ld, int tokens, int experts, int top, const int *first, int rows_per_batch, int *idx,
-                 float *weights, int *counts, int *ranks) {
+                 float *weights, int *counts, int *ranks, const RouterRule rule, float *gate, int gate_col) {
   extern __shared__ float dyn[];
   griddep_wait();
   griddep_launch();
@@ -36,12 +38,15 @@ moe_route_kernel(const float *logits, long long ld, int tokens, int experts, int
       idx[(long long)t * top + k] = -1;
       weights[(long long)t * top + k] = 0.f;
     }
+    if (gate && lane == 0) gate[t] = 0.f;
     return;
   }
-  float *z = dyn + warp * experts;
+  float *z = dyn + warp * (RULE ? rule_floats(experts, rule) : experts);
   for (int e = lane; e < experts; e += 32) z[e] = logits[(long long)t * ld + e];
+  if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-logits[(long long)t * ld + gate_col]));
   __syncwarp();
-  route_warp(z, experts, top, idx + (long long)t * top, weights + (long long)t * top, counts, ranks ? ranks + (long long)t * top : nullptr);
+  if (RULE) route_warp_rule(z, experts, top, rule, idx + (long long)t * top, weights + (long long)t * top, counts, ranks ? ranks + (long long)t * top : nullptr);
+  else route_warp(z, experts, top, idx + (long long)t * top, weights + (long long)t * top, counts, ranks ? ranks + (long long)t * top : nullptr);
 }
 
 constexpr int kPlanThreads = 1024;
@@ -99,8 +104,9 @@ moe_permute_kernel(const uint4 *x, long long ldx16, int packs, int tokens, int t
     int dest = -1;                                 // lane k: destination of choice k0 + k
     if (k0 + lane < top) {
       const int e = idx[a0 + k0 + lane];
-      if (e >= 0) {
-        dest = offsets[e] + ranks[a0 + k0 + lane];
+      const int rank = e >= 0 ? ranks[a0 + k0 + lane] : -1;
+      if (rank >= 0) {                             // (a choice that stands for the input itself has no rank)
+        dest = offsets[e] + rank;
         if (dest >= max_rows) dest = -1;
       }
       rows[a0 + k0 + lane] = dest;
@@ -117,15 +123,17 @@ moe_permute_kernel(const uint4 *x, long long ldx16, int packs, int tokens, int t
   }
 }
 
+// n2: columns of y (a gated unit reads twice as many, in the 8 + 8 order)
 template <typename T>
-__global__ void gated_act_kernel(const T *x, long long ldx, T *y, long long ldy, int n1, int half, float limit, float alpha) {
+__global__ void unit_act_kernel(const T *x, long long ldx, T *y, long long ldy, int n1, int n2, int unit, float limit, float alpha) {
   griddep_wait();
   griddep_launch();
   const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= (long long)n1 * half) return;
-  const long long m = i / half;
-  const int c = (int)(i - m * half), col = (c >> 3) * 16 + (c & 7);
-  y[m * ldy + c] = from_f32<T>(gated_value(to_f32<T>(x[m * ldx + col]), to_f32<T>(x[m * ldx + col + 8]), limit, alpha));
+  if (i >= (long long)n1 * n2) return;
+  const long long m = i / n2;
+  const int c = (int)(i - m * n2), col = (c >> 3) * 16 + (c & 7);
+  if (unit == EB_UNIT_GELU) y[m * ldy + c] = from_f32<T>(gelu_erf_value(to_f32<T>(x[m * ldx + c])));
+  else y[m * ldy + c] = from_f32<T>(unit_value(unit, to_f32<T>(x[m * ldx + col]), to_f32<T>(x[m * ldx + col + 8]), limit, alpha));
 }
 
 // ---- the weight-streaming grouped product ---------------------------------------------------------
@@ -140,7 +148,7 @@ struct SkinnyParams {
   const int *idx;              // group of list entry i, or null: every group has all rows
   int rows;                    // list entries
   int N, K;
-  int gated;
+  int unit;
   float limit, alpha;
   int ksplit;                  // the warps of a CTA share 16 weight rows and take this many columns each (0: own rows, all columns)
 };
@@ -231,8 +239,11 @@ __device__ __forceinline__ void skinny_tile(const SkinnyParams &p, int group, in
       if (r >= n) continue;
       const int i = list ? list[base + r] : base + r;
       T *c = C + (long long)i * p.ldc;
-      if (p.gated) {
-        if (row0 + g + 8 < p.N) c[row0 / 2 + g] = from_f32<T>(gated_value(acc[j][e], acc[j][2 + e], p.limit, p.alpha));
+      if (p.unit == EB_UNIT_CLAMPED || p.unit == EB_UNIT_GEGLU) {
+        if (row0 + g + 8 < p.N) c[row0 / 2 + g] = from_f32<T>(unit_value(p.unit, acc[j][e], acc[j][2 + e], p.limit, p.alpha));
+      } else if (p.unit == EB_UNIT_GELU) {
+        if (row0 + g < p.N) c[row0 + g] = from_f32<T>(gelu_erf_value(acc[j][e]));
+        if (row0 + g + 8 < p.N) c[row0 + g + 8] = from_f32<T>(gelu_erf_value(acc[j][2 + e]));
       } else {
         if (row0 + g < p.N) c[row0 + g] = from_f32<T>(acc[j][e]);
         if (row0 + g + 8 < p.N) c[row0 + g + 8] = from_f32<T>(acc[j][2 + e]);
@@ -273,22 +284,37 @@ __global__ void __launch_bounds__(128) grouped_skinny_kernel(const SkinnyParams 
 
 using namespace eb;
 
-extern "C" int eb_moe_route(const float *logits, long long ld, int tokens, int experts, int top, const int32_t *first, int rows_per_batch,
-                            int32_t *idx, float *weights, int32_t *counts, int32_t *ranks, void *stream) {
+template <bool RULE>
+static int route_impl(const float *logits, long long ld, int tokens, int experts, int top, const int32_t *first, int rows_per_batch,
+                      int32_t *idx, float *weights, int32_t *counts, int32_t *ranks, const RouterRule &rule, float *gate, int gate_col, void *stream) {
   if (tokens == 0) return EB_OK;
   EB_REQUIRE(logits && idx && weights, "moe_route: null pointer");
   EB_REQUIRE(tokens > 0 && experts > 0 && experts <= kMaxExperts && top > 0 && top <= experts && ld >= experts,
              "moe_route: bad sizes (%d tokens, %d experts, top %d)", tokens, experts, top);
   EB_REQUIRE((counts == nullptr) == (ranks == nullptr), "moe_route: counts and ranks go together");
   EB_REQUIRE(!first || rows_per_batch > 0, "moe_route: first needs rows_per_batch");
-  const size_t smem = (size_t)kRouteWarps * experts * sizeof(float);
-  if (smem > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+  const size_t smem = (size_t)kRouteWarps * (RULE ? rule_floats(experts, rule) : experts) * sizeof(float);
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(moe_route_kernel<RULE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
     cudaGetLastError();
     return fail(EB_ECUDA, "moe_route: cannot reserve %zu bytes of shared memory", smem);
   }
-  launch_pdl(moe_route_kernel, dim3((tokens + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), smem, as_stream(stream), logits, ld,
-             tokens, experts, top, first, rows_per_batch, idx, weights, counts, ranks);
+  launch_pdl(moe_route_kernel<RULE>, dim3((tokens + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32), smem, as_stream(stream), logits, ld,
+             tokens, experts, top, first, rows_per_batch, idx, weights, counts, ranks, rule, gate, gate_col);
   return check_launch("moe_route");
+}
+
+extern "C" int eb_moe_route(const float *logits, long long ld, int tokens, int experts, int top, const int32_t *first, int rows_per_batch,
+                            int32_t *idx, float *weights, int32_t *counts, int32_t *ranks, void *stream) {
+  return route_impl<false>(logits, ld, tokens, experts, top, first, rows_per_batch, idx, weights, counts, ranks, RouterRule{}, nullptr, 0, stream);
+}
+
+extern "C" int eb_moe_route_rule(const float *logits, long long ld, int tokens, int choices, int experts, int top, const float *correction,
+                                 int groups, int keep, const int32_t *first, int rows_per_batch, int32_t *idx, float *weights, int32_t *counts,
+                                 int32_t *ranks, float *shared_gate, void *stream) {
+  RouterRule rule;
+  if (int rc = make_rule("moe_route", choices, experts, top, correction, groups, keep, &rule)) return rc;
+  EB_REQUIRE(!shared_gate || ld > choices, "moe_route: the shared expert's gate is the logit behind the choices");
+  return route_impl<true>(logits, ld, tokens, choices, top, first, rows_per_batch, idx, weights, counts, ranks, rule, shared_gate, choices, stream);
 }
 
 extern "C" int eb_moe_plan(int32_t *counts, int experts, int32_t *offsets, int32_t *tile_group, int max_tiles, int32_t *live_tiles,
@@ -314,25 +340,33 @@ extern "C" int eb_moe_permute(const void *x, long long ldx, int n2, int dtype, i
   return check_launch("moe_permute");
 }
 
-extern "C" int eb_gated_act(const void *x, long long ldx, void *y, long long ldy, int n1, int half, float limit, float alpha, int dtype,
-                            void *stream) {
+extern "C" int eb_unit_act(const void *x, long long ldx, void *y, long long ldy, int n1, int n2, int unit, float limit, float alpha, int dtype,
+                           void *stream) {
   if (n1 == 0) return EB_OK;
-  EB_REQUIRE(dtype_ok(dtype) && x && y, "gated_act: bad dtype or null pointer");
-  EB_REQUIRE(n1 > 0 && half > 0 && half % 8 == 0 && ldx >= 2 * half && ldy >= half, "gated_act: bad sizes");
-  const long long total = (long long)n1 * half;
-  EB_REQUIRE((total + 255) / 256 < (1ll << 31), "gated_act: too many elements");
+  EB_REQUIRE(dtype_ok(dtype) && x && y, "unit_act: bad dtype or null pointer");
+  EB_REQUIRE(unit >= EB_UNIT_CLAMPED && unit <= EB_UNIT_GELU, "unit_act: unknown unit %d", unit);
+  EB_REQUIRE(n1 > 0 && n2 > 0 && n2 % 8 == 0 && ldx >= (unit == EB_UNIT_GELU ? n2 : 2 * n2) && ldy >= n2, "unit_act: bad sizes");
+  const long long total = (long long)n1 * n2;
+  EB_REQUIRE((total + 255) / 256 < (1ll << 31), "unit_act: too many elements");
   const dim3 g((unsigned)((total + 255) / 256)), b(256);
   cudaStream_t st = as_stream(stream);
-  if (dtype == EB_F32) launch_pdl(gated_act_kernel<float>, g, b, 0, st, (const float *)x, ldx, (float *)y, ldy, n1, half, limit, alpha);
-  else if (dtype == EB_F16) launch_pdl(gated_act_kernel<__half>, g, b, 0, st, (const __half *)x, ldx, (__half *)y, ldy, n1, half, limit, alpha);
-  else launch_pdl(gated_act_kernel<__nv_bfloat16>, g, b, 0, st, (const __nv_bfloat16 *)x, ldx, (__nv_bfloat16 *)y, ldy, n1, half, limit, alpha);
-  return check_launch("gated_act");
+  if (dtype == EB_F32) launch_pdl(unit_act_kernel<float>, g, b, 0, st, (const float *)x, ldx, (float *)y, ldy, n1, n2, unit, limit, alpha);
+  else if (dtype == EB_F16) launch_pdl(unit_act_kernel<__half>, g, b, 0, st, (const __half *)x, ldx, (__half *)y, ldy, n1, n2, unit, limit, alpha);
+  else launch_pdl(unit_act_kernel<__nv_bfloat16>, g, b, 0, st, (const __nv_bfloat16 *)x, ldx, (__nv_bfloat16 *)y, ldy, n1, n2, unit, limit, alpha);
+  return check_launch("unit_act");
+}
+
+extern "C" int eb_gated_act(const void *x, long long ldx, void *y, long long ldy, int n1, int half, float limit, float alpha, int dtype,
+                            void *stream) {
+  return eb_unit_act(x, ldx, y, ldy, n1, half, EB_UNIT_CLAMPED, limit, alpha, dtype, stream);
 }
 
 extern "C" int eb_grouped_skinny(const void *A, long long lda, long long a_group_stride, int a_div, const void *W, long long w_group_stride,
                                  long long ldw, void *C, long long ldc, long long c_group_stride, const int32_t *idx, int rows, int groups,
-                                 int N, int K, int gated, float limit, float alpha, int dtype, void *stream) {
+                                 int N, int K, int unit, float limit, float alpha, int dtype, void *stream) {
   if (rows == 0 || groups == 0) return EB_OK;
+  const bool gated = unit == EB_UNIT_CLAMPED || unit == EB_UNIT_GEGLU;
+  EB_REQUIRE(unit >= EB_UNIT_NONE && unit <= EB_UNIT_GELU, "grouped_skinny: unknown unit %d", unit);
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "grouped_skinny: fp16 or bf16 only (dtype %d)", dtype);
   EB_REQUIRE(A && W && C, "grouped_skinny: null pointer");
   EB_REQUIRE(rows > 0 && groups > 0 && groups <= 65535 && N > 0 && K > 0 && a_div > 0, "grouped_skinny: bad sizes");
@@ -344,7 +378,7 @@ extern "C" int eb_grouped_skinny(const void *A, long long lda, long long a_group
   SkinnyParams p{};
   p.A = A; p.lda = lda; p.a_gs = a_group_stride; p.a_div = a_div; p.W = W; p.w_gs = w_group_stride; p.ldw = ldw;
   p.C = C; p.ldc = ldc; p.c_gs = c_group_stride; p.idx = idx; p.rows = rows; p.N = N; p.K = K;
-  p.gated = gated; p.limit = limit; p.alpha = alpha;
+  p.unit = unit; p.limit = limit; p.alpha = alpha;
   // Too few strips to give every SM a CTA of four: with many columns the four warps share a strip
   // and split its columns, with few the CTAs get fewer warps.  (The choice depends on the weights'
   // shape alone, so a row's result does not change with the batch.)

@@ -11,6 +11,11 @@
 //   stream_update     the residual step of blocks that normalise in front of AND behind a
 //                     sublayer: x += norm(y * sigmoid(gate)) * w_out, then h = norm(x) * w_next for
 //                     the sublayer that follows.  With `src` it starts the stream: x = scale * src.
+//   stream_add        the residual step of blocks that normalise in front of a sublayer only:
+//                     x += scale * Y, then h = norm(x) * w_next.  Y is a row, the sum of two rows
+//                     normalised each by itself (mixers side by side), or what a mixture of experts
+//                     with identity experts and a gated shared expert produced for the token.
+//                     Optionally the router of the mixture that follows is evaluated on h.
 //
 // One CTA per row, the row register-resident in packs of 8; statistics, weights and the residual
 // are fp32 throughout.
@@ -225,6 +230,199 @@ struct StreamParams {
   int n2;
 };
 
+struct AddParams {
+  const void *src, *src2;      // T rows: x = src + src2 instead of x as it is (null: x as it is; src2 may be null)
+  long long lds, lds2;
+  const void *y, *y2;          // T rows (y: expert rows with a mixture)
+  long long ldy, ldy2;
+  const float *w, *w2;         // [n2]: y and y2 are normalised and multiplied by these
+  // mixture: sum_k weights[t*top+k] * (idx < experts ? y[rows ? rows[...] : t*top+k] : ident[t]) + gate[t] * shared[t]
+  const int *idx, *rows;
+  const float *weights, *gate;
+  int top, experts;
+  const void *ident, *shared;
+  long long ldi, ldsh;
+  float scale;
+  float *x;
+  long long ldx;
+  const void *w_next;
+  float next_scale;
+  void *h;
+  long long ldh;
+  float eps, inv_count;
+  int n2;
+  // router on h (null: none): [choices (+ 1 with r_gate)][n2] T
+  const void *router;
+  int choices, r_top;
+  RouterRule rule;
+  int *r_idx;
+  float *r_weights, *r_gate;
+};
+
+enum { kAddRow = 0, kAddTwo = 1, kAddMix = 2 };
+
+template <typename T, int PACKS, int FORM, int THREADS>
+__global__ void __launch_bounds__(THREADS) stream_add_kernel(const AddParams p) {
+  __shared__ float2 scratch[THREADS / 32];
+  extern __shared__ float dyn[];                   // router: [n2] row, [choices + 1] logits, the rule's own
+  const long long row = blockIdx.x;
+  const int packs = p.n2 / 8;
+  griddep_wait();
+  griddep_launch();
+  auto sum2 = [&](float2 s) {
+    s.x = warp_sum(s.x);
+    s.y = warp_sum(s.y);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = s;
+    __syncthreads();
+    s = (threadIdx.x & 31) < THREADS / 32 ? scratch[threadIdx.x & 31] : make_float2(0.f, 0.f);
+    return make_float2(warp_sum(s.x), warp_sum(s.y));
+  };
+  float xv[PACKS][8], v[PACKS][8], v2[FORM == kAddTwo ? PACKS : 1][8];
+  float2 sq = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= packs) break;
+    if (p.src) {
+      load8<T>(reinterpret_cast<const T *>(p.src) + row * p.lds + c * 8, xv[i]);
+      if (p.src2) {
+        float f[8];
+        load8<T>(reinterpret_cast<const T *>(p.src2) + row * p.lds2 + c * 8, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) xv[i][e] += f[e];
+      }
+    } else {
+      load8<float>(p.x + row * p.ldx + c * 8, xv[i]);
+    }
+    if (FORM == kAddMix) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] = 0.f;
+      float self = 0.f;
+      for (int k = 0; k < p.top; ++k) {
+        const long long a = row * p.top + k;
+        const int ex = p.idx[a];
+        const float s = p.weights[a];
+        if (ex < 0) continue;
+        if (ex >= p.experts) { self += s; continue; }
+        const long long src = p.rows ? p.rows[a] : a;
+        float f[8];
+        load8<T>(reinterpret_cast<const T *>(p.y) + src * p.ldy + c * 8, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = fmaf(s, f[e], v[i][e]);
+      }
+      if (self != 0.f) {
+        float f[8];
+        load8<T>(reinterpret_cast<const T *>(p.ident) + row * p.ldi + c * 8, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = fmaf(self, f[e], v[i][e]);
+      }
+      if (p.shared) {
+        const float s = p.gate[row];
+        float f[8];
+        load8<T>(reinterpret_cast<const T *>(p.shared) + row * p.ldsh + c * 8, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] = fmaf(s, f[e], v[i][e]);
+      }
+    } else if (p.y) {
+      load8<T>(reinterpret_cast<const T *>(p.y) + row * p.ldy + c * 8, v[i]);
+    }
+    if (FORM == kAddTwo) {
+      load8<T>(reinterpret_cast<const T *>(p.y2) + row * p.ldy2 + c * 8, v2[i]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        sq.x = fmaf(v[i][e], v[i][e], sq.x);
+        sq.y = fmaf(v2[i][e], v2[i][e], sq.y);
+      }
+    }
+  }
+  if (FORM == kAddTwo) {
+    sq = sum2(sq);
+    const float r1 = rsqrtf(sq.x * p.inv_count + p.eps), r2 = rsqrtf(sq.y * p.inv_count + p.eps);
+#pragma unroll
+    for (int i = 0; i < PACKS; ++i) {
+      const int c = threadIdx.x + i * THREADS;
+      if (c >= packs) break;
+      float a[8], b[8];
+      load8<float>(p.w + c * 8, a);
+      load8<float>(p.w2 + c * 8, b);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] = v[i][e] * r1 * a[e] + v2[i][e] * r2 * b[e];
+    }
+  }
+  float sx = 0.f;
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= packs) break;
+    if (FORM != kAddRow || p.y) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) xv[i][e] = fmaf(p.scale, v[i][e], xv[i][e]);
+    }
+    if (p.src || p.y) store8<float>(p.x + row * p.ldx + c * 8, xv[i]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sx = fmaf(xv[i][e], xv[i][e], sx);
+  }
+  if (!p.w_next) return;
+  const float r = rsqrtf(sum2(make_float2(sx, 0.f)).x * p.inv_count + p.eps) * p.next_scale;
+#pragma unroll
+  for (int i = 0; i < PACKS; ++i) {
+    const int c = threadIdx.x + i * THREADS;
+    if (c >= packs) break;
+    float wv[8];
+    load8<T>(reinterpret_cast<const T *>(p.w_next) + c * 8, wv);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) wv[e] *= xv[i][e] * r;
+    store8<T>(reinterpret_cast<T *>(p.h) + row * p.ldh + c * 8, wv);
+    if (p.router) {
+      // the router reads the row as the products do: rounded to the operand type
+#pragma unroll
+      for (int e = 0; e < 8; ++e) dyn[c * 8 + e] = to_f32<T>(from_f32<T>(wv[e]));
+    }
+  }
+  if (!p.router) return;
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float *z = dyn + p.n2;                           // the rule's numbers lie behind the choices' logits; the gate's is not among them
+  for (int e = warp; e < p.choices + (p.r_gate ? 1 : 0); e += THREADS / 32) {
+    const T *wr = reinterpret_cast<const T *>(p.router) + (long long)e * p.n2;
+    float acc = 0.f;
+#pragma unroll 4
+    for (int c = lane; c < packs; c += 32) {
+      float f[8];
+      load8<T>(wr + c * 8, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc = fmaf(f[j], dyn[c * 8 + j], acc);
+    }
+    acc = warp_sum(acc);
+    if (lane == 0) {
+      if (e < p.choices) z[e] = acc;
+      else p.r_gate[row] = 1.f / (1.f + expf(-acc));
+    }
+  }
+  __syncthreads();
+  if (warp == 0) route_warp_rule(z, p.choices, p.r_top, p.rule, p.r_idx + row * p.r_top, p.r_weights + row * p.r_top, nullptr, nullptr);
+}
+
+template <typename T, int FORM> int launch_add(const AddParams &p, int n1, cudaStream_t st) {
+  const int packs = p.n2 / 8, threads = p.router ? 1024 : kNormThreads, per = (packs + threads - 1) / threads;
+  const size_t smem = p.router ? (size_t)(p.n2 + rule_floats(p.choices, p.rule)) * sizeof(float) : 0;
+  const dim3 g(n1), b(threads);
+  auto go = [&](auto kern) -> int {
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+      cudaGetLastError();
+      return fail(EB_ECUDA, "stream_add: cannot reserve %zu bytes of shared memory", smem);
+    }
+    launch_pdl(kern, g, b, smem, st, p);
+    return check_launch("stream_add");
+  };
+  if (p.router) return per <= 1 ? go(stream_add_kernel<T, 1, FORM, 1024>) : go(stream_add_kernel<T, 2, FORM, 1024>);
+  if (per <= 1) return go(stream_add_kernel<T, 1, FORM, kNormThreads>);
+  if (per <= 2) return go(stream_add_kernel<T, 2, FORM, kNormThreads>);
+  if (per <= 4) return go(stream_add_kernel<T, 4, FORM, kNormThreads>);
+  return go(stream_add_kernel<T, 8, FORM, kNormThreads>);
+}
+
 template <typename T, int PACKS>
 __global__ void __launch_bounds__(kNormThreads) stream_update_kernel(const StreamParams p) {
   constexpr int THREADS = kNormThreads;
@@ -429,4 +627,45 @@ extern "C" int eb_stream_update(const void *src, long long lds, float src_scale,
   if (dtype == EB_F32) return launch_stream<float>(p, n1, st);
   if (dtype == EB_F16) return launch_stream<__half>(p, n1, st);
   return launch_stream<__nv_bfloat16>(p, n1, st);
+}
+
+extern "C" int eb_stream_add(const void *src, long long lds, const void *src2, long long lds2, const void *y, long long ldy, const float *w,
+                             const void *y2, long long ldy2, const float *w2, const int32_t *idx, const int32_t *rows, const float *weights, int top,
+                             int experts, const void *ident, long long ldi, const void *shared, long long ldsh, const float *gate, float scale,
+                             float *x, long long ldx, const void *w_next, float next_scale, void *h, long long ldh, float eps, int n1, int n2,
+                             int count, const void *router, int choices, int r_experts, int r_top, const float *r_correction, int r_groups,
+                             int r_keep, int32_t *r_idx, float *r_weights, float *r_gate, int dtype, void *stream) {
+  if (n1 == 0) return EB_OK;
+  EB_REQUIRE(dtype_ok(dtype), "stream_add: bad dtype %d", dtype);
+  EB_REQUIRE(x && (src || y || w_next), "stream_add: null pointer");
+  EB_REQUIRE(n1 > 0 && n2 > 0 && n2 % 8 == 0 && n2 <= kMaxNormWidth, "stream_add: width %d must be a multiple of 8, at most %d", n2, kMaxNormWidth);
+  EB_REQUIRE(count > 0 && count <= n2, "stream_add: the mean is over 1..n2 elements");
+  const void *rows_p[] = {src, src2, y, y2, ident, shared, h};
+  const long long rows_ld[] = {lds, lds2, ldy, ldy2, ldi, ldsh, ldh};
+  for (int i = 0; i < 7; ++i)
+    EB_REQUIRE(!rows_p[i] || (rows_ld[i] >= n2 && rows_ld[i] % 8 == 0 && aligned16(rows_p[i])), "stream_add: row strides must be multiples of 8 and >= n2, rows 16-byte aligned");
+  EB_REQUIRE(ldx >= n2 && ldx % 8 == 0 && aligned16(x) && aligned16(w) && aligned16(w2) && aligned16(w_next) && aligned16(router),
+             "stream_add: row strides must be multiples of 8 and >= n2, pointers 16-byte aligned");
+  EB_REQUIRE(!src2 || src, "stream_add: a second start row without a first");
+  EB_REQUIRE(!y2 || (y && w && w2 && !idx), "stream_add: two rows need their weights");
+  EB_REQUIRE(y2 || !w, "stream_add: a weight without a second row");
+  EB_REQUIRE(!idx || (y && weights && ident && top > 0 && experts >= 0), "stream_add: a mixture needs expert rows, weights, top and the input rows");
+  EB_REQUIRE(!shared || (idx && gate), "stream_add: a shared expert goes with a mixture and its gate");
+  EB_REQUIRE(!w_next || h, "stream_add: no place for the normalised row");
+  AddParams p{};
+  if (router) {
+    EB_REQUIRE(w_next && r_idx && r_weights, "stream_add: the router reads h and needs its outputs");
+    if (int rc = make_rule("stream_add", choices, r_experts, r_top, r_correction, r_groups, r_keep, &p.rule)) return rc;
+  }
+  p.src = src; p.lds = lds; p.src2 = src2; p.lds2 = lds2; p.y = y; p.ldy = ldy; p.y2 = y2; p.ldy2 = ldy2; p.w = w; p.w2 = w2;
+  p.idx = idx; p.rows = rows; p.weights = weights; p.gate = gate; p.top = top; p.experts = experts; p.ident = ident; p.ldi = ldi;
+  p.shared = shared; p.ldsh = ldsh; p.scale = scale; p.x = x; p.ldx = ldx; p.w_next = w_next; p.next_scale = next_scale; p.h = h; p.ldh = ldh;
+  p.eps = eps; p.inv_count = 1.f / (float)count; p.n2 = n2;
+  p.router = router; p.choices = choices; p.r_top = r_top; p.r_idx = r_idx; p.r_weights = r_weights; p.r_gate = r_gate;
+  cudaStream_t st = as_stream(stream);
+#define EB_ADD(T) (idx ? launch_add<T, kAddMix>(p, n1, st) : y2 ? launch_add<T, kAddTwo>(p, n1, st) : launch_add<T, kAddRow>(p, n1, st))
+  if (dtype == EB_F32) return EB_ADD(float);
+  if (dtype == EB_F16) return EB_ADD(__half);
+  return EB_ADD(__nv_bfloat16);
+#undef EB_ADD
 }

@@ -52,4 +52,103 @@ __device__ __forceinline__ void route_warp(float *z, int experts, int top, int *
   }
 }
 
+// How a router chooses beyond the plain softmax scores.
+struct RouterRule {
+  const float *correction = nullptr;   // [choices] added to the scores for the choice alone, or null
+  int groups = 1, keep = 1;            // equal groups of neighbours; only the best `keep` (by their largest choice score) are open
+  int real = 0;                        // choices below this are experts with rows, the others stand for the input itself
+};
+
+__host__ __device__ inline int rule_floats(int choices, const RouterRule &r) { return 2 * choices + 2 * r.groups; }
+
+inline int make_rule(const char *name, int choices, int experts, int top, const float *correction, int groups, int keep, RouterRule *r) {
+  if (choices <= 0 || choices > kMaxExperts || experts < 0 || experts > choices) return fail(EB_EINVAL, "%s: bad router (%d choices, %d experts)", name, choices, experts);
+  if (groups <= 0 || keep <= 0 || keep > groups || choices % groups != 0) return fail(EB_EINVAL, "%s: %d choices in %d groups of which %d are kept", name, choices, groups, keep);
+  if (top <= 0 || top > choices / groups * keep) return fail(EB_EINVAL, "%s: top %d of %d open choices", name, top, choices / groups * keep);
+  r->correction = correction;
+  r->groups = groups;
+  r->keep = keep;
+  r->real = experts;
+  return EB_OK;
+}
+
+// The largest of v[0..n) that is above -inf, and its index (the lowest among equals; n or more if there is none).
+__device__ __forceinline__ void warp_argmax(const float *v, int n, float &best, int &bi) {
+  best = -INFINITY;
+  bi = 0x7fffffff;
+  for (int e = threadIdx.x & 31; e < n; e += 32) {
+    const float x = v[e];
+    if (x > best) { best = x; bi = e; }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
+  }
+}
+
+// route_warp with a rule; z has room for rule_floats() numbers.  The `top` choices with the largest
+// score + correction among the open groups are taken; their weights are their scores, divided by
+// their sum (+ 1e-20).
+__device__ __forceinline__ void route_warp_rule(float *z, int choices, int top, const RouterRule &rule, int *idx, float *weights, int *counts, int *ranks) {
+  const int lane = threadIdx.x & 31;
+  float *c = z + choices, *gs = c + choices, *open = gs + rule.groups;
+  float m = -FLT_MAX;
+  for (int e = lane; e < choices; e += 32) m = fmaxf(m, z[e]);
+  m = warp_max(m);
+  float s = 0.f;
+  for (int e = lane; e < choices; e += 32) s += expf(z[e] - m);
+  const float inv = 1.f / warp_sum(s);
+  for (int e = lane; e < choices; e += 32) {
+    const float sc = expf(z[e] - m) * inv;
+    z[e] = sc;
+    c[e] = sc + (rule.correction ? rule.correction[e] : 0.f);
+  }
+  __syncwarp();
+  if (rule.keep < rule.groups) {
+    const int per = choices / rule.groups;
+    for (int g = 0; g < rule.groups; ++g) {
+      float b = -INFINITY;
+      for (int e = lane; e < per; e += 32) b = fmaxf(b, c[g * per + e]);
+      b = warp_max(b);
+      if (lane == 0) { gs[g] = b; open[g] = 0.f; }
+    }
+    __syncwarp();
+    for (int k = 0; k < rule.keep; ++k) {
+      float best;
+      int bi;
+      warp_argmax(gs, rule.groups, best, bi);
+      if (lane == 0 && bi < rule.groups) { gs[bi] = -INFINITY; open[bi] = 1.f; }
+      __syncwarp();
+    }
+    for (int e = lane; e < choices; e += 32)
+      if (open[e / per] == 0.f) c[e] = -INFINITY;
+    __syncwarp();
+  }
+  float total = 0.f;
+  for (int k0 = 0; k0 < top; k0 += 32) {
+    int mine = 0;                                    // lane k: choice k0 + k
+    float score = 0.f;
+    const int n = min(32, top - k0);
+    for (int k = 0; k < n; ++k) {
+      float best;
+      int bi;
+      warp_argmax(c, choices, best, bi);
+      if (bi >= choices) bi = 0;                     // logits that are not numbers: any valid choice
+      if (lane == k) { mine = bi; score = z[bi]; }
+      __syncwarp();
+      if (lane == 0) c[bi] = -INFINITY;
+      __syncwarp();
+    }
+    total += warp_sum(score);
+    if (lane < n) {
+      idx[k0 + lane] = mine;
+      weights[k0 + lane] = score;
+      if (counts) ranks[k0 + lane] = mine < rule.real ? atomicAdd(counts + mine * kCountStride, 1) : -1;
+    }
+  }
+  for (int k = lane; k < top; k += 32) weights[k] = weights[k] / (total + 1e-20f);       // (this lane's own entries)
+}
+
 }  // namespace eb

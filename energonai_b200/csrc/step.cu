@@ -36,6 +36,12 @@ struct StepParams {
   int hidden;
   void *hidden_out;            // [batch][ld_hidden] T
   long long ld_hidden;
+  // bigram table (null: none): the row (previous token * mul_prev + token * mul_cur) mod pair_rows goes to
+  // pair_out; the previous token stands in the column before the new one
+  const void *pair_emb;
+  long long pair_rows, mul_prev, mul_cur;
+  void *pair_out;              // [batch][ld_pair] T
+  long long ld_pair;
   int *counter;                // zero between launches
 };
 
@@ -113,6 +119,15 @@ __global__ void __launch_bounds__(kStepThreads) greedy_step_kernel(const StepPar
     }
   }
 
+  if (p.pair_emb) {
+    // (no column in front of the new token: the table's last row, as for the first token of a sequence)
+    const long long r = col > 0 && col <= p.out_cols ? (p.out_ids[(long long)b * p.ld_out + col - 1] * p.mul_prev + token * p.mul_cur) % p.pair_rows
+                                                     : p.pair_rows;
+    const T *w = reinterpret_cast<const T *>(p.pair_emb) + (r < 0 ? 0 : r) * p.hidden;
+    T *o = reinterpret_cast<T *>(p.pair_out) + (long long)b * p.ld_pair;
+    for (int d = tid; d < p.hidden; d += kStepThreads) o[d] = w[d];
+  }
+
   // every CTA has read the position scalars: the last one advances them
   __syncthreads();
   if (tid == 0) {
@@ -140,10 +155,11 @@ void launch_step(int emb_dtype, int batch, cudaStream_t st, const StepParams &p)
 }
 }  // namespace
 
-extern "C" int eb_greedy_step(const void *logits, long long ld_logits, int batch, int vocab, int dtype, int64_t *out_ids,
+static int greedy_impl(const void *logits, long long ld_logits, int batch, int vocab, int dtype, int64_t *out_ids,
                               long long ld_out, int out_cols, int64_t *tok, int32_t *kv_state, const void *word_emb,
                               long long vocab_start, int vocab_rows, const void *pos_emb, int pos_rows, int add_pos, int hidden,
-                              int emb_dtype, void *hidden_out, long long ld_hidden, int32_t *counter, void *stream) {
+                              int emb_dtype, void *hidden_out, long long ld_hidden, int32_t *counter, const void *pair_emb, long long pair_rows,
+                              long long mul_prev, long long mul_cur, void *pair_out, long long ld_pair, void *stream) {
   if (batch == 0) return EB_OK;
   EB_REQUIRE(dtype_ok(dtype) && (!word_emb || dtype_ok(emb_dtype)), "greedy_step: bad dtype %d / %d", dtype, emb_dtype);
   EB_REQUIRE(batch > 0 && batch <= 65535 && vocab > 0, "greedy_step: bad batch %d or vocabulary %d", batch, vocab);
@@ -161,10 +177,33 @@ extern "C" int eb_greedy_step(const void *logits, long long ld_logits, int batch
   p.word_emb = word_emb; p.vocab_start = vocab_start; p.vocab_rows = vocab_rows;
   p.pos_emb = pos_emb; p.pos_rows = pos_rows; p.add_pos = add_pos; p.hidden = hidden;
   p.hidden_out = hidden_out; p.ld_hidden = ld_hidden; p.counter = counter;
+  if (pair_emb) {
+    EB_REQUIRE(word_emb && pair_out && pair_rows > 0 && ld_pair >= hidden, "greedy_step: the bigram rows go with the embedding and need their output and size");
+    EB_REQUIRE(mul_prev >= 0 && mul_cur >= 0 && mul_prev < (1ll << 31) && mul_cur < (1ll << 31), "greedy_step: bad bigram factors");
+  }
+  p.pair_emb = pair_emb; p.pair_rows = pair_rows; p.mul_prev = mul_prev; p.mul_cur = mul_cur; p.pair_out = pair_out; p.ld_pair = ld_pair;
   cudaStream_t st = as_stream(stream);
   if (!word_emb) emb_dtype = EB_F16;
   if (dtype == EB_F32) launch_step<float>(emb_dtype, batch, st, p);
   else if (dtype == EB_F16) launch_step<__half>(emb_dtype, batch, st, p);
   else launch_step<__nv_bfloat16>(emb_dtype, batch, st, p);
   return check_launch("greedy_step");
+}
+
+extern "C" int eb_greedy_step(const void *logits, long long ld_logits, int batch, int vocab, int dtype, int64_t *out_ids,
+                              long long ld_out, int out_cols, int64_t *tok, int32_t *kv_state, const void *word_emb,
+                              long long vocab_start, int vocab_rows, const void *pos_emb, int pos_rows, int add_pos, int hidden,
+                              int emb_dtype, void *hidden_out, long long ld_hidden, int32_t *counter, void *stream) {
+  return greedy_impl(logits, ld_logits, batch, vocab, dtype, out_ids, ld_out, out_cols, tok, kv_state, word_emb, vocab_start, vocab_rows, pos_emb,
+                     pos_rows, add_pos, hidden, emb_dtype, hidden_out, ld_hidden, counter, nullptr, 0, 0, 0, nullptr, 0, stream);
+}
+
+extern "C" int eb_greedy_step_bigram(const void *logits, long long ld_logits, int batch, int vocab, int dtype, int64_t *out_ids,
+                              long long ld_out, int out_cols, int64_t *tok, int32_t *kv_state, const void *word_emb,
+                              long long vocab_start, int vocab_rows, const void *pos_emb, int pos_rows, int add_pos, int hidden,
+                              int emb_dtype, void *hidden_out, long long ld_hidden, int32_t *counter, const void *pair_emb, long long pair_rows,
+                                     long long mul_prev, long long mul_cur, void *pair_out, long long ld_pair, void *stream) {
+  EB_REQUIRE(pair_emb, "greedy_step: null bigram table");
+  return greedy_impl(logits, ld_logits, batch, vocab, dtype, out_ids, ld_out, out_cols, tok, kv_state, word_emb, vocab_start, vocab_rows, pos_emb,
+                     pos_rows, add_pos, hidden, emb_dtype, hidden_out, ld_hidden, counter, pair_emb, pair_rows, mul_prev, mul_cur, pair_out, ld_pair, stream);
 }

@@ -1,0 +1,119 @@
+"""Python entry to the decaying-memory kernels: state-space (eb_short_conv, eb_ssm_*, eb_gate_group_norm) and gated
+linear (eb_gla_*) layers."""
+import torch
+
+from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
+
+
+def _rows(t, what):
+    if t.dim() != 2 or t.stride(1) != 1:
+        raise RuntimeError(f"{what} must be [rows, columns] with contiguous rows")
+    return t.stride(0)
+
+
+def _state(S, heads, dk, dv):
+    if S.dim() != 4 or tuple(S.shape[1:]) != (heads, dk, dv) or S.dtype != torch.float32 or not S.is_contiguous():
+        raise RuntimeError("decaying memory: the state is fp32 [batch, heads, dk, dv]")
+    return S.shape[0]
+
+
+def _per_head(heads, *vectors):
+    if any(v.dtype != torch.float32 or v.numel() != heads or not v.is_contiguous() for v in vectors):
+        raise RuntimeError("state space: one fp32 number per head")
+
+
+def short_conv(x, w, b, ring, batch, first=None):
+    """Causal convolution per channel and SiLU of a prompt: x [batch*seq, C] (row stride allowed), w [taps, C], b [C];
+    the last inputs go to ring [batch, rows, C].  Returns [batch*seq, C]."""
+    require_cuda(x, w, b, ring, first)
+    ldx, (n, C) = _rows(x, "short_conv: x"), x.shape
+    if w.shape[1] != C or b.numel() != C or not w.is_contiguous() or any(t.dtype != x.dtype for t in (w, b, ring)) or n % batch:
+        raise RuntimeError("short_conv: w [taps, C], b [C] of one dtype, whole sequences")
+    if ring.dim() != 3 or ring.shape[0] != batch or ring.shape[2] != C or ring.stride(2) != 1:
+        raise RuntimeError("short_conv: the ring is [batch, rows, C]")
+    out = torch.empty((n, C), dtype=x.dtype, device=x.device)
+    check(lib().eb_short_conv(ptr(x), ldx, ptr(w), ptr(b), ptr(out), C, batch, n // batch, C, w.shape[0], ptr(first), ptr(ring), ring.stride(0),
+                              ring.stride(1), ring.shape[1], dtype_code(x.dtype), stream_ptr()), "short_conv")
+    return out
+
+
+def ssm_prompt(xbc, dt, dt_bias, a_log, skip, S, heads, groups, dk, dv, first=None):
+    """A prompt through the state-space recurrence; xbc [batch*seq, heads*dv + 2*groups*dk] behind the convolution, dt
+    fp32 [batch*seq, >= heads].  S is overwritten with the state behind the last token.  Returns [batch*seq, heads*dv]."""
+    require_cuda(xbc, dt, dt_bias, a_log, skip, S, first)
+    B, n = _state(S, heads, dk, dv), xbc.shape[0]
+    _per_head(heads, dt_bias, a_log, skip)
+    if xbc.shape[1] != heads * dv + 2 * groups * dk or dt.dtype != torch.float32 or dt.shape[0] != n or dt.shape[1] < heads or n % B:
+        raise RuntimeError("state space: rows [x | B | C], dt fp32, whole sequences")
+    y = torch.empty((n, heads * dv), dtype=xbc.dtype, device=xbc.device)
+    check(lib().eb_ssm_scan(ptr(xbc), _rows(xbc, "xbc"), ptr(dt), _rows(dt, "dt"), ptr(dt_bias), ptr(a_log), ptr(skip), ptr(first), ptr(y), heads * dv,
+                            ptr(S), B, n // B, heads, groups, dk, dv, dtype_code(xbc.dtype), stream_ptr()), "ssm_scan")
+    return y
+
+
+def ssm_step(xbc, conv_w, conv_b, ring, pos_device, dt, dt_bias, a_log, skip, S, heads, groups, dk, dv, first=None):
+    """One token per sequence, xbc [batch, ...] in front of the convolution; the ring and S go on.  Returns [batch, heads*dv]."""
+    require_cuda(xbc, conv_w, conv_b, ring, pos_device, dt, dt_bias, a_log, skip, S, first)
+    B = _state(S, heads, dk, dv)
+    _per_head(heads, dt_bias, a_log, skip)
+    C = heads * dv + 2 * groups * dk
+    if tuple(xbc.shape) != (B, C) or dt.dtype != torch.float32 or dt.shape[0] != B or conv_w.shape[1] != C or not conv_w.is_contiguous() or any(
+            t.dtype != xbc.dtype for t in (conv_w, conv_b, ring)) or tuple(ring.shape[::2]) != (B, C) or ring.stride(2) != 1:
+        raise RuntimeError("state space: one row [x | B | C] per sequence, convolution and ring of its dtype")
+    y = torch.empty((B, heads * dv), dtype=xbc.dtype, device=xbc.device)
+    check(lib().eb_ssm_step(ptr(xbc), _rows(xbc, "xbc"), ptr(conv_w), ptr(conv_b), conv_w.shape[0], ptr(ring), ring.stride(0), ring.stride(1),
+                            ring.shape[1], ptr(pos_device), ptr(first), ptr(dt), _rows(dt, "dt"), ptr(dt_bias), ptr(a_log), ptr(skip), ptr(y),
+                            heads * dv, ptr(S), B, heads, groups, dk, dv, dtype_code(xbc.dtype), stream_ptr()), "ssm_step")
+    return y
+
+
+def gate_group_norm(y, z, norm, eps, heads, dv, parts):
+    """unit(y * silu(z)) * norm, unit over `parts` equal parts of the heads * dv real columns of y [rows, heads*padded]."""
+    require_cuda(y, z, norm)
+    rows, width = y.shape
+    if z.shape != y.shape or any(t.dtype != y.dtype for t in (z, norm)) or norm.numel() != width or width % heads:
+        raise RuntimeError("gate_group_norm: y and z are [rows, heads*dv] of one dtype, the norm has one entry per column")
+    pad = width // heads
+    out = (torch.empty if pad == dv else torch.zeros)((rows, width), dtype=y.dtype, device=y.device)
+    check(lib().eb_gate_group_norm(ptr(y), _rows(y, "y"), ptr(z), _rows(z, "z"), ptr(norm), float(eps), ptr(out), width, rows, heads, int(dv), pad,
+                                   int(parts), dtype_code(y.dtype), stream_ptr()), "gate_group_norm")
+    return out
+
+
+def _qkv(q, k, v, heads, S):
+    dk, dv = q.shape[1] // heads, v.shape[1] // heads
+    if any(t.dim() != 2 or t.stride(1) != 1 or t.stride(0) != q.stride(0) or t.dtype != q.dtype for t in (q, k, v)):
+        raise RuntimeError("gated linear: q, k and v are column ranges of one row layout")
+    if q.shape[1] != heads * dk or k.shape[1] != heads * dk or v.shape[1] != heads * dv:
+        raise RuntimeError("gated linear: q, k and v hold whole heads")
+    return _state(S, heads, dk, dv), dk, dv
+
+
+def gla_prompt(q, k, v, z, tau, scale, S, heads, first=None):
+    """A prompt through the gated linear recurrence: q, k [batch*seq, heads*dk], v [batch*seq, heads*dv] (column views of one
+    projection), z fp32 [batch*seq, heads*dk].  S is overwritten.  Returns [batch*seq, heads*dv]."""
+    require_cuda(q, k, v, z, S, first)
+    B, dk, dv = _qkv(q, k, v, heads, S)
+    n = q.shape[0]
+    if z.dtype != torch.float32 or tuple(z.shape) != (n, heads * dk) or n % B:
+        raise RuntimeError("gated linear: z is fp32 [rows, heads*dk], whole sequences")
+    o = torch.empty((n, heads * dv), dtype=q.dtype, device=q.device)
+    check(lib().eb_gla_scan(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(z), _rows(z, "z"), float(tau), float(scale), ptr(first), ptr(o), heads * dv, ptr(S),
+                            B, n // B, heads, dk, dv, dtype_code(q.dtype), stream_ptr()), "gla_scan")
+    return o
+
+
+def gla_step(q, k, v, g, low, w2, b2, tau, scale, norm, dv_count, eps, S, heads):
+    """One token per sequence: z = w2 low + b2, S goes on; returns unit(o_h) * norm * silu(g), [batch, heads*dv]."""
+    require_cuda(q, k, v, g, low, w2, b2, norm, S)
+    B, dk, dv = _qkv(q, k, v, heads, S)
+    rank = w2.shape[1]
+    if q.shape[0] != B or g.shape != v.shape or any(t.stride(0) != q.stride(0) or t.dtype != q.dtype for t in (g, low)) or low.shape[1] != rank:
+        raise RuntimeError("gated linear: one row per sequence, gate and low-rank part in the same row layout")
+    if not w2.is_contiguous() or w2.shape[0] != heads * dk or b2.numel() != heads * dk or norm.numel() != heads * dv or any(
+            t.dtype != q.dtype for t in (w2, b2, norm)):
+        raise RuntimeError("gated linear: w2 [heads*dk, rank], b2 [heads*dk], norm [heads*dv] of the operand dtype")
+    out = torch.empty((B, heads * dv), dtype=q.dtype, device=q.device)
+    check(lib().eb_gla_step(ptr(q), ptr(k), ptr(v), ptr(g), ptr(low), q.stride(0), ptr(w2), ptr(b2), rank, float(tau), float(scale), ptr(norm),
+                            int(dv_count), float(eps), ptr(out), heads * dv, ptr(S), B, heads, dk, dv, dtype_code(q.dtype), stream_ptr()), "gla_step")
+    return out

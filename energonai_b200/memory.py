@@ -61,13 +61,13 @@ def memory_step(q, k, v, g, gates, bias, cap, scale, norm, dv_count, eps, state,
     return out
 
 
-def head_norm_gate(o, g, norm, heads, dv_count, eps):
-    """unit(o_h) * norm * sigmoid(g) for rows o [rows, heads*dv]; unit over the first dv_count of a head."""
+def head_norm_gate(o, g, norm, heads, dv_count, eps, silu=False):
+    """unit(o_h) * norm * sigmoid(g), or silu(g) instead, for rows o [rows, heads*dv]; unit over the first dv_count of a head."""
     require_cuda(o, g, norm)
     rows, width = o.shape
     if g.shape != o.shape or g.dtype != o.dtype or norm.dtype != o.dtype or norm.numel() != width or o.stride(1) != 1 or g.stride(1) != 1 or width % heads:
         raise RuntimeError("head_norm_gate: o and g are [rows, heads*dv] of one dtype, the norm has one entry per column")
     out = torch.empty((rows, width), dtype=o.dtype, device=o.device)
-    check(lib().eb_head_norm_gate(ptr(o), o.stride(0), ptr(g), g.stride(0), ptr(norm), float(eps), ptr(out), width, rows, heads, width // heads,
-                                  int(dv_count), dtype_code(o.dtype), stream_ptr()), "head_norm_gate")
+    check(lib().eb_head_norm_gate_act(ptr(o), o.stride(0), ptr(g), g.stride(0), ptr(norm), float(eps), ptr(out), width, rows, heads, width // heads,
+                                  int(dv_count), 1 if silu else 0, dtype_code(o.dtype), stream_ptr()), "head_norm_gate")
     return out

@@ -1,4 +1,4 @@
-"""config.json of a layer-listed decoder -> LatentDecoderConfig or SandwichDecoderConfig.
+"""config.json of a layer-listed decoder -> LatentDecoderConfig, SandwichDecoderConfig or HybridDecoderConfig.
 
     {"architecture": ..., "vocab": V, "width": W, "norm": {"eps": e},
      "layers": [{"type": "latent_attention",
@@ -175,3 +175,190 @@ class SandwichDecoderConfig:
             layers.append(SandwichLayerConfig(mixer, mlp))
         return cls(vocab=int(d["vocab"]), width=int(d["width"]), eps=float(d["norm"]["eps"]), embed_scale=float(d["embedding"]["scale"]),
                    layers=layers)
+
+
+# ---- decoders of state-space layers and of attention beside gated linear attention -----------------------
+#
+#     {"architecture": ..., "vocab": V, "width": W, "norm": {"eps": e}, "residual_mult": m, "logit_scale": s,
+#      "embedding": {"bigram": {"buckets", "mul_prev", "mul_cur"}?},
+#      "layers": [{"type": "mamba2", "mixer": {"heads", "vdim", "state", "groups", "conv", "norm_groups"}, "mlp": ...},
+#                 {"type": "parallel", "mixer": {"left": {"heads", "kv_heads", "dim", "vdim", "scale", "mask": {"size"}?,
+#                                                         "rot": {"dims", "base", "scaling": {"factor"}?}?},
+#                                                "right": {"heads", "dim", "vdim", "tau"}},
+#                  "mlp": {"kind": "dense", "ff"} |
+#                         {"kind": "moe", "router": {"experts", "top", "identity"?, "groups": {"count", "keep"}?},
+#                          "expert": {"ff"}, "shared": {"ff"}?} | null}, ...]}
+
+@dataclass
+class StateSpaceConfig:
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int                # taps of the convolution, the current token's included
+    norm_groups: int
+
+
+@dataclass
+class ChunkAttentionConfig:
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    chunk: int = 0           # 0: none
+    rot_dims: int = 0        # 0: no rotation
+    rot_base: float = 1.0
+    rot_factor: float = 1.0  # every frequency is divided by it
+
+    @property
+    def vdim(self):
+        return self.dim      # the values are the keys
+
+
+@dataclass
+class GatedLinearConfig:
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: Optional[int] = None      # of the decay's projection; the checkpoint's shapes give it (with_shapes)
+
+
+@dataclass
+class ParallelConfig:
+    left: ChunkAttentionConfig
+    right: GatedLinearConfig
+
+
+@dataclass
+class RoutedConfig:
+    experts: int
+    top: int
+    ff: int
+    identity: int = 0        # further choices, which return the input itself
+    groups: int = 1
+    keep: int = 1
+    shared_ff: int = 0       # 0: no shared expert
+
+
+@dataclass
+class HybridLayerConfig:
+    mixer: Union[StateSpaceConfig, ParallelConfig]
+    mlp: Optional[Union[DenseConfig, RoutedConfig]] = None
+
+
+@dataclass
+class BigramConfig:
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+def _need(ok, where, what):
+    if not ok:
+        raise ValueError(f"{where}: {what}")
+
+
+def _sizes(where, d, *names):
+    out = [int(d[n]) for n in names]
+    _need(all(v > 0 for v in out), where, f"{', '.join(names)} must be positive (got {out})")
+    return out
+
+
+@dataclass
+class HybridDecoderConfig:
+    vocab: int
+    width: int
+    eps: float
+    residual_mult: float
+    logit_scale: float
+    layers: List[HybridLayerConfig]
+    bigram: Optional[BigramConfig] = None
+
+    @staticmethod
+    def _mixer(where, kind, m):
+        if kind == "mamba2":
+            _known(where, m, ("heads", "vdim", "state", "groups", "conv", "norm_groups"))
+            c = StateSpaceConfig(*_sizes(where, m, "heads", "vdim", "state", "groups", "conv", "norm_groups"))
+            _need(c.heads % c.groups == 0, where, f"{c.heads} heads do not share {c.groups} groups")
+            _need(c.heads * c.vdim % c.norm_groups == 0, where, f"{c.heads * c.vdim} columns have no {c.norm_groups} equal parts")
+            return c
+        if kind != "parallel":
+            raise ValueError(f"{where}: unknown type {kind!r}")
+        _known(where, m, ("left", "right"))
+        a, r = m["left"], m["right"]
+        _known(where, a, ("heads", "kv_heads", "dim", "vdim", "scale", "mask", "rot"))
+        heads, kv_heads, dim, vdim = _sizes(where, a, "heads", "kv_heads", "dim", "vdim")
+        _need(heads % kv_heads == 0, where, f"{heads} heads do not share {kv_heads} key / value heads")
+        _need(vdim == dim, where, f"the values are the keys: vdim {vdim} is not dim {dim}")
+        left = ChunkAttentionConfig(heads, kv_heads, dim, float(a["scale"]))
+        if a.get("mask"):
+            _known(where, a["mask"], ("size",))
+            left.chunk, = _sizes(where, a["mask"], "size")
+        if a.get("rot"):
+            rot = a["rot"]
+            _known(where, rot, ("dims", "base", "scaling"))
+            left.rot_dims, left.rot_base = int(rot["dims"]), float(rot["base"])
+            _need(0 <= left.rot_dims <= dim and left.rot_dims % 2 == 0 and left.rot_base > 0, where, f"{left.rot_dims} rotated dimensions of {dim}")
+            if rot.get("scaling"):
+                _known(where, rot["scaling"], ("factor",))
+                left.rot_factor = float(rot["scaling"]["factor"])
+                _need(left.rot_factor > 0, where, f"a rotation slowed down by {left.rot_factor}")
+        _known(where, r, ("heads", "dim", "vdim", "tau", "rank"))
+        right = GatedLinearConfig(*_sizes(where, r, "heads", "dim", "vdim"), tau=float(r["tau"]), rank=int(r["rank"]) if r.get("rank") else None)
+        _need(right.tau > 0, where, f"tau {right.tau}")
+        return ParallelConfig(left, right)
+
+    @staticmethod
+    def _mlp(where, f):
+        if f is None:
+            return None
+        if f["kind"] == "dense":
+            _known(where, f, ("kind", "ff"))
+            return DenseConfig(*_sizes(where, f, "ff"))
+        if f["kind"] != "moe":
+            raise ValueError(f"{where}: unknown feed-forward kind {f['kind']!r}")
+        _known(where, f, ("kind", "router", "expert", "shared"))
+        r = f["router"]
+        _known(where, r, ("experts", "top", "identity", "groups"))
+        _known(where, f["expert"], ("ff",))
+        c = RoutedConfig(*_sizes(where, r, "experts", "top"), *_sizes(where, f["expert"], "ff"), identity=int(r.get("identity") or 0))
+        if r.get("groups"):
+            _known(where, r["groups"], ("count", "keep"))
+            c.groups, c.keep = _sizes(where, r["groups"], "count", "keep")
+        if f.get("shared"):
+            _known(where, f["shared"], ("ff",))
+            c.shared_ff, = _sizes(where, f["shared"], "ff")
+        choices = c.experts + c.identity
+        _need(c.identity >= 0 and choices % c.groups == 0 and c.keep <= c.groups, where, f"{choices} choices in {c.groups} groups of which {c.keep} are kept")
+        _need(c.top <= choices // c.groups * c.keep, where, f"top {c.top} of {choices // c.groups * c.keep} open choices")
+        return c
+
+    @classmethod
+    def from_dict(cls, d):
+        layers = []
+        for i, ly in enumerate(d["layers"]):
+            where = f"layer {i}"
+            _known(where, ly, ("type", "mixer", "mlp"))
+            layers.append(HybridLayerConfig(cls._mixer(where, ly["type"], ly["mixer"]), cls._mlp(where, ly.get("mlp"))))
+        _known("model", d, ("architecture", "vocab", "width", "norm", "residual_mult", "logit_scale", "embedding", "layers"))
+        _known("norm", d["norm"], ("eps",))
+        emb = d.get("embedding") or {}
+        _known("embedding", emb, ("bigram",))
+        bigram = None
+        if emb.get("bigram"):
+            _known("bigram", emb["bigram"], ("buckets", "mul_prev", "mul_cur"))
+            b = emb["bigram"]
+            bigram = BigramConfig(*_sizes("bigram", b, "buckets"), int(b["mul_prev"]), int(b["mul_cur"]))
+            _need(0 <= bigram.mul_prev < 1 << 31 and 0 <= bigram.mul_cur < 1 << 31, "bigram", "its factors are not negative")
+        return cls(*_sizes("model", d, "vocab", "width"), eps=float(d["norm"]["eps"]), residual_mult=float(d["residual_mult"]),
+                   logit_scale=float(d["logit_scale"]), layers=layers, bigram=bigram)
+
+    def with_shapes(self, shapes):
+        """Takes the sizes that only a checkpoint gives, {tensor name: shape}: the rank of each decay projection."""
+        for i, lc in enumerate(self.layers):
+            if isinstance(lc.mixer, ParallelConfig) and f"l{i}.mix.right.a1" in shapes:
+                rank = int(shapes[f"l{i}.mix.right.a1"][0])
+                _need(lc.mixer.right.rank in (None, rank), f"layer {i}", f"the decay's projection has rank {rank}, the configuration asks for {lc.mixer.right.rank}")
+                lc.mixer.right.rank = rank
+        return self

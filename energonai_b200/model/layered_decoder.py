@@ -19,9 +19,12 @@ class LayeredDecoder(GenerationModel):
     """A subclass fills self.layers in build_layers() and supplies
       caches()                    {layer: RingCache or RecurrentState} of an empty state
       run(rows, ctx, on_layer)    embedding rows (operand dtype) through all layers -> (x, h): the fp32
-                                  stream, and its final norm if it is at hand (else None)"""
+                                  stream, and its final norm if it is at hand (else None)
+    and, where the rows are more than the tokens' own,
+      embed_prompt(input_ids), embed_step(tokens)    what run() takes as rows"""
     eos_token_id = -1            # the configurations name no stop token
     norm_offset = 0.0            # 1.0: norm weights are stored around zero
+    tied = False                 # the head is the embedding table
 
     def __init__(self, config, dtype=torch.bfloat16, device=None):
         super().__init__()
@@ -31,11 +34,11 @@ class LayeredDecoder(GenerationModel):
         self.config, self.dtype = config, dtype
         self.vocab, self.width, self.hidden_size = config.vocab, config.width, round_up(config.width, 8)
         kw = dict(dtype=dtype, device=device)
-        self.embed = init_weight(self.vocab, self.hidden_size, **kw)
+        self.embed = init_weight(round_up(self.vocab, 8) if self.tied else self.vocab, self.hidden_size, **kw)
         self.layers = nn.ModuleList()
         self.build_layers(config, **kw)
         self.norm = RMSNorm1D(self.hidden_size, eps=config.eps, count=self.width, offset=self.norm_offset, **kw)
-        self.head = init_weight(round_up(self.vocab, 8), self.hidden_size, **kw)
+        self.head = self.embed if self.tied else init_weight(round_up(self.vocab, 8), self.hidden_size, **kw)
         self.state = self.new_state()
         self._reserve = 0
 
@@ -64,7 +67,13 @@ class LayeredDecoder(GenerationModel):
         if self.state.padded and self.dtype != torch.float32:
             mask = (torch.arange(S, device=dev)[None, :] < self.state.first[:, None]).to(self.dtype) * -10000.0
         ctx = PromptContext(self.state, B, S, mask)
-        return self.run(nn.functional.embedding(input_ids.reshape(-1), self.embed), ctx, on_layer)[0]
+        return self.run(self.embed_prompt(input_ids), ctx, on_layer)[0]
+
+    def embed_prompt(self, input_ids):
+        return nn.functional.embedding(input_ids.reshape(-1), self.embed)
+
+    def embed_step(self, tokens):
+        return nn.functional.embedding(tokens.reshape(-1), self.embed)
 
     def _step(self, rows):
         x, h = self.run(rows, StepContext(self.state))
@@ -76,7 +85,7 @@ class LayeredDecoder(GenerationModel):
         if tokens.numel() != self.state.batch:
             raise ValueError(f"step: {tokens.numel()} tokens for {self.state.batch} sequences")
         self.state.ensure(self.state.length + 1)
-        logits = self._step(nn.functional.embedding(tokens.reshape(-1), self.embed))
+        logits = self._step(self.embed_step(tokens))
         self.state.advance()
         return logits
 

@@ -6,7 +6,7 @@ from typing import Callable, Optional
 import torch
 from torch import dtype, nn
 
-from ..gemm import project, project_parts, xielu_params
+from ..gemm import project, project_parts, project_unit, xielu_params
 from ..nn import Linear1D_Col, Linear1D_Row, init_weight
 from .sequence_state import round_up
 
@@ -71,3 +71,22 @@ class XIELUFeedForward(nn.Module):
         """-> (y, pre-activation of its gate)."""
         u = project_parts(h, self.up, bias=self.bias, xielu=(self.act, self.ff_padded))
         return project(u[:, :self.ff_padded], self.down), u[:, self.ff_padded:]
+
+
+class GEGLUFeedForward(nn.Module):
+    """W_down (gelu_tanh(W_gate h) * (W_up h)); gates and ups interleaved in blocks of 8 rows, the unit in the epilogue
+    of their product."""
+
+    def __init__(self, width, ff, dtype, device=None):
+        super().__init__()
+        kw = dict(dtype=dtype, device=device)
+        self.ff, self.ff_padded = ff, round_up(ff, 8)
+        self.gate_up = init_weight(2 * self.ff_padded, width, **kw)
+        self.down = init_weight(width, self.ff_padded, **kw)
+
+    def router_for_step(self, tokens):
+        return None
+
+    def forward(self, h, first=None, rows_per_batch=1, routed=None):
+        """-> what stream_add adds."""
+        return dict(y=project(project_unit(h, self.gate_up, "geglu"), self.down))

@@ -58,16 +58,16 @@ class RingCache(KVCache):
 
 
 class RecurrentState:
-    """fp32 tensors [batch, ...] that a recurrent layer carries from token to token; `shapes` gives each
-    one's size per sequence.  A new batch starts from zero."""
+    """fp32 tensors (or of another type) [batch, ...] that a recurrent layer carries from token to token;
+    `shapes` gives each one's size per sequence.  A new batch starts from zero."""
 
-    def __init__(self, shapes):
-        self.shapes, self.tensors, self.len = [tuple(s) for s in shapes], None, 0
+    def __init__(self, shapes, dtype=torch.float32):
+        self.shapes, self.dtype, self.tensors, self.len = [tuple(s) for s in shapes], dtype, None, 0
 
     def prepare(self, batch, positions, dtype, device):
         t = self.tensors
         if t is None or t[0].shape[0] != batch or t[0].device != device:
-            self.tensors = [torch.zeros((batch,) + s, dtype=torch.float32, device=device) for s in self.shapes]
+            self.tensors = [torch.zeros((batch,) + s, dtype=self.dtype, device=device) for s in self.shapes]
         else:
             for x in t:
                 x.zero_()
@@ -80,7 +80,7 @@ class RecurrentState:
         self.tensors = [t.index_select(0, rows) for t in self.tensors]
 
     def fork(self):
-        out = RecurrentState(self.shapes)
+        out = RecurrentState(self.shapes, self.dtype)
         out.tensors, out.len = self.tensors, self.len
         return out
 
@@ -97,7 +97,7 @@ class SequenceState:
     successor) lives on the device, where captured steps advance it."""
 
     def __init__(self, caches):
-        self.caches = caches                    # {layer: RingCache or RecurrentState}
+        self.caches = caches                    # {layer, or (layer, part): RingCache or RecurrentState}
         self.first = self.kv_state = None
         self.batch, self.length, self.padded = 0, 0, False
 

@@ -10,6 +10,42 @@ ROW_TILE = 128           # rows of one expert come in tiles of this many in the 
 SKINNY_MAX_ENTRIES = 10240   # (token, choice) pairs the weight-streaming product sorts in shared memory
 
 
+UNITS = {None: 0, "clamped": 1, "geglu": 2, "gelu": 3}      # EB_UNIT_*
+GATED = ("clamped", "geglu")
+
+
+def unit_code(unit, gate):
+    """(code, limit, alpha, columns per result) of a unit; gate = (limit, alpha) alone names the clamped one."""
+    if gate is not None and unit is None:
+        unit = "clamped"
+    limit, alpha = gate if gate is not None else (0.0, 0.0)
+    return UNITS[unit], float(limit), float(alpha), 2 if unit in GATED else 1
+
+
+class RouterRule:
+    """How a router chooses: `choices` softmax scores, those from `experts` on standing for the input itself;
+    correction fp32 [choices] or None is added for the choice; of `groups` equal groups the best `keep`
+    are open; the weights of the chosen are their scores over their sum."""
+
+    def __init__(self, choices, experts, correction=None, groups=1, keep=1):
+        self.choices, self.experts, self.correction, self.groups, self.keep = choices, experts, correction, groups, keep
+
+
+def route_rule(logits, rule, top, first=None, rows_per_batch=0, counts=None, gated=False):
+    """logits [T, >= choices (+ 1 if gated)] fp32 -> (idx, weights, ranks or None, shared gate or None)."""
+    require_cuda(logits, first, counts, rule.correction)
+    if logits.dim() != 2 or logits.dtype != torch.float32 or logits.stride(1) != 1 or logits.shape[1] < rule.choices + int(gated):
+        raise RuntimeError("moe route: logits must be fp32 [tokens, choices]")
+    T, dev = logits.shape[0], logits.device
+    idx = torch.empty((T, top), dtype=torch.int32, device=dev)
+    w = torch.empty((T, top), dtype=torch.float32, device=dev)
+    ranks = torch.empty((T, top), dtype=torch.int32, device=dev) if counts is not None else None
+    gate = torch.empty(T, dtype=torch.float32, device=dev) if gated else None
+    check(lib().eb_moe_route_rule(ptr(logits), logits.stride(0), T, rule.choices, rule.experts, top, ptr(rule.correction), rule.groups, rule.keep,
+                                  ptr(first), rows_per_batch, ptr(idx), ptr(w), ptr(counts), ptr(ranks), ptr(gate), stream_ptr()), "moe_route")
+    return idx, w, ranks, gate
+
+
 def new_counts(experts, device):
     """Zeroed row counters of the experts; route() fills them, SortedRows zeroes them again."""
     return torch.zeros(experts * COUNT_STRIDE, dtype=torch.int32, device=device)
@@ -50,38 +86,43 @@ class SortedRows:
                                    ptr(self.rows), ptr(self.x), self.x.stride(0), n, stream_ptr()), "moe_permute")
 
 
-def grouped_gemm(a, w, plan, gate=None):
-    """a [rows of the plan, K], w [experts, N, K] -> [rows, N], or [rows, N/2] with gate = (limit,
-    alpha): the clamped gated unit on columns in blocks of 8 gates and their 8 ups."""
+def grouped_gemm(a, w, plan, gate=None, unit=None):
+    """a [rows of the plan, K], w [experts, N, K] -> [rows, N], or a unit of it: "gelu"; gated ones give
+    [rows, N/2] from columns in blocks of 8 gates and their 8 ups ("geglu"; gate = (limit, alpha): the
+    clamped one)."""
     require_cuda(a, w)
     E, N, K = w.shape
     M = a.shape[0]
     if not w.is_contiguous() or a.dtype != w.dtype or a.shape[1] != K or a.stride(1) != 1:
         raise RuntimeError("grouped gemm: a [rows, K] and contiguous w [experts, N, K] of one dtype required")
-    limit, alpha = gate if gate is not None else (0.0, 0.0)
+    code, limit, alpha, per = unit_code(unit, gate)
     if a.dtype == torch.float32:
         out = torch.empty((M, N), dtype=a.dtype, device=a.device)
         check(lib().eb_gemm_f32(ptr(a), a.stride(0), 0, ptr(w), K, N * K, ptr(out), N, 0, M, N, K, 1, ptr(plan.tile_group),
                                 ptr(plan.live_tiles), None, 0, None, stream_ptr()), "gemm_f32")
-        return gated_act(out, limit, alpha) if gate is not None else out
-    out = torch.empty((M, N // 2 if gate is not None else N), dtype=a.dtype, device=a.device)
+        return unit_act(out, unit, gate) if code else out
+    out = torch.empty((M, N // per), dtype=a.dtype, device=a.device)
     check(lib().eb_gemm_grouped(ptr(a), a.stride(0), ptr(w), K, ptr(out), out.stride(0), M, N, K, E, ptr(plan.tile_group),
-                                ptr(plan.live_tiles), 1 if gate is not None else 0, float(limit), float(alpha), dtype_code(a.dtype),
-                                stream_ptr()), "gemm_grouped")
+                                ptr(plan.live_tiles), code, limit, alpha, dtype_code(a.dtype), stream_ptr()), "gemm_grouped")
     return out
 
 
-def gated_act(x, limit, alpha):
-    """[n, 2*half] in the 8 + 8 column order -> [n, half]."""
+def unit_act(x, unit=None, gate=None):
+    """A unit alone: [n, N] -> [n, N], or, gated, [n, 2*half] in the 8 + 8 column order -> [n, half]."""
     require_cuda(x)
-    half = x.shape[1] // 2
-    y = torch.empty((x.shape[0], half), dtype=x.dtype, device=x.device)
-    check(lib().eb_gated_act(ptr(x), x.stride(0), ptr(y), half, x.shape[0], half, float(limit), float(alpha), dtype_code(x.dtype),
-                             stream_ptr()), "gated_act")
+    code, limit, alpha, per = unit_code(unit, gate)
+    n = x.shape[1] // per
+    y = torch.empty((x.shape[0], n), dtype=x.dtype, device=x.device)
+    check(lib().eb_unit_act(ptr(x), x.stride(0), ptr(y), n, x.shape[0], n, code, limit, alpha, dtype_code(x.dtype), stream_ptr()), "unit_act")
     return y
 
 
-def skinny_experts(a, w, idx, a_div, gate=None):
+def gated_act(x, limit, alpha):
+    """[n, 2*half] in the 8 + 8 column order -> [n, half], the clamped unit."""
+    return unit_act(x, gate=(limit, alpha))
+
+
+def skinny_experts(a, w, idx, a_div, gate=None, unit=None):
     """Generation steps: entry i of idx (flattened [T, top]) multiplies row i // a_div of a by the
     weights w [experts, N, K] of expert idx[i] -> [T * top, N or N/2]; rows of unrouted entries are
     not written."""
@@ -90,11 +131,10 @@ def skinny_experts(a, w, idx, a_div, gate=None):
     n = idx.numel()
     if not w.is_contiguous() or a.dtype != w.dtype or a.shape[1] != K or a.stride(1) != 1 or a.shape[0] * a_div < n:
         raise RuntimeError("skinny product: a [rows, K] and contiguous w [experts, N, K] of one dtype required")
-    limit, alpha = gate if gate is not None else (0.0, 0.0)
-    out = torch.empty((n, N // 2 if gate is not None else N), dtype=a.dtype, device=a.device)
+    code, limit, alpha, per = unit_code(unit, gate)
+    out = torch.empty((n, N // per), dtype=a.dtype, device=a.device)
     check(lib().eb_grouped_skinny(ptr(a), a.stride(0), 0, a_div, ptr(w), N * K, K, ptr(out), out.stride(0), 0, ptr(idx), n, E, N, K,
-                                  1 if gate is not None else 0, float(limit), float(alpha), dtype_code(a.dtype), stream_ptr()),
-          "grouped_skinny")
+                                  code, limit, alpha, dtype_code(a.dtype), stream_ptr()), "grouped_skinny")
     return out
 
 

@@ -1,4 +1,4 @@
-"""Python entry to the RMS-norm kernels (eb_rms_norm / eb_rms_residual / eb_stream_update)."""
+"""Python entry to the RMS-norm kernels (eb_rms_norm / eb_rms_residual / eb_stream_update / eb_stream_add)."""
 import torch
 
 from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
@@ -79,3 +79,43 @@ def stream_update(x, eps, count=None, src=None, src_scale=1.0, y=None, gate=None
                                  ld(x, "x"), ptr(w_next), ptr(h), n2, float(eps), n1, n2, count or n2, dtype_code(t.dtype), stream_ptr()),
           "stream_update")
     return h
+
+
+def stream_add(x, eps, count=None, src=None, src2=None, y=None, w=None, y2=None, w2=None, mix=None, ident=None, experts=0, shared=None, gate=None,
+               scale=1.0, w_next=None, next_scale=1.0, router=None):
+    """The residual step of blocks with a norm in front of every sublayer only; x [n1, n2] fp32 in place:
+      x = src + src2 (if src is given);  x += scale * Y;  returns h = norm(x) * w_next * next_scale (None
+      without w_next).
+    Y is y; with y2, norm(y) * w + norm(y2) * w2 (w, w2 fp32); with mix = (idx, rows or None, weights), the
+    weighted sum of a token's expert rows y, of ident for choices from `experts` on, and gate * shared.
+    router = (weight, RouterRule, top, gated): returns (h, (idx, weights, shared gate or None)) of the
+    mixture that follows."""
+    require_cuda(x, src, src2, y, w, y2, w2, ident, shared, gate, w_next)
+    n1, n2 = x.shape
+    t = next((a for a in (src, y, w_next) if a is not None), None)
+    if t is None or x.dtype != torch.float32 or any(a is not None and a.dtype != t.dtype for a in (src, src2, y, y2, ident, shared, w_next)):
+        raise RuntimeError("stream_add: x is fp32, the other rows share a dtype")
+    if any(a is not None and tuple(a.shape) != (n1, n2) for a in (src, src2, y if mix is None else None, y2, ident, shared)) or any(
+            a is not None and a.shape[-1] != n2 for a in (y, w, w2, w_next)):
+        raise RuntimeError("stream_add: everything is [rows, width] of one width")
+    if any(a is not None and a.dtype != torch.float32 for a in (w, w2, gate)):
+        raise RuntimeError("stream_add: w, w2 and gate are fp32")
+    idx, rows, weights = mix if mix is not None else (None, None, None)
+    h = torch.empty((n1, n2), dtype=t.dtype, device=x.device) if w_next is not None else None
+    ld = lambda a, what: _rows(a, f"stream_add: {what}") if a is not None else 0
+    rw = r_idx = r_w = r_gate = rule = None
+    top = 0
+    if router is not None:
+        rw, rule, top, gated = router
+        if rw.dtype != t.dtype or not rw.is_contiguous() or rw.shape[1] != n2 or rw.shape[0] < rule.choices + int(gated):
+            raise RuntimeError("stream_add: the router weight must be contiguous [choices, width]")
+        r_idx = torch.empty((n1, top), dtype=torch.int32, device=x.device)
+        r_w = torch.empty((n1, top), dtype=torch.float32, device=x.device)
+        r_gate = torch.empty(n1, dtype=torch.float32, device=x.device) if gated else None
+    check(lib().eb_stream_add(ptr(src), ld(src, "src"), ptr(src2), ld(src2, "src2"), ptr(y), ld(y, "y"), ptr(w), ptr(y2), ld(y2, "y2"), ptr(w2),
+                              ptr(idx), ptr(rows), ptr(weights), idx.shape[1] if idx is not None else 0, int(experts), ptr(ident), ld(ident, "ident"),
+                              ptr(shared), ld(shared, "shared"), ptr(gate), float(scale), ptr(x), ld(x, "x"), ptr(w_next), float(next_scale), ptr(h), n2,
+                              float(eps), n1, n2, count or n2, ptr(rw), rule.choices if rule else 0, rule.experts if rule else 0, top,
+                              ptr(rule.correction) if rule else None, rule.groups if rule else 1, rule.keep if rule else 1, ptr(r_idx), ptr(r_w),
+                              ptr(r_gate), dtype_code(t.dtype), stream_ptr()), "stream_add")
+    return (h, (r_idx, r_w, r_gate)) if router is not None else h

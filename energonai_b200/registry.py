@@ -15,8 +15,9 @@ DTYPES = {"float32": torch.float32, "float16": torch.float16, "bfloat16": torch.
 
 
 class Architecture:
-    """config: class with from_dict(); model: class taking (config, dtype, device); convert(state,
-    model): checkpoint tensors -> the model's parameters."""
+    """config: class with from_dict() and, where only a checkpoint's shapes give some size, with_shapes();
+    model: class taking (config, dtype, device); convert(state, model): checkpoint tensors -> the model's
+    parameters."""
 
     def __init__(self, name, config, model, convert):
         self.name, self.config, self.model, self.convert = name, config, model, convert
@@ -56,7 +57,7 @@ def read_config(folder):
 
 def load_model(folder, dtype="bfloat16", device=None):
     """The model of a folder, its weights loaded, on `device` (default: the current GPU)."""
-    from .utils import load_checkpoint
+    from .utils import load_checkpoint, load_state_dict
     _populate()
     config = read_config(folder)
     name = config.get("architecture")
@@ -64,9 +65,13 @@ def load_model(folder, dtype="bfloat16", device=None):
         raise ValueError(f"{folder}: architecture {name!r} is not registered (known: {', '.join(sorted(_ARCHITECTURES))})")
     arch = _ARCHITECTURES[name]
     dtype = DTYPES[dtype] if isinstance(dtype, str) else dtype
-    model = arch.model(arch.config.from_dict(config), dtype=dtype)
     weights = os.path.join(folder, "model.safetensors")
-    load_checkpoint(weights if os.path.exists(weights) else folder, model, preprocess_fn=lambda state: arch.convert(state, model))
+    weights = weights if os.path.exists(weights) else folder
+    sizes = arch.config.from_dict(config)
+    if hasattr(sizes, "with_shapes"):
+        sizes = sizes.with_shapes({k: tuple(v.shape) for k, v in load_state_dict(weights).items()})
+    model = arch.model(sizes, dtype=dtype)
+    load_checkpoint(weights, model, preprocess_fn=lambda state: arch.convert(state, model))
     return model.to(device if device is not None else torch.device("cuda", torch.cuda.current_device())).eval()
 
 
@@ -79,9 +84,11 @@ def _populate():
         return
     _done = True
     from . import model as M
-    from .model.config import LatentDecoderConfig, SandwichDecoderConfig
+    from .model.config import HybridDecoderConfig, LatentDecoderConfig, SandwichDecoderConfig
+    from .model.hybrid_decoder import HybridDecoder
     from .model.latent_decoder import LatentDecoder
     from .model.sandwich_decoder import SandwichDecoder
+    from .utils.checkpointing_moponex import processing_Moponex
     from .utils.checkpointing_mutolix import processing_Mutolix
     from .utils.checkpointing_tulezen import processing_Tulezen
     for name in ("opt_125M", "opt_6B", "opt_13B", "opt_30B", "opt_66B", "opt_175B", "gpt2_small", "gpt2_large", "gpt2_8B", "gpt3",
@@ -89,3 +96,4 @@ def _populate():
         register_factory(name, getattr(M, name))
     register_architecture("Tulezen", LatentDecoderConfig, LatentDecoder, processing_Tulezen)
     register_architecture("Mutolix", SandwichDecoderConfig, SandwichDecoder, processing_Mutolix)
+    register_architecture("Moponex", HybridDecoderConfig, HybridDecoder, processing_Moponex)

@@ -48,6 +48,16 @@ extern "C" {
 #define EB_ACT_GELU_ERF 3  /* torch.nn.functional.gelu                                      */
 #define EB_ACT_XIELU 4     /* eb_gemm_parts, eb_gemm_f32                                    */
 
+/* units of a feed-forward, fp32 on the accumulators.  The gated ones read columns in blocks of 8 gates g
+ * and their 8 ups u and give half as many:
+ *   CLAMPED  g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit)
+ *   GEGLU    gelu_tanh(g) u
+ *   GELU     gelu(x) of every column, the erf form (no gate) */
+#define EB_UNIT_NONE 0
+#define EB_UNIT_CLAMPED 1
+#define EB_UNIT_GEGLU 2
+#define EB_UNIT_GELU 3
+
 /* flags for eb_gemm */
 #define EB_GEMM_STATIC_W 1 /* W is constant (model weights): the kernel may start reading it while
                               earlier work of the stream is still running */
@@ -353,21 +363,24 @@ EB_API size_t eb_decode_chain_workspace_bytes(const eb_chain_op *ops, int n_ops,
  * multiplied by the weights of group tile_group[i].  W holds the groups' [N, K] matrices one below
  * the other ([groups * N, K], rows ldw apart); only the first *live_tiles row tiles are processed
  * (both device memory, read at run time).  M, a multiple of 128, is the room A and C have.
- * gated != 0: the columns of a group come in blocks of 8 gates and their 8 ups and
- *   C[m][8b + j] = g * sigmoid(alpha * g) * (u + 1),  g = min(gate, limit), u = clamp(up, -limit, limit)
- * (C is [M, N/2]), the activation in fp32 on the accumulators.  fp16 / bf16. */
+ * unit: EB_UNIT_* (a gated one: C is [M, N/2]).  fp16 / bf16. */
 EB_API int eb_gemm_grouped(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, int M, int N, int K,
-                    int groups, const int32_t *tile_group, const int32_t *live_tiles, int gated, float limit, float alpha,
+                    int groups, const int32_t *tile_group, const int32_t *live_tiles, int unit, float limit, float alpha,
                     int dtype, void *stream);
+
+/* C = gated unit of (A . W^T), W [N, K] in blocks of 8 gate rows and their 8 up rows, C [M, N/2]: eb_gemm with a
+ * gated unit, in both orientations (workspace as eb_gemm). */
+EB_API int eb_gemm_gated(const void *A, long long lda, const void *W, long long ldw, void *C, long long ldc, int M, int N, int K, int unit,
+                  float limit, float alpha, int dtype, int flags, void *workspace, size_t workspace_bytes, void *stream);
 
 /* The same kind of product for a handful of rows per group (generation steps), as one pass over
  * the weights of the groups that have rows.  idx != NULL: entry i of the list (rows entries)
  * belongs to group idx[i] (negative: none), reads row i / a_div of A and writes row i of C.  idx
  * NULL: every group takes all rows, with group strides on A and C (heads of an absorbed attention
- * projection).  Strides in elements; gated as above. */
+ * projection).  Strides in elements; unit as above. */
 EB_API int eb_grouped_skinny(const void *A, long long lda, long long a_group_stride, int a_div, const void *W,
                       long long w_group_stride, long long ldw, void *C, long long ldc, long long c_group_stride,
-                      const int32_t *idx, int rows, int groups, int N, int K, int gated, float limit, float alpha, int dtype,
+                      const int32_t *idx, int rows, int groups, int N, int K, int unit, float limit, float alpha, int dtype,
                       void *stream);
 
 /* C = A . W^T in true 32-bit.  Strided groups, or row tiles with their group (one of the two).  A single
@@ -378,7 +391,10 @@ EB_API int eb_gemm_f32(const float *A, long long lda, long long a_group_stride, 
                 const int32_t *tile_group, const int32_t *live_tiles, const float *bias, int act_cols, const float *act_params,
                 void *stream);
 
-/* The gated activation alone: x [n1, 2*half] in the 8 + 8 column order -> y [n1, half]. */
+/* A unit alone: x [n1, n2] or, gated, [n1, 2*n2] in the 8 + 8 column order -> y [n1, n2].
+ * eb_gated_act: the clamped one. */
+EB_API int eb_unit_act(const void *x, long long ldx, void *y, long long ldy, int n1, int n2, int unit, float limit, float alpha,
+                int dtype, void *stream);
 EB_API int eb_gated_act(const void *x, long long ldx, void *y, long long ldy, int n1, int half, float limit, float alpha,
                  int dtype, void *stream);
 
@@ -391,12 +407,22 @@ EB_API int eb_gated_act(const void *x, long long ldx, void *y, long long ldy, in
 EB_API int eb_moe_route(const float *logits, long long ld, int tokens, int experts, int top, const int32_t *first,
                  int rows_per_batch, int32_t *idx, float *weights, int32_t *counts, int32_t *ranks, void *stream);
 
+/* Router with a rule.  Scores are the softmax over all `choices` logits, of which the first `experts` are experts
+ * and the others stand for the input itself (they take no ticket: rank -1).  Choice scores are score +
+ * correction (or NULL).  The choices form `groups` equal groups of neighbours; only the `keep` groups with
+ * the largest choice score in them are open.  The `top` largest choice scores of the open groups are
+ * chosen; the weights are their scores, divided by their sum (+ 1e-20).  shared_gate (or NULL)[t] =
+ * sigmoid of the logit behind the choices (0 for padding).  Otherwise as eb_moe_route. */
+EB_API int eb_moe_route_rule(const float *logits, long long ld, int tokens, int choices, int experts, int top, const float *correction,
+                      int groups, int keep, const int32_t *first, int rows_per_batch, int32_t *idx, float *weights, int32_t *counts,
+                      int32_t *ranks, float *shared_gate, void *stream);
+
 /* Row layout in which every expert owns whole 128-row tiles: offsets[e], tile_group[] (at most
  * max_tiles), *live_tiles; counts are zeroed for the next batch. */
 EB_API int eb_moe_plan(int32_t *counts, int experts, int32_t *offsets, int32_t *tile_group, int max_tiles, int32_t *live_tiles,
                 void *stream);
 
-/* rows[t][k] = offsets[idx] + rank (or -1) and out[rows[t][k]] = x[t]. */
+/* rows[t][k] = offsets[idx] + rank (or -1: no index or no rank) and out[rows[t][k]] = x[t]. */
 EB_API int eb_moe_permute(const void *x, long long ldx, int n2, int dtype, int tokens, int top, const int32_t *idx,
                    const int32_t *ranks, const int32_t *offsets, int32_t *rows, void *out, long long ldo, int max_rows,
                    void *stream);
@@ -431,6 +457,22 @@ EB_API int eb_stream_update(const void *src, long long lds, float src_scale, con
                      long long ldg, const float *w_out, float *x, long long ldx, const void *w_next, void *h, long long ldh,
                      float eps, int n1, int n2, int count, int dtype, void *stream);
 
+/* The residual step of blocks with a norm in front of every sublayer only, per row of n2 elements (means over
+ * the first `count`):
+ *   x = src + src2               if src (embedding rows, `dtype`; src2 or NULL), else x as it is (fp32)
+ *   x += scale * Y               Y = y;  with y2: norm(y) * w + norm(y2) * w2 (w, w2 fp32);  with idx, the output of
+ *                                a mixture: sum_k weights[t][k] * (idx[t][k] < experts ? y[rows ? rows[t][k] :
+ *                                t*top + k] : ident[t]) over the k with idx >= 0, + gate[t] * shared[t]
+ *   h = norm(x) * w_next * next_scale          if w_next; h in `dtype`
+ * router (or NULL, [choices (+ 1 with r_gate)][n2]): the router of the mixture that follows is evaluated on
+ * h, by the rule of eb_moe_route_rule (r_gate: its shared_gate). */
+EB_API int eb_stream_add(const void *src, long long lds, const void *src2, long long lds2, const void *y, long long ldy, const float *w,
+                  const void *y2, long long ldy2, const float *w2, const int32_t *idx, const int32_t *rows, const float *weights,
+                  int top, int experts, const void *ident, long long ldi, const void *shared, long long ldsh, const float *gate,
+                  float scale, float *x, long long ldx, const void *w_next, float next_scale, void *h, long long ldh, float eps,
+                  int n1, int n2, int count, const void *router, int choices, int r_experts, int r_top, const float *r_correction,
+                  int r_groups, int r_keep, int32_t *r_idx, float *r_weights, float *r_gate, int dtype, void *stream);
+
 /* Queries, keys and values of a projected row [q: heads*dk | k: kv_heads*dk | v: kv_heads*dv] made ready
  * for attention.  q and k are divided by the root mean square over ALL their rows (counts q_count and
  * k_count: heads may be zero-padded) and multiplied by q_norm / k_norm; q also by
@@ -445,6 +487,61 @@ EB_API int eb_attention_inputs(const void *proj, long long ldp, int heads, int k
                         void *q_out, long long ldq, void *k_cache, long long k_batch_stride, long long k_row_stride,
                         void *v_cache, long long v_batch_stride, long long v_row_stride, int cache_rows, int n1,
                         int rows_per_batch, const int32_t *pos_device, const int32_t *first, int dtype, void *stream);
+
+/* Queries and keys of a projected row [q: heads*dk | k: kv_heads*dk], every head by itself:
+ *   z = q_h / sqrt(mean over dk_count + eps) * q_norm  (k_norm for keys), then for i < pairs
+ *   (z_2i, z_2i+1) turned by the angle p * freq[i],     p = pos0 + s - first[b]
+ * q goes to q_out; the key to k_out (or NULL) and, with the value, which is the key as projected, to the
+ * ring caches: row b*rows_per_batch + s of n1 to row (pos0 + s) mod ring_rows of sequence b (of a longer
+ * prompt only the last ring_rows positions).  pos0 from pos_device (NULL: 0). */
+EB_API int eb_attention_rotary(const void *proj, long long ldp, int heads, int kv_heads, int dk, int dk_count, const void *q_norm,
+                        const void *k_norm, float eps, const float *freq, int pairs, void *q_out, long long ldq, void *k_out,
+                        long long ldk, void *k_cache, long long k_batch_stride, long long k_row_stride, void *v_cache,
+                        long long v_batch_stride, long long v_row_stride, int ring_rows, int n1, int rows_per_batch,
+                        const int32_t *pos_device, const int32_t *first, int dtype, void *stream);
+
+/* ---- decaying memories --------------------------------------------------------------------------- */
+
+/* Recurrent layers whose fp32 state per head is a matrix S [dk][dv] that decays.  Everything between the
+ * projections and S is fp32; head sizes are multiples of 8 (zero-padded); rows in front of first[b] are
+ * padding: they add nothing and forget nothing.
+ *
+ * State space:  dt' = softplus(dt + dt_bias[h]);  S' = exp(-exp(a_log[h]) dt') S + dt' B x^T;  y = S'^T C + skip[h] x,
+ * B and C shared by heads / groups heads.  xbc rows: [x: heads*dv | B: groups*dk | C: groups*dk].
+ * Gated linear:  S' = diag(sigmoid(z)^(1/tau)) S + k v^T;  o = S'^T (q scale).  z [row][heads*dk]. */
+
+/* Causal convolution per channel and SiLU of a prompt: out[t] = silu(b + sum_j w[j] x[t - (taps-1) + j]), w [taps]
+ * [channels], inputs in front of first[b] zero.  The last ring_rows inputs also go to the ring, position p
+ * in row p mod ring_rows. */
+EB_API int eb_short_conv(const void *x, long long ldx, const void *w, const void *b, void *out, long long ldo, int batch, int seq,
+                  int channels, int taps, const int32_t *first, void *ring, long long ring_batch_stride, long long ring_ld,
+                  int ring_rows, int dtype, void *stream);
+
+/* A whole prompt from an empty state, token by token on the CUDA cores, any sizes; xbc behind the convolution. */
+EB_API int eb_ssm_scan(const void *xbc, long long ldx, const float *dt, long long ldt, const float *dt_bias, const float *a_log,
+                const float *skip, const int32_t *first, void *y, long long ldy, float *S, int batch, int seq, int heads,
+                int groups, int dk, int dv, int dtype, void *stream);
+EB_API int eb_gla_scan(const void *q, const void *k, const void *v, long long ldp, const float *z, long long ldz, float tau,
+                float scale, const int32_t *first, void *o, long long ldo, float *S, int batch, int seq, int heads, int dk,
+                int dv, int dtype, void *stream);
+
+/* One token per sequence; xbc in front of the convolution, whose earlier inputs are read from the ring (and
+ * this one's put there). */
+EB_API int eb_ssm_step(const void *xbc, long long ldx, const void *conv_w, const void *conv_b, int taps, void *ring,
+                long long ring_batch_stride, long long ring_ld, int ring_rows, const int32_t *pos_device, const int32_t *first,
+                const float *dt, long long ldt, const float *dt_bias, const float *a_log, const float *skip, void *y,
+                long long ldy, float *S, int batch, int heads, int groups, int dk, int dv, int dtype, void *stream);
+
+/* One token per sequence: z = w2 low + b2 (w2 [heads*dk][rank]), the state goes on, and
+ * out[h] = unit(o_h) * norm * silu(g), unit(o) = o / sqrt(mean over dv_count of o^2 + eps). */
+EB_API int eb_gla_step(const void *q, const void *k, const void *v, const void *g, const void *low, long long ldp, const void *w2,
+                const void *b2, int rank, float tau, float scale, const void *norm, int dv_count, float eps, void *out,
+                long long ldo, float *S, int batch, int heads, int dk, int dv, int dtype, void *stream);
+
+/* out = unit(y * silu(z)) * norm, unit over `parts` equal parts of the heads*dv real columns (heads of dv
+ * columns padded to dv_padded; padding columns of out are not written). */
+EB_API int eb_gate_group_norm(const void *y, long long ldy, const void *z, long long ldz, const void *norm, float eps, void *out,
+                       long long ldo, int rows, int heads, int dv, int dv_padded, int parts, int dtype, void *stream);
 
 /* ---- matrix memory ------------------------------------------------------------------------------ */
 
@@ -482,6 +579,9 @@ EB_API int eb_memory_step(const void *q, const void *k, const void *v, const voi
  * (dv_count of them real). */
 EB_API int eb_head_norm_gate(const void *o, long long ldo, const void *g, long long ldg, const void *norm, float eps, void *out,
                       long long ld_out, int rows, int heads, int dv, int dv_count, int dtype, void *stream);
+/* silu != 0: the gate is g * sigmoid(g). */
+EB_API int eb_head_norm_gate_act(const void *o, long long ldo, const void *g, long long ldg, const void *norm, float eps, void *out,
+                          long long ld_out, int rows, int heads, int dv, int dv_count, int silu, int dtype, void *stream);
 
 /* ---- the tail of a greedy generation step ----------------------------------------------------- */
 
@@ -501,6 +601,14 @@ EB_API int eb_greedy_step(const void *logits, long long ld_logits, int batch, in
                    long long ld_out, int out_cols, int64_t *tok, int32_t *kv_state, const void *word_emb,
                    long long vocab_start, int vocab_rows, const void *pos_emb, int pos_rows, int add_pos, int hidden,
                    int emb_dtype, void *hidden_out, long long ld_hidden, int32_t *counter, void *stream);
+
+/* eb_greedy_step with a bigram table: pair_out[b] = pair_emb[(previous token * mul_prev + token * mul_cur) mod pair_rows],
+ * the previous token being out_ids[b][kv_state[1] - 1]. */
+EB_API int eb_greedy_step_bigram(const void *logits, long long ld_logits, int batch, int vocab, int dtype, int64_t *out_ids,
+                   long long ld_out, int out_cols, int64_t *tok, int32_t *kv_state, const void *word_emb,
+                   long long vocab_start, int vocab_rows, const void *pos_emb, int pos_rows, int add_pos, int hidden,
+                   int emb_dtype, void *hidden_out, long long ld_hidden, int32_t *counter, const void *pair_emb, long long pair_rows,
+                   long long mul_prev, long long mul_cur, void *pair_out, long long ld_pair, void *stream);
 
 /* ---- fused attention ----------------------------------------------------------------------- */
 
@@ -542,6 +650,16 @@ EB_API int eb_attention_prefill_window_tc(const void *q, const void *k, const vo
                             int heads, int q_len, int kv_len, int head_dim, int window, float scale, int dtype,
                             void *stream);
 
+/* eb_attention_prefill_tc of a sequence with itself (len queries and keys) with a chunk mask and a sink: kv_group
+ * query heads share a key / value head; row i sees the keys j <= i with floor((i - f) / chunk) =
+ * floor((j - f) / chunk), f = first[b] (chunk 0: all from f on; rows in front of f, padding, see only
+ * themselves); sinks (or NULL) [heads]: exp(sinks[h]) joins the softmax denominator. */
+EB_API int eb_attention_prefill_chunk_tc(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+                            long long q_row_stride, long long k_batch_stride, long long k_row_stride, long long v_batch_stride,
+                            long long v_row_stride, long long o_batch_stride, long long o_row_stride, int batch, int heads,
+                            int kv_group, int len, int head_dim, int chunk, const int32_t *first, const float *sinks,
+                            float scale, int dtype, void *stream);
+
 /* table[h][d] = r1[h] log2(1 + r2[h] d), d < len: the distance bias of eb_attention_prefill_biased_tc. */
 EB_API int eb_distance_bias(const float *r1, const float *r2, int heads, int len, float *table, void *stream);
 
@@ -567,6 +685,13 @@ EB_API int eb_attention_group_decode(const void *q, const void *k, const void *v
                               long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int cache_rows,
                               const int32_t *pos_device, const int32_t *first, const float *bias_r1, const float *bias_r2,
                               int sink, float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes, void *stream);
+/* With a chunk mask and a sink as eb_attention_prefill_chunk_tc, no bias.  chunk > 0: the cache is a ring,
+ * position p in row p mod ring_rows, that holds at least what of the chunk has come. */
+EB_API int eb_attention_group_decode_chunk(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
+                              long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                              long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int ring_rows, int chunk,
+                              const int32_t *pos_device, const int32_t *first, const float *sinks, float scale, int dtype,
+                              int nsplit, void *scratch, size_t scratch_bytes, void *stream);
 EB_API size_t eb_attention_group_decode_scratch_bytes(int batch, int heads, int kv_heads, int head_dim, int nsplit);
 
 /* Windowed causal attention for any head sizes and fp32 / fp16 / bf16 on the CUDA cores: query row
@@ -582,6 +707,14 @@ EB_API int eb_attention_plain(const void *q, const void *k, const void *v, void 
                        int kv_group, int q_len, int k_dim, int v_dim, int window, int ring_rows, const int32_t *pos_device,
                        const int32_t *first, const float *bias_r1, const float *bias_r2, int sink, float scale, int dtype,
                        void *stream);
+
+/* The same with a chunk mask and a sink per head (as eb_attention_prefill_chunk_tc) instead of window and bias. */
+EB_API int eb_attention_plain_chunk(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
+                       long long q_head_stride, long long k_batch_stride, long long k_row_stride, long long k_head_stride,
+                       long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
+                       long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
+                       int v_dim, int chunk, int ring_rows, const int32_t *pos_device, const int32_t *first, const float *sinks,
+                       float scale, int dtype, void *stream);
 
 /* Generation step of latent attention with absorbed projections: q [batch][heads * rank] are the
  * queries in latent space, the cached latent row of a position is key and value of every head,
