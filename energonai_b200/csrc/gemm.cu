@@ -1357,6 +1357,7 @@ namespace eb {
 int attention_tc_status(int *out4, bool clear);   // attention_tc.cu
 int latent_status(int *out4, bool clear);         // latent_attention.cu
 int memory_tc_status(int *out4, bool clear);      // matrix_memory_tc.cu
+int decay_tc_status(int *out4, bool clear);       // decay_memory_tc.cu
 }
 
 extern "C" int eb_device_status(int *out4, int clear) {
@@ -1387,6 +1388,12 @@ extern "C" int eb_device_status(int *out4, int clear) {
   if (host[0] == 0 && mem[0] != 0) {
     for (int i = 0; i < 4; ++i) host[i] = mem[i];
     host[1] += 300;
+  }
+  int dec[4] = {0, 0, 0, 0};                       // decaying memories: 400+
+  if (eb::decay_tc_status(dec, clear != 0) != EB_OK) return fail(EB_ECUDA, "device_status: cannot read the status word");
+  if (host[0] == 0 && dec[0] != 0) {
+    for (int i = 0; i < 4; ++i) host[i] = dec[i];
+    host[1] += 400;
   }
   if (out4)
     for (int i = 0; i < 4; ++i) out4[i] = host[i];

@@ -22,6 +22,17 @@ def _per_head(heads, *vectors):
         raise RuntimeError("state space: one fp32 number per head")
 
 
+KEY_HEADS = (64, 128)            # key head sizes of the chunked tensor-core kernels
+PAIRED_VALUE_HEAD = 64           # two value heads of this size share a CTA there
+
+
+def chunk_heads(dim, vdim, dtype):
+    """Padded (key, value) head sizes of the chunked kernels, or None where they do not serve."""
+    if dtype != torch.bfloat16 or dim > KEY_HEADS[-1]:
+        return None
+    return min(n for n in KEY_HEADS if n >= dim), -(-vdim // 8) * 8
+
+
 def short_conv(x, w, b, ring, batch, first=None):
     """Causal convolution per channel and SiLU of a prompt: x [batch*seq, C] (row stride allowed), w [taps, C], b [C];
     the last inputs go to ring [batch, rows, C].  Returns [batch*seq, C]."""
@@ -37,8 +48,9 @@ def short_conv(x, w, b, ring, batch, first=None):
     return out
 
 
-def ssm_prompt(xbc, dt, dt_bias, a_log, skip, S, heads, groups, dk, dv, first=None):
-    """A prompt through the state-space recurrence; xbc [batch*seq, heads*dv + 2*groups*dk] behind the convolution, dt
+def ssm_prompt(xbc, dt, dt_bias, a_log, skip, S, heads, groups, dk, dv, first=None, chunked=False):
+    """A prompt through the state-space recurrence, token by token on the CUDA cores or (chunked: bf16, dk of KEY_HEADS)
+    128 tokens at a time on the tensor cores; xbc [batch*seq, heads*dv + 2*groups*dk] behind the convolution, dt
     fp32 [batch*seq, >= heads].  S is overwritten with the state behind the last token.  Returns [batch*seq, heads*dv]."""
     require_cuda(xbc, dt, dt_bias, a_log, skip, S, first)
     B, n = _state(S, heads, dk, dv), xbc.shape[0]
@@ -46,8 +58,9 @@ def ssm_prompt(xbc, dt, dt_bias, a_log, skip, S, heads, groups, dk, dv, first=No
     if xbc.shape[1] != heads * dv + 2 * groups * dk or dt.dtype != torch.float32 or dt.shape[0] != n or dt.shape[1] < heads or n % B:
         raise RuntimeError("state space: rows [x | B | C], dt fp32, whole sequences")
     y = torch.empty((n, heads * dv), dtype=xbc.dtype, device=xbc.device)
-    check(lib().eb_ssm_scan(ptr(xbc), _rows(xbc, "xbc"), ptr(dt), _rows(dt, "dt"), ptr(dt_bias), ptr(a_log), ptr(skip), ptr(first), ptr(y), heads * dv,
-                            ptr(S), B, n // B, heads, groups, dk, dv, dtype_code(xbc.dtype), stream_ptr()), "ssm_scan")
+    run, name = (lib().eb_ssm_chunks, "ssm_chunks") if chunked else (lib().eb_ssm_scan, "ssm_scan")
+    check(run(ptr(xbc), _rows(xbc, "xbc"), ptr(dt), _rows(dt, "dt"), ptr(dt_bias), ptr(a_log), ptr(skip), ptr(first), ptr(y), heads * dv, ptr(S), B, n // B,
+              heads, groups, dk, dv, dtype_code(xbc.dtype), stream_ptr()), name)
     return y
 
 
@@ -89,15 +102,22 @@ def _qkv(q, k, v, heads, S):
     return _state(S, heads, dk, dv), dk, dv
 
 
-def gla_prompt(q, k, v, z, tau, scale, S, heads, first=None):
+def gla_prompt(q, k, v, z, tau, scale, S, heads, first=None, chunked=False):
     """A prompt through the gated linear recurrence: q, k [batch*seq, heads*dk], v [batch*seq, heads*dv] (column views of one
-    projection), z fp32 [batch*seq, heads*dk].  S is overwritten.  Returns [batch*seq, heads*dv]."""
+    projection), z fp32 [batch*seq, heads*dk]; chunked as in ssm_prompt.  S is overwritten.  Returns [batch*seq,
+    heads*dv]."""
     require_cuda(q, k, v, z, S, first)
     B, dk, dv = _qkv(q, k, v, heads, S)
     n = q.shape[0]
     if z.dtype != torch.float32 or tuple(z.shape) != (n, heads * dk) or n % B:
         raise RuntimeError("gated linear: z is fp32 [rows, heads*dk], whole sequences")
     o = torch.empty((n, heads * dv), dtype=q.dtype, device=q.device)
+    if chunked:
+        nbytes = lib().eb_gla_chunks_workspace_bytes(B, n // B, heads, dk)
+        ws = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
+        check(lib().eb_gla_chunks(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(z), _rows(z, "z"), float(tau), float(scale), ptr(first), ptr(o), heads * dv, ptr(S),
+                                  B, n // B, heads, dk, dv, dtype_code(q.dtype), ptr(ws), nbytes, stream_ptr()), "gla_chunks", launches=2)
+        return o
     check(lib().eb_gla_scan(ptr(q), ptr(k), ptr(v), q.stride(0), ptr(z), _rows(z, "z"), float(tau), float(scale), ptr(first), ptr(o), heads * dv, ptr(S),
                             B, n // B, heads, dk, dv, dtype_code(q.dtype), stream_ptr()), "gla_scan")
     return o

@@ -5,7 +5,7 @@ import torch
 from torch import nn
 
 from ..attention import attention_group_decode_chunk, attention_plain, attention_prefill_chunk, attention_rotary
-from ..decay import gla_prompt, gla_step
+from ..decay import chunk_heads, gla_prompt, gla_step
 from ..gemm import project
 from ..memory import head_norm_gate
 from ..nn import init_weight
@@ -64,7 +64,10 @@ class GatedLinearAttention(nn.Module):
         kw = dict(dtype=dtype, device=device)
         self.layer, self.eps, self.heads, self.dim, self.vdim, self.tau, self.rank = layer, eps, cfg.heads, cfg.dim, cfg.vdim, cfg.tau, cfg.rank
         self.scale = cfg.dim ** -0.5
-        self.dk, self.dv, self.low = round_up(cfg.dim, 8), round_up(cfg.vdim, 8), round_up(cfg.rank, 8)
+        padded = chunk_heads(cfg.dim, cfg.vdim, dtype)                                     # prompts on the tensor cores
+        self.chunked = padded is not None
+        self.dk, self.dv = padded if self.chunked else (round_up(cfg.dim, 8), round_up(cfg.vdim, 8))
+        self.low = round_up(cfg.rank, 8)
         qk, vg = self.heads * self.dk, self.heads * self.dv
         self.splits = [qk, qk, vg, vg, self.low]
         self.columns = sum(self.splits)
@@ -82,7 +85,7 @@ class GatedLinearAttention(nn.Module):
         if not ctx.is_prompt:
             return gla_step(q, k, v, g, low, self.a2, self.a2_bias, self.tau, self.scale, self.norm, self.vdim, self.eps, S, self.heads)
         z = project(low, self.a2, bias=self.a2_bias, out_dtype=torch.float32)
-        o = gla_prompt(q, k, v, z, self.tau, self.scale, S, self.heads, first=ctx.first)
+        o = gla_prompt(q, k, v, z, self.tau, self.scale, S, self.heads, first=ctx.first, chunked=self.chunked)
         return head_norm_gate(o, g, self.norm, self.heads, self.vdim, self.eps, silu=True)
 
 

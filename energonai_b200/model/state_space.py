@@ -7,7 +7,7 @@ recurrent one and the convolution's last inputs, a ring as long as its taps."""
 import torch
 from torch import nn
 
-from ..decay import gate_group_norm, short_conv, ssm_prompt, ssm_step
+from ..decay import PAIRED_VALUE_HEAD, chunk_heads, gate_group_norm, short_conv, ssm_prompt, ssm_step
 from ..gemm import project, project_parts
 from ..nn import init_weight
 from .sequence_state import RecurrentState, RingCache, round_up
@@ -19,7 +19,9 @@ class StateSpace(nn.Module):
         kw = dict(dtype=dtype, device=device)
         self.layer, self.eps = layer, eps
         self.heads, self.vdim, self.state, self.groups, self.norm_groups = cfg.heads, cfg.vdim, cfg.state, cfg.groups, cfg.norm_groups
-        self.dk, self.dv = round_up(cfg.state, 8), round_up(cfg.vdim, 8)
+        padded = chunk_heads(cfg.state, max(cfg.vdim, PAIRED_VALUE_HEAD), dtype)           # prompts on the tensor cores
+        self.chunked = padded is not None
+        self.dk, self.dv = padded if self.chunked else (round_up(cfg.state, 8), round_up(cfg.vdim, 8))
         self.inner = self.heads * self.dv
         self.channels = self.inner + 2 * self.groups * self.dk
         self.tail = self.inner + self.channels
@@ -43,7 +45,7 @@ class StateSpace(nn.Module):
         sizes = (self.heads, self.groups, self.dk, self.dv)
         if ctx.is_prompt:
             xbc = short_conv(xbc, self.conv_w, self.conv_b, ring, ctx.batch, first=ctx.first)
-            y = ssm_prompt(xbc, dt, self.dt_bias, self.a_log, self.skip, S, *sizes, first=ctx.first)
+            y = ssm_prompt(xbc, dt, self.dt_bias, self.a_log, self.skip, S, *sizes, first=ctx.first, chunked=self.chunked)
         else:
             y = ssm_step(xbc, self.conv_w, self.conv_b, ring, ctx.pos, dt, self.dt_bias, self.a_log, self.skip, S, *sizes, first=ctx.first)
         return project(gate_group_norm(y, z, self.norm, self.eps, self.heads, self.vdim, self.norm_groups), self.out_proj)

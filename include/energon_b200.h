@@ -525,6 +525,17 @@ EB_API int eb_gla_scan(const void *q, const void *k, const void *v, long long ld
                 float scale, const int32_t *first, void *o, long long ldo, float *S, int batch, int seq, int heads, int dk,
                 int dv, int dtype, void *stream);
 
+/* The same on the tensor cores, 128 tokens at a time: bf16, dk 64 or 128 (heads zero-padded to it), the state and all
+ * gates fp32, what enters the state as an operand split into two bf16 parts.  Waits are bounded ("where"
+ * codes 400 and up).  eb_gla_chunks: two launches, workspace of eb_gla_chunks_workspace_bytes. */
+EB_API int eb_ssm_chunks(const void *xbc, long long ldx, const float *dt, long long ldt, const float *dt_bias, const float *a_log,
+                  const float *skip, const int32_t *first, void *y, long long ldy, float *S, int batch, int seq, int heads,
+                  int groups, int dk, int dv, int dtype, void *stream);
+EB_API int eb_gla_chunks(const void *q, const void *k, const void *v, long long ldp, const float *z, long long ldz, float tau,
+                  float scale, const int32_t *first, void *o, long long ldo, float *S, int batch, int seq, int heads, int dk,
+                  int dv, int dtype, void *workspace, size_t workspace_bytes, void *stream);
+EB_API size_t eb_gla_chunks_workspace_bytes(int batch, int seq, int heads, int dk);
+
 /* One token per sequence; xbc in front of the convolution, whose earlier inputs are read from the ring (and
  * this one's put there). */
 EB_API int eb_ssm_step(const void *xbc, long long ldx, const void *conv_w, const void *conv_b, int taps, void *ring,
