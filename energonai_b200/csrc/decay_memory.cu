@@ -46,7 +46,7 @@ template <typename T> __device__ __forceinline__ void store_pack(T *p, const flo
 }
 
 // ---- convolution of a prompt ---------------------------------------------------------------------------
-constexpr int kConvThreads = 128, kConvStrip = 16;
+constexpr int kConvThreads = 128, kConvStrip = 32;
 
 struct ConvParams {
   const void *x;
@@ -61,70 +61,90 @@ struct ConvParams {
   int ring_rows;
 };
 
-// Thread = 8 channels of kConvStrip tokens; TAPS > 0: the window in registers, else read again per token.
+// silu of what becomes a 16-bit operand, and of 32-bit models
+template <typename T> __device__ __forceinline__ float conv_silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+template <> __device__ __forceinline__ float conv_silu<float>(float x) { return silu(x); }
+
+// Four channels as 32-bit numbers
+template <typename T> __device__ __forceinline__ void load4(const T *p, float (&f)[4]) {
+  const uint2 w = *reinterpret_cast<const uint2 *>(p);
+  const float2 a = unpack2<T>(w.x), b = unpack2<T>(w.y);
+  f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+}
+template <> __device__ __forceinline__ void load4<float>(const float *p, float (&f)[4]) {
+  const float4 a = *reinterpret_cast<const float4 *>(p);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+}
+template <typename T> __device__ __forceinline__ void store4(T *p, const float (&f)[4]) {
+  *reinterpret_cast<uint2 *>(p) = make_uint2(pack2<T>(f[0], f[1]), pack2<T>(f[2], f[3]));
+}
+template <> __device__ __forceinline__ void store4<float>(float *p, const float (&f)[4]) { *reinterpret_cast<float4 *>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+
+// Thread = 4 channels of kConvStrip tokens; TAPS > 0: the window in registers, else read again per token.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(kConvThreads) short_conv_kernel(const ConvParams p) {
   griddep_wait();
   griddep_launch();
-  const int c = (blockIdx.x * kConvThreads + threadIdx.x) * 8, b = blockIdx.z, t0 = blockIdx.y * kConvStrip;
+  const int c = (blockIdx.x * kConvThreads + threadIdx.x) * 4, b = blockIdx.z, t0 = blockIdx.y * kConvStrip;
   if (c >= p.C) return;
   const int first = p.first ? p.first[b] : 0, taps = TAPS > 0 ? TAPS : p.taps;
   const T *x = reinterpret_cast<const T *>(p.x) + (long long)b * p.seq * p.ldx + c;
   T *out = reinterpret_cast<T *>(p.out) + (long long)b * p.seq * p.ldo + c;
   T *ring = reinterpret_cast<T *>(p.ring) + b * p.ring_bs + c;
   const T *w = reinterpret_cast<const T *>(p.w) + c;
-  auto input = [&](int t, float (&f)[8]) {
+  auto input = [&](int t, float (&f)[4]) {
     if (t >= first && t < p.seq) {
-      load_pack<T>(x + (long long)t * p.ldx, f);
+      load4<T>(x + (long long)t * p.ldx, f);
     } else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) f[e] = 0.f;
+      for (int e = 0; e < 4; ++e) f[e] = 0.f;
     }
   };
-  float bias[8];
-  load_pack<T>(reinterpret_cast<const T *>(p.b) + c, bias);
-  auto finish = [&](int t, const float (&cur)[8], float (&acc)[8]) {
+  float bias[4];
+  load4<T>(reinterpret_cast<const T *>(p.b) + c, bias);
+  auto finish = [&](int t, const float (&cur)[4], float (&acc)[4]) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = silu(acc[e]);
-    store_pack<T>(out + (long long)t * p.ldo, acc);
-    if (p.seq - t <= p.ring_rows) store_pack<T>(ring + (long long)(t % p.ring_rows) * p.ring_ld, cur);
+    for (int e = 0; e < 4; ++e) acc[e] = conv_silu<T>(acc[e]);
+    store4<T>(out + (long long)t * p.ldo, acc);
+    if (p.seq - t <= p.ring_rows) store4<T>(ring + (long long)(t % p.ring_rows) * p.ring_ld, cur);
   };
   if constexpr (TAPS > 0) {
-    float wv[TAPS][8], win[TAPS][8];                 // win[j]: the input j tokens before the last TAPS - 1
+    constexpr int kGroup = 8;                        // tokens whose inputs are in flight together
+    float wv[TAPS][4], in[TAPS - 1 + kGroup][4];     // in[TAPS - 1 + i]: token i of the group
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) load_pack<T>(w + (long long)j * p.C, wv[j]);
+    for (int j = 0; j < TAPS; ++j) load4<T>(w + (long long)j * p.C, wv[j]);
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) input(t0 - (TAPS - 1) + j, win[j + 1]);
+    for (int j = 0; j < TAPS - 1; ++j) input(t0 - (TAPS - 1) + j, in[j]);
+#pragma unroll 1
+    for (int i0 = 0; i0 < kConvStrip; i0 += kGroup) {
 #pragma unroll
-    for (int i0 = 0; i0 < kConvStrip; i0 += 4) {
-      float next[4][8];
+      for (int i = 0; i < kGroup; ++i) input(t0 + i0 + i, in[TAPS - 1 + i]);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) input(t0 + i0 + i, next[i]);
+      for (int i = 0; i < kGroup; ++i) {
+        float acc[4];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        float acc[8];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-#pragma unroll
-          for (int j = 0; j < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
-          win[TAPS - 1][e] = next[i][e];
+        for (int e = 0; e < 4; ++e) {
           acc[e] = bias[e];
 #pragma unroll
-          for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(wv[j][e], win[j][e], acc[e]);
+          for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(wv[j][e], in[i + j][e], acc[e]);
         }
-        if (t0 + i0 + i < p.seq) finish(t0 + i0 + i, win[TAPS - 1], acc);
+        if (t0 + i0 + i < p.seq) finish(t0 + i0 + i, in[TAPS - 1 + i], acc);
       }
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) in[j][e] = in[kGroup + j][e];
     }
   } else {
     for (int t = t0; t < min(p.seq, t0 + kConvStrip); ++t) {
-      float acc[8], f[8], wv[8];
+      float acc[4], f[4], wv[4];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = bias[e];
+      for (int e = 0; e < 4; ++e) acc[e] = bias[e];
       for (int j = 0; j < taps; ++j) {
         input(t - (taps - 1) + j, f);
-        load_pack<T>(w + (long long)j * p.C, wv);
+        load4<T>(w + (long long)j * p.C, wv);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = fmaf(wv[e], f[e], acc[e]);
+        for (int e = 0; e < 4; ++e) acc[e] = fmaf(wv[e], f[e], acc[e]);
       }
       finish(t, f, acc);
     }
@@ -132,7 +152,7 @@ __global__ void __launch_bounds__(kConvThreads) short_conv_kernel(const ConvPara
 }
 
 template <typename T> int launch_conv(const ConvParams &p, int B, cudaStream_t st) {
-  const dim3 g((p.C / 8 + kConvThreads - 1) / kConvThreads, (p.seq + kConvStrip - 1) / kConvStrip, B), b(kConvThreads);
+  const dim3 g((p.C / 4 + kConvThreads - 1) / kConvThreads, (p.seq + kConvStrip - 1) / kConvStrip, B), b(kConvThreads);
   switch (p.taps) {
     case 2: launch_pdl(short_conv_kernel<T, 2>, g, b, 0, st, p); break;
     case 3: launch_pdl(short_conv_kernel<T, 3>, g, b, 0, st, p); break;
@@ -268,7 +288,7 @@ __global__ void __launch_bounds__(kStepThreads, 4) ssm_step_kernel(const SsmStep
     // (the row of this position is none of the rows that are read)
     if (keep) ring[(long long)(pos % p.ring_rows) * p.ring_ld + ch] = cur;
     // what the projection and the convolution give is an operand: rounded as a prompt's is
-    return to_f32<T>(from_f32<T>(silu(acc)));
+    return to_f32<T>(from_f32<T>(conv_silu<T>(acc)));
   };
   const bool lead = blockIdx.x == 0 && h % (p.heads / p.groups) == 0;
   const int b0 = p.heads * p.dv + g * p.dk, c1 = b0 + p.groups * p.dk;

@@ -578,32 +578,39 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_prepare_kernel(const Prep
   const long long row0 = (long long)b * p.seq + t0;
   const T *q = reinterpret_cast<const T *>(p.q) + row0 * p.ldp + h * DK, *k = reinterpret_cast<const T *>(p.k) + row0 * p.ldp + h * DK;
 
-  // keys (zero for padding and behind the end), log decays and their running sums
-  for (int i = tid; i < kChunk * kPacks; i += kPrepThreads) {
-    const int r = i / kPacks, x = (i % kPacks) * 8;
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (r >= first && r < n) v = *reinterpret_cast<const uint4 *>(k + (long long)r * p.ldp + x);
-    *reinterpret_cast<uint4 *>(ks + r * kLd + x) = v;
+  // keys (zero for padding and behind the end) on their way to shared memory, queries to registers
+  constexpr int kIters = kChunk * kPacks / kPrepThreads, kRowStep = kPrepThreads / kPacks;
+  const int r_of = tid / kPacks, x_of = (tid % kPacks) * 8;
+  uint4 qv[kIters];
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int r = r_of + i * kRowStep;
+    const bool ok = r >= first && r < n;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(s32(ks + r * kLd + x_of)), "l"(ok ? k + (long long)r * p.ldp + x_of : k), "r"(ok ? 16 : 0) : "memory");
   }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) qv[i] = *reinterpret_cast<const uint4 *>(q + (long long)min(r_of + i * kRowStep, n - 1) * p.ldp + x_of);
+  // log decays and their running sums
   {
+    constexpr int kBatch = 32;
     const int d = tid % DK, part = tid / DK;
     const float *z = p.z + row0 * p.ldz + h * DK + d;
     float run = 0.f;
 #pragma unroll 1
-    for (int i0 = 0; i0 < kTokens; i0 += 8) {
-      float zz[8];
+    for (int i0 = 0; i0 < kTokens; i0 += kBatch) {
+      float zz[kBatch];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        const int r = part * kTokens + i0 + i;
-        zz[i] = r < n ? z[(long long)r * p.ldz] : 0.f;
-      }
+      for (int i = 0; i < kBatch; ++i) zz[i] = z[(long long)min(part * kTokens + i0 + i, n - 1) * p.ldz];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < kBatch; ++i) {
         const int r = part * kTokens + i0 + i;
-        if (r >= first && r < n) run += log_decay_gla(zz[i], p.inv_tau) * kLog2eDecay;
+        const float l = log_decay_gla(zz[i], p.inv_tau) * kLog2eDecay;
+        run += r >= first && r < n ? l : 0.f;
         Lm[r * kLd + d] = run;
       }
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     ends[tid] = run;
     __syncthreads();
     float before = 0.f;
@@ -617,10 +624,12 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_prepare_kernel(const Prep
   // Q exp(L_t) and K exp(L_end - L_s)
   T *qt = reinterpret_cast<T *>(p.qt) + row0 * p.heads * DK + h * DK, *khi = reinterpret_cast<T *>(p.khi) + row0 * p.heads * DK + h * DK,
     *klo = reinterpret_cast<T *>(p.klo) + row0 * p.heads * DK + h * DK;
-  for (int i = tid; i < n * kPacks; i += kPrepThreads) {
-    const int r = i / kPacks, x = (i % kPacks) * 8;
-    const uint4 qv = *reinterpret_cast<const uint4 *>(q + (long long)r * p.ldp + x), kv = *reinterpret_cast<const uint4 *>(ks + r * kLd + x);
-    const uint32_t qw[4] = {qv.x, qv.y, qv.z, qv.w}, kw[4] = {kv.x, kv.y, kv.z, kv.w};
+#pragma unroll
+  for (int i = 0; i < kIters; ++i) {
+    const int r = r_of + i * kRowStep, x = x_of;
+    if (r >= n) break;
+    const uint4 kv = *reinterpret_cast<const uint4 *>(ks + r * kLd + x);
+    const uint32_t qw[4] = {qv[i].x, qv[i].y, qv[i].z, qv[i].w}, kw[4] = {kv.x, kv.y, kv.z, kv.w};
     uint32_t a[4], hi[4], lo[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
@@ -635,67 +644,78 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gla_prepare_kernel(const Prep
     *reinterpret_cast<uint4 *>(klo + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   }
 
-  // P: warp = block of 16 rows; lane (g, t): rows g and g + 8, columns 2 t and 2 t + 1 of every 8 keys
-  const int g = lane >> 2, t = lane & 3, m0 = warp * 16;
+  // P: blocks of 16 rows against tiles of 8 keys; lane (g, t): rows g and g + 8, columns 2 t and 2 t + 1 of a tile.  Block
+  // w has 2 w + 2 tiles; the warps of blocks w and 7 - w share theirs, 9 each.
+  const int g = lane >> 2, t = lane & 3, low = min(warp, 7 - warp);
   T *pm = reinterpret_cast<T *>(p.pm) + row0 * p.heads * kChunk + h * kChunk;
-  if (m0 < n) {
+  auto block = [&](int w, int tile0, int tile1) {
+    const int m0 = w * 16;
+    if (m0 >= n) return;
+    const float *base = Lm + (m0 - 1) * kLd;                     // L in front of the block (0 for the first)
+    auto before = [&](int x) { return m0 > 0 ? *reinterpret_cast<const float2 *>(base + x) : make_float2(0.f, 0.f); };
     float spread = 0.f;
-    for (int d = lane; d < DK; d += 32) spread = fmaxf(spread, (m0 > 0 ? Lm[(m0 - 1) * kLd + d] : 0.f) - Lm[(m0 + 15) * kLd + d]);
+    for (int d = lane; d < DK; d += 32) spread = fmaxf(spread, (m0 > 0 ? base[d] : 0.f) - Lm[(m0 + 15) * kLd + d]);
     const bool direct = warp_max(spread) > kSafeLog2;
-    const int tiles = direct ? 2 * warp : 2 * warp + 2;          // tiles of 8 keys that go through the tensor cores
-    float acc[kChunk / 8][4];
+    uint32_t a[DK / 16][4], a_lo[DK / 16][4];
 #pragma unroll
-    for (int i = 0; i < kChunk / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-#pragma unroll 1
-    for (int kk = 0; kk < DK; kk += 16) {
-      const int x0 = kk + 2 * t, x1 = x0 + 8;
-      float2 b0 = make_float2(0.f, 0.f), b1 = b0;                // L in front of the block
-      if (m0 > 0) {
-        b0 = *reinterpret_cast<const float2 *>(Lm + (m0 - 1) * kLd + x0);
-        b1 = *reinterpret_cast<const float2 *>(Lm + (m0 - 1) * kLd + x1);
-      }
-      uint32_t a[4], a_lo[4];
+    for (int kk = 0; kk < DK / 16; ++kk)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int r = m0 + g + 8 * (i & 1), x = i < 2 ? x0 : x1;
-        const float2 bb = i < 2 ? b0 : b1, l = *reinterpret_cast<const float2 *>(Lm + r * kLd + x);
+        const int r = m0 + g + 8 * (i & 1), x = kk * 16 + 2 * t + (i < 2 ? 0 : 8);
+        const float2 bb = before(x), l = *reinterpret_cast<const float2 *>(Lm + r * kLd + x);
         const float2 f = r < n ? unpack2<T>(*reinterpret_cast<const uint32_t *>(q + (long long)r * p.ldp + x)) : make_float2(0.f, 0.f);
-        split2(f.x * p.scale * ex2(l.x - bb.x), f.y * p.scale * ex2(l.y - bb.y), a[i], a_lo[i]);
+        split2(f.x * p.scale * ex2(l.x - bb.x), f.y * p.scale * ex2(l.y - bb.y), a[kk][i], a_lo[kk][i]);
       }
+#pragma unroll 1
+    for (int i = tile0; i < tile1; ++i) {
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      if (direct && i >= 2 * w) {
+#pragma unroll 1
+        for (int e = 0; e < 4; ++e) {
+          const int r = m0 + g + 8 * (e >> 1), s = i * 8 + 2 * t + (e & 1);
+          float sum = 0.f;
+          if (s <= r && r < n)
+            for (int d = 0; d < DK; ++d)
+              sum = fmaf(to_f32<T>(q[(long long)r * p.ldp + d]) * p.scale * ex2(Lm[r * kLd + d] - Lm[s * kLd + d]), to_f32<T>(ks[s * kLd + d]), sum);
+          if (e == 0) acc[0] = sum;
+          else if (e == 1) acc[1] = sum;
+          else if (e == 2) acc[2] = sum;
+          else acc[3] = sum;
+        }
+      } else {
+        const int s = i * 8 + g;
 #pragma unroll
-      for (int i = 0; i < kChunk / 8; ++i) {
-        if (i < tiles) {
-          const int s = i * 8 + g;
+        for (int kk = 0; kk < DK / 16; ++kk) {
+          const int x0 = kk * 16 + 2 * t, x1 = x0 + 8;
+          const float2 b0 = before(x0), b1 = before(x1);
           const float2 l0 = *reinterpret_cast<const float2 *>(Lm + s * kLd + x0), l1 = *reinterpret_cast<const float2 *>(Lm + s * kLd + x1);
           const float2 f0 = unpack2<T>(*reinterpret_cast<const uint32_t *>(ks + s * kLd + x0)), f1 = unpack2<T>(*reinterpret_cast<const uint32_t *>(ks + s * kLd + x1));
           uint32_t k0, k0_lo, k1, k1_lo;
           split2(f0.x * ex2(b0.x - l0.x), f0.y * ex2(b0.y - l0.y), k0, k0_lo);
           split2(f1.x * ex2(b1.x - l1.x), f1.y * ex2(b1.y - l1.y), k1, k1_lo);
-          mma_bf16(acc[i], a, k0, k1);
-          mma_bf16(acc[i], a_lo, k0, k1);
-          mma_bf16(acc[i], a, k0_lo, k1_lo);
+          mma_bf16(acc, a[kk], k0, k1);
+          mma_bf16(acc, a_lo[kk], k0, k1);
+          mma_bf16(acc, a[kk], k0_lo, k1_lo);
         }
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < kChunk / 8; ++i) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = m0 + g + 8 * (e >> 1), s = i * 8 + 2 * t + (e & 1);
-        if (direct && i >= 2 * warp && i < 2 * warp + 2 && s <= r && r < n) {
-          float sum = 0.f;
-          for (int d = 0; d < DK; ++d)
-            sum = fmaf(to_f32<T>(q[(long long)r * p.ldp + d]) * p.scale * ex2(Lm[r * kLd + d] - Lm[s * kLd + d]), to_f32<T>(ks[s * kLd + d]), sum);
-          acc[i][e] = sum;
-        }
-        if (s > r) acc[i][e] = 0.f;
       }
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int r = m0 + g + 8 * e;
-        if (r < n) *reinterpret_cast<uint32_t *>(pm + (long long)r * p.heads * kChunk + i * 8 + 2 * t) = pack2<T>(acc[i][2 * e], acc[i][2 * e + 1]);
+        const int r = m0 + g + 8 * e, s = i * 8 + 2 * t;
+        if (r < n)
+          *reinterpret_cast<uint32_t *>(pm + (long long)r * p.heads * kChunk + s) = pack2<T>(s <= r ? acc[2 * e] : 0.f, s + 1 <= r ? acc[2 * e + 1] : 0.f);
       }
     }
+  };
+  // keys behind a block are hidden from it
+  for (int i = tid; i < n * (kChunk / 8); i += kPrepThreads) {
+    const int r = i / (kChunk / 8), s = i % (kChunk / 8);
+    if (s >= 2 * (r / 16) + 2) *reinterpret_cast<uint4 *>(pm + (long long)r * p.heads * kChunk + s * 8) = make_uint4(0, 0, 0, 0);
+  }
+  // (tile 7 - 2 low on of the larger block is its own warp's)
+#pragma unroll 1
+  for (int turn = 0; turn < 2; ++turn) {
+    if (warp < 4) block(turn == 0 ? low : 7 - low, 0, turn == 0 ? 2 * low + 2 : 7 - 2 * low);
+    else if (turn == 0) block(warp, 7 - 2 * low, 2 * warp + 2);
   }
 }
 

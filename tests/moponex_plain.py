@@ -218,3 +218,130 @@ def greedy(cfg, tensors, tokens, new):
         gap = min(gap, float(top.values[0] - top.values[1]))
         tokens.append(int(top.indices[0]))
     return tokens, gap
+
+
+# ---- small models of the tests' own ------------------------------------------------------------------
+def dense_mlp(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe_mlp(experts, top, ff, identity=0, groups=None, shared=None):
+    r = {"experts": experts, "top": top}
+    if identity:
+        r["identity"] = identity
+    if groups:
+        r["groups"] = {"count": groups[0], "keep": groups[1]}
+    out = {"kind": "moe", "router": r, "expert": {"ff": ff}}
+    if shared:
+        out["shared"] = {"ff": shared}
+    return out
+
+
+def ssm_layer(heads, vdim, state, groups=1, conv=4, norm_groups=1, mlp=None):
+    return {"type": "mamba2", "mlp": mlp,
+            "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups}}
+
+
+def parallel_layer(left, right, mlp=None):
+    """left = (heads, kv_heads, dim, scale, chunk, (rotated dims, base, factor or None) or None), right = (heads, dim, vdim,
+    tau, rank)."""
+    H, G, d, scale, chunk, rot = left
+    a = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": scale}
+    if chunk:
+        a["mask"] = {"size": chunk}
+    if rot:
+        a["rot"] = {"dims": rot[0], "base": rot[1]}
+        if rot[2]:
+            a["rot"]["scaling"] = {"factor": rot[2]}
+    return {"type": "parallel", "mlp": mlp, "rank": right[4],
+            "mixer": {"left": a, "right": {"heads": right[0], "dim": right[1], "vdim": right[2], "tau": right[3]}}}
+
+
+def make_config(layers, width, vocab, eps=2e-5, mult=0.6, logit_scale=0.3, bigram=(97, 31, 7)):
+    """The ranks of the decay projections are not part of a configuration: make_tensors() takes them from `layers`,
+    and `ranks` keeps them (see with_ranks)."""
+    emb = {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))} if bigram else {}
+    return {"architecture": "Moponex", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": mult, "logit_scale": logit_scale,
+            "embedding": emb, "layers": [{k: v for k, v in ly.items() if k != "rank"} for ly in layers], "ranks": [ly.get("rank") for ly in layers]}
+
+
+def file_config(cfg):
+    """What config.json holds."""
+    return {k: v for k, v in cfg.items() if k != "ranks"}
+
+
+def with_ranks(cfg):
+    """For models built without a checkpoint: the ranks stand in the configuration."""
+    out = file_config(cfg)
+    out["layers"] = [dict(ly, mixer=dict(ly["mixer"], right=dict(ly["mixer"]["right"], rank=r))) if r else ly for ly, r in zip(cfg["layers"], cfg["ranks"])]
+    return out
+
+
+def make_tensors(cfg, seed):
+    """Random bfloat16 tensors of a configuration.  Projections keep the scale of their input; decays are mostly slow,
+    so that far tokens still count; sinks are about as large as scores; corrections decide choices; norm
+    weights move away from one."""
+    g = torch.Generator().manual_seed(seed)
+    W, t = cfg["width"], {}
+
+    def mat(name, rows, cols, gain=1.0):
+        t[name] = (torch.randn(rows, cols, generator=g) * gain / cols ** 0.5).bfloat16()
+
+    def vec(name, n, mean, spread=0.3):
+        t[name] = (mean + spread * torch.randn(n, generator=g)).bfloat16()
+    mat("embed", cfg["vocab"], W, W ** 0.5 * 0.7)
+    if cfg["embedding"].get("bigram"):
+        mat("bigram", cfg["embedding"]["bigram"]["buckets"] + 1, W, W ** 0.5 * 0.5)
+    vec("final.norm", W, 1.0)
+    for i, (ly, rank) in enumerate(zip(cfg["layers"], cfg["ranks"])):
+        p, m, f = f"l{i}.", ly["mixer"], ly["mlp"]
+        vec(p + "norm1", W, 1.0)
+        if ly["type"] == "mamba2":
+            H, P, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+            channels = H * P + 2 * G * N
+            mat(p + "mix.in", H * P + channels + H, W, 1.2)
+            mat(p + "mix.conv", channels, m["conv"], 1.3)
+            vec(p + "mix.conv.b", channels, 0.0)
+            vec(p + "mix.dt_bias", H, -2.0, 0.7)
+            vec(p + "mix.A_log", H, -2.0, 1.2)
+            vec(p + "mix.D", H, 0.7)
+            vec(p + "mix.norm", H * P, 1.0)
+            mat(p + "mix.o", W, H * P, 1.5)
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d = a["heads"], a["kv_heads"], a["dim"]
+            for name, n in (("q", H), ("k", G)):
+                mat(p + "mix.left." + name, n * d, W)
+                vec(p + f"mix.left.{name}.b", n * d, 0.0)
+                vec(p + f"mix.left.{name}.norm", d, 1.4)
+            vec(p + "mix.left.sink", H, 2.0, 1.5)
+            mat(p + "mix.left.o", W, H * d)
+            H, d, dv = r["heads"], r["dim"], r["vdim"]
+            for name, n in (("q", d), ("k", d), ("v", dv), ("g", dv)):
+                mat(p + "mix.right." + name, H * n, W, 1.2)
+            mat(p + "mix.right.a1", rank, W)
+            mat(p + "mix.right.a2", H * d, rank)
+            vec(p + "mix.right.a2.b", H * d, 1.5, 1.5)
+            vec(p + "mix.right.norm", dv, 1.0)
+            mat(p + "mix.right.o", W, H * dv)
+            vec(p + "mix.left.out", W, 1.0)
+            vec(p + "mix.right.out", W, 0.8)
+        if f is None:
+            continue
+        vec(p + "norm2", W, 1.0)
+        if f["kind"] == "dense":
+            for name, rows, cols in (("gate", f["ff"], W), ("up", f["ff"], W), ("down", W, f["ff"])):
+                mat(p + "mlp." + name, rows, cols, 1.3)
+            continue
+        r = f["router"]
+        n = r["experts"] + r.get("identity", 0)
+        mat(p + "mlp.router", n, W, 2.0)
+        vec(p + "mlp.correction", n, -1.0, 0.15)
+        for e in range(r["experts"]):
+            mat(f"{p}mlp.e{e}.up", f["expert"]["ff"], W, 1.3)
+            mat(f"{p}mlp.e{e}.down", W, f["expert"]["ff"], 1.3)
+        if f.get("shared"):
+            mat(p + "mlp.shared.up", f["shared"]["ff"], W, 1.3)
+            mat(p + "mlp.shared.down", W, f["shared"]["ff"], 1.3)
+            mat(p + "mlp.shared.sg", 1, W)
+    return t
