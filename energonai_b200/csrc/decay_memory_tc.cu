@@ -61,7 +61,9 @@ struct ChunkParams {
 struct SsmGates {
   float g2[kChunk];            // L_t
   float u2[kChunk];            // log2(dt_s) - L_s
+  float wk[kChunk];            // exp(L at the end of its block of 32 tokens - L_s) dt_s
   float w[kChunk];             // exp(L_end - L_s) dt_s
+  float end[kChunk / 32];      // L at the end of each block
   float decay, pad[3];         // exp(L_end)
 };
 
@@ -155,10 +157,11 @@ decay_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
       for (int c = 0; c < nc; ++c) {
         const int before = (c - 1) & 1;
         if (c > 0 && !bar_wait(k_empty, before, abort_flag, 1)) break;
-        bar_expect_tx(k_full, SSM ? L::kOp : 2 * L::kOp);
+        bar_expect_tx(k_full, SSM ? L::kOp + L::kWide : 2 * L::kOp);
         tile(k_addr, &tm_k, k_full, hk * DK, kSub, c);
         if (!SSM) tile(k2_addr, &tm_k2, k_full, hk * DK, kSub, c);
         if (SSM) {
+          tile(vhi_addr, &tm_v, k_full, col0, 2, c);           // (the values that are weighted in place)
           if (c > 0 && !bar_wait(q_empty, before, abort_flag, 2)) break;
           bar_expect_tx(q_full, L::kOp);
           tile(q_addr, &tm_q, q_full, hk * DK, kSub, c);
@@ -281,10 +284,12 @@ decay_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
           end = __shfl_sync(0xffffffffu, x, 31);
           g.g2[i + lane] = x;
           g.u2[i + lane] = log2f(dt) - x;
-          g.w[i + lane] = dt;
+          g.wk[i + lane] = dt * ex2(end - x);
+          if (lane == 0) g.end[i / 32] = end;
         }
+        __syncwarp();
 #pragma unroll 1
-        for (int i = lane; i < kChunk; i += 32) g.w[i] *= ex2(end - g.g2[i]);                  // (this lane's own entries)
+        for (int i = lane; i < kChunk; i += 32) g.w[i] = g.wk[i] * ex2(end - g.end[i / 32]);
         if (lane == 0) g.decay = ex2(end);
         __syncwarp();
         if (lane == 0) bar_arrive(g_full + 8 * slot);
@@ -317,15 +322,25 @@ decay_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
           } else {
             float x[32];
             tc_ld32(t_lane + kColA + cc * 32, x);
+            if (cc < quarter) {                        // the row's part of the decay times the key's
+              const float from_end = ex2(g2 - g.end[cc]);
 #pragma unroll
-            for (int e = 0; e < 32; e += 4) {
-              float4 u = *reinterpret_cast<const float4 *>(g.u2 + cc * 32 + e);
-              add2(u.x, u.y, u.x, u.y, g2, g2);
-              add2(u.z, u.w, u.z, u.w, g2, g2);
-              mul2(x[e], x[e + 1], x[e], x[e + 1], ex2(u.x), ex2(u.y));
-              mul2(x[e + 2], x[e + 3], x[e + 2], x[e + 3], ex2(u.z), ex2(u.w));
-            }
-            if (cc == quarter) {
+              for (int e = 0; e < 32; e += 4) {
+                float4 u = *reinterpret_cast<const float4 *>(g.wk + cc * 32 + e);
+                mul2(u.x, u.y, u.x, u.y, from_end, from_end);
+                mul2(u.z, u.w, u.z, u.w, from_end, from_end);
+                mul2(x[e], x[e + 1], x[e], x[e + 1], u.x, u.y);
+                mul2(x[e + 2], x[e + 3], x[e + 2], x[e + 3], u.z, u.w);
+              }
+            } else {
+#pragma unroll
+              for (int e = 0; e < 32; e += 4) {
+                float4 u = *reinterpret_cast<const float4 *>(g.u2 + cc * 32 + e);
+                add2(u.x, u.y, u.x, u.y, g2, g2);
+                add2(u.z, u.w, u.z, u.w, g2, g2);
+                mul2(x[e], x[e + 1], x[e], x[e + 1], ex2(u.x), ex2(u.y));
+                mul2(x[e + 2], x[e + 3], x[e + 2], x[e + 3], ex2(u.z), ex2(u.w));
+              }
 #pragma unroll
               for (int e = 0; e < 32; ++e) x[e] = e < lane ? x[e] : (e == lane ? x[e] + skip : 0.f);
             }
@@ -440,32 +455,39 @@ decay_chunk_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_consta
         }
       }
       if constexpr (SSM) {
-        if (!wait(v_full, ph, 24)) { alive = false; break; }
-        const uint8_t *v_ptr = smem + L::kV;
+        if (!wait(k_full, ph, 24)) { alive = false; break; }
         uint8_t *hi_ptr = smem + L::kV2, *lo_ptr = smem + L::kV3;
-        // thread = 8 columns of every 8th row
+        // thread = 8 columns of every 8th row, in place; the rows of a batch are read before any of them is written
         const int piece = tid & 15, r0 = tid >> 4;
         const float *w = gates[slot * 2 + (two ? piece >> 3 : 0)].w;
         const uint32_t off = (uint32_t)(piece >> 3) * kAtom;
-#pragma unroll 4
-        for (int i = 0; i < kChunk / 8; ++i) {
-          const int r = r0 + 8 * i;
-          const uint32_t at = off + r * 128 + (((piece & 7) ^ (r & 7)) << 4);
-          const uint4 v = *reinterpret_cast<const uint4 *>(v_ptr + at);
-          const uint32_t vv[4] = {v.x, v.y, v.z, v.w};
-          const float ws = w[r];
-          uint32_t hi[4], lo[4];
+#pragma unroll 1
+        for (int i0 = 0; i0 < kChunk / 8; i0 += 8) {
+          uint4 v[8];
+          float ws[8];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            float2 f = unpack2<T>(vv[e]);
-            mul2(f.x, f.y, f.x, f.y, ws, ws);
-            hi[e] = pack2<T>(f.x, f.y);
-            const float2 x = unpack2<T>(hi[e]);
-            add2(f.x, f.y, f.x, f.y, -x.x, -x.y);
-            lo[e] = pack2<T>(f.x, f.y);
+          for (int i = 0; i < 8; ++i) {
+            const int r = r0 + 8 * (i0 + i);
+            v[i] = *reinterpret_cast<const uint4 *>(hi_ptr + off + r * 128 + (((piece & 7) ^ (r & 7)) << 4));
+            ws[i] = w[r];
           }
-          *reinterpret_cast<uint4 *>(hi_ptr + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4 *>(lo_ptr + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const int r = r0 + 8 * (i0 + i);
+            const uint32_t at = off + r * 128 + (((piece & 7) ^ (r & 7)) << 4), vv[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              float2 f = unpack2<T>(vv[e]);
+              mul2(f.x, f.y, f.x, f.y, ws[i], ws[i]);
+              hi[e] = pack2<T>(f.x, f.y);
+              const float2 x = unpack2<T>(hi[e]);
+              add2(f.x, f.y, f.x, f.y, -x.x, -x.y);
+              lo[e] = pack2<T>(f.x, f.y);
+            }
+            *reinterpret_cast<uint4 *>(hi_ptr + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            *reinterpret_cast<uint4 *>(lo_ptr + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          }
         }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
         __syncwarp();

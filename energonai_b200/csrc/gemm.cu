@@ -315,7 +315,7 @@ __device__ __forceinline__ int group_row(const GemmParams &p, int lane_tile) { r
 __device__ __forceinline__ float apply_act(float v, int act) {
   if (act == EB_ACT_RELU) return fmaxf(v, 0.f);
   if (act == EB_ACT_GELU_TANH) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * v * (1.f + 0.044715f * v * v)));
-  if (act == EB_ACT_GELU_ERF) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
+  if (act == EB_ACT_GELU_ERF) return gelu_erf_fast(v);
   return v;
 }
 
@@ -730,6 +730,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
                     } else if (act == EB_ACT_XIELU) {
 #pragma unroll
                       for (int j = 0; j < 8; ++j) vv[j] = xielu_fast(vv[j], act0, act1);
+                    } else if (act == EB_ACT_GELU_ERF) {
+#pragma unroll
+                      for (int j = 0; j < 8; ++j) vv[j] = gelu_erf_fast(vv[j]);
                     } else if (act != EB_ACT_NONE) {
 #pragma unroll
                       for (int j = 0; j < 8; ++j) vv[j] = apply_act(vv[j], act);
@@ -1020,6 +1023,9 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
             } else if (act == EB_ACT_XIELU) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) y[j] = xielu_fast(y[j], act0, act1);
+            } else if (act == EB_ACT_GELU_ERF) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) y[j] = gelu_erf_fast(y[j]);
             } else if (act != EB_ACT_NONE) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) y[j] = apply_act(y[j], act);

@@ -242,8 +242,8 @@ __device__ __forceinline__ void skinny_tile(const SkinnyParams &p, int group, in
       if (p.unit == EB_UNIT_CLAMPED || p.unit == EB_UNIT_GEGLU) {
         if (row0 + g + 8 < p.N) c[row0 / 2 + g] = from_f32<T>(unit_value(p.unit, acc[j][e], acc[j][2 + e], p.limit, p.alpha));
       } else if (p.unit == EB_UNIT_GELU) {
-        if (row0 + g < p.N) c[row0 + g] = from_f32<T>(gelu_erf_value(acc[j][e]));
-        if (row0 + g + 8 < p.N) c[row0 + g + 8] = from_f32<T>(gelu_erf_value(acc[j][2 + e]));
+        if (row0 + g < p.N) c[row0 + g] = from_f32<T>(gelu_erf_fast(acc[j][e]));
+        if (row0 + g + 8 < p.N) c[row0 + g + 8] = from_f32<T>(gelu_erf_fast(acc[j][2 + e]));
       } else {
         if (row0 + g < p.N) c[row0 + g] = from_f32<T>(acc[j][e]);
         if (row0 + g + 8 < p.N) c[row0 + g + 8] = from_f32<T>(acc[j][2 + e]);

@@ -1,8 +1,8 @@
 """Throughput of the layer-listed decoders (latent attention / mixture of experts, matrix memory / grouped
-attention) at sizes that resemble a real model's layers (random weights), beside an OPT-shaped
-PipelineModel of equal width, heads, depth and weights per token, and the time of every kernel next to
-its roofline and to the like kernel of the other model.  `bench.py --design tulezen | mutolix` prints
-the result as one JSON line."""
+attention, state space / chunk attention beside gated linear attention) at sizes that resemble a real model's
+layers (random weights), beside an OPT-shaped PipelineModel of equal width, heads, depth and weights per
+token, and the time of every kernel next to its roofline and to the like kernel of another model.
+`bench.py --design tulezen | mutolix | moponex` prints the result as one JSON line."""
 import json
 import os
 import statistics
@@ -352,7 +352,228 @@ def mutolix_kernel_table(z, B, S, T):
     return rows, {}
 
 
+MOPONEX_SIZES = {
+    # alternating parallel layers (chunk attention | gated linear attention, dense feed-forward) and state-space layers
+    # (routed experts); g*: the gated linear heads, s*: the state space's
+    "2048": dict(width=2048, heads=16, kv_heads=4, dim=128, chunk=1024, gheads=8, gdim=128, gvdim=256, rank=16, ff=5632, sheads=64, svdim=64, state=128,
+                 sgroups=1, norm_groups=1, experts=62, identity=2, groups=8, keep=4, top=6, eff=1024, shared=2048, layers=8, vocab=32768),
+    "4096": dict(width=4096, heads=32, kv_heads=8, dim=128, chunk=2048, gheads=16, gdim=128, gvdim=256, rank=16, ff=11264, sheads=128, svdim=64, state=128,
+                 sgroups=8, norm_groups=8, experts=30, identity=2, groups=4, keep=2, top=4, eff=2048, shared=4096, layers=6, vocab=32768),
+}
+
+
+def make_moponex(z):
+    from ..registry import build_model
+    par = {"type": "parallel", "mlp": {"kind": "dense", "ff": z["ff"]},
+           "mixer": {"left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                              "mask": {"size": z["chunk"]}, "rot": {"dims": z["dim"] // 2, "base": 1e4, "scaling": {"factor": 4.0}}},
+                     "right": {"heads": z["gheads"], "dim": z["gdim"], "vdim": z["gvdim"], "tau": 16.0, "rank": z["rank"]}}}
+    ssm = {"type": "mamba2", "mixer": {"heads": z["sheads"], "vdim": z["svdim"], "state": z["state"], "groups": z["sgroups"], "conv": 4,
+                                       "norm_groups": z["norm_groups"]},
+           "mlp": {"kind": "moe", "expert": {"ff": z["eff"]}, "shared": {"ff": z["shared"]},
+                   "router": {"experts": z["experts"], "top": z["top"], "identity": z["identity"], "groups": {"count": z["groups"], "keep": z["keep"]}}}}
+    torch.manual_seed(1)
+    return build_model("Moponex", dtype=torch.bfloat16, device="cuda", config_dict={
+        "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.7, "logit_scale": 0.5, "layers": [par, ssm] * (z["layers"] // 2),
+        "embedding": {"bigram": {"buckets": z["vocab"] - 1, "mul_prev": 31, "mul_cur": 7}}})
+
+
+def moponex_as_opt(z):
+    """The feed-forward size with which an OPT layer has as many weights per token as a layer here has on average."""
+    w = z["width"]
+    par = w * (2 * z["heads"] * z["dim"] + z["kv_heads"] * z["dim"] + 2 * z["gheads"] * z["gdim"] + 3 * z["gheads"] * z["gvdim"] + 3 * z["ff"])
+    ssm = w * (3 * z["sheads"] * z["svdim"] + 2 * z["sgroups"] * z["state"] + 2 * z["shared"] + 2 * z["top"] * z["eff"])
+    ffn = ((par + ssm) / 2 / w - 4 * w) / 2
+    return dict(z, top=1, ff=int(ffn / 1.5))
+
+
+def moponex_kernel_table(z, B, S, T):
+    """As kernel_table, for the state-space / chunk-attention / gated-linear decoder."""
+    from ..attention import (attention_decode, attention_group_decode_chunk, attention_inputs, attention_prefill, attention_prefill_chunk, attention_rotary)
+    from ..decay import gate_group_norm, gla_prompt, gla_step, short_conv, ssm_prompt, ssm_step
+    from ..gemm import gemm, project_parts, project_unit
+    from ..kernel.cuda_native.layer_norm import layer_norm_forward
+    from ..memory import head_norm_gate, memory_prompt, memory_step
+    from ..moe import RouterRule, SortedRows, grouped_gemm, new_counts, route, route_rule, skinny_experts
+    from ..norm import rms_residual, stream_add, stream_update
+    bf, f32, dev = torch.bfloat16, torch.float32, "cuda"
+    W, H, G, d, ff = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
+    GH, gd, gv, rank = z["gheads"], z["gdim"], z["gvdim"], z["rank"]
+    SH, sv, N, SG = z["sheads"], z["svdim"], z["state"], z["sgroups"]
+    E, K, eff, n = z["experts"], z["top"], z["eff"], z["experts"] + z["identity"]
+    rnd = lambda *s, dtype=bf: (torch.randn(*s, device=dev, dtype=torch.float32) * 0.05).to(dtype)
+    rows = []
+
+    def add(phase, name, like, us, nbytes, flops=0.0):
+        rows.append((phase, name, like, us, float(nbytes), float(flops)))
+
+    def product(phase, name, M, Nn, Kd, like=None, unit=None, act=None, tail=0, out32=False):
+        Nn += tail
+        cols = Nn // 2 if unit == "geglu" else Nn
+        nb = 2 * (Nn * Kd + M * Kd) + (4 if out32 else 2) * M * (cols + tail)
+        ws = [rnd(Nn, Kd) for _ in range(copies(2 * Nn * Kd, 32))]
+        xs = [rnd(M, Kd) for _ in range(4)]
+        bias = rnd(Nn)
+        if unit:
+            call = lambda w, x: project_unit(x, w, unit)
+        elif tail:
+            call = lambda w, x: project_parts(x, w, tail_col=Nn - tail)
+        else:
+            call = lambda w, x: gemm(x, w, bias=bias if act else None, act=act, out_dtype=f32 if out32 else None, static_weight=True)
+        add(phase, name, like, time_calls([lambda w=w, x=xs[i % 4]: call(w, x) for i, w in enumerate(ws)]), nb, 2.0 * M * Nn * Kd)
+
+    inner, chan = SH * sv, SH * sv + 2 * SG * N
+    n_ssm, n_par = inner + chan, (H + G) * d + 2 * GH * (gd + gv) + rank
+    qk, vg = GH * gd, GH * gv
+    nw, w32, lw, lb = rnd(W), torch.ones(W, device=dev), rnd(W), rnd(W)
+    per_head = [torch.full((SH,), v, device=dev) for v in (-2.0, -1.0, 1.0)]
+    conv_w, conv_b, ssm_norm = rnd(4, chan), rnd(chan), rnd(inner)
+    a2, a2b, gnorm = rnd(qk, rank), rnd(qk), rnd(vg)
+    qn, kn, freq, sinks = rnd(d), rnd(d), torch.rand(d // 4, device=dev), torch.zeros(H, device=dev)
+    corr = torch.rand(n, device=dev) * 0.01 - 1.0
+    rule = RouterRule(n, E, corr, z["groups"], z["keep"])
+    R = min(z["chunk"], S)
+    mbias = tuple(torch.zeros(GH, device=dev) + x for x in (0.0, 4.0))
+
+    def gemms(phase, M):
+        product(phase, "gemm in_proj (state space)", M, n_ssm, W, tail=SH)
+        product(phase, "gemm in_proj (parallel)", M, n_par, W)
+        product(phase, "gemm out_proj", M, W, H * d)
+        product(phase, "gemm gate_up + geglu", M, 2 * ff, W, like="gemm fc1 relu (OPT)", unit="geglu")
+        product(phase, "gemm fc1 relu (OPT)", M, 2 * ff, W, act="relu")
+        product(phase, "gemm down", M, W, ff)
+        product(phase, "gemm shared up + gelu", M, z["shared"], W, like="gemm out_proj", unit="gelu")
+
+    # ---- generation step ----
+    gemms("step", B)
+    pos = torch.tensor([S - 1], dtype=torch.int32, device=dev)
+    nb = 8 * B * SH * N * sv
+    states = [rnd(B, SH, N, sv, dtype=f32) for _ in range(copies(nb / 2))]
+    row, dt, ring = rnd(B, n_ssm), rnd(B, SH, dtype=f32), rnd(B, 4, chan)
+    add("step", "ssm_step", "memory_step (Mutolix)", time_calls([lambda s=s: ssm_step(row[:, inner:], conv_w, conv_b, ring, pos, dt, *per_head, s, SH, SG, N, sv)
+                                                                 for s in states]), nb + 2 * B * (6 * chan + inner))
+    del states
+    y = rnd(B, inner)
+    add("step", "gate_group_norm", "layer_norm (OPT)", time_calls([lambda: gate_group_norm(y, row[:, :inner], ssm_norm, 1e-6, SH, sv, z["norm_groups"])] * 16), 6 * B * inner)
+    nb = 8 * B * GH * gd * gv
+    states = [rnd(B, GH, gd, gv, dtype=f32) for _ in range(copies(nb / 2))]
+    row = rnd(B, n_par)
+    q, k, v, g, low = row[:, (H + G) * d:].split([qk, qk, vg, vg, rank], 1)
+    add("step", "gla_step", "memory_step (Mutolix)", time_calls([lambda s=s: gla_step(q, k, v, g, low, a2, a2b, 16.0, gd ** -0.5, gnorm, gv, 1e-6, s, GH) for s in states]),
+        nb + 2 * B * (2 * qk + 3 * vg) + 2 * qk * rank)
+    gates = rnd(B, 2 * GH, dtype=f32)
+    extra = [[rnd(B, GH, gd, dtype=f32), torch.zeros(B, GH, device=dev)] for _ in states]
+    add("step", "memory_step (Mutolix)", None, time_calls([lambda s=s, e=e: memory_step(q, k, v, g, gates, mbias, 15.0, gd ** -0.5, gnorm, gv, 1e-6, [s] + e, GH)
+                                                           for s, e in zip(states, extra)]), nb + 2 * B * (2 * qk + 3 * vg))
+    del states, extra
+    kv = [rnd(B, R, 2 * G * d) for _ in range(copies(B * R * 2 * G * d * 2))]
+    qr = rnd(B, H * d)
+    add("step", "attention_group_decode chunk", "attention_decode (OPT)", time_calls([lambda c=c: attention_group_decode_chunk(
+        qr, c[:, :, :G * d], c[:, :, G * d:], d, pos, 0.09, z["chunk"], sinks=sinks) for c in kv]), 4 * B * (((S - 1) % z["chunk"]) + 1) * G * d + 4 * B * H * d)
+    add("step", "attention_rotary", "layer_norm (OPT)", time_calls([lambda c=c: attention_rotary(row, H, G, d, d, qn, kn, 1e-6, freq, c[:, :, :G * d], c[:, :, G * d:], 1,
+                                                                                                 pos_device=pos) for c in kv]), 4 * B * H * d + 6 * B * G * d)
+    del kv
+    kv = [rnd(B, R, 3 * H * d) for _ in range(copies(B * R * 2 * H * d * 2))]
+    add("step", "attention_decode (OPT)", None, time_calls([lambda c=c: attention_decode(
+        c[:, :, 2 * H * d:], c[:, :, :H * d], c[:, :, H * d:2 * H * d], d, R, q_in_cache=True) for c in kv]), 4 * B * R * H * d)
+    del kv
+    x, y, y2 = torch.randn(B, W, device=dev), rnd(B, W), rnd(B, W)
+    add("step", "stream_add", "layer_norm (OPT)", time_calls([lambda: stream_add(x, 1e-6, y=y, scale=0.7, w_next=nw)] * 16), 12 * B * W)
+    add("step", "stream_add, two rows", "layer_norm (OPT)", time_calls([lambda: stream_add(x, 1e-6, y=y, w=w32, y2=y2, w2=w32, scale=0.7, w_next=nw)] * 16), 14 * B * W)
+    routers = [rnd(n + 8, W) for _ in range(16)]
+    add("step", "stream_add + router", "rms_residual + router (Tulezen)", time_calls([lambda r=r: stream_add(x, 1e-6, y=y, scale=0.7, w_next=nw, router=(r, rule, K, True))
+                                                                                      for r in routers]), 12 * B * W + 2 * (n + 1) * W)
+    xt = rnd(B, W)
+    add("step", "rms_residual + router (Tulezen)", None, time_calls([lambda r=r: rms_residual(y, nw, 1e-5, x, xt=xt, router=(r, n, K)) for r in routers]), 12 * B * W + 2 * n * W)
+    add("step", "layer_norm (OPT)", None, time_calls([lambda: layer_norm_forward(xt, lw, lb, 1e-5)] * 16), 4 * B * W)
+    n_w = max(2, min(8, -(-FLUSH_BYTES // (4 * E * eff * W))))
+    ups, downs = [rnd(E, eff, W) for _ in range(n_w)], [rnd(E, W, eff) for _ in range(n_w)]
+    idx, w, _, gate = route_rule(torch.randn(B, n + 1, device=dev), rule, K, gated=True)
+    live = idx[idx < E]
+    act_e, pairs = int(live.unique().numel()), int(live.numel())
+    a = rnd(B * K, eff)
+    add("step", "experts up + gelu", "gemm out_proj", time_calls([lambda u=u: skinny_experts(xt, u, idx, K, unit="gelu") for u in ups]),
+        2 * (act_e * eff * W + B * W + pairs * eff), 2.0 * pairs * eff * W)
+    add("step", "experts down", "gemm out_proj", time_calls([lambda u=u: skinny_experts(a, u, idx, 1) for u in downs]), 2 * (act_e * eff * W + pairs * (W + eff)),
+        2.0 * pairs * eff * W)
+    ym, sh = rnd(B * K, W), rnd(B, W)
+    add("step", "stream_add of a mixture", "layer_norm (OPT)", time_calls([lambda: stream_add(
+        x, 1e-6, y=ym, mix=(idx, None, w), ident=xt, experts=E, shared=sh, gate=gate, scale=0.7, w_next=nw)] * 16), 12 * B * W + 2 * (pairs + B) * W)
+
+    # ---- prompt ----
+    seq = min(S, T)
+    nB = T // seq
+    gemms("prompt", T)
+    product("prompt", "gemm decay logits", T, qk, rank, out32=True)
+    projs = [rnd(T, n_ssm) for _ in range(3)]
+    ring = rnd(nB, 4, chan)
+    add("prompt", "short_conv", "layer_norm (OPT)", time_calls([lambda r=r: short_conv(r[:, inner:], conv_w, conv_b, ring, nB) for r in projs]), 4 * T * chan)
+    xbc, dt = [short_conv(r[:, inner:], conv_w, conv_b, ring, nB) for r in projs], rnd(T, SH, dtype=f32)
+    state = torch.empty(nB, SH, N, sv, device=dev)
+    add("prompt", "ssm_chunks", "memory_chunks (Mutolix)", time_calls([lambda r=r: ssm_prompt(r, dt, *per_head, state, SH, SG, N, sv, chunked=True) for r in xbc]),
+        2 * T * (chan + inner) + 4 * T * SH + 4 * nB * SH * N * sv, 4.0 * T * SH * N * sv)
+    ys = [rnd(T, inner) for _ in range(3)]
+    add("prompt", "gate_group_norm", "layer_norm (OPT)", time_calls([lambda y=y, r=r: gate_group_norm(y, r[:, :inner], ssm_norm, 1e-6, SH, sv, z["norm_groups"])
+                                                                     for y, r in zip(ys, projs)]), 6 * T * inner)
+    del projs, xbc, ys, state
+    projs = [rnd(T, n_par) for _ in range(3)]
+    zl = rnd(T, qk, dtype=f32) + 2.0
+    state = torch.empty(nB, GH, gd, gv, device=dev)
+    part = lambda r: r[:, (H + G) * d:(H + G) * d + 2 * qk + vg].split([qk, qk, vg], 1)
+    add("prompt", "gla_chunks", "memory_chunks (Mutolix)", time_calls([lambda r=r: gla_prompt(*part(r), zl, 16.0, gd ** -0.5, state, GH, chunked=True) for r in projs]),
+        4 * T * (qk + vg) + 4 * T * qk + 4 * nB * GH * gd * gv, 4.0 * T * GH * gd * gv)
+    gates, ms = rnd(T, 2 * GH, dtype=f32), [state, torch.empty(nB, GH, gd, device=dev), torch.empty(nB, GH, device=dev)]
+    add("prompt", "memory_chunks (Mutolix)", None, time_calls([lambda r=r: memory_prompt(*part(r), gates, mbias, 15.0, gd ** -0.5, ms, GH, chunked=True) for r in projs]),
+        4 * T * (qk + vg) + 8 * T * GH + 4 * nB * GH * gd * gv, 4.0 * T * GH * gd * gv)
+    os_ = [rnd(T, vg) for _ in range(4)]
+    add("prompt", "head_norm_gate", "layer_norm (OPT)", time_calls([lambda o=o: head_norm_gate(o, projs[0][:, -vg - rank:-rank], gnorm, GH, gv, 1e-6, silu=True) for o in os_]),
+        6 * T * vg)
+    rb = rnd(nB, min(z["chunk"], seq), 2 * G * d)
+    add("prompt", "attention_rotary", "layer_norm (OPT)", time_calls([lambda r=r: attention_rotary(
+        r, H, G, d, d, qn, kn, 1e-6, freq, rb[:, :, :G * d], rb[:, :, G * d:], seq, keys=True) for r in projs]), 4 * T * (H + G) * d + 4 * nB * rb.shape[1] * G * d)
+    del projs, os_, state, ms
+    q3, k3, v3, kv3 = rnd(nB, seq, H * d), rnd(nB, seq, G * d), rnd(nB, seq, G * d), rnd(nB, seq, 2 * H * d)
+    c = z["chunk"]
+    seen = sum(i % c + 1 for i in range(seq))
+    add("prompt", "attention chunk", "attention causal (OPT)", time_calls([lambda: attention_prefill_chunk(q3, k3, v3, d, c, sinks=sinks)] * 4), 2 * T * (2 * H + 2 * G) * d,
+        4.0 * nB * H * d * seen)
+    add("prompt", "attention causal (OPT)", None, time_calls([lambda: attention_prefill(q3, kv3[:, :, :H * d], kv3[:, :, H * d:], d)] * 4), 2 * T * 4 * H * d,
+        4.0 * nB * H * d * seq * (seq + 1) / 2)
+    del q3, k3, v3, kv3
+    xs = [torch.randn(T, W, device=dev) for _ in range(copies(12 * T * W, 8))]
+    ys = [rnd(T, W) for _ in xs]
+    add("prompt", "stream_add", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(x, 1e-6, y=y, scale=0.7, w_next=nw) for x, y in zip(xs, ys)]), 12 * T * W)
+    add("prompt", "stream_add, two rows", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(x, 1e-6, y=y, w=w32, y2=ys[0], w2=w32, scale=0.7, w_next=nw)
+                                                                          for x, y in zip(xs[1:], ys[1:])]), 14 * T * W)
+    add("prompt", "layer_norm (OPT)", None, time_calls([lambda t=t: layer_norm_forward(t, lw, lb, 1e-5) for t in ys]), 4 * T * W)
+    logits = torch.randn(T, n + 8, device=dev)
+    counts, n0, n1 = [new_counts(E, dev) for _ in range(3)]
+    add("prompt", "moe route by rule", "moe route (Tulezen)", time_calls([lambda: route_rule(logits, rule, K, counts=n0, gated=True)] * 4), 4 * T * n + 12 * T * K)
+    n2 = new_counts(n, dev)
+    add("prompt", "moe route (Tulezen)", None, time_calls([lambda: route(logits, n, K, counts=n2)] * 4), 4 * T * n + 12 * T * K)
+    idx, w, ranks, gate = route_rule(logits, rule, K, counts=counts, gated=True)
+    keep = counts.clone()
+
+    def sort_rows():
+        n1.copy_(keep)
+        return SortedRows(ys[0], idx, ranks, n1)
+    plan = sort_rows()
+    pairs = int((idx < E).sum())
+    add("prompt", "moe plan + permute", "layer_norm (OPT)", time_calls([sort_rows] * 4), 2 * T * W + 2 * pairs * W)
+    add("prompt", "grouped up + gelu", "gemm out_proj", time_calls([lambda u=u: grouped_gemm(plan.x, u, plan, unit="gelu") for u in ups]),
+        2 * (E * eff * W + pairs * (W + eff)), 2.0 * pairs * eff * W)
+    act = grouped_gemm(plan.x, ups[0], plan, unit="gelu")
+    add("prompt", "grouped down", "gemm out_proj", time_calls([lambda u=u: grouped_gemm(act, u, plan) for u in downs]),
+        2 * (E * eff * W + pairs * (W + eff)), 2.0 * pairs * eff * W)
+    ym = grouped_gemm(act, downs[0], plan)
+    add("prompt", "stream_add of a mixture", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(
+        x, 1e-6, y=ym, mix=(idx, plan.rows, w), ident=y, experts=E, shared=ys[0], gate=gate, scale=0.7, w_next=nw) for x, y in zip(xs[1:], ys[1:])]),
+        12 * T * W + 2 * (pairs + T) * W)
+    return rows, {"active_experts": act_e, "sorted_rows": int(plan.live_tiles.item()) * 128, "routed_rows": pairs}
+
+
 DESIGNS = {
+    "moponex": dict(sizes=MOPONEX_SIZES, runs=RUNS, make=make_moponex, as_opt=moponex_as_opt, table=moponex_kernel_table),
     "tulezen": dict(sizes=SIZES, runs=RUNS, make=make_tulezen, as_opt=lambda z: z, table=kernel_table),
     "mutolix": dict(sizes=MUTOLIX_SIZES, runs=RUNS, make=make_mutolix, as_opt=mutolix_as_opt, table=mutolix_kernel_table),
 }
