@@ -99,7 +99,8 @@ __global__ void attention_rotary_kernel(const RotaryParams p) {
 
 template <typename T> int launch_rotary(const RotaryParams &p, int n1, cudaStream_t st) {
   const int all = p.heads + p.kv_heads, need = (p.dk / 2 + 31) / 32;
-  const dim3 g(n1), b(32 * (all < 8 ? all : 8));
+  const int most = n1 >= 4 * sm_count() ? 8 : 16;           // few rows: fewer heads one after the other
+  const dim3 g(n1), b(32 * (all < most ? all : most));
   if (need <= 1) launch_pdl(attention_rotary_kernel<T, 1>, g, b, 0, st, p);
   else if (need <= 2) launch_pdl(attention_rotary_kernel<T, 2>, g, b, 0, st, p);
   else if (need <= 4) launch_pdl(attention_rotary_kernel<T, 4>, g, b, 0, st, p);

@@ -45,7 +45,7 @@ moe_route_kernel(const float *logits, long long ld, int tokens, int experts, int
   for (int e = lane; e < experts; e += 32) z[e] = logits[(long long)t * ld + e];
   if (gate && lane == 0) gate[t] = 1.f / (1.f + expf(-logits[(long long)t * ld + gate_col]));
   __syncwarp();
-  if (RULE) route_warp_rule(z, experts, top, rule, idx + (long long)t * top, weights + (long long)t * top, counts, ranks ? ranks + (long long)t * top : nullptr);
+  if (RULE) route_warp_rule<false>(z, experts, top, rule, idx + (long long)t * top, weights + (long long)t * top, counts, ranks ? ranks + (long long)t * top : nullptr);
   else route_warp(z, experts, top, idx + (long long)t * top, weights + (long long)t * top, counts, ranks ? ranks + (long long)t * top : nullptr);
 }
 

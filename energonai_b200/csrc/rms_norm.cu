@@ -299,17 +299,29 @@ __global__ void __launch_bounds__(THREADS) stream_add_kernel(const AddParams p) 
 #pragma unroll
       for (int e = 0; e < 8; ++e) v[i][e] = 0.f;
       float self = 0.f;
-      for (int k = 0; k < p.top; ++k) {
-        const long long a = row * p.top + k;
-        const int ex = p.idx[a];
-        const float s = p.weights[a];
-        if (ex < 0) continue;
-        if (ex >= p.experts) { self += s; continue; }
-        const long long src = p.rows ? p.rows[a] : a;
-        float f[8];
-        load8<T>(reinterpret_cast<const T *>(p.y) + src * p.ldy + c * 8, f);
+      constexpr int kAhead = 4;                    // choices whose rows are in flight together
+      for (int k0 = 0; k0 < p.top; k0 += kAhead) {
+        float s[kAhead], f[kAhead][8];
+        long long src[kAhead];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) v[i][e] = fmaf(s, f[e], v[i][e]);
+        for (int k = 0; k < kAhead; ++k) {
+          const bool in = k0 + k < p.top;
+          const long long a = row * p.top + (in ? k0 + k : 0);
+          const int ex = p.idx[a];
+          s[k] = p.weights[a];
+          src[k] = p.rows ? p.rows[a] : a;
+          if (in && ex >= p.experts) self += s[k];
+          if (!in || ex < 0 || ex >= p.experts) src[k] = -1;
+        }
+#pragma unroll
+        for (int k = 0; k < kAhead; ++k)
+          if (src[k] >= 0) load8<T>(reinterpret_cast<const T *>(p.y) + src[k] * p.ldy + c * 8, f[k]);
+#pragma unroll
+        for (int k = 0; k < kAhead; ++k) {
+          if (src[k] < 0) continue;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) v[i][e] = fmaf(s[k], f[k][e], v[i][e]);
+        }
       }
       if (self != 0.f) {
         float f[8];
@@ -401,7 +413,7 @@ __global__ void __launch_bounds__(THREADS) stream_add_kernel(const AddParams p) 
     }
   }
   __syncthreads();
-  if (warp == 0) route_warp_rule(z, p.choices, p.r_top, p.rule, p.r_idx + row * p.r_top, p.r_weights + row * p.r_top, nullptr, nullptr);
+  if (warp == 0) route_warp_rule<true>(z, p.choices, p.r_top, p.rule, p.r_idx + row * p.r_top, p.r_weights + row * p.r_top, nullptr, nullptr);
 }
 
 template <typename T, int FORM> int launch_add(const AddParams &p, int n1, cudaStream_t st) {

@@ -52,6 +52,8 @@ __device__ __forceinline__ void route_warp(float *z, int experts, int top, int *
   }
 }
 
+constexpr int kRankChoices = 128;
+
 // How a router chooses beyond the plain softmax scores.
 struct RouterRule {
   const float *correction = nullptr;   // [choices] added to the scores for the choice alone, or null
@@ -90,7 +92,9 @@ __device__ __forceinline__ void warp_argmax(const float *v, int n, float &best, 
 
 // route_warp with a rule; z has room for rule_floats() numbers.  The `top` choices with the largest
 // score + correction among the open groups are taken; their weights are their scores, divided by
-// their sum (+ 1e-20).
+// their sum (+ 1e-20).  RANKS: up to kRankChoices choices each one's rank is counted, which takes a warp by itself less
+// time than picking one after the other (and many warps together more).
+template <bool RANKS>
 __device__ __forceinline__ void route_warp_rule(float *z, int choices, int top, const RouterRule &rule, int *idx, float *weights, int *counts, int *ranks) {
   const int lane = threadIdx.x & 31;
   float *c = z + choices, *gs = c + choices, *open = gs + rule.groups;
@@ -108,25 +112,75 @@ __device__ __forceinline__ void route_warp_rule(float *z, int choices, int top, 
   __syncwarp();
   if (rule.keep < rule.groups) {
     const int per = choices / rule.groups;
-    for (int g = 0; g < rule.groups; ++g) {
-      float b = -INFINITY;
-      for (int e = lane; e < per; e += 32) b = fmaxf(b, c[g * per + e]);
-      b = warp_max(b);
-      if (lane == 0) { gs[g] = b; open[g] = 0.f; }
-    }
-    __syncwarp();
-    for (int k = 0; k < rule.keep; ++k) {
-      float best;
-      int bi;
-      warp_argmax(gs, rule.groups, best, bi);
-      if (lane == 0 && bi < rule.groups) { gs[bi] = -INFINITY; open[bi] = 1.f; }
+    if (rule.groups <= 32) {                         // lane = group: its rank among them
+      float mine = -INFINITY;
+      if (lane < rule.groups)
+        for (int e = 0; e < per; ++e) mine = fmaxf(mine, c[lane * per + e]);
+      int before = 0;
+      for (int g = 0; g < rule.groups; ++g) {
+        const float other = __shfl_sync(0xffffffffu, mine, g);
+        before += other > mine || (other == mine && g < lane);
+      }
+      if (lane < rule.groups) open[lane] = before < rule.keep ? 1.f : 0.f;
       __syncwarp();
+    } else {
+      for (int g = lane; g < rule.groups; g += 32) {
+        float b = -INFINITY;
+        for (int e = 0; e < per; ++e) b = fmaxf(b, c[g * per + e]);
+        gs[g] = b;
+        open[g] = 0.f;
+      }
+      __syncwarp();
+      for (int k = 0; k < rule.keep; ++k) {
+        float best;
+        int bi;
+        warp_argmax(gs, rule.groups, best, bi);
+        if (lane == 0 && bi < rule.groups) { gs[bi] = -INFINITY; open[bi] = 1.f; }
+        __syncwarp();
+      }
     }
     for (int e = lane; e < choices; e += 32)
       if (open[e / per] == 0.f) c[e] = -INFINITY;
     __syncwarp();
   }
   float total = 0.f;
+  if (RANKS && choices <= kRankChoices) {
+    // every choice's rank among all; the first `top` are taken.  (Logits that are not numbers leave places of the list
+    // untaken: any valid choices stand there.)
+    for (int k = lane; k < top; k += 32) {
+      idx[k] = k;
+      weights[k] = 0.f;
+      if (counts) ranks[k] = -1;
+    }
+    __syncwarp();
+    float mine[kRankChoices / 32];
+    int before[kRankChoices / 32];
+#pragma unroll
+    for (int i = 0; i < kRankChoices / 32; ++i) {
+      mine[i] = lane + 32 * i < choices ? c[lane + 32 * i] : -INFINITY;
+      before[i] = 0;
+    }
+    for (int e = 0; e < choices; ++e) {
+      const float other = c[e];
+#pragma unroll
+      for (int i = 0; i < kRankChoices / 32; ++i)
+        if (32 * i < choices) before[i] += other > mine[i] || (other == mine[i] && e < lane + 32 * i);
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kRankChoices / 32; ++i)
+      if (lane + 32 * i < choices && before[i] < top) sum += z[lane + 32 * i];
+    total = warp_sum(sum) + 1e-20f;
+#pragma unroll
+    for (int i = 0; i < kRankChoices / 32; ++i) {
+      const int e = lane + 32 * i, k = before[i];
+      if (e >= choices || k >= top) continue;
+      idx[k] = e;
+      weights[k] = z[e] / total;
+      if (counts) ranks[k] = e < rule.real ? atomicAdd(counts + e * kCountStride, 1) : -1;
+    }
+    return;
+  }
   for (int k0 = 0; k0 < top; k0 += 32) {
     int mine = 0;                                    // lane k: choice k0 + k
     float score = 0.f;

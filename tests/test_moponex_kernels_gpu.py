@@ -81,7 +81,7 @@ def test_units_of_experts(dtype, unit):
 
 
 # ---- router ---------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("T,E,identity,top,groups,keep", [(33, 16, 0, 4, 1, 1), (40, 13, 2, 3, 3, 2), (7, 5, 1, 2, 2, 1), (20, 60, 4, 40, 4, 3), (9, 3, 0, 1, 3, 1),
+@pytest.mark.parametrize("T,E,identity,top,groups,keep", [(33, 16, 0, 4, 1, 1), (40, 13, 2, 3, 3, 2), (7, 5, 1, 2, 2, 1), (20, 60, 4, 40, 4, 3), (11, 130, 6, 40, 34, 20), (9, 3, 0, 1, 3, 1),
                                                           (12, 250, 6, 8, 8, 4)])
 def test_router_rule(T, E, identity, top, groups, keep):
     from energonai_b200.moe import RouterRule, new_counts, route_rule
