@@ -259,7 +259,7 @@ struct AddParams {
   float *r_weights, *r_gate;
 };
 
-enum { kAddRow = 0, kAddTwo = 1, kAddMix = 2 };
+enum { kAddRow = 0, kAddTwo = 1, kAddMix = 2, kAddMixFew = 3 };      // kAddMixFew: few rows, several choices' rows in flight per thread
 
 template <typename T, int PACKS, int FORM, int THREADS>
 __global__ void __launch_bounds__(THREADS) stream_add_kernel(const AddParams p) {
@@ -295,11 +295,11 @@ __global__ void __launch_bounds__(THREADS) stream_add_kernel(const AddParams p) 
     } else {
       load8<float>(p.x + row * p.ldx + c * 8, xv[i]);
     }
-    if (FORM == kAddMix) {
+    if (FORM >= kAddMix) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) v[i][e] = 0.f;
       float self = 0.f;
-      constexpr int kAhead = 4;                    // choices whose rows are in flight together
+      constexpr int kAhead = FORM == kAddMixFew ? 4 : 1;
       for (int k0 = 0; k0 < p.top; k0 += kAhead) {
         float s[kAhead], f[kAhead][8];
         long long src[kAhead];
@@ -675,7 +675,7 @@ extern "C" int eb_stream_add(const void *src, long long lds, const void *src2, l
   p.eps = eps; p.inv_count = 1.f / (float)count; p.n2 = n2;
   p.router = router; p.choices = choices; p.r_top = r_top; p.r_idx = r_idx; p.r_weights = r_weights; p.r_gate = r_gate;
   cudaStream_t st = as_stream(stream);
-#define EB_ADD(T) (idx ? launch_add<T, kAddMix>(p, n1, st) : y2 ? launch_add<T, kAddTwo>(p, n1, st) : launch_add<T, kAddRow>(p, n1, st))
+#define EB_ADD(T) (idx ? (n1 < 4 * sm_count() ? launch_add<T, kAddMixFew>(p, n1, st) : launch_add<T, kAddMix>(p, n1, st)) : y2 ? launch_add<T, kAddTwo>(p, n1, st) : launch_add<T, kAddRow>(p, n1, st))
   if (dtype == EB_F32) return EB_ADD(float);
   if (dtype == EB_F16) return EB_ADD(__half);
   return EB_ADD(__nv_bfloat16);

@@ -178,6 +178,19 @@ def test_stream_add_of_a_mixture_and_the_router_behind_it(dtype, width, experts,
         assert (rg is None) == (not gated) and (rg is None or torch.allclose(rg.cpu().double(), torch.sigmoid(z[:, n]), rtol=1e-4))
 
 
+def test_stream_add_of_a_mixture_of_many_rows():
+    from energonai_b200.norm import stream_add
+    T, width, E, top = 700, 72, 5, 3
+    g = torch.Generator().manual_seed(2)
+    y, h0, sh, x0 = rnd(T * top, width, seed=1), rnd(T, width, seed=2), rnd(T, width, seed=3), rnd(T, width, seed=4)
+    idx, w, gate = torch.randint(0, E + 2, (T, top), generator=g).to(torch.int32), torch.rand(T, top, generator=g), torch.rand(T, generator=g)
+    rows = torch.where(idx[..., None] < E, y.view(T, top, width), h0[:, None])
+    want = x0.double() + 0.5 * ((w[..., None].double() * rows.double()).sum(1) + gate[:, None].double() * sh.double())
+    x = x0.cuda()
+    stream_add(x, 1e-5, y=y.cuda(), mix=(idx.cuda(), None, w.cuda()), ident=h0.cuda(), experts=E, shared=sh.cuda(), gate=gate.cuda(), scale=0.5)
+    assert rel(x, want) < 2e-6
+
+
 # ---- bigram rows in the tail of a step ---------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", [F32, BF16])
 def test_greedy_step_with_bigram_rows(dtype):
