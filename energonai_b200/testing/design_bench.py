@@ -366,16 +366,16 @@ def make_moponex(z):
     from ..registry import build_model
     par = {"type": "parallel", "mlp": {"kind": "dense", "ff": z["ff"]},
            "mixer": {"left": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
-                              "mask": {"size": z["chunk"]}, "rot": {"dims": z["dim"] // 2, "base": 1e4, "scaling": {"factor": 4.0}}},
-                     "right": {"heads": z["gheads"], "dim": z["gdim"], "vdim": z["gvdim"], "tau": 16.0, "rank": z["rank"]}}}
+                              "mask": {"size": z["chunk"]}, "rot": {"dims": z["dim"] // 2, "base": 5e5, "scaling": {"factor": 4.0}}},
+                     "right": {"heads": z["gheads"], "dim": z["gdim"], "vdim": z["gvdim"], "tau": 12.0, "rank": z["rank"]}}}
     ssm = {"type": "mamba2", "mixer": {"heads": z["sheads"], "vdim": z["svdim"], "state": z["state"], "groups": z["sgroups"], "conv": 4,
                                        "norm_groups": z["norm_groups"]},
            "mlp": {"kind": "moe", "expert": {"ff": z["eff"]}, "shared": {"ff": z["shared"]},
                    "router": {"experts": z["experts"], "top": z["top"], "identity": z["identity"], "groups": {"count": z["groups"], "keep": z["keep"]}}}}
     torch.manual_seed(1)
     return build_model("Moponex", dtype=torch.bfloat16, device="cuda", config_dict={
-        "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.7, "logit_scale": 0.5, "layers": [par, ssm] * (z["layers"] // 2),
-        "embedding": {"bigram": {"buckets": z["vocab"] - 1, "mul_prev": 31, "mul_cur": 7}}})
+        "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.8, "logit_scale": 0.25, "layers": [par, ssm] * (z["layers"] // 2),
+        "embedding": {"bigram": {"buckets": z["vocab"] - 1, "mul_prev": 1021, "mul_cur": 13}}})
 
 
 def moponex_as_opt(z):
@@ -459,7 +459,7 @@ def moponex_kernel_table(z, B, S, T):
     states = [rnd(B, GH, gd, gv, dtype=f32) for _ in range(copies(nb / 2))]
     row = rnd(B, n_par)
     q, k, v, g, low = row[:, (H + G) * d:].split([qk, qk, vg, vg, rank], 1)
-    add("step", "gla_step", "memory_step (Mutolix)", time_calls([lambda s=s: gla_step(q, k, v, g, low, a2, a2b, 16.0, gd ** -0.5, gnorm, gv, 1e-6, s, GH) for s in states]),
+    add("step", "gla_step", "memory_step (Mutolix)", time_calls([lambda s=s: gla_step(q, k, v, g, low, a2, a2b, 12.0, gd ** -0.5, gnorm, gv, 1e-6, s, GH) for s in states]),
         nb + 2 * B * (2 * qk + 3 * vg) + 2 * qk * rank)
     gates = rnd(B, 2 * GH, dtype=f32)
     extra = [[rnd(B, GH, gd, dtype=f32), torch.zeros(B, GH, device=dev)] for _ in states]
@@ -478,10 +478,10 @@ def moponex_kernel_table(z, B, S, T):
         c[:, :, 2 * H * d:], c[:, :, :H * d], c[:, :, H * d:2 * H * d], d, R, q_in_cache=True) for c in kv]), 4 * B * R * H * d)
     del kv
     x, y, y2 = torch.randn(B, W, device=dev), rnd(B, W), rnd(B, W)
-    add("step", "stream_add", "layer_norm (OPT)", time_calls([lambda: stream_add(x, 1e-6, y=y, scale=0.7, w_next=nw)] * 16), 12 * B * W)
-    add("step", "stream_add, two rows", "layer_norm (OPT)", time_calls([lambda: stream_add(x, 1e-6, y=y, w=w32, y2=y2, w2=w32, scale=0.7, w_next=nw)] * 16), 14 * B * W)
+    add("step", "stream_add", "layer_norm (OPT)", time_calls([lambda: stream_add(x, 1e-6, y=y, scale=0.8, w_next=nw)] * 16), 12 * B * W)
+    add("step", "stream_add, two rows", "layer_norm (OPT)", time_calls([lambda: stream_add(x, 1e-6, y=y, w=w32, y2=y2, w2=w32, scale=0.8, w_next=nw)] * 16), 14 * B * W)
     routers = [rnd(n + 8, W) for _ in range(16)]
-    add("step", "stream_add + router", "rms_residual + router (Tulezen)", time_calls([lambda r=r: stream_add(x, 1e-6, y=y, scale=0.7, w_next=nw, router=(r, rule, K, True))
+    add("step", "stream_add + router", "rms_residual + router (Tulezen)", time_calls([lambda r=r: stream_add(x, 1e-6, y=y, scale=0.8, w_next=nw, router=(r, rule, K, True))
                                                                                       for r in routers]), 12 * B * W + 2 * (n + 1) * W)
     xt = rnd(B, W)
     add("step", "rms_residual + router (Tulezen)", None, time_calls([lambda r=r: rms_residual(y, nw, 1e-5, x, xt=xt, router=(r, n, K)) for r in routers]), 12 * B * W + 2 * n * W)
@@ -498,7 +498,7 @@ def moponex_kernel_table(z, B, S, T):
         2.0 * pairs * eff * W)
     ym, sh = rnd(B * K, W), rnd(B, W)
     add("step", "stream_add of a mixture", "layer_norm (OPT)", time_calls([lambda: stream_add(
-        x, 1e-6, y=ym, mix=(idx, None, w), ident=xt, experts=E, shared=sh, gate=gate, scale=0.7, w_next=nw)] * 16), 12 * B * W + 2 * (pairs + B) * W)
+        x, 1e-6, y=ym, mix=(idx, None, w), ident=xt, experts=E, shared=sh, gate=gate, scale=0.8, w_next=nw)] * 16), 12 * B * W + 2 * (pairs + B) * W)
 
     # ---- prompt ----
     seq = min(S, T)
@@ -520,7 +520,7 @@ def moponex_kernel_table(z, B, S, T):
     zl = rnd(T, qk, dtype=f32) + 2.0
     state = torch.empty(nB, GH, gd, gv, device=dev)
     part = lambda r: r[:, (H + G) * d:(H + G) * d + 2 * qk + vg].split([qk, qk, vg], 1)
-    add("prompt", "gla_chunks", "memory_chunks (Mutolix)", time_calls([lambda r=r: gla_prompt(*part(r), zl, 16.0, gd ** -0.5, state, GH, chunked=True) for r in projs]),
+    add("prompt", "gla_chunks", "memory_chunks (Mutolix)", time_calls([lambda r=r: gla_prompt(*part(r), zl, 12.0, gd ** -0.5, state, GH, chunked=True) for r in projs]),
         4 * T * (qk + vg) + 4 * T * qk + 4 * nB * GH * gd * gv, 4.0 * T * GH * gd * gv)
     gates, ms = rnd(T, 2 * GH, dtype=f32), [state, torch.empty(nB, GH, gd, device=dev), torch.empty(nB, GH, device=dev)]
     add("prompt", "memory_chunks (Mutolix)", None, time_calls([lambda r=r: memory_prompt(*part(r), gates, mbias, 15.0, gd ** -0.5, ms, GH, chunked=True) for r in projs]),
@@ -542,8 +542,8 @@ def moponex_kernel_table(z, B, S, T):
     del q3, k3, v3, kv3
     xs = [torch.randn(T, W, device=dev) for _ in range(copies(12 * T * W, 8))]
     ys = [rnd(T, W) for _ in xs]
-    add("prompt", "stream_add", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(x, 1e-6, y=y, scale=0.7, w_next=nw) for x, y in zip(xs, ys)]), 12 * T * W)
-    add("prompt", "stream_add, two rows", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(x, 1e-6, y=y, w=w32, y2=ys[0], w2=w32, scale=0.7, w_next=nw)
+    add("prompt", "stream_add", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(x, 1e-6, y=y, scale=0.8, w_next=nw) for x, y in zip(xs, ys)]), 12 * T * W)
+    add("prompt", "stream_add, two rows", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(x, 1e-6, y=y, w=w32, y2=ys[0], w2=w32, scale=0.8, w_next=nw)
                                                                           for x, y in zip(xs[1:], ys[1:])]), 14 * T * W)
     add("prompt", "layer_norm (OPT)", None, time_calls([lambda t=t: layer_norm_forward(t, lw, lb, 1e-5) for t in ys]), 4 * T * W)
     logits = torch.randn(T, n + 8, device=dev)
@@ -567,7 +567,7 @@ def moponex_kernel_table(z, B, S, T):
         2 * (E * eff * W + pairs * (W + eff)), 2.0 * pairs * eff * W)
     ym = grouped_gemm(act, downs[0], plan)
     add("prompt", "stream_add of a mixture", "layer_norm (OPT)", time_calls([lambda x=x, y=y: stream_add(
-        x, 1e-6, y=ym, mix=(idx, plan.rows, w), ident=y, experts=E, shared=ys[0], gate=gate, scale=0.7, w_next=nw) for x, y in zip(xs[1:], ys[1:])]),
+        x, 1e-6, y=ym, mix=(idx, plan.rows, w), ident=y, experts=E, shared=ys[0], gate=gate, scale=0.8, w_next=nw) for x, y in zip(xs[1:], ys[1:])]),
         12 * T * W + 2 * (pairs + T) * W)
     return rows, {"active_experts": act_e, "sorted_rows": int(plan.live_tiles.item()) * 128, "routed_rows": pairs}
 

@@ -257,7 +257,7 @@ def parallel_layer(left, right, mlp=None):
             "mixer": {"left": a, "right": {"heads": right[0], "dim": right[1], "vdim": right[2], "tau": right[3]}}}
 
 
-def make_config(layers, width, vocab, eps=2e-5, mult=0.6, logit_scale=0.3, bigram=(97, 31, 7)):
+def make_config(layers, width, vocab, eps=2e-5, mult=0.6, logit_scale=0.3, bigram=(97, 29, 11)):
     """The ranks of the decay projections are not part of a configuration: make_tensors() takes them from `layers`,
     and `ranks` keeps them (see with_ranks)."""
     emb = {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))} if bigram else {}

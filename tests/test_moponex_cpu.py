@@ -27,7 +27,7 @@ def config():
 def test_configuration_reads_every_size_and_rejects_what_it_does_not_know():
     c = HybridDecoderConfig.from_dict(P.file_config(config()))
     assert (c.vocab, c.width, c.eps, c.residual_mult, c.logit_scale, len(c.layers)) == (83, 52, 2e-5, 0.6, 0.3, 4)
-    assert (c.bigram.buckets, c.bigram.mul_prev, c.bigram.mul_cur) == (97, 31, 7)
+    assert (c.bigram.buckets, c.bigram.mul_prev, c.bigram.mul_cur) == (97, 29, 11)
     a, r = c.layers[0].mixer.left, c.layers[0].mixer.right
     assert (a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.chunk, a.rot_dims, a.rot_base, a.rot_factor) == (6, 2, 12, 12, 0.4, 9, 8, 100.0, 3.0)
     assert (r.heads, r.dim, r.vdim, r.tau, r.rank) == (3, 20, 28, 4.0, None) and c.layers[0].mlp.ff == 44

@@ -22,16 +22,16 @@ ODD = P.make_config([P.parallel_layer((6, 2, 12, 0.4, 9, (8, 100.0, 3.0)), (3, 2
                      P.ssm_layer(6, 10, 12, groups=3, conv=3, norm_groups=4, mlp=P.moe_mlp(7, 3, 20, identity=2, groups=(3, 2), shared=12)),
                      P.parallel_layer((2, 2, 9, 0.5, 0, None), (1, 8, 12, 1.0, 16), P.moe_mlp(5, 2, 12)),
                      P.ssm_layer(4, 16, 24, groups=4, conv=2, norm_groups=1),
-                     P.parallel_layer((4, 1, 16, 0.3, 33, (16, 5000.0, None)), (2, 12, 8, 16.0, 8), P.moe_mlp(8, 4, 8, identity=4, groups=(4, 3)))],
+                     P.parallel_layer((4, 1, 16, 0.3, 33, (16, 5000.0, None)), (2, 12, 8, 20.0, 8), P.moe_mlp(8, 4, 8, identity=4, groups=(4, 3)))],
                     width=52, vocab=83)
 # sizes that fill or exceed the tensor-core tiles; two heads per tile and one
 WIDE = P.make_config([P.ssm_layer(4, 64, 128, groups=2, mlp=P.moe_mlp(12, 3, 40, identity=4, groups=(4, 2), shared=72)),
-                      P.parallel_layer((20, 1, 64, 0.12, 130, (32, 10000.0, 2.0)), (2, 128, 136, 16.0, 16), P.dense_mlp(136)),
+                      P.parallel_layer((20, 1, 64, 0.12, 130, (48, 20000.0, 2.0)), (2, 128, 136, 12.0, 16), P.dense_mlp(136)),
                       P.ssm_layer(3, 136, 70, groups=1, norm_groups=3), P.parallel_layer((4, 2, 100, 0.1, 64, (100, 300.0, None)), (3, 50, 64, 2.0, 24)),
                       P.ssm_layer(5, 40, 20, groups=5, norm_groups=5, mlp=P.dense_mlp(64))], width=192, vocab=334, eps=1e-6, mult=1.0, logit_scale=1.0)
 # head sizes the tensor-core kernels do not have; heads, ranks, groups and taps of one; no bigram rows
-HUGE = P.make_config([P.parallel_layer((2, 1, 140, 0.08, 20, (40, 1000.0, 8.0)), (1, 136, 24, 8.0, 1), P.moe_mlp(3, 1, 16)),
-                      P.ssm_layer(1, 8, 136, conv=5), P.parallel_layer((1, 1, 2, 1.0, 1, (2, 10.0, None)), (1, 1, 1, 16.0, 3), P.dense_mlp(24)),
+HUGE = P.make_config([P.parallel_layer((2, 1, 140, 0.08, 20, (40, 1000.0, 8.0)), (1, 136, 24, 6.0, 1), P.moe_mlp(3, 1, 16)),
+                      P.ssm_layer(1, 8, 136, conv=5), P.parallel_layer((1, 1, 2, 1.0, 1, (2, 10.0, None)), (1, 1, 1, 9.0, 3), P.dense_mlp(24)),
                       P.ssm_layer(2, 1, 1, conv=1, norm_groups=2)], width=40, vocab=64, bigram=None)
 CONFIGS = {"odd": ODD, "wide": WIDE, "huge": HUGE}
 
@@ -131,6 +131,18 @@ def test_unequal_batch_against_each_alone(name, lens, dtype):
         for k in range(out.shape[0] - n):
             alone.append(model.step(torch.tensor([toks[r][n + k]], device="cuda")))
         check(out, torch.cat(alone), dtype)
+
+
+def test_float16():
+    """The third number format: tensor-core products and attention, recurrences on the CUDA cores."""
+    from energonai_b200.registry import build_model
+    from energonai_b200.utils import processing_Moponex
+    t = P.make_tensors(ODD, 1)
+    model = build_model("Moponex", config_dict=P.with_ranks(ODD), dtype=torch.float16)
+    model.load_state_dict(processing_Moponex(t, model))
+    model, toks = model.cuda().eval(), tokens(ODD, 60)
+    got = [prompt_logits(model, toks[:40])] + [model.step(torch.tensor([x], device="cuda")) for x in toks[40:]]
+    check(torch.cat(got), P.forward(ODD, t, toks)[0], "float16")
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
