@@ -161,7 +161,7 @@ def attention_plain(q, k, v, heads, k_dim, v_dim, window=0, scale=1.0, first=Non
     return out
 
 
-LATENT_WIDTHS = (64, 128, 256, 384, 512)      # latent widths of the tensor-core generation kernel
+LATENT_WIDTHS = (64, 128, 192, 256, 320, 384, 512)      # latent widths of the tensor-core generation kernel
 
 
 def pick_latent_nsplit(batch, heads, keys, sm_count=148):
@@ -175,10 +175,12 @@ def pick_latent_nsplit(batch, heads, keys, sm_count=148):
     return 4 if 4 <= want < 8 else (2 if 2 <= want < 4 else (9 if want == 8 else want))
 
 
-def latent_decode(q, cache, rank, heads, window, pos_device, scale, first=None, nsplit=None):
+def latent_decode(q, cache, rank, heads, window, pos_device, scale, first=None, sinks=None, nsplit=None):
     """Generation step over a latent ring cache: q [B, heads*rank] (absorbed queries), cache [B,
-    rows, rank], pos_device int32 scalar (the query's position).  Returns [B, heads*rank]."""
+    rows, rank], pos_device int32 scalar (the query's position); sinks fp32 [heads] or None: exp of it joins the
+    softmax denominator.  Returns [B, heads*rank]."""
     require_cuda(q, cache, pos_device, first)
+    _check_sinks(sinks, heads)
     B = q.shape[0]
     rows = cache.shape[1]
     out = torch.empty((B, heads * rank), dtype=q.dtype, device=q.device)
@@ -186,8 +188,8 @@ def latent_decode(q, cache, rank, heads, window, pos_device, scale, first=None, 
         nsplit = pick_latent_nsplit(B, heads, min(window, rows) if window > 0 else rows)
     nbytes = lib().eb_latent_decode_scratch_bytes(B, heads, rank, nsplit)
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
-    check(lib().eb_latent_decode(ptr(q), q.stride(0), ptr(cache), cache.stride(0), cache.stride(1), rows, ptr(out), out.stride(0), B,
-                                 heads, rank, int(window), ptr(pos_device), ptr(first), float(scale), dtype_code(q.dtype), nsplit,
+    check(lib().eb_latent_decode_sink(ptr(q), q.stride(0), ptr(cache), cache.stride(0), cache.stride(1), rows, ptr(out), out.stride(0), B,
+                                 heads, rank, int(window), ptr(pos_device), ptr(first), ptr(sinks), float(scale), dtype_code(q.dtype), nsplit,
                                  ptr(scratch), nbytes, stream_ptr()), "latent_decode", launches=2 if nbytes else 1)
     return out
 
@@ -341,3 +343,178 @@ def attention_group_decode_chunk(q, k, v, head_dim, pos_device, scale, chunk, si
                                                 dtype_code(q.dtype), nsplit, ptr(scratch), scratch.numel() if scratch is not None else 0,
                                                 stream_ptr()), "attention_group_decode_chunk")
     return out
+
+
+def distance_slopes(heads, device=None):
+    """Slopes of a bias linear in the distance: 2^(-8 (h + 1) / heads) for head h, fp32."""
+    h = torch.arange(1, heads + 1, dtype=torch.float64)
+    return torch.exp2(-8 * h / heads).to(dtype=torch.float32, device=device)
+
+
+def _check_slopes(slopes, heads):
+    require_cuda(slopes)
+    if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != heads or not slopes.is_contiguous()):
+        raise RuntimeError("attention: one fp32 slope per query head")
+
+
+def _check_gate(gate, out):
+    require_cuda(gate)
+    if gate is not None and (gate.shape != out.shape or gate.dtype != out.dtype or gate.stride(-1) != 1):
+        raise RuntimeError("attention: the gate is laid out like the output")
+
+
+def attention_values(k, v, kv_heads, dv_count, eps, k_cache, v_cache, keep, rows_per_batch, pos_device=None, first=None):
+    """Values v [rows, kv_heads*dv] over their head's root mean square, in place, and keys k [rows, kv_heads*dk] and
+    values to a cache [batch, keep + ring rows, ...] (RingCache(keep=...)).  k and v are column views of one
+    projection."""
+    require_cuda(k, v, k_cache, v_cache, pos_device, first)
+    n1 = k.shape[0]
+    if k.stride(1) != 1 or v.stride(1) != 1 or k.stride(0) != v.stride(0) or any(t.dtype != k.dtype for t in (v, k_cache, v_cache)):
+        raise RuntimeError("attention_values: k and v are column ranges of one row layout, caches of their dtype")
+    if n1 % rows_per_batch or k.shape[1] % kv_heads or v.shape[1] % kv_heads:
+        raise RuntimeError("attention_values: whole sequences and whole heads")
+    for t, x in ((k_cache, k), (v_cache, v)):
+        if t.dim() != 3 or t.stride(2) != 1 or t.shape[0] != n1 // rows_per_batch or t.shape[2] != x.shape[1] or t.shape[1] != k_cache.shape[1] or t.shape[1] <= keep:
+            raise RuntimeError("attention_values: caches are [batch, keep + ring rows, kv_heads*dim]")
+    check(lib().eb_attention_values(ptr(k), ptr(v), k.stride(0), kv_heads, k.shape[1] // kv_heads, v.shape[1] // kv_heads, int(dv_count), float(eps),
+                                    ptr(k_cache), k_cache.stride(0), k_cache.stride(1), ptr(v_cache), v_cache.stride(0), v_cache.stride(1), int(keep),
+                                    k_cache.shape[1] - keep, n1, rows_per_batch, ptr(pos_device), ptr(first), dtype_code(k.dtype), stream_ptr()),
+          "attention_values")
+
+
+def sigmoid_gate(y, gate, out=None):
+    """y * sigmoid(gate), rows [n, columns] (row strides allowed)."""
+    out = torch.empty_like(y) if out is None else out
+    require_cuda(y, out)
+    _check_gate(gate, y)
+    if y.dim() != 2 or y.stride(1) != 1 or out.shape != y.shape or out.dtype != y.dtype or out.stride(1) != 1:
+        raise RuntimeError("sigmoid_gate: rows of one dtype")
+    check(lib().eb_sigmoid_gate(ptr(y), y.stride(0), ptr(gate), gate.stride(0), ptr(out), out.stride(0), y.shape[0], y.shape[1], dtype_code(y.dtype),
+                                stream_ptr()), "sigmoid_gate")
+    return out
+
+
+def attention_plain_capped(q, k, v, heads, k_dim, v_dim, window=0, keep=0, kept_rows=0, scale=1.0, first=None, pos_device=None, kv_heads=None, slopes=None,
+                           cap=0.0, sink=False):
+    """attention_plain with a window that keeps the first `keep` positions visible, scores capped by cap * tanh(score / cap)
+    (0: not) and slopes * distance taken off; kept_rows: rows in front of the ring in k / v that hold those
+    positions (keep, or 0: position j is row j mod rows)."""
+    require_cuda(q, k, v, first, pos_device)
+    _check_slopes(slopes, heads)
+    B, Sq, _ = q.shape
+    out = torch.empty((B, Sq, heads * v_dim), dtype=q.dtype, device=q.device)
+    if any(t.stride(2) != 1 for t in (q, k, v)) or k.shape[1] != v.shape[1]:
+        raise RuntimeError("attention: contiguous last dims and one number of key / value rows required")
+    check(lib().eb_attention_plain_capped(ptr(q), ptr(k), ptr(v), ptr(out), q.stride(0), q.stride(1), k_dim, k.stride(0), k.stride(1), k_dim,
+                                          v.stride(0), v.stride(1), v_dim, out.stride(0), out.stride(1), v_dim, B, heads, heads // (kv_heads or heads), Sq,
+                                          k_dim, v_dim, int(window), int(keep), int(kept_rows), k.shape[1] - kept_rows, ptr(pos_device), ptr(first),
+                                          ptr(slopes), float(cap), 1 if sink else 0, float(scale), dtype_code(q.dtype), stream_ptr()), "attention_plain_capped")
+    return out
+
+
+def _prompt_views(q, k, v, k_dim, v_dim, gate, out):
+    require_cuda(q, k, v, out)
+    B, S, H, G = q.shape[0], q.shape[1], q.shape[2] // k_dim, k.shape[2] // k_dim
+    if k.shape[1] != S or v.shape[:2] != k.shape[:2] or v.shape[2] != G * v_dim or H % G:
+        raise RuntimeError("attention: a whole prompt with query heads in equal groups")
+    if out is None:
+        out = torch.empty((B, S, H * v_dim), dtype=q.dtype, device=q.device)
+    _check_gate(gate, out)
+    strides = [x for t, d in ((q, k_dim), (k, k_dim), (v, v_dim), (out, v_dim)) for x in _bsh_strides(t, d)]
+    return B, S, H, G, out, strides + (list(_bsh_strides(gate, v_dim)) if gate is not None else [0, 0])
+
+
+def attention_prefill_gated(q, k, v, k_dim, v_dim, sinks=None, first=None, gate=None, scale=None, out=None):
+    """attention_prefill_chunk without chunks, with value heads of v_dim (64 or k_dim), the output times sigmoid(gate)."""
+    B, S, H, G, out, strides = _prompt_views(q, k, v, k_dim, v_dim, gate, out)
+    require_cuda(first)
+    _check_sinks(sinks, H)
+    scale = k_dim ** -0.5 if scale is None else scale
+    check(lib().eb_attention_prefill_gated_tc(ptr(q), ptr(k), ptr(v), ptr(out), ptr(gate), *strides, B, H, H // G, S, k_dim, v_dim, ptr(first), ptr(sinks),
+                                              float(scale), dtype_code(q.dtype), stream_ptr()), "attention_prefill_gated_tc")
+    return out
+
+
+def attention_prefill_capped(q, k, v, k_dim, v_dim, window=0, keep=0, slopes=None, cap=0.0, sink=True, first=None, gate=None, scale=None, out=None):
+    """Prompt attention (tensor-core kernel) by the rule of attention_plain_capped, the output times sigmoid(gate)."""
+    B, S, H, G, out, strides = _prompt_views(q, k, v, k_dim, v_dim, gate, out)
+    require_cuda(first)
+    _check_slopes(slopes, H)
+    scale = k_dim ** -0.5 if scale is None else scale
+    check(lib().eb_attention_prefill_capped_tc(ptr(q), ptr(k), ptr(v), ptr(out), ptr(gate), *strides, B, H, H // G, S, k_dim, v_dim, int(window), int(keep),
+                                               ptr(first), ptr(slopes), float(cap), 1 if sink else 0, float(scale), dtype_code(q.dtype), stream_ptr()),
+          "attention_prefill_capped_tc")
+    return out
+
+
+def attention_group_decode_capped(q, k, v, head_dim, pos_device, scale, window=0, keep=0, slopes=None, cap=0.0, sink=True, first=None, gate=None, out=None,
+                                  nsplit=None):
+    """Generation step of attention_prefill_capped: q [B, H*D], k / v [B, keep + ring rows, G*D] cache views, pos_device int32
+    scalar (the query's position).  Returns [B, H*D]."""
+    require_cuda(q, k, v, pos_device, first, out)
+    B, HD = q.shape
+    H, G, rows = HD // head_dim, k.shape[2] // head_dim, k.shape[1] - keep
+    _check_slopes(slopes, H)
+    ks, vs = _bsh_strides(k, head_dim), _bsh_strides(v, head_dim)
+    if out is None:
+        out = torch.empty((B, HD), dtype=q.dtype, device=q.device)
+    _check_gate(gate, out)
+    if nsplit is None:
+        nsplit = pick_group_nsplit(B, G * -(-(H // G) // 16), rows + keep)
+    nbytes = lib().eb_attention_group_decode_scratch_bytes(B, H, G, head_dim, nsplit)
+    scratch = _get_scratch(q.device, nbytes) if nbytes else None
+    check(lib().eb_attention_group_decode_capped(ptr(q), ptr(k), ptr(v), ptr(out), ptr(gate), q.stride(0), ks[0], ks[1], vs[0], vs[1], out.stride(0),
+                                                 gate.stride(0) if gate is not None else 0, B, H, G, head_dim, int(keep), rows, int(window),
+                                                 ptr(pos_device), ptr(first), ptr(slopes), float(cap), 1 if sink else 0, float(scale),
+                                                 dtype_code(q.dtype), nsplit, ptr(scratch), scratch.numel() if scratch is not None else 0,
+                                                 stream_ptr()), "attention_group_decode_capped")
+    return out
+
+
+def yarn_rotation(dims, base, scaling=None):
+    """(angle per position of each neighbouring pair, fp32 [dims / 2]; factor of sine and cosine).  scaling (YaRN) =
+    (factor, original, fast, slow): pairs that turn fewer than `slow` times over `original` positions are slowed
+    down by factor, those that turn more than `fast` times are not, with a linear ramp between them."""
+    import math
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    freq = float(base) ** (-2 * i / max(1, dims))
+    if scaling is None:
+        return freq.float(), 1.0
+    factor, original, fast, slow = scaling
+    pair_of = lambda turns: dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(pair_of(fast)), 0), min(math.ceil(pair_of(slow)), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
+    return (freq / factor * ramp + freq * (1 - ramp)).float(), 0.1 * math.log(factor) + 1
+
+
+def latent_inputs(proj, q_cols, q_count, q_norm, eps, row=None, rows_per_batch=1, pos_device=None, first=None):
+    """Rows [query latent | cached row] of a projection -> the normalised query latent [rows, q_cols] and the rows that go to
+    the cache.  row = dict(cols, rot_col, count, norm, freq, factor, ring, keep_rows): the part from rot_col on is
+    turned; ring [batch, rows, cols]; keep_rows: also returns the rows themselves (else None).  None: no latent."""
+    row = row or {}
+    ring, norm, freq = row.get("ring"), row.get("norm"), row.get("freq")
+    require_cuda(proj, q_norm, ring, norm, freq, pos_device, first)
+    n1, cols = proj.shape[0], row.get("cols", 0)
+    if proj.dim() != 2 or proj.stride(1) != 1 or q_norm.numel() != q_cols or any(t is not None and t.dtype != proj.dtype for t in (q_norm, norm, ring)):
+        raise RuntimeError("latent_inputs: rows, norms and cache of one dtype")
+    if ring is not None and (ring.dim() != 3 or ring.stride(2) != 1 or ring.shape[0] * rows_per_batch != n1 or ring.shape[2] < cols or norm.numel() != row["rot_col"]
+                             or freq.dtype != torch.float32 or not freq.is_contiguous()):
+        raise RuntimeError("latent_inputs: the cache is [batch, rows, columns], the norm has an entry per column of the latent")
+    q = torch.empty((n1, q_cols), dtype=proj.dtype, device=proj.device)
+    rows = torch.empty((n1, cols), dtype=proj.dtype, device=proj.device) if row.get("keep_rows") else None
+    check(lib().eb_latent_inputs(ptr(proj), proj.stride(0), q_cols, int(q_count), ptr(q_norm), ptr(q), q_cols, cols, row.get("rot_col", 0),
+                                 int(row.get("count", 0)), ptr(norm), freq.numel() if freq is not None else 0, ptr(freq), float(row.get("factor", 1.0)),
+                                 float(eps), ptr(rows), cols, ptr(ring), ring.stride(0) if ring is not None else 0,
+                                 ring.stride(1) if ring is not None else 0, ring.shape[1] if ring is not None else 0, n1, rows_per_batch, ptr(pos_device),
+                                 ptr(first), dtype_code(proj.dtype), stream_ptr()), "latent_inputs")
+    return q, rows
+
+
+def rotate_heads(x, heads, head_cols, col, freq, factor, rows_per_batch, pos_device=None, first=None):
+    """Turns the pairs from column `col` of every head of rows x, in place."""
+    require_cuda(x, freq, pos_device, first)
+    if x.dim() != 2 or x.stride(1) != 1 or x.shape[1] != heads * head_cols or freq.dtype != torch.float32 or not freq.is_contiguous() or x.shape[0] % rows_per_batch:
+        raise RuntimeError("rotate_heads: rows of whole heads, frequencies in fp32")
+    check(lib().eb_rotate_heads(ptr(x), x.stride(0), heads, head_cols, int(col), freq.numel(), ptr(freq), float(factor), x.shape[0], rows_per_batch,
+                                ptr(pos_device), ptr(first), dtype_code(x.dtype), stream_ptr()), "rotate_heads")
+    return x

@@ -21,7 +21,8 @@ NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", 
               "-diag-suppress", "177,550"]
 # Recurrences add up the logarithms of their gates over a whole sequence: an approximation's bias would
 # add up with them, so these files get the accurate functions; so do angles that grow with the position.
-ACCURATE = {"matrix_memory.cu", "matrix_memory_tc.cu", "decay_memory.cu", "decay_memory_tc.cu", "attention_rotary.cu"}
+ACCURATE = {"matrix_memory.cu", "matrix_memory_tc.cu", "decay_memory.cu", "decay_memory_tc.cu", "attention_rotary.cu", "latent_inputs.cu",
+            "selective_scan.cu"}
 
 
 def nvcc_flags(source):

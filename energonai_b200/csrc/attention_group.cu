@@ -7,6 +7,10 @@
 // A chunk mask (a position sees only its own chunk of so many positions, counted from the sequence's first)
 // goes with a ring cache: position p in row p mod rows.
 //
+// A window may keep the first positions visible; the cache then has rows for them in front of its ring.  With it go
+// capped scores, cap tanh(score / cap), and a bias linear in the distance.  The output may be multiplied by the
+// sigmoid of a gate.
+//
 // Scores: scale q.k - r1 ln(1 + r2 distance), optionally a sink (one more in the denominator, or exp of a
 // number per head), all fp32;
 // an attention weight is rounded once, as an operand of the value product.
@@ -28,15 +32,27 @@ struct GroupParams {
   int group, blocks, cache_rows, nsplit, sink;      // blocks: CTAs of up to 16 heads per group
   const int *pos_dev, *first;
   const float *r1, *r2;
+  int window, keep;                                 // window form: of which the first `keep` cache rows hold the first positions
+  const float *slopes;                              // ... per head, slope * distance is taken off, or null
+  float cap_log2, cap_scale;                        // ... cap * log2(e) and scale / cap, or 0
+  const void *gate;                                 // [B][heads * D] or null
+  long long g_bs;
   float scale_log2;
   float *scratch;                                   // [unit][nsplit][16][D + 2]
   int *counters;
 };
 
+enum { kAll, kChunk, kWindow };                       // what of the past is visible
+
+// tanh by an exponential and a reciprocal: the error of the special function for tanh would be multiplied by the cap
+__device__ __forceinline__ float tanh_exp(float z) { return 1.f - __fdividef(2.f, 1.f + __expf(2.f * z)); }
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
 // WIDE: groups of more than 8 heads; else the second half of the tile's rows is not looked at.
-template <typename T, int D, bool WIDE, bool RING>
+template <typename T, int D, bool WIDE, int FORM>
 __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(const GroupParams p) {
   extern __shared__ __align__(128) uint8_t smem[];
+  constexpr bool RING = FORM == kChunk, WINDOW = FORM == kWindow;
   constexpr int kTileBytes = kTile * D * 2, kLd = D + 2, kHalves = WIDE ? 2 : 1;
   const uint32_t k_s = (uint32_t)__cvta_generic_to_shared(smem), v_s = k_s + kStages * kTileBytes;
   float *red = reinterpret_cast<float *>(smem);     // after the key loop: [4 warps][16][D + 2]
@@ -48,13 +64,17 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   const int split = blockIdx.x, hk = blockIdx.y / p.blocks, hb = blockIdx.y % p.blocks, b = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int h0 = hk * p.group + hb * kRowsPerCta, nh = min(kRowsPerCta, p.group - hb * kRowsPerCta);
-  const int pos = RING ? max(*p.pos_dev, 0) : min(max(*p.pos_dev, 0), p.cache_rows - 1), Sk = pos + 1;
+  const int pos = RING || WINDOW ? max(*p.pos_dev, 0) : min(max(*p.pos_dev, 0), p.cache_rows - 1);
   int lo = p.first ? min(max(p.first[b], 0), pos) : 0;
+  const int start = lo;
+  if (WINDOW) lo = max(p.window > 0 ? max(lo, pos - p.window + 1) : lo, pos - p.cache_rows + 1);
+  // window form: entries are counted, first the kept positions in front of the window, then those of the window
+  const int kept = WINDOW ? min(p.keep, lo - start) : 0, Sk = WINDOW ? kept + pos + 1 - lo : pos + 1;
   if (RING) lo = max(lo + (pos - lo) / p.chunk * p.chunk, pos - p.cache_rows + 1);
   // tile n holds the positions from base + 64 n on
-  const int base = RING ? lo : lo / kTile * kTile, tiles = (Sk - base + kTile - 1) / kTile, per = (tiles + p.nsplit - 1) / p.nsplit;
+  const int base = WINDOW ? 0 : RING ? lo : lo / kTile * kTile, tiles = (Sk - base + kTile - 1) / kTile, per = (tiles + p.nsplit - 1) / p.nsplit;
   const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
-  const int r0 = RING ? base % p.cache_rows : 0;
+  const int r0 = RING ? base % p.cache_rows : WINDOW ? lo % p.cache_rows : 0;
 
   const T *qb = reinterpret_cast<const T *>(p.q) + b * p.q_bs + (long long)h0 * D;
   const T *kb = reinterpret_cast<const T *>(p.k) + b * p.k_bs + hk * D;
@@ -63,6 +83,11 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
     if (RING) {
       load_warp_ring<T, D>(k_s + buf * kTileBytes, kb, p.k_rs, n * kTile, Sk - base, r0, p.cache_rows, warp, lane);
       load_warp_ring<T, D>(v_s + buf * kTileBytes, vb, p.v_rs, n * kTile, Sk - base, r0, p.cache_rows, warp, lane);
+      return;
+    }
+    if (WINDOW) {
+      load_warp_kept<T, D>(k_s + buf * kTileBytes, kb, p.k_rs, n * kTile, Sk, kept, p.keep, r0, p.cache_rows, warp, lane);
+      load_warp_kept<T, D>(v_s + buf * kTileBytes, vb, p.v_rs, n * kTile, Sk, kept, p.keep, r0, p.cache_rows, warp, lane);
       return;
     }
     load_warp_rows<T, D>(k_s + buf * kTileBytes, kb, p.k_rs, base + n * kTile, Sk, warp, lane);
@@ -87,6 +112,11 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
 #pragma unroll
     for (int r = 0; r < 2; ++r)
       if (row_ok[r]) { r1[r] = p.r1[h0 + g + 8 * r]; r2[r] = p.r2[h0 + g + 8 * r]; }
+  }
+  if (WINDOW && p.slopes) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (row_ok[r]) r1[r] = p.slopes[h0 + g + 8 * r] * kLog2eGroup;
   }
   float o[D / 8][4];
 #pragma unroll
@@ -117,8 +147,15 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int j = base + n * kTile + warp * 16 + i * 8 + 2 * t + e;
-          float x = s[i][2 * r + e] * p.scale_log2 - r1[r] * log2f(fmaf(r2[r], (float)max(pos - j, 0), 1.f));
-          if (j > pos || j < lo || !row_ok[r]) x = -INFINITY;
+          float x = s[i][2 * r + e] * p.scale_log2;
+          if (WINDOW) {
+            if (p.cap_scale > 0.f) x = p.cap_log2 * tanh_exp(s[i][2 * r + e] * p.cap_scale);
+            x -= r1[r] * (float)(pos - (j < kept ? start + j : lo + j - kept));
+            if (j >= Sk || !row_ok[r]) x = -INFINITY;
+          } else {
+            x -= r1[r] * log2f(fmaf(r2[r], (float)max(pos - j, 0), 1.f));
+            if (j > pos || j < lo || !row_ok[r]) x = -INFINITY;
+          }
           s[i][2 * r + e] = x;
           mx = fmaxf(mx, x);
         }
@@ -185,6 +222,11 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
     l_out = l;
     return acc;
   };
+  const T *gate = p.gate ? reinterpret_cast<const T *>(p.gate) + b * p.g_bs + (long long)h0 * D : nullptr;
+  auto result = [&](float acc, float l, int i) {
+    const float y = l > 0.f ? acc / l : 0.f;
+    return from_f32<T>(gate ? y * sigmoid_fast(to_f32<T>(gate[i])) : y);
+  };
   T *out = reinterpret_cast<T *>(p.o) + b * p.o_bs + (long long)h0 * D;
   const int unit = b * gridDim.y + blockIdx.y;
   float *slot = p.nsplit > 1 ? p.scratch + ((size_t)unit * p.nsplit + split) * (kRowsPerCta * kLd) : nullptr;
@@ -205,7 +247,7 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
       acc = fmaf(part[d], f, acc);
     }
     if (!slot) {
-      out[row * D + d] = from_f32<T>(l > 0.f ? acc / l : 0.f);
+      out[row * D + d] = result(acc, l, i);
     } else {
       slot[row * kLd + d] = acc;
       if (d == 0) { slot[row * kLd + D] = m; slot[row * kLd + D + 1] = l; }
@@ -225,13 +267,13 @@ __global__ void __launch_bounds__(kGroupThreads) attention_group_decode_kernel(c
   for (int i = threadIdx.x; i < nh * D; i += kGroupThreads) {
     float m, l;
     const float acc = merge(all, p.nsplit, kRowsPerCta * kLd, i / D, i % D, p.sink != 0, m, l);
-    out[i] = from_f32<T>(l > 0.f ? acc / l : 0.f);
+    out[i] = result(acc, l, i);
   }
 }
 
-template <typename T, int D, bool WIDE, bool RING> int launch_group_as(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
+template <typename T, int D, bool WIDE, int FORM> int launch_group_as(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
   constexpr size_t smem = 2 * kStages * (size_t)kTile * D * 2;
-  auto kern = attention_group_decode_kernel<T, D, WIDE, RING>;
+  auto kern = attention_group_decode_kernel<T, D, WIDE, FORM>;
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -246,9 +288,10 @@ template <typename T, int D, bool WIDE, bool RING> int launch_group_as(const Gro
   return check_launch("attention_group_decode");
 }
 
-template <typename T, int D> int launch_group(const GroupParams &p, int kv_heads, int B, cudaStream_t st) {
-  if (p.chunk > 0) return p.group > 8 ? launch_group_as<T, D, true, true>(p, kv_heads, B, st) : launch_group_as<T, D, false, true>(p, kv_heads, B, st);
-  return p.group > 8 ? launch_group_as<T, D, true, false>(p, kv_heads, B, st) : launch_group_as<T, D, false, false>(p, kv_heads, B, st);
+template <typename T, int D> int launch_group(const GroupParams &p, int form, int kv_heads, int B, cudaStream_t st) {
+#define EB_GROUP(FORM) (p.group > 8 ? launch_group_as<T, D, true, FORM>(p, kv_heads, B, st) : launch_group_as<T, D, false, FORM>(p, kv_heads, B, st))
+  return form == kWindow ? EB_GROUP(kWindow) : form == kChunk ? EB_GROUP(kChunk) : EB_GROUP(kAll);
+#undef EB_GROUP
 }
 
 inline int head_blocks(int heads, int kv_heads) { return (heads / kv_heads + kRowsPerCta - 1) / kRowsPerCta; }
@@ -263,12 +306,20 @@ extern "C" size_t eb_attention_group_decode_scratch_bytes(int batch, int heads, 
   return kCounterSlots * sizeof(int) + (size_t)batch * kv_heads * head_blocks(heads, kv_heads) * nsplit * kRowsPerCta * (head_dim + 2) * sizeof(float);
 }
 
+struct GroupWindow {
+  int window, keep;
+  const float *slopes;
+  float cap;
+  const void *gate;
+  long long gate_batch_stride;
+};
+
 static int group_decode_impl(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
                                          long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
                                          long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int cache_rows,
                                          const int32_t *pos_device, const int32_t *first, const float *bias_r1, const float *bias_r2, int sink,
                                          const float *sinks, int chunk, float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes,
-                                         void *stream) {
+                                         void *stream, const GroupWindow *win = nullptr) {
   if (batch == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "attention_group_decode: fp16 or bf16 only (dtype %d)", dtype);
   EB_REQUIRE(head_dim == 64 || head_dim == 128, "attention_group_decode: head_dim %d not supported (64 or 128)", head_dim);
@@ -284,6 +335,12 @@ static int group_decode_impl(const void *q, const void *k, const void *v, void *
   p.v_rs = v_row_stride; p.o_bs = out_batch_stride; p.group = heads / kv_heads; p.blocks = head_blocks(heads, kv_heads);
   p.cache_rows = cache_rows; p.nsplit = nsplit; p.sink = sink; p.sinks = sinks; p.chunk = chunk; p.pos_dev = pos_device; p.first = first; p.r1 = bias_r1; p.r2 = bias_r2;
   p.scale_log2 = scale * kLog2eGroup;
+  if (win) {
+    EB_REQUIRE(win->window >= 0 && win->keep >= 0 && win->cap >= 0.f && (!win->gate || win->gate_batch_stride % 8 == 0), "attention_group_decode: bad window form");
+    p.window = win->window; p.keep = win->keep; p.slopes = win->slopes; p.gate = win->gate; p.g_bs = win->gate_batch_stride;
+    if (win->cap > 0.f) { p.cap_log2 = win->cap * kLog2eGroup; p.cap_scale = scale / win->cap; }
+  }
+  const int form = win ? kWindow : chunk > 0 ? kChunk : kAll;
   EB_REQUIRE((long long)kv_heads * p.blocks <= 65535, "attention_group_decode: too many heads");
   if (nsplit > 1) {
     const size_t need = eb_attention_group_decode_scratch_bytes(batch, heads, kv_heads, head_dim, nsplit);
@@ -293,8 +350,8 @@ static int group_decode_impl(const void *q, const void *k, const void *v, void *
     p.scratch = reinterpret_cast<float *>(reinterpret_cast<char *>(scratch) + kCounterSlots * sizeof(int));
   }
   cudaStream_t st = as_stream(stream);
-  if (dtype == EB_F16) return head_dim == 64 ? launch_group<__half, 64>(p, kv_heads, batch, st) : launch_group<__half, 128>(p, kv_heads, batch, st);
-  return head_dim == 64 ? launch_group<__nv_bfloat16, 64>(p, kv_heads, batch, st) : launch_group<__nv_bfloat16, 128>(p, kv_heads, batch, st);
+  if (dtype == EB_F16) return head_dim == 64 ? launch_group<__half, 64>(p, form, kv_heads, batch, st) : launch_group<__half, 128>(p, form, kv_heads, batch, st);
+  return head_dim == 64 ? launch_group<__nv_bfloat16, 64>(p, form, kv_heads, batch, st) : launch_group<__nv_bfloat16, 128>(p, form, kv_heads, batch, st);
 }
 
 extern "C" int eb_attention_group_decode(const void *q, const void *k, const void *v, void *out, long long q_batch_stride,
@@ -316,4 +373,15 @@ extern "C" int eb_attention_group_decode_chunk(const void *q, const void *k, con
   return group_decode_impl(q, k, v, out, q_batch_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride, out_batch_stride, batch, heads,
                            kv_heads, head_dim, ring_rows, pos_device, first, nullptr, nullptr, sinks ? 1 : 0, sinks, chunk, scale, dtype, nsplit, scratch,
                            scratch_bytes, stream);
+}
+
+extern "C" int eb_attention_group_decode_capped(const void *q, const void *k, const void *v, void *out, const void *gate, long long q_batch_stride,
+                                         long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                                         long long out_batch_stride, long long gate_batch_stride, int batch, int heads, int kv_heads, int head_dim,
+                                         int keep, int ring_rows, int window, const int32_t *pos_device, const int32_t *first, const float *slopes,
+                                         float cap, int sink, float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes, void *stream) {
+  const GroupWindow win{window, keep, slopes, cap, gate, gate_batch_stride};
+  return group_decode_impl(q, k, v, out, q_batch_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride, out_batch_stride, batch, heads,
+                           kv_heads, head_dim, ring_rows, pos_device, first, nullptr, nullptr, sink, nullptr, 0, scale, dtype, nsplit, scratch,
+                           scratch_bytes, stream, &win);
 }

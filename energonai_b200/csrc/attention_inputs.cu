@@ -145,6 +145,89 @@ template <typename T> int launch_inputs(const InputParams &p, int n1, cudaStream
   return check_launch("attention_inputs");
 }
 
+// ---- keys and values for a cache with kept first positions ----
+struct ValueParams {
+  const void *k;
+  void *v;                     // column ranges of rows ld apart; v is normalised in place
+  long long ld;
+  int heads, dk, dv;
+  float inv_count, eps;
+  void *kc, *vc;               // cache row 0: `keep` rows of the first positions, then the ring
+  long long k_bs, k_rs, v_bs, v_rs;
+  int keep, ring_rows, n1, rows_per_batch;
+  const int *pos_dev, *first;
+};
+
+// A warp per (row, key / value head): the value over its root mean square, then key and value to the cache.
+template <typename T>
+__global__ void __launch_bounds__(256) attention_values_kernel(const ValueParams p) {
+  griddep_wait();
+  griddep_launch();
+  constexpr int N = Vec16<T>::N;
+  const int lane = threadIdx.x & 31;
+  const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), row = unit / p.heads;
+  if (row >= p.n1) return;
+  const int h = (int)(unit - row * p.heads);
+  const long long b = row / p.rows_per_batch;
+  const int s = (int)(row - b * p.rows_per_batch), col = (p.pos_dev ? *p.pos_dev : 0) + s, at = col - (p.first ? p.first[b] : 0);
+  const bool in_ring = col >= 0 && p.rows_per_batch - s <= p.ring_rows, kept = at >= 0 && at < p.keep;
+  const long long ring = p.keep + (in_ring ? col % p.ring_rows : 0);
+  T *v = reinterpret_cast<T *>(p.v) + row * p.ld + h * p.dv;
+  T *kc = reinterpret_cast<T *>(p.kc) + b * p.k_bs + h * p.dk, *vc = reinterpret_cast<T *>(p.vc) + b * p.v_bs + h * p.dv;
+  float sq = 0.f;
+  for (int i = lane * N; i < p.dv; i += 32 * N) {
+    Vec16<T> w;
+    float f[N];
+    w.load(v + i);
+    w.unpack(f);
+#pragma unroll
+    for (int e = 0; e < N; ++e) sq = fmaf(f[e], f[e], sq);
+  }
+  const float r = 1.f / sqrtf(warp_sum(sq) * p.inv_count + p.eps);
+  for (int i = lane * N; i < p.dv; i += 32 * N) {
+    Vec16<T> w;
+    float f[N];
+    w.load(v + i);
+    w.unpack(f);
+#pragma unroll
+    for (int e = 0; e < N; ++e) f[e] *= r;
+    w.pack(f);
+    w.store(v + i);
+    if (in_ring) w.store(vc + ring * p.v_rs + i);
+    if (kept) w.store(vc + at * p.v_rs + i);
+  }
+  if (!in_ring && !kept) return;
+  const T *k = reinterpret_cast<const T *>(p.k) + row * p.ld + h * p.dk;
+  for (int i = lane * N; i < p.dk; i += 32 * N) {
+    Vec16<T> w;
+    w.load(k + i);
+    if (in_ring) w.store(kc + ring * p.k_rs + i);
+    if (kept) w.store(kc + at * p.k_rs + i);
+  }
+}
+
+// ---- a gate on the concatenated heads ----
+template <typename T>
+__global__ void __launch_bounds__(256) sigmoid_gate_kernel(const T *y, long long ldy, const T *g, long long ldg, T *out, long long ldo, int n1, int n2) {
+  griddep_wait();
+  griddep_launch();
+  constexpr int N = Vec16<T>::N;
+  const long long per = n2 / N;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n1 * per; i += (long long)gridDim.x * blockDim.x) {
+    const long long row = i / per, c = (i - row * per) * N;
+    Vec16<T> a, b;
+    float fa[N], fb[N];
+    a.load(y + row * ldy + c);
+    b.load(g + row * ldg + c);
+    a.unpack(fa);
+    b.unpack(fb);
+#pragma unroll
+    for (int e = 0; e < N; ++e) fa[e] /= 1.f + expf(-fb[e]);
+    a.pack(fa);
+    a.store(out + row * ldo + c);
+  }
+}
+
 }  // namespace
 }  // namespace eb
 
@@ -180,4 +263,49 @@ extern "C" int eb_attention_inputs(const void *proj, long long ldp, int heads, i
   if (dtype == EB_F32) return launch_inputs<float>(p, n1, st);
   if (dtype == EB_F16) return launch_inputs<__half>(p, n1, st);
   return launch_inputs<__nv_bfloat16>(p, n1, st);
+}
+
+extern "C" int eb_attention_values(const void *k, void *v, long long ld, int kv_heads, int dk, int dv, int dv_count, float eps, void *k_cache,
+                                   long long k_batch_stride, long long k_row_stride, void *v_cache, long long v_batch_stride, long long v_row_stride,
+                                   int keep, int ring_rows, int n1, int rows_per_batch, const int32_t *pos_device, const int32_t *first, int dtype,
+                                   void *stream) {
+  if (n1 == 0) return EB_OK;
+  EB_REQUIRE(dtype_ok(dtype), "attention_values: bad dtype %d", dtype);
+  EB_REQUIRE(k && v && k_cache && v_cache, "attention_values: null pointer");
+  EB_REQUIRE(kv_heads > 0 && dk > 0 && dk % 8 == 0 && dv > 0 && dv % 8 == 0 && dv_count > 0 && dv_count <= dv, "attention_values: head sizes must be multiples of 8 (%d, %d)", dk, dv);
+  EB_REQUIRE(n1 > 0 && rows_per_batch > 0 && n1 % rows_per_batch == 0 && keep >= 0 && ring_rows > 0, "attention_values: bad row counts");
+  const long long strides[] = {ld, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride};
+  for (long long s : strides) EB_REQUIRE(s % 8 == 0, "attention_values: strides must be multiples of 8 elements");
+  EB_REQUIRE(ld >= (long long)kv_heads * dk && ld >= (long long)kv_heads * dv && k_row_stride >= (long long)kv_heads * dk && v_row_stride >= (long long)kv_heads * dv,
+             "attention_values: row strides smaller than the rows they hold");
+  EB_REQUIRE(aligned16(k) && aligned16(v) && aligned16(k_cache) && aligned16(v_cache), "attention_values: pointers must be 16-byte aligned");
+  ValueParams p{};
+  p.k = k; p.v = v; p.ld = ld; p.heads = kv_heads; p.dk = dk; p.dv = dv; p.inv_count = 1.f / (float)dv_count; p.eps = eps; p.kc = k_cache; p.vc = v_cache;
+  p.k_bs = k_batch_stride; p.k_rs = k_row_stride; p.v_bs = v_batch_stride; p.v_rs = v_row_stride; p.keep = keep; p.ring_rows = ring_rows; p.n1 = n1;
+  p.rows_per_batch = rows_per_batch; p.pos_dev = pos_device; p.first = first;
+  cudaStream_t st = as_stream(stream);
+  const long long warps = (long long)n1 * kv_heads, per = warps < 8ll * sm_count() ? 1 : 8;       // few rows: a warp per CTA
+  const dim3 g((unsigned)((warps + per - 1) / per)), t((unsigned)(32 * per));
+  if (dtype == EB_F32) launch_pdl(attention_values_kernel<float>, g, t, 0, st, p);
+  else if (dtype == EB_F16) launch_pdl(attention_values_kernel<__half>, g, t, 0, st, p);
+  else launch_pdl(attention_values_kernel<__nv_bfloat16>, g, t, 0, st, p);
+  return check_launch("attention_values");
+}
+
+extern "C" int eb_sigmoid_gate(const void *y, long long ldy, const void *g, long long ldg, void *out, long long ldo, int n1, int n2, int dtype,
+                               void *stream) {
+  if (n1 == 0) return EB_OK;
+  EB_REQUIRE(dtype_ok(dtype), "sigmoid_gate: bad dtype %d", dtype);
+  EB_REQUIRE(y && g && out && aligned16(y) && aligned16(g) && aligned16(out), "sigmoid_gate: null or misaligned pointer");
+  EB_REQUIRE(n1 > 0 && n2 > 0 && n2 % 8 == 0 && ldy >= n2 && ldg >= n2 && ldo >= n2 && ldy % 8 == 0 && ldg % 8 == 0 && ldo % 8 == 0,
+             "sigmoid_gate: rows of a multiple of 8 columns");
+  cudaStream_t st = as_stream(stream);
+  const long long packs = (long long)n1 * n2 / (dtype == EB_F32 ? 4 : 8), blocks = (packs + 255) / 256;
+  const dim3 grid((unsigned)(blocks < 16ll * sm_count() ? blocks : 16ll * sm_count())), t(256);
+#define EB_GATE(T) launch_pdl(sigmoid_gate_kernel<T>, grid, t, 0, st, (const T *)y, ldy, (const T *)g, ldg, (T *)out, ldo, n1, n2)
+  if (dtype == EB_F32) EB_GATE(float);
+  else if (dtype == EB_F16) EB_GATE(__half);
+  else EB_GATE(__nv_bfloat16);
+#undef EB_GATE
+  return check_launch("sigmoid_gate");
 }

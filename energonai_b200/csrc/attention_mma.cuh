@@ -83,5 +83,23 @@ __device__ __forceinline__ void load_warp_ring(uint32_t tile, const T *base, lon
   }
 }
 
+// The same with `kept` rows in front: entry rel < kept is row rel, the others follow in the ring, which begins at
+// row ring0 (its first wanted row is r0).
+template <typename T, int D>
+__device__ __forceinline__ void load_warp_kept(uint32_t tile, const T *base, long long rs, int rel0, int count, int kept, int ring0, int r0, int R, int warp,
+                                               int lane) {
+  constexpr int kChunks = D / 8, kRowStep = 32 / kChunks, kIters = 16 / kRowStep;
+  const int c = lane % kChunks, rl = lane / kChunks;
+#pragma unroll
+  for (int k = 0; k < kIters; ++k) {
+    const int i = warp * 16 + rl + k * kRowStep, rel = rel0 + i;
+    const bool ok = rel < count;
+    int r = r0 + rel - kept;
+    if (r >= R) r -= R;
+    r = rel < kept ? rel : ring0 + r;
+    cp_async16(tile + tile_off<D>(i, c), ok ? base + (long long)r * rs + c * 8 : base, ok);
+  }
+}
+
 }  // namespace
 }  // namespace eb

@@ -34,6 +34,12 @@
 // padding) do the same with another lower bound, and a number per head may join the softmax as a
 // score without a value.
 //
+// The capped form bounds scores by cap tanh(score / cap) and takes slope * distance off; a window may keep the
+// first positions of a sequence visible, whose key tiles then come first in the walk of both row tiles (they
+// are numbered as if they lay right in front of the window's first tile).  While no score of 32 keys is
+// above 0.35 cap, tanh is its Taylor series (five terms leave 1e-7 of the argument); otherwise it takes an
+// exponential and a reciprocal.  The output may be multiplied by the sigmoid of a gate.
+//
 // Every mbarrier wait is bounded; a wait that runs out is recorded, the CTA's roles leave (each
 // decision made uniform over the warp first), copies in flight are given time to land, TMEM is
 // freed and the kernel returns.
@@ -50,16 +56,17 @@ constexpr int kKeys = 128;                 // keys per tile
 constexpr int kTcThreads = 64 + kTiles * 128;
 
 // Shared-memory plan per head_dim.  With head_dim 128 everything but a second V stage fits.
-template <int D> struct TcSmem {
-  static constexpr uint32_t kQBytes = (D / 64) * kRows * 128, kKBytes = (D / 64) * kKeys * 128, kVBytes = (D / 64) * kKeys * 128,
+template <int D, int DV> struct TcSmem {
+  static constexpr uint32_t kQBytes = (D / 64) * kRows * 128, kKBytes = (D / 64) * kKeys * 128, kVBytes = (DV / 64) * kKeys * 128,
                             kPBytes = 2 * kRows * 128;
-  static constexpr int kVStages = D > 64 ? 1 : 2;
+  static constexpr int kVStages = DV > 64 ? 1 : 2;
   static constexpr size_t kTotal = 1024 + 1024 + (size_t)kTiles * kQBytes + 2 * kKBytes + (size_t)kVStages * kVBytes + (size_t)kTiles * kPBytes;
 };
 constexpr float kLog2eTc = 1.4426950408889634f;
 // From this distance on r1 log2(1 + r2 d) is interpolated between d, d - 16 and d - 32: the third derivative
 // is at most 2 r1 / (ln 2 d^3), so the parabola is off by less than 1e-5 r1.
 constexpr int kFarKeys = 512;
+constexpr float kSmallTanh = 0.35f;        // below this argument the capped form takes the series
 constexpr float kRescaleLog2 = 8.f;         // the accumulated row is rescaled when its maximum grows by more than 2^8
 
 struct TcParams {
@@ -72,6 +79,11 @@ struct TcParams {
   const float *sinks;                      // plain form: per head, a score without a value (null: none)
   int chunk;                               // > 0: row i sees only the keys of its chunk, counted from `first`
   const int *first;                        // [B] padding rows in front of each sequence (they see themselves), or null
+  int keep;                                // capped form: so many positions from `first` on stay visible behind the window
+  const float *slopes;                     // ... slopes[h] * distance is taken off, or null
+  float cap_log2, cap_scale;               // ... cap * log2(e) and scale / cap (0: no cap)
+  const void *gate;                        // output times sigmoid(gate), laid out like it with strides of its own, or null
+  long long g_bs, g_rs;
   int mask_vec;                            // mask rows start on 16-byte boundaries
   float scale_log2;                        // scale * log2(e)
   const void *mask;                        // additive [B][>= Sk] in T, or null
@@ -84,17 +96,30 @@ struct TcParams {
 // Shared memory (1024-aligned): [1 KB barriers, TMEM slot, abort flag][Q: 2 row tiles x D/64
 // sub-tiles of 128 rows x 128 B][K ring: 2 x D/64 sub-tiles][V ring: kVStages x D/64 sub-tiles
 // of 128 key rows x 128 B][P: 2 row tiles x 2 sub-tiles of 128 rows x 128 B].
-template <typename T, int D, bool BIAS>
+enum { kFormPlain, kFormBias, kFormCapped };
+
+// tanh(z) / z for |z| <= kSmallTanh, two at a time, w = z^2
+__device__ __forceinline__ void tanh_series(float &p0, float &p1, float w0, float w1) {
+  constexpr float c4 = 62.f / 2835.f, c3 = -17.f / 315.f, c2 = 2.f / 15.f, c1 = -1.f / 3.f;
+  fma2(p0, p1, w0, w1, c4, c4, c3, c3);
+  fma2(p0, p1, p0, p1, w0, w1, c2, c2);
+  fma2(p0, p1, p0, p1, w0, w1, c1, c1);
+  fma2(p0, p1, p0, p1, w0, w1, 1.f, 1.f);
+}
+__device__ __forceinline__ float tanh_exp(float z) { return 1.f - __fdividef(2.f, 1.f + ex2(z * (2.f * kLog2eTc))); }
+
+template <typename T, int D, int DV, int FORM>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                             const __grid_constant__ CUtensorMap tm_v, const TcParams p) {
-  constexpr int kSub = D / 64;                                   // 64-column sub-tiles of Q / K
-  constexpr int kVStages = TcSmem<D>::kVStages;
-  constexpr uint32_t kQBytes = TcSmem<D>::kQBytes, kKBytes = TcSmem<D>::kKBytes, kVBytes = TcSmem<D>::kVBytes,
-                     kPBytes = TcSmem<D>::kPBytes;
+  constexpr bool BIAS = FORM == kFormBias, CAPPED = FORM == kFormCapped;
+  constexpr int kSub = D / 64, kSubV = DV / 64;                  // 64-column sub-tiles of Q / K and V
+  using Smem = TcSmem<D, DV>;
+  constexpr int kVStages = Smem::kVStages;
+  constexpr uint32_t kQBytes = Smem::kQBytes, kKBytes = Smem::kKBytes, kVBytes = Smem::kVBytes, kPBytes = Smem::kPBytes;
   constexpr uint32_t kTmemCols = 512, kPvCol = 2 * kKeys;
   constexpr int kBf16 = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
-  constexpr uint32_t kIdescS = tc_idesc(kKeys, kBf16), kIdescPV = tc_idesc(D, kBf16) | (1u << 16);   // bit 16: B is N-major
+  constexpr uint32_t kIdescS = tc_idesc(kKeys, kBf16), kIdescPV = tc_idesc(DV, kBf16) | (1u << 16);   // bit 16: B is N-major
 
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = s32(smem_raw);
@@ -117,8 +142,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   const int first = p.first ? p.first[b] : 0;
   // first key that the row at position i sees
   auto seen_from = [&](int i) {
-    if (p.window > 0) return i - p.window + 1;
+    if (!CAPPED && p.window > 0) return i - p.window + 1;
     const int f = min(first, max(i, 0));
+    if (CAPPED) return p.window > 0 ? max(f, i - p.window + 1) : f;
     return p.chunk > 0 && i > f ? f + (i - f) / p.chunk * p.chunk : f;
   };
   // key tiles each row tile walks: all of them, or up to its last row's diagonal; none for a
@@ -136,6 +162,16 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     nmax = max(nmax, nt[t]);
   }
   if (jmin > nmax) jmin = nmax;
+  // tiles with kept positions in front of the window, numbered [jmin, jwin)
+  const int jwin = jmin, kept_tile = first / kKeys;
+  if (CAPPED && p.keep > 0 && p.window > 0 && nmax > 0) {
+    const int kept = min((min(first + p.keep, p.Sk) - 1) / kKeys + 1, jmin) - kept_tile;
+    if (kept > 0) {
+      jmin -= kept;
+      ks[0] = ks[1] = jmin;
+    }
+  }
+  auto tile_of = [&](int j) { return CAPPED && j < jwin ? kept_tile + j - jmin : j; };
 
   if (threadIdx.x == 0) {
     asm volatile("prefetch.tensormap [%0];" ::"l"(&tm_q) : "memory");
@@ -183,7 +219,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         bar_expect_tx(k_full + 8 * st, kKBytes);
 #pragma unroll
         for (int kb = 0; kb < kSub; ++kb)
-          tma_load_3d(k_addr + st * kKBytes + kb * kKeys * 128, &tm_k, k_full + 8 * st, hk * D + kb * 64, j * kKeys, b);
+          tma_load_3d(k_addr + st * kKBytes + kb * kKeys * 128, &tm_k, k_full + 8 * st, hk * D + kb * 64, tile_of(j) * kKeys, b);
         return true;
       };
       bool ok = load_k(jmin);
@@ -193,8 +229,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         if (i >= kVStages && !bar_wait(v_empty + 8 * vs, (vu - 1) & 1, abort_flag, 9)) break;
         bar_expect_tx(v_full + 8 * vs, kVBytes);
 #pragma unroll
-        for (int kb = 0; kb < kSub; ++kb)
-          tma_load_3d(v_addr + vs * kVBytes + kb * kKeys * 128, &tm_v, v_full + 8 * vs, hk * D + kb * 64, j * kKeys, b);
+        for (int kb = 0; kb < kSubV; ++kb)
+          tma_load_3d(v_addr + vs * kVBytes + kb * kKeys * 128, &tm_v, v_full + 8 * vs, hk * DV + kb * 64, tile_of(j) * kKeys, b);
       }
     }
   } else if (warp == 1) {
@@ -257,9 +293,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     uint8_t *p_row = p_ptr + t * kPBytes + row * 128;
     const T *mrow = p.mask ? reinterpret_cast<const T *>(p.mask) + (long long)b * p.mask_bs : nullptr;
     const int vis_end = p.causal ? min(p.Sk, qi + shift + 1) : p.Sk;               // keys [0, vis_end) are visible to this row
-    const int vis_begin = seen_from(qi + shift);                                   // ... from this key on
+    const int vis_begin = CAPPED ? max(first, seen_from(qi + shift)) : seen_from(qi + shift);      // ... from this key on
+    const int kept_end = CAPPED ? first + p.keep : 0;                              // (capped: and [first, kept_end))
     // m_ref: the maximum the accumulated row and l_run are scaled by (a sink is a score of 0 seen already)
-    float m_ref = BIAS && p.sink ? 0.f : -1e30f, l_run = BIAS && p.sink ? 1.f : 0.f;
+    const bool zero_sink = (BIAS || CAPPED) && p.sink;
+    float m_ref = zero_sink ? 0.f : -1e30f, l_run = zero_sink ? 1.f : 0.f;
     if (!BIAS && p.sinks) {
       m_ref = p.sinks[h] * kLog2eTc;
       l_run = 1.f;
@@ -269,9 +307,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     // whole range.  fp16 does not, and a negative r1 raises scores: there the maximum includes it.
     const float *bias = BIAS ? p.bias + (long long)h * p.bias_ld : nullptr;
     const bool bias_in_max = BIAS && (!kBf16 || bias[1] < 0.f);
+    const float slope = CAPPED && p.slopes ? p.slopes[h] * kLog2eTc : 0.f;
+    // capped score of a raw product without the bias, in the log2 domain
+    auto capped = [&](float x) { return p.cap_scale > 0.f ? p.cap_log2 * tanh_exp(x * p.cap_scale) : x * p.scale_log2; };
     bool alive = ntiles > 0;
     for (int j = first_tile; j < ntiles && alive; ++j) {
-      const int key0 = j * kKeys;
+      const int key0 = tile_of(j) * kKeys;
       // Work per chunk of 32 keys, decided for the warp as a whole (tensor-memory loads are
       // warp-wide): 0 = hidden from every row of the warp (behind the diagonal or the end of the
       // sequence): nothing to read, P = 0; 1 = visible to every row and no mask value set: one
@@ -282,17 +323,18 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
       // which was the largest stall.  So it packs the classes and reads mask values again.)
       int cls[kKeys / 32];
       float mval[kKeys / 32];
-      uint32_t classes = 0;
+      uint32_t classes = 0, small = 0;              // (small: bit c, the series serves chunk c)
 #pragma unroll
       for (int c = 0; c < kKeys / 32; ++c) {
         const int kb = key0 + c * 32;
         float mv = 0.f;
         if (mrow && kb + lane < p.Sk) mv = to_f32<T>(mrow[kb + lane]) * kLog2eTc;
         mval[c] = mv;
-        const bool hidden = __all_sync(0xffffffffu, kb >= vis_end || kb + 32 <= vis_begin);
-        const bool simple = __all_sync(0xffffffffu, kb >= vis_begin && kb + 32 <= vis_end && mv == 0.f);
+        const bool unkept = !CAPPED || kb >= kept_end || kb + 32 <= first, kept = CAPPED && kb >= first && kb + 32 <= min(kept_end, vis_end);
+        const bool hidden = __all_sync(0xffffffffu, kb >= vis_end || (kb + 32 <= vis_begin && unkept));
+        const bool simple = __all_sync(0xffffffffu, ((kb >= vis_begin && kb + 32 <= vis_end) || kept) && mv == 0.f);
         cls[c] = hidden ? 0 : (simple ? 1 : 2);
-        if (BIAS) classes |= (uint32_t)cls[c] << (2 * c);
+        if (BIAS || CAPPED) classes |= (uint32_t)cls[c] << (2 * c);
       }
       auto mask_value = [&](int c) { return mrow && key0 + c * 32 + lane < p.Sk ? to_f32<T>(mrow[key0 + c * 32 + lane]) * kLog2eTc : 0.f; };
       if (!__all_sync(0xffffffffu, bar_wait(my_s_full, (j - first_tile) & 1, abort_flag, 7))) { alive = false; break; }
@@ -325,7 +367,40 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           }
         }
       };
-      if constexpr (BIAS) {
+      // the largest capped score of a chunk, less the bias of its nearest key: an upper bound that is at most 31 slopes
+      // (or, with the series, twice its range) too high, which the range of bf16 and fp32 takes
+      auto visible = [&](int key) { return key < vis_end && (key >= vis_begin || (key >= first && key < kept_end)); };
+      auto bound = [&](int c, int kind) {
+        if (kind == 0) return;
+        float x[32], top = -INFINITY, big = 0.f;
+        tc_ld32(t_s + c * 32, x);
+        const int kb = key0 + c * 32;
+        if (kind == 1) {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) big = fmaxf(big, fabsf(x[e]));
+          if (__all_sync(0xffffffffu, big * p.cap_scale <= kSmallTanh)) {
+            small |= 1u << c;
+            top = big;
+          } else {
+#pragma unroll
+            for (int e = 0; e < 32; ++e) top = fmaxf(top, x[e]);
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < 32; ++e) top = fmaxf(top, visible(kb + e) ? x[e] : -INFINITY);
+        }
+        if (kBf16) {
+          if (top > -INFINITY) m_tile = fmaxf(m_tile, ((small >> c) & 1 ? top * p.scale_log2 : capped(top)) - slope * (float)max(0, qi + shift - kb - 31));
+        } else {
+#pragma unroll
+          for (int e = 0; e < 32; ++e)
+            if (kind == 1 || visible(kb + e)) m_tile = fmaxf(m_tile, capped(x[e]) - slope * (float)(qi + shift - kb - e));
+        }
+      };
+      if constexpr (CAPPED) {
+#pragma unroll 1
+        for (int c = 0; c < kKeys / 32; ++c) bound(c, (classes >> (2 * c)) & 3);
+      } else if constexpr (BIAS) {
 #pragma unroll 1
         for (int c = 0; c < kKeys / 32; ++c) maximum(c, (classes >> (2 * c)) & 3, mask_value(c));
       } else {
@@ -348,7 +423,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         if (j > first_tile) {
           tc_fence_after();
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             float x[32];
             tc_ld32(t_pv + c * 32, x);
 #pragma unroll
@@ -371,7 +446,30 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
         float x[32];
         tc_ld32(t_s + c * 32, x);
         const int gap = qi + shift - (key0 + c * 32);
-        if (kind == 1 && BIAS) {
+        if (CAPPED) {
+          const int kb = key0 + c * 32;
+          const float base = neg_m - slope * (float)(qi + shift - kb);
+          if ((small >> c) & 1) {
+#pragma unroll
+            for (int e = 0; e < 32; e += 2) {
+              float z0, z1, p0, p1, b0, b1;
+              mul2(z0, z1, x[e], x[e + 1], p.cap_scale, p.cap_scale);
+              mul2(z0, z1, z0, z1, z0, z1);
+              tanh_series(p0, p1, z0, z1);
+              mul2(x[e], x[e + 1], x[e], x[e + 1], p.scale_log2, p.scale_log2);
+              fma2(b0, b1, (float)e, (float)(e + 1), slope, slope, base, base);
+              fma2(x[e], x[e + 1], x[e], x[e + 1], p0, p1, b0, b1);
+            }
+#pragma unroll
+            for (int e = 0; e < 32; ++e) x[e] = ex2(x[e]);
+          } else {
+#pragma unroll
+            for (int e = 0; e < 32; ++e) {
+              const float v = ex2(capped(x[e]) + fmaf((float)e, slope, base));
+              x[e] = kind == 1 || visible(kb + e) ? v : 0.f;
+            }
+          }
+        } else if (kind == 1 && BIAS) {
           // far from the diagonal the bias of a chunk's 32 keys is a parabola through three of them
           if (q0 + t * kRows + quarter * 32 + shift - (key0 + c * 32) - 32 >= kFarKeys) {
             const float b0 = __ldg(bias + gap), b1 = __ldg(bias + gap - 16), b2 = __ldg(bias + gap - 32);
@@ -420,7 +518,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
           *reinterpret_cast<uint4 *>(dst + ((((c & 1) * 4 + g) ^ (row & 7)) << 4)) = w;
         }
       };
-      if constexpr (BIAS) {
+      if constexpr (BIAS || CAPPED) {
 #pragma unroll 1
         for (int c = 0; c < kKeys / 32; ++c) weights(c, (classes >> (2 * c)) & 3, mask_value(c));
       } else {
@@ -439,12 +537,24 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
     if (alive) {
       tc_fence_after();
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      T *orow = reinterpret_cast<T *>(p.o) + (long long)b * p.o_bs + (long long)qi * p.o_rs + h * D;
+      T *orow = reinterpret_cast<T *>(p.o) + (long long)b * p.o_bs + (long long)qi * p.o_rs + h * DV;
+      const T *grow = p.gate ? reinterpret_cast<const T *>(p.gate) + (long long)b * p.g_bs + (long long)qi * p.g_rs + h * DV : nullptr;
 #pragma unroll 1
-      for (int c = 0; c < D / 32; ++c) {
+      for (int c = 0; c < DV / 32; ++c) {
         float x[32];
         tc_ld32(t_pv + c * 32, x);                 // warp-wide: rows behind the end of the sequence read too, and store nothing
         if (qi < p.Sq) {
+          if (grow) {
+#pragma unroll
+            for (int g = 0; g < 4; ++g) {
+              Vec16<T> w;
+              float f[8];
+              w.load(grow + c * 32 + g * 8);
+              w.unpack(f);
+#pragma unroll
+              for (int e = 0; e < 8; ++e) x[g * 8 + e] = __fdividef(x[g * 8 + e], 1.f + ex2(-f[e] * kLog2eTc));
+            }
+          }
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
             uint4 w;
@@ -483,10 +593,10 @@ __global__ void distance_bias_kernel(const float *r1, const float *r2, int len, 
   if (d < len) out[(long long)h * len + d] = r1[h] * log2f(fmaf(r2[h], (float)d, 1.f));
 }
 
-template <typename T, int D, bool BIAS>
+template <typename T, int D, int DV, int FORM>
 int launch_tc(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const TcParams &p, cudaStream_t st) {
-  constexpr size_t smem = TcSmem<D>::kTotal;
-  auto kern = attention_prefill_tc_kernel<T, D, BIAS>;
+  constexpr size_t smem = TcSmem<D, DV>::kTotal;
+  auto kern = attention_prefill_tc_kernel<T, D, DV, FORM>;
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -511,16 +621,26 @@ int attention_tc_status(int *out4, bool clear) { return tc_status(out4, clear); 
 
 using namespace eb;
 
+struct TcCapped {
+  int keep;
+  const float *slopes;
+  float cap;
+};
+
 static int prefill_tc_impl(const void *q, const void *k, const void *v, void *out, const void *mask,
                                        long long q_batch_stride, long long q_row_stride, long long k_batch_stride,
                                        long long k_row_stride, long long v_batch_stride, long long v_row_stride,
                                        long long o_batch_stride, long long o_row_stride, long long mask_batch_stride, int batch,
                                        int heads, int q_len, int kv_len, int head_dim, int causal, int window, float scale,
                                        int dtype, void *stream, int kv_group = 1, const float *bias = nullptr, long long bias_ld = 0,
-                                       int sink = 0, const float *sinks = nullptr, int chunk = 0, const int32_t *first = nullptr) {
+                                       int sink = 0, const float *sinks = nullptr, int chunk = 0, const int32_t *first = nullptr,
+                                       int v_dim = 0, const TcCapped *capped = nullptr, const void *gate = nullptr, long long g_batch_stride = 0,
+                                       long long g_row_stride = 0) {
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "attention_prefill: fp16 or bf16 only (dtype %d)", dtype);
+  if (v_dim == 0) v_dim = head_dim;
   EB_REQUIRE(head_dim == 64 || head_dim == 128, "attention_prefill: head_dim %d not supported (64 or 128)", head_dim);
+  EB_REQUIRE(v_dim == head_dim || (v_dim == 64 && !bias), "attention_prefill: value heads of %d not supported (64 or as the keys)", v_dim);
   EB_REQUIRE(batch > 0 && heads > 0 && q_len > 0 && kv_len > 0, "attention_prefill: negative or zero size");
   EB_REQUIRE(heads <= 65535 && batch <= 65535, "attention_prefill: batch and heads are limited to 65535");
   EB_REQUIRE(q && k && v && out, "attention_prefill: null pointer");
@@ -532,10 +652,11 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   EB_REQUIRE(scale > 0.f, "attention_prefill: the scale must be positive");
   EB_REQUIRE(window >= 0 && (window == 0 || causal), "attention_prefill: a window needs the causal mask");
   cudaStream_t st = as_stream(stream);
-  const long long hd = (long long)heads * head_dim, hkd = hd / kv_group;
+  EB_REQUIRE(!gate || (aligned16(gate) && g_batch_stride % 8 == 0 && g_row_stride % 8 == 0), "attention_prefill: the gate's rows start on 16-byte boundaries");
+  const long long hd = (long long)heads * head_dim, hkd = hd / kv_group, hvd = (long long)heads / kv_group * v_dim;
   CUtensorMap mq, mk, mv;
   int rc;
-  if ((rc = tc_map3(&mv, v, dtype, hkd, kv_len, batch, v_row_stride, v_batch_stride, kKeys))) return rc;
+  if ((rc = tc_map3(&mv, v, dtype, hvd, kv_len, batch, v_row_stride, v_batch_stride, kKeys))) return rc;
   if ((rc = tc_map3(&mq, q, dtype, hd, q_len, batch, q_row_stride, q_batch_stride, kRows))) return rc;
   if ((rc = tc_map3(&mk, k, dtype, hkd, kv_len, batch, k_row_stride, k_batch_stride, kKeys))) return rc;
   TcParams p{};
@@ -546,9 +667,18 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   p.o = out; p.o_bs = o_batch_stride; p.o_rs = o_row_stride;
   p.group = kv_group; p.bias = bias; p.bias_ld = bias_ld; p.sink = sink;
   p.sinks = sinks; p.chunk = chunk; p.first = first;
-#define EB_TC(T, D) (bias ? launch_tc<T, D, true>(mq, mk, mv, p, st) : launch_tc<T, D, false>(mq, mk, mv, p, st))
-  if (dtype == EB_F16) return head_dim == 64 ? EB_TC(__half, 64) : EB_TC(__half, 128);
-  return head_dim == 64 ? EB_TC(__nv_bfloat16, 64) : EB_TC(__nv_bfloat16, 128);
+  p.gate = gate; p.g_bs = g_batch_stride; p.g_rs = g_row_stride;
+  if (capped) {
+    EB_REQUIRE(capped->keep >= 0 && capped->cap >= 0.f && !mask && !bias && !chunk, "attention_prefill: bad capped form");
+    p.keep = capped->keep; p.slopes = capped->slopes;
+    p.cap_log2 = capped->cap * kLog2eTc; p.cap_scale = capped->cap > 0.f ? scale / capped->cap : 0.f;
+  }
+#define EB_TC(T, D, DV) (capped ? launch_tc<T, D, DV, kFormCapped>(mq, mk, mv, p, st) : launch_tc<T, D, DV, kFormPlain>(mq, mk, mv, p, st))
+#define EB_TC_B(T, D) (bias ? launch_tc<T, D, D, kFormBias>(mq, mk, mv, p, st) : EB_TC(T, D, D))
+  if (v_dim != head_dim) return dtype == EB_F16 ? EB_TC(__half, 128, 64) : EB_TC(__nv_bfloat16, 128, 64);
+  if (dtype == EB_F16) return head_dim == 64 ? EB_TC_B(__half, 64) : EB_TC_B(__half, 128);
+  return head_dim == 64 ? EB_TC_B(__nv_bfloat16, 64) : EB_TC_B(__nv_bfloat16, 128);
+#undef EB_TC_B
 #undef EB_TC
 }
 
@@ -605,4 +735,28 @@ extern "C" int eb_attention_prefill_chunk_tc(const void *q, const void *k, const
   return prefill_tc_impl(q, k, v, out, nullptr, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
                          o_batch_stride, o_row_stride, 0, batch, heads, len, len, head_dim, 1, 0, scale, dtype, stream, kv_group, nullptr, 0, 0,
                          sinks, chunk, first);
+}
+
+extern "C" int eb_attention_prefill_gated_tc(const void *q, const void *k, const void *v, void *out, const void *gate, long long q_batch_stride,
+                                       long long q_row_stride, long long k_batch_stride, long long k_row_stride, long long v_batch_stride,
+                                       long long v_row_stride, long long o_batch_stride, long long o_row_stride, long long g_batch_stride,
+                                       long long g_row_stride, int batch, int heads, int kv_group, int len, int k_dim, int v_dim,
+                                       const int32_t *first, const float *sinks, float scale, int dtype, void *stream) {
+  EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_prefill: %d heads do not share keys in groups of %d", heads, kv_group);
+  return prefill_tc_impl(q, k, v, out, nullptr, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
+                         o_batch_stride, o_row_stride, 0, batch, heads, len, len, k_dim, 1, 0, scale, dtype, stream, kv_group, nullptr, 0, 0,
+                         sinks, 0, first, v_dim, nullptr, gate, g_batch_stride, g_row_stride);
+}
+
+extern "C" int eb_attention_prefill_capped_tc(const void *q, const void *k, const void *v, void *out, const void *gate, long long q_batch_stride,
+                                       long long q_row_stride, long long k_batch_stride, long long k_row_stride, long long v_batch_stride,
+                                       long long v_row_stride, long long o_batch_stride, long long o_row_stride, long long g_batch_stride,
+                                       long long g_row_stride, int batch, int heads, int kv_group, int len, int k_dim, int v_dim, int window,
+                                       int keep, const int32_t *first, const float *slopes, float cap, int sink, float scale, int dtype,
+                                       void *stream) {
+  EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_prefill: %d heads do not share keys in groups of %d", heads, kv_group);
+  const TcCapped capped{keep, slopes, cap};
+  return prefill_tc_impl(q, k, v, out, nullptr, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
+                         o_batch_stride, o_row_stride, 0, batch, heads, len, len, k_dim, 1, window, scale, dtype, stream, kv_group, nullptr, 0, sink,
+                         nullptr, 0, first, v_dim, &capped, gate, g_batch_stride, g_row_stride);
 }

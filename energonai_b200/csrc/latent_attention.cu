@@ -52,6 +52,7 @@ struct LatentParams {
   const int *pos_dev;          // position of the query, the same for every sequence
   const int *first;            // [B] first position of each sequence, or null
   float scale_log2;
+  const float *sinks;          // per head: exp of it joins the softmax denominator, or null
   float *part_o;               // [B][heads][nsplit][R]; null: the splits are a cluster
   float *part_ml;              // [B][heads][nsplit][2]
 };
@@ -238,6 +239,18 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const LatentParam
   float m_run[MT][2], l_run[2] = {0.f, 0.f};
 #pragma unroll
   for (int m = 0; m < MT; ++m) m_run[m][0] = m_run[m][1] = -1e30f;
+  if (p.sinks && split == 0) {                      // a score that every head has seen already; one thread per row counts it
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int h = h0 + m * 16 + g + e * 8;
+        if (h < p.heads) {
+          m_run[m][e] = p.sinks[h] * kLog2eLat;
+          if (m == mt && kg == 0 && tq == 0) l_run[e] = 1.f;
+        }
+      }
+  }
   const int key_w = kg * 8 * kNT;
   // A wait that ran out is not acted on before the end: the barriers below stay matched, the
   // remaining waits are skipped, the result is unspecified and the status word says so.
@@ -346,13 +359,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_c, const LatentParam
       for (int n = 0; n < kON; n += 2) {
         uint32_t vf[4];
         // 16 keys x 16 columns: matrices (keys 0-7, cols 0-7), (8-15, 0-7), (0-7, 8-15), (8-15, 8-15);
-        // with one 8-column tile per warp the upper half of the lanes repeats the lower's rows
-        const int ch = kON >= 2 ? warp * kON + n + (lane >> 4) : warp;
+        // for the last of an odd number of 8-column tiles the upper half of the lanes repeats the lower's rows
+        const int ch = kON >= 2 ? warp * kON + min(n + (lane >> 4), kON - 1) : warp;
         lat_ldm4t(vf, cs + lat_tile_off(k * 16 + (lane & 15), ch, kSubBytes));
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
           lat_mma<T>(acc[m][n], pf[m], vf[0], vf[1]);
-          if (kON >= 2) lat_mma<T>(acc[m][n + (kON >= 2 ? 1 : 0)], pf[m], vf[2], vf[3]);
+          if (n + 1 < kON) lat_mma<T>(acc[m][n + 1 < kON ? n + 1 : n], pf[m], vf[2], vf[3]);
         }
       }
     }
@@ -565,7 +578,9 @@ template <typename T> int launch_latent_r(const CUtensorMap &map, const LatentPa
   switch (R) {
     case 64: return launch_latent_mt<T, 64>(map, p, B, st);
     case 128: return launch_latent_mt<T, 128>(map, p, B, st);
+    case 192: return launch_latent_mt<T, 192>(map, p, B, st);
     case 256: return launch_latent_mt<T, 256>(map, p, B, st);
+    case 320: return launch_latent_mt<T, 320>(map, p, B, st);
     case 384: return launch_latent_mt<T, 384>(map, p, B, st);
     default: return launch_latent_mt<T, 512>(map, p, B, st);
   }
@@ -585,7 +600,18 @@ struct PlainParams {
   int sink;                    // one is added to the softmax denominator
   const float *sinks;          // per head: exp of it is (instead of one)
   int chunk;                   // > 0: a position sees only its own chunk of so many, counted from first
+  int keep, kept_rows;         // the first `keep` positions stay visible; cache rows in front of the ring that hold them
+  const float *slopes;         // per head: slope * distance is taken off the score, or null
+  float cap_log2, inv_cap;     // score <- cap tanh(score / cap), or inv_cap 0
 };
+
+// tanh of a score over its cap: of 32-bit models by the library (not the approximation that fast math puts in its
+// place, whose error the cap would multiply)
+template <typename T> __device__ __forceinline__ float capped_tanh(float x) { return 1.f - __fdividef(2.f, 1.f + __expf(2.f * x)); }
+template <> __device__ __forceinline__ float capped_tanh<float>(float x) {
+  const float a = fabsf(x), e = expm1f(-2.f * a);
+  return copysignf(__fdiv_rn(-e, 2.f + e), x);
+}
 
 template <typename T>
 __global__ void attention_plain_kernel(const PlainParams p) {
@@ -605,28 +631,37 @@ __global__ void attention_plain_kernel(const PlainParams p) {
   if (p.window > 0) lo = max(lo, pos - p.window + 1);
   if (p.chunk > 0 && pos > lo) lo += (pos - lo) / p.chunk * p.chunk;
   lo = max(lo, max(0, pos - p.ring_rows + 1));
+  const int start = p.first ? min(p.first[b], lo) : 0, kept = min(p.keep, lo - start), count = kept + pos + 1 - lo;
+  // entry n of what is visible: its position, and its row
+  auto position = [&](int n) { return n < kept ? start + n : lo + n - kept; };
+  auto row_of = [&](int n) {
+    if (n < kept && p.kept_rows > 0) return (long long)n;
+    return (long long)(p.kept_rows + position(n) % p.ring_rows);
+  };
   const T *K = reinterpret_cast<const T *>(p.k) + b * p.k_bs + h / p.group * p.k_hs, *V = reinterpret_cast<const T *>(p.v) + b * p.v_bs + h / p.group * p.v_hs;
-  const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f;
+  const float r1 = p.r1 ? p.r1[h] : 0.f, r2 = p.r1 ? p.r2[h] : 0.f, slope = p.slopes ? p.slopes[h] * kLog2eLat : 0.f;
   float m = p.sinks ? p.sinks[h] * kLog2eLat : p.sink ? 0.f : -1e30f, l = p.sinks || p.sink ? 1.f : 0.f;      // the sink: a score without a value
-  for (int j0 = lo; j0 <= pos; j0 += 32) {
-    const int j = j0 + lane;
+  for (int n0 = 0; n0 < count; n0 += 32) {
     float s = -INFINITY;
-    if (j <= pos) {
-      const T *kr = K + (long long)(j % p.ring_rows) * p.k_rs;
+    if (n0 + lane < count) {
+      const int j = position(n0 + lane);
+      const T *kr = K + row_of(n0 + lane) * p.k_rs;
       float a = 0.f;
       for (int d = 0; d < p.dk; ++d) a = fmaf(sq[d], to_f32<T>(kr[d]), a);
       s = a * p.scale_log2;
+      if (p.inv_cap > 0.f) s = p.cap_log2 * capped_tanh<T>(a * p.inv_cap);
       if (p.r1) s -= r1 * log2f(fmaf(r2, (float)(pos - j), 1.f));
+      s -= slope * (float)(pos - j);
     }
     const float mn = fmaxf(m, warp_max(s)), alpha = exp2f(m - mn), pj = exp2f(s - mn);
     m = mn;
     l = l * alpha + warp_sum(pj);
-    const int n = min(32, pos + 1 - j0);
+    const int n = min(32, count - n0);
     for (int d = lane; d - lane < p.dv; d += 32) {
       float a = d < p.dv ? so[d] * alpha : 0.f;
       for (int jj = 0; jj < n; ++jj) {
         const float w = __shfl_sync(0xffffffffu, pj, jj);
-        if (d < p.dv) a = fmaf(w, to_f32<T>(V[(long long)((j0 + jj) % p.ring_rows) * p.v_rs + d]), a);
+        if (d < p.dv) a = fmaf(w, to_f32<T>(V[row_of(n0 + jj) * p.v_rs + d]), a);
       }
       if (d < p.dv) so[d] = a;
     }
@@ -676,10 +711,18 @@ extern "C" int eb_latent_decode(const void *q, long long q_batch_stride, const v
                                 long long cache_row_stride, int ring_rows, void *out, long long out_batch_stride, int batch, int heads,
                                 int rank, int window, const int32_t *pos_device, const int32_t *first, float scale, int dtype,
                                 int nsplit, void *scratch, size_t scratch_bytes, void *stream) {
+  return eb_latent_decode_sink(q, q_batch_stride, cache, cache_batch_stride, cache_row_stride, ring_rows, out, out_batch_stride, batch, heads, rank, window,
+                               pos_device, first, nullptr, scale, dtype, nsplit, scratch, scratch_bytes, stream);
+}
+
+extern "C" int eb_latent_decode_sink(const void *q, long long q_batch_stride, const void *cache, long long cache_batch_stride,
+                                long long cache_row_stride, int ring_rows, void *out, long long out_batch_stride, int batch, int heads,
+                                int rank, int window, const int32_t *pos_device, const int32_t *first, const float *sinks, float scale, int dtype,
+                                int nsplit, void *scratch, size_t scratch_bytes, void *stream) {
   if (batch == 0 || heads == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "latent_decode: fp16 or bf16 only (dtype %d)", dtype);
-  EB_REQUIRE(rank == 64 || rank == 128 || rank == 256 || rank == 384 || rank == 512,
-             "latent_decode: latent width %d not supported (64, 128, 256, 384 or 512)", rank);
+  EB_REQUIRE(rank == 64 || rank == 128 || rank == 192 || rank == 256 || rank == 320 || rank == 384 || rank == 512,
+             "latent_decode: latent width %d not supported (64, 128, 192, 256, 320, 384 or 512)", rank);
   EB_REQUIRE(batch > 0 && batch <= 65535 && heads > 0 && ring_rows > 0 && window >= 0 && nsplit >= 1 && nsplit <= 1024, "latent_decode: bad sizes");
   EB_REQUIRE(q && cache && out && pos_device, "latent_decode: null pointer");
   EB_REQUIRE(aligned16(q) && aligned16(cache) && aligned16(out), "latent_decode: pointers must be 16-byte aligned");
@@ -688,7 +731,7 @@ extern "C" int eb_latent_decode(const void *q, long long q_batch_stride, const v
   LatentParams p{};
   p.q = q; p.q_bs = q_batch_stride; p.c = cache; p.c_bs = cache_batch_stride; p.c_ld = cache_row_stride; p.ring_rows = ring_rows;
   p.o = out; p.o_bs = out_batch_stride; p.heads = heads; p.window = window; p.nsplit = nsplit;
-  p.pos_dev = pos_device; p.first = first; p.scale_log2 = scale * kLog2eLat;
+  p.pos_dev = pos_device; p.first = first; p.sinks = sinks; p.scale_log2 = scale * kLog2eLat;
   if (nsplit > 1 && !latent_clustered(nsplit)) {
     const size_t need = eb_latent_decode_scratch_bytes(batch, heads, rank, nsplit);
     EB_REQUIRE(scratch && scratch_bytes >= need && aligned16(scratch), "latent_decode: %d splits need a scratch of %zu bytes", nsplit, need);
@@ -706,7 +749,8 @@ static int plain_impl(const void *q, const void *k, const void *v, void *out, lo
                                   long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
                                   long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
                                   int v_dim, int window, int ring_rows, const int32_t *pos_device, const int32_t *first, const float *bias_r1,
-                                  const float *bias_r2, int sink, const float *sinks, int chunk, float scale, int dtype, void *stream) {
+                                  const float *bias_r2, int sink, const float *sinks, int chunk, float scale, int dtype, void *stream,
+                                  int keep = 0, int kept_rows = 0, const float *slopes = nullptr, float cap = 0.f) {
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype_ok(dtype), "attention_plain: bad dtype %d", dtype);
   EB_REQUIRE(q && k && v && out, "attention_plain: null pointer");
@@ -715,7 +759,10 @@ static int plain_impl(const void *q, const void *k, const void *v, void *out, lo
   EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_plain: %d heads do not share keys in groups of %d", heads, kv_group);
   EB_REQUIRE((bias_r1 == nullptr) == (bias_r2 == nullptr), "attention_plain: the distance bias has two numbers per head");
   PlainParams p{};
+  EB_REQUIRE(keep >= 0 && (kept_rows == 0 || kept_rows == keep) && cap >= 0.f, "attention_plain: a cache keeps all %d first positions or none", keep);
   p.group = kv_group; p.r1 = bias_r1; p.r2 = bias_r2; p.sink = sink; p.sinks = sinks; p.chunk = chunk;
+  p.keep = keep; p.kept_rows = kept_rows; p.slopes = slopes;
+  if (cap > 0.f) { p.cap_log2 = cap * kLog2eLat; p.inv_cap = scale / cap; }
   p.q = q; p.k = k; p.v = v; p.o = out;
   p.q_bs = q_batch_stride; p.q_rs = q_row_stride; p.q_hs = q_head_stride;
   p.k_bs = k_batch_stride; p.k_rs = k_row_stride; p.k_hs = k_head_stride;
@@ -750,4 +797,15 @@ extern "C" int eb_attention_plain_chunk(const void *q, const void *k, const void
   return plain_impl(q, k, v, out, q_batch_stride, q_row_stride, q_head_stride, k_batch_stride, k_row_stride, k_head_stride, v_batch_stride,
                     v_row_stride, v_head_stride, o_batch_stride, o_row_stride, o_head_stride, batch, heads, kv_group, q_len, k_dim, v_dim, 0,
                     ring_rows, pos_device, first, nullptr, nullptr, 0, sinks, chunk, scale, dtype, stream);
+}
+
+extern "C" int eb_attention_plain_capped(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
+                                  long long q_head_stride, long long k_batch_stride, long long k_row_stride, long long k_head_stride,
+                                  long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
+                                  long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
+                                  int v_dim, int window, int keep, int kept_rows, int ring_rows, const int32_t *pos_device, const int32_t *first,
+                                  const float *slopes, float cap, int sink, float scale, int dtype, void *stream) {
+  return plain_impl(q, k, v, out, q_batch_stride, q_row_stride, q_head_stride, k_batch_stride, k_row_stride, k_head_stride, v_batch_stride,
+                    v_row_stride, v_head_stride, o_batch_stride, o_row_stride, o_head_stride, batch, heads, kv_group, q_len, k_dim, v_dim, window,
+                    ring_rows, pos_device, first, nullptr, nullptr, sink, nullptr, 0, scale, dtype, stream, keep, kept_rows, slopes, cap);
 }

@@ -1,5 +1,5 @@
 """Python entry to the decaying-memory kernels: state-space (eb_short_conv, eb_ssm_*, eb_gate_group_norm) and gated
-linear (eb_gla_*) layers."""
+linear (eb_gla_*) layers, and the state space with a state per channel (eb_selective_*)."""
 import torch
 
 from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
@@ -136,4 +136,55 @@ def gla_step(q, k, v, g, low, w2, b2, tau, scale, norm, dv_count, eps, S, heads)
     out = torch.empty((B, heads * dv), dtype=q.dtype, device=q.device)
     check(lib().eb_gla_step(ptr(q), ptr(k), ptr(v), ptr(g), ptr(low), q.stride(0), ptr(w2), ptr(b2), rank, float(tau), float(scale), ptr(norm),
                             int(dv_count), float(eps), ptr(out), heads * dv, ptr(S), B, heads, dk, dv, dtype_code(q.dtype), stream_ptr()), "gla_step")
+    return out
+
+
+def short_conv_step(x, w, b, ring, pos_device, first=None):
+    """short_conv of one token per sequence, x [batch, C]: earlier inputs from the ring, this one into it."""
+    require_cuda(x, w, b, ring, pos_device, first)
+    ldx, (n, C) = _rows(x, "short_conv_step: x"), x.shape
+    if w.shape[1] != C or b.numel() != C or not w.is_contiguous() or any(t.dtype != x.dtype for t in (w, b, ring)):
+        raise RuntimeError("short_conv_step: w [taps, C], b [C] of one dtype")
+    if ring.dim() != 3 or ring.shape[0] != n or ring.shape[2] != C or ring.stride(2) != 1:
+        raise RuntimeError("short_conv_step: the ring is [batch, rows, C]")
+    out = torch.empty((n, C), dtype=x.dtype, device=x.device)
+    check(lib().eb_short_conv_step(ptr(x), ldx, ptr(w), ptr(b), ptr(out), C, n, C, w.shape[0], ptr(pos_device), ptr(first), ptr(ring), ring.stride(0),
+                                   ring.stride(1), ring.shape[1], dtype_code(x.dtype), stream_ptr()), "short_conv_step")
+    return out
+
+
+def _selective(x, gate, bc, bias, a_log, skip, S, out):
+    inner, states = a_log.shape
+    if any(t.dtype != torch.float32 or not t.is_contiguous() for t in (bias, a_log, skip, S)) or bias.numel() != inner or skip.numel() != inner or tuple(S.shape[1:]) != (inner, states):
+        raise RuntimeError("selective scan: bias, skip [inner], a_log [inner, states] and the state [batch, inner, states] are fp32")
+    if x.shape[1] != inner or gate.shape != x.shape or gate.dtype != x.dtype or bc.dtype != torch.float32 or bc.shape[0] != x.shape[0] or bc.shape[1] < 2 * states:
+        raise RuntimeError("selective scan: rows x and gate [rows, inner], bc fp32 [rows, 2 * states]")
+    out = torch.empty((x.shape[0], inner), dtype=x.dtype, device=x.device) if out is None else out
+    if out.shape != x.shape or out.dtype != x.dtype:
+        raise RuntimeError("selective scan: the output is laid out like x")
+    return inner, states, out, (ptr(x), _rows(x, "x"), ptr(gate), _rows(gate, "gate"))
+
+
+def selective_scan(x, gate, z, bc, bias, a_log, skip, S, first=None, out=None):
+    """A prompt through the recurrence with a state per channel: x [batch*seq, inner] behind the convolution, gate alike, z fp32
+    [batch*seq, inner] (projected steps without their bias), bc fp32 [batch*seq, >= 2 * states] (B | C).  S [batch, inner,
+    states] is overwritten with the state behind the last token.  Returns (S^T C + skip x) * silu(gate)."""
+    require_cuda(x, gate, z, bc, bias, a_log, skip, S, first, out)
+    inner, states, out, rows = _selective(x, gate, bc, bias, a_log, skip, S, out)
+    B = S.shape[0]
+    if z.dtype != torch.float32 or tuple(z.shape) != tuple(x.shape) or x.shape[0] % B:
+        raise RuntimeError("selective scan: z is fp32 [rows, inner], whole sequences")
+    check(lib().eb_selective_scan(*rows, ptr(z), _rows(z, "z"), ptr(bc), _rows(bc, "bc"), ptr(bias), ptr(a_log), ptr(skip), ptr(first), ptr(out),
+                                  _rows(out, "out"), ptr(S), B, x.shape[0] // B, inner, states, dtype_code(x.dtype), stream_ptr()), "selective_scan")
+    return out
+
+
+def selective_step(x, gate, low, w, bc, bias, a_log, skip, S, out=None):
+    """One token per sequence: z = low @ w.T (low [batch, rank], w [inner, rank]); S goes on.  Returns as selective_scan."""
+    require_cuda(x, gate, low, w, bc, bias, a_log, skip, S, out)
+    inner, states, out, rows = _selective(x, gate, bc, bias, a_log, skip, S, out)
+    if x.shape[0] != S.shape[0] or not w.is_contiguous() or w.shape[0] != inner or low.shape != (x.shape[0], w.shape[1]) or any(t.dtype != x.dtype for t in (low, w)):
+        raise RuntimeError("selective scan: low [batch, rank] and w [inner, rank] of the rows' dtype")
+    check(lib().eb_selective_step(*rows, ptr(low), _rows(low, "low"), ptr(w), w.shape[1], ptr(bc), _rows(bc, "bc"), ptr(bias), ptr(a_log), ptr(skip),
+                                  ptr(out), _rows(out, "out"), ptr(S), x.shape[0], inner, states, dtype_code(x.dtype), stream_ptr()), "selective_step")
     return out

@@ -148,22 +148,25 @@ def project_parts(x, w, bias=None, xielu=None, tail_col=None):
     return out if tail_col is None else (out[:, :tail_col], out[:, tail_col:])
 
 
-def project_unit(x, w, unit):
+def project_unit(x, w, unit, out=None):
     """A feed-forward's first product with its unit in the epilogue: "gelu" of x @ w.T, or "geglu", w in blocks of
-    8 gate rows and their 8 up rows -> half as many columns."""
+    8 gate rows and their 8 up rows -> half as many columns (out: rows that receive them, a row stride allowed)."""
     from .moe import UNITS, unit_act
+    if out is not None and (out.dtype != x.dtype or out.stride(-1) != 1 or tuple(out.shape) != (x.shape[0], w.shape[0] // (1 if unit == "gelu" else 2))):
+        raise RuntimeError("project_unit: the result has another shape")
     if w.dtype == torch.float32:
-        return unit_act(gemm_f32(x, w), unit)
+        return unit_act(gemm_f32(x, w), unit, out=out)
     if unit == "gelu":
-        return gemm(x, w, act="gelu", static_weight=True)
+        return gemm(x, w, act="gelu", static_weight=True, out=out)
     require_cuda(x, w)
     if x.dim() != 2 or x.stride(1) != 1 or not w.is_contiguous() or x.dtype != w.dtype or x.shape[1] != w.shape[1]:
         raise RuntimeError("project_unit: x [M,K] and contiguous w [N,K] of one dtype required")
     (M, K), N = x.shape, w.shape[0]
-    out = torch.empty((M, N // 2), dtype=x.dtype, device=x.device)
+    out = torch.empty((M, N // 2), dtype=x.dtype, device=x.device) if out is None else out
+    require_cuda(out)
     nbytes = lib().eb_gemm_workspace_bytes(M, N, K)
     ws = workspace(x.device, nbytes) if nbytes else None
-    check(lib().eb_gemm_gated(ptr(x), x.stride(0), ptr(w), K, ptr(out), N // 2, M, N, K, UNITS[unit], 0.0, 0.0, dtype_code(x.dtype), 1, ptr(ws),
+    check(lib().eb_gemm_gated(ptr(x), x.stride(0), ptr(w), K, ptr(out), out.stride(0), M, N, K, UNITS[unit], 0.0, 0.0, dtype_code(x.dtype), 1, ptr(ws),
                               ws.numel() if ws is not None else 0, stream_ptr()), "gemm_gated")
     return out
 

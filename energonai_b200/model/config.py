@@ -1,4 +1,5 @@
-"""config.json of a layer-listed decoder -> LatentDecoderConfig, SandwichDecoderConfig or HybridDecoderConfig.
+"""config.json of a layer-listed decoder -> LatentDecoderConfig, SandwichDecoderConfig, HybridDecoderConfig or
+ParallelDecoderConfig.
 
     {"architecture": ..., "vocab": V, "width": W, "norm": {"eps": e},
      "layers": [{"type": "latent_attention",
@@ -362,3 +363,121 @@ class HybridDecoderConfig:
                 _need(lc.mixer.right.rank in (None, rank), f"layer {i}", f"the decay's projection has rank {rank}, the configuration asks for {lc.mixer.right.rank}")
                 lc.mixer.right.rank = rank
         return self
+
+
+# ---- decoders whose mixer and feed-forward read the stream side by side ----------------------------------
+#
+#     {"architecture": ..., "vocab": V, "width": W, "norm": {"eps": e}, "canon": {"taps": t},
+#      "layers": [{"type": "latent_attention",
+#                  "mixer": {"heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale", "kv_from"?,
+#                            "rot": {"dims", "base", "scaling": {"factor", "original", "fast", "slow"}?}}, "mlp": ...},
+#                 {"type": "mamba1", "mixer": {"inner", "state", "dt_rank", "conv"}, "mlp": ...},
+#                 {"type": "attention", "mixer": {"heads", "kv_heads", "dim", "vdim", "scale", "softcap"?,
+#                                                 "mask": {"size", "keep_first"?}?}, "mlp": {"kind": "dense", "ff"} | null}, ...]}
+
+@dataclass
+class RotaryLatentConfig:
+    heads: int
+    dim: int                 # of a query or key head, without the rotated part
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rot_base: float
+    rot_scaling: Optional[tuple] = None      # (factor, original, fast, slow)
+    kv_from: Optional[int] = None
+
+
+@dataclass
+class SelectiveScanConfig:
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int                # taps of the convolution, the current token's included
+
+
+@dataclass
+class CappedAttentionConfig:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    softcap: float = 0.0     # 0: none
+    window: int = 0          # 0: none
+    keep_first: int = 0      # positions that stay visible behind the window
+
+
+@dataclass
+class ParallelLayerConfig:
+    mixer: Union[RotaryLatentConfig, SelectiveScanConfig, CappedAttentionConfig]
+    mlp: Optional[DenseConfig] = None
+
+
+@dataclass
+class ParallelDecoderConfig:
+    vocab: int
+    width: int
+    eps: float
+    taps: int                # of the convolution in front of every sublayer
+    layers: List[ParallelLayerConfig]
+
+    @staticmethod
+    def _mixer(where, kind, m):
+        if kind == "mamba1":
+            _known(where, m, ("inner", "state", "dt_rank", "conv"))
+            c = SelectiveScanConfig(*_sizes(where, m, "inner", "state", "dt_rank", "conv"))
+            _need(c.state <= 256, where, f"{c.state} states per channel (at most 256)")
+            return c
+        if kind == "attention":
+            _known(where, m, ("heads", "kv_heads", "dim", "vdim", "scale", "softcap", "mask"))
+            c = CappedAttentionConfig(*_sizes(where, m, "heads", "kv_heads", "dim", "vdim"), scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0))
+            _need(c.heads % c.kv_heads == 0, where, f"{c.heads} heads do not share {c.kv_heads} key / value heads")
+            _need(c.softcap >= 0, where, f"scores capped at {c.softcap}")
+            if m.get("mask"):
+                _known(where, m["mask"], ("size", "keep_first"))
+                c.window, = _sizes(where, m["mask"], "size")
+                c.keep_first = int(m["mask"].get("keep_first") or 0)
+                _need(c.keep_first >= 0, where, f"a window that keeps {c.keep_first} positions")
+            return c
+        _need(kind == "latent_attention", where, f"unknown type {kind!r}")
+        _known(where, m, ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale", "rot", "kv_from"))
+        rot, src = m["rot"], m.get("kv_from")
+        _known(where, rot, ("dims", "base", "scaling"))
+        c = RotaryLatentConfig(*_sizes(where, m, "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank"), scale=float(m["scale"]),
+                               rot_base=float(rot["base"]), kv_from=None if src is None else int(src))
+        _need(int(rot["dims"]) == c.rot_dim and c.rot_dim % 2 == 0 and c.rot_base > 0, where, f"{rot['dims']} of {c.rot_dim} dimensions rotated")
+        if rot.get("scaling"):
+            s = rot["scaling"]
+            _known(where, s, ("factor", "original", "fast", "slow"))
+            c.rot_scaling = tuple(float(s[k]) for k in ("factor", "original", "fast", "slow"))
+            _need(all(v > 0 for v in c.rot_scaling) and c.rot_base != 1, where, f"rotation scaled by {c.rot_scaling}")
+        return c
+
+    @classmethod
+    def from_dict(cls, d):
+        _known("model", d, ("architecture", "vocab", "width", "norm", "canon", "layers"))
+        _known("norm", d["norm"], ("eps",))
+        _known("canon", d["canon"], ("taps",))
+        layers = []
+        for i, ly in enumerate(d["layers"]):
+            where = f"layer {i}"
+            _known(where, ly, ("type", "mixer", "mlp"))
+            mlp, f = None, ly.get("mlp")
+            if f is not None:
+                _need(f.get("kind", "dense") == "dense", where, f"unknown feed-forward kind {f.get('kind')!r}")
+                _known(where, f, ("kind", "ff"))
+                mlp = DenseConfig(*_sizes(where, f, "ff"))
+            c = cls._mixer(where, ly["type"], ly["mixer"])
+            src = getattr(c, "kv_from", None)
+            if src is not None:
+                _need(0 <= src < i and isinstance(layers[src].mixer, RotaryLatentConfig), where, f"kv_from must name an earlier latent layer (got {src})")
+                other = layers[src].mixer
+                _need(other.kv_from is None, where, f"layer {src} has no latents of its own")
+                same = lambda m: (m.kv_rank, m.rot_dim, m.rot_base, m.rot_scaling)
+                _need(same(other) == same(c), where, f"its latents and rotation differ from those of layer {src}")
+            layers.append(ParallelLayerConfig(c, mlp))
+        taps, = _sizes("canon", d["canon"], "taps")
+        _need(taps <= 16, "canon", f"a convolution of {taps} taps (at most 16)")
+        return cls(*_sizes("model", d, "vocab", "width"), eps=float(d["norm"]["eps"]), taps=taps, layers=layers)

@@ -16,12 +16,13 @@ columns change no product.
 import torch
 from torch import nn
 
-from ..attention import (LATENT_WIDTHS, attention_plain, attention_prefill_window, latent_decode)
+from ..attention import (LATENT_WIDTHS, attention_plain, attention_prefill_gated, attention_prefill_window, latent_decode, latent_inputs, rotate_heads,
+                         sigmoid_gate, yarn_rotation)
 from ..gemm import project
 from ..moe import per_head
 from ..nn import RMSNorm1D, init_weight
 from ..norm import rms_norm
-from .sequence_state import round_up
+from .sequence_state import RingCache, round_up
 
 
 class LatentAttention(nn.Module):
@@ -84,3 +85,76 @@ class LatentAttention(nn.Module):
                                 first=ctx.first, pos_device=ctx.pos, shared_kv=True).view(B, -1)
         v = per_head(o, self.kv_up[self.q_rows:].view(self.heads, self.dv, self.rank))
         return project(v, self.out_proj)
+
+
+class RotaryLatentAttention(nn.Module):
+    """Latent attention whose query comes out of a latent of its own and has a rotated part; the key's rotated part is common
+    to all heads and cached behind the latent, as one row.  A number per head joins the softmax as a score without
+    a value, and the concatenated heads are multiplied by the sigmoid of a gate.
+
+    The key up-projection carries the rotated part through with ones, so that a head's whole key, or the absorbed
+    query, is one linear map of the cached row.  One product of h gives query latent, cached row and gate."""
+    output_bias = False
+
+    def __init__(self, layer, width, cfg, eps, dtype, device=None):
+        super().__init__()
+        kw = dict(dtype=dtype, device=device)
+        self.layer, self.eps, self.heads, self.scale, self.kv_from = layer, eps, cfg.heads, cfg.scale, cfg.kv_from
+        self.dim, self.rot_dim, self.vdim, self.q_rank, self.kv_rank = cfg.dim, cfg.rot_dim, cfg.vdim, cfg.q_rank, cfg.kv_rank
+        self.rot_at, self.rot_col = round_up(cfg.dim, 8), round_up(cfg.kv_rank, 8)         # where the rotated part begins in a head, in a row
+        key, row = self.rot_at + cfg.rot_dim, self.rot_col + cfg.rot_dim
+        self.tensor_core_prompt = dtype != torch.float32 and max(key, cfg.vdim) <= 128 and cfg.scale > 0
+        if self.tensor_core_prompt:
+            self.dv = 64 if cfg.vdim <= 64 else 128
+            self.dk = max(self.dv, 64 if key <= 64 else 128)
+        else:
+            self.dk, self.dv = round_up(key, 8), round_up(cfg.vdim, 8)
+        self.tensor_core_step = dtype != torch.float32 and row <= LATENT_WIDTHS[-1]
+        self.rank = min(w for w in LATENT_WIDTHS if w >= row) if self.tensor_core_step else round_up(row, 8)
+        self.q_cols, self.q_rows, self.columns = round_up(cfg.q_rank, 8), cfg.heads * self.dk, cfg.heads * self.dv
+        own = cfg.kv_from is None
+        ones = lambda n: nn.Parameter(torch.ones(n, **kw), requires_grad=False)
+        self.in_proj = init_weight(self.q_cols + (self.rank if own else 0) + self.columns, width, **kw)      # query latent | row | gate
+        self.q_norm, self.latent_norm = ones(self.q_cols), ones(self.rot_col) if own else None
+        self.q_up = init_weight(self.q_rows, self.q_cols, **kw)
+        self.kv_up = init_weight(self.q_rows + self.columns, self.rank, **kw)              # keys | values, head by head
+        self.k_absorb = init_weight(self.heads, self.rank, self.dk, **kw)                  # a head's key map, transposed
+        self.sinks = nn.Parameter(torch.zeros(self.heads, dtype=torch.float32, device=device), requires_grad=False)
+        freq, self.factor = yarn_rotation(cfg.rot_dim, cfg.rot_base, cfg.rot_scaling)
+        self.register_buffer("freq", freq.to(device=device), persistent=False)
+
+    @property
+    def source(self):
+        return self.layer if self.kv_from is None else self.kv_from
+
+    def caches(self):
+        return {self.layer: RingCache(self.rank)} if self.kv_from is None else {}
+
+    def forward(self, h, ctx, out):
+        """h [rows, width] -> out [rows, columns]; rows of this layer's own latents are cached."""
+        B, S, H = ctx.batch, ctx.seq, self.heads
+        cache, where = ctx.state.caches[self.source].buf, dict(rows_per_batch=S, pos_device=ctx.pos, first=ctx.first)
+        proj = project(h, self.in_proj)
+        gate, row = proj[:, proj.shape[1] - self.columns:], None
+        if self.kv_from is None:
+            row = dict(cols=self.rank, rot_col=self.rot_col, count=self.kv_rank, norm=self.latent_norm, freq=self.freq, factor=self.factor, ring=cache,
+                       keep_rows=ctx.is_prompt)
+        q, rows = latent_inputs(proj, self.q_cols, self.q_rank, self.q_norm, self.eps, row=row, **where)
+        q = rotate_heads(project(q, self.q_up), H, self.dk, self.rot_at, self.freq, self.factor, **where)
+        if ctx.is_prompt:
+            if rows is not None:
+                ctx.latents[self.layer] = rows
+            kv = project(ctx.latents[self.source], self.kv_up).view(B, S, -1)
+            q, k, v = q.view(B, S, -1), kv[:, :, :self.q_rows], kv[:, :, self.q_rows:]
+            if self.tensor_core_prompt:
+                return attention_prefill_gated(q, k, v, self.dk, self.dv, sinks=self.sinks, first=ctx.first, gate=gate.view(B, S, -1), scale=self.scale,
+                                               out=out.view(B, S, -1))
+            o = attention_plain(q, k, v, H, self.dk, self.dv, scale=self.scale, first=ctx.first, chunk=0, sinks=self.sinks)
+            return sigmoid_gate(o.view(B * S, -1), gate, out=out)
+        qa = per_head(q, self.k_absorb)
+        if self.tensor_core_step:
+            o = latent_decode(qa, cache, self.rank, H, 0, ctx.pos, self.scale, first=ctx.first, sinks=self.sinks)
+        else:
+            o = attention_plain(qa.view(B, 1, -1), cache, cache, H, self.rank, self.rank, scale=self.scale, first=ctx.first, pos_device=ctx.pos,
+                                shared_kv=True, chunk=0, sinks=self.sinks).view(B, -1)
+        return sigmoid_gate(per_head(o, self.kv_up[self.q_rows:].view(H, self.dv, self.rank)), gate, out=out)

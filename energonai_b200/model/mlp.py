@@ -77,15 +77,20 @@ class GEGLUFeedForward(nn.Module):
     """W_down (gelu_tanh(W_gate h) * (W_up h)); gates and ups interleaved in blocks of 8 rows, the unit in the epilogue
     of their product."""
 
-    def __init__(self, width, ff, dtype, device=None):
+    def __init__(self, width, ff, dtype, device=None, down=True):
+        """down=False: the output product belongs to the block (see inner())."""
         super().__init__()
         kw = dict(dtype=dtype, device=device)
         self.ff, self.ff_padded = ff, round_up(ff, 8)
         self.gate_up = init_weight(2 * self.ff_padded, width, **kw)
-        self.down = init_weight(width, self.ff_padded, **kw)
+        self.down = init_weight(width, self.ff_padded, **kw) if down else None
 
     def router_for_step(self, tokens):
         return None
+
+    def inner(self, h, out):
+        """The unit's columns alone, into `out` [rows, ff_padded] (blocks that share one output product)."""
+        return project_unit(h, self.gate_up, "geglu", out=out)
 
     def forward(self, h, first=None, rows_per_batch=1, routed=None):
         """-> what stream_add adds."""

@@ -14,16 +14,17 @@ def round_up(n, m):
 
 
 class RingCache(KVCache):
-    """[batch, rows, width] ring: position p lives in row p mod rows.  `window` is the longest window of
+    """[batch, keep + rows, width]: `keep` rows for the first positions of each sequence, if a window keeps them
+    visible, and a ring in which position p lives in row p mod rows.  `window` is the longest window of
     the layers that read it (0: unlimited), so rows = min(positions, window).  A ring shorter than its
     window has never wrapped, which is why it can grow like a KVCache."""
 
-    def __init__(self, width, window=0, reserve=256):
+    def __init__(self, width, window=0, reserve=256, keep=0):
         super().__init__(reserve)
-        self.width, self.window = width, window
+        self.width, self.window, self.kept = width, window, keep
 
     def rows_for(self, positions):
-        return min(positions, self.window) if self.window > 0 else positions
+        return self.kept + (min(positions, self.window) if self.window > 0 else positions)
 
     def prepare(self, batch, positions, dtype, device):
         """For a new batch: room for `positions`; memory kept from an earlier batch of the same size
@@ -37,21 +38,23 @@ class RingCache(KVCache):
         rows = self.rows_for(positions)
         have = self.buf.shape[1]
         if rows > have:
-            self.ensure(self.buf.shape[0], self.rows_for(positions + self.reserve), self.width, self.buf.dtype, self.buf.device, exact=True)
-            self.buf[:, have:].zero_()
+            old = self.buf
+            self.buf = torch.zeros((old.shape[0], self.rows_for(positions + self.reserve), self.width), dtype=old.dtype, device=old.device)
+            self.buf[:, :have] = old
 
     def keep(self, rows):
         self.buf = self.buf.index_select(0, rows)
 
     def fork(self):
         """The same memory under another owner (which then keeps its own sequences)."""
-        out = RingCache(self.width, self.window, self.reserve)
+        out = RingCache(self.width, self.window, self.reserve, self.kept)
         out.buf, out.len = self.buf, self.len
         return out
 
     def room(self):
         """Positions it can take; None if it holds its whole window."""
-        return self.buf.shape[1] if self.window <= 0 or self.buf.shape[1] < self.window else None
+        rows = self.buf.shape[1] - self.kept
+        return rows if self.window <= 0 or rows < self.window else None
 
     def pointers(self):
         return (self.buf.data_ptr(),)

@@ -107,13 +107,13 @@ def grouped_gemm(a, w, plan, gate=None, unit=None):
     return out
 
 
-def unit_act(x, unit=None, gate=None):
+def unit_act(x, unit=None, gate=None, out=None):
     """A unit alone: [n, N] -> [n, N], or, gated, [n, 2*half] in the 8 + 8 column order -> [n, half]."""
-    require_cuda(x)
+    require_cuda(x, out)
     code, limit, alpha, per = unit_code(unit, gate)
     n = x.shape[1] // per
-    y = torch.empty((x.shape[0], n), dtype=x.dtype, device=x.device)
-    check(lib().eb_unit_act(ptr(x), x.stride(0), ptr(y), n, x.shape[0], n, code, limit, alpha, dtype_code(x.dtype), stream_ptr()), "unit_act")
+    y = torch.empty((x.shape[0], n), dtype=x.dtype, device=x.device) if out is None else out
+    check(lib().eb_unit_act(ptr(x), x.stride(0), ptr(y), y.stride(0), x.shape[0], n, code, limit, alpha, dtype_code(x.dtype), stream_ptr()), "unit_act")
     return y
 
 

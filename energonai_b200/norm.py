@@ -1,4 +1,5 @@
-"""Python entry to the RMS-norm kernels (eb_rms_norm / eb_rms_residual / eb_stream_update / eb_stream_add)."""
+"""Python entry to the RMS-norm kernels (eb_rms_norm / eb_rms_residual / eb_stream_update / eb_stream_add /
+eb_stream_conv)."""
 import torch
 
 from ._lib import lib, check, dtype_code, ptr, stream_ptr, require_cuda
@@ -119,3 +120,33 @@ def stream_add(x, eps, count=None, src=None, src2=None, y=None, w=None, y2=None,
                               ptr(rule.correction) if rule else None, rule.groups if rule else 1, rule.keep if rule else 1, ptr(r_idx), ptr(r_w),
                               ptr(r_gate), dtype_code(t.dtype), stream_ptr()), "stream_add")
     return (h, (r_idx, r_w, r_gate)) if router is not None else h
+
+
+CONV_TAPS = (2, 3, 4, 8, 16)          # sizes of the tap tables stream_conv takes (pad in front with zero rows)
+
+
+def stream_conv(x, k1, ring, eps, batch, count=None, src=None, y=None, k2=None, first=None, pos_device=None):
+    """The residual step of blocks whose two sublayers read the same stream through a norm and a short causal convolution of
+    the normed rows over time; x [rows, n2] fp32 (not read if src, the embedding rows, is given):
+      x' = (src or x) + y;  u = x' over its root mean square;  h1_t = sum_j k1[j] u_(t - taps + 1 + j);  h2 with k2
+    k1, k2 fp32 [taps, n2] (k2 None: one sublayer).  The last rows u go to ring [batch, rows, n2].  pos_device (int32
+    scalar): a step, one row per sequence, earlier rows from the ring.  Returns (x', h1, h2 or None)."""
+    require_cuda(x, src, y, k1, k2, ring, first, pos_device)
+    t, like = src if src is not None else y, x if x is not None else src
+    n1, n2 = like.shape
+    taps = k1.shape[0]
+    if t is None or ring.dtype != t.dtype or any(a is not None and (a.dtype != t.dtype or tuple(a.shape) != (n1, n2)) for a in (src, y)) or (
+            x is not None and (x.dtype != torch.float32 or tuple(x.shape) != (n1, n2))):
+        raise RuntimeError("stream_conv: rows [rows, width]; x is fp32, the others and the ring share a dtype")
+    if any(k is not None and (k.dtype != torch.float32 or not k.is_contiguous() or tuple(k.shape) != (taps, n2)) for k in (k1, k2)):
+        raise RuntimeError("stream_conv: tap tables are contiguous fp32 [taps, width]")
+    if n1 % batch or ring.dim() != 3 or ring.shape[0] != batch or ring.shape[2] != n2 or ring.stride(2) != 1 or (pos_device is not None and n1 != batch):
+        raise RuntimeError("stream_conv: the ring is [batch, rows, width]; a step has one row per sequence")
+    x_out = torch.empty((n1, n2), dtype=torch.float32, device=t.device)
+    h1 = torch.empty((n1, n2), dtype=t.dtype, device=t.device)
+    h2 = torch.empty_like(h1) if k2 is not None else None
+    ld = lambda a, what: _rows(a, f"stream_conv: {what}") if a is not None else n2
+    check(lib().eb_stream_conv(ptr(src), ld(src, "src"), ptr(x) if src is None else None, n2, ptr(y), ld(y, "y"), ptr(x_out), ptr(k1), ptr(k2), taps,
+                               ptr(h1), ptr(h2), n2, ptr(ring), ring.stride(0), ring.stride(1), ring.shape[1], batch, n1 // batch, n2, count or n2,
+                               float(eps), ptr(first), ptr(pos_device), dtype_code(t.dtype), stream_ptr()), "stream_conv")
+    return x_out, h1, h2

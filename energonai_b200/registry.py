@@ -84,16 +84,19 @@ def _populate():
         return
     _done = True
     from . import model as M
-    from .model.config import HybridDecoderConfig, LatentDecoderConfig, SandwichDecoderConfig
+    from .model.config import HybridDecoderConfig, LatentDecoderConfig, ParallelDecoderConfig, SandwichDecoderConfig
     from .model.hybrid_decoder import HybridDecoder
     from .model.latent_decoder import LatentDecoder
+    from .model.parallel_decoder import ParallelDecoder
     from .model.sandwich_decoder import SandwichDecoder
     from .utils.checkpointing_moponex import processing_Moponex
     from .utils.checkpointing_mutolix import processing_Mutolix
     from .utils.checkpointing_tulezen import processing_Tulezen
+    from .utils.checkpointing_tupidra import processing_Tupidra
     for name in ("opt_125M", "opt_6B", "opt_13B", "opt_30B", "opt_66B", "opt_175B", "gpt2_small", "gpt2_large", "gpt2_8B", "gpt3",
                  "hf_gpt2", "bert_small", "bert_large", "bert_8B", "bert_175B"):
         register_factory(name, getattr(M, name))
     register_architecture("Tulezen", LatentDecoderConfig, LatentDecoder, processing_Tulezen)
     register_architecture("Mutolix", SandwichDecoderConfig, SandwichDecoder, processing_Mutolix)
     register_architecture("Moponex", HybridDecoderConfig, HybridDecoder, processing_Moponex)
+    register_architecture("Tupidra", ParallelDecoderConfig, ParallelDecoder, processing_Tupidra)

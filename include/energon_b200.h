@@ -473,6 +473,19 @@ EB_API int eb_stream_add(const void *src, long long lds, const void *src2, long 
                   int n1, int n2, int count, const void *router, int choices, int r_experts, int r_top, const float *r_correction,
                   int r_groups, int r_keep, int32_t *r_idx, float *r_weights, float *r_gate, int dtype, void *stream);
 
+/* The residual step of blocks whose two sublayers read the same stream, each through a norm and a causal
+ * convolution of the normed rows over time, per row of n2 elements (means over the first `count`):
+ *   x_out = (src, else x_in) + y (or NULL);  u = x_out / sqrt(mean(x_out^2) + eps)
+ *   h1_t = sum_j k1[j] u_(t - taps + 1 + j),  h2_t likewise with k2 (h2 NULL: one sublayer)
+ * k1, k2 fp32 [taps][n2] (norm weight times tap, one more for the current token's; taps 2, 3, 4, 8 or 16), rows in front
+ * of first[b] count as zero.  Rows b*seq + s; the last ring_rows rows u also go to the ring, position p in row
+ * p mod ring_rows.  x_out must not be x_in.  With pos_device: one token per sequence at that position (seq 1; in place
+ * allowed), earlier rows come from the ring. */
+EB_API int eb_stream_conv(const void *src, long long lds, const float *x_in, long long ldx, const void *y, long long ldy, float *x_out,
+                   const float *k1, const float *k2, int taps, void *h1, void *h2, long long ldh, void *ring,
+                   long long ring_batch_stride, long long ring_ld, int ring_rows, int batch, int seq, int n2, int count, float eps,
+                   const int32_t *first, const int32_t *pos_device, int dtype, void *stream);
+
 /* Queries, keys and values of a projected row [q: heads*dk | k: kv_heads*dk | v: kv_heads*dv] made ready
  * for attention.  q and k are divided by the root mean square over ALL their rows (counts q_count and
  * k_count: heads may be zero-padded) and multiplied by q_norm / k_norm; q also by
@@ -499,6 +512,34 @@ EB_API int eb_attention_rotary(const void *proj, long long ldp, int heads, int k
                         long long ldk, void *k_cache, long long k_batch_stride, long long k_row_stride, void *v_cache,
                         long long v_batch_stride, long long v_row_stride, int ring_rows, int n1, int rows_per_batch,
                         const int32_t *pos_device, const int32_t *first, int dtype, void *stream);
+
+/* Every value head is divided by its root mean square (over dv_count columns), in place, and key and value go to a
+ * cache of `keep` rows for the first positions of a sequence followed by a ring of ring_rows rows: position col =
+ * pos0 + s of row b*rows_per_batch + s to ring row col mod ring_rows (of a longer prompt only the last ring_rows
+ * positions) and, while col - first[b] < keep, to that row in front.  k and v are column ranges of rows ld apart. */
+EB_API int eb_attention_values(const void *k, void *v, long long ld, int kv_heads, int dk, int dv, int dv_count, float eps, void *k_cache,
+                        long long k_batch_stride, long long k_row_stride, void *v_cache, long long v_batch_stride, long long v_row_stride,
+                        int keep, int ring_rows, int n1, int rows_per_batch, const int32_t *pos_device, const int32_t *first, int dtype,
+                        void *stream);
+
+/* out = y * sigmoid(g), rows of n2 columns. */
+EB_API int eb_sigmoid_gate(const void *y, long long ldy, const void *g, long long ldg, void *out, long long ldo, int n1, int n2, int dtype,
+                    void *stream);
+
+/* Rows [query latent: q_cols | c | rotated key part] of a projection, the latter two row_cols together, the rotated part
+ * from rot_col on (row_cols and q_cols multiples of 8, zero-padded):
+ *   q_out = norm(query latent) * q_norm                     norm(z) = z / sqrt(sum(z^2) / count + eps)
+ *   row   = [norm(c) * c_norm | (u, v) turned by p freq[i] and times factor, for its first `pairs` neighbouring pairs | 0]
+ * at position p = pos0 + s - first[b].  The row goes to ring row (pos0 + s) mod ring_rows (as eb_attention_rotary) and to
+ * rows_out (or NULL).  ring NULL: only the query latent. */
+EB_API int eb_latent_inputs(const void *proj, long long ldp, int q_cols, int q_count, const void *q_norm, void *q_out, long long ldq,
+                     int row_cols, int rot_col, int c_count, const void *c_norm, int pairs, const float *freq, float factor, float eps,
+                     void *rows_out, long long ldr, void *ring, long long ring_batch_stride, long long ring_ld, int ring_rows, int n1,
+                     int rows_per_batch, const int32_t *pos_device, const int32_t *first, int dtype, void *stream);
+
+/* The pairs from column `col` of every head (head_cols columns) of rows x, turned in place as above. */
+EB_API int eb_rotate_heads(void *x, long long ldx, int heads, int head_cols, int col, int pairs, const float *freq, float factor, int n1,
+                    int rows_per_batch, const int32_t *pos_device, const int32_t *first, int dtype, void *stream);
 
 /* ---- decaying memories --------------------------------------------------------------------------- */
 
@@ -553,6 +594,30 @@ EB_API int eb_gla_step(const void *q, const void *k, const void *v, const void *
  * columns padded to dv_padded; padding columns of out are not written). */
 EB_API int eb_gate_group_norm(const void *y, long long ldy, const void *z, long long ldz, const void *norm, float eps, void *out,
                        long long ldo, int rows, int heads, int dv, int dv_padded, int parts, int dtype, void *stream);
+
+/* ---- selective state space (a state per channel) ----------------------------------------------------- */
+
+/* Channel c of `inner`, state n of `states` (multiples of 8 and 4, zero-padded):
+ *   dt = softplus(z_c + bias[c]);  S[c][n] = exp(-exp(a_log[c][n]) dt) S[c][n] + dt x_c B_n;  y_c = sum_n S[c][n] C_n + skip[c] x_c
+ *   out_c = y_c silu(gate_c)
+ * x is behind the convolution (eb_short_conv), bc rows are [B: states | C: states] and, like z and the state
+ * S [batch][inner][states], fp32.
+ *
+ * eb_selective_scan: a whole prompt from an empty state, rows b*seq + s; rows in front of first[b] add nothing and
+ * forget nothing. */
+EB_API int eb_selective_scan(const void *x, long long ldx, const void *gate, long long ldg, const float *z, long long ldz, const float *bc,
+                      long long ldbc, const float *bias, const float *a_log, const float *skip, const int32_t *first, void *out,
+                      long long ldo, float *S, int batch, int seq, int inner, int states, int dtype, void *stream);
+
+/* One token per sequence, the state goes on; z = w low, w [inner][rank] (rank a multiple of 8, zero-padded). */
+EB_API int eb_selective_step(const void *x, long long ldx, const void *gate, long long ldg, const void *low, long long ldl, const void *w,
+                      int rank, const float *bc, long long ldbc, const float *bias, const float *a_log, const float *skip, void *out,
+                      long long ldo, float *S, int batch, int inner, int states, int dtype, void *stream);
+
+/* eb_short_conv of one token per sequence: earlier inputs come from the ring, this one goes there. */
+EB_API int eb_short_conv_step(const void *x, long long ldx, const void *w, const void *b, void *out, long long ldo, int batch, int channels,
+                       int taps, const int32_t *pos_device, const int32_t *first, void *ring, long long ring_batch_stride,
+                       long long ring_ld, int ring_rows, int dtype, void *stream);
 
 /* ---- matrix memory ------------------------------------------------------------------------------ */
 
@@ -685,6 +750,22 @@ EB_API int eb_attention_prefill_biased_tc(const void *q, const void *k, const vo
                             int heads, int kv_group, int q_len, int kv_len, int head_dim, int window, const float *bias_table,
                             int bias_len, int sink, float scale, int dtype, void *stream);
 
+/* eb_attention_prefill_chunk_tc without chunks, with value heads of v_dim (64 or k_dim) and the output times
+ * sigmoid(gate), gate (or NULL) laid out like the output. */
+EB_API int eb_attention_prefill_gated_tc(const void *q, const void *k, const void *v, void *out, const void *gate, long long q_batch_stride,
+                            long long q_row_stride, long long k_batch_stride, long long k_row_stride, long long v_batch_stride,
+                            long long v_row_stride, long long o_batch_stride, long long o_row_stride, long long g_batch_stride,
+                            long long g_row_stride, int batch, int heads, int kv_group, int len, int k_dim, int v_dim,
+                            const int32_t *first, const float *sinks, float scale, int dtype, void *stream);
+
+/* The rule of eb_attention_plain_capped for a prompt on the tensor cores, with a gate as above. */
+EB_API int eb_attention_prefill_capped_tc(const void *q, const void *k, const void *v, void *out, const void *gate, long long q_batch_stride,
+                            long long q_row_stride, long long k_batch_stride, long long k_row_stride, long long v_batch_stride,
+                            long long v_row_stride, long long o_batch_stride, long long o_row_stride, long long g_batch_stride,
+                            long long g_row_stride, int batch, int heads, int kv_group, int len, int k_dim, int v_dim, int window,
+                            int keep, const int32_t *first, const float *slopes, float cap, int sink, float scale, int dtype,
+                            void *stream);
+
 /* Generation step for query heads in groups that share a key / value head: q [batch][heads*head_dim], one
  * row per sequence at position pos (device scalar); k / v rows first[b] .. pos of the cache,
  *   s_j = scale q.k_j - r1[h] ln(1 + r2[h] (pos - j));   out = sum_j exp(s_j) v_j / ([sink] + sum_j exp(s_j)).
@@ -703,6 +784,13 @@ EB_API int eb_attention_group_decode_chunk(const void *q, const void *k, const v
                               long long out_batch_stride, int batch, int heads, int kv_heads, int head_dim, int ring_rows, int chunk,
                               const int32_t *pos_device, const int32_t *first, const float *sinks, float scale, int dtype,
                               int nsplit, void *scratch, size_t scratch_bytes, void *stream);
+/* The rule of eb_attention_plain_capped over a cache of `keep` rows for the first positions and a ring of ring_rows rows
+ * (eb_attention_values fills it), the output times sigmoid(gate), gate (or NULL) [batch][heads*head_dim]. */
+EB_API int eb_attention_group_decode_capped(const void *q, const void *k, const void *v, void *out, const void *gate, long long q_batch_stride,
+                              long long k_batch_stride, long long k_row_stride, long long v_batch_stride, long long v_row_stride,
+                              long long out_batch_stride, long long gate_batch_stride, int batch, int heads, int kv_heads, int head_dim,
+                              int keep, int ring_rows, int window, const int32_t *pos_device, const int32_t *first, const float *slopes,
+                              float cap, int sink, float scale, int dtype, int nsplit, void *scratch, size_t scratch_bytes, void *stream);
 EB_API size_t eb_attention_group_decode_scratch_bytes(int batch, int heads, int kv_heads, int head_dim, int nsplit);
 
 /* Windowed causal attention for any head sizes and fp32 / fp16 / bf16 on the CUDA cores: query row
@@ -727,11 +815,23 @@ EB_API int eb_attention_plain_chunk(const void *q, const void *k, const void *v,
                        int v_dim, int chunk, int ring_rows, const int32_t *pos_device, const int32_t *first, const float *sinks,
                        float scale, int dtype, void *stream);
 
+/* The same with a window that keeps the first positions of a sequence visible, capped scores and a linear bias:
+ * position i sees max(first[b], i - window + 1) .. i and first[b] .. first[b] + keep - 1 (up to itself; window 0: all),
+ *   s = cap tanh(scale q.k / cap) - slopes[h] (i - j)            (cap 0: no cap; slopes NULL: no bias)
+ * and sink != 0 adds one to the softmax denominator.  kept_rows: cache rows in front of the ring which hold the
+ * first `keep` positions of each sequence (keep or 0; 0: position j is always row j mod ring_rows). */
+EB_API int eb_attention_plain_capped(const void *q, const void *k, const void *v, void *out, long long q_batch_stride, long long q_row_stride,
+                       long long q_head_stride, long long k_batch_stride, long long k_row_stride, long long k_head_stride,
+                       long long v_batch_stride, long long v_row_stride, long long v_head_stride, long long o_batch_stride,
+                       long long o_row_stride, long long o_head_stride, int batch, int heads, int kv_group, int q_len, int k_dim,
+                       int v_dim, int window, int keep, int kept_rows, int ring_rows, const int32_t *pos_device, const int32_t *first,
+                       const float *slopes, float cap, int sink, float scale, int dtype, void *stream);
+
 /* Generation step of latent attention with absorbed projections: q [batch][heads * rank] are the
  * queries in latent space, the cached latent row of a position is key and value of every head,
  *   out[b][h] = sum_j softmax_j(scale * q[b][h] . c[b][j]) c[b][j]
  * over the positions max(first[b], pos - window + 1) .. pos (window 0: all), position j in cache row
- * j mod ring_rows.  rank 64, 128, 256, 384 or 512.  Every cache row must hold finite numbers, also
+ * j mod ring_rows.  rank 64, 128, 192, 256, 320, 384 or 512.  Every cache row must hold finite numbers, also
  * those no position has been written to yet (they are multiplied by a weight of exactly 0).
  * nsplit > 1 splits the positions over that many CTAs per (sequence, head tile): 2, 4 or 8 are
  * clusters that merge their parts on chip, any other number merges in a second launch through
@@ -739,6 +839,11 @@ EB_API int eb_attention_plain_chunk(const void *q, const void *k, const void *v,
 EB_API int eb_latent_decode(const void *q, long long q_batch_stride, const void *cache, long long cache_batch_stride,
                      long long cache_row_stride, int ring_rows, void *out, long long out_batch_stride, int batch, int heads,
                      int rank, int window, const int32_t *pos_device, const int32_t *first, float scale, int dtype,
+                     int nsplit, void *scratch, size_t scratch_bytes, void *stream);
+/* sinks (or NULL): exp(sinks[h]) joins the softmax denominator. */
+EB_API int eb_latent_decode_sink(const void *q, long long q_batch_stride, const void *cache, long long cache_batch_stride,
+                     long long cache_row_stride, int ring_rows, void *out, long long out_batch_stride, int batch, int heads,
+                     int rank, int window, const int32_t *pos_device, const int32_t *first, const float *sinks, float scale, int dtype,
                      int nsplit, void *scratch, size_t scratch_bytes, void *stream);
 EB_API size_t eb_latent_decode_scratch_bytes(int batch, int heads, int rank, int nsplit);
 
