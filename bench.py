@@ -862,7 +862,7 @@ def main():
                          "5 = OPT-66B bucketed decode, 2 = BERT-large block on the kernel API")
     ap.add_argument("--layers", type=int, default=0, help="debug: fewer layers (marks the line as reduced)")
     ap.add_argument("--new-tokens", type=int, default=0, help="debug: fewer generation steps (marks the line as reduced)")
-    ap.add_argument("--design", choices=["tulezen", "mutolix", "moponex"], help="instead of a configuration: throughput and kernel table of this decoder at "
+    ap.add_argument("--design", choices=["tulezen", "mutolix", "moponex", "tupidra"], help="instead of a configuration: throughput and kernel table of this decoder at "
                     "sizes like a real model's layers, beside an OPT-shaped model of equal size")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
     ap.add_argument("--no-check", action="store_true", help="skip the verification against the oracle")

@@ -166,10 +166,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   const int jwin = jmin, kept_tile = first / kKeys;
   if (CAPPED && p.keep > 0 && p.window > 0 && nmax > 0) {
     const int kept = min((min(first + p.keep, p.Sk) - 1) / kKeys + 1, jmin) - kept_tile;
-    if (kept > 0) {
-      jmin -= kept;
-      ks[0] = ks[1] = jmin;
-    }
+    jmin -= max(kept, 0);
+    ks[0] = ks[1] = jmin;
   }
   auto tile_of = [&](int j) { return CAPPED && j < jwin ? kept_tile + j - jmin : j; };
 
@@ -651,8 +649,9 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   EB_REQUIRE(kv_len >= q_len || !causal, "attention_prefill: causal attention needs kv_len >= q_len");
   EB_REQUIRE(scale > 0.f, "attention_prefill: the scale must be positive");
   EB_REQUIRE(window >= 0 && (window == 0 || causal), "attention_prefill: a window needs the causal mask");
-  cudaStream_t st = as_stream(stream);
+  EB_REQUIRE(!capped || (capped->keep >= 0 && capped->cap >= 0.f && !mask && !bias && !chunk), "attention_prefill: bad capped form");
   EB_REQUIRE(!gate || (aligned16(gate) && g_batch_stride % 8 == 0 && g_row_stride % 8 == 0), "attention_prefill: the gate's rows start on 16-byte boundaries");
+  cudaStream_t st = as_stream(stream);
   const long long hd = (long long)heads * head_dim, hkd = hd / kv_group, hvd = (long long)heads / kv_group * v_dim;
   CUtensorMap mq, mk, mv;
   int rc;
@@ -669,7 +668,6 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   p.sinks = sinks; p.chunk = chunk; p.first = first;
   p.gate = gate; p.g_bs = g_batch_stride; p.g_rs = g_row_stride;
   if (capped) {
-    EB_REQUIRE(capped->keep >= 0 && capped->cap >= 0.f && !mask && !bias && !chunk, "attention_prefill: bad capped form");
     p.keep = capped->keep; p.slopes = capped->slopes;
     p.cap_log2 = capped->cap * kLog2eTc; p.cap_scale = capped->cap > 0.f ? scale / capped->cap : 0.f;
   }

@@ -203,6 +203,23 @@ __device__ __forceinline__ void tcgen05_mma_f16(uint32_t d_tmem, uint64_t a_desc
       ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
       : "memory");
 }
+// The same as calls of a whole warp with warp-uniform operands, of which one elected lane acts: descriptors and addresses
+// stay in uniform registers.  In a branch that only one lane takes every operand is moved there first, and those
+// moves set the pace of the weight stream (0.37 us per k-block whatever the tile's width).
+__device__ __forceinline__ void tcgen05_commit_warp(uint32_t bar) {
+  asm volatile(
+      "{\n\t.reg .pred q;\n\telect.sync _|q, 0xffffffff;\n\t"
+      "@q tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];\n\t}" ::"r"(bar)
+      : "memory");
+}
+__device__ __forceinline__ void tcgen05_mma_f16_warp(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\telect.sync _|q, 0xffffffff;\n\t"
+      "setp.ne.b32 p, %4, 0;\n\t"
+      "@q tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+      ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(accumulate)
+      : "memory");
+}
 __device__ __forceinline__ void tmem_ld16(uint32_t taddr, float *v) {
   uint32_t r[16];
   asm volatile(
@@ -474,37 +491,35 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
     }
     }   // mover lanes
   } else if (warp == 1) {
-    // ---------------- MMA issuer ----------------
+    // ---------------- MMA issuer (whole warp, every decision uniform over it) ----------------
     griddep_wait();
-    if (lane == 0) {
-      Scheduler<BN, SWAP> sched(p);
-      Segment s;
-      int stage = 0, acc = 0;
-      uint32_t phase = 0, acc_phase = 0;
-      bool ok = true;
-      while (ok && sched.next(s)) {
-        if (!mbar_wait(tempty_bar + 8 * acc, acc_phase ^ 1u, abort_flag, 2)) break;
+    Scheduler<BN, SWAP> sched(p);
+    Segment s;
+    int stage = 0, acc = 0;
+    uint32_t phase = 0, acc_phase = 0;
+    bool ok = true;
+    while (ok && sched.next(s)) {
+      if (!__all_sync(0xffffffffu, mbar_wait(tempty_bar + 8 * acc, acc_phase ^ 1u, abort_flag, 2))) break;
+      tcgen05_fence_after();
+      const uint32_t d_tmem = tmem_base + acc * BN;
+      for (int sk = s.sk0; sk < s.sk1; ++sk) {
+        if (!__all_sync(0xffffffffu, mbar_wait(full_bar + 8 * stage, phase, abort_flag, 3))) { ok = false; break; }
         tcgen05_fence_after();
-        const uint32_t d_tmem = tmem_base + acc * BN;
-        for (int sk = s.sk0; sk < s.sk1; ++sk) {
-          if (!mbar_wait(full_bar + 8 * stage, phase, abort_flag, 3)) { ok = false; break; }
-          tcgen05_fence_after();
-          for (int j = 0; j < kpb && sk * kpb + j < p.kblocks; ++j) {
-            const uint32_t st_addr = tiles_addr + stage * stage_bytes;
-            const uint64_t a_desc = make_smem_desc(st_addr + j * lane_bytes), b_desc = make_smem_desc(st_addr + col_base + j * kColBytes);
+        for (int j = 0; j < kpb && sk * kpb + j < p.kblocks; ++j) {
+          const uint32_t st_addr = tiles_addr + stage * stage_bytes;
+          const uint64_t a_desc = make_smem_desc(st_addr + j * lane_bytes), b_desc = make_smem_desc(st_addr + col_base + j * kColBytes);
 #pragma unroll
-            for (int k = 0; k < kBlockK / kUmmaK; ++k) {
-              // advancing 16 elements along K inside the swizzle atom = +32 bytes = +2 in the address field
-              tcgen05_mma_f16(d_tmem, a_desc + 2 * k, b_desc + 2 * k, kIdesc, (sk > s.sk0 || j > 0 || k > 0) ? 1u : 0u);
-            }
+          for (int k = 0; k < kBlockK / kUmmaK; ++k) {
+            // advancing 16 elements along K inside the swizzle atom = +32 bytes = +2 in the address field
+            tcgen05_mma_f16_warp(d_tmem, a_desc + 2 * k, b_desc + 2 * k, kIdesc, (sk > s.sk0 || j > 0 || k > 0) ? 1u : 0u);
           }
-          tcgen05_commit(empty_bar + 8 * stage);   // frees the stage once these MMAs have read it
-          if (++stage == stages) { stage = 0; phase ^= 1u; }
         }
-        if (!ok) break;
-        tcgen05_commit(tfull_bar + 8 * acc);        // accumulator complete
-        if (++acc == 2) { acc = 0; acc_phase ^= 1u; }
+        tcgen05_commit_warp(empty_bar + 8 * stage);   // frees the stage once these MMAs have read it
+        if (++stage == stages) { stage = 0; phase ^= 1u; }
       }
+      if (!ok) break;
+      tcgen05_commit_warp(tfull_bar + 8 * acc);        // accumulator complete
+      if (++acc == 2) { acc = 0; acc_phase ^= 1u; }
     }
   } else {
     // ---------------- epilogue (warps 2..5) ----------------
@@ -1531,19 +1546,40 @@ static int gemm_impl(const void *A, long long lda, const void *W, long long ldw,
   }
   p.lane_rows = M; p.col_rows = N;
   const long long lane_tiles = (M + kLanes - 1) / kLanes;
-  const bool wide = lane_tiles * ((N + 255) / 256) >= sm_count();   // enough 128x256 tiles to fill the machine
-  const int bn = wide ? 256 : 128;
+  // Tile width: a k-block costs a CTA about 0.45 / 0.30 / 0.23 / 0.19 us with 256 / 128 / 64 / 32 columns (2, 2 and 3 k-blocks
+  // per stage for the narrow ones, whose pace is the hand-over of a stage), and the tiles come in waves of one per
+  // SM.  What a row's result is does not depend on the choice.
+  struct Form { int bn, kpb, stages; float us; };
+  constexpr Form forms[] = {{256, 1, 4, 0.45f}, {128, 2, 3, 0.30f}, {64, 2, 4, 0.23f}, {32, 3, 3, 0.19f}};
+  auto waves = [&](int cols) { return (lane_tiles * ((N + cols - 1) / cols) + sm_count() - 1) / sm_count(); };
+  Form form = forms[0];
+  if (p.rs) {                                          // (its epilogue turns 64 columns around behind 1-block stages)
+    if (lane_tiles * ((N + 255) / 256) < sm_count()) form = {128, 1, 6, 0.f};
+  } else {
+    float best = 0.f;
+    for (const Form &f : forms) {
+      const float us = (float)waves(f.bn) * ((float)p.kblocks * f.us + 2.f);
+      if (f.bn == 256 || us < best) { best = us; form = f; }
+    }
+  }
+  const int bn = form.bn;
   const long long tiles = lane_tiles * ((N + bn - 1) / bn);
   const int grid = (int)(tiles < sm_count() ? tiles : sm_count());
-  p.stages = wide ? 4 : 6;
-  p.kpb = 1;
+  p.kpb = form.kpb;
+  p.stages = form.stages;
   // (+ 18 KB behind the stages: the staging rows of the reduce-scatter epilogue)
-  const size_t smem = kBarrierBytes + 1024 + (size_t)p.stages * (kLanes * 128 + bn * 128) + (p.rs ? 4 * 32 * 72 * 2 : 0);
+  const size_t smem = kBarrierBytes + 1024 + (size_t)p.stages * p.kpb * (kLanes * 128 + bn * 128) + (p.rs ? 4 * 32 * 72 * 2 : 0);
   if ((rc = make_map(&tl, A, dtype, M, K, lda, kLanes))) return rc;
   if ((rc = make_map(&tc, W, dtype, N, K, ldw, bn))) return rc;
   if (bn == 256)
     return dtype == EB_F16 ? launch<__half, 256, false>(tl, tc, p, grid, smem, st)
                            : launch<__nv_bfloat16, 256, false>(tl, tc, p, grid, smem, st);
+  if (bn == 64)
+    return dtype == EB_F16 ? launch<__half, 64, false>(tl, tc, p, grid, smem, st)
+                           : launch<__nv_bfloat16, 64, false>(tl, tc, p, grid, smem, st);
+  if (bn == 32)
+    return dtype == EB_F16 ? launch<__half, 32, false>(tl, tc, p, grid, smem, st)
+                           : launch<__nv_bfloat16, 32, false>(tl, tc, p, grid, smem, st);
   return dtype == EB_F16 ? launch<__half, 128, false>(tl, tc, p, grid, smem, st)
                          : launch<__nv_bfloat16, 128, false>(tl, tc, p, grid, smem, st);
 }

@@ -7,9 +7,9 @@
 // no product to put on the tensor cores: the exponentials set the pace (one per channel, state and token on
 // the special-function units).
 //
-//   scan          a prompt: a channel's states over the lanes of a group, 4 or 8 per lane in registers, 32 tokens at
-//                 a time through shared memory; steps, products dt x and the gate are formed by the whole CTA
-//                 around each chunk, the sums over a group's lanes are taken for four tokens together.
+//   scan          a prompt: a channel's states over the lanes of a group, a few per lane in registers, up to 32
+//                 tokens at a time through shared memory; steps, products dt x and the gate are formed by the whole
+//                 CTA around each chunk, the sums over a group's lanes are taken for four tokens together.
 //   scan_step     one token per sequence: the step's projection (dt_rank numbers per channel), the pass over the
 //                 state and the gate in one launch; a CTA keeps its channels for several sequences, so that
 //                 their projection is read once.
@@ -18,20 +18,20 @@
 // State, steps, decays, B and C are fp32.  (Compiled without fast math: decays add up over a sequence.)
 #include "common.cuh"
 #include "decay_gates.cuh"
+#include "packed_math.cuh"
 
 namespace eb {
 namespace {
 
 constexpr float kLog2eScan = 1.4426950408889634f;
 
-__device__ __forceinline__ float pow2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 template <typename T> __device__ __forceinline__ float gate_silu(float x) { return silu_fast(x); }
 template <> __device__ __forceinline__ float gate_silu<float>(float x) { return x / (1.f + expf(-x)); }
+
+// log(1 + exp(x)); 16-bit models take the special-function unit's exponential (2^-22 of the result)
+template <typename T> __device__ __forceinline__ float step_size(float x) { return fmaxf(x, 0.f) + log1p_unit(ex2(-fabsf(x) * kLog2eScan)); }
+template <> __device__ __forceinline__ float step_size<float>(float x) { return softplus(x); }
 
 template <typename T> struct Two;
 template <> struct Two<float> {
@@ -90,22 +90,22 @@ template <int LPC, typename F> __device__ __forceinline__ void group_sum4(float 
   }
 }
 
-// NS: states per lane; LPC: lanes per channel (NS * LPC >= states)
-template <int LPC> constexpr int scan_threads = LPC * 8 > 128 ? LPC * 8 : 128;
+// NS: states per lane; LPC: lanes per channel, or per pair of them (CPT 2); NS * LPC >= states
+template <int LPC, int CPT> constexpr int scan_threads = LPC * 8 / CPT > 128 ? LPC * 8 / CPT : 128;
 
-template <typename T, int NS, int LPC>
-__global__ void __launch_bounds__(scan_threads<LPC>) selective_scan_kernel(const SelScanParams p) {
+template <typename T, int NS, int LPC, int CPT>
+__global__ void __launch_bounds__(scan_threads<LPC, CPT>) selective_scan_kernel(const SelScanParams p) {
   using W = Two<T>;
   using R = typename W::R;
-  constexpr int kSelThreads = scan_threads<LPC>, kScanTokens = LPC == 1 ? 8 : LPC == 2 ? 16 : NS * LPC <= 32 ? 32 : NS * LPC <= 64 ? 16 : 8;
-  constexpr int CH = kSelThreads / LPC, NP = NS * LPC;            // channels of this CTA, states with padding
-  constexpr int kPairs = CH / 2, kRowsPass = kSelThreads / kPairs;       // elementwise: thread = two channels of a token,
-  constexpr int kPasses = kScanTokens > kRowsPass ? kScanTokens / kRowsPass : 1;                          // this often per chunk
-  constexpr int kBcVec = kScanTokens * 2 * NP / 4, kBcIters = (kBcVec + kSelThreads - 1) / kSelThreads;
-  static_assert(CH >= 2 && (kPasses == 1 || kRowsPass * kPasses == kScanTokens), "a chunk is whole passes");
-  __shared__ __align__(16) float2 s_dt[2][kScanTokens][CH];       // (step, step * input)
-  __shared__ __align__(16) float s_bc[2][kScanTokens][2 * NP];
-  __shared__ float s_y[2][kScanTokens][CH + 1];
+  constexpr int kThreads = scan_threads<LPC, CPT>, CH = CPT * kThreads / LPC, NP = NS * LPC;        // channels of this CTA, states with padding
+  constexpr int kTokens = CH * CPT >= 128 ? 8 : CH >= 64 ? 16 : NP <= 32 ? 32 : NP <= 64 ? 16 : 8;
+  constexpr int kPairs = CH / 2, kRowsPass = kThreads / kPairs;   // elementwise: thread = two channels of a token,
+  constexpr int kPasses = kTokens > kRowsPass ? kTokens / kRowsPass : 1;                                  // this often per chunk
+  constexpr int kBcVec = kTokens * 2 * NP / 4, kBcIters = (kBcVec + kThreads - 1) / kThreads;
+  static_assert(kPasses == 1 || kRowsPass * kPasses == kTokens, "a chunk is whole passes");
+  __shared__ __align__(16) float4 s_dt[2][kTokens][kPairs];       // of two channels: step, step * input
+  __shared__ __align__(16) float s_bc[2][kTokens][2 * NP];
+  __shared__ __align__(8) float s_y[2][kTokens][CH + 2];
 
   griddep_wait();
   griddep_launch();
@@ -114,7 +114,7 @@ __global__ void __launch_bounds__(scan_threads<LPC>) selective_scan_kernel(const
   const long long row0 = (long long)b * p.seq;
   // elementwise role: channels c0 + 2 * pc and the next, tokens pr + kRowsPass * i of a chunk
   const int pc = tid % kPairs, pr = tid / kPairs, ec = c0 + 2 * pc;
-  const bool has_e = ec < p.inner && pr < kScanTokens;            // (inner is even)
+  const bool has_e = ec < p.inner && pr < kTokens;                // (inner is even)
   const float2 bias = has_e ? *reinterpret_cast<const float2 *>(p.bias + ec) : make_float2(0.f, 0.f);
   const float2 skip = has_e ? *reinterpret_cast<const float2 *>(p.skip + ec) : make_float2(0.f, 0.f);
   R xr[kPasses], gr[kPasses];
@@ -134,7 +134,7 @@ __global__ void __launch_bounds__(scan_threads<LPC>) selective_scan_kernel(const
     }
 #pragma unroll
     for (int i = 0; i < kBcIters; ++i) {
-      const int v = tid + i * kSelThreads, t = t0 + v / (2 * NP / 4), n = v % (2 * NP / 4) * 4;     // n: column of the padded row
+      const int v = tid + i * kThreads, t = t0 + v / (2 * NP / 4), n = v % (2 * NP / 4) * 4;        // n: column of the padded row
       const int half = n >= NP, at = n - half * NP;
       bcr[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (v < kBcVec && t < p.seq && at < p.states) bcr[i] = *reinterpret_cast<const float4 *>(p.bc + (row0 + t) * p.ldbc + half * p.states + at);
@@ -144,77 +144,105 @@ __global__ void __launch_bounds__(scan_threads<LPC>) selective_scan_kernel(const
 #pragma unroll
     for (int i = 0; i < kPasses; ++i) {
       const int r = pr + kRowsPass * i, t = t0 + r;
-      if (r >= kScanTokens) continue;
+      if (r >= kTokens) continue;
       const bool live = t >= first && t < p.seq;
       const float2 x = W::get(xr[i]);
-      const float d0 = live ? softplus(zr[i].x + bias.x) : 0.f, d1 = live ? softplus(zr[i].y + bias.y) : 0.f;
-      *reinterpret_cast<float4 *>(&s_dt[buf][r][2 * pc]) = make_float4(d0, live ? d0 * x.x : 0.f, d1, live ? d1 * x.y : 0.f);
+      const float d0 = live ? step_size<T>(zr[i].x + bias.x) : 0.f, d1 = live ? step_size<T>(zr[i].y + bias.y) : 0.f;
+      s_dt[buf][r][pc] = make_float4(d0, live ? d0 * x.x : 0.f, d1, live ? d1 * x.y : 0.f);
     }
 #pragma unroll
     for (int i = 0; i < kBcIters; ++i) {
-      const int v = tid + i * kSelThreads;
+      const int v = tid + i * kThreads;
       if (v < kBcVec) *reinterpret_cast<float4 *>(&s_bc[buf][v / (2 * NP / 4)][v % (2 * NP / 4) * 4]) = bcr[i];
     }
   };
 
-  // scan role: channel c, states sub * NS ..
-  const int ch = tid / LPC, sub = tid % LPC, c = c0 + ch;
-  float A[NS], S[NS];
+  // scan role: CPT channels from c on, states sub * NS ..
+  const int cp = tid / LPC, sub = tid % LPC, c = c0 + CPT * cp;
+  float A[CPT][NS], S[CPT][NS];
 #pragma unroll
-  for (int n = 0; n < NS; ++n) {
-    const int s = sub * NS + n;
-    A[n] = c < p.inner && s < p.states ? -expf(p.a_log[(long long)c * p.states + s]) * kLog2eScan : 0.f;
-    S[n] = 0.f;
-  }
+  for (int k = 0; k < CPT; ++k)
+#pragma unroll
+    for (int n = 0; n < NS; ++n) {
+      const int s = sub * NS + n;
+      A[k][n] = c < p.inner && s < p.states ? -expf(p.a_log[(long long)(c + k) * p.states + s]) * kLog2eScan : 0.f;
+      S[k][n] = 0.f;
+    }
   fetch(0);
   prepare(0, 0);
   __syncthreads();
-  const int chunks = (p.seq + kScanTokens - 1) / kScanTokens;
-  for (int k = 0; k < chunks; ++k) {
-    const int buf = k & 1, t0 = k * kScanTokens;
+  const int chunks = (p.seq + kTokens - 1) / kTokens;
+  for (int j = 0; j < chunks; ++j) {
+    const int buf = j & 1, t0 = j * kTokens;
     R xk[kPasses], gk[kPasses];
 #pragma unroll
     for (int i = 0; i < kPasses; ++i) { xk[i] = xr[i]; gk[i] = gr[i]; }
-    const bool more = k + 1 < chunks;
-    if (more) fetch(t0 + kScanTokens);
+    const bool more = j + 1 < chunks;
+    if (more) fetch(t0 + kTokens);
 #pragma unroll 2
-    for (int t = 0; t < kScanTokens; t += 4) {
-      float y[4];
+    for (int t = 0; t < kTokens; t += 4) {
+      float y[CPT][4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float2 d = s_dt[buf][t + i][ch];
+        float d[2 * CPT];                            // (step, step * input) of the channels
+        if constexpr (CPT == 2) {
+          const float4 v = s_dt[buf][t + i][cp];
+          d[0] = v.x; d[1] = v.y; d[2] = v.z; d[3] = v.w;
+        } else {
+          const float2 v = reinterpret_cast<const float2 *>(s_dt[buf][t + i])[cp];
+          d[0] = v.x; d[1] = v.y;
+        }
         const float *B = &s_bc[buf][t + i][sub * NS], *C = B + NP;
-        float acc = 0.f;
+        float acc[CPT][2] = {}, bb[4], cc[4];
 #pragma unroll
-        for (int n4 = 0; n4 < NS; n4 += 4) {
-          const float4 bv = *reinterpret_cast<const float4 *>(B + n4), cv = *reinterpret_cast<const float4 *>(C + n4);
-          const float bb[4] = {bv.x, bv.y, bv.z, bv.w}, cc[4] = {cv.x, cv.y, cv.z, cv.w};
+        for (int n = 0; n < NS; n += 2) {
+          float2 bv, cv;
+          if (NS % 4 == 0 && n % 4 == 0) {
+            const float4 b4 = *reinterpret_cast<const float4 *>(B + n), c4 = *reinterpret_cast<const float4 *>(C + n);
+            bb[0] = b4.x; bb[1] = b4.y; bb[2] = b4.z; bb[3] = b4.w;
+            cc[0] = c4.x; cc[1] = c4.y; cc[2] = c4.z; cc[3] = c4.w;
+          }
+          if (NS % 4 == 0) {
+            bv = make_float2(bb[n % 4], bb[n % 4 + 1]);
+            cv = make_float2(cc[n % 4], cc[n % 4 + 1]);
+          } else {
+            bv = *reinterpret_cast<const float2 *>(B + n);
+            cv = *reinterpret_cast<const float2 *>(C + n);
+          }
 #pragma unroll
-          for (int n = 0; n < 4; ++n) {
-            S[n4 + n] = fmaf(pow2(d.x * A[n4 + n]), S[n4 + n], d.y * bb[n]);
-            acc = fmaf(S[n4 + n], cc[n], acc);
+          for (int k = 0; k < CPT; ++k) {
+            float *s = S[k] + n, e0, e1, b0, b1;
+            mul2(e0, e1, d[2 * k], d[2 * k], A[k][n], A[k][n + 1]);
+            mul2(b0, b1, d[2 * k + 1], d[2 * k + 1], bv.x, bv.y);
+            fma2(s[0], s[1], ex2(e0), ex2(e1), s[0], s[1], b0, b1);
+            fma2(acc[k][0], acc[k][1], s[0], s[1], cv.x, cv.y, acc[k][0], acc[k][1]);
           }
         }
-        y[i] = acc;
+#pragma unroll
+        for (int k = 0; k < CPT; ++k) y[k][i] = acc[k][0] + acc[k][1];
       }
-      group_sum4<LPC>(y, sub, [&](int i, float v) { s_y[buf][t + i][ch] = v; });
+#pragma unroll
+      for (int k = 0; k < CPT; ++k) group_sum4<LPC>(y[k], sub, [&](int i, float v) { s_y[buf][t + i][CPT * cp + k] = v; });
     }
-    if (more) prepare(t0 + kScanTokens, buf ^ 1);
+    if (more) prepare(t0 + kTokens, buf ^ 1);
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < kPasses; ++i) {
       const int r = pr + kRowsPass * i, t = t0 + r;
-      if (t >= p.seq || !has_e) continue;
-      const float2 x = W::get(xk[i]), g = W::get(gk[i]);
-      const float y0 = fmaf(skip.x, x.x, s_y[buf][r][2 * pc]), y1 = fmaf(skip.y, x.y, s_y[buf][r][2 * pc + 1]);
-      *reinterpret_cast<R *>(reinterpret_cast<T *>(p.out) + (row0 + t) * p.ldo + ec) = W::put(y0 * gate_silu<T>(g.x), y1 * gate_silu<T>(g.y));
+      if (t >= p.seq || !has_e || r >= kTokens) continue;
+      const float2 x = W::get(xk[i]), g = W::get(gk[i]), y = *reinterpret_cast<const float2 *>(&s_y[buf][r][2 * pc]);
+      *reinterpret_cast<R *>(reinterpret_cast<T *>(p.out) + (row0 + t) * p.ldo + ec) =
+          W::put(fmaf(skip.x, x.x, y.x) * gate_silu<T>(g.x), fmaf(skip.y, x.y, y.y) * gate_silu<T>(g.y));
     }
   }
   if (c < p.inner) {
-    float *dst = p.S + ((long long)b * p.inner + c) * p.states + sub * NS;
 #pragma unroll
-    for (int n = 0; n < NS; n += 4)
-      if (sub * NS + n < p.states) *reinterpret_cast<float4 *>(dst + n) = make_float4(S[n], S[n + 1], S[n + 2], S[n + 3]);
+    for (int k = 0; k < CPT; ++k) {
+      float *dst = p.S + ((long long)b * p.inner + c + k) * p.states + sub * NS;
+#pragma unroll
+      for (int n = 0; n < NS; n += 2)
+        if (sub * NS + n < p.states) *reinterpret_cast<float2 *>(dst + n) = make_float2(S[k][n], S[k][n + 1]);
+    }
   }
 }
 
@@ -268,14 +296,14 @@ __global__ void __launch_bounds__(kSelStepThreads) selective_step_kernel(const S
     for (int r = sub * 8; r < p.rank; r += LPC * 8) z = dot8<T>(w + r, low + r, z);
 #pragma unroll
     for (int o = LPC / 2; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-    const float dt = softplus(z + bias), dx = dt * x;
+    const float dt = step_size<T>(z + bias), dx = dt * x;
     float y = 0.f;
 #pragma unroll
     for (int n = 0; n < NS / 4; ++n) {
-      S4[n].x = fmaf(pow2(dt * A[4 * n]), S4[n].x, dx * B4[n].x);
-      S4[n].y = fmaf(pow2(dt * A[4 * n + 1]), S4[n].y, dx * B4[n].y);
-      S4[n].z = fmaf(pow2(dt * A[4 * n + 2]), S4[n].z, dx * B4[n].z);
-      S4[n].w = fmaf(pow2(dt * A[4 * n + 3]), S4[n].w, dx * B4[n].w);
+      S4[n].x = fmaf(ex2(dt * A[4 * n]), S4[n].x, dx * B4[n].x);
+      S4[n].y = fmaf(ex2(dt * A[4 * n + 1]), S4[n].y, dx * B4[n].y);
+      S4[n].z = fmaf(ex2(dt * A[4 * n + 2]), S4[n].z, dx * B4[n].z);
+      S4[n].w = fmaf(ex2(dt * A[4 * n + 3]), S4[n].w, dx * B4[n].w);
       y = fmaf(S4[n].x, C4[n].x, fmaf(S4[n].y, C4[n].y, fmaf(S4[n].z, C4[n].z, fmaf(S4[n].w, C4[n].w, y))));
       if (mine && sub * NS + 4 * n < p.states) *reinterpret_cast<float4 *>(Sp + 4 * n) = S4[n];
     }
@@ -324,29 +352,36 @@ __global__ void __launch_bounds__(128) conv_step_kernel(const ConvStepParams p) 
   *reinterpret_cast<R *>(reinterpret_cast<T *>(p.out) + b * p.ldo + c) = W::put(gate_silu<T>(acc.x), gate_silu<T>(acc.y));
 }
 
-template <typename T, int NS, int LPC> int launch_scan(const SelScanParams &p, bool step, cudaStream_t st) {
-  if (!step) {
-    constexpr int CH = scan_threads<LPC> / LPC;
-    launch_pdl(selective_scan_kernel<T, NS, LPC>, dim3((p.inner + CH - 1) / CH, p.batch), dim3(scan_threads<LPC>), 0, st, p);
-    return check_launch("selective_scan");
-  }
+template <typename T, int NS, int LPC, int CPT> int launch_scan(const SelScanParams &p, cudaStream_t st) {
+  constexpr int kThreads = scan_threads<LPC, CPT>, CH = CPT * kThreads / LPC;
+  launch_pdl(selective_scan_kernel<T, NS, LPC, CPT>, dim3((p.inner + CH - 1) / CH, p.batch), dim3(kThreads), 0, st, p);
+  return check_launch("selective_scan");
+}
+
+template <typename T, int NS, int LPC> int launch_step(SelScanParams p, cudaStream_t st) {
   constexpr int CH = kSelStepThreads / LPC;
-  SelScanParams q = p;
   const int tiles = (p.inner + CH - 1) / CH;
-  q.per_cta = 1;
-  while (q.per_cta < 8 && (long long)tiles * ((p.batch + 2 * q.per_cta - 1) / (2 * q.per_cta)) >= 4ll * sm_count()) q.per_cta *= 2;
-  launch_pdl(selective_step_kernel<T, NS, LPC>, dim3(tiles, (p.batch + q.per_cta - 1) / q.per_cta), dim3(kSelStepThreads), 0, st, q);
+  p.per_cta = 1;
+  while (p.per_cta < 8 && (long long)tiles * ((p.batch + 2 * p.per_cta - 1) / (2 * p.per_cta)) >= 4ll * sm_count()) p.per_cta *= 2;
+  launch_pdl(selective_step_kernel<T, NS, LPC>, dim3(tiles, (p.batch + p.per_cta - 1) / p.per_cta), dim3(kSelStepThreads), 0, st, p);
   return check_launch("selective_step");
 }
 
+// 16 states: with few warps the machine wants many short chains, with plenty fewer loads of B and C per state
+template <typename T> int launch_scan16(const SelScanParams &p, cudaStream_t st) {
+  const double warps = (double)p.batch * p.inner * 16 / 128 / (4.0 * sm_count());      // per scheduler, four states per thread
+  if (warps < 1.5) return launch_scan<T, 2, 8, 1>(p, st);
+  return warps < 8.0 ? launch_scan<T, 2, 8, 2>(p, st) : launch_scan<T, 4, 4, 2>(p, st);
+}
+
 template <typename T> int launch_sel(const SelScanParams &p, bool step, cudaStream_t st) {
-  if (p.states <= 4) return launch_scan<T, 4, 1>(p, step, st);
-  if (p.states <= 8) return launch_scan<T, 4, 2>(p, step, st);
-  if (p.states <= 16) return launch_scan<T, 4, 4>(p, step, st);
-  if (p.states <= 32) return launch_scan<T, 4, 8>(p, step, st);
-  if (p.states <= 64) return launch_scan<T, 8, 8>(p, step, st);
-  if (p.states <= 128) return launch_scan<T, 8, 16>(p, step, st);
-  return launch_scan<T, 8, 32>(p, step, st);
+  if (p.states <= 4) return step ? launch_step<T, 4, 1>(p, st) : launch_scan<T, 4, 1, 1>(p, st);
+  if (p.states <= 8) return step ? launch_step<T, 4, 2>(p, st) : launch_scan<T, 2, 4, 1>(p, st);
+  if (p.states <= 16) return step ? launch_step<T, 4, 4>(p, st) : launch_scan16<T>(p, st);
+  if (p.states <= 32) return step ? launch_step<T, 4, 8>(p, st) : launch_scan<T, 4, 8, 1>(p, st);
+  if (p.states <= 64) return step ? launch_step<T, 8, 8>(p, st) : launch_scan<T, 4, 16, 1>(p, st);
+  if (p.states <= 128) return step ? launch_step<T, 8, 16>(p, st) : launch_scan<T, 8, 16, 1>(p, st);
+  return step ? launch_step<T, 8, 32>(p, st) : launch_scan<T, 8, 32, 1>(p, st);
 }
 
 int check_scan(const char *what, const SelScanParams &p) {

@@ -8,16 +8,14 @@
 // fp32 table k[j] = w (c_j + [j is the current token]) per sublayer.  Stream, sums and taps are fp32; u is
 // rounded only where it goes to the ring.
 //
-// Prompt: a CTA walks kStrip tokens of a sequence, a thread owning 4 columns (or several packs of 4); the last
-// taps - 1 rows u stay in its registers.  The rows in front of the strip are recomputed (so x is written to
-// another buffer than it is read from); four tokens share one reduction.  Step: one CTA per sequence, the
-// rows in front from the ring.
+// Prompt: a CTA walks a strip of a sequence's tokens, a thread owning 4 columns (or several packs of 4); the last
+// rows u stay in its registers.  The rows in front of the strip are recomputed (so x is written to
+// another buffer than it is read from); a group of tokens shares one reduction.  Step: one CTA per sequence,
+// the rows in front from the ring.
 #include "common.cuh"
 
 namespace eb {
 namespace {
-
-constexpr int kGroup = 4;                          // tokens per reduction
 
 struct StreamConvParams {
   const void *src;                                 // embedding rows (T) or null
@@ -64,26 +62,72 @@ __device__ __forceinline__ float sum4(const float (&v)[4], int lane) {
   return s;
 }
 
-// PACKS: packs of 4 columns per thread.
-template <typename T, int TAPS, int PACKS, bool STEP>
+__device__ __forceinline__ void copy_async(void *dst, const void *src, int bytes, bool live) {
+  const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+  const int n = live ? bytes : 0;                  // the rest is filled with zeros
+  if (bytes == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(n) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(d), "l"(src), "r"(n) : "memory");
+}
+
+// The sums of part[0 .. warps) over all warps, in every thread.
+__device__ __forceinline__ void total4(const float4 *part, int warps, int lane, float (&total)[4]) {
+  const float4 q = lane < warps ? part[lane] : make_float4(0.f, 0.f, 0.f, 0.f);
+  const float v[4] = {q.x, q.y, q.z, q.w}, s = sum4(v, lane);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) total[i] = __shfl_sync(0xffffffffu, s, 8 * i);
+}
+
+// A prompt.  Every thread copies the columns of the next group of tokens that it will need itself into shared memory
+// while it works on this one; rows are read from there twice, for the sums and for the norm.  PACKS: packs of 4
+// columns per thread, G: tokens per group.
+template <typename T, int TAPS, int PACKS, int G>
 __global__ void __launch_bounds__(1024) stream_conv_kernel(const StreamConvParams p) {
-  constexpr int kBack = TAPS - 1;
-  constexpr bool kKeep = TAPS <= 4 && PACKS == 1 && !STEP;       // the tap tables stay in registers
+  constexpr int kBack = TAPS - 1, kLead = (kBack + G - 1) / G * G;
+  constexpr bool kKeep = TAPS <= 4 && PACKS == 1;                // the tap tables stay in registers
   __shared__ float4 part[2][32];
+  extern __shared__ __align__(16) uint8_t sm[];
   griddep_wait();
   griddep_launch();
-  const int b = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-  const int pos = STEP ? max(*p.pos_dev, 0) : 0;
-  const int first = p.first ? p.first[b] : 0;
-  const int t0 = STEP ? pos : blockIdx.x * p.strip, t1 = STEP ? pos + 1 : min(p.seq, t0 + p.strip);
-  const long long row0 = STEP ? (long long)b - pos : (long long)b * p.seq;          // row of token t: row0 + t
+  const int b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, n = blockDim.x;
+  const int first = p.first ? p.first[b] : 0, t0 = blockIdx.x * p.strip, t1 = min(p.seq, t0 + p.strip);
+  const long long row0 = (long long)b * p.seq;
+  float *sx = reinterpret_cast<float *>(sm);                     // [2][G][PACKS][n] packs of x, or of src
+  T *sy = reinterpret_cast<T *>(sm + (size_t)2 * G * PACKS * n * 16);
+  auto slot = [&](int st, int i, int k) { return (((st * G + i) * PACKS + k) * n + tid) * 4; };
   int col[PACKS];
   bool on[PACKS];
 #pragma unroll
   for (int k = 0; k < PACKS; ++k) {
-    col[k] = (threadIdx.x + k * blockDim.x) * 4;
+    col[k] = (tid + k * n) * 4;
     on[k] = col[k] < p.n2;
   }
+  auto live = [&](int t) { return t >= t0 - kBack && t >= 0 && t < t1; };
+  auto fetch = [&](int g0, int st) {
+#pragma unroll
+    for (int i = 0; i < G; ++i) {
+      const int t = g0 + i;
+#pragma unroll
+      for (int k = 0; k < PACKS; ++k) {
+        const bool ok = live(t) && on[k];
+        const long long at = ok ? row0 + t : row0;
+        const int c = on[k] ? col[k] : 0;
+        if (p.src) copy_async(sx + slot(st, i, k), reinterpret_cast<const T *>(p.src) + at * p.lds + c, 4 * sizeof(T), ok);
+        else copy_async(sx + slot(st, i, k), p.x_in + at * p.ldx + c, 16, ok);
+        if (p.y) copy_async(sy + slot(st, i, k), reinterpret_cast<const T *>(p.y) + at * p.ldy + c, 4 * sizeof(T), ok);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  auto row = [&](int st, int i, int k, float (&x)[4]) {
+    if (p.src) ld4<T>(reinterpret_cast<const T *>(sx + slot(st, i, k)), x);
+    else ld4<float>(sx + slot(st, i, k), x);
+    if (p.y) {
+      float y[4];
+      ld4<T>(sy + slot(st, i, k), y);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[e] += y[e];
+    }
+  };
   T *ring = reinterpret_cast<T *>(p.ring) + b * p.ring_bs;
   float c1[kKeep ? TAPS : 1][4], c2[kKeep ? TAPS : 1][4];
   if constexpr (kKeep) {
@@ -94,55 +138,36 @@ __global__ void __launch_bounds__(1024) stream_conv_kernel(const StreamConvParam
         if (p.h2) ld4<float>(p.k2 + (long long)j * p.n2 + col[0], c2[j]);
       }
   }
-  constexpr int G = STEP ? 1 : kGroup;
-  float u[PACKS][kBack + G][4];                      // u[.][kBack + i]: token i of the group
+  float u[PACKS][TAPS][4];                           // the last rows; u[.][kBack]: the current one
 #pragma unroll
   for (int k = 0; k < PACKS; ++k)
 #pragma unroll
-    for (int j = 0; j < kBack; ++j) {
+    for (int j = 0; j < TAPS; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) u[k][j][e] = 0.f;
-      const int t = pos - kBack + j;
-      if (STEP && on[k] && t >= first) ld4<T>(ring + (long long)(t % p.ring_rows) * p.ring_ld + col[k], u[k][j]);
-    }
-  int buf = 0;
-  constexpr int kLead = STEP ? 0 : (kBack + kGroup - 1) / kGroup * kGroup;
+  int st = 0;
+  fetch(t0 - kLead, 0);
 #pragma unroll 1
-  for (int g0 = t0 - kLead; g0 < t1; g0 += G) {
+  for (int g0 = t0 - kLead; g0 < t1; g0 += G, st ^= 1) {
+    if (g0 + G < t1) fetch(g0 + G, st ^ 1);
+    else asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
     float sq[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-    for (int i = 0; i < G; ++i) {
-      const int t = g0 + i;
-      const bool live = t >= t0 - kBack && t >= 0 && t < t1;
+    for (int i = 0; i < G; ++i)
 #pragma unroll
       for (int k = 0; k < PACKS; ++k) {
-        float (&x)[4] = u[k][kBack + i];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) x[e] = 0.f;
-        if (!live || !on[k]) continue;
-        if (p.src) ld4<T>(reinterpret_cast<const T *>(p.src) + (row0 + t) * p.lds + col[k], x);
-        else ld4<float>(p.x_in + (row0 + t) * p.ldx + col[k], x);
-        if (p.y) {
-          float y[4];
-          ld4<T>(reinterpret_cast<const T *>(p.y) + (row0 + t) * p.ldy + col[k], y);
-#pragma unroll
-          for (int e = 0; e < 4; ++e) x[e] += y[e];
-        }
-        if (t >= t0 && (p.src || p.y || p.x_in != p.x_out)) st4<float>(p.x_out + (row0 + t) * p.ldx + col[k], x);
+        float x[4];
+        row(st, i, k, x);
+        if (g0 + i >= t0 && g0 + i < t1 && on[k]) st4<float>(p.x_out + (row0 + g0 + i) * p.ldx + col[k], x);
 #pragma unroll
         for (int e = 0; e < 4; ++e) sq[i] = fmaf(x[e], x[e], sq[i]);
       }
-    }
     const float s = sum4(sq, lane);
-    if ((lane & 7) == 0) reinterpret_cast<float *>(&part[buf][warp])[lane >> 3] = s;
+    if ((lane & 7) == 0) reinterpret_cast<float *>(&part[st][warp])[lane >> 3] = s;
     __syncthreads();
-    float4 tot = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int w = 0; w < warps; ++w) {
-      const float4 q = part[buf][w];
-      tot.x += q.x; tot.y += q.y; tot.z += q.z; tot.w += q.w;
-    }
-    buf ^= 1;
-    const float total[4] = {tot.x, tot.y, tot.z, tot.w};
+    float total[4];
+    total4(part[st], n >> 5, lane, total);
 #pragma unroll
     for (int i = 0; i < G; ++i) {
       const int t = g0 + i;
@@ -151,65 +176,147 @@ __global__ void __launch_bounds__(1024) stream_conv_kernel(const StreamConvParam
 #pragma unroll
       for (int k = 0; k < PACKS; ++k) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) u[k][kBack + i][e] *= r;
+        for (int j = 0; j < kBack; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) u[k][j][e] = u[k][j + 1][e];
+        row(st, i, k, u[k][kBack]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) u[k][kBack][e] *= r;
         if (!out || !on[k]) continue;
-        float a1[4] = {0.f, 0.f, 0.f, 0.f}, a2[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j) {
-          float w[4];
-          if constexpr (!kKeep) ld4<float>(p.k1 + (long long)j * p.n2 + col[k], w);
-#pragma unroll
-          for (int e = 0; e < 4; ++e) a1[e] = fmaf(kKeep ? c1[kKeep ? j : 0][e] : w[e], u[k][i + j][e], a1[e]);
-        }
-        st4<T>(reinterpret_cast<T *>(p.h1) + (row0 + t) * p.ldh + col[k], a1);
-        if (p.h2) {
+        auto conv = [&](const float *table, const float (&kept)[kKeep ? TAPS : 1][4], void *h) {
+          float a[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
           for (int j = 0; j < TAPS; ++j) {
             float w[4];
-            if constexpr (!kKeep) ld4<float>(p.k2 + (long long)j * p.n2 + col[k], w);
+            if constexpr (!kKeep) ld4<float>(table + (long long)j * p.n2 + col[k], w);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) a2[e] = fmaf(kKeep ? c2[kKeep ? j : 0][e] : w[e], u[k][i + j][e], a2[e]);
+            for (int e = 0; e < 4; ++e) a[e] = fmaf(kKeep ? kept[kKeep ? j : 0][e] : w[e], u[k][j][e], a[e]);
           }
-          st4<T>(reinterpret_cast<T *>(p.h2) + (row0 + t) * p.ldh + col[k], a2);
-        }
-        if (STEP || p.seq - t <= p.ring_rows) st4<T>(ring + (long long)(t % p.ring_rows) * p.ring_ld + col[k], u[k][kBack + i]);
+          st4<T>(reinterpret_cast<T *>(h) + (row0 + t) * p.ldh + col[k], a);
+        };
+        conv(p.k1, c1, p.h1);
+        if (p.h2) conv(p.k2, c2, p.h2);
+        if (p.seq - t <= p.ring_rows) st4<T>(ring + (long long)(t % p.ring_rows) * p.ring_ld + col[k], u[k][kBack]);
       }
     }
-#pragma unroll
-    for (int k = 0; k < PACKS; ++k)
-#pragma unroll
-      for (int j = 0; j < kBack; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) u[k][j][e] = u[k][G + j][e];
   }
 }
 
-template <typename T, int TAPS, int PACKS> int launch_packs(StreamConvParams p, int batch, bool step, cudaStream_t st) {
-  const int threads = ((p.n2 / 4 + PACKS - 1) / PACKS + 31) / 32 * 32;
-  if (step) {
-    launch_pdl(stream_conv_kernel<T, TAPS, PACKS, true>, dim3(1, batch), dim3(threads), 0, st, p);
-    return check_launch("stream_conv");
+// One token per sequence.
+template <typename T, int PACKS>
+__global__ void __launch_bounds__(1024) stream_conv_step_kernel(const StreamConvParams p, int taps) {
+  __shared__ float4 part[32];
+  griddep_wait();
+  griddep_launch();
+  const int b = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int first = p.first ? p.first[b] : 0, pos = max(*p.pos_dev, 0);
+  T *ring = reinterpret_cast<T *>(p.ring) + b * p.ring_bs;
+  float x[PACKS][4], sq[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int k = 0; k < PACKS; ++k) {
+    const int col = (tid + k * blockDim.x) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[k][e] = 0.f;
+    if (col >= p.n2) continue;
+    if (p.src) ld4<T>(reinterpret_cast<const T *>(p.src) + b * p.lds + col, x[k]);
+    else ld4<float>(p.x_in + b * p.ldx + col, x[k]);
+    if (p.y) {
+      float y[4];
+      ld4<T>(reinterpret_cast<const T *>(p.y) + b * p.ldy + col, y);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[k][e] += y[e];
+    }
+    st4<float>(p.x_out + b * p.ldx + col, x[k]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) sq[0] = fmaf(x[k][e], x[k][e], sq[0]);
   }
-  // strips as long as leaves about three CTAs of 512 threads per SM
-  p.strip = 4 * kGroup;
-  while (p.strip < 32 && (long long)batch * ((p.seq + p.strip - 1) / p.strip) > 6ll * sm_count()) p.strip *= 2;
-  while (p.strip > kGroup && (long long)batch * ((p.seq + p.strip - 1) / p.strip) < 2ll * sm_count()) p.strip /= 2;
-  launch_pdl(stream_conv_kernel<T, TAPS, PACKS, false>, dim3((p.seq + p.strip - 1) / p.strip, batch), dim3(threads), 0, st, p);
+  // what the ring gives is added up before the sum is known
+  float a1[PACKS][4], a2[PACKS][4];
+#pragma unroll
+  for (int k = 0; k < PACKS; ++k) {
+    const int col = (tid + k * blockDim.x) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) a1[k][e] = a2[k][e] = 0.f;
+    if (col >= p.n2) continue;
+#pragma unroll 4
+    for (int j = 0; j < taps - 1; ++j) {
+      const int t = pos - (taps - 1) + j;
+      if (t < first) continue;
+      float u[4], w1[4], w2[4];
+      ld4<T>(ring + (long long)(t % p.ring_rows) * p.ring_ld + col, u);
+      ld4<float>(p.k1 + (long long)j * p.n2 + col, w1);
+      if (p.h2) ld4<float>(p.k2 + (long long)j * p.n2 + col, w2);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        a1[k][e] = fmaf(w1[e], u[e], a1[k][e]);
+        if (p.h2) a2[k][e] = fmaf(w2[e], u[e], a2[k][e]);
+      }
+    }
+  }
+  const float s = warp_sum(sq[0]);
+  if (lane == 0) part[warp].x = s;
+  __syncthreads();
+  const float r = rsqrtf(warp_sum(lane < (blockDim.x >> 5) ? part[lane].x : 0.f) * p.inv_count + p.eps);
+#pragma unroll
+  for (int k = 0; k < PACKS; ++k) {
+    const int col = (tid + k * blockDim.x) * 4;
+    if (col >= p.n2) continue;
+    float w[4];
+    ld4<float>(p.k1 + (long long)(taps - 1) * p.n2 + col, w);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      x[k][e] *= r;
+      a1[k][e] = fmaf(w[e], x[k][e], a1[k][e]);
+    }
+    st4<T>(reinterpret_cast<T *>(p.h1) + b * p.ldh + col, a1[k]);
+    if (p.h2) {
+      ld4<float>(p.k2 + (long long)(taps - 1) * p.n2 + col, w);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) a2[k][e] = fmaf(w[e], x[k][e], a2[k][e]);
+      st4<T>(reinterpret_cast<T *>(p.h2) + b * p.ldh + col, a2[k]);
+    }
+    st4<T>(ring + (long long)(pos % p.ring_rows) * p.ring_ld + col, x[k]);
+  }
+}
+
+template <typename T, int TAPS, int PACKS, int G> int launch_prompt(StreamConvParams p, int batch, cudaStream_t st) {
+  const int threads = ((p.n2 / 4 + PACKS - 1) / PACKS + 31) / 32 * 32;
+  const size_t smem = (size_t)2 * G * PACKS * threads * (16 + 4 * sizeof(T));
+  auto kern = stream_conv_kernel<T, TAPS, PACKS, G>;
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    cudaGetLastError();
+    return fail(EB_ECUDA, "stream_conv: cannot reserve %zu bytes of shared memory", smem);
+  }
+  // one strip per CTA the machine holds, of 8 to 64 tokens
+  const int fit = (int)((220 * 1024) / (smem + 2048)), regs = 1024 / threads, per_sm = fit < regs ? (fit < 1 ? 1 : fit) : regs;
+  const long long slots = (long long)per_sm * sm_count(), want = ((long long)batch * p.seq + slots - 1) / slots;
+  p.strip = (int)((want < 8 ? 8 : want > 64 ? 64 : want) + G - 1) / G * G;
+  launch_pdl(kern, dim3((p.seq + p.strip - 1) / p.strip, batch), dim3(threads), smem, st, p);
   return check_launch("stream_conv");
 }
 
-template <typename T, int TAPS> int launch_taps(const StreamConvParams &p, int batch, bool step, cudaStream_t st) {
-  if (p.n2 <= 4096) return launch_packs<T, TAPS, 1>(p, batch, step, st);
-  return launch_packs<T, TAPS, 4>(p, batch, step, st);
+template <typename T> int launch_step(const StreamConvParams &p, int taps, int batch, cudaStream_t st) {
+  auto go = [&](auto kern, int packs) {
+    const int threads = ((p.n2 / 4 + packs - 1) / packs + 31) / 32 * 32;
+    launch_pdl(kern, dim3(batch), dim3(threads), 0, st, p, taps);
+    return check_launch("stream_conv");
+  };
+  return p.n2 <= 4096 ? go(stream_conv_step_kernel<T, 1>, 1) : go(stream_conv_step_kernel<T, 4>, 4);
+}
+
+template <typename T, int TAPS> int launch_taps(const StreamConvParams &p, int batch, cudaStream_t st) {
+  if (p.n2 <= 4096) return launch_prompt<T, TAPS, 1, sizeof(T) == 2 ? 4 : 2>(p, batch, st);
+  return launch_prompt<T, TAPS, 4, 1>(p, batch, st);
 }
 
 template <typename T> int launch_stream_conv(const StreamConvParams &p, int taps, int batch, bool step, cudaStream_t st) {
+  if (step) return launch_step<T>(p, taps, batch, st);
   switch (taps) {
-    case 2: return launch_taps<T, 2>(p, batch, step, st);
-    case 3: return launch_taps<T, 3>(p, batch, step, st);
-    case 4: return launch_taps<T, 4>(p, batch, step, st);
-    case 8: return launch_taps<T, 8>(p, batch, step, st);
-    default: return launch_taps<T, 16>(p, batch, step, st);
+    case 2: return launch_taps<T, 2>(p, batch, st);
+    case 3: return launch_taps<T, 3>(p, batch, st);
+    case 4: return launch_taps<T, 4>(p, batch, st);
+    case 8: return launch_taps<T, 8>(p, batch, st);
+    default: return launch_taps<T, 16>(p, batch, st);
   }
 }
 

@@ -6,6 +6,7 @@
 #include <cuda.h>
 
 #include "common.cuh"
+#include "packed_math.cuh"
 
 namespace eb {
 namespace {
@@ -115,30 +116,6 @@ __device__ __forceinline__ void tc_st32(uint32_t taddr, const float *v) {
         "r"(__float_as_uint(v[24])), "r"(__float_as_uint(v[25])), "r"(__float_as_uint(v[26])), "r"(__float_as_uint(v[27])),
         "r"(__float_as_uint(v[28])), "r"(__float_as_uint(v[29])), "r"(__float_as_uint(v[30])), "r"(__float_as_uint(v[31]))
       : "memory");
-}
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// Two fp32 operations in one instruction.
-__device__ __forceinline__ void fma2(float &x0, float &x1, float a0, float a1, float b0, float b1, float c0, float c1) {
-  asm("{\n\t.reg .b64 a, b, c, d;\n\t"
-      "mov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\t"
-      "fma.rn.f32x2 d, a, b, c;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(x0), "=f"(x1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1), "f"(c0), "f"(c1));
-}
-__device__ __forceinline__ void mul2(float &x0, float &x1, float a0, float a1, float b0, float b1) {
-  asm("{\n\t.reg .b64 a, b, d;\n\t"
-      "mov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\t"
-      "mul.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(x0), "=f"(x1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1));
-}
-__device__ __forceinline__ void add2(float &x0, float &x1, float a0, float a1, float b0, float b1) {
-  asm("{\n\t.reg .b64 a, b, d;\n\t"
-      "mov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\t"
-      "add.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
-      : "=f"(x0), "=f"(x1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1));
 }
 __device__ __forceinline__ void tc_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 // K-major tile of 128-byte rows with the 128-byte swizzle; 8-row groups 1024 bytes apart.

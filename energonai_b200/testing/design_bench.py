@@ -1,8 +1,9 @@
 """Throughput of the layer-listed decoders (latent attention / mixture of experts, matrix memory / grouped
-attention, state space / chunk attention beside gated linear attention) at sizes that resemble a real model's
+attention, state space / chunk attention beside gated linear attention, selective state space / capped attention /
+rotary latent attention beside dense feed-forwards) at sizes that resemble a real model's
 layers (random weights), beside an OPT-shaped PipelineModel of equal width, heads, depth and weights per
 token, and the time of every kernel next to its roofline and to the like kernel of another model.
-`bench.py --design tulezen | mutolix | moponex` prints the result as one JSON line."""
+`bench.py --design tulezen | mutolix | moponex | tupidra` prints the result as one JSON line."""
 import json
 import os
 import statistics
@@ -24,7 +25,8 @@ FLUSH_BYTES = 400 << 20      # a timed kernel cycles through operand copies of a
 def peaks():
     path = os.path.join(os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)))), "MEASURED_PEAKS.json")
     d = json.load(open(path)) if os.path.exists(path) else {}
-    return {"hbm": d.get("hbm_gbs", 6650.0) * 1e9, "tensor": d.get("bf16_tflops", 1590.0) * 1e12,
+    # sfu: special-function results per second, 16 per clock on each of 148 SMs at 1.965 GHz (nominal)
+    return {"hbm": d.get("hbm_gbs", 6650.0) * 1e9, "tensor": d.get("bf16_tflops", 1590.0) * 1e12, "sfu": 16 * 148 * 1.965e9,
             "kind": "measured" if d else "fallback"}
 
 
@@ -572,7 +574,218 @@ def moponex_kernel_table(z, B, S, T):
     return rows, {"active_experts": act_e, "sorted_rows": int(plan.live_tiles.item()) * 128, "routed_rows": pairs}
 
 
+TUPIDRA_SIZES = {
+    # a selective state space (inner, state, dt_rank), a capped attention (heads on kv_heads, window, keep) and two rotary latent
+    # attentions (l*: heads of ldim + rot / lvdim, q_rank, kv_rank), the second on the latents of the first; every layer
+    # with a dense feed-forward beside its mixer
+    "2048": dict(width=2048, inner=4096, state=16, dt_rank=128, heads=16, kv_heads=4, dim=128, window=1024, keep=64, lheads=32, ldim=64, rot=32, lvdim=64,
+                 q_rank=768, kv_rank=256, ff=5632, layers=8, vocab=32768),
+    "4096": dict(width=4096, inner=8192, state=16, dt_rank=256, heads=32, kv_heads=8, dim=128, window=4096, keep=64, lheads=32, ldim=96, rot=32, lvdim=128,
+                 q_rank=1536, kv_rank=480, ff=11264, layers=8, vocab=32768),
+}
+
+
+def make_tupidra(z):
+    from ..registry import build_model
+    ff = {"kind": "dense", "ff": z["ff"]}
+    scan = {"type": "mamba1", "mlp": ff, "mixer": {"inner": z["inner"], "state": z["state"], "dt_rank": z["dt_rank"], "conv": 4}}
+    att = {"type": "attention", "mlp": ff, "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                                                     "softcap": 50.0, "mask": {"size": z["window"], "keep_first": z["keep"]}}}
+    mix = {"heads": z["lheads"], "dim": z["ldim"], "rot_dim": z["rot"], "vdim": z["lvdim"], "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+           "scale": (z["ldim"] + z["rot"]) ** -0.5,
+           "rot": {"dims": z["rot"], "base": 1e5, "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    layers = []
+    for i in range(0, z["layers"], 4):
+        layers += [scan, att, {"type": "latent_attention", "mlp": ff, "mixer": mix}, {"type": "latent_attention", "mlp": ff, "mixer": dict(mix, kv_from=i + 2)}]
+    torch.manual_seed(1)
+    return build_model("Tupidra", config_dict={"vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "canon": {"taps": 4}, "layers": layers},
+                       dtype=torch.bfloat16, device="cuda")
+
+
+def tupidra_as_opt(z):
+    """The feed-forward size with which an OPT layer has as many weights as a layer here has on average."""
+    w, h = z["width"], z["heads"] * z["dim"]
+    scan = z["inner"] * (3 * w + 2 * z["dt_rank"] + 2 * z["state"])
+    att = w * (3 * h + 2 * z["kv_heads"] * z["dim"])
+    lh, key = z["lheads"], z["ldim"] + z["rot"]
+    latent = w * (z["q_rank"] + 2 * lh * z["lvdim"]) + lh * (key * z["q_rank"] + (z["ldim"] + z["lvdim"]) * z["kv_rank"])
+    latents = w * (z["kv_rank"] + z["rot"])
+    ffn = ((scan + att + 2 * latent + latents) / 4 / w + 3 * z["ff"] - 4 * w) / 2
+    return dict(z, top=1, ff=int(ffn / 1.5))
+
+
+def tupidra_kernel_table(z, B, S, T):
+    """As kernel_table, for the selective-scan / capped-attention / rotary-latent decoder."""
+    from ..attention import (LATENT_WIDTHS, attention_decode, attention_group_decode, attention_group_decode_capped, attention_prefill, attention_prefill_biased,
+                             attention_prefill_capped, attention_prefill_gated, attention_rotary, attention_values, distance_bias, distance_slopes, latent_decode,
+                             latent_inputs, rotate_heads, sigmoid_gate)
+    from ..decay import selective_scan, selective_step, short_conv, short_conv_step, ssm_prompt, ssm_step
+    from ..gemm import gemm, project_parts, project_unit
+    from ..kernel.cuda_native.layer_norm import layer_norm_forward
+    from ..moe import per_head
+    from ..norm import rms_norm, stream_add, stream_conv
+    bf, f32, dev = torch.bfloat16, torch.float32, "cuda"
+    W, H, G, d, ff, C, N, dr = (z[k] for k in ("width", "heads", "kv_heads", "dim", "ff", "inner", "state", "dt_rank"))
+    LH, ld, rot, lv, qr, kr = (z[k] for k in ("lheads", "ldim", "rot", "lvdim", "q_rank", "kv_rank"))
+    dk, R = 64 if ld + rot <= 64 else 128, min(w for w in LATENT_WIDTHS if w >= kr + rot)
+    win, keep = z["window"], z["keep"]
+    rnd = lambda *s, dtype=bf: (torch.randn(*s, device=dev, dtype=torch.float32) * 0.05).to(dtype)
+    rows = []
+
+    def add(phase, name, like, us, nbytes, flops=0.0, sfu=0.0):
+        rows.append((phase, name, like, us, float(nbytes), float(flops), float(sfu)))
+
+    def product(phase, name, M, Nn, Kd, like=None, unit=None, act=None, tail=0, out32=False, bias=False):
+        Nn += tail
+        cols = Nn // 2 if unit == "geglu" else Nn
+        nb = 2 * (Nn * Kd + M * Kd) + (4 if out32 else 2) * M * (cols + tail)
+        ws = [rnd(Nn, Kd) for _ in range(copies(2 * Nn * Kd, 32))]
+        xs = [rnd(M, Kd) for _ in range(4)]
+        b = rnd(Nn)
+        if unit:
+            call = lambda w, x: project_unit(x, w, unit)
+        elif tail:
+            call = lambda w, x: project_parts(x, w, tail_col=Nn - tail)
+        else:
+            call = lambda w, x: gemm(x, w, bias=b if act or bias else None, act=act, out_dtype=f32 if out32 else None, static_weight=True)
+        add(phase, name, like, time_calls([lambda w=w, x=xs[i % 4]: call(w, x) for i, w in enumerate(ws)]), nb, 2.0 * M * Nn * Kd)
+
+    def gemms(phase, M):
+        product(phase, "gemm in_proj (scan)", M, 2 * C, W)
+        product(phase, "gemm x_proj", M, dr, C, tail=2 * N)
+        product(phase, "gemm in_proj (attention)", M, (2 * H + 2 * G) * d, W, bias=True)
+        product(phase, "gemm in_proj (latent)", M, qr + R + LH * lv, W)
+        product(phase, "gemm query up", M, LH * dk, qr)
+        product(phase, "gemm gate_up + geglu", M, 2 * ff, W, like="gemm fc1 relu (OPT)", unit="geglu")
+        product(phase, "gemm fc1 relu (OPT)", M, 2 * ff, W, act="relu")
+        product(phase, "gemm out (scan | mlp)", M, W, C + ff)
+        product(phase, "gemm out (attention | mlp)", M, W, H * d + ff, bias=True)
+
+    scan_p = [torch.full((C,), -3.0, device=dev), torch.rand(C, N, device=dev), torch.ones(C, device=dev)]
+    conv_w, conv_b, dtw = rnd(4, C), rnd(C), rnd(C, dr)
+    k1, k2, lw, lb, nw = torch.rand(4, W, device=dev), torch.rand(4, W, device=dev), rnd(W), rnd(W), rnd(W)
+    slopes, rule = distance_slopes(H, dev), dict(window=win, keep=keep, cap=50.0)
+    sinks, freq, qn, cn = torch.zeros(LH, device=dev), torch.rand(rot // 2, device=dev), rnd(qr), rnd(kr)
+    pos = torch.tensor([S - 1], dtype=torch.int32, device=dev)
+    held = min(win, S)
+    seen = held + min(keep, max(0, S - held))
+
+    # ---- generation step ----
+    gemms("step", B)
+    nb = 8 * B * C * N
+    states = [rnd(B, C, N, dtype=f32) for _ in range(copies(nb / 2))]
+    xz, low, bc, x1 = rnd(B, 2 * C), rnd(B, dr), rnd(B, 2 * N, dtype=f32), rnd(B, C)
+    ring = rnd(B, 4, C)
+    add("step", "short_conv_step", "layer_norm (OPT)", time_calls([lambda: short_conv_step(xz[:, :C], conv_w, conv_b, ring, pos)] * 16), 12 * B * C)
+    add("step", "selective_step", "ssm_step (Moponex)", time_calls([lambda s=s: selective_step(x1, xz[:, C:], low, dtw, bc, *scan_p, s) for s in states]),
+        nb + 6 * B * C + 2 * C * dr + 4 * C * N)
+    SH, sn = C // 64, max(8, N)
+    smalls = [s.view(B, SH, sn, -1) for s in states] if N * 64 % sn == 0 else None
+    per = [torch.full((SH,), v, device=dev) for v in (-2.0, -1.0, 1.0)]
+    sw, sb, srow, sring, sdt = rnd(4, C + 2 * sn), rnd(C + 2 * sn), rnd(B, C + 2 * sn), rnd(B, 4, C + 2 * sn), rnd(B, SH, dtype=f32)
+    add("step", "ssm_step (Moponex)", None, time_calls([lambda s=s: ssm_step(srow, sw, sb, sring, pos, sdt, *per, s, SH, 1, sn, 64) for s in smalls]),
+        nb + 2 * B * (6 * (C + 2 * sn) + C))
+    del states, smalls
+    kv = [rnd(B, keep + held, 2 * G * d) for _ in range(copies(B * held * 2 * G * d * 2))]
+    pr = rnd(B, (2 * H + 2 * G) * d)
+    q, k, v, g = pr.split([H * d, G * d, G * d, H * d], 1)
+    add("step", "attention_group_decode capped", "attention_group_decode (Mutolix)", time_calls([lambda c=c: attention_group_decode_capped(
+        q, c[:, :, :G * d], c[:, :, G * d:], d, pos, 0.09, slopes=slopes, gate=g, **rule) for c in kv]), 4 * B * seen * G * d + 6 * B * H * d)
+    bias_h = tuple(torch.rand(H, device=dev) for _ in range(2))
+    qc, last = q.contiguous(), torch.tensor([held - 1], dtype=torch.int32, device=dev)
+    add("step", "attention_group_decode (Mutolix)", None, time_calls([lambda c=c: attention_group_decode(
+        qc, c[:, :, :G * d], c[:, :, G * d:], d, last, 0.09, bias=bias_h) for c in kv]), 4 * B * held * G * d + 4 * B * H * d)
+    add("step", "attention_values", "attention_rotary (Moponex)", time_calls([lambda c=c: attention_values(
+        k, v, G, d, 1e-6, c[:, :, :G * d], c[:, :, G * d:], keep, 1, pos_device=pos) for c in kv]), 10 * B * G * d)
+    hn, hf = rnd(d), torch.rand(d // 4, device=dev)
+    add("step", "attention_rotary (Moponex)", None, time_calls([lambda c=c: attention_rotary(pr, H, G, d, d, hn, hn, 1e-6, hf, c[:, :, :G * d], c[:, :, G * d:], 1,
+                                                                                             pos_device=pos) for c in kv]), 4 * B * H * d + 6 * B * G * d)
+    del kv
+    cache = [rnd(B, S, R) for _ in range(copies(B * S * R * 2))]
+    qa = rnd(B, LH * R)
+    lat = lambda sk: time_calls([lambda c=c: latent_decode(qa, c, R, LH, 0, pos, 0.05, sinks=sk) for c in cache])
+    add("step", "latent_decode with sinks", "latent_decode (Tulezen)", lat(sinks), 2 * B * S * R + 4 * B * LH * R, 4.0 * B * LH * S * R)
+    add("step", "latent_decode (Tulezen)", None, lat(None), 2 * B * S * R + 4 * B * LH * R, 4.0 * B * LH * S * R)
+    pl = rnd(B, qr + R + LH * lv)
+    row = lambda c, **kw: dict(cols=R, rot_col=kr, count=kr, norm=cn, freq=freq, factor=1.2, ring=c, **kw)
+    add("step", "latent_inputs", "rms_norm to ring (Tulezen)", time_calls([lambda c=c: latent_inputs(pl, qr, qr, qn, 1e-6, row=row(c), pos_device=pos) for c in cache]),
+        4 * B * (qr + R))
+    rn = rnd(R)
+    add("step", "rms_norm to ring (Tulezen)", None, time_calls([lambda c=c: rms_norm(pl[:, :R], rn, 1e-5, write_out=False, ring=c, pos_device=pos) for c in cache]), 4 * B * R)
+    del cache
+    qh, o, vo, gl = rnd(B, LH * dk), rnd(B, LH * R), rnd(B, LH * lv), pl[:, qr + R:]
+    add("step", "rotate_heads", "attention_rotary (Moponex)", time_calls([lambda: rotate_heads(qh, LH, dk, ld, freq, 1.2, 1, pos_device=pos)] * 16), 4 * B * LH * rot)
+    ups = [rnd(LH, R, dk) for _ in range(copies(LH * R * dk * 2, 48))]
+    add("step", "per_head key absorb", "gemm query up", time_calls([lambda w=w: per_head(qh, w) for w in ups]), 2 * (LH * R * dk + B * LH * (R + dk)))
+    add("step", "per_head value up", "gemm query up", time_calls([lambda w=w: per_head(o, w.view(-1)[:LH * lv * R].view(LH, lv, R)) for w in ups]),
+        2 * (LH * R * lv + B * LH * (R + lv)))
+    del ups
+    add("step", "sigmoid_gate", "layer_norm (OPT)", time_calls([lambda: sigmoid_gate(vo, gl)] * 16), 6 * B * LH * lv)
+    x, y, xt, rr = torch.randn(B, W, device=dev), rnd(B, W), rnd(B, W), rnd(B, 4, W)
+    add("step", "stream_conv", "stream_add (Moponex)", time_calls([lambda: stream_conv(x, k1, rr, 1e-6, B, y=y, k2=k2, pos_device=pos)] * 16), 22 * B * W + 32 * W)
+    add("step", "stream_add (Moponex)", None, time_calls([lambda: stream_add(x, 1e-6, y=y, w_next=nw)] * 16), 12 * B * W)
+    add("step", "layer_norm (OPT)", None, time_calls([lambda: layer_norm_forward(xt, lw, lb, 1e-5)] * 16), 4 * B * W)
+
+    # ---- prompt ----
+    seq = min(S, T)
+    nB = T // seq
+    gemms("prompt", T)
+    product("prompt", "gemm step logits", T, C, dr, out32=True)
+    product("prompt", "gemm kv up", T, LH * (dk + lv), R)
+    xzs, zs, bc = [rnd(T, 2 * C) for _ in range(3)], rnd(T, C, dtype=f32), rnd(T, 2 * N, dtype=f32)
+    ring = rnd(nB, 4, C)
+    add("prompt", "short_conv", "layer_norm (OPT)", time_calls([lambda r=r: short_conv(r[:, :C], conv_w, conv_b, ring, nB) for r in xzs]), 4 * T * C)
+    state = torch.empty(nB, C, N, device=dev)
+    add("prompt", "selective_scan", "ssm_chunks (Moponex)", time_calls([lambda r=r: selective_scan(r[:, :C], r[:, C:], zs, bc, *scan_p, state) for r in xzs]),
+        10 * T * C + 8 * T * N + 4 * nB * C * N, 0.0, float(T) * C * N)
+    del xzs, zs, state
+    sx, sdt, sst = rnd(T, C + 256), rnd(T, SH, dtype=f32), torch.empty(nB, SH, 128, 64, device=dev)
+    add("prompt", "ssm_chunks (Moponex)", None, time_calls([lambda: ssm_prompt(sx, sdt, *per, sst, SH, 1, 128, 64, chunked=True)] * 4),
+        2 * T * (2 * C + 256) + 4 * T * SH + 4 * nB * C * 128, 4.0 * T * C * 128)
+    del sx, sst
+    q3, kv3, g3 = rnd(nB, seq, H * d), rnd(nB, seq, 2 * G * d), rnd(nB, seq, H * d)
+    k3, v3 = kv3[:, :, :G * d], kv3[:, :, G * d:]
+    pairs = sum(min(i + 1, win) + min(keep, max(0, i + 1 - win)) for i in range(seq))
+    full = seq * (seq + 1) / 2
+    add("prompt", "attention capped", "attention biased (Mutolix)", time_calls([lambda: attention_prefill_capped(q3, k3, v3, d, d, slopes=slopes, gate=g3, **rule)] * 4),
+        2 * T * (3 * H + 2 * G) * d, 4.0 * nB * H * d * pairs)
+    table = distance_bias(*bias_h, seq)
+    add("prompt", "attention biased (Mutolix)", None, time_calls([lambda: attention_prefill_biased(q3, k3, v3, d, table)] * 4), 2 * T * (2 * H + 2 * G) * d, 4.0 * nB * H * d * full)
+    cb = rnd(nB, keep + min(win, seq), 2 * G * d)
+    kvs = [rnd(T, 2 * G * d) for _ in range(copies(T * G * d * 10, 16))]
+    add("prompt", "attention_values", "attention_rotary (Moponex)", time_calls([lambda r=r: attention_values(
+        r[:, :G * d], r[:, G * d:], G, d, 1e-6, cb[:, :, :G * d], cb[:, :, G * d:], keep, seq) for r in kvs]), 4 * T * G * d + 4 * nB * cb.shape[1] * G * d + 2 * nB * cb.shape[1] * G * d)
+    projs = [rnd(T, (H + G) * d) for _ in range(3)]
+    add("prompt", "attention_rotary (Moponex)", None, time_calls([lambda r=r: attention_rotary(
+        r, H, G, d, d, hn, hn, 1e-6, hf, cb[:, :, :G * d], cb[:, :, G * d:], seq, keys=True) for r in projs]), 4 * T * (H + G) * d + 4 * nB * cb.shape[1] * G * d)
+    del q3, kv3, g3, k3, v3, kvs, cb, projs
+    q3, kv3, g3 = rnd(nB, seq, LH * dk), rnd(nB, seq, LH * (dk + lv)), rnd(nB, seq, LH * lv)
+    k3, v3 = kv3[:, :, :LH * dk], kv3[:, :, LH * dk:]
+    add("prompt", "attention latent", "attention causal (OPT)", time_calls([lambda: attention_prefill_gated(q3, k3, v3, dk, lv, sinks=sinks, gate=g3)] * 4),
+        2 * T * (2 * dk + 3 * lv) * LH, 2.0 * nB * LH * (dk + lv) * full)
+    del kv3, g3, k3, v3
+    q4, kv4 = rnd(nB, seq, H * d), rnd(nB, seq, 2 * H * d)
+    add("prompt", "attention causal (OPT)", None, time_calls([lambda: attention_prefill(q4, kv4[:, :, :H * d], kv4[:, :, H * d:], d)] * 4), 8 * T * H * d, 4.0 * nB * H * d * full)
+    del q4, kv4
+    pls, lc = [rnd(T, qr + R + LH * lv) for _ in range(3)], rnd(nB, seq, R)
+    add("prompt", "latent_inputs", "rms_norm latent (Tulezen)", time_calls([lambda r=r: latent_inputs(r, qr, qr, qn, 1e-6, row=row(lc, keep_rows=True), rows_per_batch=seq) for r in pls]),
+        T * (4 * qr + 6 * R))
+    cs = [rnd(T, R) for _ in range(copies(4 * T * R))]
+    add("prompt", "rms_norm latent (Tulezen)", None, time_calls([lambda t=t: rms_norm(t, rn, 1e-5, ring=lc, rows_per_batch=seq) for t in cs]), 6 * T * R)
+    del pls, cs, lc
+    qs = [q3.view(T, -1)] + [rnd(T, LH * dk) for _ in range(3)]
+    add("prompt", "rotate_heads", "attention_rotary (Moponex)", time_calls([lambda r=r: rotate_heads(r, LH, dk, ld, freq, 1.2, seq) for r in qs]), 4 * T * LH * rot)
+    del qs, q3
+    xs = [torch.randn(T, W, device=dev) for _ in range(copies(14 * T * W, 8))]
+    ys, rr = [rnd(T, W) for _ in xs], rnd(nB, 4, W)
+    add("prompt", "stream_conv", "stream_add (Moponex)", time_calls([lambda x=x, y=y: stream_conv(x, k1, rr, 1e-6, nB, y=y, k2=k2) for x, y in zip(xs, ys)]), 14 * T * W)
+    add("prompt", "stream_add (Moponex)", None, time_calls([lambda x=x, y=y: stream_add(x, 1e-6, y=y, w_next=nw) for x, y in zip(xs, ys)]), 12 * T * W)
+    add("prompt", "layer_norm (OPT)", None, time_calls([lambda t=t: layer_norm_forward(t, lw, lb, 1e-5) for t in ys]), 4 * T * W)
+    return rows, {}
+
+
 DESIGNS = {
+    "tupidra": dict(sizes=TUPIDRA_SIZES, runs=RUNS, make=make_tupidra, as_opt=tupidra_as_opt, table=tupidra_kernel_table),
     "moponex": dict(sizes=MOPONEX_SIZES, runs=RUNS, make=make_moponex, as_opt=moponex_as_opt, table=moponex_kernel_table),
     "tulezen": dict(sizes=SIZES, runs=RUNS, make=make_tulezen, as_opt=lambda z: z, table=kernel_table),
     "mutolix": dict(sizes=MUTOLIX_SIZES, runs=RUNS, make=make_mutolix, as_opt=mutolix_as_opt, table=mutolix_kernel_table),
@@ -582,10 +795,11 @@ DESIGNS = {
 def table_with_fractions(rows):
     pk = peaks()
     out = []
-    for phase, name, like, us, nbytes, flops in rows:
-        roof = max(nbytes / pk["hbm"], flops / pk["tensor"]) * 1e6
-        out.append({"phase": phase, "kernel": name, "us": round(us, 2), "roofline_us": round(roof, 2), "frac": round(roof / us, 3), "like": like,
-                    "bound": "hbm" if nbytes / pk["hbm"] >= flops / pk["tensor"] else "tensor"})
+    for phase, name, like, us, *work in rows:
+        times = {what: n / pk[what] * 1e6 for what, n in zip(("hbm", "tensor", "sfu"), work)}
+        bound = max(times, key=times.get)
+        out.append({"phase": phase, "kernel": name, "us": round(us, 2), "roofline_us": round(times[bound], 2), "frac": round(times[bound] / us, 3), "like": like,
+                    "bound": bound})
     by = {(r["phase"], r["kernel"]): r["frac"] for r in out}
     for r in out:
         if r["like"]:

@@ -189,3 +189,96 @@ def greedy(cfg, tensors, tokens, new):
         gap = min(gap, float(top.values[0] - top.values[1]))
         tokens.append(int(top.indices[0]))
     return tokens, gap
+
+
+# ---- small models of the tests' own ------------------------------------------------------------------
+def dense_mlp(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def scan_layer(inner, state, dt_rank, conv=4, mlp=None):
+    return {"type": "mamba1", "mlp": mlp, "mixer": {"inner": inner, "state": state, "dt_rank": dt_rank, "conv": conv}}
+
+
+def attention_layer(heads, kv_heads, dim, vdim, scale, cap=None, mask=None, mlp=None):
+    """mask = (window, kept first positions)."""
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+    if cap:
+        m["softcap"] = cap
+    if mask:
+        m["mask"] = {"size": mask[0], "keep_first": mask[1]}
+    return {"type": "attention", "mlp": mlp, "mixer": m}
+
+
+def latent_layer(heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, base, scaling=None, kv_from=None, mlp=None):
+    """scaling = (factor, original, fast, slow)."""
+    rot = {"dims": rot_dim, "base": base}
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank, "scale": scale, "rot": rot}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "latent_attention", "mlp": mlp, "mixer": m}
+
+
+def make_config(layers, width, vocab, taps=4, eps=2e-5):
+    return {"architecture": "Tupidra", "vocab": vocab, "width": width, "norm": {"eps": eps}, "canon": {"taps": taps}, "layers": layers}
+
+
+def make_tensors(cfg, seed):
+    """Random bfloat16 tensors of a configuration.  Projections keep the scale of their input; decays are mostly slow, so
+    that far tokens still count; sinks are about as large as scores; norm weights move away from one."""
+    g = torch.Generator().manual_seed(seed)
+    W, t, taps = cfg["width"], {}, cfg["canon"]["taps"]
+
+    def mat(name, rows, cols, gain=1.0):
+        t[name] = (torch.randn(rows, cols, generator=g) * gain / cols ** 0.5).bfloat16()
+
+    def vec(name, n, mean, spread=0.3):
+        t[name] = (mean + spread * torch.randn(n, generator=g)).bfloat16()
+    mat("embed", cfg["vocab"], W, W ** 0.5)
+    mat("head", cfg["vocab"], W)
+    vec("final.norm", W, 1.0)
+    for i, ly in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}.", ly["mixer"], ly["mlp"]
+        q = p + "mix."
+        vec(p + "norm1", W, 1.0)
+        mat(p + "canon1", W, taps, 0.7)
+        if ly["type"] == "mamba1":
+            C, N, R = m["inner"], m["state"], m["dt_rank"]
+            mat(q + "in", 2 * C, W, 1.2)
+            mat(q + "conv", C, m["conv"], 1.3)
+            vec(q + "conv.b", C, 0.0)
+            mat(q + "x", R + 2 * N, C, 0.8)
+            mat(q + "dt", C, R)
+            vec(q + "dt.b", C, -3.0, 0.7)
+            t[q + "A_log"] = (torch.randn(C, N, generator=g) - 0.5).bfloat16()
+            vec(q + "D", C, 0.7)
+            mat(q + "o", W, C, 0.5)
+        elif ly["type"] == "attention":
+            H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            for name, n in (("q", H * d), ("k", G * d), ("v", G * dv)):
+                mat(q + name, n, W, 1.2)
+                vec(f"{q}{name}.b", n, 0.0)
+            mat(q + "g", H * dv, W, 1.5)
+            mat(q + "o", W, H * dv, 3.5)
+            vec(q + "o.b", W, 0.0)
+        else:
+            H, d, r, dv, qr, kr = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank"))
+            mat(q + "dq", qr, W)
+            vec(q + "dq.norm", qr, 1.0)
+            mat(q + "uq", H * (d + r), qr, 1.2)
+            if m.get("kv_from") is None:
+                mat(q + "dkv", kr + r, W)
+                vec(q + "dkv.norm", kr, 1.0)
+            mat(q + "uk", H * d, kr, 1.2)
+            mat(q + "uv", H * dv, kr, 1.2)
+            vec(q + "sink", H, 1.0, 1.0)
+            mat(q + "g", H * dv, W, 1.5)
+            mat(q + "o", W, H * dv, 3.5)
+        if f is not None:
+            vec(p + "norm2", W, 1.0)
+            mat(p + "canon2", W, taps, 0.7)
+            for name, rows, cols in (("gate", f["ff"], W), ("up", f["ff"], W), ("down", W, f["ff"])):
+                mat(p + "mlp." + name, rows, cols, 1.3)
+    return t
