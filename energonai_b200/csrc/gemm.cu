@@ -491,35 +491,47 @@ gemm_kernel(const __grid_constant__ CUtensorMap tm_lane, const __grid_constant__
     }
     }   // mover lanes
   } else if (warp == 1) {
-    // ---------------- MMA issuer (whole warp, every decision uniform over it) ----------------
+    // ---------------- MMA issuer ----------------
+    // The whole warp, every decision uniform over it; for the widest tiles, whose MMAs are long enough for one
+    // lane to issue, one lane (with the whole warp, short K ran 15 % slower there: 56 us -> 65 us at 8192 x 4096 x 768).
+    constexpr bool kWarpIssue = BN < 256;
     griddep_wait();
-    Scheduler<BN, SWAP> sched(p);
-    Segment s;
-    int stage = 0, acc = 0;
-    uint32_t phase = 0, acc_phase = 0;
-    bool ok = true;
-    while (ok && sched.next(s)) {
-      if (!__all_sync(0xffffffffu, mbar_wait(tempty_bar + 8 * acc, acc_phase ^ 1u, abort_flag, 2))) break;
-      tcgen05_fence_after();
-      const uint32_t d_tmem = tmem_base + acc * BN;
-      for (int sk = s.sk0; sk < s.sk1; ++sk) {
-        if (!__all_sync(0xffffffffu, mbar_wait(full_bar + 8 * stage, phase, abort_flag, 3))) { ok = false; break; }
+    if (kWarpIssue || lane == 0) {
+      auto wait = [&](uint32_t bar, uint32_t parity, int where) {
+        const bool good = mbar_wait(bar, parity, abort_flag, where);
+        return kWarpIssue ? __all_sync(0xffffffffu, good) != 0 : good;
+      };
+      auto commit = [&](uint32_t bar) { kWarpIssue ? tcgen05_commit_warp(bar) : tcgen05_commit(bar); };
+      Scheduler<BN, SWAP> sched(p);
+      Segment s;
+      int stage = 0, acc = 0;
+      uint32_t phase = 0, acc_phase = 0;
+      bool ok = true;
+      while (ok && sched.next(s)) {
+        if (!wait(tempty_bar + 8 * acc, acc_phase ^ 1u, 2)) break;
         tcgen05_fence_after();
-        for (int j = 0; j < kpb && sk * kpb + j < p.kblocks; ++j) {
-          const uint32_t st_addr = tiles_addr + stage * stage_bytes;
-          const uint64_t a_desc = make_smem_desc(st_addr + j * lane_bytes), b_desc = make_smem_desc(st_addr + col_base + j * kColBytes);
+        const uint32_t d_tmem = tmem_base + acc * BN;
+        for (int sk = s.sk0; sk < s.sk1; ++sk) {
+          if (!wait(full_bar + 8 * stage, phase, 3)) { ok = false; break; }
+          tcgen05_fence_after();
+          for (int j = 0; j < kpb && sk * kpb + j < p.kblocks; ++j) {
+            const uint32_t st_addr = tiles_addr + stage * stage_bytes;
+            const uint64_t a_desc = make_smem_desc(st_addr + j * lane_bytes), b_desc = make_smem_desc(st_addr + col_base + j * kColBytes);
 #pragma unroll
-          for (int k = 0; k < kBlockK / kUmmaK; ++k) {
-            // advancing 16 elements along K inside the swizzle atom = +32 bytes = +2 in the address field
-            tcgen05_mma_f16_warp(d_tmem, a_desc + 2 * k, b_desc + 2 * k, kIdesc, (sk > s.sk0 || j > 0 || k > 0) ? 1u : 0u);
+            for (int k = 0; k < kBlockK / kUmmaK; ++k) {
+              // advancing 16 elements along K inside the swizzle atom = +32 bytes = +2 in the address field
+              const uint32_t add = (sk > s.sk0 || j > 0 || k > 0) ? 1u : 0u;
+              if constexpr (kWarpIssue) tcgen05_mma_f16_warp(d_tmem, a_desc + 2 * k, b_desc + 2 * k, kIdesc, add);
+              else tcgen05_mma_f16(d_tmem, a_desc + 2 * k, b_desc + 2 * k, kIdesc, add);
+            }
           }
+          commit(empty_bar + 8 * stage);            // frees the stage once these MMAs have read it
+          if (++stage == stages) { stage = 0; phase ^= 1u; }
         }
-        tcgen05_commit_warp(empty_bar + 8 * stage);   // frees the stage once these MMAs have read it
-        if (++stage == stages) { stage = 0; phase ^= 1u; }
+        if (!ok) break;
+        commit(tfull_bar + 8 * acc);                // accumulator complete
+        if (++acc == 2) { acc = 0; acc_phase ^= 1u; }
       }
-      if (!ok) break;
-      tcgen05_commit_warp(tfull_bar + 8 * acc);        // accumulator complete
-      if (++acc == 2) { acc = 0; acc_phase ^= 1u; }
     }
   } else {
     // ---------------- epilogue (warps 2..5) ----------------

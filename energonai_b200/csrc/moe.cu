@@ -271,7 +271,7 @@ __global__ void __launch_bounds__(128) grouped_skinny_kernel(const SkinnyParams 
   const int row0 = (SPLIT ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * 16;
   if (n == 0 || row0 >= p.N) return;
   const int *l = p.idx ? list : nullptr;
-  for (int base = 0; base < n; base += 32) {
+  for (int base = blockIdx.z * 32; base < n; base += 32 * gridDim.z) {
     const int m = min(32, n - base);
     if (m <= 8) skinny_tile<T, 1, 8, SPLIT>(p, group, row0, l, base, m, part);
     else if (m <= 16) skinny_tile<T, 2, 4, SPLIT>(p, group, row0, l, base, m, part);
@@ -387,7 +387,8 @@ extern "C" int eb_grouped_skinny(const void *A, long long lda, long long a_group
   const bool few = (long long)((strips + warps - 1) / warps) * groups < 2ll * sm_count(), split = few && K >= 256;
   if (split) p.ksplit = ((K + warps - 1) / warps + 31) / 32 * 32;
   while (!split && warps > 1 && (long long)((strips + warps - 1) / warps) * groups < 2ll * sm_count()) warps >>= 1;
-  const dim3 g(split ? strips : (strips + warps - 1) / warps, groups), b(warps * 32);
+  // (groups without a list: the rows come 32 to a CTA, side by side)
+  const dim3 g(split ? strips : (strips + warps - 1) / warps, groups, idx ? 1 : (rows + 31) / 32), b(warps * 32);
   const size_t smem = idx ? (size_t)rows * sizeof(int) : 0;
   cudaStream_t st = as_stream(stream);
   if (dtype == EB_F16) launch_pdl(split ? grouped_skinny_kernel<__half, true> : grouped_skinny_kernel<__half, false>, g, b, smem, st, p);

@@ -33,6 +33,17 @@ template <> __device__ __forceinline__ float gate_silu<float>(float x) { return 
 template <typename T> __device__ __forceinline__ float step_size(float x) { return fmaxf(x, 0.f) + log1p_unit(ex2(-fabsf(x) * kLog2eScan)); }
 template <> __device__ __forceinline__ float step_size<float>(float x) { return softplus(x); }
 
+// One element's step, S' = exp(dt rate) S + in.  16-bit models: a power of two (rates times log2 e).  32-bit models form
+// exp - 1: a slow decay is close to one, and the rounding of one, always to the same side, adds up over a sequence.
+template <typename T> struct Decay {
+  static constexpr float kScale = kLog2eScan;
+  static __device__ __forceinline__ float step(float S, float e, float in) { return fmaf(ex2(e), S, in); }
+};
+template <> struct Decay<float> {
+  static constexpr float kScale = 1.f;
+  static __device__ __forceinline__ float step(float S, float e, float in) { return fmaf(expm1f(e), S, S + in); }
+};
+
 template <typename T> struct Two;
 template <> struct Two<float> {
   using R = float2;
@@ -165,7 +176,7 @@ __global__ void __launch_bounds__(scan_threads<LPC, CPT>) selective_scan_kernel(
 #pragma unroll
     for (int n = 0; n < NS; ++n) {
       const int s = sub * NS + n;
-      A[k][n] = c < p.inner && s < p.states ? -expf(p.a_log[(long long)(c + k) * p.states + s]) * kLog2eScan : 0.f;
+      A[k][n] = c < p.inner && s < p.states ? -expf(p.a_log[(long long)(c + k) * p.states + s]) * Decay<T>::kScale : 0.f;
       S[k][n] = 0.f;
     }
   fetch(0);
@@ -214,7 +225,12 @@ __global__ void __launch_bounds__(scan_threads<LPC, CPT>) selective_scan_kernel(
             float *s = S[k] + n, e0, e1, b0, b1;
             mul2(e0, e1, d[2 * k], d[2 * k], A[k][n], A[k][n + 1]);
             mul2(b0, b1, d[2 * k + 1], d[2 * k + 1], bv.x, bv.y);
-            fma2(s[0], s[1], ex2(e0), ex2(e1), s[0], s[1], b0, b1);
+            if constexpr (sizeof(T) == 2) {
+              fma2(s[0], s[1], ex2(e0), ex2(e1), s[0], s[1], b0, b1);
+            } else {
+              s[0] = Decay<T>::step(s[0], e0, b0);
+              s[1] = Decay<T>::step(s[1], e1, b1);
+            }
             fma2(acc[k][0], acc[k][1], s[0], s[1], cv.x, cv.y, acc[k][0], acc[k][1]);
           }
         }
@@ -271,7 +287,7 @@ __global__ void __launch_bounds__(kSelStepThreads) selective_step_kernel(const S
   const bool mine = blockIdx.x * CH + ch < p.inner;
   float A[NS];
 #pragma unroll
-  for (int n = 0; n < NS; ++n) A[n] = sub * NS + n < p.states ? -expf(p.a_log[(long long)c * p.states + sub * NS + n]) * kLog2eScan : 0.f;
+  for (int n = 0; n < NS; ++n) A[n] = sub * NS + n < p.states ? -expf(p.a_log[(long long)c * p.states + sub * NS + n]) * Decay<T>::kScale : 0.f;
   const float bias = p.bias[c], skip = p.skip[c];
   const T *w = reinterpret_cast<const T *>(p.w) + (long long)c * p.rank;
   griddep_wait();
@@ -300,10 +316,10 @@ __global__ void __launch_bounds__(kSelStepThreads) selective_step_kernel(const S
     float y = 0.f;
 #pragma unroll
     for (int n = 0; n < NS / 4; ++n) {
-      S4[n].x = fmaf(ex2(dt * A[4 * n]), S4[n].x, dx * B4[n].x);
-      S4[n].y = fmaf(ex2(dt * A[4 * n + 1]), S4[n].y, dx * B4[n].y);
-      S4[n].z = fmaf(ex2(dt * A[4 * n + 2]), S4[n].z, dx * B4[n].z);
-      S4[n].w = fmaf(ex2(dt * A[4 * n + 3]), S4[n].w, dx * B4[n].w);
+      S4[n].x = Decay<T>::step(S4[n].x, dt * A[4 * n], dx * B4[n].x);
+      S4[n].y = Decay<T>::step(S4[n].y, dt * A[4 * n + 1], dx * B4[n].y);
+      S4[n].z = Decay<T>::step(S4[n].z, dt * A[4 * n + 2], dx * B4[n].z);
+      S4[n].w = Decay<T>::step(S4[n].w, dt * A[4 * n + 3], dx * B4[n].w);
       y = fmaf(S4[n].x, C4[n].x, fmaf(S4[n].y, C4[n].y, fmaf(S4[n].z, C4[n].z, fmaf(S4[n].w, C4[n].w, y))));
       if (mine && sub * NS + 4 * n < p.states) *reinterpret_cast<float4 *>(Sp + 4 * n) = S4[n];
     }
