@@ -161,7 +161,7 @@ def attention_plain(q, k, v, heads, k_dim, v_dim, window=0, scale=1.0, first=Non
     return out
 
 
-LATENT_WIDTHS = (64, 128, 192, 256, 320, 384, 512)      # latent widths of the tensor-core generation kernel
+LATENT_WIDTHS = (64, 128, 192, 256, 320, 384, 512, 576)      # latent widths of the tensor-core generation kernel
 
 
 def pick_latent_nsplit(batch, heads, keys, sm_count=148):
@@ -412,6 +412,9 @@ def attention_plain_capped(q, k, v, heads, k_dim, v_dim, window=0, keep=0, kept_
     return out
 
 
+PROMPT_HEADS = ((64, 64), (128, 64), (128, 128), (192, 64), (192, 128))       # key / value head sizes of attention_prefill_gated
+
+
 def _prompt_views(q, k, v, k_dim, v_dim, gate, out):
     require_cuda(q, k, v, out)
     B, S, H, G = q.shape[0], q.shape[1], q.shape[2] // k_dim, k.shape[2] // k_dim
@@ -425,7 +428,7 @@ def _prompt_views(q, k, v, k_dim, v_dim, gate, out):
 
 
 def attention_prefill_gated(q, k, v, k_dim, v_dim, sinks=None, first=None, gate=None, scale=None, out=None):
-    """attention_prefill_chunk without chunks, with value heads of v_dim (64 or k_dim), the output times sigmoid(gate)."""
+    """attention_prefill_chunk without chunks, with heads of k_dim / v_dim (PROMPT_HEADS), the output times sigmoid(gate)."""
     B, S, H, G, out, strides = _prompt_views(q, k, v, k_dim, v_dim, gate, out)
     require_cuda(first)
     _check_sinks(sinks, H)

@@ -11,7 +11,7 @@
 // swizzle, rows beyond the sequence read as zeros).  V is used as it lies in memory: for the
 // second product the contraction index (keys) runs down the rows of the tile, which the shared-
 // memory descriptor expresses as an N-major B operand, so nothing is transposed.
-// A CTA serves two row tiles (256 query rows).  Warp roles (320 threads): warp 0 issues
+// A CTA serves two row tiles (256 query rows; with query heads of 192 one).  Warp roles (320 threads): warp 0 issues
 // TMA, warp 1 issues the MMAs, warps 2-5 and 6-9 are the softmax of row tile 0 and 1: thread r
 // owns query row r, reads its score row from TMEM (tcgen05.ld), keeps the running maximum / sum
 // (fp32, log2 domain) and writes the probabilities as the 16-bit, swizzled A operand of the second
@@ -51,12 +51,13 @@ namespace eb {
 namespace {
 
 // (kRows of tc_ops.cuh: query rows per row tile)
-constexpr int kTiles = 2;                  // row tiles per CTA, each with its own four softmax warps
 constexpr int kKeys = 128;                 // keys per tile
-constexpr int kTcThreads = 64 + kTiles * 128;
+constexpr int kMaxTiles = 2;
 
-// Shared-memory plan per head_dim.  With head_dim 128 everything but a second V stage fits.
+// Shared-memory plan per head size.  With head_dim 128 everything but a second V stage fits, with 192 one row tile does.
 template <int D, int DV> struct TcSmem {
+  static constexpr int kTiles = D > 128 ? 1 : kMaxTiles;       // row tiles per CTA, each with its own four softmax warps
+  static constexpr int kThreads = 64 + kTiles * 128;
   static constexpr uint32_t kQBytes = (D / 64) * kRows * 128, kKBytes = (D / 64) * kKeys * 128, kVBytes = (DV / 64) * kKeys * 128,
                             kPBytes = 2 * kRows * 128;
   static constexpr int kVStages = DV > 64 ? 1 : 2;
@@ -109,13 +110,13 @@ __device__ __forceinline__ void tanh_series(float &p0, float &p1, float w0, floa
 __device__ __forceinline__ float tanh_exp(float z) { return 1.f - __fdividef(2.f, 1.f + ex2(z * (2.f * kLog2eTc))); }
 
 template <typename T, int D, int DV, int FORM>
-__global__ void __launch_bounds__(kTcThreads, 1)
+__global__ void __launch_bounds__(TcSmem<D, DV>::kThreads, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                             const __grid_constant__ CUtensorMap tm_v, const TcParams p) {
   constexpr bool BIAS = FORM == kFormBias, CAPPED = FORM == kFormCapped;
   constexpr int kSub = D / 64, kSubV = DV / 64;                  // 64-column sub-tiles of Q / K and V
   using Smem = TcSmem<D, DV>;
-  constexpr int kVStages = Smem::kVStages;
+  constexpr int kVStages = Smem::kVStages, kTiles = Smem::kTiles;
   constexpr uint32_t kQBytes = Smem::kQBytes, kKBytes = Smem::kKBytes, kVBytes = Smem::kVBytes, kPBytes = Smem::kPBytes;
   constexpr uint32_t kTmemCols = 512, kPvCol = 2 * kKeys;
   constexpr int kBf16 = std::is_same<T, __nv_bfloat16>::value ? 1 : 0;
@@ -167,7 +168,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __gr
   if (CAPPED && p.keep > 0 && p.window > 0 && nmax > 0) {
     const int kept = min((min(first + p.keep, p.Sk) - 1) / kKeys + 1, jmin) - kept_tile;
     jmin -= max(kept, 0);
-    ks[0] = ks[1] = jmin;
+#pragma unroll
+    for (int t = 0; t < kTiles; ++t) ks[t] = jmin;
   }
   auto tile_of = [&](int j) { return CAPPED && j < jwin ? kept_tile + j - jmin : j; };
 
@@ -594,6 +596,8 @@ __global__ void distance_bias_kernel(const float *r1, const float *r2, int len, 
 template <typename T, int D, int DV, int FORM>
 int launch_tc(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const TcParams &p, cudaStream_t st) {
   constexpr size_t smem = TcSmem<D, DV>::kTotal;
+  constexpr int kTiles = TcSmem<D, DV>::kTiles;
+  static_assert(smem <= 227 * 1024, "shared memory");
   auto kern = attention_prefill_tc_kernel<T, D, DV, FORM>;
   static bool configured[64] = {};
   int dev = 0;
@@ -606,7 +610,7 @@ int launch_tc(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &m
     configured[dev] = true;
   }
   dim3 grid((p.Sq + kTiles * kRows - 1) / (kTiles * kRows), p.H, p.B);
-  launch_pdl(kern, grid, dim3(kTcThreads), smem, st, mq, mk, mv, p);
+  launch_pdl(kern, grid, dim3(TcSmem<D, DV>::kThreads), smem, st, mq, mk, mv, p);
   return check_launch("attention_prefill");
 }
 
@@ -637,8 +641,9 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   if (batch == 0 || heads == 0 || q_len == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "attention_prefill: fp16 or bf16 only (dtype %d)", dtype);
   if (v_dim == 0) v_dim = head_dim;
-  EB_REQUIRE(head_dim == 64 || head_dim == 128, "attention_prefill: head_dim %d not supported (64 or 128)", head_dim);
-  EB_REQUIRE(v_dim == head_dim || (v_dim == 64 && !bias), "attention_prefill: value heads of %d not supported (64 or as the keys)", v_dim);
+  const bool large = head_dim == 192 && v_dim != 192 && !capped && !bias;             // (plain form, with smaller value heads)
+  EB_REQUIRE(head_dim == 64 || head_dim == 128 || large, "attention_prefill: head_dim %d not supported (64 or 128)", head_dim);
+  EB_REQUIRE(v_dim == head_dim || (v_dim == 64 && !bias) || (large && v_dim == 128), "attention_prefill: value heads of %d not supported", v_dim);
   EB_REQUIRE(batch > 0 && heads > 0 && q_len > 0 && kv_len > 0, "attention_prefill: negative or zero size");
   EB_REQUIRE(heads <= 65535 && batch <= 65535, "attention_prefill: batch and heads are limited to 65535");
   EB_REQUIRE(q && k && v && out, "attention_prefill: null pointer");
@@ -673,6 +678,10 @@ static int prefill_tc_impl(const void *q, const void *k, const void *v, void *ou
   }
 #define EB_TC(T, D, DV) (capped ? launch_tc<T, D, DV, kFormCapped>(mq, mk, mv, p, st) : launch_tc<T, D, DV, kFormPlain>(mq, mk, mv, p, st))
 #define EB_TC_B(T, D) (bias ? launch_tc<T, D, D, kFormBias>(mq, mk, mv, p, st) : EB_TC(T, D, D))
+  if (large) {
+    if (v_dim == 64) return dtype == EB_F16 ? launch_tc<__half, 192, 64, kFormPlain>(mq, mk, mv, p, st) : launch_tc<__nv_bfloat16, 192, 64, kFormPlain>(mq, mk, mv, p, st);
+    return dtype == EB_F16 ? launch_tc<__half, 192, 128, kFormPlain>(mq, mk, mv, p, st) : launch_tc<__nv_bfloat16, 192, 128, kFormPlain>(mq, mk, mv, p, st);
+  }
   if (v_dim != head_dim) return dtype == EB_F16 ? EB_TC(__half, 128, 64) : EB_TC(__nv_bfloat16, 128, 64);
   if (dtype == EB_F16) return head_dim == 64 ? EB_TC_B(__half, 64) : EB_TC_B(__half, 128);
   return head_dim == 64 ? EB_TC_B(__nv_bfloat16, 64) : EB_TC_B(__nv_bfloat16, 128);
@@ -716,8 +725,8 @@ extern "C" int eb_attention_prefill_biased_tc(const void *q, const void *k, cons
                                        int heads, int kv_group, int q_len, int kv_len, int head_dim, int window, const float *bias_table,
                                        int bias_len, int sink, float scale, int dtype, void *stream) {
   EB_REQUIRE(kv_group > 0 && heads % kv_group == 0, "attention_prefill: %d heads do not share keys in groups of %d", heads, kv_group);
-  EB_REQUIRE(bias_table && bias_len >= kv_len + kTiles * kRows, "attention_prefill: the bias table needs %d distances, has %d",
-             kv_len + kTiles * kRows, bias_len);
+  EB_REQUIRE(bias_table && bias_len >= kv_len + kMaxTiles * kRows, "attention_prefill: the bias table needs %d distances, has %d",
+             kv_len + kMaxTiles * kRows, bias_len);
   return prefill_tc_impl(q, k, v, out, mask, q_batch_stride, q_row_stride, k_batch_stride, k_row_stride, v_batch_stride, v_row_stride,
                          o_batch_stride, o_row_stride, mask_batch_stride, batch, heads, q_len, kv_len, head_dim, 1, window, scale, dtype,
                          stream, kv_group, bias_table, bias_len, sink);

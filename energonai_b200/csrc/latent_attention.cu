@@ -125,7 +125,7 @@ __device__ __forceinline__ float4 cluster_ld4(uint32_t addr) {
   return v;
 }
 
-// R: latent width (multiple of 64, at most 512); MT: 16-head tiles per CTA (1 or 2).
+// R: latent width (multiple of 64, at most 576); MT: 16-head tiles per CTA (1 or 2).
 //
 // The visible positions lie in a cyclic range of cache rows; the CTA walks its share of the 64-row
 // tiles of that range in ROW order (a softmax does not care about order), so a tile is one
@@ -582,7 +582,8 @@ template <typename T> int launch_latent_r(const CUtensorMap &map, const LatentPa
     case 256: return launch_latent_mt<T, 256>(map, p, B, st);
     case 320: return launch_latent_mt<T, 320>(map, p, B, st);
     case 384: return launch_latent_mt<T, 384>(map, p, B, st);
-    default: return launch_latent_mt<T, 512>(map, p, B, st);
+    case 512: return launch_latent_mt<T, 512>(map, p, B, st);
+    default: return launch_latent_mt<T, 576>(map, p, B, st);
   }
 }
 
@@ -721,8 +722,8 @@ extern "C" int eb_latent_decode_sink(const void *q, long long q_batch_stride, co
                                 int nsplit, void *scratch, size_t scratch_bytes, void *stream) {
   if (batch == 0 || heads == 0) return EB_OK;
   EB_REQUIRE(dtype == EB_F16 || dtype == EB_BF16, "latent_decode: fp16 or bf16 only (dtype %d)", dtype);
-  EB_REQUIRE(rank == 64 || rank == 128 || rank == 192 || rank == 256 || rank == 320 || rank == 384 || rank == 512,
-             "latent_decode: latent width %d not supported (64, 128, 192, 256, 320, 384 or 512)", rank);
+  EB_REQUIRE(rank == 64 || rank == 128 || rank == 192 || rank == 256 || rank == 320 || rank == 384 || rank == 512 || rank == 576,
+             "latent_decode: latent width %d not supported (64, 128, 192, 256, 320, 384, 512 or 576)", rank);
   EB_REQUIRE(batch > 0 && batch <= 65535 && heads > 0 && ring_rows > 0 && window >= 0 && nsplit >= 1 && nsplit <= 1024, "latent_decode: bad sizes");
   EB_REQUIRE(q && cache && out && pos_device, "latent_decode: null pointer");
   EB_REQUIRE(aligned16(q) && aligned16(cache) && aligned16(out), "latent_decode: pointers must be 16-byte aligned");

@@ -16,7 +16,7 @@ columns change no product.
 import torch
 from torch import nn
 
-from ..attention import (LATENT_WIDTHS, attention_plain, attention_prefill_gated, attention_prefill_window, latent_decode, latent_inputs, rotate_heads,
+from ..attention import (LATENT_WIDTHS, PROMPT_HEADS, attention_plain, attention_prefill_gated, attention_prefill_window, latent_decode, latent_inputs, rotate_heads,
                          sigmoid_gate, yarn_rotation)
 from ..gemm import project
 from ..moe import per_head
@@ -103,12 +103,9 @@ class RotaryLatentAttention(nn.Module):
         self.dim, self.rot_dim, self.vdim, self.q_rank, self.kv_rank = cfg.dim, cfg.rot_dim, cfg.vdim, cfg.q_rank, cfg.kv_rank
         self.rot_at, self.rot_col = round_up(cfg.dim, 8), round_up(cfg.kv_rank, 8)         # where the rotated part begins in a head, in a row
         key, row = self.rot_at + cfg.rot_dim, self.rot_col + cfg.rot_dim
-        self.tensor_core_prompt = dtype != torch.float32 and max(key, cfg.vdim) <= 128 and cfg.scale > 0
-        if self.tensor_core_prompt:
-            self.dv = 64 if cfg.vdim <= 64 else 128
-            self.dk = max(self.dv, 64 if key <= 64 else 128)
-        else:
-            self.dk, self.dv = round_up(key, 8), round_up(cfg.vdim, 8)
+        fits = [h for h in PROMPT_HEADS if h[0] >= key and h[1] >= cfg.vdim]
+        self.tensor_core_prompt = dtype != torch.float32 and bool(fits) and cfg.scale > 0
+        self.dk, self.dv = min(fits) if self.tensor_core_prompt else (round_up(key, 8), round_up(cfg.vdim, 8))
         self.tensor_core_step = dtype != torch.float32 and row <= LATENT_WIDTHS[-1]
         self.rank = min(w for w in LATENT_WIDTHS if w >= row) if self.tensor_core_step else round_up(row, 8)
         self.q_cols, self.q_rows, self.columns = round_up(cfg.q_rank, 8), cfg.heads * self.dk, cfg.heads * self.dv

@@ -750,8 +750,8 @@ EB_API int eb_attention_prefill_biased_tc(const void *q, const void *k, const vo
                             int heads, int kv_group, int q_len, int kv_len, int head_dim, int window, const float *bias_table,
                             int bias_len, int sink, float scale, int dtype, void *stream);
 
-/* eb_attention_prefill_chunk_tc without chunks, with value heads of v_dim (64 or k_dim) and the output times
- * sigmoid(gate), gate (or NULL) laid out like the output. */
+/* eb_attention_prefill_chunk_tc without chunks, with value heads of v_dim and the output times sigmoid(gate), gate (or
+ * NULL) laid out like the output.  k_dim / v_dim: 64 / 64, 128 / 64 or 128, 192 / 64 or 128. */
 EB_API int eb_attention_prefill_gated_tc(const void *q, const void *k, const void *v, void *out, const void *gate, long long q_batch_stride,
                             long long q_row_stride, long long k_batch_stride, long long k_row_stride, long long v_batch_stride,
                             long long v_row_stride, long long o_batch_stride, long long o_row_stride, long long g_batch_stride,
@@ -831,7 +831,7 @@ EB_API int eb_attention_plain_capped(const void *q, const void *k, const void *v
  * queries in latent space, the cached latent row of a position is key and value of every head,
  *   out[b][h] = sum_j softmax_j(scale * q[b][h] . c[b][j]) c[b][j]
  * over the positions max(first[b], pos - window + 1) .. pos (window 0: all), position j in cache row
- * j mod ring_rows.  rank 64, 128, 192, 256, 320, 384 or 512.  Every cache row must hold finite numbers, also
+ * j mod ring_rows.  rank 64, 128, 192, 256, 320, 384, 512 or 576.  Every cache row must hold finite numbers, also
  * those no position has been written to yet (they are multiplied by a weight of exactly 0).
  * nsplit > 1 splits the positions over that many CTAs per (sequence, head tile): 2, 4 or 8 are
  * clusters that merge their parts on chip, any other number merges in a second launch through

@@ -80,10 +80,12 @@ def test_padded_sizes():
     m = registry.build_model("Tupidra", config_dict=config(), dtype=torch.float32).layers
     assert (m[1].mixer.dk, m[1].mixer.dv, m[1].mixer.tensor_core) == (16, 24, False)
     assert (m[2].mixer.dk, m[2].mixer.dv, m[2].mixer.rank) == (24, 16, 32) and (m[4].mixer.dk, m[4].mixer.dv) == (32, 24)
-    wide = P.make_config([P.latent_layer(2, 64, 40, 60, 8, 250, 0.1, 10.0), P.latent_layer(2, 120, 10, 64, 8, 500, 0.1, 10.0), P.latent_layer(2, 30, 10, 100, 8, 20, 0.1, 10.0)], 64, 50)
+    wide = P.make_config([P.latent_layer(2, 64, 40, 60, 8, 250, 0.1, 10.0), P.latent_layer(2, 120, 10, 64, 8, 500, 0.1, 10.0), P.latent_layer(2, 30, 10, 100, 8, 20, 0.1, 10.0),
+                          P.latent_layer(2, 190, 10, 64, 8, 600, 0.1, 10.0)], 64, 50)
     m = registry.build_model("Tupidra", config_dict=wide, dtype=torch.bfloat16).layers
     at = lambda i: (m[i].mixer.dk, m[i].mixer.dv, m[i].mixer.rank, m[i].mixer.tensor_core_prompt, m[i].mixer.tensor_core_step)
-    assert at(0) == (128, 64, 320, True, True) and at(1) == (136, 64, 520, False, False) and at(2) == (128, 128, 64, True, True)
+    assert at(0) == (128, 64, 320, True, True) and at(1) == (192, 64, 576, True, True) and at(2) == (128, 128, 64, True, True)
+    assert at(3) == (208, 64, 616, False, False)
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -286,10 +288,10 @@ def test_kernels_validate_before_any_cuda_call():
     assert L.eb_rotate_heads(a, 16, 1, 16, 8, 5, a, 1.0, 1, 1, None, None, B16, None) == -1 and L.eb_rotate_heads(a, 16, 1, 16, 7, 2, a, 1.0, 1, 1, None, None, B16, None) == -1
     pre = lambda k=64, v=64, group=1, window=0, keep=0, cap=1.0, scale=0.1, gate=None: L.eb_attention_prefill_capped_tc(
         a, a, a, a, gate, *[64] * 10, 1, 2, group, 8, k, v, window, keep, None, a, cap, 1, scale, B16, None)
-    assert pre(group=3) == -1 and pre(k=96) == -1 and pre(v=128) == -1 and pre(keep=-1) == -1 and pre(cap=-1.0) == -1 and pre(scale=0.0) == -1 and pre(window=-1) == -1
+    assert pre(group=3) == -1 and pre(k=96) == -1 and pre(k=192) == -1 and pre(v=128) == -1 and pre(keep=-1) == -1 and pre(cap=-1.0) == -1 and pre(scale=0.0) == -1 and pre(window=-1) == -1
     assert pre(gate=a + 2) == -1 and "gate" in err()
     gated = lambda k=64, v=64, group=1: L.eb_attention_prefill_gated_tc(a, a, a, a, None, *[64] * 10, 1, 2, group, 8, k, v, None, None, 0.1, B16, None)
-    assert gated(group=3) == -1 and gated(k=32) == -1 and gated(v=32) == -1
+    assert gated(group=3) == -1 and gated(k=32) == -1 and gated(v=32) == -1 and gated(k=192, v=192) == -1 and gated(k=256) == -1
     dec = lambda kv=2, keep=0, cap=0.0, nsplit=1, window=4: L.eb_attention_group_decode_capped(a, a, a, a, None, 256, 640, 128, 640, 128, 256, 0, 1, 4, kv, 64, keep, 5, window, a, None,
                                                                                               None, cap, 1, 1.0, B16, nsplit, None, 0, None)
     assert dec(kv=3) == -1 and dec(keep=-1) == -1 and dec(cap=-1.0) == -1 and dec(nsplit=2) == -1 and dec(window=-1) == -1

@@ -270,7 +270,7 @@ def test_latent_inputs(dtype, q_cols, q_count, rank, kv, rot):
 
 
 @pytest.mark.parametrize("dtype", [BF16, F16])
-@pytest.mark.parametrize("n,H,dk,dv", [(3, 2, 64, 64), (200, 3, 128, 64), (300, 2, 128, 128), (520, 1, 128, 64)])
+@pytest.mark.parametrize("n,H,dk,dv", [(3, 2, 64, 64), (200, 3, 128, 64), (300, 2, 128, 128), (520, 1, 128, 64), (1, 1, 192, 128), (390, 3, 192, 128), (257, 2, 192, 64)])
 def test_gated_prompt_attention_with_sinks(dtype, n, H, dk, dv):
     from energonai_b200.attention import attention_prefill_gated
     B, first = 2, [0, min(n - 1, 140)]
@@ -285,7 +285,7 @@ def test_gated_prompt_attention_with_sinks(dtype, n, H, dk, dv):
         assert rel(got[b, first[b]:], o * torch.sigmoid(g[b, first[b]:].double())) < tol(dtype)
 
 
-@pytest.mark.parametrize("R,H,n", [(64, 3, 20), (192, 16, 130), (192, 20, 600), (320, 5, 700), (320, 33, 64), (512, 17, 300)])
+@pytest.mark.parametrize("R,H,n", [(64, 3, 20), (192, 16, 130), (192, 20, 600), (320, 5, 700), (320, 33, 64), (512, 17, 300), (576, 3, 700), (576, 18, 130)])
 def test_latent_decode_with_sinks(R, H, n):
     """The sink joins once, whatever the splits."""
     from energonai_b200.attention import attention_plain, latent_decode
