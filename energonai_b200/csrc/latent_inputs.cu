@@ -104,7 +104,7 @@ struct RotateParams {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(128) rotate_heads_kernel(const RotateParams p) {
+__global__ void __launch_bounds__(512) rotate_heads_kernel(const RotateParams p) {
   using P = Pair<T>;
   using R = typename P::R;
   extern __shared__ float2 cs[];                   // [pairs]
@@ -180,8 +180,9 @@ extern "C" int eb_rotate_heads(void *x, long long ldx, int heads, int head_cols,
   p.freq = freq; p.factor = factor; p.pos_dev = pos_device; p.first = first;
   cudaStream_t st = as_stream(stream);
   const size_t smem = (size_t)pairs * sizeof(float2);
-  if (dtype == EB_F32) launch_pdl(rotate_heads_kernel<float>, dim3(n1), dim3(128), smem, st, p);
-  else if (dtype == EB_F16) launch_pdl(rotate_heads_kernel<__half>, dim3(n1), dim3(128), smem, st, p);
-  else launch_pdl(rotate_heads_kernel<__nv_bfloat16>, dim3(n1), dim3(128), smem, st, p);
+  const dim3 t(n1 < 4 * sm_count() && heads * pairs > 256 ? 512 : 128);                    // few rows: fewer pairs one after the other
+  if (dtype == EB_F32) launch_pdl(rotate_heads_kernel<float>, dim3(n1), t, smem, st, p);
+  else if (dtype == EB_F16) launch_pdl(rotate_heads_kernel<__half>, dim3(n1), t, smem, st, p);
+  else launch_pdl(rotate_heads_kernel<__nv_bfloat16>, dim3(n1), t, smem, st, p);
   return check_launch("rotate_heads");
 }

@@ -580,8 +580,8 @@ TUPIDRA_SIZES = {
     # with a dense feed-forward beside its mixer
     "2048": dict(width=2048, inner=4096, state=16, dt_rank=128, heads=16, kv_heads=4, dim=128, window=1024, keep=64, lheads=32, ldim=64, rot=32, lvdim=64,
                  q_rank=768, kv_rank=256, ff=5632, layers=8, vocab=32768),
-    "4096": dict(width=4096, inner=8192, state=16, dt_rank=256, heads=32, kv_heads=8, dim=128, window=4096, keep=64, lheads=32, ldim=96, rot=32, lvdim=128,
-                 q_rank=1536, kv_rank=480, ff=11264, layers=8, vocab=32768),
+    "4096": dict(width=4096, inner=8192, state=16, dt_rank=256, heads=32, kv_heads=8, dim=128, window=4096, keep=64, lheads=32, ldim=128, rot=64, lvdim=128,
+                 q_rank=1536, kv_rank=512, ff=11264, layers=8, vocab=32768),
 }
 
 
@@ -616,7 +616,7 @@ def tupidra_as_opt(z):
 
 def tupidra_kernel_table(z, B, S, T):
     """As kernel_table, for the selective-scan / capped-attention / rotary-latent decoder."""
-    from ..attention import (LATENT_WIDTHS, attention_decode, attention_group_decode, attention_group_decode_capped, attention_prefill, attention_prefill_biased,
+    from ..attention import (LATENT_WIDTHS, PROMPT_HEADS, attention_decode, attention_group_decode, attention_group_decode_capped, attention_prefill, attention_prefill_biased,
                              attention_prefill_capped, attention_prefill_gated, attention_rotary, attention_values, distance_bias, distance_slopes, latent_decode,
                              latent_inputs, rotate_heads, sigmoid_gate)
     from ..decay import selective_scan, selective_step, short_conv, short_conv_step, ssm_prompt, ssm_step
@@ -627,7 +627,7 @@ def tupidra_kernel_table(z, B, S, T):
     bf, f32, dev = torch.bfloat16, torch.float32, "cuda"
     W, H, G, d, ff, C, N, dr = (z[k] for k in ("width", "heads", "kv_heads", "dim", "ff", "inner", "state", "dt_rank"))
     LH, ld, rot, lv, qr, kr = (z[k] for k in ("lheads", "ldim", "rot", "lvdim", "q_rank", "kv_rank"))
-    dk, R = 64 if ld + rot <= 64 else 128, min(w for w in LATENT_WIDTHS if w >= kr + rot)
+    dk, R = min(h for h in PROMPT_HEADS if h[0] >= ld + rot and h[1] >= lv)[0], min(w for w in LATENT_WIDTHS if w >= kr + rot)
     win, keep = z["window"], z["keep"]
     rnd = lambda *s, dtype=bf: (torch.randn(*s, device=dev, dtype=torch.float32) * 0.05).to(dtype)
     rows = []
